@@ -44,7 +44,12 @@ typedef enum {
 } mpk_dtype;
 
 /* execution modes, python/mirage/mpk/persistent_kernel.py:169 */
-typedef enum { MPK_MODE_OFFLINE = 0, MPK_MODE_ONLINE_NOTOKEN = 1 } mpk_mode;
+typedef enum {
+  MPK_MODE_OFFLINE = 0,        /* all requests known at launch: prompts first, then greedy / sampled decoding until EOS or full */
+  MPK_MODE_ONLINE_NOTOKEN = 1, /* the caller describes every batch itself                                                     */
+  MPK_MODE_ONLINE = 2          /* the device schedules as offline, but token-table rows are requests the host posts, extends,
+                                  holds and closes between launches through request_ctl (see mpk_config)                      */
+} mpk_mode;
 
 /* io_category of PersistentKernel.new_tensor, persistent_kernel.py:546-568 */
 typedef enum { MPK_IO_CUDA = 0, MPK_IO_SYMMETRIC = 1 } mpk_io_category;
@@ -55,7 +60,7 @@ typedef enum {
   MPK_OP_EMBED = 1,             /* embed_layer              :586  in: ids, table        out: y            params: [input_source]          */
   MPK_OP_RMSNORM = 2,           /* rmsnorm_layer            :609  in: x, gamma          out: y                                            */
   MPK_OP_RMSNORM_LINEAR = 3,    /* rmsnorm_linear_layer     :627  in: x, gamma, W       out: y                                            */
-  MPK_OP_LINEAR = 4,            /* linear_layer             :1731 in: x, W              out: y                                            */
+  MPK_OP_LINEAR = 4,            /* linear_layer             :1731 in: x, W              out: y            params: optional [activation: 0 none, 1 squared relu (hybrid graphs)] */
   MPK_OP_LINEAR_RESIDUAL = 5,   /* linear_with_residual_layer :1762 in: x, W, residual  out: y            params: [enable_residual]       */
   MPK_OP_SPLITK_LINEAR = 6,     /* splitk_linear_layer      :1706 in: x, W              out: y (y += x W^T)                               */
   MPK_OP_ATTENTION = 7,         /* attention_layer          :648  in: qkv,k,v,qn,kn,cos,sin out: o       params: [hq, hkv, qk_norm, rope] */
@@ -94,7 +99,29 @@ typedef enum {
                                    (softmax over the experts, top-k by value with ties to the lower index, weights renormalised
                                    over the selected experts; the logits are left as they are)  params: optional [first, end]
                                    of the experts this rank runs */
+  ,
+  /* Hybrid graphs (no reference counterpart): float32 residual stream, attention with free head sizes, recurrent layers.
+   * A graph with one of these may hold, besides them, embed, linear, argmax and sampling layers; all floats in params
+   * are bit patterns.  Linears write float32 where the output tensor is float32; float32 linear inputs select 32-bit
+   * arithmetic for the whole graph. */
+  MPK_OP_RESIDUAL_NORM = 32,    /* x += norm(y) | y; out = norm(x)   in: x (f32, in place), y, weight of y's norm, weight of the output norm
+                                   out: out   (all but x optional)   params: [eps, weights stored around zero] */
+  MPK_OP_QKV_APPEND = 33,       /* rotate q and k, unit RMS norm, append k / v rows   in: projections, cos, sin  out: q, k_cache, v_cache
+                                   tensors: proj, q, k_cache, v_cache, cos, sin
+                                   params: [hq, hkv, dim, vdim, q_col, k_col, v_col, rotated dims, unit norm, eps] */
+  MPK_OP_EXT_ATTENTION = 34,    /* tensors: q, k_cache, v_cache, out
+                                   params: [hq, hkv, vdim, out_col, scale, soft cap (0: none), sink, out_scale] */
+  MPK_OP_SHORT_CONV = 35,       /* causal per-channel convolution   tensors: in, in_bias, taps, bias, state, out (biases optional)
+                                   params: [in_col, activation: 0 none, 1 silu] */
+  MPK_OP_RGLRU = 36,            /* gated diagonal recurrence        tensors: u, proj, y_bias, ra, ra_bias, ri, ri_bias, lambda, state, out
+                                   params: [y_col, out_col, out_scale, decay constant] */
+  MPK_OP_MLSTM = 37             /* matrix-memory recurrence         tensors: proj, i_bias, f_bias, norm, state, n_m state, scratch, out
+                                   params: [heads, dim, vdim, q_col, k_col, v_col, gate_col, i_col, f_col, gate cap, eps, q scale, chunks] */
 } mpk_op;
+
+/* Value columns a task of an MPK_OP_MLSTM layer walks at a time; the layer's `chunks` parameter (and the second state
+ * tensor [slots, heads, chunks, dim + 1]) may be at most ceil(vdim / this).  */
+#define MPK_MLSTM_COLUMNS(dim) ((dim) <= 256 ? 64 : (dim) <= 512 ? 32 : 16)
 
 /* Constructor arguments of PersistentKernel (persistent_kernel.py:349-369) plus the
  * meta tensors it hands to init_func (:2494-2506).  All pointers are DEVICE
@@ -131,6 +158,13 @@ typedef struct {
                                         [2] task end (globaltimer ns), [3] worker << 40 | event << 8 | task type, [4..7] phase stamps
                                         whose meaning depends on the task type; mirage_b200/profiler.py converts to a Chrome trace */
   uint64_t profiler_entries;
+  int32_t *state_slots;              /* [max_num_batched_requests] recurrent-state slot of each batch slot; optional with a batching
+                                        task (the library allocates it), the caller's in online_notoken (NULL: batch slot = state slot) */
+  int32_t *request_ctl;              /* online mode: [2][total_num_requests].  Row 0, written by the host between launches: 0 free,
+                                        1 run (prompt, then decode until EOS or the table is full), 2 hold (run the prompt_lengths[r]
+                                        tokens supplied so far, keep pages and state), 3 close (run what is supplied, then retire; the
+                                        device sets 0 when it retires the request, at the start of a launch).  Row 1 is the device's. */
+  int32_t *request_ids;              /* [max_num_batched_requests] token-table row of each batch slot, -1: empty; optional */
 } mpk_config;
 
 /* What the device reported after the most recent launch. */

@@ -29,8 +29,11 @@ OP_MLA_KV_GATHER, OP_MLA_DECODE, OP_MLA_REDUCE = 25, 26, 27
 OP_SAMPLING_PARTIAL, OP_SAMPLING_REDUCE = 28, 29
 OP_ARGMAX_EXCHANGE = 30
 OP_MOE_TOPK_SOFTMAX = 31
+OP_RESIDUAL_NORM, OP_QKV_APPEND, OP_EXT_ATTENTION, OP_SHORT_CONV, OP_RGLRU, OP_MLSTM = 32, 33, 34, 35, 36, 37
 IO_CUDA, IO_SYMMETRIC = 0, 1
-MODE_OFFLINE, MODE_ONLINE_NOTOKEN = 0, 1
+MODE_OFFLINE, MODE_ONLINE_NOTOKEN, MODE_ONLINE = 0, 1, 2
+# control words of online mode (request_ctl)
+REQ_FREE, REQ_RUN, REQ_HOLD, REQ_CLOSE = 0, 1, 2, 3
 
 
 class MpkConfig(C.Structure):
@@ -45,6 +48,7 @@ class MpkConfig(C.Structure):
         ("qo_indptr", C.c_void_p), ("paged_kv_indptr", C.c_void_p), ("paged_kv_indices", C.c_void_p),
         ("paged_kv_last_page_len", C.c_void_p), ("paged_kv_indices_snapshot", C.c_void_p),
         ("profiler_buffer", C.c_void_p), ("profiler_entries", C.c_uint64),
+        ("state_slots", C.c_void_p), ("request_ctl", C.c_void_p), ("request_ids", C.c_void_p),
     ]
 
 

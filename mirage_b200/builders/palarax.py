@@ -1,0 +1,287 @@
+"""Palarax decoder on a `PersistentKernel`: configuration, weight preparation, recurrent state and layer sequence.
+
+A float32 residual stream with a norm before and after every sublayer.  Two kinds of mixers:
+
+  mlstm     [q | k | v | gate | i | f] in one linear -> matrix-memory recurrence with its head norm and gate -> output linear
+  parallel  [q | k | y | x] in one linear -> { rotation, unit norms, cache rows -> attention with soft cap and sink } beside
+            { short convolution -> gated diagonal recurrence }; both write their columns of one buffer, already scaled,
+            and one linear over [left.o | right.o] adds them up
+
+and a squared-relu feed-forward.  Linear weights of the bf16 graph are padded to a multiple of 64 input columns (the
+tensor path's k granularity), the activation buffers in front of them likewise: the padding columns stay zero.
+"""
+from __future__ import annotations
+
+import json
+import os
+from dataclasses import dataclass
+from typing import Any, Dict, List, Optional, Tuple
+
+import torch
+
+from ..mpk import register_model_builder
+from ..persistent_kernel import DTensor, PersistentKernel, bfloat16, float32, int64
+
+
+def _round_up(n: int, m: int) -> int:
+    return -(-n // m) * m
+
+
+@dataclass(frozen=True)
+class MlstmSpec:
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+
+@dataclass(frozen=True)
+class AttentionSpec:
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    rot_base: float
+    rot_dims: int
+    scale: float
+    softcap: float
+
+
+@dataclass(frozen=True)
+class RgLruSpec:
+    width: int
+    blocks: int
+    taps: int
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    left: AttentionSpec
+    right: RgLruSpec
+    left_scale: float
+    right_scale: float
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: Any                # MlstmSpec or ParallelSpec
+    ff: Optional[int]         # width of the feed-forward, None: the layer has none
+
+
+@dataclass(frozen=True)
+class PalaraxConfig:
+    vocab: int
+    width: int
+    eps: float
+    layers: Tuple[LayerSpec, ...]
+
+    DECAY = 8.0               # constant of the diagonal recurrence's log decay
+
+    @classmethod
+    def from_dict(cls, c: Dict[str, Any]) -> "PalaraxConfig":
+        layers = []
+        for n, entry in enumerate(c["layers"]):
+            m = entry["mixer"]
+            if entry["type"] == "mlstm":
+                mixer = MlstmSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"]))
+            elif entry["type"] == "parallel":
+                l, r = m["left"], m["right"]
+                left = AttentionSpec(int(l["heads"]), int(l["kv_heads"]), int(l["dim"]), int(l["vdim"]),
+                                     float(l["rot"]["base"]), int(l["rot"]["dims"]), float(l["scale"]), float(l["softcap"]))
+                right = RgLruSpec(int(r["width"]), int(r["blocks"]), int(r["conv"]))
+                if left.heads % left.kv_heads or left.rot_dims % 2 or left.rot_dims > left.dim or right.width % right.blocks:
+                    raise ValueError(f"layer {n}: sizes do not divide")
+                if left.vdim != left.dim:
+                    raise ValueError(f"layer {n}: keys serve as values, but dim {left.dim} != vdim {left.vdim}")
+                mixer = ParallelSpec(left, right, float(m["left_scale"]), float(m["right_scale"]))
+            else:
+                raise ValueError(f"layer {n}: unknown mixer {entry['type']!r}")
+            mlp = entry.get("mlp")
+            if mlp is not None and mlp["kind"] != "dense":
+                raise ValueError(f"layer {n}: unknown feed-forward {mlp['kind']!r}")
+            layers.append(LayerSpec(mixer, None if mlp is None else int(mlp["ff"])))
+        return cls(int(c["vocab"]), int(c["width"]), float(c["norm"]["eps"]), tuple(layers))
+
+    @classmethod
+    def from_checkpoint(cls, path: str) -> "PalaraxConfig":
+        with open(os.path.join(path, "config.json")) as f:
+            return cls.from_dict(json.load(f))
+
+
+def _rotary_tables(base: float, dims: int, positions: int, device) -> Tuple[torch.Tensor, torch.Tensor]:
+    """float32 cos / sin [positions, dims / 2] of position * base^(-2i / dims); the angles are formed in 64-bit."""
+    if dims == 0:
+        z = torch.zeros(1, 1, dtype=torch.float32, device=device)
+        return z, z.clone()
+    f = float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+    a = torch.arange(positions, dtype=torch.float64)[:, None] * f
+    return a.cos().float().to(device), a.sin().float().to(device)
+
+
+def allocate_state(c: PalaraxConfig, *, slots: int, max_num_pages: int, page_size: int, dtype: torch.dtype, device,
+                   num_workers: int) -> List[Dict[str, torch.Tensor]]:
+    """Per layer: what a sequence leaves behind.  Attention caches are paged [pages, page, kv heads, head size rounded up
+    to 8] in the activation type; recurrent state is float32 and indexed by state slot."""
+    z32 = lambda *s: torch.zeros(*s, dtype=torch.float32, device=device)
+    out = []
+    for layer in c.layers:
+        m = layer.mixer
+        if isinstance(m, MlstmSpec):
+            chunks = PersistentKernel.mlstm_chunks(num_workers, slots, m.heads, m.dim, m.vdim)
+            out.append({"memory": z32(slots, m.heads, m.dim, _round_up(m.vdim, 4)),
+                        "normaliser": z32(slots, m.heads, chunks, m.dim + 1)})
+        else:
+            shape = lambda d: (max_num_pages, page_size, m.left.kv_heads, _round_up(d, 8))
+            out.append({"k": torch.zeros(shape(m.left.dim), dtype=dtype, device=device),
+                        "v": torch.zeros(shape(m.left.vdim), dtype=dtype, device=device),
+                        "conv": z32(slots, max(m.right.taps - 1, 1), m.right.width),
+                        "diag": z32(slots, m.right.width)})
+    return out
+
+
+@dataclass
+class PalaraxModelConfig:
+    """What the builder needs beside the kernel: shapes, weights under their checkpoint names, state, activation type."""
+    config: PalaraxConfig
+    state_dict: Dict[str, torch.Tensor]
+    state: List[Dict[str, torch.Tensor]]
+    dtype: torch.dtype = torch.bfloat16
+    sampling_seed: Optional[int] = None    # None: greedy argmax; an int: Gumbel-max sampling
+
+    def check_valid(self):
+        assert self.state_dict is not None and len(self.state) == len(self.config.layers)
+        assert self.dtype in (torch.bfloat16, torch.float32)
+
+
+@register_model_builder("palarax")
+class PalaraxBuilder:
+    def __init__(self, mpk: PersistentKernel):
+        self.mpk = mpk
+        self.logits: Optional[DTensor] = None
+        self.hidden: Optional[DTensor] = None      # float32 residual stream
+        self._buffers: Dict[Tuple[str, int], DTensor] = {}
+        self._tables: Dict[Tuple[float, int], Tuple[DTensor, DTensor]] = {}
+
+    # -- helpers
+    def _buf(self, tag: str, width: int, dt) -> DTensor:
+        """One buffer per purpose and width, shared by all layers."""
+        key = (tag, width)
+        if key not in self._buffers:
+            self._buffers[key] = self.mpk.new_tensor(dims=(self.mpk.max_num_batched_tokens, width), dtype=dt,
+                                                     name=f"{tag}_{width}")
+        return self._buffers[key]
+
+    def _kpad(self, k: int) -> int:
+        return _round_up(k, 64) if self.act is bfloat16 else k
+
+    def _weight(self, name: str, parts: List[torch.Tensor], dim: int = 0) -> DTensor:
+        """The parts side by side along `dim`, input columns padded."""
+        w = torch.cat(parts, dim) if len(parts) > 1 else parts[0]
+        pad = self._kpad(w.shape[1]) - w.shape[1]
+        w = torch.nn.functional.pad(w, (0, pad)) if pad else w
+        return self.mpk.attach_input(w.contiguous(), name=name)
+
+    def _att(self, name: str) -> DTensor:
+        return self.mpk.attach_input(self.sd[name].contiguous(), name=name)
+
+    def _linear(self, x: DTensor, w: DTensor, y: DTensor, activation: str = None):
+        self.mpk.linear_layer(input=x, weight=w, output=y, grid_dim=(96, 1, 1), block_dim=(128, 1, 1), activation=activation)
+
+    def _rotary(self, base: float, dims: int) -> Tuple[DTensor, DTensor]:
+        key = (base, dims)
+        if key not in self._tables:
+            dev = self.sd["embed"].device
+            cos, sin = _rotary_tables(base, dims, self.mpk.max_seq_length, dev)
+            n = len(self._tables)
+            self._tables[key] = (self.mpk.attach_input(cos, name=f"cos_{n}"), self.mpk.attach_input(sin, name=f"sin_{n}"))
+        return self._tables[key]
+
+    # -- mixers: `h` is the normed input; return the mixer's float32 output
+    def _mlstm(self, p: str, m: MlstmSpec, st: Dict[str, torch.Tensor], h: DTensor) -> DTensor:
+        mpk, sd = self.mpk, self.sd
+        qk, v = m.heads * m.dim, m.heads * m.vdim
+        proj = self._buf("proj", 2 * qk + 2 * v + 2 * m.heads, float32)
+        self._linear(h, self._weight(p + "qkvgif", [sd[p + n] for n in ("q", "k", "v", "g", "i", "f")]), proj)
+        out = self._buf("mixed", self._kpad(v), self.act)
+        mpk.mlstm_layer(proj, self._att(p + "i.b"), self._att(p + "f.b"), self._att(p + "norm"),
+                        mpk.attach_input(st["memory"], name=p + "memory"),
+                        mpk.attach_input(st["normaliser"], name=p + "normaliser"), self._buf("readout", v, float32), out,
+                        heads=m.heads, dim=m.dim, vdim=m.vdim, q_col=0, k_col=qk, v_col=2 * qk, gate_col=2 * qk + v,
+                        i_col=2 * qk + 2 * v, f_col=2 * qk + 2 * v + m.heads, gate_cap=m.gate_cap, eps=self.eps,
+                        q_scale=m.dim ** -0.5)
+        y = self._buf("sublayer", self.width, float32)
+        self._linear(out, self._weight(p + "o.padded", [sd[p + "o"]]), y)
+        return y
+
+    def _parallel(self, p: str, m: ParallelSpec, st: Dict[str, torch.Tensor], h: DTensor) -> DTensor:
+        mpk, sd = self.mpk, self.sd
+        l, r, pl, pr = m.left, m.right, p + "left.", p + "right."
+        nq, nk = l.heads * l.dim, l.kv_heads * l.dim
+        k_col, y_col, x_col = nq, nq + nk, nq + nk + r.width
+        proj = self._buf("proj", x_col + r.width, float32)
+        self._linear(h, self._weight(p + "qkyx", [sd[pl + "q"], sd[pl + "k"], sd[pr + "y"], sd[pr + "x"]]), proj)
+        left_out = l.heads * l.vdim
+        mixed = self._buf("mixed", self._kpad(left_out + r.width), self.act)
+        # left branch
+        kc, vc = mpk.attach_input(st["k"], name=pl + "k_cache"), mpk.attach_input(st["v"], name=pl + "v_cache")
+        q = self._buf("q", l.heads * kc.dim(3), self.act)
+        cos, sin = self._rotary(l.rot_base, l.rot_dims)
+        mpk.qkv_append_layer(proj, q, kc, vc, cos, sin, heads=l.heads, kv_heads=l.kv_heads, dim=l.dim, vdim=l.vdim, q_col=0,
+                             k_col=k_col, v_col=k_col, rot_dims=l.rot_dims, unit_norm=True, eps=self.eps)
+        mpk.ext_attention_layer(q, kc, vc, mixed, heads=l.heads, kv_heads=l.kv_heads, vdim=l.vdim, scale=l.scale,
+                                softcap=l.softcap, sink=True, out_col=0, out_scale=m.left_scale)
+        # right branch
+        u = self._buf("conv_out", r.width, float32)
+        mpk.short_conv_layer(proj, self._att(pr + "conv"), mpk.attach_input(st["conv"], name=pr + "conv_state"), u,
+                             input_bias=self._att(pr + "x.b"), bias=self._att(pr + "conv.b"), in_col=x_col)
+        mpk.rglru_layer(u, proj, self._att(pr + "y.b"), self._att(pr + "ra"), self._att(pr + "ra.b"), self._att(pr + "ri"),
+                        self._att(pr + "ri.b"), self._att(pr + "lam"), mpk.attach_input(st["diag"], name=pr + "state"), mixed,
+                        y_col=y_col, out_col=left_out, out_scale=m.right_scale, decay=PalaraxConfig.DECAY)
+        y = self._buf("sublayer", self.width, float32)
+        self._linear(mixed, self._weight(p + "o", [sd[pl + "o"], sd[pr + "o"]], dim=1), y)
+        return y
+
+    def build_from_config(self, mc: PalaraxModelConfig):
+        mpk, c, sd = self.mpk, mc.config, mc.state_dict
+        self.sd, self.eps, self.width = sd, c.eps, c.width
+        self.act = float32 if mc.dtype == torch.float32 else bfloat16
+        mbt = mpk.max_num_batched_tokens
+        if tuple(sd["embed"].shape) != (c.vocab, c.width):
+            raise ValueError(f"embedding is {tuple(sd['embed'].shape)}, configuration says {(c.vocab, c.width)}")
+        table = self._weight("embed", [sd["embed"]])
+        x = self._buf("stream", c.width, float32)
+        h = self._buf("normed", self._kpad(c.width), self.act)
+        mpk.embed_layer(input=mpk.attach_input(mpk.meta_tensors["input_tokens"], name="input_token"), weight=table, output=x,
+                        grid_dim=(1, 1, 1), block_dim=(128, 1, 1), input_source=1)
+
+        def norm(y: Optional[str], post: Optional[str], nxt: str):
+            mpk.residual_norm_layer(x, y, self._att(post) if post else None, self._att(nxt), h, eps=c.eps, zero_centered=True)
+
+        # a sublayer's closing norm and the next one's opening norm are one task
+        y, post = None, None
+        for n, layer in enumerate(c.layers):
+            p = f"l{n}."
+            norm(y, post, p + "norm1")
+            mixer = self._mlstm if isinstance(layer.mixer, MlstmSpec) else self._parallel
+            y, post = mixer(p + "mix.", layer.mixer, mc.state[n], h), p + "norm1b"
+            if layer.ff is not None:
+                norm(y, post, p + "norm2")
+                mid = self._buf("ff", self._kpad(layer.ff), self.act)
+                # (a padded buffer is wider than the weight has rows: the linear fills its leading columns)
+                self._linear(h, self._weight(p + "mlp.up.padded", [sd[p + "mlp.up"]]), mid, activation="relu2")
+                y, post = self._buf("sublayer", c.width, float32), p + "norm2b"
+                self._linear(mid, self._weight(p + "mlp.down.padded", [sd[p + "mlp.down"]]), y)
+        norm(y, post, "final.norm")
+        self.hidden = x
+        self.logits = mpk.new_tensor(dims=(mbt, c.vocab), dtype=float32, name="logits")
+        self._linear(h, table, self.logits)
+        out = mpk.attach_input(mpk.meta_tensors["output_tokens"], name="output_token")
+        if mc.sampling_seed is not None:
+            mpk.sampling_sm100_layer(logits=self.logits, output=out, grid_dim=(mbt, 1, 1), block_dim=(256, 1, 1),
+                                     seed=mc.sampling_seed)
+            return
+        parts = max(1, min(mpk.num_workers, c.vocab // 64))
+        part_v = mpk.new_tensor(dims=(mbt, parts), dtype=float32, name="argmax_part_value")
+        part_i = mpk.new_tensor(dims=(mbt, parts), dtype=int64, name="argmax_part_index")
+        mpk.argmax_partial_layer(input=self.logits, output=(part_v, part_i), grid_dim=(parts, 1, 1), block_dim=(128, 1, 1))
+        mpk.argmax_reduce_layer(input=(part_v, part_i), output=out, grid_dim=(1, 1, 1), block_dim=(128, 1, 1))

@@ -1,4 +1,5 @@
-// The decode megakernel: one launch executes one iteration of the task graph.
+// The decode megakernel: one launch executes one iteration of the task graph.  Included by the files that
+// instantiate it (decoder_kernels.cu, hybrid_kernels.cu).
 //
 // Replaces the reference's persistent runtime (worker/scheduler loops and queues,
 // include/mirage/persistent_kernel/persistent_kernel.cuh:513-1082) and the task bodies
@@ -20,6 +21,7 @@
 // Every wait (event counter, mbarrier) is bounded by a wall-clock budget; on expiry the
 // CTA records where it gave up, raises a global abort flag that all other waits poll,
 // drains its own in-flight copies and returns.
+#pragma once
 #include <cuda_bf16.h>
 #include <cuda_fp8.h>
 #include <cuda_runtime.h>
@@ -43,7 +45,6 @@ struct Smem {
   uint32_t *tmem_holder;   // tensor-memory base address written by tcgen05.alloc
 };
 
-constexpr int kMiscBytes = 1536;
 constexpr int kStashRing = 16;     // attention stash records of the general instantiation (32 bytes each, after the flags)
 
 __device__ __forceinline__ Smem carve(uint8_t *base, const KernelParams &P) {
@@ -130,7 +131,7 @@ __device__ void prefetch_attention_kv_l2(const Ctx &c, const TaskDesc *d, int la
 // A linear task streams its weight panel [n0, n1) x K as chunks of 16 rows x KC columns (KC <= 1024):
 // one cp.async.bulk per row segment, rows padded by 16 bytes in shared memory so that ldmatrix reads
 // are bank-conflict free.  Order: k tile (activation tile) -> 16-row group -> k chunk.
-template <bool GENERAL>
+template <bool GENERAL, int HYB>
 __device__ void streamer_loop(const Ctx &c, int t_begin, int t_end) {
   const KernelParams &P = c.P;
   const int lane = threadIdx.x & 31;
@@ -146,8 +147,8 @@ __device__ void streamer_loop(const Ctx &c, int t_begin, int t_end) {
   // The whole warp walks the task list; lane 0 owns the barrier traffic, lane r copies row r of a chunk.
   for (int t = t_begin; t < t_end && ok; ++t) {
     const TaskDesc *d = &P.tasks[t];
-    if (d->type == TASK_ATTENTION && P.kv_l2_prefetch) prefetch_attention_kv_l2<GENERAL>(c, d, lane, t);
-    if (d->type != TASK_LINEAR && !(GENERAL && d->type == TASK_MOE_GEMM)) continue;
+    if (!HYB && d->type == TASK_ATTENTION && P.kv_l2_prefetch) prefetch_attention_kv_l2<GENERAL>(c, d, lane, t);
+    if (d->type != TASK_LINEAR && !(GENERAL && !HYB && d->type == TASK_MOE_GEMM)) continue;
     if (d->flags & TF_STREAM_AFTER_DEP) {
       if (lane == 0)
         for (int i = 0; i < kMaxDeps && ok; ++i)
@@ -164,7 +165,7 @@ __device__ void streamer_loop(const Ctx &c, int t_begin, int t_end) {
       // 128-byte-swizzled layout the MMA reads.  Order: k tile -> row tile -> k blocks.
       const uint8_t *tmap = reinterpret_cast<const uint8_t *>(P.tmaps) + (size_t)d->a[L_TMAP] * 128;
       const int rows = d->a[L_N1] - d->a[L_N0], RB = d->a[L_ROWS];
-      const int kbe = (d->flags & TF_FP8) ? 2 * kTcKBlock : kTcKBlock;   // elements of one 128-byte k block
+      const int kbe = (!HYB && (d->flags & TF_FP8)) ? 2 * kTcKBlock : kTcKBlock;   // elements of one 128-byte k block
       const int nkb = d->a[L_KC] / kbe, kbt = d->a[L_KT] / kbe, kball = d->a[L_K] / kbe;
       const int tiles = (rows + RB - 1) / RB;
       const uint32_t tx = (uint32_t)(nkb * RB * 128);
@@ -188,19 +189,19 @@ __device__ void streamer_loop(const Ctx &c, int t_begin, int t_end) {
     const uint8_t *W = reinterpret_cast<const uint8_t *>(d->p[0]);
     const int n0 = d->a[L_N0], n1 = d->a[L_N1], K = d->a[L_K], ldw = d->a[L_LDW];
     const int KT = d->a[L_KT], KC = d->a[L_KC], R = d->a[L_ROWS];
-    const uint32_t esz = (GENERAL && (d->flags & TF_FP8)) ? 1u : 2u;   // e4m3 or bf16 weights
+    const uint32_t esz = (GENERAL && !HYB && (d->flags & TF_FP8)) ? 1u : 2u;   // e4m3 or bf16 weights
     const uint32_t seg_bytes = (uint32_t)KC * esz;
     const uint32_t row_stride = seg_bytes + kRowPadBytes;
     // an expert task repeats the panel loop once per active expert (the list is final: the task waited for it)
     int reps = 1;
     const int *act = nullptr;
-    if (GENERAL && d->type == TASK_MOE_GEMM) {
+    if (GENERAL && !HYB && d->type == TASK_MOE_GEMM) {
       act = reinterpret_cast<const int *>(d->p[5]);
       reps = min(__ldcg(&act[d->a[M_NEXP]]), d->a[M_NEXP]);
     }
     for (int rep = 0; rep < reps && ok; ++rep) {
     const uint8_t *Wp = W;
-    if (GENERAL && act != nullptr) Wp = W + (size_t)__ldcg(&act[rep]) * (size_t)d->a[M_ESTRIDE] * esz;
+    if (GENERAL && !HYB && act != nullptr) Wp = W + (size_t)__ldcg(&act[rep]) * (size_t)d->a[M_ESTRIDE] * esz;
     for (int kt = 0; kt < K && ok; kt += KT) {
       for (int r0 = n0; r0 < n1 && ok; r0 += R) {
         const int rows = min(R, n1 - r0);
@@ -635,22 +636,22 @@ __device__ void stage_x(const Ctx &c, const TaskDesc &d, int B, int k0, int KT, 
 // Sum the 8 warps' partial tiles of one 16-row group and run the epilogue for its rows.
 // WIDE = false: at most 8 tokens, every warp holds the same token tile (the batch-1 hot path, all constants);
 // WIDE = true: warp w holds token tile w % NT (8 tokens each) and every (8 / NT)-th k step.
-template <bool WIDE>
+template <bool WIDE, int HYB>
 __device__ __forceinline__ void linear_output(const Ctx &c, const TaskDesc &d, int NT, int r0, int rows,
                                               const float *part, int item);
 
-template <bool WIDE>
+template <bool WIDE, int HYB>
 __device__ __forceinline__ void linear_group_epilogue(const Ctx &c, const TaskDesc &d, int B, int NT, int r0, int rows,
                                                       const float *part) {
   if (!WIDE) {
     const int tid = threadIdx.x;
-    if (tid < 128 && (tid >> 4) < B) linear_output<false>(c, d, 1, r0, rows, part, tid);
+    if (tid < 128 && (tid >> 4) < B) linear_output<false, HYB>(c, d, 1, r0, rows, part, tid);
   } else {
-    for (int item = threadIdx.x; item < B * 16; item += kConsumerThreads) linear_output<true>(c, d, NT, r0, rows, part, item);
+    for (int item = threadIdx.x; item < B * 16; item += kConsumerThreads) linear_output<true, HYB>(c, d, NT, r0, rows, part, item);
   }
 }
 
-template <bool WIDE>
+template <bool WIDE, int HYB>
 __device__ __forceinline__ void linear_output(const Ctx &c, const TaskDesc &d, int NT, int r0, int rows,
                                               const float *part, int item) {
   const KernelParams &P = c.P;
@@ -699,6 +700,11 @@ __device__ __forceinline__ void linear_output(const Ctx &c, const TaskDesc &d, i
       __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(d.p[2]);
       out[(size_t)b * d.a[L_LDO] + ((col >> 2) << 1) + (r & 1)] = __float2bfloat16_rn(a * round_bf16(u));
     }
+  } else if (HYB && epi == EPI_STORE_F32) {
+    reinterpret_cast<float *>(d.p[2])[(size_t)b * d.a[L_LDO] + col] = v;
+  } else if (HYB && epi == EPI_RELU2) {
+    const float a = fmaxf(v, 0.f);
+    reinterpret_cast<__nv_bfloat16 *>(d.p[2])[(size_t)b * d.a[L_LDO] + col] = __float2bfloat16_rn(a * a);
   } else {
     __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(d.p[2]);
     if (epi == EPI_RESIDUAL) {
@@ -709,7 +715,7 @@ __device__ __forceinline__ void linear_output(const Ctx &c, const TaskDesc &d, i
   }
 }
 
-template <bool WIDE, bool TPX = false>
+template <bool WIDE, bool TPX = false, int HYB = 0>
 __device__ __forceinline__ void run_linear(const Ctx &c, const TaskDesc &d, LinearState &ls, int task,
                                            const uint4 (&gpre)[2], bool ok) {
   const KernelParams &P = c.P;
@@ -800,7 +806,7 @@ __device__ __forceinline__ void run_linear(const Ctx &c, const TaskDesc &d, Line
         }
         if (!multi_tile) {
           consumer_sync();
-          linear_group_epilogue<WIDE>(c, d, B, NT, r0, min(R, n1 - r0), part);
+          linear_group_epilogue<WIDE, HYB>(c, d, B, NT, r0, min(R, n1 - r0), part);
         }
       }
       ++group_seq;
@@ -812,7 +818,7 @@ __device__ __forceinline__ void run_linear(const Ctx &c, const TaskDesc &d, Line
     consumer_sync();
     int gi = 0;
     for (int r0 = n0; r0 < n1; r0 += R, ++gi)
-      linear_group_epilogue<WIDE>(c, d, B, NT, r0, min(R, n1 - r0), c.s.partial + (size_t)(gi & 1) * (8 * 16 * 8));
+      linear_group_epilogue<WIDE, HYB>(c, d, B, NT, r0, min(R, n1 - r0), c.s.partial + (size_t)(gi & 1) * (8 * 16 * 8));
   }
 }
 
@@ -849,6 +855,7 @@ __device__ __forceinline__ EmitArgs emit_args(const Ctx &c, const TaskDesc &d) {
   return e;
 }
 
+template <int HYB>
 __device__ __forceinline__ void linear_emit(const Ctx &c, const EmitArgs &e, int b, int col, float v, float u, float resv) {
   if (e.epi == EPI_PUSH_LL) {
     // one 32-bit word per element: bf16 partial sum in the low half, sequence number in the high half
@@ -868,11 +875,17 @@ __device__ __forceinline__ void linear_emit(const Ctx &c, const EmitArgs &e, int
       const float a = round_bf16(silu_f(round_bf16(v)));
       e.out[(size_t)b * e.ldo + ((col >> 2) << 1) + (col & 1)] = __float2bfloat16_rn(a * round_bf16(u));
     }
+  } else if (HYB && e.epi == EPI_STORE_F32) {
+    reinterpret_cast<float *>(e.out)[(size_t)b * e.ldo + col] = v;
+  } else if (HYB && e.epi == EPI_RELU2) {
+    const float a = fmaxf(v, 0.f);
+    e.out[(size_t)b * e.ldo + col] = __float2bfloat16_rn(a * a);
   } else {
     e.out[(size_t)b * e.ldo + col] = __float2bfloat16_rn(v + resv);   // resv: the residual element, or 0
   }
 }
 
+template <int HYB>
 __device__ void run_linear_tc(const Ctx &c, const TaskDesc &d, LinearState &ls, int task, const uint4 (&gpre)[2], bool ok) {
   const KernelParams &P = c.P;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -987,7 +1000,7 @@ __device__ void run_linear_tc(const Ctx &c, const TaskDesc &d, LinearState &ls, 
           const float v = __uint_as_float(r[j]);
           const float u = (epi == EPI_SILU_PAIR) ? __shfl_down_sync(0xffffffffu, v, 2) : 0.f;
           const int b = half * nh + c0 + j;
-          if (row_ok && b < B) linear_emit(c, ea, b, n0 + row, v, u, resv[j]);
+          if (row_ok && b < B) linear_emit<HYB>(c, ea, b, n0 + row, v, u, resv[j]);
         }
         if (tid == 0 && prof && tile == 0 && c0 == 0) P.profiler[(size_t)task * 8 + 7] = globaltimer_ns();
       }
@@ -1163,7 +1176,7 @@ __device__ void run_linear_fp8_tc(const Ctx &c, const TaskDesc &d, LinearState &
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
           const int b = half * nh + c0 + j;
-          if (row_ok && b < B) linear_emit(c, ea, b, n0 + row, __uint_as_float(r[j]), 0.f, resv[j]);
+          if (row_ok && b < B) linear_emit<0>(c, ea, b, n0 + row, __uint_as_float(r[j]), 0.f, resv[j]);
         }
       }
     }
@@ -1347,7 +1360,7 @@ __device__ __forceinline__ void run_linear_fp8(const Ctx &c, const TaskDesc &d, 
         }
         if (!multi_tile) {
           consumer_sync();
-          linear_group_epilogue<true>(c, d, B, NT, r0, min(R, n1 - r0), part);
+          linear_group_epilogue<true, 0>(c, d, B, NT, r0, min(R, n1 - r0), part);
         }
       }
       ++group_seq;
@@ -1358,7 +1371,7 @@ __device__ __forceinline__ void run_linear_fp8(const Ctx &c, const TaskDesc &d, 
     consumer_sync();
     int gi = 0;
     for (int r0 = n0; r0 < n1; r0 += R, ++gi)
-      linear_group_epilogue<true>(c, d, B, NT, r0, min(R, n1 - r0), c.s.partial + (size_t)(gi & 1) * (8 * 16 * 8));
+      linear_group_epilogue<true, 0>(c, d, B, NT, r0, min(R, n1 - r0), c.s.partial + (size_t)(gi & 1) * (8 * 16 * 8));
   }
   ls.stage = stage;
   ls.phase = phase;
@@ -3239,9 +3252,12 @@ __device__ __forceinline__ void sample_merge(float &v, long long &i, float v2, l
 
 // One column range of the vocabulary: key = bf16(logit + bf16(noise)), noise by groups of four columns from one
 // Philox block whose subsequence is (row within the reference task) * V + first column of the group.
+__device__ __forceinline__ float logit_value(const __nv_bfloat16 *p) { return bf16_to_f(__ldcg(p)); }
+__device__ __forceinline__ float logit_value(const float *p) { return round_bf16(__ldcg(p)); }
+template <typename LOGIT>
 __device__ void run_sampling_partial(const Ctx &c, const TaskDesc &d) {
   const int B = active_tokens(c.P);
-  const __nv_bfloat16 *logits = reinterpret_cast<const __nv_bfloat16 *>(d.p[0]);
+  const LOGIT *logits = reinterpret_cast<const LOGIT *>(d.p[0]);
   __nv_bfloat16 *pv = reinterpret_cast<__nv_bfloat16 *>(d.p[1]);
   long long *pi = reinterpret_cast<long long *>(d.p[2]);
   const int c0 = d.a[0], c1 = d.a[1], cid = d.a[2], ldl = d.a[3], ldp = d.a[4];
@@ -3262,7 +3278,7 @@ __device__ void run_sampling_partial(const Ctx &c, const TaskDesc &d) {
         const int j = q * 4 + e;
         if (j >= c0 && j < c1) {
           const float noise = bf16_to_f(__float2bfloat16_rn(gumbel_noise(rr[e])));
-          const float k = bf16_to_f(__float2bfloat16_rn(bf16_to_f(__ldcg(&logits[(size_t)b * ldl + j])) + noise));
+          const float k = bf16_to_f(__float2bfloat16_rn(logit_value(&logits[(size_t)b * ldl + j]) + noise));
           sample_merge(v, i, k, (long long)j);
         }
       }
@@ -3455,6 +3471,12 @@ __device__ void run_ar_push(const Ctx &c, const TaskDesc &d) {
 // TASK_BATCH: device-side continuous batching, block-parallel.
 // Same result, array by array, as the reference's single-threaded
 // prepare_next_batch (include/mirage/persistent_kernel/persistent_kernel.cuh:206-368).
+// Two additions:
+//   * every live request owns a recurrent-state slot (M.state_slots[batch slot]): the lowest free one when it is
+//     admitted, kept while the batch is compacted around it, free again when it retires;
+//   * online mode (M.request_ctl given): rows of the token table are requests the host posts, extends and closes
+//     while the loop runs (REQ_* in runtime_types.h), admitted in row order; a request advances no further than the
+//     tokens the host has supplied (REQ_HOLD) or decodes on its own (REQ_RUN), and never further than the free pages.
 // ---------------------------------------------------------------------------
 __device__ __noinline__ void run_batch(const Ctx c) {
   if (c.tmem_base & 0x80000000u) {   // called for TASK_ARGMAX_EXCHANGE (see task_other)
@@ -3479,11 +3501,23 @@ __device__ __noinline__ void run_batch(const Ctx c) {
   int *n_src = n_old + mbr;        // [mbr]  old kv offset of carried pages
   int *n_newoff = n_src + mbr;     // [mbr]  offset into freshly allocated pages
   int *n_step = n_newoff + mbr;    // [mbr]  token read offset in `tokens`
-  int *sc = n_step + mbr;          // scalars: [0] head [1] tail [2] next_req [3] num_reqs [4] num_tokens [5] num_pages
+  int *s_slot = n_step + mbr;      // [mbr]  state slot per old batch slot
+  int *n_slot = s_slot + mbr;      // [mbr]  state slot per new batch slot
+  int *s_used = n_slot + mbr;      // [mbr]  state slot taken
+  int *sc = s_used + mbr;          // scalars: [0] head [1] tail [2] next_req [3] num_reqs [4] num_tokens [5] num_pages
+  int *s_ctl = sc + 16;            // [total_num_requests] online mode: control word | live << 8
+  const bool online = M.request_ctl != nullptr;
+  const int R = P.total_num_requests;
 
   const int prev_tokens = M.qo_indptr[mbr];   // active tokens of the previous iteration (0 after a reset)
   if (tid < 3) sc[tid] = M.sched_scalars[tid];
   for (int i = tid; i <= mbr; i += kConsumerThreads) s_kv[i] = M.paged_kv_indptr[i];
+  for (int i = tid; i < mbr; i += kConsumerThreads) {
+    s_slot[i] = M.state_slots[i];
+    s_used[i] = 0;
+  }
+  if (online)
+    for (int r = tid; r < R; r += kConsumerThreads) s_ctl[r] = (M.request_ctl[r] & 0xff) | (M.request_ctl[R + r] ? 0x100 : 0);
   consumer_sync();
   // Step 1: commit outputs, advance steps, retire finished requests.
   // s_rid: request id, -1 for an empty slot, -2 for a request retired in this step.
@@ -3500,8 +3534,18 @@ __device__ __noinline__ void run_batch(const Ctx c) {
           M.tokens[(size_t)rid * S + step + j + 1] = M.output_tokens[qo + j];
       step_new = step + n;
       M.step[rid] = step_new;
-      const bool done = (step_new + 1 >= S) ||
-                        (M.tokens[(size_t)rid * S + step_new] == P.eos_token_id && step_new >= plen);
+      bool done = (step_new + 1 >= S) ||
+                  (M.tokens[(size_t)rid * S + step_new] == P.eos_token_id && step_new >= plen);
+      if (online) {
+        const int ctl = s_ctl[rid] & 0xff;
+        if (ctl == REQ_HOLD) done = false;
+        else if (ctl == REQ_CLOSE) done = step_new >= plen;
+        if (done) {
+          s_ctl[rid] = 0;
+          M.request_ctl[rid] = REQ_FREE;
+          M.request_ctl[R + rid] = 0;
+        }
+      }
       if (done) {
         freed = s_kv[i + 1] - s_kv[i];
         rid = -2;
@@ -3536,6 +3580,7 @@ __device__ __noinline__ void run_batch(const Ctx c) {
   if (tid == 0) {
     int num_reqs = 0, num_tokens = 0, num_pages = 0, new_pages = 0;
     int head = sc[0];
+    const int avail = sc[1] + s_free[mbr] - head;   // free pages
     for (int i = 0; i < mbr; ++i) {
       const int rid = s_rid[i];
       if (rid < 0) continue;
@@ -3543,6 +3588,12 @@ __device__ __noinline__ void run_batch(const Ctx c) {
       int nn = s_plen[i] - step;
       nn = (nn > 0) ? min(nn, mbt - num_tokens) : min(1, mbt - num_tokens);
       const int n_old_pages = s_kv[i + 1] - s_kv[i];
+      if (online) {
+        if (s_plen[i] <= step && (s_ctl[rid] & 0xff) != REQ_RUN) nn = 0;
+        nn = max(0, min(nn, (n_old_pages + avail - new_pages) * PS - step));
+      }
+      n_slot[num_reqs] = s_slot[i];
+      if ((unsigned)s_slot[i] < (unsigned)mbr) s_used[s_slot[i]] = 1;
       const int np = (step + nn + PS - 1) / PS;
       n_rid[num_reqs] = rid;
       n_tok[num_reqs] = num_tokens;
@@ -3556,10 +3607,22 @@ __device__ __noinline__ void run_batch(const Ctx c) {
       num_tokens += nn;
       ++num_reqs;
     }
-    int next = sc[2];
+    int next = online ? 0 : sc[2], slot = 0;
     while (num_reqs < mbr && num_tokens < mbt && next < P.total_num_requests) {
-      const int nn = min(M.prompt_lengths[next], mbt - num_tokens);
+      int nn = mbt - num_tokens;
+      if (online) {
+        const int ctl = s_ctl[next];
+        if (ctl != REQ_RUN && ctl != REQ_HOLD && ctl != REQ_CLOSE) { ++next; continue; }   // free row, or live already
+        nn = min(nn, (avail - new_pages) * PS);
+        if (nn <= 0) break;
+        M.step[next] = 0;
+        M.request_ctl[R + next] = 1;
+      }
+      nn = min(M.prompt_lengths[next], nn);
       const int np = (nn + PS - 1) / PS;
+      while (slot < mbr - 1 && s_used[slot]) ++slot;
+      s_used[slot] = 1;
+      n_slot[num_reqs] = slot;
       n_rid[num_reqs] = next;
       n_tok[num_reqs] = num_tokens;
       n_pg[num_reqs] = num_pages;
@@ -3581,7 +3644,7 @@ __device__ __noinline__ void run_batch(const Ctx c) {
     sc[6] = head;              // ring position of the first fresh page
     sc[0] = head + new_pages;
     sc[1] = sc[1] + s_free[mbr];
-    sc[2] = next;
+    sc[2] = online ? 0 : next;
   }
   consumer_sync();
   const int num_reqs = sc[3], num_tokens = sc[4], num_pages = sc[5], head0 = sc[6];
@@ -3602,6 +3665,7 @@ __device__ __noinline__ void run_batch(const Ctx c) {
   for (int k = tid; k < mbr; k += kConsumerThreads) {
     if (k < num_reqs) {
       M.request_ids[k] = n_rid[k];
+      M.state_slots[k] = n_slot[k];
       M.qo_indptr[k] = n_tok[k];
       M.paged_kv_indptr[k] = n_pg[k];
       const int tot = n_step[k] + (n_tok[k + 1] - n_tok[k]);
@@ -3634,6 +3698,12 @@ __device__ __noinline__ void run_batch(const Ctx c) {
   }
 }
 
+}  // namespace mpk
+
+#include "hybrid_tasks.cuh"
+
+namespace mpk {
+
 // ---------------------------------------------------------------------------
 // compute warps: walk the task list
 // ---------------------------------------------------------------------------
@@ -3664,7 +3734,7 @@ __device__ __forceinline__ bool wait_dependencies(const Ctx &c, const TaskDesc &
 
 // Each task kind has its own non-inlined runner so that register allocation of the heavy bodies
 // (attention) does not leak into the weight-streaming loop.
-template <bool GENERAL, bool TPX>
+template <bool GENERAL, bool TPX, int HYB>
 __device__ __forceinline__ bool task_linear(const Ctx &c, const TaskDesc &d, int t, bool ok, TaskTimes &tt,
                                          LinearState &ls) {
   const int tid = threadIdx.x;
@@ -3678,10 +3748,10 @@ __device__ __forceinline__ bool task_linear(const Ctx &c, const TaskDesc &d, int
   }
   ok = wait_dependencies(c, d, t, ok, tt);
   // the weight chunks must be consumed even when the launch is being abandoned or no token is active
-  if (GENERAL && (d.flags & TF_TC) && (d.flags & TF_FP8)) run_linear_fp8_tc(c, d, ls, t, ok);
-  else if (GENERAL && (d.flags & TF_TC)) run_linear_tc(c, d, ls, t, gpre, ok);
-  else if (GENERAL && (d.flags & TF_FP8)) run_linear_fp8(c, d, ls, t, ok);
-  else run_linear<GENERAL, TPX>(c, d, ls, t, gpre, ok);
+  if (GENERAL && !HYB && (d.flags & TF_TC) && (d.flags & TF_FP8)) run_linear_fp8_tc(c, d, ls, t, ok);
+  else if (GENERAL && (d.flags & TF_TC)) run_linear_tc<HYB>(c, d, ls, t, gpre, ok);
+  else if (GENERAL && !HYB && (d.flags & TF_FP8)) run_linear_fp8(c, d, ls, t, ok);
+  else run_linear<GENERAL, TPX, HYB>(c, d, ls, t, gpre, ok);
   return ok;
 }
 
@@ -3717,10 +3787,14 @@ __device__ __forceinline__ bool task_attention(const Ctx &c, const TaskDesc &d, 
   return ok;
 }
 
-template <bool GENERAL, bool TPX>
+template <bool GENERAL, bool TPX, int HYB>
 __device__ __forceinline__ bool task_other(const Ctx &c, const TaskDesc &d, int t, bool ok, TaskTimes &tt) {
   ok = wait_dependencies(c, d, t, ok, tt);
   if (!ok) return false;
+  if (HYB) {
+    run_hybrid_task<HYB>(c, d);
+    return true;
+  }
   switch (d.type) {
     // (the argmax exchange of multi-rank graphs shares the batching task's out-of-line function and its call site: a
     // second call in this switch moved the register allocation of the linear loop; bit 31 of the tensor-memory field,
@@ -3747,7 +3821,7 @@ __device__ __forceinline__ bool task_other(const Ctx &c, const TaskDesc &d, int 
     case TASK_MLA_APPEND: if (GENERAL) run_mla_append(c, d); break;
     case TASK_MLA_DECODE: if (GENERAL) run_mla_decode(c, d); break;
     case TASK_MLA_REDUCE: if (GENERAL) run_mla_reduce(c, d); break;
-    case TASK_SAMPLING_PARTIAL: if (GENERAL) run_sampling_partial(c, d); break;
+    case TASK_SAMPLING_PARTIAL: if (GENERAL) run_sampling_partial<__nv_bfloat16>(c, d); break;
     case TASK_SAMPLING_REDUCE: if (GENERAL) run_sampling_reduce(c, d); break;
     case TASK_AR_PUSH: if (GENERAL && TPX) run_ar_push(c, d); break;
     default: break;
@@ -3755,7 +3829,7 @@ __device__ __forceinline__ bool task_other(const Ctx &c, const TaskDesc &d, int 
   return true;
 }
 
-template <bool GENERAL, bool TPX>
+template <bool GENERAL, bool TPX, int HYB>
 __device__ void consumer_loop(const Ctx &c, int t_begin, int t_end) {
   const KernelParams &P = c.P;
   const int tid = threadIdx.x;
@@ -3771,12 +3845,12 @@ __device__ void consumer_loop(const Ctx &c, int t_begin, int t_end) {
     if (fetch) nxt = __ldg(reinterpret_cast<const uint4 *>(&P.tasks[t + 1]) + (tid - 224));
     TaskTimes tt{0, 0, (P.profiler != nullptr) && (uint64_t)(t + 1) * 8 <= P.profiler_entries};
     const uint32_t type = d.type;
-    if (type == TASK_LINEAR) ok = task_linear<GENERAL, TPX>(c, d, t, ok, tt, ls);
-    else if (GENERAL && type == TASK_MOE_GEMM) {
+    if (HYB != HYB_F32 && type == TASK_LINEAR) ok = task_linear<GENERAL, TPX, HYB>(c, d, t, ok, tt, ls);
+    else if (GENERAL && !HYB && type == TASK_MOE_GEMM) {
       ok = wait_dependencies(c, d, t, ok, tt);
       run_moe_gemm(c, d, ls, t, ok);
-    } else if (type == TASK_ATTENTION) ok = task_attention<GENERAL>(c, d, t, ok, tt);
-    else ok = task_other<GENERAL, TPX>(c, d, t, ok, tt);
+    } else if (!HYB && type == TASK_ATTENTION) ok = task_attention<GENERAL>(c, d, t, ok, tt);
+    else ok = task_other<GENERAL, TPX, HYB>(c, d, t, ok, tt);
     if (fetch) reinterpret_cast<uint4 *>(&c.s.desc[(t + 1 - t_begin) & 1])[tid - 224] = nxt;
     const int trig = d.trig_event;
     const uint32_t tflags = d.flags;
@@ -3812,7 +3886,10 @@ __device__ void consumer_loop(const Ctx &c, int t_begin, int t_end) {
 // single-GPU paths had been tuned sits behind it -- the allreduce prologue with all ranks' loads in flight (batch-1
 // kernel), the argmax exchange of a sharded lm_head -- so that the single-GPU instantiations <*, false> stay exactly
 // the code that was measured: both run at the register cap, where unrelated code moves their allocation.
-template <bool GENERAL, bool TPX = false>
+// HYB marks the instantiations of graphs with recurrent or extended-attention layers (hybrid_tasks.cuh): they hold the
+// linear bodies and the hybrid tasks only.  HYB_BF16 serves in bf16; HYB_F32 computes everything in 32-bit floats and has
+// no tensor-core code at all.
+template <bool GENERAL, bool TPX = false, int HYB = 0>
 __global__ void __launch_bounds__(kBlockThreads, 1) mpk_megakernel(const __grid_constant__ KernelParams P) {
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   Smem s = carve(smem_raw, P);
@@ -3843,9 +3920,9 @@ __global__ void __launch_bounds__(kBlockThreads, 1) mpk_megakernel(const __grid_
         use_tmem ? *reinterpret_cast<volatile uint32_t *>(s.tmem_holder) : 0u};
   const int t_begin = P.worker_begin[blockIdx.x], t_end = P.worker_begin[blockIdx.x + 1];
   if (tid >= kConsumerThreads) {
-    streamer_loop<GENERAL>(c, t_begin, t_end);
+    streamer_loop<GENERAL, HYB>(c, t_begin, t_end);
   } else {
-    consumer_loop<GENERAL, TPX>(c, t_begin, t_end);
+    consumer_loop<GENERAL, TPX, HYB>(c, t_begin, t_end);
   }
   if (use_tmem) tc_fence_before_sync();
   __syncthreads();
@@ -3878,72 +3955,3 @@ __global__ void __launch_bounds__(kBlockThreads, 1) mpk_megakernel(const __grid_
 
 }  // namespace mpk
 
-// ---------------------------------------------------------------------------
-// host-side launch glue (called from the C ABI implementation)
-// ---------------------------------------------------------------------------
-extern "C" int mpk_kernel_smem_bytes(int num_stages, int stage_bytes, int x_tile_bytes) {
-  return num_stages * stage_bytes + x_tile_bytes + mpk::kPartialBytes + mpk::kMiscBytes;
-}
-
-// The limit is a property of the function on the current device, shared by every handle of the process: it is raised
-// to the device's opt-in maximum (not to this handle's need), so that preparing a graph with a small footprint cannot
-// lower it under a graph prepared earlier.
-extern "C" int mpk_kernel_prepare(int smem_bytes) {
-  int dev = 0, limit = 0;
-  cudaError_t e = cudaGetDevice(&dev);
-  if (e == cudaSuccess) e = cudaDeviceGetAttribute(&limit, cudaDevAttrMaxSharedMemoryPerBlockOptin, dev);
-  if (e != cudaSuccess) return (int)e;
-  if (smem_bytes > limit) return (int)cudaErrorInvalidValue;
-  smem_bytes = limit;
-  e = cudaFuncSetAttribute(mpk::mpk_megakernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_bytes);
-  if (e == cudaSuccess)
-    e = cudaFuncSetAttribute(mpk::mpk_megakernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_bytes);
-  if (e == cudaSuccess)
-    e = cudaFuncSetAttribute(mpk::mpk_megakernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_bytes);
-  if (e == cudaSuccess)
-    e = cudaFuncSetAttribute(mpk::mpk_megakernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_bytes);
-  return e == cudaSuccess ? 0 : (int)e;
-}
-
-extern "C" int mpk_kernel_launch(const mpk::KernelParams *params, int smem_bytes, void *stream) {
-  if (params->general_kernel && params->world_size > 1)
-    mpk::mpk_megakernel<true, true><<<params->num_workers, mpk::kBlockThreads, smem_bytes, (cudaStream_t)stream>>>(*params);
-  else if (params->general_kernel)
-    mpk::mpk_megakernel<true><<<params->num_workers, mpk::kBlockThreads, smem_bytes, (cudaStream_t)stream>>>(*params);
-  else if (params->world_size > 1 && params->tp_extensions)
-    mpk::mpk_megakernel<false, true><<<params->num_workers, mpk::kBlockThreads, smem_bytes, (cudaStream_t)stream>>>(*params);
-  else
-    mpk::mpk_megakernel<false><<<params->num_workers, mpk::kBlockThreads, smem_bytes, (cudaStream_t)stream>>>(*params);
-  cudaError_t e = cudaGetLastError();
-  return e == cudaSuccess ? 0 : (int)e;
-}
-
-__global__ void mpk_shuffle_rows_kernel(uint8_t *dst, const uint8_t *const *srcs, const int64_t *rows_per_group,
-                                        const int64_t *prefix_rows, int n, int64_t group_rows_total,
-                                        int64_t row_bytes, int64_t total_rows) {
-  // dst row r: group g = r / group_rows_total, offset o within the group; tensor i with prefix[i] <= o < prefix[i+1]
-  for (int64_t r = blockIdx.x; r < total_rows; r += gridDim.x) {
-    const int64_t g = r / group_rows_total, o = r - g * group_rows_total;
-    int i = 0;
-    while (i + 1 < n && o >= prefix_rows[i + 1]) ++i;
-    const uint8_t *src = srcs[i] + ((g * rows_per_group[i]) + (o - prefix_rows[i])) * row_bytes;
-    uint8_t *d = dst + r * row_bytes;
-    if (row_bytes % 16 == 0) {
-      for (int64_t b = threadIdx.x * 16; b < row_bytes; b += blockDim.x * 16)
-        *reinterpret_cast<uint4 *>(d + b) = *reinterpret_cast<const uint4 *>(src + b);
-    } else {   // narrow rows (e.g. the packed scale words of a small weight): 4-byte words
-      for (int64_t b = threadIdx.x * 4; b < row_bytes; b += blockDim.x * 4)
-        *reinterpret_cast<uint32_t *>(d + b) = *reinterpret_cast<const uint32_t *>(src + b);
-    }
-  }
-}
-
-extern "C" int mpk_shuffle_rows_launch(void *dst, const void *const *srcs_dev, const int64_t *rows_per_group_dev,
-                                       const int64_t *prefix_rows_dev, int n, int64_t group_rows_total,
-                                       int64_t row_bytes, int64_t total_rows, void *stream) {
-  mpk_shuffle_rows_kernel<<<1024, 256, 0, (cudaStream_t)stream>>>(
-      (uint8_t *)dst, (const uint8_t *const *)srcs_dev, rows_per_group_dev, prefix_rows_dev, n, group_rows_total,
-      row_bytes, total_rows);
-  cudaError_t e = cudaGetLastError();
-  return e == cudaSuccess ? 0 : (int)e;
-}

@@ -6,6 +6,7 @@
 // launches the pre-built megakernel once per decode iteration.
 #include <cuda.h>
 #include <cuda_runtime.h>
+#include <dlfcn.h>
 
 #include <algorithm>
 #include <cstdio>
@@ -19,14 +20,47 @@
 #include "runtime_types.h"
 #include "task_graph.h"
 
-extern "C" int mpk_kernel_smem_bytes(int num_stages, int stage_bytes, int x_tile_bytes);
-extern "C" int mpk_kernel_prepare(int smem_bytes);
-extern "C" int mpk_kernel_launch(const mpk::KernelParams *params, int smem_bytes, void *stream);
 extern "C" int mpk_shuffle_rows_launch(void *dst, const void *const *srcs_dev, const int64_t *rows_per_group_dev,
                                        const int64_t *prefix_rows_dev, int n, int64_t group_rows_total,
                                        int64_t row_bytes, int64_t total_rows, void *stream);
 
 using namespace mpk;
+
+// The megakernel instantiations live in one library per family, beside this one; a graph loads the family it needs.
+struct KernelFamily {
+  int (*prepare)(int smem_bytes, int flags) = nullptr;
+  int (*launch)(const KernelParams *params, int smem_bytes, void *stream) = nullptr;
+};
+
+static int load_family(bool hybrid, KernelFamily *out, std::string *err) {
+  static KernelFamily loaded[2];
+  KernelFamily &f = loaded[hybrid ? 1 : 0];
+  if (!f.launch) {
+    Dl_info info;
+    if (!dladdr(reinterpret_cast<const void *>(&load_family), &info) || !info.dli_fname) {
+      *err = "cannot locate the library's own path";
+      return MPK_ERR_STATE;
+    }
+    std::string dir(info.dli_fname);
+    const size_t cut = dir.rfind('/');
+    dir = cut == std::string::npos ? std::string(".") : dir.substr(0, cut);
+    const std::string path = dir + (hybrid ? "/libmpk_b200_hybrid.so" : "/libmpk_b200_decoder.so");
+    void *so = dlopen(path.c_str(), RTLD_NOW | RTLD_LOCAL);
+    if (!so) {
+      *err = std::string("kernel library not loaded: ") + dlerror() + " (build it with `python mirage_b200/build.py`)";
+      return MPK_ERR_STATE;
+    }
+    f.prepare = reinterpret_cast<int (*)(int, int)>(dlsym(so, "mpk_family_prepare"));
+    f.launch = reinterpret_cast<int (*)(const KernelParams *, int, void *)>(dlsym(so, "mpk_family_launch"));
+    if (!f.prepare || !f.launch) {
+      f = KernelFamily();
+      *err = "kernel library without its entry points: " + path;
+      return MPK_ERR_STATE;
+    }
+  }
+  *out = f;
+  return MPK_OK;
+}
 
 struct mpk_handle {
   mpk_config cfg;
@@ -49,11 +83,12 @@ struct mpk_handle {
   uint64_t counters_bytes = 0;
   void *peer_comm[kMaxWorld] = {};
   bool peer_opened[kMaxWorld] = {};
-  int32_t *d_request_ids = nullptr, *d_page_queue = nullptr, *d_sched = nullptr;
+  int32_t *d_request_ids = nullptr, *d_state_slots = nullptr, *d_page_queue = nullptr, *d_sched = nullptr;
   float *d_attn_scratch = nullptr;
   unsigned int *d_attn_tickets = nullptr;
   void *d_tmaps = nullptr;            // tensor maps of the tcgen05 linear tasks
   KernelParams params;
+  KernelFamily kernels;
   uint64_t fake_ptr = 0x100000;       // dry-run address allocator
 };
 
@@ -182,6 +217,11 @@ int mpk_create(const mpk_config *cfg, mpk_handle **out) {
     if (cfg->page_size < 1 || cfg->max_num_pages < 1 || cfg->max_seq_length < 1)
       return set_err(h, MPK_ERR_INVALID, "page_size, max_num_pages, max_seq_length must be >= 1");
     const bool online = cfg->mode == MPK_MODE_ONLINE_NOTOKEN;
+    if (cfg->mode < MPK_MODE_OFFLINE || cfg->mode > MPK_MODE_ONLINE) return set_err(h, MPK_ERR_INVALID, "unknown mode");
+    if (!cfg->dry_run && cfg->mode == MPK_MODE_ONLINE && !cfg->request_ctl)
+      return set_err(h, MPK_ERR_INVALID, "online mode needs request_ctl");
+    if (cfg->mode == MPK_MODE_ONLINE && cfg->total_num_requests > 4096)
+      return set_err(h, MPK_ERR_UNSUPPORTED, "online mode: more than 4096 token-table rows");
     if (!cfg->dry_run && (!cfg->input_tokens || !cfg->qo_indptr || !cfg->paged_kv_indptr || !cfg->paged_kv_indices ||
                           !cfg->paged_kv_last_page_len))
       return set_err(h, MPK_ERR_INVALID, "the batch description (input_tokens, qo_indptr, paged_kv_*) is required");
@@ -356,13 +396,16 @@ int mpk_compile(mpk_handle *h) {
   CompiledGraph &g = h->graph;
   if (g.num_stages > 8)   // entries 8.. of the 16-entry barrier arrays are scratch (attention stash, accumulator barrier)
     return set_err(h, MPK_ERR_UNSUPPORTED, "internal: more than 8 weight stages planned");
-  h->smem_bytes = mpk_kernel_smem_bytes(g.num_stages, g.stage_bytes, g.x_tile_bytes);
+  h->smem_bytes = g.num_stages * g.stage_bytes + g.x_tile_bytes + kPartialBytes + kMiscBytes;
   // 5. runtime buffers
   h->counters_bytes = ((uint64_t)g.num_events * 8 + 255) / 256 * 256;
   h->comm_bytes = h->counters_bytes + (uint64_t)2 * g.inbox_floats_per_buffer * 4 + 256;
   rc = dev_alloc(h, (void **)&h->comm, h->comm_bytes); if (rc) return rc;
   rc = dev_alloc(h, (void **)&h->d_status, sizeof(DeviceStatus)); if (rc) return rc;
   rc = dev_alloc(h, (void **)&h->d_request_ids, (uint64_t)cfg.max_num_batched_requests * 4); if (rc) return rc;
+  if (!cfg.test_mode && cfg.mode != MPK_MODE_ONLINE_NOTOKEN && !cfg.state_slots) {
+    rc = dev_alloc(h, (void **)&h->d_state_slots, (uint64_t)cfg.max_num_batched_requests * 4); if (rc) return rc;
+  }
   rc = dev_alloc(h, (void **)&h->d_page_queue, (uint64_t)std::max(cfg.max_num_pages, 1) * 4); if (rc) return rc;
   rc = dev_alloc(h, (void **)&h->d_sched, 64); if (rc) return rc;
   rc = dev_alloc(h, (void **)&h->d_attn_scratch, (uint64_t)g.attn_scratch_floats * 4); if (rc) return rc;
@@ -393,7 +436,9 @@ int mpk_compile(mpk_handle *h) {
   P.meta.qo_indptr = cfg.qo_indptr; P.meta.paged_kv_indptr = cfg.paged_kv_indptr;
   P.meta.paged_kv_indices = cfg.paged_kv_indices; P.meta.paged_kv_last_page_len = cfg.paged_kv_last_page_len;
   P.meta.paged_kv_indices_snapshot = snapshot;
-  P.meta.request_ids = h->d_request_ids; P.meta.page_queue = h->d_page_queue; P.meta.sched_scalars = h->d_sched;
+  P.meta.request_ids = cfg.request_ids ? cfg.request_ids : h->d_request_ids; P.meta.page_queue = h->d_page_queue; P.meta.sched_scalars = h->d_sched;
+  P.meta.state_slots = cfg.state_slots ? cfg.state_slots : h->d_state_slots;
+  P.meta.request_ctl = (cfg.mode == MPK_MODE_ONLINE && !cfg.test_mode) ? cfg.request_ctl : nullptr;
   P.attn_scratch = h->d_attn_scratch;
   P.attn_tickets = h->d_attn_tickets;
   P.profiler = cfg.profiler_buffer;
@@ -414,6 +459,7 @@ int mpk_compile(mpk_handle *h) {
   P.x_tile_bytes = g.x_tile_bytes;
   P.max_inflight = g.num_stages;
   P.general_kernel = g.general_kernel ? 1 : 0;
+  P.hybrid = g.hybrid;
   P.tmaps = h->d_tmaps;
   P.use_tmem = g.use_tmem ? 1 : 0;
   P.tc_tokens = g.tc_tokens;
@@ -432,7 +478,9 @@ int mpk_compile(mpk_handle *h) {
   P.spin_limit = 4000;   // milliseconds a launch may wait before it gives up
   if (const char *e = getenv("MPK_SPIN_LIMIT_MS")) P.spin_limit = (uint32_t)std::max(1, std::min(atoi(e), 60000));
   if (!dry) {
-    int e = mpk_kernel_prepare(h->smem_bytes);
+    rc = load_family(g.hybrid != HYB_NONE, &h->kernels, &h->error);
+    if (rc) return rc;
+    int e = h->kernels.prepare(h->smem_bytes, 0);
     if (e) return set_err(h, MPK_ERR_CUDA, std::string("cudaFuncSetAttribute(smem=") + std::to_string(h->smem_bytes) +
                                                "): " + cudaGetErrorString((cudaError_t)e));
   }
@@ -503,7 +551,9 @@ int mpk_reset(mpk_handle *h, void *cuda_stream) {
     // init_kernel, include/mirage/persistent_kernel/persistent_kernel.cuh:149-166 (offline only: in online_notoken
     // the batch description belongs to the caller and is left alone)
     CU(cudaMemsetAsync(cfg.step, 0, (size_t)cfg.total_num_requests * 4, st));
-    CU(cudaMemsetAsync(h->d_request_ids, 0xff, (size_t)cfg.max_num_batched_requests * 4, st));
+    CU(cudaMemsetAsync(h->params.meta.request_ids, 0xff, (size_t)cfg.max_num_batched_requests * 4, st));
+    CU(cudaMemsetAsync(h->params.meta.state_slots, 0, (size_t)cfg.max_num_batched_requests * 4, st));
+    if (h->params.meta.request_ctl) CU(cudaMemsetAsync(h->params.meta.request_ctl, 0, (size_t)cfg.total_num_requests * 8, st));
     CU(cudaMemsetAsync(cfg.qo_indptr, 0, (size_t)(cfg.max_num_batched_requests + 1) * 4, st));
     CU(cudaMemsetAsync(cfg.paged_kv_indptr, 0, (size_t)(cfg.max_num_batched_requests + 1) * 4, st));
     std::vector<int32_t> ring(cfg.max_num_pages);
@@ -535,7 +585,7 @@ int mpk_launch(mpk_handle *h, void *cuda_stream, int num_steps) {
   }
   CU(cudaSetDevice(h->cfg.device));
   for (int i = 0; i < num_steps; ++i) {
-    int e = mpk_kernel_launch(&h->params, h->smem_bytes, cuda_stream);
+    int e = h->kernels.launch(&h->params, h->smem_bytes, cuda_stream);
     if (e) return set_err(h, MPK_ERR_CUDA, std::string("megakernel launch: ") + cudaGetErrorString((cudaError_t)e));
   }
   return MPK_OK;

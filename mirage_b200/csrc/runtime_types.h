@@ -18,6 +18,7 @@ constexpr int kChunkColsMax = 2048;            // k extent of a chunk, at most (
 constexpr int kRowPadBytes = 16;               // shared-memory row padding: conflict-free ldmatrix
 constexpr int stage_bytes_for(int chunk_cols) { return kChunkRows * (chunk_cols * 2 + kRowPadBytes); }
 constexpr int kPartialBytes = 8 * 1024;        // per-task partial-sum slots
+constexpr int kMiscBytes = 1536;               // barriers, descriptors, flags (1 KB) + the attention stash ring
 constexpr int kMaxLinearTokens = 64;           // eight mma n-tiles of 8 tokens, one per compute warp
 constexpr int kFp8TaskRows = 64;               // weight rows of one FP8 linear task (their scales are staged in shared memory)
 constexpr int kTcSlotBytes = 16 * 1024;        // weight ring slot of graphs whose linears run on tcgen05 (1 KB multiples: swizzle atoms)
@@ -53,6 +54,38 @@ enum TaskType : uint32_t {
   TASK_ARGMAX_EXCHANGE = 22,    // argmax merge over a vocabulary sharded across ranks (pairs exchanged through the inboxes)
   TASK_AR_PUSH = 23,            // copy a column slice of a local bf16 tensor into every rank's inbox as fp32 (allreduce whose
                                 // input is not produced by a bf16 linear); fields as TASK_ALLREDUCE with p[0] = the tensor
+  // ---- hybrid graphs (recurrent and extended-attention layers; hybrid_tasks.cuh) ----
+  TASK_EMBED_F32 = 24,          // token ids -> float32 rows of a bf16 table
+  TASK_RESIDUAL_NORM = 25,      // x += norm(y) on a float32 residual stream, and the next layer's normed input
+  TASK_LINEAR_F32 = 26,         // float32 activations x bf16 weights in 32-bit arithmetic
+  TASK_QKV_APPEND = 27,         // rotation and unit norms of q and k, new k / v rows into the paged cache
+  TASK_EXT_ATTENTION = 28,      // paged attention with free head sizes, score soft cap and sink
+  TASK_SHORT_CONV = 29,         // causal per-channel convolution with carried inputs
+  TASK_RGLRU = 30,              // gated diagonal linear recurrence
+  TASK_MLSTM = 31,              // matrix-memory recurrence with exponential gates
+};
+
+// Which family of megakernel instantiations runs a graph (template parameter HYB of the kernel).
+// Query rows a bf16 extended-attention task keeps in shared memory: whole 16-row tiles, a power of two of them (the
+// warps are split over the tiles), at most as many as the graph can batch.
+#ifdef __CUDACC__
+__host__ __device__
+#endif
+constexpr int ext_attention_rows(int rows) {
+  int r = 16;
+  while (r < rows) r *= 2;
+  return r;
+}
+
+enum : int { HYB_NONE = 0, HYB_BF16 = 1, HYB_F32 = 2 };
+
+// Online mode: control word of a token-table row (KernelParams.meta.request_ctl[row], written by the host between
+// launches; request_ctl[rows + row] is the device's "live" flag).
+enum : int {
+  REQ_FREE = 0,    // row unused (the device sets it when a request retires)
+  REQ_RUN = 1,     // runs its prompt, then decodes until EOS or the table's end
+  REQ_HOLD = 2,    // runs the tokens supplied so far (prompt_lengths[row]) and then keeps its pages and state
+  REQ_CLOSE = 3,   // retires once the supplied tokens have run
 };
 
 // prologue applied while staging the activation tile of a linear task
@@ -63,6 +96,8 @@ enum Epilogue : int32_t {
   EPI_RESIDUAL = 1,     // out = bf16(acc + residual)
   EPI_PUSH_F32 = 2,     // fp32 partial rows pushed into every rank's inbox slot [my_rank] (+ counter increments)
   EPI_PUSH_LL = 3,      // {bf16 partial, 16-bit sequence} words pushed into every rank's inbox: self-validating
+  EPI_STORE_F32 = 5,    // out = acc, float32 (hybrid graphs)
+  EPI_RELU2 = 6,        // out = bf16(max(acc, 0)^2) (hybrid graphs)
   EPI_SILU_PAIR = 4,    // rows interleaved [gate, gate, up, up]: out[2k + i] = bf16(silu(gate_i)) * up_i
 };
 
@@ -150,6 +185,33 @@ enum { M_NEXP = 19, M_NTOPK, M_PER_SLOT, M_LDR, M_ESTRIDE };
 // ---- TASK_ARGMAX_EXCHANGE:  as TASK_ARGMAX_REDUCE, plus a[2] first column of this rank, p[5] word offset of the
 //      exchange area inside an inbox buffer ([world][tokens] x {value | seq, index | seq} 64-bit words), a[L_ARIDX],
 //      a[L_NAR], a[L_PARSTRIDE] as for the allreduce
+// ---- hybrid tasks --------------------------------------------------------------
+// ---- TASK_EMBED_F32: p[0] ids  p[1] table bf16  p[2] out f32;  a[E_*] as TASK_EMBED (a[E_AUX] = vocabulary)
+// ---- TASK_RESIDUAL_NORM: rows [a[0], a[1]), width a[2]; p[0] x f32 (in place)  p[1] y f32 or null  p[2] weight of y's norm or
+//      null (plain sum)  p[3] weight of the output norm or null  p[4] out (bf16, f32 with flag 1) or null;
+//      a[3] ld x  a[4] ld y  a[5] ld out  a[6] eps bits  a[7] flags (1: out f32, 2: weights stored around zero)
+// ---- TASK_LINEAR_F32: p[0] W bf16 [N, K]  p[1] x f32  p[2] out f32;  a[0] n0  a[1] n1  a[2] K  a[3] ldw  a[4] ld x  a[5] ld out
+//      a[6] activation (0 none, 1 squared relu)  a[7] tokens per shared-memory tile
+// ---- TASK_QKV_APPEND: tokens [a[0], a[1]); p[0] projections f32  p[1] q out  p[2] k cache  p[3] v cache  p[4] cos f32  p[5] sin f32
+//      p[6] v source (null: the k columns before rotation and norm)
+//      a[QA_*] below
+enum { QA_T0 = 0, QA_T1, QA_LDP, QA_QOFF, QA_KOFF, QA_VOFF, QA_HQ, QA_HKV, QA_DIM, QA_DIMP, QA_VDIM, QA_VDIMP, QA_ROT, QA_NORM,
+       QA_EPS, QA_PAGE, QA_LDQ, QA_ROWS };
+// ---- TASK_EXT_ATTENTION: p[0] q [tokens, hq * dimp]  p[1] k cache  p[2] v cache  p[3] out;  a[XA_*] below
+enum { XA_SLOT = 0, XA_HEAD, XA_CHUNK, XA_NCHUNK, XA_HQ, XA_HKV, XA_DIMP, XA_VDIM, XA_VDIMP, XA_PAGE, XA_LDQ, XA_LDO, XA_OCOL,
+       XA_SCALE, XA_CAP, XA_SINK, XA_OSCALE, XA_TICKET, XA_SREC, XA_WINDOW };
+// ---- TASK_SHORT_CONV: channels [a[0], a[1]); p[0] in f32  p[1] in bias bf16 or null  p[2] taps bf16 [channels, taps]
+//      p[3] bias bf16 or null  p[4] carried inputs f32 [slots, taps - 1, channels]  p[5] out f32
+//      a[2] channels  a[3] taps  a[4] ld in  a[5] in column offset  a[6] ld out  a[7] activation (0 none, 1 silu)
+// ---- TASK_RGLRU: p[0] u f32 [tokens, width]  p[1] projections f32 (output branch)  p[2] y bias bf16  p[3] ra  p[4] ra bias  p[5] ri
+//      p[6] ri bias  p[7] lambda (bf16, all);  a[GL_*]; state and output pointers are 64-bit values in a[GL_STATE], a[GL_OUT]
+enum { GL_BLOCK = 0, GL_C0, GL_C1, GL_BS, GL_WIDTH, GL_LDU, GL_LDP, GL_YOFF, GL_LDO, GL_OCOL, GL_OSCALE, GL_OUTF32, GL_GATE_C, GL_TG,
+       GL_STATE = 20, GL_OUT = 22 };
+// ---- TASK_MLSTM: p[0] projections f32  p[1] input-gate bias  p[2] forget-gate bias  p[3] output norm weight (bf16)
+//      p[4] matrix state f32 [slots, heads, dim, vdimp]  p[5] normaliser state f32 [slots, heads, chunks, dim + 1] (n, then m)
+//      p[6] readout scratch f32 [tokens, heads * vdim]  p[7] out;  a[ML_*]
+enum { ML_SLOT = 0, ML_HEAD, ML_CHUNK, ML_NCHUNK, ML_H, ML_DIM, ML_VDIM, ML_VDIMP, ML_V0, ML_V1, ML_CAP, ML_EPS, ML_LDP, ML_QOFF,
+       ML_KOFF, ML_VOFF, ML_GOFF, ML_IOFF, ML_FOFF, ML_LDO, ML_OUTF32, ML_QSCALE, ML_TICKET, ML_TC, ML_LDR };
 // ---- TASK_ALLREDUCE:       p[0] inbox base p[1] residual (or null) p[2] out
 //  a[0] c0 a[1] c1 (columns) a[2] world a[3] slot stride (floats) a[4] ld_out a[5] ld_res a[6] N
 //  a[7] allreduce index  a[8] allreduces per iteration  a[9] stride between the two inbox buffers (floats)
@@ -168,6 +230,8 @@ struct BatchMeta {
   int32_t *request_ids;      // [max_num_batched_requests]
   int32_t *page_queue;       // [max_num_pages]
   int32_t *sched_scalars;    // [0] page_queue_head [1] page_queue_tail [2] next_request_id
+  int32_t *state_slots;      // [max_num_batched_requests] recurrent-state slot of each batch slot
+  int32_t *request_ctl;      // [2][total_num_requests] online mode only, else null
 };
 
 struct DeviceStatus {
@@ -215,6 +279,7 @@ struct KernelParams {
   int32_t ll_buffer_words;              // words between the two inbox buffers
   int32_t tp_extensions;                // batch-1 graphs of several ranks: run the instantiation with the argmax exchange and the
                                         // all-ranks-in-flight allreduce prologue (set when the graph holds an exchange task)
+  int32_t hybrid;                       // host side: HYB_* family of the graph
   int32_t general_kernel;               // host side: launch the instantiation with FP8 and > 8-token linear tasks
   int32_t x_tile_bytes;                 // bytes reserved for the activation tile
   uint32_t spin_limit;                  // polls before a wait gives up

@@ -11,7 +11,6 @@ namespace mpk {
 namespace {
 
 constexpr int kSmemBudget = 232448;   // 227 KB opt-in dynamic shared memory per CTA on sm_100
-constexpr int kMiscBytesHost = 1536;   // barriers, descriptors, flags (1 KB) + the attention stash ring
 constexpr int ST_META = 0;            // batch description written by the batching task
 constexpr int ST_META_OUT = 1;        // output_tokens (written by argmax, read by the batching task)
 
@@ -44,6 +43,8 @@ struct Builder {
   std::vector<std::vector<TaskDesc>> per_worker;
   std::vector<std::vector<int>> per_worker_exec;
   int rot = 0;
+  int hybrid_tickets = 0;   // arrival tickets handed to the tasks of hybrid graphs
+  std::map<int, std::map<int, int>> slices;   // storage -> (first column -> id) of outputs that layers write by column range
 
   Builder(GraphInputs i, CompiledGraph *out, std::string *e)
       : in(i), g(out), err(e), cfg(*i.cfg), T(*i.tensors), L(*i.layers), W(i.num_workers) {
@@ -57,6 +58,7 @@ struct Builder {
   // expert / latent-attention / sampling layer)?
   bool general_graph() const {
     if (nb_max > 8 || cfg.max_num_batched_tokens > 8) return true;
+    if (g->hybrid) return false;
     for (const auto &l : L)
       if (l.op >= MPK_OP_QUANTIZE_FP8) return true;
     return false;
@@ -78,7 +80,7 @@ struct Builder {
   // (these tasks keep no partial sums there), and the buffer may grow until five 16 KB ring slots remain (what the
   // 129 KB bf16 tile leaves as well): at 64 tokens that admits k tiles of 2048 instead of 1024, i.e. half as many
   // stage / drain pauses per task.
-  static int64_t fp8_tc_tile_cap() { return (kSmemBudget - kMiscBytesHost - kPartialBytes - 5 * kTcSlotBytes) / 256 * 256; }
+  static int64_t fp8_tc_tile_cap() { return (kSmemBudget - kMiscBytes - kPartialBytes - 5 * kTcSlotBytes) / 256 * 256; }
   int64_t linear_tile_bytes(int64_t K) const {
     return tc_linear(K) ? (int64_t)tc_np() * K * 2 : (int64_t)nb_max * (K * 2 + kRowPadBytes);
   }
@@ -160,6 +162,16 @@ struct Builder {
       case MPK_OP_MLA_KV_GATHER: add(ins, l.t[0]); add(ins, l.t[1]); add(ins, l.t[2]); add(outs, l.t[2]); break;
       case MPK_OP_MLA_DECODE: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); add(outs, l.t[3]); break;
       case MPK_OP_MLA_REDUCE: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); break;
+      case MPK_OP_RESIDUAL_NORM:
+        for (int i = 0; i < 4; ++i) add(ins, l.t[i]);
+        if (l.t[1] >= 0) add(outs, l.t[0]);
+        add(outs, l.t[4]);
+        break;
+      case MPK_OP_QKV_APPEND: add(ins, l.t[0]); add(ins, l.t[4]); add(ins, l.t[5]); for (int i = 1; i < 4; ++i) add(outs, l.t[i]); break;
+      case MPK_OP_EXT_ATTENTION: for (int i = 0; i < 3; ++i) add(ins, l.t[i]); add(outs, l.t[3]); break;
+      case MPK_OP_SHORT_CONV: for (int i = 0; i < 5; ++i) add(ins, l.t[i]); add(outs, l.t[4]); add(outs, l.t[5]); break;
+      case MPK_OP_RGLRU: for (int i = 0; i < 9; ++i) add(ins, l.t[i]); add(outs, l.t[8]); add(outs, l.t[9]); break;
+      case MPK_OP_MLSTM: for (int i = 0; i < 6; ++i) add(ins, l.t[i]); for (int i = 4; i < 8; ++i) add(outs, l.t[i]); break;
       case MPK_OP_LINEAR_FP8_RESIDUAL: for (int i = 0; i < 5; ++i) add(ins, l.t[i]); add(outs, l.t[5]); break;
       default: break;
     }
@@ -191,7 +203,8 @@ struct Builder {
           {MPK_OP_MOE_W2_FP8, 7}, {MPK_OP_MOE_SILU_MUL, 2}, {MPK_OP_MOE_MUL_SUM_ADD, 4},
           {MPK_OP_MLA_KV_GATHER, 3}, {MPK_OP_MLA_DECODE, 4}, {MPK_OP_MLA_REDUCE, 3},
           {MPK_OP_SAMPLING_PARTIAL, 3}, {MPK_OP_SAMPLING_REDUCE, 3}, {MPK_OP_ARGMAX_EXCHANGE, 3},
-          {MPK_OP_MOE_TOPK_SOFTMAX, 4}};
+          {MPK_OP_MOE_TOPK_SOFTMAX, 4}, {MPK_OP_RESIDUAL_NORM, 5}, {MPK_OP_QKV_APPEND, 6}, {MPK_OP_EXT_ATTENTION, 4},
+          {MPK_OP_SHORT_CONV, 6}, {MPK_OP_RGLRU, 10}, {MPK_OP_MLSTM, 8}};
       auto it = need.find(L[i].op);
       if (it == need.end()) return fail(MPK_ERR_UNSUPPORTED, "layer " + std::to_string(i) + ": unknown op");
       if ((int)L[i].t.size() < it->second)
@@ -370,7 +383,12 @@ struct Builder {
     int64_t need = 24 * 1024;
     for (const auto &l : L) {
       if (l.folded) continue;
-      if (l.op == MPK_OP_LINEAR || l.op == MPK_OP_LINEAR_RESIDUAL || l.op == MPK_OP_SPLITK_LINEAR) {
+      if (hybrid_op(l.op)) {
+        need = std::max<int64_t>(need, hybrid_smem(l) - kPartialBytes);
+      } else if (g->hybrid == HYB_F32 && l.op == MPK_OP_LINEAR) {
+        const int64_t K = T[l.t[1]].dim(1);
+        need = std::max<int64_t>(need, (int64_t)linear_f32_tokens(K) * K * 4 - kPartialBytes);
+      } else if (l.op == MPK_OP_LINEAR || l.op == MPK_OP_LINEAR_RESIDUAL || l.op == MPK_OP_SPLITK_LINEAR) {
         const int64_t K = T[l.t[1]].dim(1);
         need = std::max(need, std::min<int64_t>(linear_tile_bytes(K), x_tile_cap()));
         if (tc_linear(K) && T[l.t[1]].dtype == MPK_BF16) g->use_tmem = true;
@@ -405,10 +423,10 @@ struct Builder {
         need = std::max(need, attn - kPartialBytes);
       }
     }
-    if (!no_batch_task()) need = std::max<int64_t>(need, (int64_t)(13 * cfg.max_num_batched_requests + 16) * 4 - kPartialBytes);
+    if (!no_batch_task()) need = std::max<int64_t>(need, (int64_t)(16 * cfg.max_num_batched_requests + 20 + (cfg.mode == MPK_MODE_ONLINE ? cfg.total_num_requests : 0)) * 4 - kPartialBytes);
     need = (need + 255) / 256 * 256;
     // 64 KB stages (4 KB row segments) when at least three of them fit, else 32 KB stages
-    const int64_t room = kSmemBudget - kMiscBytesHost - kPartialBytes - need;
+    const int64_t room = kSmemBudget - kMiscBytes - kPartialBytes - need;
     g->x_tile_bytes = (int)need;
     g->tc_tokens = tc_np();
     if (g->use_tmem) {
@@ -488,7 +506,9 @@ struct Builder {
     } else if (x.dim(x.dims.size() - 1) != K) {
       return fail(MPK_ERR_INVALID, "linear input width != K for " + w.name);
     }
-    if (y.dim(y.dims.size() - 1) != N) return fail(MPK_ERR_INVALID, "linear output width != N for " + w.name);
+    // (hybrid graphs: the output buffer may be padded to the k granularity of the next linear)
+    if (g->hybrid ? y.dim(y.dims.size() - 1) < N : y.dim(y.dims.size() - 1) != N)
+      return fail(MPK_ERR_INVALID, "linear output width != N for " + w.name);
     int epi = EPI_STORE;
     uint64_t res_ptr = 0;
     int ldr = 0;
@@ -502,6 +522,17 @@ struct Builder {
       epi = EPI_RESIDUAL; res_ptr = (uint64_t)y.ptr; ldr = (int)y.ld();
     }
     if (l.push) epi = l.push_ll ? EPI_PUSH_LL : EPI_PUSH_F32;
+    if (x.dtype != MPK_BF16) return fail(MPK_ERR_UNSUPPORTED, "linear input must be bf16: " + w.name);
+    if (l.op == MPK_OP_LINEAR && !l.params.empty() && l.params[0] != 0) {
+      if (g->hybrid != HYB_BF16 || l.params[0] != 1 || y.dtype != MPK_BF16)
+        return fail(MPK_ERR_UNSUPPORTED, "linear activation: squared relu into bf16, in hybrid graphs: " + w.name);
+      epi = EPI_RELU2;
+    } else if (y.dtype == MPK_F32) {
+      if (g->hybrid != HYB_BF16 || epi != EPI_STORE) return fail(MPK_ERR_UNSUPPORTED, "float32 linear output needs a hybrid graph: " + w.name);
+      epi = EPI_STORE_F32;
+    } else if (y.dtype != MPK_BF16) {
+      return fail(MPK_ERR_UNSUPPORTED, "linear output must be bf16 or float32: " + w.name);
+    }
     uint64_t out_ptr = (uint64_t)y.ptr;
     int ldo = (int)y.ld();
     const int unit = l.silu_out >= 0 ? 4 : 1;      // paired rows stay in one task
@@ -929,6 +960,277 @@ struct Builder {
     return MPK_OK;
   }
 
+  // ---- hybrid graphs: recurrent layers, extended attention, float32 residual stream --------------------------
+  static bool hybrid_op(int op) { return op >= MPK_OP_RESIDUAL_NORM && op <= MPK_OP_MLSTM; }
+  static int round_up(int64_t v, int m) { return (int)((v + m - 1) / m * m); }
+  static int bits_of(int64_t p) { return (int)(uint32_t)p; }
+
+  int classify_hybrid() {
+    bool any = false, f32 = false;
+    for (const auto &l : L) any = any || hybrid_op(l.op);
+    if (!any) return MPK_OK;
+    if (cfg.world_size > 1) return fail(MPK_ERR_UNSUPPORTED, "hybrid graphs run on one rank");
+    if (cfg.max_num_batched_tokens > kMaxLinearTokens)
+      return fail(MPK_ERR_UNSUPPORTED, "hybrid graphs batch at most 64 tokens");
+    for (size_t i = 0; i < L.size(); ++i) {
+      const LayerInfo &l = L[i];
+      if (hybrid_op(l.op) || l.op == MPK_OP_EMBED || l.op == MPK_OP_ARGMAX_PARTIAL || l.op == MPK_OP_ARGMAX_REDUCE ||
+          l.op == MPK_OP_SAMPLING_PARTIAL || l.op == MPK_OP_SAMPLING_REDUCE) continue;
+      if (l.op != MPK_OP_LINEAR) return fail(MPK_ERR_UNSUPPORTED, "layer " + std::to_string(i) + ": not available in a hybrid graph");
+      if (T[l.t[0]].dtype == MPK_F32) f32 = true;
+    }
+    g->hybrid = f32 ? HYB_F32 : HYB_BF16;
+    return MPK_OK;
+  }
+  int act_dtype() const { return g->hybrid == HYB_F32 ? MPK_F32 : MPK_BF16; }
+  bool batch_meta_given() const {
+    return cfg.dry_run || (cfg.qo_indptr && cfg.paged_kv_indptr && cfg.paged_kv_indices && cfg.paged_kv_last_page_len);
+  }
+  int linear_f32_tokens(int64_t K) const { return (int)std::max<int64_t>(1, std::min<int64_t>(nb_max, 98304 / (4 * std::max<int64_t>(K, 1)))); }
+  int xattn_width(const LayerInfo &l) const {   // padded head size of the tensor-core body
+    const int w = (int)std::max(T[l.t[1]].dim(3), T[l.t[2]].dim(3));
+    return w <= 64 ? 64 : (w <= 128 ? 128 : 256);
+  }
+  void rglru_plan(const LayerInfo &l, int *C, int *TG) const {
+    const int nb = (int)T[l.t[3]].dim(0), bs = (int)T[l.t[3]].dim(1);
+    const int chunks = std::max(1, W / std::max(nb, 1));
+    *C = std::min(std::min(bs, 64), std::max(8, round_up((bs + chunks - 1) / chunks, 2)));
+    int tg = std::min(nb_max, (int)std::max<int64_t>(8, (int64_t)65536 / (4 * (bs + 2 * *C))));
+    *TG = std::max(1, tg > 8 ? tg / 8 * 8 : tg);
+  }
+  static int mlstm_tokens(int64_t dim) { return dim <= 512 ? 16 : 8; }
+  int64_t hybrid_smem(const LayerInfo &l) const {
+    const int64_t mbr = cfg.max_num_batched_requests;
+    switch (l.op) {
+      case MPK_OP_RESIDUAL_NORM: return T[l.t[0]].dim(1) * 4 + 16;
+      case MPK_OP_EXT_ATTENTION: {
+        if (g->hybrid == HYB_F32) return 8 * T[l.t[1]].dim(3) * 4;
+        const int D = xattn_width(l), pitch = D * 2 + 16, keys = D > 128 ? 32 : 64, wmax = D > 128 ? 4 : 8;
+        const int G = (int)(l.params[0] / std::max<int64_t>(l.params[1], 1));
+        return (int64_t)std::min(wmax * 16, ext_attention_rows(cfg.max_num_batched_tokens * G)) * pitch + 4 * keys * pitch;
+      }
+      case MPK_OP_SHORT_CONV: return kMaxLinearTokens * 16 + (mbr + 1) * 4;
+      case MPK_OP_RGLRU: {
+        int C, TG;
+        rglru_plan(l, &C, &TG);
+        return kMaxLinearTokens * 16 + std::max<int64_t>((int64_t)TG * (T[l.t[3]].dim(1) + 2 * C) * 4, (mbr + 1) * 4);
+      }
+      case MPK_OP_MLSTM: {
+        const int64_t dim = l.params[1], vc = MPK_MLSTM_COLUMNS(dim), TC = mlstm_tokens(dim);
+        return 4 * (3 * kMaxLinearTokens + TC * 8 + TC * (2 * dim + vc) + TC * 8 * vc);
+      }
+      default: return 0;
+    }
+  }
+
+  int emit_linear_f32(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &x = T[l.t[0]], &w = T[l.t[1]], &y = T[l.t[2]];
+    if (w.dims.size() != 2 || w.dtype != MPK_BF16 || w.strides[1] != 1 || x.dtype != MPK_F32 || y.dtype != MPK_F32)
+      return fail(MPK_ERR_UNSUPPORTED, "32-bit linear: float32 input and output, row-major bf16 weight: " + w.name);
+    const int N = (int)w.dim(0), K = (int)w.dim(1);
+    if (x.dim(1) != K || y.dim(1) != N) return fail(MPK_ERR_INVALID, "32-bit linear: shapes disagree for " + w.name);
+    const int nt = std::min(W, N);
+    for (int i = 0; i < nt; ++i) {
+      TaskDesc d = blank(TASK_LINEAR_F32, li);
+      d.p[0] = (uint64_t)w.ptr; d.p[1] = (uint64_t)x.ptr; d.p[2] = (uint64_t)y.ptr;
+      d.a[0] = (int)((int64_t)N * i / nt); d.a[1] = (int)((int64_t)N * (i + 1) / nt);
+      d.a[2] = K; d.a[3] = (int)w.ld(); d.a[4] = (int)x.ld(); d.a[5] = (int)y.ld();
+      d.a[6] = l.params.empty() ? 0 : (int)l.params[0];
+      d.a[7] = linear_f32_tokens(K);
+      put((i + rot) % W, d, ex);
+    }
+    g->weight_bytes += (int64_t)N * K * 2;
+    return MPK_OK;
+  }
+
+  int emit_residual_norm(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &x = T[l.t[0]];
+    auto opt = [&](int i) { return l.t[i] >= 0 ? (uint64_t)T[l.t[i]].ptr : 0; };
+    const int D = (int)x.dim(1);
+    if (l.params.size() < 2 || x.dtype != MPK_F32 || x.dims.size() != 2) return fail(MPK_ERR_INVALID, "residual_norm: x must be float32 [tokens, width]");
+    if (l.t[1] >= 0 && (T[l.t[1]].dtype != MPK_F32 || T[l.t[1]].dim(1) != D)) return fail(MPK_ERR_INVALID, "residual_norm: y must be float32 of x's width");
+    for (int i = 2; i < 4; ++i)
+      if (l.t[i] >= 0 && (T[l.t[i]].dtype != MPK_BF16 || T[l.t[i]].dim(0) != D)) return fail(MPK_ERR_INVALID, "residual_norm: weights must be bf16 [width]");
+    if ((l.t[3] >= 0) != (l.t[4] >= 0)) return fail(MPK_ERR_INVALID, "residual_norm: output and its norm weight go together");
+    if (l.t[4] >= 0 && (T[l.t[4]].dtype != act_dtype() || T[l.t[4]].dim(1) < D)) return fail(MPK_ERR_INVALID, "residual_norm: output type or width");
+    const int rows = (int)std::min<int64_t>(x.dim(0), cfg.max_num_batched_tokens), nt = std::min(rows, W);
+    for (int i = 0; i < nt; ++i) {
+      TaskDesc d = blank(TASK_RESIDUAL_NORM, li);
+      d.p[0] = (uint64_t)x.ptr; d.p[1] = opt(1); d.p[2] = opt(2); d.p[3] = opt(3); d.p[4] = opt(4);
+      d.a[0] = (int)((int64_t)rows * i / nt); d.a[1] = (int)((int64_t)rows * (i + 1) / nt); d.a[2] = D;
+      d.a[3] = (int)x.ld(); d.a[4] = l.t[1] >= 0 ? (int)T[l.t[1]].ld() : 0; d.a[5] = l.t[4] >= 0 ? (int)T[l.t[4]].ld() : 0;
+      d.a[6] = bits_of(l.params[0]);
+      d.a[7] = (g->hybrid == HYB_F32 ? 1 : 0) | (l.params[1] ? 2 : 0);
+      put((i + rot) % W, d, ex);
+    }
+    return MPK_OK;
+  }
+
+  int emit_qkv_append(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &pr = T[l.t[0]], &q = T[l.t[1]], &kc = T[l.t[2]], &vc = T[l.t[3]], &cs = T[l.t[4]], &sn = T[l.t[5]];
+    if (l.params.size() < 10) return fail(MPK_ERR_INVALID, "qkv_append needs 10 parameters");
+    const int hq = (int)l.params[0], hkv = (int)l.params[1], dim = (int)l.params[2], vdim = (int)l.params[3], rdim = (int)l.params[7];
+    if (!batch_meta_given()) return fail(MPK_ERR_INVALID, "qkv_append needs the batch meta tensors");
+    if (pr.dtype != MPK_F32 || q.dtype != act_dtype() || kc.dtype != act_dtype() || vc.dtype != act_dtype() || cs.dtype != MPK_F32 || sn.dtype != MPK_F32)
+      return fail(MPK_ERR_INVALID, "qkv_append: float32 projections and tables, q and caches of the graph's activation type");
+    if (hq < 1 || hkv < 1 || hq % hkv || dim < 1 || vdim < 1 || rdim < 0 || rdim > dim || rdim % 2)
+      return fail(MPK_ERR_INVALID, "qkv_append: head counts or sizes");
+    if (kc.dims.size() != 4 || vc.dims.size() != 4 || kc.dim(1) != cfg.page_size || vc.dim(1) != cfg.page_size || kc.dim(2) != hkv ||
+        vc.dim(2) != hkv || kc.dim(3) < dim || vc.dim(3) < vdim || kc.dim(3) % 8 || vc.dim(3) % 8 || q.dim(1) != hq * kc.dim(3))
+      return fail(MPK_ERR_INVALID, "qkv_append: caches [pages, page, kv_heads, head size rounded up to 8], q [tokens, heads x that]");
+    if (l.params[4] + (int64_t)hq * dim > pr.dim(1) || l.params[5] + (int64_t)hkv * dim > pr.dim(1) || l.params[6] + (int64_t)hkv * vdim > pr.dim(1))
+      return fail(MPK_ERR_INVALID, "qkv_append: columns outside the projections");
+    if (rdim > 0 && (cs.dims.size() != 2 || cs.dim(1) != rdim / 2 || sn.dim(1) != rdim / 2 || cs.dim(0) != sn.dim(0)))
+      return fail(MPK_ERR_INVALID, "qkv_append: cos / sin tables [positions, rotated dims / 2]");
+    const int nt = std::max(1, std::min(W, (nb_max * (hq + hkv) + 7) / 8));
+    for (int i = 0; i < nt; ++i) {
+      TaskDesc d = blank(TASK_QKV_APPEND, li);
+      d.p[0] = (uint64_t)pr.ptr; d.p[1] = (uint64_t)q.ptr; d.p[2] = (uint64_t)kc.ptr; d.p[3] = (uint64_t)vc.ptr;
+      d.p[4] = (uint64_t)cs.ptr; d.p[5] = (uint64_t)sn.ptr;
+      d.a[QA_T0] = i; d.a[QA_T1] = nt; d.a[QA_LDP] = (int)pr.ld();
+      d.a[QA_QOFF] = (int)l.params[4]; d.a[QA_KOFF] = (int)l.params[5]; d.a[QA_VOFF] = (int)l.params[6];
+      d.a[QA_HQ] = hq; d.a[QA_HKV] = hkv; d.a[QA_DIM] = dim; d.a[QA_DIMP] = (int)kc.dim(3); d.a[QA_VDIM] = vdim; d.a[QA_VDIMP] = (int)vc.dim(3);
+      d.a[QA_ROT] = rdim; d.a[QA_NORM] = (int)l.params[8]; d.a[QA_EPS] = bits_of(l.params[9]); d.a[QA_PAGE] = cfg.page_size;
+      d.a[QA_LDQ] = (int)q.ld(); d.a[QA_ROWS] = rdim > 0 ? (int)cs.dim(0) : 1;
+      put((i + rot) % W, d, ex);
+    }
+    return MPK_OK;
+  }
+
+  int emit_ext_attention(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &q = T[l.t[0]], &kc = T[l.t[1]], &vc = T[l.t[2]], &o = T[l.t[3]];
+    if (l.params.size() < 8) return fail(MPK_ERR_INVALID, "ext_attention needs 8 parameters");
+    const int hq = (int)l.params[0], hkv = (int)l.params[1], vdim = (int)l.params[2], ocol = (int)l.params[3];
+    if (!batch_meta_given()) return fail(MPK_ERR_INVALID, "ext_attention needs the batch meta tensors");
+    if (hq < 1 || hkv < 1 || hq % hkv || kc.dims.size() != 4 || vc.dims.size() != 4 || kc.dim(2) != hkv || vc.dim(2) != hkv ||
+        kc.dim(1) != cfg.page_size || vc.dim(1) != cfg.page_size || kc.dim(3) % 8 || vc.dim(3) % 8 || vc.dim(3) < vdim ||
+        q.dim(1) != hq * kc.dim(3) || ocol < 0 || ocol + (int64_t)hq * vdim > o.dim(1))
+      return fail(MPK_ERR_INVALID, "ext_attention: shapes of q, caches and output disagree");
+    if (q.dtype != act_dtype() || kc.dtype != act_dtype() || vc.dtype != act_dtype() || o.dtype != act_dtype())
+      return fail(MPK_ERR_INVALID, "ext_attention: q, caches and output must have the graph's activation type");
+    if (std::max(kc.dim(3), vc.dim(3)) > (g->hybrid == HYB_F32 ? 512 : 256))
+      return fail(MPK_ERR_UNSUPPORTED, "ext_attention: head sizes up to 256 (512 in 32-bit graphs)");
+    const int slots = cfg.max_num_batched_requests, max_seq = std::max(cfg.max_seq_length, 1);
+    // chunks of a (request, kv head): enough to occupy the workers, at most ~2048 keys each, at least 128
+    int NC = std::max(std::max(1, W / std::max(slots * hkv, 1)), (max_seq + 2047) / 2048);
+    NC = std::min(std::min(NC, std::max(1, max_seq / 128)), 32);
+    const int srec = vdim + 2;
+    for (int s = 0; s < slots; ++s)
+      for (int h = 0; h < hkv; ++h)
+        for (int ch = 0; ch < NC; ++ch) {
+          TaskDesc d = blank(TASK_EXT_ATTENTION, li);
+          for (int i = 0; i < 4; ++i) d.p[i] = (uint64_t)T[l.t[i]].ptr;
+          d.a[XA_SLOT] = s; d.a[XA_HEAD] = h; d.a[XA_CHUNK] = ch; d.a[XA_NCHUNK] = NC; d.a[XA_HQ] = hq; d.a[XA_HKV] = hkv;
+          d.a[XA_DIMP] = (int)kc.dim(3); d.a[XA_VDIM] = vdim; d.a[XA_VDIMP] = (int)vc.dim(3); d.a[XA_PAGE] = cfg.page_size;
+          d.a[XA_LDQ] = (int)q.ld(); d.a[XA_LDO] = (int)o.ld(); d.a[XA_OCOL] = ocol;
+          d.a[XA_SCALE] = bits_of(l.params[4]); d.a[XA_CAP] = bits_of(l.params[5]); d.a[XA_SINK] = (int)l.params[6];
+          d.a[XA_OSCALE] = bits_of(l.params[7]);
+          d.a[XA_TICKET] = hybrid_tickets + s * hkv + h; d.a[XA_SREC] = srec;
+          put(((s * hkv + h) * NC + ch + rot) % W, d, ex);
+        }
+    hybrid_tickets += slots * hkv;
+    g->attn_scratch_floats = std::max<int64_t>(g->attn_scratch_floats, (int64_t)cfg.max_num_batched_tokens * hq * NC * srec);
+    return MPK_OK;
+  }
+
+  int emit_short_conv(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &x = T[l.t[0]], &w = T[l.t[2]], &st = T[l.t[4]], &o = T[l.t[5]];
+    if (l.params.size() < 2 || w.dims.size() != 2) return fail(MPK_ERR_INVALID, "short_conv: taps [channels, taps], params [in_col, activation]");
+    const int C = (int)w.dim(0), taps = (int)w.dim(1);
+    if (!batch_meta_given()) return fail(MPK_ERR_INVALID, "short_conv needs the batch meta tensors");
+    if (x.dtype != MPK_F32 || st.dtype != MPK_F32 || o.dtype != MPK_F32 || w.dtype != MPK_BF16 || l.params[0] + C > x.dim(1) || o.dim(1) != C ||
+        (int64_t)(st.bytes / 4) < (taps > 1 ? (int64_t)cfg.max_num_batched_requests * (taps - 1) * C : 0))
+      return fail(MPK_ERR_INVALID, "short_conv: float32 input, output and state [slots, taps - 1, channels], bf16 taps");
+    for (int i : {1, 3})
+      if (l.t[i] >= 0 && (T[l.t[i]].dtype != MPK_BF16 || T[l.t[i]].dim(0) != C)) return fail(MPK_ERR_INVALID, "short_conv: bf16 biases [channels]");
+    const int nt = std::max(1, std::min(W, C / 32));
+    for (int i = 0; i < nt; ++i) {
+      TaskDesc d = blank(TASK_SHORT_CONV, li);
+      for (int k = 0; k < 6; ++k) d.p[k] = l.t[k] >= 0 ? (uint64_t)T[l.t[k]].ptr : 0;
+      d.a[0] = (int)((int64_t)C * i / nt); d.a[1] = (int)((int64_t)C * (i + 1) / nt); d.a[2] = C; d.a[3] = taps;
+      d.a[4] = (int)x.ld(); d.a[5] = (int)l.params[0]; d.a[6] = (int)o.ld(); d.a[7] = (int)l.params[1];
+      put((i + rot) % W, d, ex);
+    }
+    return MPK_OK;
+  }
+
+  int emit_rglru(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &u = T[l.t[0]], &pr = T[l.t[1]], &ra = T[l.t[3]], &st = T[l.t[8]], &o = T[l.t[9]];
+    if (l.params.size() < 4 || ra.dims.size() != 3 || ra.dim(1) != ra.dim(2)) return fail(MPK_ERR_INVALID, "rglru: gates [blocks, size, size], 4 parameters");
+    const int nb = (int)ra.dim(0), bs = (int)ra.dim(1);
+    const int64_t width = (int64_t)nb * bs;
+    if (!batch_meta_given()) return fail(MPK_ERR_INVALID, "rglru needs the batch meta tensors");
+    if (u.dtype != MPK_F32 || pr.dtype != MPK_F32 || st.dtype != MPK_F32 || o.dtype != act_dtype() || u.dim(1) != width ||
+        l.params[0] + width > pr.dim(1) || l.params[1] + width > o.dim(1) || (int64_t)(st.bytes / 4) < (int64_t)cfg.max_num_batched_requests * width)
+      return fail(MPK_ERR_INVALID, "rglru: shapes or types of u, projections, state [slots, width] and output");
+    for (int i = 2; i < 8; ++i)
+      if (T[l.t[i]].dtype != MPK_BF16 || (int64_t)(T[l.t[i]].bytes / 2) < (i == 3 || i == 5 ? width * bs : width) || ((uint64_t)T[l.t[i]].ptr & 3))
+        return fail(MPK_ERR_INVALID, "rglru: bf16 gate weights and biases, 4-byte aligned");
+    int C, TG;
+    rglru_plan(l, &C, &TG);
+    int i = 0;
+    for (int b = 0; b < nb; ++b)
+      for (int c0 = 0; c0 < bs; c0 += C, ++i) {
+        TaskDesc d = blank(TASK_RGLRU, li);
+        for (int k = 0; k < 8; ++k) d.p[k] = (uint64_t)T[l.t[k]].ptr;
+        const uint64_t sp = (uint64_t)st.ptr, op = (uint64_t)o.ptr;
+        std::memcpy(&d.a[GL_STATE], &sp, 8);
+        std::memcpy(&d.a[GL_OUT], &op, 8);
+        d.a[GL_BLOCK] = b; d.a[GL_C0] = c0; d.a[GL_C1] = std::min(c0 + C, bs); d.a[GL_BS] = bs; d.a[GL_WIDTH] = (int)width;
+        d.a[GL_LDU] = (int)u.ld(); d.a[GL_LDP] = (int)pr.ld(); d.a[GL_YOFF] = (int)l.params[0]; d.a[GL_LDO] = (int)o.ld();
+        d.a[GL_OCOL] = (int)l.params[1]; d.a[GL_OSCALE] = bits_of(l.params[2]); d.a[GL_GATE_C] = bits_of(l.params[3]); d.a[GL_TG] = TG;
+        put((i + rot) % W, d, ex);
+      }
+    g->weight_bytes += 4 * width * bs;
+    return MPK_OK;
+  }
+
+  int emit_mlstm(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &pr = T[l.t[0]], &S = T[l.t[4]], &nm = T[l.t[5]], &raw = T[l.t[6]], &o = T[l.t[7]];
+    if (l.params.size() < 13) return fail(MPK_ERR_INVALID, "mlstm needs 13 parameters");
+    const int H = (int)l.params[0], dim = (int)l.params[1], vdim = (int)l.params[2], chunks = (int)l.params[12];
+    const int slots = cfg.max_num_batched_requests;
+    if (!batch_meta_given()) return fail(MPK_ERR_INVALID, "mlstm needs the batch meta tensors");
+    if (H < 1 || dim < 1 || vdim < 1) return fail(MPK_ERR_INVALID, "mlstm: head count or sizes");
+    if (dim > 1024) return fail(MPK_ERR_UNSUPPORTED, "mlstm: key sizes up to 1024");
+    if (pr.dtype != MPK_F32 || S.dtype != MPK_F32 || nm.dtype != MPK_F32 || raw.dtype != MPK_F32 || o.dtype != act_dtype() || S.dims.size() != 4 ||
+        S.dim(0) < slots || S.dim(1) != H || S.dim(2) != dim || S.dim(3) < vdim || S.dim(3) % 4 || raw.dim(1) < (int64_t)H * vdim ||
+        o.dim(1) < (int64_t)H * vdim)
+      return fail(MPK_ERR_INVALID, "mlstm: state [slots, heads, dim, vdim rounded up to 4], scratch and output [tokens, heads x vdim]");
+    for (int i = 3; i < 9; ++i) {
+      const int64_t w = i < 5 ? (int64_t)H * dim : (i < 7 ? (int64_t)H * vdim : H);
+      if (l.params[i] < 0 || l.params[i] + w > pr.dim(1)) return fail(MPK_ERR_INVALID, "mlstm: columns outside the projections");
+    }
+    for (int i = 1; i < 4; ++i)
+      if (T[l.t[i]].dtype != MPK_BF16 || (int64_t)(T[l.t[i]].bytes / 2) < (i == 3 ? (int64_t)H * vdim : H)) return fail(MPK_ERR_INVALID, "mlstm: bf16 biases [heads] and norm [heads x vdim]");
+    const int vc = MPK_MLSTM_COLUMNS(dim), nsub = (vdim + vc - 1) / vc;
+    if (chunks < 1 || chunks > nsub || nm.dims.size() != 4 || nm.dim(0) < slots || nm.dim(1) != H || nm.dim(2) != chunks || nm.dim(3) != dim + 1)
+      return fail(MPK_ERR_INVALID, "mlstm: chunk count or normaliser state [slots, heads, chunks, dim + 1]");
+    for (int s = 0; s < slots; ++s)
+      for (int h = 0; h < H; ++h)
+        for (int ch = 0; ch < chunks; ++ch) {
+          TaskDesc d = blank(TASK_MLSTM, li);
+          for (int k = 0; k < 8; ++k) d.p[k] = (uint64_t)T[l.t[k]].ptr;
+          d.a[ML_SLOT] = s; d.a[ML_HEAD] = h; d.a[ML_CHUNK] = ch; d.a[ML_NCHUNK] = chunks; d.a[ML_H] = H; d.a[ML_DIM] = dim;
+          d.a[ML_VDIM] = vdim; d.a[ML_VDIMP] = (int)S.dim(3);
+          d.a[ML_V0] = nsub * ch / chunks * vc; d.a[ML_V1] = std::min(nsub * (ch + 1) / chunks * vc, (int)S.dim(3));
+          d.a[ML_CAP] = bits_of(l.params[9]); d.a[ML_EPS] = bits_of(l.params[10]); d.a[ML_QSCALE] = bits_of(l.params[11]);
+          d.a[ML_LDP] = (int)pr.ld(); d.a[ML_QOFF] = (int)l.params[3]; d.a[ML_KOFF] = (int)l.params[4]; d.a[ML_VOFF] = (int)l.params[5];
+          d.a[ML_GOFF] = (int)l.params[6]; d.a[ML_IOFF] = (int)l.params[7]; d.a[ML_FOFF] = (int)l.params[8]; d.a[ML_LDO] = (int)o.ld();
+          d.a[ML_TICKET] = hybrid_tickets + s * H + h; d.a[ML_TC] = mlstm_tokens(dim); d.a[ML_LDR] = (int)raw.ld();
+          put(((s * H + h) * chunks + ch + rot) % W, d, ex);
+        }
+    hybrid_tickets += slots * H;
+    return MPK_OK;
+  }
+
   void emit_token_rows(uint32_t type, int li, int ex, uint64_t p0, uint64_t p1, uint64_t p2, int width, int ldi,
                        int ldo, int aux, int ldi2, int rows_total) {
     const int nt = std::min(rows_total, W);
@@ -947,7 +1249,13 @@ struct Builder {
     const int mbt = cfg.max_num_batched_tokens;
     switch (l.op) {
       case MPK_OP_LINEAR: case MPK_OP_LINEAR_RESIDUAL: case MPK_OP_SPLITK_LINEAR:
-        return emit_linear(li, ex);
+        return g->hybrid == HYB_F32 ? emit_linear_f32(li, ex) : emit_linear(li, ex);
+      case MPK_OP_RESIDUAL_NORM: return emit_residual_norm(li, ex);
+      case MPK_OP_QKV_APPEND: return emit_qkv_append(li, ex);
+      case MPK_OP_EXT_ATTENTION: return emit_ext_attention(li, ex);
+      case MPK_OP_SHORT_CONV: return emit_short_conv(li, ex);
+      case MPK_OP_RGLRU: return emit_rglru(li, ex);
+      case MPK_OP_MLSTM: return emit_mlstm(li, ex);
       case MPK_OP_LINEAR_FP8: case MPK_OP_LINEAR_FP8_RESIDUAL:
         return emit_linear_fp8(li, ex);
       case MPK_OP_QUANTIZE_FP8:
@@ -1093,6 +1401,13 @@ struct Builder {
       case MPK_OP_EMBED: {
         const TensorInfo &tab = T[l.t[1]], &y = T[l.t[2]];
         if (T[l.t[0]].dtype != MPK_I64) return fail(MPK_ERR_INVALID, "embed ids must be int64");
+        if (g->hybrid) {
+          // the table may be wider than the stream (padded to the projections' k granularity)
+          if (y.dtype != MPK_F32 || tab.dtype != MPK_BF16 || tab.dim(1) < y.dim(1)) return fail(MPK_ERR_INVALID, "embed in a hybrid graph: bf16 table, float32 output");
+          emit_token_rows(TASK_EMBED_F32, li, ex, (uint64_t)T[l.t[0]].ptr, (uint64_t)tab.ptr, (uint64_t)y.ptr,
+                          (int)y.dim(1), (int)tab.ld(), (int)y.ld(), (int)tab.dim(0), 0, mbt);
+          return MPK_OK;
+        }
         if (tab.dim(1) % 8 != 0) return fail(MPK_ERR_UNSUPPORTED, "embedding width must be a multiple of 8");
         emit_token_rows(TASK_EMBED, li, ex, (uint64_t)T[l.t[0]].ptr, (uint64_t)tab.ptr, (uint64_t)y.ptr,
                         (int)tab.dim(1), (int)tab.ld(), (int)y.ld(), (int)tab.dim(0), 0, mbt);
@@ -1147,6 +1462,8 @@ struct Builder {
         const int V = (int)lg.dim(1);
         if (pv.dim(1) < n || pi.dim(1) < n || pi.dtype != MPK_I64)
           return fail(MPK_ERR_INVALID, "argmax partial buffers must be [tokens, >= grid.x], index int64");
+        if (lg.dtype != (g->hybrid ? MPK_F32 : MPK_BF16) || pv.dtype != (g->hybrid && !sampling ? MPK_F32 : MPK_BF16))
+          return fail(MPK_ERR_INVALID, "argmax / sampling: bf16 logits and values (hybrid graphs: float32 logits, float32 argmax values)");
         for (int i = 0; i < n; ++i) {
           TaskDesc d = blank(sampling ? TASK_SAMPLING_PARTIAL : TASK_ARGMAX_PARTIAL, li);
           d.p[0] = (uint64_t)lg.ptr; d.p[1] = (uint64_t)pv.ptr; d.p[2] = (uint64_t)pi.ptr;
@@ -1229,8 +1546,17 @@ struct Builder {
     }
   }
 
+  // output tensor a layer writes only a column range of, and that range's first column
+  int sliced_output(const LayerInfo &l) const { return l.op == MPK_OP_EXT_ATTENTION ? l.t[3] : (l.op == MPK_OP_RGLRU ? l.t[9] : -1); }
+  int slice_column(const LayerInfo &l) const {
+    const size_t i = l.op == MPK_OP_EXT_ATTENTION ? 3 : 1;
+    return l.params.size() > i ? (int)l.params[i] : 0;
+  }
+
   int run() {
     int rc = check_arity();
+    if (rc) return rc;
+    rc = classify_hybrid();
     if (rc) return rc;
     for (const auto &l : L) if (l.folded) g->num_folded++;     // folded before materialisation (activation epilogue)
     fold_layers();
@@ -1256,6 +1582,13 @@ struct Builder {
 
     // ---- exec layers + dependencies ------------------------------------------------
     std::vector<int> exec_of_layer(L.size(), -1);
+    // Layers that write a column range of a wider tensor (the branches of a parallel mixer) do not wait for one another:
+    // every range is a storage of its own for its writers, and readers of the tensor read all of them.
+    int slice_id = 1 << 24;
+    for (const auto &l : L) {
+      const int t = sliced_output(l);
+      if (t >= 0 && !slices[T[t].storage].count(slice_column(l))) slices[T[t].storage][slice_column(l)] = slice_id++;
+    }
     if (!no_batch_task()) {
       ExecLayer b;
       b.type = TASK_BATCH;
@@ -1269,8 +1602,16 @@ struct Builder {
       e.layer = (int)i;
       std::vector<int> ins, outs;
       layer_io(L[i], &ins, &outs);
-      for (int t : ins) e.reads.push_back(T[t].storage);
-      for (int t : outs) e.writes.push_back(T[t].storage);
+      for (int t : ins) {
+        e.reads.push_back(T[t].storage);
+        auto it = slices.find(T[t].storage);
+        if (it != slices.end()) for (const auto &sl : it->second) e.reads.push_back(sl.second);
+      }
+      const int sliced = sliced_output(L[i]);
+      for (int t : outs) {
+        if (t == sliced) e.writes.push_back(slices[T[t].storage][slice_column(L[i])]);
+        else e.writes.push_back(T[t].storage);
+      }
       if (!no_batch_task()) e.reads.push_back(ST_META);
       e.remote_trigger = L[i].push && !L[i].push_ll;
       exec_of_layer[i] = (int)g->exec.size();
@@ -1330,6 +1671,7 @@ struct Builder {
       if (x.num_tasks == 0) return fail(MPK_ERR_INVALID, "layer " + std::to_string(x.layer) + " produced no task");
     }
     g->attn_tickets *= std::max(attn_ordinal, 1);
+    g->attn_tickets += hybrid_tickets;
     // ---- events: one per exec layer ---------------------------------------------------
     g->num_events = E;
     for (int e = 0; e < E; ++e) {
@@ -1368,7 +1710,7 @@ struct Builder {
     g->worker_begin[W] = (int32_t)g->tasks.size();
     g->general_kernel = cfg.max_num_batched_tokens > 8;
     for (const auto &d : g->tasks)
-      if ((d.type == TASK_LINEAR && (d.flags & TF_FP8)) || d.type >= TASK_QUANTIZE_FP8) g->general_kernel = true;
+      if (!g->hybrid && ((d.type == TASK_LINEAR && (d.flags & TF_FP8)) || d.type >= TASK_QUANTIZE_FP8)) g->general_kernel = true;
     g->num_workers = W;
     g->world_size = std::max(cfg.world_size, 1);
     // attention ticket banks: patch the ticket offset now that the bank size is known
@@ -1487,7 +1829,8 @@ std::string dump_task_graph(const CompiledGraph &g, const std::vector<TensorInfo
   static const char *names[] = {"nop", "batch", "embed", "rmsnorm", "linear", "attention", "silu_mul",
                                 "argmax_partial", "argmax_reduce", "allreduce", "elementwise_add", "tensor_init",
                                 "quantize_fp8", "moe_routing", "moe_gemm", "moe_silu_mul", "moe_mul_sum_add",
-                                "mla_append", "mla_decode", "mla_reduce", "sampling_partial", "sampling_reduce", "argmax_exchange", "ar_push"};
+                                "mla_append", "mla_decode", "mla_reduce", "sampling_partial", "sampling_reduce", "argmax_exchange", "ar_push",
+                                "embed_f32", "residual_norm", "linear_f32", "qkv_append", "ext_attention", "short_conv", "rglru", "mlstm"};
   std::ostringstream os;
   os << "{\"num_workers\": " << g.num_workers << ", \"num_tasks\": " << g.tasks.size()
      << ", \"num_events\": " << g.num_events << ", \"num_layers\": " << layers.size()
@@ -1496,7 +1839,7 @@ std::string dump_task_graph(const CompiledGraph &g, const std::vector<TensorInfo
      << ",\n \"events\": [\n";
   for (size_t e = 0; e < g.exec.size(); ++e) {
     const ExecLayer &x = g.exec[e];
-    os << "  {\"event\": " << e << ", \"type\": \"" << names[x.type < 24 ? x.type : 0] << "\", \"layer\": " << x.layer
+    os << "  {\"event\": " << e << ", \"type\": \"" << names[x.type < 32 ? x.type : 0] << "\", \"layer\": " << x.layer
        << ", \"tasks\": " << x.num_tasks << ", \"deps\": [";
     for (size_t k = 0; k < x.deps.size(); ++k) os << (k ? ", " : "") << "[" << x.deps[k] << ", " << x.dep_need[k] << "]";
     os << "]";

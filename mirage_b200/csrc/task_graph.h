@@ -92,6 +92,7 @@ struct CompiledGraph {
   int x_tile_bytes = 0;
   int num_allreduce = 0;
   bool general_kernel = false;            // FP8 tasks or more than 8 batched tokens: needs the general instantiation
+  int hybrid = 0;                         // HYB_* family: recurrent / extended-attention layers present
   bool use_tmem = false;                  // some linear runs on tcgen05: workers allocate tensor memory
   int tc_tokens = 0;                      // token rows of the tcgen05 activation operand tile
   std::vector<TmapSpec> tmaps;            // indexed by TaskDesc::a[L_TMAP]

@@ -83,6 +83,8 @@ class MPKMetadata:
         if self.weight_from_model:
             raise NotImplementedError("weight_from_model=True: loading checkpoints is outside this library; pass "
                                       "model_config.state_dict")
+        if hasattr(self.model_config, "check_valid"):      # models whose state is not one pair of cache tensors
+            return self.model_config.check_valid()
         assert self.model_config is not None and self.model_config.state_dict is not None, \
             "state_dict is required when weight_from_model is False"
         assert self.model_config.k_cache is not None and self.model_config.v_cache is not None

@@ -19,6 +19,7 @@ import ctypes as C
 import math
 import json
 import os
+import struct
 from typing import Dict, Optional, Sequence, Tuple
 
 import torch
@@ -130,8 +131,8 @@ class PersistentKernel:
     ):
         if mode not in valid_persistent_kernel_modes:
             raise ValueError(f"Invalid persistent kernel mode: {mode}")
-        if mode not in ("offline", "online_notoken") and not test_mode:
-            raise NotImplementedError(f"mode {mode!r} is not implemented by mirage_b200 (offline, online_notoken)")
+        if mode not in ("offline", "online", "online_notoken") and not test_mode:
+            raise NotImplementedError(f"mode {mode!r} is not implemented by mirage_b200 (offline, online, online_notoken)")
         if spec_decode_config is not None:
             raise NotImplementedError("speculative decoding is outside the decode path this library implements")
         self.__finalized__ = False
@@ -195,6 +196,13 @@ class PersistentKernel:
             if "paged_kv_indices_snapshot" not in mt and not dry_run:
                 mt["paged_kv_indices_snapshot"] = torch.empty(max_num_pages, dtype=torch.int32,
                                                               device=mt["tokens"].device)
+            if mode == "online":
+                # token-table rows are requests the host posts, extends and closes between launches
+                # (`request_ctl` [2, rows]; include/mpk_b200.h); `request_ids` tells which row a batch slot holds
+                for key, n in (("request_ctl", 2 * self.total_num_requests), ("request_ids", max_num_batched_requests)):
+                    if key not in mt:
+                        raise ValueError(f"meta_tensors[{key!r}] is required in online mode")
+                    assert mt[key].dtype == torch.int32 and mt[key].numel() >= n, key
         else:
             self.total_num_requests = 1
 
@@ -203,7 +211,7 @@ class PersistentKernel:
             return None if t is None or dry_run else t.data_ptr()
 
         cfg = N.MpkConfig()
-        cfg.mode = N.MODE_OFFLINE if mode == "offline" else N.MODE_ONLINE_NOTOKEN
+        cfg.mode = {"offline": N.MODE_OFFLINE, "online": N.MODE_ONLINE}.get(mode, N.MODE_ONLINE_NOTOKEN)
         cfg.test_mode, cfg.dry_run, cfg.device = int(test_mode), int(dry_run), self.device
         cfg.world_size, cfg.rank, cfg.num_workers = world_size, mpi_rank, self.num_workers
         cfg.max_seq_length, cfg.max_num_batched_requests = max_seq_length, max_num_batched_requests
@@ -216,6 +224,7 @@ class PersistentKernel:
         cfg.paged_kv_indices = ptr("paged_kv_indices_buffer")
         cfg.paged_kv_last_page_len = ptr("paged_kv_last_page_len_buffer")
         cfg.paged_kv_indices_snapshot = ptr("paged_kv_indices_snapshot")
+        cfg.state_slots, cfg.request_ctl, cfg.request_ids = ptr("state_slots"), ptr("request_ctl"), ptr("request_ids")
         if profiler_tensor is not None:
             cfg.profiler_buffer, cfg.profiler_entries = profiler_tensor.data_ptr(), profiler_tensor.numel()
         self._cfg = cfg
@@ -320,9 +329,14 @@ class PersistentKernel:
         assert input.num_dims == 2 and weight_linear.num_dims == 2 and output.num_dims == 2
         self._layer(N.OP_RMSNORM_LINEAR, [input, weight_norm, weight_linear, output], grid_dim)
 
-    def linear_layer(self, input: DTensor, weight: DTensor, output: DTensor, grid_dim: tuple, block_dim: tuple):
+    LINEAR_ACTIVATIONS = {None: 0, "relu2": 1}
+
+    def linear_layer(self, input: DTensor, weight: DTensor, output: DTensor, grid_dim: tuple, block_dim: tuple,
+                     activation: str = None):
+        """`activation` (squared relu, in hybrid graphs) is applied to the fp32 accumulator before the store."""
         assert input.num_dims == 2 and weight.num_dims == 2 and output.num_dims == 2
-        self._layer(N.OP_LINEAR, [input, weight, output], grid_dim)
+        act = self.LINEAR_ACTIVATIONS[activation]
+        self._layer(N.OP_LINEAR, [input, weight, output], grid_dim, [act] if act else [])
 
     def linear_with_residual_layer(self, input: DTensor, weight: DTensor, residual: DTensor, output: DTensor,
                                    grid_dim: tuple, block_dim: tuple):
@@ -485,13 +499,81 @@ class PersistentKernel:
         self._layer(N.OP_LINEAR_FP8_RESIDUAL, [input_fp8, input_scale, weight_fp8, weight_scale, residual, output],
                     grid_dim, [1])
 
+    # ---- hybrid graphs: float32 residual stream, attention with free head sizes, recurrent layers ------------
+    # (no reference counterpart; one of these layers makes the graph a hybrid graph, see include/mpk_b200.h)
+    @staticmethod
+    def _bits(x: float) -> int:
+        return struct.unpack("i", struct.pack("f", float(x)))[0]
+
+    def residual_norm_layer(self, x: DTensor, y: Optional[DTensor] = None, post_weight: Optional[DTensor] = None,
+                            norm_weight: Optional[DTensor] = None, output: Optional[DTensor] = None, eps: float = 1e-6,
+                            zero_centered: bool = False):
+        """x += rmsnorm(y) * w_post on the float32 stream `x` (x += y without `post_weight`, x unchanged without `y`),
+        then output = rmsnorm(x) * w_norm.  `zero_centered`: both weights are stored around zero (1 + w is applied)."""
+        assert x.num_dims == 2
+        self._layer(N.OP_RESIDUAL_NORM, [x, y, post_weight, norm_weight, output], (1, 1, 1),
+                    [self._bits(eps), int(zero_centered)])
+
+    def qkv_append_layer(self, proj: DTensor, q: DTensor, k_cache: DTensor, v_cache: DTensor, cos: DTensor, sin: DTensor,
+                         *, heads: int, kv_heads: int, dim: int, vdim: int, q_col: int, k_col: int, v_col: int,
+                         rot_dims: int, unit_norm: bool, eps: float):
+        """Takes q / k / v columns of the float32 projections: rotates the first `rot_dims` of q and k (half-split pairs,
+        float32 tables [positions, rot_dims / 2]), divides them by their RMS (`unit_norm`), and writes q and the cache
+        rows of the new positions.  Values are taken as projected; `v_col == k_col` makes the keys the values."""
+        self._layer(N.OP_QKV_APPEND, [proj, q, k_cache, v_cache, cos, sin], (1, 1, 1),
+                    [heads, kv_heads, dim, vdim, q_col, k_col, v_col, rot_dims, int(unit_norm), self._bits(eps)])
+
+    def ext_attention_layer(self, q: DTensor, k_cache: DTensor, v_cache: DTensor, output: DTensor, *, heads: int,
+                            kv_heads: int, vdim: int, scale: float, softcap: float = 0.0, sink: bool = False,
+                            out_col: int = 0, out_scale: float = 1.0):
+        """Causal paged attention over rows a qkv_append_layer wrote.  score = softcap * tanh(scale * q.k / softcap) (no
+        cap at 0); `sink` adds one to the softmax denominator; the result times `out_scale` goes to columns
+        [out_col, out_col + heads * vdim) of `output`."""
+        self._layer(N.OP_EXT_ATTENTION, [q, k_cache, v_cache, output], (1, 1, 1),
+                    [heads, kv_heads, vdim, out_col, self._bits(scale), self._bits(softcap or 0.0), int(sink),
+                     self._bits(out_scale)])
+
+    def short_conv_layer(self, input: DTensor, taps: DTensor, state: DTensor, output: DTensor, *,
+                         input_bias: Optional[DTensor] = None, bias: Optional[DTensor] = None, in_col: int = 0,
+                         activation: str = None):
+        """Causal convolution per channel over columns [in_col, in_col + channels) of `input` (+ `input_bias`); the last
+        taps - 1 inputs of a request live in `state` [slots, taps - 1, channels]."""
+        self._layer(N.OP_SHORT_CONV, [input, input_bias, taps, bias, state, output], (1, 1, 1),
+                    [in_col, {None: 0, "silu": 1}[activation]])
+
+    def rglru_layer(self, u: DTensor, proj: DTensor, y_bias: DTensor, ra: DTensor, ra_bias: DTensor, ri: DTensor,
+                    ri_bias: DTensor, lam: DTensor, state: DTensor, output: DTensor, *, y_col: int, out_col: int = 0,
+                    out_scale: float = 1.0, decay: float = 8.0):
+        """Real-gated linear recurrent unit (De et al., "Griffin: Mixing Gated Linear Recurrences with Local Attention
+        for Efficient Language Models"): block-diagonal gates on `u`, state S <- a S + sqrt(1 - a^2) i u with
+        log a = -decay * r * softplus(lam), output out_scale * S * gelu_tanh(proj[:, y_col:] + y_bias)."""
+        self._layer(N.OP_RGLRU, [u, proj, y_bias, ra, ra_bias, ri, ri_bias, lam, state, output], (1, 1, 1),
+                    [y_col, out_col, self._bits(out_scale), self._bits(decay)])
+
+    @staticmethod
+    def mlstm_chunks(num_workers: int, slots: int, heads: int, dim: int, vdim: int) -> int:
+        """Column ranges a head's matrix memory is cut into: enough tasks to occupy the workers, at most one per column
+        block the task body walks (MPK_MLSTM_COLUMNS of include/mpk_b200.h)."""
+        cols = 64 if dim <= 256 else (32 if dim <= 512 else 16)
+        return max(1, min(-(-vdim // cols), num_workers // max(slots * heads, 1)))
+
+    def mlstm_layer(self, proj: DTensor, i_bias: DTensor, f_bias: DTensor, norm: DTensor, state: DTensor,
+                    nm_state: DTensor, scratch: DTensor, output: DTensor, *, heads: int, dim: int, vdim: int, q_col: int,
+                    k_col: int, v_col: int, gate_col: int, i_col: int, f_col: int, gate_cap: float, eps: float,
+                    q_scale: float):
+        """Matrix-memory recurrence with exponential gates (Beck et al., "xLSTM: Extended Long Short-Term Memory"):
+        float32 state [slots, heads, dim, vdim up to a multiple of 4] and [slots, heads, chunks, dim + 1] (normaliser,
+        running maximum), per-head output norm, times sigmoid of the output gate columns."""
+        self._layer(N.OP_MLSTM, [proj, i_bias, f_bias, norm, state, nm_state, scratch, output], (1, 1, 1),
+                    [heads, dim, vdim, q_col, k_col, v_col, gate_col, i_col, f_col, self._bits(gate_cap), self._bits(eps),
+                     self._bits(q_scale), nm_state.dim(2)])
+
     # ---- mixture of experts (persistent_kernel.py:1385-1704 of the reference) -------------------------------
     def moe_topk_sigmoid_routing_layer(self, input: DTensor, bias: DTensor, output: tuple, grid_dim: tuple,
                                        block_dim: tuple, num_groups: int = 8, topk_group: int = 4,
                                        routed_scaling_factor: float = 2.5, local_experts: tuple = None):
         """input [B, E] logits (zeroed by the task), bias [E] float32; output = (topk_weight [B, topk] float32,
         routing_indices [E, B] int32 holding slot + 1 or 0, mask [E + 1] int32: active experts, count last)."""
-        import struct
         assert input.num_dims == 2 and bias.num_dims == 1 and len(output) == 3
         w, idx, mask = output
         assert w.num_dims == 2 and idx.num_dims == 2 and mask.num_dims == 1
@@ -553,7 +635,6 @@ class PersistentKernel:
                     [d_k, d_v, page_size])
 
     def _mla_decode(self, q_input, kv_input, output_partial, output_lse, q_len, kv_len, sm_scale):
-        import struct
         heads = q_input.dims[-1] // 576
         scale = self.MLA_DEFAULT_SCALE if sm_scale is None else float(sm_scale)
         bits = struct.unpack("i", struct.pack("f", scale))[0]
@@ -692,7 +773,7 @@ class PersistentKernel:
         """Run the whole generation like the reference's launch: iterate until no request is left
         (offline mode), or run the graph once (online_notoken / test mode)."""
         stream = kwargs.get("default_stream", None)
-        if self.test_mode or self.mode == "online_notoken":
+        if self.test_mode or self.mode in ("online", "online_notoken"):
             self.step(1, stream)
             return
         self.reset(stream)

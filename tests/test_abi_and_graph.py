@@ -28,8 +28,8 @@ def test_library_exports_every_symbol_of_the_header():
 
 def test_config_struct_matches_header_layout():
     from mirage_b200 import _native
-    # 15 int32 (+1 pad) + int64 + 12 pointers + uint64, as in mpk_config
-    assert ctypes.sizeof(_native.MpkConfig) == 14 * 4 + 8 + 12 * 8 + 8
+    # 14 int32 + int64 + 12 pointers + uint64 + 3 pointers, as in mpk_config
+    assert ctypes.sizeof(_native.MpkConfig) == 14 * 4 + 8 + 12 * 8 + 8 + 3 * 8
     assert ctypes.sizeof(_native.MpkStatus) == 6 * 4 + 8
 
 

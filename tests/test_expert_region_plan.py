@@ -1,5 +1,5 @@
 """The expert GEMM task keeps the operands of the step it computes and of the step it prefetches in two regions of
-the activation tile, placed by a few lines of arithmetic in `run_moe_gemm` (mirage_b200/csrc/megakernel.cu): the next
+the activation tile, placed by a few lines of arithmetic in `run_moe_gemm` (mirage_b200/csrc/megakernel.cuh): the next
 region goes behind the current one if it fits, else to the front if it fits in front of the current one, else the step
 is staged only after the current one is done.  This restates that arithmetic and checks, for random token counts per
 expert and for the tile sizes the graph compiler hands out, that the two live regions never overlap and never leave
