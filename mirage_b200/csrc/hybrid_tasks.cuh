@@ -30,6 +30,9 @@ __device__ __forceinline__ float bf16_at(uint64_t base, size_t i) {
 }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// Decay factor exp(x), x <= 0, of a recurrence that applies it once per token: near 1 the last-bit error of expf has a
+// sign of its own and adds up over a long memory; 1 + expm1f(x) rounds to nearest.
+__device__ __forceinline__ float decay_exp(float x) { return x > -0.35f ? 1.0f + expm1f(x) : expf(x); }
 __device__ __forceinline__ float gelu_tanh_f(float x) {
   return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
 }
@@ -785,7 +788,7 @@ __device__ __forceinline__ void run_rglru(const Ctx &c, const TaskDesc &d) {
       const int t = i / C, ch = i - t * C, g = gch + ch;
       const float r = sigmoid_f(rs[i] + bf16_at(d.p[4], g)), gi = sigmoid_f(is[i] + bf16_at(d.p[6], g));
       const float la = -gate_c * r * softplus_f(bf16_at(d.p[7], g));
-      float a = expf(la), b = sqrtf(-expm1f(2.0f * la)) * gi * us[(size_t)t * bs + c0 + ch];
+      float a = decay_exp(la), b = sqrtf(-expm1f(2.0f * la)) * gi * us[(size_t)t * bs + c0 + ch];
       const TokenRec &tr = rec[tb + t];
       if (tr.flags & 1) {   // the request's carried state enters here; nothing flows in from the previous token
         if (!(tr.flags & 4)) b = fmaf(a, __ldcg(state + (size_t)tr.slot * width + g), b);
@@ -868,7 +871,7 @@ __device__ __forceinline__ void mlstm_body(const Ctx &c, const TaskDesc &d, cons
   }
   consumer_sync();
   for (int t = tid; t < sv.nq; t += kConsumerThreads) {
-    dec[t] = expf(dec[t]);
+    dec[t] = decay_exp(dec[t]);
     inp[t] = expf(inp[t]);
     den[t] = expf(den[t]);
   }

@@ -974,6 +974,9 @@ struct Builder {
       return fail(MPK_ERR_UNSUPPORTED, "hybrid graphs batch at most 64 tokens");
     for (size_t i = 0; i < L.size(); ++i) {
       const LayerInfo &l = L[i];
+      const int act_out = l.op == MPK_OP_RESIDUAL_NORM || l.op == MPK_OP_EXT_ATTENTION || l.op == MPK_OP_RGLRU || l.op == MPK_OP_MLSTM
+                              ? l.t.back() : -1;   // output of the graph's activation type
+      if (act_out >= 0 && T[act_out].dtype == MPK_F32) f32 = true;
       if (hybrid_op(l.op) || l.op == MPK_OP_EMBED || l.op == MPK_OP_ARGMAX_PARTIAL || l.op == MPK_OP_ARGMAX_REDUCE ||
           l.op == MPK_OP_SAMPLING_PARTIAL || l.op == MPK_OP_SAMPLING_REDUCE) continue;
       if (l.op != MPK_OP_LINEAR) return fail(MPK_ERR_UNSUPPORTED, "layer " + std::to_string(i) + ": not available in a hybrid graph");

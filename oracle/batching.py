@@ -14,10 +14,17 @@ recorded its state after every call of eight seeded scenarios (tests/golden/batc
 tests/test_batching_golden.py requires this class to reproduce them array by array -- and, where the compiled
 reference is present, 40 further random scenarios live.  tests/test_batching_oracle.py keeps the hand-derived
 traces (page counts, indptr arrays, retirement on EOS / max length) as readable documentation of the rules.
+
+Additions of this library, outside the pinned part: `state_slots` (the recurrent-state slot of each batch slot: lowest
+free one at admission, kept until retirement) and online mode (`request_ctl` given): rows of the token table are requests
+the host posts (REQ_RUN / REQ_HOLD), extends and closes; a held request runs only the tokens supplied, and no request
+runs further than the free pages allow.
 """
 from __future__ import annotations
 
 import numpy as np
+
+REQ_FREE, REQ_RUN, REQ_HOLD, REQ_CLOSE = range(4)
 
 
 class BatchState:
@@ -25,7 +32,7 @@ class BatchState:
 
     def __init__(self, tokens: np.ndarray, prompt_lengths: np.ndarray, *,
                  max_num_batched_requests: int, max_num_batched_tokens: int,
-                 max_num_pages: int, page_size: int, eos_token_id: int = -1):
+                 max_num_pages: int, page_size: int, eos_token_id: int = -1, online: bool = False):
         self.R, self.max_seq_length = tokens.shape
         self.mbr = max_num_batched_requests
         self.mbt = max_num_batched_tokens
@@ -39,6 +46,9 @@ class BatchState:
         self.step = np.zeros(self.R, np.int32)
         self.next_request_id = 0
         self.request_ids = np.full(self.mbr, -1, np.int32)
+        self.state_slots = np.zeros(self.mbr, np.int32)
+        self.request_ctl = np.zeros(self.R, np.int32) if online else None
+        self.live = set()
         self.qo_indptr = np.zeros(self.mbr + 1, np.int32)
         self.paged_kv_indptr = np.zeros(self.mbr + 1, np.int32)
         self.paged_kv_indices = np.zeros(max_num_pages, np.int32)
@@ -72,6 +82,12 @@ class BatchState:
             self.step[rid] = step + n
             done = (step + n + 1 >= S) or (
                 self.tokens[rid, step + n] == self.eos and step + n >= plen)
+            if self.request_ctl is not None:
+                ctl = int(self.request_ctl[rid])
+                done = (done and ctl == REQ_RUN) or (ctl == REQ_CLOSE and step + n >= plen)
+                if done:
+                    self.request_ctl[rid] = REQ_FREE
+                    self.live.discard(rid)
             if done:
                 self.request_ids[i] = -1
                 kv = int(self.paged_kv_indptr[i])
@@ -82,6 +98,7 @@ class BatchState:
         snapshot = self.paged_kv_indices.copy()
         # Step 3 (:259-304): running requests keep their slot order.
         num_reqs = num_tokens = num_pages = 0
+        used = set()
         for i in range(self.mbr):
             rid = int(self.request_ids[i])
             if rid == -1:
@@ -97,6 +114,12 @@ class BatchState:
                 n_new = min(n_new, self.mbt - num_tokens)
             else:
                 n_new = min(1, self.mbt - num_tokens)
+                if self.request_ctl is not None and self.request_ctl[rid] != REQ_RUN:
+                    n_new = 0
+            if self.request_ctl is not None:
+                n_new = max(0, min(n_new, (n_old + tail - head) * P - step))
+            self.state_slots[num_reqs] = self.state_slots[i]
+            used.add(int(self.state_slots[i]))
             for j in range(n_new):
                 self.input_tokens[num_tokens + j] = self.tokens[rid, step + j]
             n_pages = (step + n_new + P - 1) // P
@@ -112,13 +135,26 @@ class BatchState:
             num_reqs += 1
         # admit new requests (:306-339)
         while num_reqs < self.mbr and num_tokens < self.mbt:
-            nxt = self.next_request_id
-            if nxt >= self.total_num_requests:
-                break
+            room = self.mbt - num_tokens
+            if self.request_ctl is None:
+                nxt = self.next_request_id
+                if nxt >= self.total_num_requests:
+                    break
+            else:
+                waiting = [r for r in range(self.R) if self.request_ctl[r] != REQ_FREE and r not in self.live]
+                if not waiting or tail <= head:
+                    break
+                nxt = waiting[0]
+                room = min(room, (tail - head) * P)
+                self.step[nxt] = 0
+                self.live.add(nxt)
+            slot = min(set(range(self.mbr)) - used)
+            used.add(slot)
+            self.state_slots[num_reqs] = slot
             self.request_ids[num_reqs] = nxt
             self.qo_indptr[num_reqs] = num_tokens
             self.paged_kv_indptr[num_reqs] = num_pages
-            n_new = min(int(self.prompt_lengths[nxt]), self.mbt - num_tokens)
+            n_new = min(int(self.prompt_lengths[nxt]), room)
             for j in range(n_new):
                 self.input_tokens[num_tokens + j] = self.tokens[nxt, j]
             n_pages = (n_new + P - 1) // P
@@ -130,7 +166,8 @@ class BatchState:
             num_tokens += n_new
             num_pages += n_pages
             num_reqs += 1
-            self.next_request_id = nxt + 1
+            if self.request_ctl is None:
+                self.next_request_id = nxt + 1
         # Step 4 (:341-348)
         self.request_ids[num_reqs:] = -1
         self.qo_indptr[num_reqs:] = num_tokens

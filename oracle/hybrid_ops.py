@@ -1,0 +1,127 @@
+"""CPU oracle of the mechanisms hybrid graphs are made of: one plain, slow function each.
+
+TEST INFRASTRUCTURE ONLY.  Whole sequences in, token loops for the recurrences, in the dtype of the inputs (the tests use
+float64).  Shares nothing with the product path.
+"""
+from __future__ import annotations
+
+import math
+from typing import Dict, Optional, Tuple
+
+import torch
+
+Tensor = torch.Tensor
+
+
+def rms_unit(x: Tensor, eps: float) -> Tensor:
+    return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
+
+
+def rms_norm_around_zero(x: Tensor, w: Tensor, eps: float) -> Tensor:
+    return rms_unit(x, eps) * (1 + w)
+
+
+def residual_norm(x: Tensor, y: Optional[Tensor], w_post: Optional[Tensor], w_next: Tensor, eps: float,
+                  around_zero: bool = True) -> Tuple[Tensor, Tensor]:
+    """(new stream, normed stream)."""
+    one = 1.0 if around_zero else 0.0
+    if y is not None:
+        x = x + (y if w_post is None else rms_unit(y, eps) * (one + w_post))
+    return x, rms_unit(x, eps) * (one + w_next)
+
+
+def rotate_half_split(x: Tensor, pos: Tensor, base: float, dims: int) -> Tensor:
+    """x [tokens, heads, size]; component i < dims / 2 turns with component i + dims / 2 by pos * base^(-2 i / dims)."""
+    out = x.clone()
+    for i in range(dims // 2):
+        a = pos.to(x.dtype) * base ** (-2.0 * i / dims)
+        c, s = torch.cos(a)[:, None], torch.sin(a)[:, None]
+        u, v = x[..., i], x[..., i + dims // 2]
+        out[..., i] = u * c - v * s
+        out[..., i + dims // 2] = v * c + u * s
+    return out
+
+
+def attention(q: Tensor, k: Tensor, v: Tensor, scale: float, softcap: float = 0.0, sink: bool = False) -> Tensor:
+    """q [tokens, H, d], k [tokens, G, d], v [tokens, G, dv]: causal, grouped heads -> [tokens, H, dv]."""
+    T, H = q.shape[:2]
+    G = k.shape[1]
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for h in range(H):
+        g = h // (H // G)
+        for t in range(T):
+            s = (k[:t + 1, g] @ q[t, h]) * scale
+            if softcap:
+                s = softcap * torch.tanh(s / softcap)
+            top = torch.clamp(s.max(), min=0.0) if sink else s.max()
+            e = torch.exp(s - top)
+            total = e.sum() + (torch.exp(-top) if sink else 0.0)
+            out[t, h] = (e / total) @ v[:t + 1, g]
+    return out
+
+
+def short_conv(x: Tensor, taps: Tensor, bias: Optional[Tensor]) -> Tensor:
+    """x [tokens, C], taps [C, n] (last column: the current token)."""
+    T, C = x.shape
+    n = taps.shape[1]
+    out = torch.zeros_like(x)
+    for t in range(T):
+        acc = torch.zeros(C, dtype=x.dtype) if bias is None else bias.clone()
+        for j in range(n):
+            src = t - (n - 1) + j
+            if src >= 0:
+                acc = acc + taps[:, j] * x[src]
+        out[t] = acc
+    return out
+
+
+def gelu_tanh(z: Tensor) -> Tensor:
+    return 0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def rglru(u: Tensor, ra: Tensor, ra_b: Tensor, ri: Tensor, ri_b: Tensor, lam: Tensor, decay: float = 8.0) -> Tensor:
+    """u [tokens, width], gate matrices [blocks, size, size] -> the recurrence's state after every token."""
+    T, width = u.shape
+    nb, size = ra.shape[:2]
+    S = torch.zeros(width, dtype=u.dtype)
+    out = torch.zeros_like(u)
+    for t in range(T):
+        r, i = torch.zeros_like(S), torch.zeros_like(S)
+        for b in range(nb):
+            sl = slice(b * size, (b + 1) * size)
+            r[sl] = torch.sigmoid(ra[b] @ u[t, sl] + ra_b[b])
+            i[sl] = torch.sigmoid(ri[b] @ u[t, sl] + ri_b[b])
+        log_a = -decay * r * torch.nn.functional.softplus(lam)
+        S = torch.exp(log_a) * S + torch.sqrt(-torch.expm1(2 * log_a)) * i * u[t]
+        out[t] = S
+    return out
+
+
+def mlstm(q: Tensor, k: Tensor, v: Tensor, i_pre: Tensor, f_pre: Tensor, cap: float) -> Tensor:
+    """q (already scaled), k [tokens, H, d], v [tokens, H, dv], gate pre-activations [tokens, H] -> read-outs
+    [tokens, H, dv], with the running maximum that keeps the exponentials bounded."""
+    T, H, d = q.shape
+    i_log = cap * torch.tanh(i_pre / cap)
+    f_log = torch.nn.functional.logsigmoid(cap * torch.tanh(f_pre / cap))
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for h in range(H):
+        S = torch.zeros(d, v.shape[2], dtype=q.dtype)
+        n = torch.zeros(d, dtype=q.dtype)
+        m = torch.zeros((), dtype=q.dtype)
+        for t in range(T):
+            m_new = torch.maximum(f_log[t, h] + m, i_log[t, h])
+            keep, add = torch.exp(f_log[t, h] + m - m_new), torch.exp(i_log[t, h] - m_new)
+            m = m_new
+            S = keep * S + add * torch.outer(k[t, h], v[t, h])
+            n = keep * n + add * k[t, h]
+            out[t, h] = (q[t, h] @ S) / (torch.maximum((n @ q[t, h]).abs(), torch.exp(-m)) + 1e-6)
+    return out
+
+
+def mlstm_output(o: Tensor, norm: Tensor, gate: Tensor, eps: float) -> Tensor:
+    """Read-outs [tokens, H, dv] -> per-head unit norm, times the weight, times sigmoid(gate) [tokens, H * dv]."""
+    return rms_unit(o, eps).reshape(o.shape[0], -1) * norm * torch.sigmoid(gate)
+
+
+def squared_relu(x: Tensor) -> Tensor:
+    return torch.relu(x) ** 2
