@@ -159,26 +159,44 @@ def test_greedy_generation_through_the_scheduler(model, dtype):
     assert r.generate(prompts) == got                               # a second run starts from clean state
 
 
-def test_generation_through_the_model_wrapper_and_sampling(model):
+def test_generation_through_the_model_wrapper(model):
     import mirage_b200 as mi
     from mirage_b200.builders.palarax import PalaraxConfig, PalaraxModelConfig, allocate_state
     c, w, toks, _ = model
     cfg = PalaraxConfig.from_dict(c)
     prompts = [toks["c"][:6], toks["b"][:10]]
-    out = {}
-    for seed in (None, 17):
-        sizes = dict(max_num_batched_requests=2, max_num_batched_tokens=8, max_num_pages=8, page_size=16)
-        state = allocate_state(cfg, slots=2, max_num_pages=8, page_size=16, dtype=torch.float32, device="cuda",
-                               num_workers=mi.get_configurations_from_gpu(0)[0])
-        m = mi.MPK(mi.MPKMetadata(mode="offline", total_num_requests=2, max_seq_length=40, model_name="Palarax",
-                                  model_config=PalaraxModelConfig(cfg, {k: v.cuda() for k, v in w.items()}, state,
-                                                                  torch.float32, seed), **sizes))
-        m.build()
-        out[seed] = m.run_ids(prompts)
-        assert out[seed] == m.run_ids(prompts)
+    sizes = dict(max_num_batched_requests=2, max_num_batched_tokens=8, max_num_pages=8, page_size=16)
+    state = allocate_state(cfg, slots=2, max_num_pages=8, page_size=16, dtype=torch.float32, device="cuda",
+                           num_workers=mi.get_configurations_from_gpu(0)[0])
+    m = mi.MPK(mi.MPKMetadata(mode="offline", total_num_requests=2, max_seq_length=40, model_name="Palarax",
+                              model_config=PalaraxModelConfig(cfg, {k: v.cuda() for k, v in w.items()}, state, torch.float32), **sizes))
+    m.build()
+    m.compile()
+    out = m.run_ids(prompts)
     orc = P.PalaraxOracle(c, w)
-    assert [o[:len(p) + 5] for o, p in zip(out[None], prompts)] == [orc.greedy(p, 5) for p in prompts]
-    assert out[17] != out[None] and all(0 <= t < c["vocab"] for o in out[17] for t in o)
+    assert [o[:len(p) + 5] for o, p in zip(out, prompts)] == [orc.greedy(p, 5) for p in prompts]
+    assert m.run_ids(prompts) == out
+
+
+def test_sampled_ids_are_the_largest_keys_of_the_logits(model):
+    from oracle import sampling_ops as so
+    c, w, toks, _ = model
+    flat = dict(w)
+    flat["final.norm"] = (w["final.norm"].float() * 0.05 - 0.95).to(torch.bfloat16)   # logits small enough for the noise to decide
+    seed = 4242
+    r = runner(c, flat, torch.bfloat16, mode="offline", requests=3, slots=3, tokens=12, pages=12, max_seq=40, sampling_seed=seed)
+    r.load_prompts([toks["c"], toks["b"][:5], toks["d"]])
+    differs = 0
+    for _ in range(12):
+        r.step(1)
+        n = r.mpk.status().active_tokens
+        logits, ids = r.logits[:n].cpu(), r.meta["output_tokens"][:n, 0].cpu()
+        keys = so.sampling_keys(logits.to(torch.bfloat16), seed, 1).float()
+        top = keys.max(-1).values
+        step = 2.0 ** (torch.floor(torch.log2(top.abs().clamp_min(1e-20))) - 7)       # one bf16 step at the top key
+        assert bool((keys.gather(1, ids[:, None])[:, 0] >= top - 2 * step).all())
+        differs += int((ids != logits.argmax(-1)).sum())
+    assert differs > 0
 
 
 def test_online_scheduler_matches_its_oracle_bit_for_bit(model):
