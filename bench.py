@@ -750,6 +750,139 @@ def run_deepseek_slice(args):
         dist.destroy_process_group()
 
 
+# Palarax at real layer sizes beside Qwen3 layers of (about) the same parameter count: 6 matrix-memory layers and 2 parallel
+# layers against 8 Qwen3 layers, same width, head counts and vocabulary.
+HYBRID_SIZES = {
+    "4096": dict(width=4096, layers=8, heads=32, kv=8, dim=128, ff=16384, mheads=8, mdim=256, mvdim=512, blocks=16, qwen_ff=12288),
+    "2048": dict(width=2048, layers=8, heads=16, kv=8, dim=128, ff=8192, mheads=4, mdim=256, mvdim=512, blocks=8, qwen_ff=6144),
+}
+HYBRID_VOCAB = 32768
+
+
+def palarax_case(z, dev):
+    """(config, device weights) of one size; random weights in the ranges that keep the recurrences alive."""
+    import torch
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    ml = {"type": "mlstm", "mlp": mlp, "mixer": {"heads": z["mheads"], "dim": z["mdim"], "vdim": z["mvdim"], "gate_cap": 15.0}}
+    pa = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+                 "softcap": 50.0, "rot": {"base": 1e6, "dims": z["dim"]}},
+        "right": {"width": z["width"], "blocks": z["blocks"], "conv": 4}, "left_scale": 0.7, "right_scale": 0.7}}
+    c = {"architecture": "Palarax", "vocab": HYBRID_VOCAB, "width": z["width"], "norm": {"eps": 1e-6},
+         "layers": [pa if n % 4 == 3 else ml for n in range(z["layers"])]}
+    g = torch.Generator(device=dev).manual_seed(1)
+    rnd = lambda *s, std=None, mean=0.0: (mean + (s[-1] ** -0.5 if std is None else std) * torch.randn(
+        *s, generator=g, device=dev)).to(torch.bfloat16)
+    D, w = z["width"], {"embed": rnd(HYBRID_VOCAB, z["width"], std=1.0), "final.norm": rnd(z["width"], std=0.1)}
+    for n, layer in enumerate(c["layers"]):
+        p = f"l{n}."
+        for nm in ("norm1", "norm1b", "norm2", "norm2b"):
+            w[p + nm] = rnd(D, std=0.1)
+        w[p + "mlp.up"], w[p + "mlp.down"] = rnd(z["ff"], D), rnd(D, z["ff"])
+        if layer["type"] == "mlstm":
+            H, d, dv = z["mheads"], z["mdim"], z["mvdim"]
+            for nm, rows in (("q", H * d), ("k", H * d), ("v", H * dv), ("g", H * dv), ("i", H), ("f", H)):
+                w[p + "mix." + nm] = rnd(rows, D)
+            w[p + "mix.o"], w[p + "mix.norm"] = rnd(D, H * dv), rnd(H * dv, std=0.1, mean=1.0)
+            w[p + "mix.i.b"], w[p + "mix.f.b"] = rnd(H, std=1.0), rnd(H, std=1.0, mean=4.0)
+        else:
+            l, r = p + "mix.left.", p + "mix.right."
+            w[l + "q"], w[l + "k"], w[l + "o"] = rnd(z["heads"] * z["dim"], D), rnd(z["kv"] * z["dim"], D), rnd(D, z["heads"] * z["dim"])
+            for nm in ("y", "x"):
+                w[r + nm], w[r + nm + ".b"] = rnd(D, D), rnd(D, std=0.3)
+            w[r + "conv"], w[r + "conv.b"], w[r + "o"], w[r + "lam"] = rnd(D, 4, std=0.5), rnd(D, std=0.2), rnd(D, D), rnd(D, mean=-5.0, std=1.0)
+            for nm in ("ra", "ri"):
+                s = D // z["blocks"]
+                w[r + nm], w[r + nm + ".b"] = rnd(z["blocks"], s, s), rnd(z["blocks"], s, std=0.5)
+    return c, w
+
+
+def run_palarax(args):
+    """Prefill (one request, 64 tokens per launch) and decode (batch 1, 16, 64 at --context) of Palarax and of Qwen3 layers of
+    equal size, with the spans of every kind of task group from the in-kernel profiler.  Timed launches carry no profiler."""
+    import torch
+    from mirage_b200.builders.palarax import PalaraxConfig
+    from mirage_b200.builders.runner import DecoderShape, PalaraxRunner, Qwen3Runner
+    from mirage_b200.profiler import event_spans
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    K, Wm, ctx, page = min(args.steps, 64), max(args.warmup, 3), args.context, 64
+    peak, peak_kind = measured_peak_gbs()
+    g = torch.Generator().manual_seed(5)
+
+    def case(make, B, mbt, prompt):
+        """ms per launch, weight bytes per launch, {task type: (groups, mean us)}."""
+        max_seq = -(-(ctx + prompt + 2 * K + 4 * Wm + 16) // page) * page
+        kw = dict(total_num_requests=B, max_seq_length=max_seq, max_num_batched_requests=B, max_num_batched_tokens=mbt,
+                  max_num_pages=B * (max_seq // page), page_size=page)
+        spans, ms, clk = {}, None, None
+        for profiled in (False, True):
+            prof = torch.zeros(1 << 20, dtype=torch.int64, device=dev) if profiled else None
+            r = make(kw, prof)
+            r.load_prompts([torch.randint(0, HYBRID_VOCAB, (max(prompt, 1),), generator=g).tolist() for _ in range(B)])
+            steps = K
+            if prompt > 1:
+                lead = ctx // mbt                     # launches before the timed ones: the context of the timed tokens
+                steps = (prompt // mbt) - lead
+                r.step(lead)
+            else:
+                r.step(ctx + Wm)
+            st = r.mpk.status()
+            assert st.active_tokens == (mbt if prompt > 1 else B), st.active_tokens
+            if profiled:
+                r.step(1)
+                r.mpk.status()
+                info = r.mpk.graph_info()
+                for e in event_spans(prof, info["num_tasks"]).values():
+                    spans.setdefault(e["type"], []).append(e["us"])
+                continue
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize()
+            with ClockSampler(0) as clocks:
+                e0.record()
+                r.step(steps)
+                e1.record()
+                torch.cuda.synchronize()
+            ms, clk = e0.elapsed_time(e1) / steps, clocks.summary()
+            assert r.mpk.status().error == 0
+            wb = r.mpk.graph_info()["weight_bytes_per_step"]
+            del r
+            torch.cuda.empty_cache()
+        return ms, wb, {k: [len(v), round(sum(v) / len(v), 2)] for k, v in sorted(spans.items())}, clk
+
+    results, launches, clk = [], 0, None
+    for size, z in HYBRID_SIZES.items():
+        for model in ("palarax", "qwen3"):
+            if model == "palarax":
+                c, w = palarax_case(z, dev)
+                make = lambda kw, prof: PalaraxRunner(PalaraxConfig.from_dict(c), w, profiler_tensor=prof, **kw)
+            else:
+                shape = dict(num_layers=z["layers"], hidden_size=z["width"], num_q_heads=z["heads"], num_kv_heads=z["kv"],
+                             head_dim=z["dim"], intermediate_size=z["qwen_ff"], vocab_size=HYBRID_VOCAB)
+                w = make_gpu_weights(shape, 7, dev)
+                make = lambda kw, prof: Qwen3Runner(DecoderShape(max_position=8192, **shape), w, profiler_tensor=prof, **kw)
+            for name, B, mbt, prompt in (("prefill64", 1, 64, ctx + 1024), ("decode1", 1, 1, 1), ("decode16", 16, 16, 1),
+                                         ("decode64", 64, 64, 1)):
+                full = f"{model}_{size}_{name}"
+                if args.cases not in full:
+                    continue
+                ms, wb, spans, clk = case(make, B, mbt, prompt)
+                n = mbt if prompt > 1 else B
+                results.append({"case": full, "ms_per_launch": round(ms, 4), "tok_s": round(n * 1e3 / ms, 1), "weight_gb": round(wb / 1e9, 3),
+                                "weight_roofline_frac": round(wb / (ms * 1e-3) / 1e9 / peak, 3), "groups_us": spans})
+                launches += K
+            w = None
+            torch.cuda.empty_cache()
+    head = [r for r in results if r["case"] == "palarax_4096_decode1"] or results
+    print(json.dumps({
+        "metric": "palarax_decode_ms_per_token_bs1", "value": head[0]["ms_per_launch"], "unit": "ms/token", "n_gpus": 1, "steps": K,
+        "warmup": Wm, "ms_per_step": head[0]["ms_per_launch"], "higher_is_better": False, "scaling": "strong", "vs_baseline": None,
+        "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": "Palarax 6 matrix-memory + 2 parallel layers beside 8 Qwen3 layers, width 4096 and 2048, context %d" % ctx,
+                   "l2": "weights of a launch exceed L2; every launch re-streams them"},
+        "gpu_launches": launches, "clocks": clk, "peak_gbs": peak, "peak_kind": peak_kind, "results": results}))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -772,9 +905,12 @@ def main():
     ap.add_argument("--shard-lm-head", action="store_true",
                     help="N > 1: split the lm_head rows over the ranks and merge the ranks' argmax inside the kernel "
                          "(default: every rank keeps the whole lm_head, as the reference does)")
-    ap.add_argument("--workload", default="qwen3", choices=["qwen3", "fp8_layer", "moe_block", "mla_decode", "deepseek_slice", "moe_w13", "mla_dense"],
+    ap.add_argument("--workload", default="qwen3", choices=["qwen3", "fp8_layer", "moe_block", "mla_decode", "deepseek_slice", "moe_w13", "mla_dense",
+                                                             "palarax"],
                     help="qwen3: the headline decode benchmark; the others time one block of the FP8 / MoE / MLA "
-                         "task bodies at the shapes of the DeepSeek-V3-style parity configurations (1 GPU)")
+                         "task bodies at the shapes of the DeepSeek-V3-style parity configurations (1 GPU); palarax: prefill "
+                         "and decode of Palarax at a few sizes beside Qwen3 layers of equal size (1 GPU)")
+    ap.add_argument("--cases", default="", help="palarax: only cases whose name contains this text")
     args = ap.parse_args()
     if args.impl == "reference":
         return run_reference(args)
@@ -782,6 +918,8 @@ def main():
         return run_ref_kernel(args)
     if args.workload == "deepseek_slice":
         return run_deepseek_slice(args)
+    if args.workload == "palarax":
+        return run_palarax(args)
     if args.workload != "qwen3":
         return run_block_workload(args)
 

@@ -96,7 +96,7 @@ class Qwen3Runner(DecoderRunner):
                  device: Optional[int] = None, num_workers: int = 0, sampling_seed: Optional[int] = None,
                  shard_lm_head: bool = False,
                  fp8_state_dict: Optional[Dict[str, tuple]] = None, link_peers: bool = True,
-                 presharded: bool = False, mode: str = "offline"):
+                 presharded: bool = False, mode: str = "offline", profiler_tensor: Optional[torch.Tensor] = None):
         """`state_dict` / `fp8_state_dict` hold the whole model and are cut for this rank here, unless `presharded`:
         then they are this rank's shard already (what `checkpoint.load_sharded_state_dict` returns)."""
         dev = torch.device("cuda", torch.cuda.current_device() if device is None else device)
@@ -117,7 +117,7 @@ class Qwen3Runner(DecoderRunner):
             mode=mode, world_size=world_size, mpi_rank=rank, num_workers=num_workers,
             max_seq_length=max_seq_length, max_num_batched_requests=mbr, max_num_batched_tokens=mbt,
             max_num_pages=max_num_pages, page_size=page_size, meta_tensors=self.meta, eos_token_id=eos_token_id,
-            device=dev.index)
+            device=dev.index, profiler_tensor=profiler_tensor)
         cfg = Qwen3ModelConfig(
             hidden_size=shape.hidden_size, intermediate_size=shape.intermediate_size // world_size,
             vocab_size=shape.vocab_size, local_num_q_heads=shape.num_q_heads // world_size,

@@ -15,7 +15,8 @@ import torch
 
 TASK_NAMES = ["nop", "batch", "embed", "rmsnorm", "linear", "attention", "silu_mul", "argmax_partial", "argmax_reduce",
               "allreduce", "elementwise_add", "tensor_init", "quantize_fp8", "moe_routing", "moe_gemm", "moe_silu_mul",
-              "moe_mul_sum_add", "mla_append", "mla_decode", "mla_reduce", "sampling_partial", "sampling_reduce", "argmax_exchange", "ar_push"]
+              "moe_mul_sum_add", "mla_append", "mla_decode", "mla_reduce", "sampling_partial", "sampling_reduce", "argmax_exchange", "ar_push",
+              "embed_f32", "residual_norm", "linear_f32", "qkv_append", "ext_attention", "short_conv", "rglru", "mlstm"]
 
 
 def decode_records(profiler_buffer: torch.Tensor, num_tasks: int) -> List[Dict[str, int]]:
@@ -30,6 +31,18 @@ def decode_records(profiler_buffer: torch.Tensor, num_tasks: int) -> List[Dict[s
         tag = r[3] & 0xFFFFFFFFFFFFFFFF
         out.append({"worker": int(tag >> 40), "event": int((tag >> 8) & 0xFFFFFFFF), "type": int(tag & 0xFF),
                     "begin_ns": r[0] - t0, "ready_ns": max(r[1], r[0]) - t0, "end_ns": r[2] - t0})
+    return out
+
+
+def event_spans(profiler_buffer: torch.Tensor, num_tasks: int) -> Dict[int, Dict[str, float]]:
+    """Per event (one group of tasks cut from one layer): task type and the microseconds from its first task's ready time
+    to its last task's end."""
+    out: Dict[int, Dict[str, float]] = {}
+    for r in decode_records(profiler_buffer, num_tasks):
+        e = out.setdefault(r["event"], {"type": TASK_NAMES[r["type"]], "t0": r["ready_ns"], "t1": r["end_ns"]})
+        e["t0"], e["t1"] = min(e["t0"], r["ready_ns"]), max(e["t1"], r["end_ns"])
+    for e in out.values():
+        e["us"] = (e["t1"] - e["t0"]) / 1e3
     return out
 
 
@@ -82,6 +95,7 @@ REFERENCE_EVENT_IDS = {
     "sampling_reduce": 265,
     "argmax_exchange": 107,   # TASK_REDUCE
     "ar_push": 302,           # TASK_NVSHMEM_TILE_ALLREDUCE
+    "embed_f32": 101, "residual_norm": 119, "linear_f32": 253, "qkv_append": 257, "ext_attention": 257,
 }
 REFERENCE_WAIT_EVENT_ID = 203  # TASK_GET_NEXT_TASK: the span a worker spends waiting for a task's dependencies
 
