@@ -121,7 +121,7 @@ typedef enum {
 
 /* Value columns a task of an MPK_OP_MLSTM layer walks at a time; the layer's `chunks` parameter (and the second state
  * tensor [slots, heads, chunks, dim + 1]) may be at most ceil(vdim / this).  */
-#define MPK_MLSTM_COLUMNS(dim) ((dim) <= 256 ? 64 : (dim) <= 512 ? 32 : 16)
+#define MPK_MLSTM_COLUMNS(dim) ((dim) <= 128 ? 64 : (dim) <= 256 ? 32 : (dim) <= 512 ? 16 : 8)
 
 /* Constructor arguments of PersistentKernel (persistent_kernel.py:349-369) plus the
  * meta tensors it hands to init_func (:2494-2506).  All pointers are DEVICE

@@ -222,6 +222,11 @@ class PalaraxBuilder:
         self._linear(h, self._weight(p + "qkyx", [sd[pl + "q"], sd[pl + "k"], sd[pr + "y"], sd[pr + "x"]]), proj)
         left_out = l.heads * l.vdim
         mixed = self._buf("mixed", self._kpad(left_out + r.width), self.act)
+        # right branch, first half: a worker runs its tasks in layer order, so what is short and early in both branches comes
+        # first, and no branch waits behind the other's long task
+        u = self._buf("conv_out", r.width, float32)
+        mpk.short_conv_layer(proj, self._att(pr + "conv"), mpk.attach_input(st["conv"], name=pr + "conv_state"), u,
+                             input_bias=self._att(pr + "x.b"), bias=self._att(pr + "conv.b"), in_col=x_col)
         # left branch
         kc, vc = mpk.attach_input(st["k"], name=pl + "k_cache"), mpk.attach_input(st["v"], name=pl + "v_cache")
         q = self._buf("q", l.heads * kc.dim(3), self.act)
@@ -230,10 +235,7 @@ class PalaraxBuilder:
                              k_col=k_col, v_col=k_col, rot_dims=l.rot_dims, unit_norm=True, eps=self.eps)
         mpk.ext_attention_layer(q, kc, vc, mixed, heads=l.heads, kv_heads=l.kv_heads, vdim=l.vdim, scale=l.scale,
                                 softcap=l.softcap, sink=True, out_col=0, out_scale=m.left_scale)
-        # right branch
-        u = self._buf("conv_out", r.width, float32)
-        mpk.short_conv_layer(proj, self._att(pr + "conv"), mpk.attach_input(st["conv"], name=pr + "conv_state"), u,
-                             input_bias=self._att(pr + "x.b"), bias=self._att(pr + "conv.b"), in_col=x_col)
+        # right branch, second half
         mpk.rglru_layer(u, proj, self._att(pr + "y.b"), self._att(pr + "ra"), self._att(pr + "ra.b"), self._att(pr + "ri"),
                         self._att(pr + "ri.b"), self._att(pr + "lam"), mpk.attach_input(st["diag"], name=pr + "state"), mixed,
                         y_col=y_col, out_col=left_out, out_scale=m.right_scale, decay=PalaraxConfig.DECAY)

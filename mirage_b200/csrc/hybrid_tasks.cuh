@@ -13,6 +13,10 @@
 //
 // HYB = HYB_BF16: matrix operands, the KV cache and the operands handed to projections are bf16, everything else is
 // float32.  HYB = HYB_F32: those are float32 as well.
+//
+// The bodies are functions of their own (__noinline__): inlined side by side into the task switch they share one register
+// allocation, and every variant added makes the linear loop and the others spill.  They take the context by value: a
+// reference would keep it in local memory for the whole kernel.
 #pragma once
 #include "megakernel.cuh"
 
@@ -40,6 +44,12 @@ __device__ __forceinline__ float warp_max(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
   return v;
+}
+// Phase stamp i (0..3) of a task's profiler record.
+__device__ __forceinline__ void stamp(const Ctx &c, int task, int i) {
+  const KernelParams &P = c.P;
+  if (threadIdx.x == 0 && P.profiler != nullptr && (uint64_t)(task + 1) * 8 <= P.profiler_entries)
+    P.profiler[(size_t)task * 8 + 4 + i] = globaltimer_ns();
 }
 // Sum over the 256 compute threads (slots: 8 floats of shared memory; the caller keeps two calls apart with a barrier
 // or with different slots).
@@ -172,8 +182,83 @@ __device__ __forceinline__ void residual_norm_rows(const Ctx &c, const TaskDesc 
     consumer_sync();   // the reduction slots are used again by the next row
   }
 }
+// Four bf16 values as floats (8-byte aligned).
+__device__ __forceinline__ float4 bf16x4_at(uint64_t base, int i) {
+  const uint2 v = __ldg(reinterpret_cast<const uint2 *>(base + 2ull * i));
+  return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y));
+}
+__device__ __forceinline__ void store_elt4(__nv_bfloat16 *p, float4 v) {
+  *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+}
+__device__ __forceinline__ void store_elt4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+
+// The same for aligned rows of at most 4096 columns: row, sublayer output and both weights sit in registers, every load of
+// a row is in flight before the first reduction.
 template <int HYB>
-__device__ __forceinline__ void run_residual_norm(const Ctx &c, const TaskDesc &d) {
+__device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc &d) {
+  typedef typename HybElt<HYB>::T T;
+  constexpr int NV = 4;
+  const int B = active_tokens(c.P);
+  const int t0 = d.a[0], t1 = min(d.a[1], B), W = d.a[2], tid = threadIdx.x;
+  const float eps = __int_as_float(d.a[6]);
+  const float off = (d.a[7] & 2) ? 1.0f : 0.0f;
+  const bool has_y = d.p[1] != 0, has_post = d.p[2] != 0, has_out = d.p[3] != 0;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int t = t0; t < t1; ++t) {
+    float *x = reinterpret_cast<float *>(d.p[0]) + (size_t)t * d.a[3];
+    const float *y = reinterpret_cast<const float *>(d.p[1]) + (size_t)t * d.a[4];
+    float4 xv[NV], yv[NV], wp[NV], wn[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int j = (i * kConsumerThreads + tid) * 4;
+      const bool in = j < W;
+      yv[i] = in && has_y ? __ldcg(reinterpret_cast<const float4 *>(y + j)) : zero;
+      xv[i] = in ? __ldcg(reinterpret_cast<const float4 *>(x + j)) : zero;
+      wp[i] = in && has_post ? bf16x4_at(d.p[2], j) : zero;
+      wn[i] = in && has_out ? bf16x4_at(d.p[3], j) : zero;
+    }
+    if (has_y) {
+      float inv = 1.f;
+      if (has_post) {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) ss += yv[i].x * yv[i].x + yv[i].y * yv[i].y + yv[i].z * yv[i].z + yv[i].w * yv[i].w;
+        inv = 1.0f / sqrtf(block_sum(ss, c.s.red) / (float)W + eps);
+      }
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const float ox = has_post ? off + wp[i].x : 1.f, oy = has_post ? off + wp[i].y : 1.f, oz = has_post ? off + wp[i].z : 1.f,
+                    ow = has_post ? off + wp[i].w : 1.f;
+        xv[i].x += yv[i].x * inv * ox; xv[i].y += yv[i].y * inv * oy;
+        xv[i].z += yv[i].z * inv * oz; xv[i].w += yv[i].w * inv * ow;
+        const int j = (i * kConsumerThreads + tid) * 4;
+        if (j < W) *reinterpret_cast<float4 *>(x + j) = xv[i];
+      }
+    }
+    if (has_out) {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) ss += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
+      const float inv = 1.0f / sqrtf(block_sum(ss, c.s.red + 8) / (float)W + eps);
+      T *out = reinterpret_cast<T *>(d.p[4]) + (size_t)t * d.a[5];
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int j = (i * kConsumerThreads + tid) * 4;
+        if (j < W)
+          store_elt4(out + j, make_float4(xv[i].x * inv * (off + wn[i].x), xv[i].y * inv * (off + wn[i].y), xv[i].z * inv * (off + wn[i].z),
+                                          xv[i].w * inv * (off + wn[i].w)));
+      }
+    }
+    if (t + 1 < t1) consumer_sync();   // the reduction slots are used again by the next row
+  }
+}
+template <int HYB>
+__device__ __noinline__ void run_residual_norm(const Ctx c, const TaskDesc &d) {
+  if (d.a[2] <= 4096 && ((d.a[2] | d.a[3] | d.a[4] | d.a[5]) & 3) == 0 && ((d.p[0] | d.p[1] | d.p[4]) & 15) == 0 &&
+      ((d.p[2] | d.p[3]) & 7) == 0) {
+    residual_norm_wide<HYB>(c, d);
+    return;
+  }
   if (((d.a[2] | d.a[3] | d.a[4]) & 3) == 0 && ((d.p[0] | d.p[1]) & 15) == 0) residual_norm_rows<HYB, 4>(c, d);
   else residual_norm_rows<HYB, 1>(c, d);
 }
@@ -225,7 +310,7 @@ __device__ __forceinline__ void run_linear_f32(const Ctx &c, const TaskDesc &d) 
 // page of its position together with the value row.
 // ---------------------------------------------------------------------------
 template <int HYB>
-__device__ __forceinline__ void run_qkv_append(const Ctx &c, const TaskDesc &d) {
+__device__ __noinline__ void run_qkv_append(const Ctx c, const TaskDesc &d) {
   typedef typename HybElt<HYB>::T T;
   const KernelParams &P = c.P;
   const int B = active_tokens(P);
@@ -313,26 +398,32 @@ __device__ __forceinline__ void attn_emit_row(const Ctx &c, const TaskDesc &d, c
     const float L = l * w + (o.sink ? exp_dom<HYB>(-M) : 0.f);
     const float f = L > 0.f ? w / L * o.oscale : 0.f;
     T *out = reinterpret_cast<T *>(d.p[3]) + (size_t)tok * o.ldo + o.ocol + (size_t)hq_idx * o.vdim;
-    for (int j = lane; j < o.vdim; j += 32) store_elt(out + j, val(j) * f);
+    for (int j0 = 0; j0 < o.vdim; j0 += 32) {   // (val may shuffle: the whole warp calls it)
+      const float v = val(j0 + lane);
+      if (j0 + lane < o.vdim) store_elt(out + j0 + lane, v * f);
+    }
   } else {
     float *rec = c.P.attn_scratch + (((size_t)tok * o.hq + hq_idx) * o.NC + o.chunk) * o.srec;
     if (lane == 0) {
       __stcg(rec, m);
       __stcg(rec + 1, l);
     }
-    for (int j = lane; j < o.vdim; j += 32) __stcg(rec + 2 + j, val(j));
+    for (int j0 = 0; j0 < o.vdim; j0 += 32) {
+      const float v = val(j0 + lane);
+      if (j0 + lane < o.vdim) __stcg(rec + 2 + j0 + lane, v);
+    }
   }
 }
 
 // Merge of the chunks' records by the last arriver.  NC <= 32.
 template <int HYB>
-__device__ __forceinline__ void attn_merge(const Ctx &c, const TaskDesc &d, const AttnOut &o, int rows) {
+__device__ __noinline__ void attn_merge(const Ctx c, const TaskDesc &d, const AttnOut &o, int part, int row0, int row1) {
   typedef typename HybElt<HYB>::T T;
   const KernelParams &P = c.P;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   consumer_sync();
   if (threadIdx.x == 0) {
-    unsigned int *ticket = &P.attn_tickets[d.a[XA_TICKET]];
+    unsigned int *ticket = &P.attn_tickets[d.a[XA_TICKET] + part];
     unsigned int old;
     asm volatile("atom.acq_rel.gpu.global.add.u32 %0, [%1], 1;" : "=r"(old) : "l"(ticket) : "memory");
     const bool last = old + 1u == (unsigned)o.n_act;
@@ -341,57 +432,298 @@ __device__ __forceinline__ void attn_merge(const Ctx &c, const TaskDesc &d, cons
   }
   consumer_sync();
   if (c.s.flags[1] == 0) return;
-  for (int r = warp; r < rows; r += 8) {
+  // an item is 32 output columns of a row; its chunks' records are fetched sixteen at a time
+  const int cols = (o.vdim + 31) >> 5;
+  for (int item = warp + row0 * cols; item < row1 * cols; item += 8) {
+    const int r = item / cols, j = (item - r * cols) * 32 + lane;
     const int tok = o.q0 + r / o.G, hq_idx = o.head * o.G + r % o.G;
     const float *rec = P.attn_scratch + ((size_t)tok * o.hq + hq_idx) * o.NC * o.srec;
     const bool v = lane < o.n_act;
     const float m = v ? __ldcg(rec + (size_t)lane * o.srec) : -INFINITY;
     const float l = v ? __ldcg(rec + (size_t)lane * o.srec + 1) : 0.f;
+    float x[16], x2[16];
+#pragma unroll
+    for (int u = 0; u < 16; ++u) x[u] = (u < o.n_act && j < o.vdim) ? __ldcg(rec + (size_t)u * o.srec + 2 + j) : 0.f;
+    if (o.n_act > 16) {
+#pragma unroll
+      for (int u = 0; u < 16; ++u) x2[u] = (16 + u < o.n_act && j < o.vdim) ? __ldcg(rec + (size_t)(16 + u) * o.srec + 2 + j) : 0.f;
+    }
     float M = warp_max(m);
     if (o.sink) M = fmaxf(M, 0.f);
     const float w = m == -INFINITY ? 0.f : exp_dom<HYB>(m - M);
     const float L = warp_sum(l * w) + (o.sink ? exp_dom<HYB>(-M) : 0.f);
     const float f = L > 0.f ? o.oscale / L : 0.f;
-    T *out = reinterpret_cast<T *>(d.p[3]) + (size_t)tok * o.ldo + o.ocol + (size_t)hq_idx * o.vdim;
-    for (int j0 = 0; j0 < o.vdim; j0 += 32) {
-      const int j = j0 + lane;
-      float acc = 0.f;
-      for (int u = 0; u < o.n_act; ++u) {
-        const float wu = __shfl_sync(0xffffffffu, w, u);
-        if (j < o.vdim && wu > 0.f) acc = fmaf(wu, __ldcg(rec + (size_t)u * o.srec + 2 + j), acc);
-      }
-      if (j < o.vdim) store_elt(out + j, acc * f);
+    float acc = 0.f;
+#pragma unroll
+    for (int u = 0; u < 16; ++u) acc = fmaf(__shfl_sync(0xffffffffu, w, u), x[u], acc);
+    if (o.n_act > 16) {
+#pragma unroll
+      for (int u = 0; u < 16; ++u) acc = fmaf(__shfl_sync(0xffffffffu, w, 16 + u), x2[u], acc);
+    }
+    if (j < o.vdim)
+      store_elt(reinterpret_cast<T *>(d.p[3]) + (size_t)tok * o.ldo + o.ocol + (size_t)hq_idx * o.vdim + j, acc * f);
+  }
+}
+
+// What a warp's 16-row tile needs to know of its queries.
+struct AttnRows {
+  float scale, cap, cap2;
+  int kend;         // keys of the task
+  int p_lo, p_hi;   // last key this lane's two rows see
+  int p_all;        // keys up to here are seen by every row of the tile
+  bool two;         // rows 8 .. 15 of the tile hold queries
+};
+__device__ __forceinline__ AttnRows attn_rows(const TaskDesc &d, const SeqView &sv, int G, int first, int n, int kend) {
+  AttnRows w;
+  w.scale = __int_as_float(d.a[XA_SCALE]);
+  w.cap = __int_as_float(d.a[XA_CAP]);
+  w.cap2 = w.cap > 0.f ? 2.0f * 1.4426950408889634f / w.cap : 0.f;
+  w.kend = kend;
+  const int r = first + ((threadIdx.x & 31) >> 2);
+  w.p_lo = sv.pos0 + r / G;
+  w.p_hi = sv.pos0 + (r + 8) / G;
+  w.p_all = min(sv.pos0 + first / G, kend - 1);
+  w.two = n > 8;
+  return w;
+}
+// Eight keys (rows at kaddr / vaddr, this lane's ldmatrix addresses) against a 16-row query tile: scores, online softmax,
+// P V.  key0 is below w.kend.
+template <int D, int ON, bool TWO>
+__device__ __forceinline__ void attn_octet(const AttnRows &w, const uint32_t (&qf)[TWO ? 1 : D / 16][2], uint32_t qa, uint32_t kaddr,
+                                           uint32_t vaddr, int key0, float (&m_run)[2], float (&l_run)[2], float (&o)[ON / 8][4]) {
+  float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int kk = 0; kk < D / 32; ++kk) {
+    uint32_t b[4];
+    ldmatrix_x4(b, kaddr + kk * 64u);
+    if (!TWO) {
+      const uint32_t a0[4] = {qf[TWO ? 0 : 2 * kk][0], 0u, qf[TWO ? 0 : 2 * kk][1], 0u};
+      const uint32_t a1[4] = {qf[TWO ? 0 : 2 * kk + 1][0], 0u, qf[TWO ? 0 : 2 * kk + 1][1], 0u};
+      mma_bf16_16816(s, a0, b[0], b[1]);
+      mma_bf16_16816(s2, a1, b[2], b[3]);
+    } else {
+      uint32_t a0[4], a1[4];
+      ldmatrix_x4(a0, qa + kk * 64u);
+      ldmatrix_x4(a1, qa + kk * 64u + 32u);
+      mma_bf16_16816(s, a0, b[0], b[1]);
+      mma_bf16_16816(s2, a1, b[2], b[3]);
     }
   }
+  float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    if (e >= 2 && !(TWO && w.two)) { s[e] = -INFINITY; continue; }
+    s[e] = attn_score<HYB_BF16>(s[e] + s2[e], w.scale, w.cap, w.cap2);
+  }
+  if (key0 + 7 > w.p_all) {
+    const int key = key0 + 2 * (threadIdx.x & 3);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int kpos = key + (e & 1);
+      if (kpos >= w.kend || kpos > (e < 2 ? w.p_lo : w.p_hi)) s[e] = -INFINITY;
+    }
+  }
+  mx[0] = fmaxf(s[0], s[1]);
+  mx[1] = fmaxf(s[2], s[3]);
+  float ms[2], corr[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
+    mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
+    const float mn = fmaxf(m_run[i], mx[i]);
+    ms[i] = mn == -INFINITY ? 0.f : mn;
+    corr[i] = exp2f(m_run[i] - ms[i]);
+    m_run[i] = mn;
+  }
+  if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
+    l_run[0] *= corr[0];
+    l_run[1] *= corr[1];
+#pragma unroll
+    for (int i = 0; i < ON / 8; ++i) {
+      o[i][0] *= corr[0]; o[i][1] *= corr[0];
+      o[i][2] *= corr[1]; o[i][3] *= corr[1];
+    }
+  }
+  float p[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    p[e] = exp2f(s[e] - ms[e >> 1]);
+    l_run[e >> 1] += p[e];
+  }
+  const uint32_t h0 = pack_bf16(p[0], p[1]), h1 = pack_bf16(p[2], p[3]);
+  const uint32_t r0 = pack_bf16(p[0] - bf16_lo(h0), p[1] - bf16_hi(h0)), r1 = pack_bf16(p[2] - bf16_lo(h1), p[3] - bf16_hi(h1));
+  // value and remainder side by side in one k = 16 product: the V octet serves both halves
+  const uint32_t pa[4] = {h0, h1, r0, r1};
+#pragma unroll
+  for (int vq = 0; vq < ON / 32; ++vq) {
+    uint32_t b[4];
+    ldmatrix_x4_trans(b, vaddr + vq * 64u);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) mma_bf16_16816(o[4 * vq + i], pa, b[i], b[i]);
+  }
+}
+
+// Rows [first, first + nrow) from the records [split][row of `stride`] of (max, sum, D columns) in shared memory.
+template <int D>
+__device__ __forceinline__ void attn_emit_splits(const Ctx &c, const TaskDesc &d, const AttnOut &ao, const float *comb, int stride, int WK,
+                                                 int first, int nrow) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int r = warp; r < nrow; r += 8) {
+    const float *cr = comb + (size_t)r * (D + 2);
+    const size_t step = (size_t)stride * (D + 2);
+    // lane w holds split w's weight
+    const float mw = lane < WK ? cr[lane * step] : -INFINITY;
+    const float M = warp_max(mw);
+    const float wgt = mw == -INFINITY ? 0.f : exp2f(mw - M);
+    const float L = warp_sum(lane < WK ? cr[lane * step + 1] * wgt : 0.f);
+    attn_emit_row<HYB_BF16>(c, d, ao, first + r, M, L, [&](int j) {
+      float v = 0.f;
+      for (int w = 0; w < WK; ++w) v = fmaf(__shfl_sync(0xffffffffu, wgt, w), cr[w * step + 2 + min(j, D - 1)], v);
+      return v;
+    });
+  }
+}
+
+// One tile of query rows (decoding, or a task's share of a prompt portion): every warp streams its own octets of keys, w,
+// w + 8, ..., through its own ring -- no block barrier in the loop -- and the eight partial results are combined at the end.
+template <int D, bool TWO>
+__device__ __noinline__ void ext_attention_stream(const Ctx c, const TaskDesc &d, const SeqView sv, const AttnOut &ao, int k0, int k1,
+                                                  int row0, int nrow, int task) {
+  constexpr int PITCH = D * 2 + 16, STEP = 16 * PITCH, PIECES = D / 8, RSTEP = 32 / PIECES;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int nstg = d.a[XA_STAGES], page = d.a[XA_PAGE];
+  const int kend = min(k1, sv.pos0 + (row0 + nrow - 1) / ao.G + 1);
+  const int noct = kend > k0 ? (kend - k0 + 7) >> 3 : 0, mine = noct > warp ? (noct - warp + 7) >> 3 : 0;
+  uint8_t *qs = c.s.xtile;                                                      // [16][PITCH]
+  const uint32_t ring = smem_u32(qs) + (16 + warp * nstg * 16) * PITCH;         // this warp's stages: eight K rows, then eight V rows
+  // (everything below is live through the key loop: 32-bit offsets in units of 16 bytes)
+  const int piece = lane % PIECES, rl = lane / PIECES;
+  const uint32_t krow = d.a[XA_HKV] * (d.a[XA_DIMP] >> 3), vrow = d.a[XA_HKV] * (d.a[XA_VDIMP] >> 3);   // between positions
+  const bool kin = piece < (d.a[XA_DIMP] >> 3), vin = piece < (d.a[XA_VDIMP] >> 3);
+  const uint4 *kg = reinterpret_cast<const uint4 *>(d.p[1]) + ao.head * (d.a[XA_DIMP] >> 3) + piece + rl * krow;
+  const uint4 *vg = reinterpret_cast<const uint4 *>(d.p[2]) + ao.head * (d.a[XA_VDIMP] >> 3) + piece + rl * vrow;
+  const int32_t *pages = c.P.meta.paged_kv_indices + sv.kv0;
+  // page of the next octet to request, looked up one request ahead of its use
+  int pos = k0 + warp * 8;
+  int pid = pos < kend ? __ldcg(pages + pos / page) : 0;
+  auto issue = [&](int slot) {
+    if (pos < kend) {
+      const uint32_t row = (uint32_t)pid * page + pos % page;
+      const uint32_t dst = ring + slot * STEP + rl * PITCH + piece * 16;
+      const int left = kend - pos - rl;   // rows of this lane's stride that exist
+#pragma unroll
+      for (int i = 0; i < 8 / RSTEP; ++i) {
+        const uint32_t kd = dst + i * RSTEP * PITCH, vd = kd + 8 * PITCH;
+        const bool in = i * RSTEP < left;
+        if (in && kin) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(kd), "l"(kg + (size_t)((row + i * RSTEP) * krow)) : "memory");
+        else asm volatile("st.shared.v4.b32 [%0], {%1,%1,%1,%1};" ::"r"(kd), "r"(0) : "memory");
+        if (in && vin) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(vd), "l"(vg + (size_t)((row + i * RSTEP) * vrow)) : "memory");
+        else asm volatile("st.shared.v4.b32 [%0], {%1,%1,%1,%1};" ::"r"(vd), "r"(0) : "memory");
+      }
+      pos += 64;
+      pid = pos < kend ? __ldcg(pages + pos / page) : 0;
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  for (int i = 0; i < nstg - 1; ++i) issue(i);
+  {
+    const uint8_t *qg = reinterpret_cast<const uint8_t *>(d.p[0]);
+    const int G = ao.G, kp = d.a[XA_DIMP] >> 3;
+    for (int i = tid; i < 16 * PIECES; i += kConsumerThreads) {
+      const int r = i / PIECES, p = i % PIECES, row = row0 + r;
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (r < nrow && p < kp)
+        v = __ldcg(reinterpret_cast<const uint4 *>(qg + ((size_t)(sv.q0 + row / G) * d.a[XA_LDQ] + (size_t)(ao.head * G + row % G) * kp * 8) * 2) + p);
+      *reinterpret_cast<uint4 *>(qs + r * PITCH + p * 16) = v;
+    }
+  }
+  consumer_sync();
+  stamp(c, task, 0);
+  const AttnRows w = attn_rows(d, sv, ao.G, row0, nrow, kend);
+  const uint32_t qa = smem_u32(qs) + (uint32_t)((lane & 15) * PITCH + (lane >> 4) * 16);
+  uint32_t qf[TWO ? 1 : D / 16][2];   // rows 0 .. 7 only: two of a fragment's four registers
+  if (!TWO) {
+#pragma unroll
+    for (int kk = 0; kk < D / 16; ++kk)
+      ldmatrix_x2(qf[TWO ? 0 : kk], smem_u32(qs) + (uint32_t)((lane & 7) * PITCH + ((lane >> 3) & 1) * 16 + kk * 32));
+  }
+  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  float o[D / 8][4];
+#pragma unroll
+  for (int i = 0; i < D / 8; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
+  const uint32_t lane_off = (uint32_t)((lane & 7) * PITCH + (lane >> 3) * 16);
+  int slot = 0;
+#pragma unroll 1
+  for (int i = 0; i < mine; ++i) {
+    if (nstg >= 4) asm volatile("cp.async.wait_group 2;" ::: "memory");
+    else if (nstg == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
+    else asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncwarp();   // the octet has landed for every lane, and every lane is done with the slot refilled next
+    issue(slot == 0 ? nstg - 1 : slot - 1);
+    const uint32_t ka = ring + slot * STEP + lane_off;
+    attn_octet<D, D, TWO>(w, qf, qa, ka, ka + 8 * PITCH, k0 + (warp + 8 * i) * 8, m_run, l_run, o);
+    if (++slot == nstg) slot = 0;
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  consumer_sync();   // the rings become the combine area
+  stamp(c, task, 2);
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    l_run[i] += __shfl_xor_sync(0xffffffffu, l_run[i], 1);
+    l_run[i] += __shfl_xor_sync(0xffffffffu, l_run[i], 2);
+  }
+  float *comb = reinterpret_cast<float *>(qs + 16 * PITCH);   // [8 warps][16 rows][D + 2]
+  float *c0 = comb + (size_t)(warp * 16 + (lane >> 2)) * (D + 2), *c1 = c0 + 8 * (D + 2);
+  if ((lane & 3) == 0) {
+    c0[0] = m_run[0]; c0[1] = l_run[0];
+    c1[0] = m_run[1]; c1[1] = l_run[1];
+  }
+#pragma unroll
+  for (int i = 0; i < D / 8; ++i) {
+    const int col = 2 + i * 8 + 2 * (lane & 3);
+    *reinterpret_cast<float2 *>(c0 + col) = make_float2(o[i][0], o[i][1]);
+    if (w.two) *reinterpret_cast<float2 *>(c1 + col) = make_float2(o[i][2], o[i][3]);
+  }
+  consumer_sync();
+  attn_emit_splits<D>(c, d, ao, comb, 16, 8, row0, nrow);
 }
 
 // bf16: QK^T and PV on mma.sync.  Head sizes are padded to D columns in shared memory.  The eight warps are split over
 // row tiles (16 rows), key octets and, for D = 256, halves of the output columns; the key split is combined in shared
 // memory.  The probabilities enter PV as a bf16 value and a bf16 remainder, so that the weights keep 16 bits.
 template <int D>
-__device__ __forceinline__ void ext_attention_mma(const Ctx &c, const TaskDesc &d, const SeqView &sv, const AttnOut &ao, int k0, int k1,
-                                                  int rows) {
+__device__ __noinline__ void ext_attention_mma(const Ctx c, const TaskDesc &d, const SeqView sv, const AttnOut &ao, int k0, int k1,
+                                                  int row0, int rows, int task) {
   constexpr int ON = D < 128 ? D : 128, WN = D / ON, KEYS = D > 128 ? 32 : 64, NSUB = KEYS / 8, PITCH = D * 2 + 16;
   constexpr int WMAX = 8 / WN, MROWS = WMAX * 16, TILE = KEYS * PITCH;
   const KernelParams &P = c.P;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int G = ao.G, hkv = d.a[XA_HKV], dimp = d.a[XA_DIMP], vdimp = d.a[XA_VDIMP], page = d.a[XA_PAGE];
-  const float scale = __int_as_float(d.a[XA_SCALE]), cap = __int_as_float(d.a[XA_CAP]);
-  const float cap2 = cap > 0.f ? 2.0f * 1.4426950408889634f / cap : 0.f;
-  const int RB = min(MROWS, ext_attention_rows(P.max_num_batched_tokens * G));
+  const int RB = min(MROWS, ext_attention_rows(P.max_num_batched_tokens * G));   // rows of a block (all of them in small graphs)
   uint8_t *qs = c.s.xtile;                // [RB][PITCH]
-  uint8_t *st = qs + RB * PITCH;          // two stages of K rows, V rows
+  uint8_t *st = qs + RB * PITCH;          // ring of stages, each KEYS K rows, then KEYS V rows
+  const int nstg = d.a[XA_STAGES];
+  int *cells = reinterpret_cast<int *>(st + nstg * 2 * TILE);   // [kXaCells] cache row (page * page size + offset) of every eighth key
   const uint8_t *qg = reinterpret_cast<const uint8_t *>(d.p[0]);
   const uint8_t *kg = reinterpret_cast<const uint8_t *>(d.p[1]), *vg = reinterpret_cast<const uint8_t *>(d.p[2]);
   const int kp = dimp >> 3, vp = vdimp >> 3;   // 16-byte pieces of a row
+  // eight consecutive keys lie in one page when pages hold a multiple of eight positions
+  const int ncell = (page & 7) == 0 && k1 - k0 <= 8 * kXaCells ? (k1 - k0 + 7) >> 3 : 0;
+  auto cell_row = [&](int key) {
+    const int pg = key / page;
+    return __ldcg(&P.meta.paged_kv_indices[sv.kv0 + pg]) * page + (key - pg * page);
+  };
+  for (int i = tid; i < ncell; i += kConsumerThreads) cells[i] = cell_row(k0 + 8 * i);
 
-  for (int rb = 0; rb < rows; rb += RB) {
+  for (int rb = row0; rb < rows; rb += RB) {
     const int nrow = min(RB, rows - rb), mt = (nrow + 15) >> 4;
     const int WM = mt <= 1 ? 1 : (mt <= 2 ? 2 : (mt <= 4 ? 4 : WMAX));
     const int WK = WMAX / WM;                                      // <= NSUB
     const int wn = warp % WN, w2 = warp / WN, wm = w2 % WM, wk = w2 / WM;
     const int kend = min(k1, sv.pos0 + (rb + nrow - 1) / G + 1);   // keys past the last row's position are not needed
-    if (rb > 0) consumer_sync();
+    if (rb > row0) consumer_sync();
     for (int i = tid; i < WM * 16 * (D / 8); i += kConsumerThreads) {
       const int r = i / (D / 8), p = i - r * (D / 8);
       uint4 v = make_uint4(0, 0, 0, 0);
@@ -401,16 +733,18 @@ __device__ __forceinline__ void ext_attention_mma(const Ctx &c, const TaskDesc &
       }
       *reinterpret_cast<uint4 *>(qs + r * PITCH + p * 16) = v;
     }
-    auto issue = [&](int base, int stage) {
-      for (int i = tid; i < KEYS * (D / 8); i += kConsumerThreads) {
-        const int r = i / (D / 8), p = i - r * (D / 8), key = base + r;
-        uint8_t *kd = st + stage * 2 * TILE + r * PITCH + p * 16, *vd = kd + TILE;
+    auto issue = [&](int it, int stg) {
+      const int base = k0 + it * KEYS;
+      const int p = tid % (D / 8);
+      uint8_t *dst = st + stg * 2 * TILE + (tid / (D / 8)) * PITCH + p * 16;
+      constexpr int STEP = kConsumerThreads / (D / 8);   // rows of a pass
+#pragma unroll
+      for (int pass = 0; pass < KEYS / STEP; ++pass) {
+        const int key = base + pass * STEP + tid / (D / 8);
+        uint8_t *kd = dst + pass * STEP * PITCH, *vd = kd + TILE;
         const bool in = key < kend;
         size_t cell = 0;
-        if (in) {
-          const int pg = key / page;
-          cell = ((size_t)__ldcg(&P.meta.paged_kv_indices[sv.kv0 + pg]) * page + (key - pg * page)) * hkv + ao.head;
-        }
+        if (in) cell = (size_t)(ncell > 0 ? cells[(key - k0) >> 3] + ((key - k0) & 7) : cell_row(key)) * hkv + ao.head;
         // pieces outside the row or past the last key are zeros: a masked key has weight 0, and 0 x NaN would be NaN
         if (in && p < kp) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(kd)), "l"(kg + (cell * kp + p) * 16) : "memory");
         else *reinterpret_cast<uint4 *>(kd) = make_uint4(0, 0, 0, 0);
@@ -425,98 +759,41 @@ __device__ __forceinline__ void ext_attention_mma(const Ctx &c, const TaskDesc &
     for (int i = 0; i < ON / 8; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
-    const int r_lo = rb + wm * 16 + (lane >> 2);
-    const int p_lo = sv.pos0 + r_lo / G, p_hi = sv.pos0 + (r_lo + 8) / G;   // last key each row sees
+    const AttnRows w = attn_rows(d, sv, G, rb + wm * 16, nrow - wm * 16, kend);
     const int ntiles = kend > k0 ? (kend - k0 + KEYS - 1) / KEYS : 0;
-    if (ntiles > 0) issue(k0, 0);
-    for (int it = 0; it < ntiles; ++it) {
-      if (it + 1 < ntiles) issue(k0 + (it + 1) * KEYS, (it + 1) & 1);
-      if (it + 1 < ntiles) asm volatile("cp.async.wait_group 1;" ::: "memory");
-      else asm volatile("cp.async.wait_group 0;" ::: "memory");
-      consumer_sync();
-      const int base = k0 + it * KEYS;
-      const uint32_t kt = smem_u32(st + (it & 1) * 2 * TILE), vt = kt + TILE;
-      if (wm < mt) {
-        float s[NSUB][4];
-#pragma unroll
-        for (int j = 0; j < NSUB; ++j)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
-        const uint32_t qa = smem_u32(qs) + (uint32_t)((wm * 16 + (lane & 15)) * PITCH + (lane >> 4) * 16);
-#pragma unroll
-        for (int kk = 0; kk < D / 32; ++kk) {
-          uint32_t a0[4], a1[4];
-          ldmatrix_x4(a0, qa + kk * 64u);
-          ldmatrix_x4(a1, qa + kk * 64u + 32u);
-#pragma unroll
-          for (int j = 0; j < NSUB; ++j) {
-            if ((j & (WK - 1)) == wk) {
-              uint32_t b[4];
-              ldmatrix_x4(b, kt + (uint32_t)((j * 8 + (lane & 7)) * PITCH + (lane >> 3) * 16) + kk * 64u);
-              mma_bf16_16816(s[j], a0, b[0], b[1]);
-              mma_bf16_16816(s[j], a1, b[2], b[3]);
-            }
-          }
-        }
-        float mx[2] = {-INFINITY, -INFINITY};
-#pragma unroll
-        for (int j = 0; j < NSUB; ++j) {
-          if ((j & (WK - 1)) == wk) {
-            const int key = base + j * 8 + 2 * (lane & 3);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              const int kpos = key + (e & 1);
-              const bool ok = kpos < kend && kpos <= (e < 2 ? p_lo : p_hi);
-              s[j][e] = ok ? attn_score<HYB_BF16>(s[j][e], scale, cap, cap2) : -INFINITY;
-              mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
-            }
-          }
-        }
-        float corr[2], ms[2];
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
-          mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
-          const float mn = fmaxf(m_run[i], mx[i]);
-          ms[i] = mn == -INFINITY ? 0.f : mn;
-          corr[i] = exp2f(m_run[i] - ms[i]);
-          m_run[i] = mn;
-          l_run[i] *= corr[i];
-        }
-        if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
-#pragma unroll
-          for (int i = 0; i < ON / 8; ++i) {
-            o[i][0] *= corr[0]; o[i][1] *= corr[0];
-            o[i][2] *= corr[1]; o[i][3] *= corr[1];
-          }
-        }
-#pragma unroll
-        for (int j = 0; j < NSUB; ++j) {
-          if ((j & (WK - 1)) == wk) {
-            float p[4];
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              p[e] = exp2f(s[j][e] - ms[e >> 1]);
-              l_run[e >> 1] += p[e];
-            }
-            const uint32_t h0 = pack_bf16(p[0], p[1]), h1 = pack_bf16(p[2], p[3]);
-            const uint32_t r0 = pack_bf16(p[0] - bf16_lo(h0), p[1] - bf16_hi(h0)), r1 = pack_bf16(p[2] - bf16_lo(h1), p[3] - bf16_hi(h1));
-            const uint32_t va = vt + (uint32_t)((j * 8 + (lane & 7)) * PITCH + (lane >> 3) * 16 + wn * ON * 2);
-#pragma unroll
-            for (int vq = 0; vq < ON / 32; ++vq) {
-              uint32_t b[4];
-              ldmatrix_x4_trans(b, va + vq * 64u);
-#pragma unroll
-              for (int i = 0; i < 4; ++i) {
-                mma_bf16_1688(o[4 * vq + i], h0, h1, b[i]);
-                mma_bf16_1688(o[4 * vq + i], r0, r1, b[i]);
-              }
-            }
-          }
-        }
-      }
-      consumer_sync();   // the stage is refilled by the next trip
+    consumer_sync();   // queries and cells
+    stamp(c, task, 0);
+    // nstg - 1 tiles in flight; one commit per trip, empty past the last tile, so that the wait counts trips
+    for (int i = 0; i < nstg - 1; ++i) {
+      if (i < ntiles) issue(i, i);
+      else asm volatile("cp.async.commit_group;" ::: "memory");
     }
+    const uint32_t qa = smem_u32(qs) + (uint32_t)((wm * 16 + (lane & 15)) * PITCH + (lane >> 4) * 16);
+    const uint32_t qf[1][2] = {{0u, 0u}};   // (the fragments come from shared memory)
+    const uint32_t lane_off = (uint32_t)((lane & 7) * PITCH + (lane >> 3) * 16);
+    int stg = 0;
+    for (int it = 0; it < ntiles; ++it) {
+      if (nstg >= 4) asm volatile("cp.async.wait_group 2;" ::: "memory");
+      else if (nstg == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
+      else asm volatile("cp.async.wait_group 0;" ::: "memory");
+      consumer_sync();   // tile `it` has landed for everyone, and everyone is done with the stage refilled next
+      if (it == 0) stamp(c, task, 1);
+      if (it + nstg - 1 < ntiles) issue(it + nstg - 1, stg == 0 ? nstg - 1 : stg - 1);
+      else asm volatile("cp.async.commit_group;" ::: "memory");
+      const int base = k0 + it * KEYS;
+      const uint32_t kt = smem_u32(st + stg * 2 * TILE) + lane_off, vt = kt + TILE + wn * ON * 2;
+      if (++stg == nstg) stg = 0;
+      if (wm >= mt) continue;
+      // this warp's octets of keys, one at a time
+#pragma unroll 1
+      for (int j = wk; j < NSUB; j += WK) {
+        const int key0 = base + j * 8;
+        if (key0 >= kend) break;
+        attn_octet<D, ON, true>(w, qf, qa, kt + (uint32_t)(j * 8 * PITCH), vt + (uint32_t)(j * 8 * PITCH), key0, m_run, l_run, o);
+      }
+    }
+    consumer_sync();   // the stages become the combine area
+    stamp(c, task, 2);
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       l_run[i] += __shfl_xor_sync(0xffffffffu, l_run[i], 1);
@@ -535,40 +812,17 @@ __device__ __forceinline__ void ext_attention_mma(const Ctx &c, const TaskDesc &
       for (int i = 0; i < ON / 8; ++i) {
         const int col = 2 + wn * ON + i * 8 + 2 * (lane & 3);
         *reinterpret_cast<float2 *>(c0 + col) = make_float2(o[i][0], o[i][1]);
-        *reinterpret_cast<float2 *>(c1 + col) = make_float2(o[i][2], o[i][3]);
+        if (w.two) *reinterpret_cast<float2 *>(c1 + col) = make_float2(o[i][2], o[i][3]);
       }
     }
     consumer_sync();
-    for (int r = warp; r < nrow; r += 8) {
-      const float *cr = comb + (size_t)r * (D + 2);
-      const size_t step = (size_t)WM * 16 * (D + 2);
-      float M = -INFINITY, L = 0.f, wgt[8];
-#pragma unroll
-      for (int w = 0; w < 8; ++w)
-        if (w < WK) M = fmaxf(M, cr[w * step]);
-#pragma unroll
-      for (int w = 0; w < 8; ++w) {
-        wgt[w] = 0.f;
-        if (w < WK) {
-          const float mw = cr[w * step];
-          wgt[w] = mw == -INFINITY ? 0.f : exp2f(mw - M);
-          L += cr[w * step + 1] * wgt[w];
-        }
-      }
-      attn_emit_row<HYB_BF16>(c, d, ao, rb + r, M, L, [&](int j) {
-        float v = 0.f;
-#pragma unroll
-        for (int w = 0; w < 8; ++w)
-          if (w < WK) v += wgt[w] * cr[w * step + 2 + j];
-        return v;
-      });
-    }
+    attn_emit_splits<D>(c, d, ao, comb, WM * 16, WK, rb, nrow);
   }
 }
 
 // 32-bit: one warp per row, 32 keys at a time (a lane per key for the scores, a lane per output column for PV)
-__device__ __forceinline__ void ext_attention_f32(const Ctx &c, const TaskDesc &d, const SeqView &sv, const AttnOut &ao, int k0, int k1,
-                                                  int rows) {
+__device__ __noinline__ void ext_attention_f32(const Ctx c, const TaskDesc &d, const SeqView sv, const AttnOut &ao, int k0, int k1,
+                                                  int row0, int rows) {
   constexpr int NO = 16;   // output columns per lane: value sizes up to 512
   const KernelParams &P = c.P;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -581,7 +835,7 @@ __device__ __forceinline__ void ext_attention_f32(const Ctx &c, const TaskDesc &
     const int pg = key / page;
     return ((size_t)__ldcg(&P.meta.paged_kv_indices[sv.kv0 + pg]) * page + (key - pg * page)) * hkv + ao.head;
   };
-  for (int r = warp; r < rows; r += 8) {
+  for (int r = row0 + warp; r < rows; r += 8) {
     const int kend = min(k1, sv.pos0 + r / G + 1);
     __syncwarp();
     for (int i = lane; i < dimp; i += 32) q[i] = __ldcg(qg + (size_t)(sv.q0 + r / G) * d.a[XA_LDQ] + (size_t)(ao.head * G + r % G) * dimp + i);
@@ -629,48 +883,125 @@ __device__ __forceinline__ void ext_attention_f32(const Ctx &c, const TaskDesc &
 }
 
 template <int HYB>
-__device__ __forceinline__ void run_ext_attention(const Ctx &c, const TaskDesc &d) {
+__device__ __forceinline__ void run_ext_attention(const Ctx &c, const TaskDesc &d, int task) {
   const SeqView sv = seq_view(c.P, d.a[XA_SLOT]);
   if (sv.nq <= 0) return;
-  AttnOut ao;
+  // shared by the block, in shared memory: in registers it would be live through the key loops (every thread writes the
+  // same values, and the previous task is done with it)
+  AttnOut &ao = *reinterpret_cast<AttnOut *>(c.s.red);
   ao.hq = d.a[XA_HQ];
   ao.G = ao.hq / d.a[XA_HKV];
   ao.head = d.a[XA_HEAD];
   ao.q0 = sv.q0;
   ao.NC = d.a[XA_NCHUNK];
-  ao.chunk = d.a[XA_CHUNK];
   ao.vdim = d.a[XA_VDIM];
   ao.ldo = d.a[XA_LDO];
   ao.ocol = d.a[XA_OCOL];
   ao.srec = d.a[XA_SREC];
   ao.oscale = __int_as_float(d.a[XA_OSCALE]);
   ao.sink = d.a[XA_SINK] != 0;
-  const int len = sv.pos0 + sv.nq, rows = sv.nq * ao.G;
-  const int per = max(128, ((len + ao.NC - 1) / ao.NC + 63) & ~63);   // keys of a chunk
+  // The NC tasks of a (request, kv head) are split over the 16-row query tiles first and over the keys with what is left:
+  // a prompt portion has rows enough and needs no merge, a decoded token has one tile and all its tasks share the keys.
+  const int len = sv.pos0 + sv.nq, rows = sv.nq * ao.G, tiles = (rows + 15) >> 4;
+  const int parts = min(ao.NC, tiles), ksplit = ao.NC / parts;
+  const int part = d.a[XA_CHUNK] % parts;
+  ao.chunk = d.a[XA_CHUNK] / parts;
+  const int per = max(64, ((len + ksplit - 1) / ksplit + 63) & ~63);   // keys of a chunk
   ao.n_act = (len + per - 1) / per;
-  if (ao.chunk >= ao.n_act) return;
+  if (ao.chunk >= ao.n_act) return;   // (n_act <= ksplit: this also ends the tasks beyond parts * ksplit)
   const int k0 = ao.chunk * per, k1 = min(len, k0 + per);
+  const int row0 = tiles * part / parts * 16, row1 = min(rows, tiles * (part + 1) / parts * 16);
   if (HYB == HYB_F32) {
-    ext_attention_f32(c, d, sv, ao, k0, k1, rows);
+    ext_attention_f32(c, d, sv, ao, k0, k1, row0, row1);
   } else {
     const int w = max(d.a[XA_DIMP], d.a[XA_VDIMP]);
-    if (w <= 64) ext_attention_mma<64>(c, d, sv, ao, k0, k1, rows);
-    else if (w <= 128) ext_attention_mma<128>(c, d, sv, ao, k0, k1, rows);
-    else ext_attention_mma<256>(c, d, sv, ao, k0, k1, rows);
+    const bool one = row1 - row0 <= 16 && (d.a[XA_PAGE] & 7) == 0;
+    if (w <= 64) {
+      if (one && row1 - row0 <= 8) ext_attention_stream<64, false>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
+      else if (one) ext_attention_stream<64, true>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
+      else ext_attention_mma<64>(c, d, sv, ao, k0, k1, row0, row1, task);
+    } else if (w <= 128) {
+      if (one && row1 - row0 <= 8) ext_attention_stream<128, false>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
+      else if (one) ext_attention_stream<128, true>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
+      else ext_attention_mma<128>(c, d, sv, ao, k0, k1, row0, row1, task);
+    } else {
+      ext_attention_mma<256>(c, d, sv, ao, k0, k1, row0, row1, task);
+    }
   }
-  if (ao.n_act > 1) attn_merge<HYB>(c, d, ao, rows);
+  stamp(c, task, 3);
+  if (ao.n_act > 1) attn_merge<HYB>(c, d, ao, part, row0, row1);
 }
 
 // ---------------------------------------------------------------------------
 // TASK_SHORT_CONV: out[t][ch] = bias[ch] + sum_j taps[ch][j] in[t - (taps - 1) + j][ch], inputs before the portion come
 // from the carried state (zeros before the sequence).  A task owns a channel range of every request.
 // ---------------------------------------------------------------------------
-__device__ __forceinline__ void run_short_conv(const Ctx &c, const TaskDesc &d) {
+// Up to kConvWindow + 1 taps: a warp takes 32 channels and a run of up to eight consecutive tokens, with every input it
+// needs (the tokens of its run, the ones before them, carried ones where a request starts) in registers before anything
+// is stored.
+constexpr int kConvWindow = 4;
+__device__ __forceinline__ void short_conv_window(const Ctx &c, const TaskDesc &d, const TokenRec *rec, int B) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int C = d.a[2], taps = d.a[3], hist = taps - 1;
+  const float *in = reinterpret_cast<const float *>(d.p[0]) + d.a[5];
+  float *state = reinterpret_cast<float *>(d.p[4]);
+  float *out = reinterpret_cast<float *>(d.p[5]);
+  const int per = (B + 7) >> 3, t0 = warp * per, n = max(0, min(per, B - t0));
+  for (int cb = d.a[0]; cb < d.a[1]; cb += 32) {
+    const int ch = cb + lane;
+    const bool ok = ch < d.a[1];
+    float x[8 + kConvWindow], w[kConvWindow + 1];
+    float prev[8][kConvWindow];   // prev[u][j]: the input j + 1 tokens before token t0 + u
+    const float ib = (ok && d.p[1]) ? bf16_at(d.p[1], ch) : 0.f, ob = (ok && d.p[3]) ? bf16_at(d.p[3], ch) : 0.f;
+#pragma unroll
+    for (int j = 0; j <= kConvWindow; ++j) w[j] = (ok && j <= hist) ? bf16_at(d.p[2], (size_t)ch * taps + hist - j) : 0.f;
+#pragma unroll
+    for (int i = 0; i < 8 + kConvWindow; ++i) {   // x[i]: batch token t0 - kConvWindow + i
+      const int t = t0 - kConvWindow + i;
+      x[i] = (ok && t >= 0 && i < n + kConvWindow) ? __ldcg(in + (size_t)t * d.a[4] + ch) + ib : 0.f;
+    }
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+      const int t = t0 + u;
+      const TokenRec r = rec[u < n ? t : 0];
+#pragma unroll
+      for (int j = 0; j < kConvWindow; ++j) {
+        const int src = t - 1 - j;
+        prev[u][j] = src >= r.q0 ? x[kConvWindow + u - 1 - j] : 0.f;
+        if (ok && u < n && j < hist && src < r.q0 && !(r.flags & 4))
+          prev[u][j] = __ldcg(state + ((size_t)r.slot * hist + (hist + src - r.q0)) * C + ch);
+      }
+    }
+    consumer_sync();   // all carried inputs have been read
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+      if (!ok || u >= n) continue;
+      const TokenRec r = rec[t0 + u];
+      const float cur = x[kConvWindow + u];
+      float v = fmaf(w[0], cur, ob);
+#pragma unroll
+      for (int j = 0; j < kConvWindow; ++j) v = fmaf(w[j + 1], prev[u][j], v);
+      if (d.a[7] == 1) v = v * sigmoid_f(v);
+      out[(size_t)(t0 + u) * d.a[6] + ch] = v;
+      if (r.flags & 2) {   // the last `hist` inputs, oldest first
+#pragma unroll
+        for (int j = 0; j < kConvWindow; ++j)
+          if (j < hist) state[((size_t)r.slot * hist + hist - 1 - j) * C + ch] = j == 0 ? cur : prev[u][j - 1];
+      }
+    }
+  }
+}
+
+__device__ __noinline__ void run_short_conv(const Ctx c, const TaskDesc &d) {
   const KernelParams &P = c.P;
   const int B = active_tokens(P);
   if (B <= 0) return;
   TokenRec *rec = reinterpret_cast<TokenRec *>(c.s.xtile);
   token_map(P, B, rec, reinterpret_cast<int *>(c.s.xtile + kTokenMapBytes));
+  if (d.a[3] <= kConvWindow + 1) {
+    short_conv_window(c, d, rec, B);
+    return;
+  }
   const int c0 = d.a[0], nc = d.a[1] - c0, C = d.a[2], taps = d.a[3], hist = taps - 1;
   const float *in = reinterpret_cast<const float *>(d.p[0]) + d.a[5];
   float *state = reinterpret_cast<float *>(d.p[4]);
@@ -705,7 +1036,7 @@ __device__ __forceinline__ void run_short_conv(const Ctx &c, const TaskDesc &d) 
 // TASK_RGLRU: channels [c0, c1) of one block of the block-diagonal gates, all requests.
 //   r = sigmoid(Ra u + ra), i = sigmoid(Ri u + ri), log a = -c r softplus(lambda), S = a S + sqrt(1 - a^2) i u,
 //   out = scale * S * gelu_tanh(y)
-// Gate products in 32-bit: a warp takes two channels (four weight rows) and eight tokens at a time.
+// Gate products, plain form: a warp takes two channels (four weight rows) and eight tokens at a time.
 // ---------------------------------------------------------------------------
 template <int HYB, bool PAIR>
 __device__ __forceinline__ void rglru_gates(const TaskDesc &d, const float *us, float *rs, float *is, int nt) {
@@ -756,42 +1087,162 @@ __device__ __forceinline__ void rglru_gates(const TaskDesc &d, const float *us, 
   }
 }
 
+// The gate products on the tensor cores without losing 32-bit precision: the weights are bf16 as they are, u is the exact
+// sum of three bf16 numbers, so three products with float32 accumulation give u's full mantissa.  A unit is (16 rows of one
+// gate matrix, half of the columns); `af` holds the first unit's first kGateSteps weight fragments, loaded before the tokens
+// were known.
+constexpr int kGateSteps = 8;
+struct GateUnit {
+  uint64_t w;        // gate matrix
+  int ch, k0, k1;    // first channel of the 16 (relative to the task), column range
+  int mat;
+};
+__device__ __forceinline__ GateUnit gate_unit(const TaskDesc &d, int u) {
+  const int bs = d.a[GL_BS], half = ((bs + 31) >> 5) << 4;
+  GateUnit g;
+  g.mat = (u >> 1) & 1;
+  g.w = d.p[g.mat ? 5 : 3];
+  g.ch = (u >> 2) * 16;
+  g.k0 = (u & 1) ? half : 0;
+  g.k1 = (u & 1) ? bs : min(half, bs);
+  return g;
+}
+__device__ __forceinline__ void gate_fragment(const TaskDesc &d, const GateUnit &g, int k, uint32_t (&a)[4]) {
+  const int lane = threadIdx.x & 31, bs = d.a[GL_BS], c0 = d.a[GL_C0], C = d.a[GL_C1] - c0;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {   // rows g, g + 8; columns 2 q, 2 q + 8
+    const int ch = g.ch + (lane >> 2) + (i & 1) * 8, col = k + 2 * (lane & 3) + (i >> 1) * 8;
+    a[i] = (ch < C && col < g.k1) ? __ldg(reinterpret_cast<const uint32_t *>(g.w + 2 * (((size_t)d.a[GL_BLOCK] * bs + c0 + ch) * bs + col))) : 0u;
+  }
+}
+// us: [3][TG][pitch] bf16 (columns past bs are zeros); part: [half][matrix][TG][C] sums.
+__device__ __forceinline__ void rglru_gates_mma(const TaskDesc &d, const __nv_bfloat16 *us, int pitch, float *part, int nt,
+                                                uint32_t (&af)[kGateSteps][4], bool have) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int C = d.a[GL_C1] - d.a[GL_C0], TG = d.a[GL_TG], units = ((C + 15) >> 4) * 4;
+  for (int u = warp; u < units; u += 8) {
+    const GateUnit g = gate_unit(d, u);
+    for (int n0 = 0; n0 < nt; n0 += 32) {
+      float acc[4][4];
+#pragma unroll
+      for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
+      for (int kb = g.k0; kb < g.k1; kb += 16 * kGateSteps) {
+        if (!have) {
+#pragma unroll
+          for (int st = 0; st < kGateSteps; ++st) gate_fragment(d, g, kb + 16 * st, af[st]);
+        }
+        have = false;
+#pragma unroll
+        for (int st = 0; st < kGateSteps; ++st) {
+          const int k = kb + 16 * st;
+          if (k >= g.k1) break;
+#pragma unroll
+          for (int n = 0; n < 4; ++n) {
+            if (n0 + n * 8 >= nt) break;
+            const __nv_bfloat16 *x = us + (size_t)(n0 + n * 8 + (lane >> 2)) * pitch + k + 2 * (lane & 3);
+#pragma unroll
+            for (int h = 0; h < 3; ++h) {
+              const uint32_t *xp = reinterpret_cast<const uint32_t *>(x + (size_t)h * TG * pitch);
+              mma_bf16_16816(acc[n], af[st], xp[0], xp[4]);
+            }
+          }
+        }
+      }
+      float *out = part + (size_t)((u & 1) * 2 + g.mat) * TG * C;
+#pragma unroll
+      for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int t = n0 + n * 8 + 2 * (lane & 3) + (e & 1), ch = g.ch + (lane >> 2) + (e >> 1) * 8;
+          if (t < nt && ch < C) out[(size_t)t * C + ch] = acc[n][e];
+        }
+    }
+  }
+}
+
 template <int HYB>
-__device__ __forceinline__ void run_rglru(const Ctx &c, const TaskDesc &d) {
+__device__ __noinline__ void run_rglru(const Ctx c, const TaskDesc &d) {
   typedef typename HybElt<HYB>::T T;
   const KernelParams &P = c.P;
   const int B = active_tokens(P);
   if (B <= 0) return;
-  const int tid = threadIdx.x;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int bs = d.a[GL_BS], c0 = d.a[GL_C0], C = d.a[GL_C1] - c0, TG = d.a[GL_TG], blk = d.a[GL_BLOCK], width = d.a[GL_WIDTH];
+  const bool mma = HYB == HYB_BF16 && (bs & 1) == 0;
+  const int gch = blk * bs + c0;   // first channel of this task
+  uint32_t af[kGateSteps][4];
+  if (mma && warp < ((C + 15) >> 4) * 4) {
+    const GateUnit g = gate_unit(d, warp);
+#pragma unroll
+    for (int st = 0; st < kGateSteps; ++st) gate_fragment(d, g, g.k0 + 16 * st, af[st]);
+  }
   float *state = *reinterpret_cast<float *const *>(&d.a[GL_STATE]);
   T *outp = *reinterpret_cast<T *const *>(&d.a[GL_OUT]);
   const float oscale = __int_as_float(d.a[GL_OSCALE]), gate_c = __int_as_float(d.a[GL_GATE_C]);
   TokenRec *rec = reinterpret_cast<TokenRec *>(c.s.xtile);
-  float *us = reinterpret_cast<float *>(c.s.xtile + kTokenMapBytes);   // [TG][bs]
-  float *rs = us + (size_t)TG * bs;                                     // [TG][C]  gate r, then a
-  float *is = rs + (size_t)TG * C;                                      // [TG][C]  gate i, then b, then S
+  float *chp = reinterpret_cast<float *>(c.s.xtile + kTokenMapBytes);   // [4][64] per channel: gate biases, decay * softplus(lambda), y bias
+  float *part = chp + 256;                                              // [half][matrix][TG][C]; [0][0] then holds a, [0][1] b and then S
+  float *us = part + 4 * (size_t)TG * C;                                // [TG][bs], or three bf16 parts [3][TG][pitch]
+  const int pitch = ((bs + 15) & ~15) + 8;
+  __nv_bfloat16 *uh = reinterpret_cast<__nv_bfloat16 *>(us);
+  if (tid < C) {
+    chp[tid] = bf16_at(d.p[4], gch + tid);
+    chp[64 + tid] = bf16_at(d.p[6], gch + tid);
+    chp[128 + tid] = gate_c * softplus_f(bf16_at(d.p[7], gch + tid));
+    chp[192 + tid] = bf16_at(d.p[2], gch + tid);
+  }
   token_map(P, B, rec, reinterpret_cast<int *>(us));
-  const int gch = blk * bs + c0;   // first channel of this task
+  float *rs = part, *is = part + (size_t)TG * C;
   float carry = 0.f;               // state of channel tid between token groups
   for (int tb = 0; tb < B; tb += TG) {
     const int nt = min(TG, B - tb);
-    for (int i = tid; i < nt * bs; i += kConsumerThreads) {
-      const int t = i / bs, k = i - t * bs;
-      us[i] = __ldcg(reinterpret_cast<const float *>(d.p[0]) + (size_t)(tb + t) * d.a[GL_LDU] + (size_t)blk * bs + k);
+    const float *ug = reinterpret_cast<const float *>(d.p[0]) + (size_t)tb * d.a[GL_LDU] + (size_t)blk * bs;
+    const float *yg = reinterpret_cast<const float *>(d.p[1]) + (size_t)tb * d.a[GL_LDP] + d.a[GL_YOFF] + gch;
+    for (int t = warp; t < nt; t += 8) {
+#pragma unroll 8
+      for (int k = lane; k < (mma ? pitch - 8 : bs); k += 32) {
+        const float v = k < bs ? __ldcg(ug + (size_t)t * d.a[GL_LDU] + k) : 0.f;
+        if (mma) {
+          const __nv_bfloat16 h = __float2bfloat16_rn(v);
+          const float r1 = v - bf16_to_f(h);
+          const __nv_bfloat16 m = __float2bfloat16_rn(r1);
+          uh[(size_t)t * pitch + k] = h;
+          uh[(size_t)(TG + t) * pitch + k] = m;
+          uh[(size_t)(2 * TG + t) * pitch + k] = __float2bfloat16_rn(r1 - bf16_to_f(m));
+        } else {
+          us[(size_t)t * bs + k] = v;
+        }
+      }
+    }
+    // the elementwise inputs of this thread's first items travel while the gates are formed
+    float y0[4], u0[4];
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const int i = tid + q * kConsumerThreads, t = i / C, ch = i - t * C;
+      y0[q] = i < nt * C ? __ldcg(yg + (size_t)t * d.a[GL_LDP] + ch) : 0.f;
+      u0[q] = i < nt * C ? __ldcg(ug + (size_t)t * d.a[GL_LDU] + c0 + ch) : 0.f;
     }
     consumer_sync();
-    if ((bs & 1) == 0) rglru_gates<HYB, true>(d, us, rs, is, nt);
+    if (mma) rglru_gates_mma(d, uh, pitch, part, nt, af, tb == 0 && warp < ((C + 15) >> 4) * 4);
+    else if ((bs & 1) == 0) rglru_gates<HYB, true>(d, us, rs, is, nt);
     else rglru_gates<HYB, false>(d, us, rs, is, nt);
     consumer_sync();
-    for (int i = tid; i < nt * C; i += kConsumerThreads) {
-      const int t = i / C, ch = i - t * C, g = gch + ch;
-      const float r = sigmoid_f(rs[i] + bf16_at(d.p[4], g)), gi = sigmoid_f(is[i] + bf16_at(d.p[6], g));
-      const float la = -gate_c * r * softplus_f(bf16_at(d.p[7], g));
-      float a = decay_exp(la), b = sqrtf(-expm1f(2.0f * la)) * gi * us[(size_t)t * bs + c0 + ch];
+#pragma unroll 1
+    for (int q = 0; q * kConsumerThreads < nt * C; ++q) {
+      const int i = tid + q * kConsumerThreads;
+      if (i >= nt * C) break;
+      const int t = i / C, ch = i - t * C;
+      float rp = rs[i], ip = is[i];
+      if (mma) { rp += part[2 * (size_t)TG * C + i]; ip += part[3 * (size_t)TG * C + i]; }
+      const float u = q == 0 ? u0[0] : q == 1 ? u0[1] : q == 2 ? u0[2] : q == 3 ? u0[3] : __ldcg(ug + (size_t)t * d.a[GL_LDU] + c0 + ch);
+      const float r = sigmoid_f(rp + chp[ch]), gi = sigmoid_f(ip + chp[64 + ch]);
+      const float la = -r * chp[128 + ch];
+      float a = decay_exp(la), b = sqrtf(-expm1f(2.0f * la)) * gi * u;
       const TokenRec &tr = rec[tb + t];
       if (tr.flags & 1) {   // the request's carried state enters here; nothing flows in from the previous token
-        if (!(tr.flags & 4)) b = fmaf(a, __ldcg(state + (size_t)tr.slot * width + g), b);
+        if (!(tr.flags & 4)) b = fmaf(a, __ldcg(state + (size_t)tr.slot * width + gch + ch), b);
         a = 0.f;
       }
       rs[i] = a;
@@ -800,6 +1251,7 @@ __device__ __forceinline__ void run_rglru(const Ctx &c, const TaskDesc &d) {
     consumer_sync();
     if (tid < C) {
       float S = carry;
+#pragma unroll 4
       for (int t = 0; t < nt; ++t) {
         S = fmaf(rs[(size_t)t * C + tid], S, is[(size_t)t * C + tid]);
         is[(size_t)t * C + tid] = S;
@@ -807,67 +1259,133 @@ __device__ __forceinline__ void run_rglru(const Ctx &c, const TaskDesc &d) {
       carry = S;
     }
     consumer_sync();
-    for (int i = tid; i < nt * C; i += kConsumerThreads) {
-      const int t = i / C, ch = i - t * C, g = gch + ch;
+#pragma unroll 1
+    for (int q = 0; q * kConsumerThreads < nt * C; ++q) {
+      const int i = tid + q * kConsumerThreads;
+      if (i >= nt * C) break;
+      const int t = i / C, ch = i - t * C;
       const float S = is[i];
       const TokenRec &tr = rec[tb + t];
-      if (tr.flags & 2) state[(size_t)tr.slot * width + g] = S;
-      const float y = gelu_tanh_f(__ldcg(reinterpret_cast<const float *>(d.p[1]) + (size_t)(tb + t) * d.a[GL_LDP] + d.a[GL_YOFF] + g) +
-                                  bf16_at(d.p[2], g));
-      store_elt(outp + (size_t)(tb + t) * d.a[GL_LDO] + d.a[GL_OCOL] + g, S * y * oscale);
+      if (tr.flags & 2) state[(size_t)tr.slot * width + gch + ch] = S;
+      const float yp = q == 0 ? y0[0] : q == 1 ? y0[1] : q == 2 ? y0[2] : q == 3 ? y0[3] : __ldcg(yg + (size_t)t * d.a[GL_LDP] + ch);
+      store_elt(outp + (size_t)(tb + t) * d.a[GL_LDO] + d.a[GL_OCOL] + gch + ch, S * gelu_tanh_f(yp + chp[192 + ch]) * oscale);
     }
     consumer_sync();
   }
 }
 
 // ---------------------------------------------------------------------------
-// TASK_MLSTM: (request, head, range of value columns).  Matrix memory S [dim, columns] in registers, 4 columns x RPT
-// rows per thread; the columns of the task are walked in sub-blocks of 4 CQ.  Per token
+// TASK_MLSTM: (request, head, range of value columns).  Matrix memory S [dim, columns] in registers: a thread holds RPT
+// consecutive rows of 4 columns, the block 4 CQ columns of all rows (256 RPT / CQ of them; keys and queries are padded with
+// zeros up to that, so padding rows stay zero); the columns of the task are walked in sub-blocks.  Per token
 //   m' = max(f + m, i), S = exp(f + m - m') S + exp(i - m') k v^T, n likewise, o = S^T q / (max(|n q|, exp(-m')) + 1e-6)
 // Every task keeps its own copy of (n, m), so that tasks of one head share nothing while they run.  The normalised and
 // gated output needs the whole head: the last task of the (request, head) to finish writes it.
 // ---------------------------------------------------------------------------
-template <int HYB, int RPT>
-__device__ __forceinline__ void mlstm_body(const Ctx &c, const TaskDesc &d, const SeqView &sv, int CQ) {
+struct MlstmView {
+  const float *proj;   // projections of the request's first token
+  float *nm, *S, *raw;
+  int ldp, H, h, dim, vdim, vdimp, V0, V1, chunks;
+  bool fresh;
+};
+__device__ __forceinline__ MlstmView mlstm_view(const TaskDesc &d, const SeqView &sv) {
+  MlstmView m;
+  m.ldp = d.a[ML_LDP]; m.H = d.a[ML_H]; m.h = d.a[ML_HEAD]; m.dim = d.a[ML_DIM]; m.vdim = d.a[ML_VDIM]; m.vdimp = d.a[ML_VDIMP];
+  m.V0 = d.a[ML_V0]; m.V1 = d.a[ML_V1]; m.chunks = d.a[ML_NCHUNK];
+  m.fresh = sv.pos0 == 0;
+  m.proj = reinterpret_cast<const float *>(d.p[0]) + (size_t)sv.q0 * m.ldp;
+  m.nm = reinterpret_cast<float *>(d.p[5]) + ((size_t)(sv.slot * m.H + m.h) * m.chunks + d.a[ML_CHUNK]) * (m.dim + 1);
+  m.S = reinterpret_cast<float *>(d.p[4]) + (size_t)(sv.slot * m.H + m.h) * m.dim * m.vdimp;
+  m.raw = reinterpret_cast<float *>(d.p[6]) + (size_t)sv.q0 * d.a[ML_LDR] + (size_t)m.h * m.vdim;
+  return m;
+}
+// log gates from the pre-activations
+__device__ __forceinline__ float mlstm_log_i(float pre, float cap) { return cap * tanhf(pre / cap); }
+__device__ __forceinline__ float mlstm_log_f(float pre, float cap) { return -softplus_f(-cap * tanhf(pre / cap)); }
+
+// True for the task that finishes a (request, head).  Ends with a barrier.
+__device__ __forceinline__ bool mlstm_last(const Ctx &c, const TaskDesc &d, int chunks) {
+  consumer_sync();
+  if (chunks == 1) return true;
+  if (threadIdx.x == 0) {
+    unsigned int *ticket = &c.P.attn_tickets[d.a[ML_TICKET]];
+    unsigned int old;
+    asm volatile("atom.acq_rel.gpu.global.add.u32 %0, [%1], 1;" : "=r"(old) : "l"(ticket) : "memory");
+    const bool last = old + 1u == (unsigned)chunks;
+    if (last) *reinterpret_cast<volatile unsigned int *>(ticket) = 0u;
+    c.s.flags[1] = last ? 1 : 0;
+  }
+  consumer_sync();
+  return c.s.flags[1] != 0;
+}
+
+// One step of S and the read-out for this thread's rows (k scaled by the input gate).
+template <int RPT>
+__device__ __forceinline__ float4 mlstm_step(float4 (&S)[RPT], float a, const float4 v, const float *kt, const float *qt) {
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < RPT; i += 4) {
+    const float4 k4 = *reinterpret_cast<const float4 *>(kt + i), q4 = *reinterpret_cast<const float4 *>(qt + i);
+    const float k[4] = {k4.x, k4.y, k4.z, k4.w}, q[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float4 &s = S[i + e];
+      s.x = fmaf(a, s.x, k[e] * v.x); o.x = fmaf(q[e], s.x, o.x);
+      s.y = fmaf(a, s.y, k[e] * v.y); o.y = fmaf(q[e], s.y, o.y);
+      s.z = fmaf(a, s.z, k[e] * v.z); o.z = fmaf(q[e], s.z, o.z);
+      s.w = fmaf(a, s.w, k[e] * v.w); o.w = fmaf(q[e], s.w, o.w);
+    }
+  }
+  return o;
+}
+// Sum over the row groups of a warp (lanes that differ above bit log2(CQ)); valid in lanes < CQ.
+template <int CQ>
+__device__ __forceinline__ float4 mlstm_warp_rows(float4 o) {
+#pragma unroll
+  for (int s = CQ; s < 32; s <<= 1) {
+    o.x += __shfl_xor_sync(0xffffffffu, o.x, s);
+    o.y += __shfl_xor_sync(0xffffffffu, o.y, s);
+    o.z += __shfl_xor_sync(0xffffffffu, o.z, s);
+    o.w += __shfl_xor_sync(0xffffffffu, o.w, s);
+  }
+  return o;
+}
+
+// A portion of several tokens.
+template <int HYB, int CQ, int RPT>
+__device__ __noinline__ void mlstm_portion(const Ctx c, const TaskDesc &d, const SeqView sv, int task) {
   typedef typename HybElt<HYB>::T T;
-  const KernelParams &P = c.P;
+  constexpr int VC = 4 * CQ, RG = kConsumerThreads / CQ, ROWS = RG * RPT;
+  constexpr int NR = (ROWS + kConsumerThreads - 1) / kConsumerThreads;   // rows of n per thread
+  const MlstmView m = mlstm_view(d, sv);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int H = d.a[ML_H], h = d.a[ML_HEAD], dim = d.a[ML_DIM], vdim = d.a[ML_VDIM], vdimp = d.a[ML_VDIMP], TC = d.a[ML_TC];
-  const int vc = 4 * CQ, RG = kConsumerThreads / CQ, qd = tid % CQ, rg = tid / CQ;
-  const float *proj = reinterpret_cast<const float *>(d.p[0]) + (size_t)sv.q0 * d.a[ML_LDP];
-  const int ldp = d.a[ML_LDP];
-  const bool fresh = sv.pos0 == 0;
-  float *nm = reinterpret_cast<float *>(d.p[5]) + ((size_t)(sv.slot * H + h) * d.a[ML_NCHUNK] + d.a[ML_CHUNK]) * (dim + 1);
-  float *Sg = reinterpret_cast<float *>(d.p[4]) + (size_t)(sv.slot * H + h) * dim * vdimp;
-  float *raw = reinterpret_cast<float *>(d.p[6]) + (size_t)sv.q0 * d.a[ML_LDR] + (size_t)h * vdim;
+  const int qd = tid % CQ, r0 = tid / CQ * RPT, TC = d.a[ML_TC];
   // shared memory
   float *dec = reinterpret_cast<float *>(c.s.xtile);   // [64] exp(f + m - m')
   float *inp = dec + kMaxLinearTokens;                 // [64] exp(i - m')
   float *den = inp + kMaxLinearTokens;                 // [64] exp(-m'), then the denominator
   float *nred = den + kMaxLinearTokens;                // [TC][8]
-  float *ks = nred + TC * 8;                           // [TC][dim] input-scaled keys
-  float *qs = ks + (size_t)TC * dim;                   // [TC][dim]
-  float *vs = qs + (size_t)TC * dim;                   // [TC][vc]
-  float *red = vs + (size_t)TC * vc;                   // [TC][8 warps][vc]
+  float *ks = nred + TC * 8;                           // [TC][ROWS] input-scaled keys
+  float *qs = ks + (size_t)TC * ROWS;                  // [TC][ROWS]
+  float *vs = qs + (size_t)TC * ROWS;                  // [TC][VC]
+  float *red = vs + (size_t)TC * VC;                   // [TC][8 warps][VC]
   const float cap = __int_as_float(d.a[ML_CAP]), qscale = __int_as_float(d.a[ML_QSCALE]);
   // gates of all tokens, then the running maximum (one thread: a handful of operations per token)
   for (int t = tid; t < sv.nq; t += kConsumerThreads) {
-    const float ip = __ldcg(proj + (size_t)t * ldp + d.a[ML_IOFF] + h) + bf16_at(d.p[1], h);
-    const float fp = __ldcg(proj + (size_t)t * ldp + d.a[ML_FOFF] + h) + bf16_at(d.p[2], h);
-    inp[t] = cap * tanhf(ip / cap);
-    dec[t] = -softplus_f(-cap * tanhf(fp / cap));
+    inp[t] = mlstm_log_i(__ldcg(m.proj + (size_t)t * m.ldp + d.a[ML_IOFF] + m.h) + bf16_at(d.p[1], m.h), cap);
+    dec[t] = mlstm_log_f(__ldcg(m.proj + (size_t)t * m.ldp + d.a[ML_FOFF] + m.h) + bf16_at(d.p[2], m.h), cap);
   }
   consumer_sync();
   if (tid == 0) {
-    float m = fresh ? 0.f : __ldcg(nm + dim);
+    float run = m.fresh ? 0.f : __ldcg(m.nm + m.dim);
     for (int t = 0; t < sv.nq; ++t) {
-      const float fm = dec[t] + m, i = inp[t];
-      m = fmaxf(fm, i);
-      dec[t] = fm - m;
-      inp[t] = i - m;
-      den[t] = -m;
+      const float fm = dec[t] + run, i = inp[t];
+      run = fmaxf(fm, i);
+      dec[t] = fm - run;
+      inp[t] = i - run;
+      den[t] = -run;
     }
-    nm[dim] = m;
+    m.nm[m.dim] = run;
   }
   consumer_sync();
   for (int t = tid; t < sv.nq; t += kConsumerThreads) {
@@ -875,66 +1393,53 @@ __device__ __forceinline__ void mlstm_body(const Ctx &c, const TaskDesc &d, cons
     inp[t] = expf(inp[t]);
     den[t] = expf(den[t]);
   }
-  constexpr int NR = 4;   // rows of n per thread: dim <= 1024
+  stamp(c, task, 0);
   float n[NR];
 #pragma unroll
   for (int i = 0; i < NR; ++i) {
     const int row = tid + i * kConsumerThreads;
-    n[i] = (!fresh && row < dim) ? __ldcg(nm + row) : 0.f;
+    n[i] = (!m.fresh && row < m.dim) ? __ldcg(m.nm + row) : 0.f;
   }
-  for (int v0 = d.a[ML_V0]; v0 < d.a[ML_V1]; v0 += vc) {
-    const bool col_ok = v0 + 4 * qd < vdimp && v0 + 4 * qd < d.a[ML_V1];
-    const bool first = v0 == d.a[ML_V0];
+  for (int v0 = m.V0; v0 < m.V1; v0 += VC) {
+    const bool col_ok = v0 + 4 * qd < m.V1;
+    const bool first = v0 == m.V0;
     float4 S[RPT];
+    float *Sp = m.S + (size_t)r0 * m.vdimp + v0 + 4 * qd;
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
-      const int row = rg + i * RG;
       S[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (!fresh && col_ok && row < dim) S[i] = __ldcg(reinterpret_cast<const float4 *>(Sg + (size_t)row * vdimp + v0 + 4 * qd));
+      if (!m.fresh && col_ok && r0 + i < m.dim) S[i] = __ldcg(reinterpret_cast<const float4 *>(Sp + (size_t)i * m.vdimp));
     }
     for (int tb = 0; tb < sv.nq; tb += TC) {
       const int nt = min(TC, sv.nq - tb);
       consumer_sync();   // gates are final / the previous trip's readers are done
-      for (int i = tid; i < nt * dim; i += kConsumerThreads) {
-        const int t = i / dim, r = i - t * dim;
-        const float *pr = proj + (size_t)(tb + t) * ldp + h * dim + r;
-        ks[i] = __ldcg(pr + d.a[ML_KOFF]) * inp[tb + t];
-        qs[i] = __ldcg(pr + d.a[ML_QOFF]) * qscale;
-      }
-      for (int i = tid; i < nt * vc; i += kConsumerThreads) {
-        const int t = i / vc, col = v0 + i - t * vc;
-        vs[i] = col < vdim ? __ldcg(proj + (size_t)(tb + t) * ldp + d.a[ML_VOFF] + (size_t)h * vdim + col) : 0.f;
+      // warp w takes tokens w, w + 8; a lane's loads of a token are independent and in flight together
+      const float *pk = m.proj + (size_t)tb * m.ldp + d.a[ML_KOFF] + m.h * m.dim, *pq = m.proj + (size_t)tb * m.ldp + d.a[ML_QOFF] + m.h * m.dim;
+      const float *pv = m.proj + (size_t)tb * m.ldp + d.a[ML_VOFF] + (size_t)m.h * m.vdim + v0;
+      for (int t = warp; t < nt; t += 8) {
+        const float in = inp[tb + t];
+#pragma unroll 8
+        for (int r = lane; r < ROWS; r += 32) {
+          const bool ok = r < m.dim;
+          ks[(size_t)t * ROWS + r] = ok ? __ldcg(pk + (size_t)t * m.ldp + r) * in : 0.f;
+          qs[(size_t)t * ROWS + r] = ok ? __ldcg(pq + (size_t)t * m.ldp + r) * qscale : 0.f;
+        }
+#pragma unroll
+        for (int r = lane; r < VC; r += 32) vs[t * VC + r] = v0 + r < m.vdim ? __ldcg(pv + (size_t)t * m.ldp + r) : 0.f;
       }
       consumer_sync();
       for (int t = 0; t < nt; ++t) {
         const float a = dec[tb + t];
-        const float4 v = *reinterpret_cast<const float4 *>(vs + t * vc + 4 * qd);
-        const float *kt = ks + (size_t)t * dim, *qt = qs + (size_t)t * dim;
-        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-        for (int i = 0; i < RPT; ++i) {
-          const int row = rg + i * RG;
-          if (row < dim) {
-            const float k = kt[row], q = qt[row];
-            S[i].x = fmaf(a, S[i].x, k * v.x); o.x = fmaf(q, S[i].x, o.x);
-            S[i].y = fmaf(a, S[i].y, k * v.y); o.y = fmaf(q, S[i].y, o.y);
-            S[i].z = fmaf(a, S[i].z, k * v.z); o.z = fmaf(q, S[i].z, o.z);
-            S[i].w = fmaf(a, S[i].w, k * v.w); o.w = fmaf(q, S[i].w, o.w);
-          }
-        }
-        for (int s = CQ; s < 32; s <<= 1) {
-          o.x += __shfl_xor_sync(0xffffffffu, o.x, s);
-          o.y += __shfl_xor_sync(0xffffffffu, o.y, s);
-          o.z += __shfl_xor_sync(0xffffffffu, o.z, s);
-          o.w += __shfl_xor_sync(0xffffffffu, o.w, s);
-        }
-        if (lane < CQ) *reinterpret_cast<float4 *>(red + (size_t)(t * 8 + warp) * vc + 4 * lane) = o;
+        const float *kt = ks + (size_t)t * ROWS, *qt = qs + (size_t)t * ROWS;
+        const float4 v = *reinterpret_cast<const float4 *>(vs + t * VC + 4 * qd);
+        const float4 o = mlstm_warp_rows<CQ>(mlstm_step<RPT>(S, a, v, kt + r0, qt + r0));
+        if (lane < CQ) *reinterpret_cast<float4 *>(red + (size_t)(t * 8 + warp) * VC + 4 * lane) = o;
         if (first) {
           float p = 0.f;
 #pragma unroll
           for (int i = 0; i < NR; ++i) {
             const int row = tid + i * kConsumerThreads;
-            if (row < dim) {
+            if (row < ROWS) {
               n[i] = fmaf(a, n[i], kt[row]);
               p = fmaf(n[i], qt[row], p);
             }
@@ -953,63 +1458,175 @@ __device__ __forceinline__ void mlstm_body(const Ctx &c, const TaskDesc &d, cons
         }
         consumer_sync();
       }
-      for (int i = tid; i < nt * vc; i += kConsumerThreads) {
-        const int t = i / vc, j = i - t * vc;
+      for (int i = tid; i < nt * VC; i += kConsumerThreads) {
+        const int t = i / VC, j = i % VC;
         float s = 0.f;
 #pragma unroll
-        for (int w = 0; w < 8; ++w) s += red[(size_t)(t * 8 + w) * vc + j];
-        if (v0 + j < vdim && v0 + j < d.a[ML_V1]) __stcg(raw + (size_t)(tb + t) * d.a[ML_LDR] + v0 + j, s / den[tb + t]);
+        for (int w = 0; w < 8; ++w) s += red[(size_t)(t * 8 + w) * VC + j];
+        if (v0 + j < m.vdim && v0 + j < m.V1) __stcg(m.raw + (size_t)(tb + t) * d.a[ML_LDR] + v0 + j, s / den[tb + t]);
       }
     }
 #pragma unroll
-    for (int i = 0; i < RPT; ++i) {
-      const int row = rg + i * RG;
-      if (col_ok && row < dim) *reinterpret_cast<float4 *>(Sg + (size_t)row * vdimp + v0 + 4 * qd) = S[i];
-    }
+    for (int i = 0; i < RPT; ++i)
+      if (col_ok && r0 + i < m.dim) *reinterpret_cast<float4 *>(Sp + (size_t)i * m.vdimp) = S[i];
   }
 #pragma unroll
   for (int i = 0; i < NR; ++i) {
     const int row = tid + i * kConsumerThreads;
-    if (row < dim) nm[row] = n[i];
+    if (row < m.dim) m.nm[row] = n[i];
   }
+  stamp(c, task, 1);
   // ---- output of the head
-  consumer_sync();
-  if (d.a[ML_NCHUNK] > 1) {
-    if (tid == 0) {
-      unsigned int *ticket = &P.attn_tickets[d.a[ML_TICKET]];
-      unsigned int old;
-      asm volatile("atom.acq_rel.gpu.global.add.u32 %0, [%1], 1;" : "=r"(old) : "l"(ticket) : "memory");
-      const bool last = old + 1u == (unsigned)d.a[ML_NCHUNK];
-      if (last) *reinterpret_cast<volatile unsigned int *>(ticket) = 0u;
-      c.s.flags[1] = last ? 1 : 0;
-    }
-    consumer_sync();
-    if (c.s.flags[1] == 0) return;
-  }
+  if (!mlstm_last(c, d, m.chunks)) return;
+  stamp(c, task, 2);
   const float eps = __int_as_float(d.a[ML_EPS]);
-  T *out = reinterpret_cast<T *>(d.p[7]) + (size_t)sv.q0 * d.a[ML_LDO] + (size_t)h * vdim;
+  T *out = reinterpret_cast<T *>(d.p[7]) + (size_t)sv.q0 * d.a[ML_LDO] + (size_t)m.h * m.vdim;
   for (int t = warp; t < sv.nq; t += 8) {
-    const float *rt = raw + (size_t)t * d.a[ML_LDR];
+    const float *rt = m.raw + (size_t)t * d.a[ML_LDR];
+    const float *gt = m.proj + (size_t)t * m.ldp + d.a[ML_GOFF] + (size_t)m.h * m.vdim;
     float ss = 0.f;
-    for (int j = lane; j < vdim; j += 32) { const float v = __ldcg(rt + j); ss += v * v; }
-    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
-    for (int j = lane; j < vdim; j += 32) {
-      const float g = __ldcg(proj + (size_t)t * ldp + d.a[ML_GOFF] + (size_t)h * vdim + j);
-      store_elt(out + (size_t)t * d.a[ML_LDO] + j, __ldcg(rt + j) * inv * bf16_at(d.p[3], (size_t)h * vdim + j) * sigmoid_f(g));
+    if (m.vdim <= 512) {   // the row and its gates in registers, all loads in flight
+      float x[16], g[16];
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const bool in = i * 32 + lane < m.vdim;
+        x[i] = in ? __ldcg(rt + i * 32 + lane) : 0.f;
+        g[i] = in ? __ldcg(gt + i * 32 + lane) : 0.f;
+      }
+#pragma unroll
+      for (int i = 0; i < 16; ++i) ss += x[i] * x[i];
+      const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)m.vdim + eps);
+#pragma unroll
+      for (int i = 0; i < 16; ++i)
+        if (i * 32 + lane < m.vdim)
+          store_elt(out + (size_t)t * d.a[ML_LDO] + i * 32 + lane, x[i] * inv * bf16_at(d.p[3], (size_t)m.h * m.vdim + i * 32 + lane) * sigmoid_f(g[i]));
+      continue;
     }
+    for (int j = lane; j < m.vdim; j += 32) { const float v = __ldcg(rt + j); ss += v * v; }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)m.vdim + eps);
+    for (int j = lane; j < m.vdim; j += 32)
+      store_elt(out + (size_t)t * d.a[ML_LDO] + j, __ldcg(rt + j) * inv * bf16_at(d.p[3], (size_t)m.h * m.vdim + j) * sigmoid_f(__ldcg(gt + j)));
   }
 }
 
+// One token (decoding): the state is what has to move.  Every thread copies its own piece of the next sub-block into its
+// own shared-memory cells while it works on the current one, starting before anything else is known of the token.
+template <int HYB, int CQ, int RPT>
+__device__ __noinline__ void mlstm_single(const Ctx c, const TaskDesc &d, const SeqView sv, int task) {
+  typedef typename HybElt<HYB>::T T;
+  constexpr int VC = 4 * CQ, RG = kConsumerThreads / CQ, ROWS = RG * RPT;
+  constexpr int NR = (ROWS + kConsumerThreads - 1) / kConsumerThreads;
+  const MlstmView m = mlstm_view(d, sv);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int qd = tid % CQ, r0 = tid / CQ * RPT;
+  float4 *ring = reinterpret_cast<float4 *>(c.s.xtile) + tid;                  // [2][RPT][256], this thread's cells
+  float *ks = reinterpret_cast<float *>(c.s.xtile) + 8 * RPT * kConsumerThreads;   // [ROWS] input-scaled keys
+  float *qs = ks + ROWS;                                                       // [ROWS]
+  float *red = qs + ROWS;                                                      // [2][8 warps][VC]
+  float *misc = red + 16 * VC;                                                 // [16]
+  const int nrow = min(RPT, m.dim - r0);                                       // real rows of this thread (may be <= 0)
+  float *Sp = m.S + (size_t)r0 * m.vdimp + m.V0 + 4 * qd;                      // its piece of the current sub-block
+  auto fetch = [&](int v0, int slot, const float *src) {
+    if (!m.fresh && v0 + 4 * qd < m.V1) {
+      const uint32_t dst = smem_u32(ring + slot * RPT * kConsumerThreads);
+#pragma unroll
+      for (int i = 0; i < RPT; ++i, src += m.vdimp)
+        if (i < nrow)
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + (uint32_t)(i * kConsumerThreads * 16)), "l"(src) : "memory");
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  fetch(m.V0, 0, Sp);
+  fetch(m.V0 + VC, 1, Sp + VC);
+  const float cap = __int_as_float(d.a[ML_CAP]), qscale = __int_as_float(d.a[ML_QSCALE]);
+  float kq[NR][2], n[NR];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int row = tid + i * kConsumerThreads;
+    const bool ok = row < m.dim;
+    kq[i][0] = ok ? __ldcg(m.proj + d.a[ML_KOFF] + m.h * m.dim + row) : 0.f;
+    kq[i][1] = ok ? __ldcg(m.proj + d.a[ML_QOFF] + m.h * m.dim + row) : 0.f;
+    n[i] = ok && !m.fresh ? __ldcg(m.nm + row) : 0.f;
+  }
+  const float li = mlstm_log_i(__ldcg(m.proj + d.a[ML_IOFF] + m.h) + bf16_at(d.p[1], m.h), cap);
+  const float fm = mlstm_log_f(__ldcg(m.proj + d.a[ML_FOFF] + m.h) + bf16_at(d.p[2], m.h), cap) + (m.fresh ? 0.f : __ldcg(m.nm + m.dim));
+  const float run = fmaxf(fm, li), a = decay_exp(fm - run), b = expf(li - run);
+  float p = 0.f;
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int row = tid + i * kConsumerThreads;
+    if (row < ROWS) {
+      const float k = kq[i][0] * b, q = kq[i][1] * qscale;
+      ks[row] = k;
+      qs[row] = q;
+      n[i] = fmaf(a, n[i], k);
+      p = fmaf(n[i], q, p);
+      if (row < m.dim) m.nm[row] = n[i];
+    }
+  }
+  const float den = fmaxf(fabsf(block_sum(p, misc)), expf(-run)) + 1e-6f;   // (its barrier also orders reads of nm[dim] before the write)
+  if (tid == 0) m.nm[m.dim] = run;
+  stamp(c, task, 0);
+  int par = 0;
+  for (int v0 = m.V0; v0 < m.V1; v0 += VC, par ^= 1, Sp += VC) {
+    const bool col_ok = v0 + 4 * qd < m.V1;
+    float4 S[RPT];
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+#pragma unroll
+    for (int i = 0; i < RPT; ++i)
+      S[i] = !m.fresh && col_ok && i < nrow ? ring[(par * RPT + i) * kConsumerThreads] : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float *pv = m.proj + d.a[ML_VOFF] + (size_t)m.h * m.vdim + v0 + 4 * qd;
+    float4 v;
+    v.x = v0 + 4 * qd < m.vdim ? __ldcg(pv) : 0.f;
+    v.y = v0 + 4 * qd + 1 < m.vdim ? __ldcg(pv + 1) : 0.f;
+    v.z = v0 + 4 * qd + 2 < m.vdim ? __ldcg(pv + 2) : 0.f;
+    v.w = v0 + 4 * qd + 3 < m.vdim ? __ldcg(pv + 3) : 0.f;
+    const float4 o = mlstm_warp_rows<CQ>(mlstm_step<RPT>(S, a, v, ks + r0, qs + r0));
+    fetch(v0 + 2 * VC, par, Sp + 2 * VC);
+    if (lane < CQ) *reinterpret_cast<float4 *>(red + (size_t)(par * 8 + warp) * VC + 4 * lane) = o;
+    float *dst = Sp;
+#pragma unroll
+    for (int i = 0; i < RPT; ++i, dst += m.vdimp)
+      if (col_ok && i < nrow) *reinterpret_cast<float4 *>(dst) = S[i];
+    consumer_sync();
+    if (tid < VC && v0 + tid < m.vdim && v0 + tid < m.V1) {
+      float s = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) s += red[(size_t)(par * 8 + w) * VC + tid];
+      __stcg(m.raw + v0 + tid, s / den);
+    }
+  }
+  stamp(c, task, 1);
+  if (!mlstm_last(c, d, m.chunks)) return;
+  stamp(c, task, 2);
+  const float *gt = m.proj + d.a[ML_GOFF] + (size_t)m.h * m.vdim;
+  T *out = reinterpret_cast<T *>(d.p[7]) + (size_t)sv.q0 * d.a[ML_LDO] + (size_t)m.h * m.vdim;
+  float ss = 0.f;
+  for (int j = tid; j < m.vdim; j += kConsumerThreads) { const float x = __ldcg(m.raw + j); ss += x * x; }
+  const float inv = 1.0f / sqrtf(block_sum(ss, misc + 8) / (float)m.vdim + __int_as_float(d.a[ML_EPS]));
+  for (int j = tid; j < m.vdim; j += kConsumerThreads)
+    store_elt(out + j, __ldcg(m.raw + j) * inv * bf16_at(d.p[3], (size_t)m.h * m.vdim + j) * sigmoid_f(__ldcg(gt + j)));
+}
+
+template <int HYB, int CQ, int RPT>
+__device__ __forceinline__ void mlstm_body(const Ctx &c, const TaskDesc &d, const SeqView &sv, int task) {
+  if (sv.nq == 1) mlstm_single<HYB, CQ, RPT>(c, d, sv, task);
+  else mlstm_portion<HYB, CQ, RPT>(c, d, sv, task);
+}
 template <int HYB>
-__device__ __forceinline__ void run_mlstm(const Ctx &c, const TaskDesc &d) {
+__device__ __forceinline__ void run_mlstm(const Ctx &c, const TaskDesc &d, int task) {
   const SeqView sv = seq_view(c.P, d.a[ML_SLOT]);
   if (sv.nq <= 0) return;
   const int dim = d.a[ML_DIM];
-  const int CQ = dim <= 256 ? 16 : (dim <= 512 ? 8 : 4);      // at most 16 rows per thread
-  const int rpt = (dim * CQ + kConsumerThreads - 1) / kConsumerThreads;
-  if (rpt <= 4) mlstm_body<HYB, 4>(c, d, sv, CQ);
-  else if (rpt <= 8) mlstm_body<HYB, 8>(c, d, sv, CQ);
-  else mlstm_body<HYB, 16>(c, d, sv, CQ);
+  switch (mlstm_quads(dim)) {
+    case 16:
+      if (mlstm_rows_per_thread(dim) == 4) mlstm_body<HYB, 16, 4>(c, d, sv, task);
+      else mlstm_body<HYB, 16, 8>(c, d, sv, task);
+      break;
+    case 8: mlstm_body<HYB, 8, 8>(c, d, sv, task); break;
+    case 4: mlstm_body<HYB, 4, 8>(c, d, sv, task); break;
+    default: mlstm_body<HYB, 2, 8>(c, d, sv, task); break;
+  }
 }
 
 // ---------------------------------------------------------------------------
@@ -1051,7 +1668,7 @@ __device__ __forceinline__ void run_argmax_reduce_f32(const Ctx &c, const TaskDe
 }
 
 template <int HYB>
-__device__ __forceinline__ void run_hybrid_task(const Ctx &c, const TaskDesc &d) {
+__device__ __forceinline__ void run_hybrid_task(const Ctx &c, const TaskDesc &d, int task) {
   switch (d.type) {
     case TASK_BATCH: {
       Ctx cc = c;
@@ -1063,10 +1680,10 @@ __device__ __forceinline__ void run_hybrid_task(const Ctx &c, const TaskDesc &d)
     case TASK_RESIDUAL_NORM: run_residual_norm<HYB>(c, d); break;
     case TASK_LINEAR_F32: if (HYB == HYB_F32) run_linear_f32(c, d); break;
     case TASK_QKV_APPEND: run_qkv_append<HYB>(c, d); break;
-    case TASK_EXT_ATTENTION: run_ext_attention<HYB>(c, d); break;
+    case TASK_EXT_ATTENTION: run_ext_attention<HYB>(c, d, task); break;
     case TASK_SHORT_CONV: run_short_conv(c, d); break;
     case TASK_RGLRU: run_rglru<HYB>(c, d); break;
-    case TASK_MLSTM: run_mlstm<HYB>(c, d); break;
+    case TASK_MLSTM: run_mlstm<HYB>(c, d, task); break;
     case TASK_ARGMAX_PARTIAL: run_argmax_partial_f32(c, d); break;
     case TASK_ARGMAX_REDUCE: run_argmax_reduce_f32(c, d); break;
     case TASK_SAMPLING_PARTIAL: run_sampling_partial<float>(c, d); break;

@@ -3792,7 +3792,7 @@ __device__ __forceinline__ bool task_other(const Ctx &c, const TaskDesc &d, int 
   ok = wait_dependencies(c, d, t, ok, tt);
   if (!ok) return false;
   if (HYB) {
-    run_hybrid_task<HYB>(c, d);
+    run_hybrid_task<HYB>(c, d, t);
     return true;
   }
   switch (d.type) {

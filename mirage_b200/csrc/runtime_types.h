@@ -66,12 +66,19 @@ enum TaskType : uint32_t {
 };
 
 // Which family of megakernel instantiations runs a graph (template parameter HYB of the kernel).
+// Thread layout of a matrix-memory task: value-column quads and key rows per thread (256 threads).
+#ifdef __CUDACC__
+#define MPK_HD __host__ __device__
+#else
+#define MPK_HD
+#endif
+MPK_HD constexpr int mlstm_quads(int dim) { return dim <= 128 ? 16 : (dim <= 256 ? 8 : (dim <= 512 ? 4 : 2)); }
+MPK_HD constexpr int mlstm_rows_per_thread(int dim) { return dim > 64 ? 8 : 4; }
+MPK_HD constexpr int mlstm_rows(int dim) { return kConsumerThreads / mlstm_quads(dim) * mlstm_rows_per_thread(dim); }
+
 // Query rows a bf16 extended-attention task keeps in shared memory: whole 16-row tiles, a power of two of them (the
 // warps are split over the tiles), at most as many as the graph can batch.
-#ifdef __CUDACC__
-__host__ __device__
-#endif
-constexpr int ext_attention_rows(int rows) {
+MPK_HD constexpr int ext_attention_rows(int rows) {
   int r = 16;
   while (r < rows) r *= 2;
   return r;
@@ -199,7 +206,8 @@ enum { QA_T0 = 0, QA_T1, QA_LDP, QA_QOFF, QA_KOFF, QA_VOFF, QA_HQ, QA_HKV, QA_DI
        QA_EPS, QA_PAGE, QA_LDQ, QA_ROWS };
 // ---- TASK_EXT_ATTENTION: p[0] q [tokens, hq * dimp]  p[1] k cache  p[2] v cache  p[3] out;  a[XA_*] below
 enum { XA_SLOT = 0, XA_HEAD, XA_CHUNK, XA_NCHUNK, XA_HQ, XA_HKV, XA_DIMP, XA_VDIM, XA_VDIMP, XA_PAGE, XA_LDQ, XA_LDO, XA_OCOL,
-       XA_SCALE, XA_CAP, XA_SINK, XA_OSCALE, XA_TICKET, XA_SREC, XA_WINDOW };
+       XA_SCALE, XA_CAP, XA_SINK, XA_OSCALE, XA_TICKET, XA_SREC, XA_STAGES };
+constexpr int kXaCells = 320;   // cache rows of a chunk's key octets kept in shared memory
 // ---- TASK_SHORT_CONV: channels [a[0], a[1]); p[0] in f32  p[1] in bias bf16 or null  p[2] taps bf16 [channels, taps]
 //      p[3] bias bf16 or null  p[4] carried inputs f32 [slots, taps - 1, channels]  p[5] out f32
 //      a[2] channels  a[3] taps  a[4] ld in  a[5] in column offset  a[6] ld out  a[7] activation (0 none, 1 silu)

@@ -994,11 +994,16 @@ struct Builder {
     const int w = (int)std::max(T[l.t[1]].dim(3), T[l.t[2]].dim(3));
     return w <= 64 ? 64 : (w <= 128 ? 128 : 256);
   }
+  // key / value tiles in flight: graphs of many tokens reserve a large activation tile anyway
+  int xattn_stages() const { return nb_max > 8 ? 3 : 2; }
+  // shared memory of a token: gate sums and u, as float32 or as three bf16 parts
+  static int64_t rglru_token_bytes(int bs, int C) { return 16 * C + 6 * (round_up(bs, 16) + 8); }
   void rglru_plan(const LayerInfo &l, int *C, int *TG) const {
     const int nb = (int)T[l.t[3]].dim(0), bs = (int)T[l.t[3]].dim(1);
     const int chunks = std::max(1, W / std::max(nb, 1));
-    *C = std::min(std::min(bs, 64), std::max(8, round_up((bs + chunks - 1) / chunks, 2)));
-    int tg = std::min(nb_max, (int)std::max<int64_t>(8, (int64_t)65536 / (4 * (bs + 2 * *C))));
+    // 16 channels are one tile of the bf16 graphs' gate products
+    *C = std::min(std::min(bs, 64), std::max(8, round_up((bs + chunks - 1) / chunks, g->hybrid == HYB_BF16 ? 16 : 2)));
+    int tg = std::min(nb_max, (int)std::max<int64_t>(8, (int64_t)65536 / rglru_token_bytes(bs, *C)));
     *TG = std::max(1, tg > 8 ? tg / 8 * 8 : tg);
   }
   static int mlstm_tokens(int64_t dim) { return dim <= 512 ? 16 : 8; }
@@ -1010,17 +1015,21 @@ struct Builder {
         if (g->hybrid == HYB_F32) return 8 * T[l.t[1]].dim(3) * 4;
         const int D = xattn_width(l), pitch = D * 2 + 16, keys = D > 128 ? 32 : 64, wmax = D > 128 ? 4 : 8;
         const int G = (int)(l.params[0] / std::max<int64_t>(l.params[1], 1));
-        return (int64_t)std::min(wmax * 16, ext_attention_rows(cfg.max_num_batched_tokens * G)) * pitch + 4 * keys * pitch;
+        return (int64_t)std::min(wmax * 16, ext_attention_rows(cfg.max_num_batched_tokens * G)) * pitch + xattn_stages() * 2 * keys * pitch +
+               kXaCells * 4;
       }
       case MPK_OP_SHORT_CONV: return kMaxLinearTokens * 16 + (mbr + 1) * 4;
       case MPK_OP_RGLRU: {
         int C, TG;
         rglru_plan(l, &C, &TG);
-        return kMaxLinearTokens * 16 + std::max<int64_t>((int64_t)TG * (T[l.t[3]].dim(1) + 2 * C) * 4, (mbr + 1) * 4);
+        const int bs = (int)T[l.t[3]].dim(1);
+        return kMaxLinearTokens * 16 + 1024 + (int64_t)TG * 16 * C + std::max<int64_t>((int64_t)round_up(TG, 8) * 6 * (round_up(bs, 16) + 8), (mbr + 1) * 4);
       }
       case MPK_OP_MLSTM: {
-        const int64_t dim = l.params[1], vc = MPK_MLSTM_COLUMNS(dim), TC = mlstm_tokens(dim);
-        return 4 * (3 * kMaxLinearTokens + TC * 8 + TC * (2 * dim + vc) + TC * 8 * vc);
+        const int64_t dim = l.params[1], vc = MPK_MLSTM_COLUMNS(dim), TC = mlstm_tokens(dim), rows = mlstm_rows((int)dim);
+        const int64_t portion = 4 * (3 * kMaxLinearTokens + TC * 8 + TC * (2 * rows + vc) + TC * 8 * vc);
+        const int64_t single = (int64_t)mlstm_rows_per_thread((int)dim) * kConsumerThreads * 32 + 4 * (2 * rows + 16 * vc + 16);
+        return std::max(portion, single);
       }
       default: return 0;
     }
@@ -1118,9 +1127,9 @@ struct Builder {
     if (std::max(kc.dim(3), vc.dim(3)) > (g->hybrid == HYB_F32 ? 512 : 256))
       return fail(MPK_ERR_UNSUPPORTED, "ext_attention: head sizes up to 256 (512 in 32-bit graphs)");
     const int slots = cfg.max_num_batched_requests, max_seq = std::max(cfg.max_seq_length, 1);
-    // chunks of a (request, kv head): enough to occupy the workers, at most ~2048 keys each, at least 128
+    // chunks of a (request, kv head): enough to occupy the workers, at most ~2048 keys each, at least 64
     int NC = std::max(std::max(1, W / std::max(slots * hkv, 1)), (max_seq + 2047) / 2048);
-    NC = std::min(std::min(NC, std::max(1, max_seq / 128)), 32);
+    NC = std::min(std::min(NC, std::max(1, max_seq / 64)), 32);
     const int srec = vdim + 2;
     for (int s = 0; s < slots; ++s)
       for (int h = 0; h < hkv; ++h)
@@ -1132,10 +1141,12 @@ struct Builder {
           d.a[XA_LDQ] = (int)q.ld(); d.a[XA_LDO] = (int)o.ld(); d.a[XA_OCOL] = ocol;
           d.a[XA_SCALE] = bits_of(l.params[4]); d.a[XA_CAP] = bits_of(l.params[5]); d.a[XA_SINK] = (int)l.params[6];
           d.a[XA_OSCALE] = bits_of(l.params[7]);
-          d.a[XA_TICKET] = hybrid_tickets + s * hkv + h; d.a[XA_SREC] = srec;
+          d.a[XA_TICKET] = hybrid_tickets + (s * hkv + h) * NC;   // one per part of the query rows
+          d.a[XA_SREC] = srec;
+          d.a[XA_STAGES] = xattn_stages();
           put(((s * hkv + h) * NC + ch + rot) % W, d, ex);
         }
-    hybrid_tickets += slots * hkv;
+    hybrid_tickets += slots * hkv * NC;
     g->attn_scratch_floats = std::max<int64_t>(g->attn_scratch_floats, (int64_t)cfg.max_num_batched_tokens * hq * NC * srec);
     return MPK_OK;
   }

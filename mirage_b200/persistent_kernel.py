@@ -554,7 +554,7 @@ class PersistentKernel:
     def mlstm_chunks(num_workers: int, slots: int, heads: int, dim: int, vdim: int) -> int:
         """Column ranges a head's matrix memory is cut into: enough tasks to occupy the workers, at most one per column
         block the task body walks (MPK_MLSTM_COLUMNS of include/mpk_b200.h)."""
-        cols = 64 if dim <= 256 else (32 if dim <= 512 else 16)
+        cols = 64 if dim <= 128 else (32 if dim <= 256 else (16 if dim <= 512 else 8))
         return max(1, min(-(-vdim // cols), num_workers // max(slots * heads, 1)))
 
     def mlstm_layer(self, proj: DTensor, i_bias: DTensor, f_bias: DTensor, norm: DTensor, state: DTensor,

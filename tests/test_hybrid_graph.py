@@ -35,12 +35,12 @@ def test_layer_sequence_and_parallel_branches(dtype, linear):
     types = [e["type"] for e in ev]
     mlstm = ["residual_norm", linear, "mlstm", linear]
     ff = ["residual_norm", linear, linear]
-    par = ["residual_norm", linear, "qkv_append", "ext_attention", "short_conv", "rglru", linear]
+    par = ["residual_norm", linear, "short_conv", "qkv_append", "ext_attention", "rglru", linear]
     assert types == ["batch", "embed_f32"] + mlstm + ff + par + mlstm + ff + par + ff + \
         ["residual_norm", linear, "argmax_partial", "argmax_reduce"]
     deps = lambda i: sorted(d[0] for d in ev[i]["deps"])
     i = types.index("qkv_append")
-    proj, attn, conv, rg, out = i - 1, i + 1, i + 2, i + 3, i + 4
+    proj, attn, conv, rg, out = i - 2, i + 1, i - 1, i + 2, i + 3
     # the branches run side by side: both hang on the projections, only the output linear waits for both
     assert deps(i) == [proj] and deps(attn) == [i] and deps(conv) == [proj] and deps(rg) == [conv] and deps(out) == [attn, rg]
 
