@@ -690,6 +690,173 @@ __device__ __noinline__ void ext_attention_stream(const Ctx c, const TaskDesc &d
   attn_emit_splits<D>(c, d, ao, comb, 16, 8, row0, nrow);
 }
 
+// At most eight query rows (decoding): the transposed products, so that no half of an accumulator is idle.  Sixteen keys
+// are the M rows of S^T = K Q^T and the reduction of O^T = V^T P^T; an 8 x 8 block of P turns from accumulator to operand
+// layout with movmatrix.  Every warp streams its own sixteen-key steps, as two octets, through its ring of four octets.
+__device__ __forceinline__ uint32_t movmatrix_trans(uint32_t v) {
+  uint32_t r;
+  asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
+  return r;
+}
+template <int D>
+__device__ __noinline__ void ext_attention_decode(const Ctx c, const TaskDesc &d, const SeqView sv, const AttnOut &ao, int k0, int k1,
+                                                  int row0, int nrow, int task) {
+  constexpr int PITCH = D * 2 + 16, OCT = 8 * PITCH, PIECES = D / 8, RSTEP = 32 / PIECES, STEPS = 2;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int page = d.a[XA_PAGE];
+  const int kend = min(k1, sv.pos0 + (row0 + nrow - 1) / ao.G + 1);
+  const int nstep = kend > k0 ? (kend - k0 + 15) >> 4 : 0, mine = nstep > warp ? (nstep - warp + 7) >> 3 : 0;
+  uint8_t *qs = c.s.xtile;                                                   // [16][PITCH]
+  // this warp's steps: sixteen K rows, then sixteen V rows
+  const uint32_t ring = smem_u32(qs) + 16 * PITCH + warp * STEPS * 4 * OCT;
+  const int piece = lane % PIECES, rl = lane / PIECES;
+  const uint32_t krow = d.a[XA_HKV] * (d.a[XA_DIMP] >> 3), vrow = d.a[XA_HKV] * (d.a[XA_VDIMP] >> 3);
+  const bool kin = piece < (d.a[XA_DIMP] >> 3), vin = piece < (d.a[XA_VDIMP] >> 3);
+  const uint4 *kg = reinterpret_cast<const uint4 *>(d.p[1]) + ao.head * (d.a[XA_DIMP] >> 3) + piece + rl * krow;
+  const uint4 *vg = reinterpret_cast<const uint4 *>(d.p[2]) + ao.head * (d.a[XA_VDIMP] >> 3) + piece + rl * vrow;
+  const int32_t *pages = c.P.meta.paged_kv_indices + sv.kv0;
+  int pos = k0 + warp * 16;
+  auto page_of = [&](int key) { return key < kend ? __ldcg(pages + key / page) : 0; };
+  int pid0 = page_of(pos), pid1 = page_of(pos + 8);   // of the next step to request
+  auto issue = [&](int slot) {
+    if (pos < kend) {
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int p0 = pos + h * 8, left = kend - p0 - rl;
+        const uint32_t row = (uint32_t)(h ? pid1 : pid0) * page + p0 % page;
+        const uint32_t dst = ring + slot * 4 * OCT + h * OCT + rl * PITCH + piece * 16;
+#pragma unroll
+        for (int i = 0; i < 8 / RSTEP; ++i) {
+          const uint32_t kd = dst + i * RSTEP * PITCH, vd = kd + 2 * OCT;
+          const bool in = i * RSTEP < left;
+          if (in && kin) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(kd), "l"(kg + (size_t)((row + i * RSTEP) * krow)) : "memory");
+          else asm volatile("st.shared.v4.b32 [%0], {%1,%1,%1,%1};" ::"r"(kd), "r"(0) : "memory");
+          if (in && vin) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(vd), "l"(vg + (size_t)((row + i * RSTEP) * vrow)) : "memory");
+          else asm volatile("st.shared.v4.b32 [%0], {%1,%1,%1,%1};" ::"r"(vd), "r"(0) : "memory");
+        }
+      }
+      pos += 128;
+      pid0 = page_of(pos);
+      pid1 = page_of(pos + 8);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  issue(0);
+  issue(1);
+  {
+    const uint8_t *qg = reinterpret_cast<const uint8_t *>(d.p[0]);
+    const int G = ao.G, kp = d.a[XA_DIMP] >> 3;
+    for (int i = tid; i < 8 * PIECES; i += kConsumerThreads) {
+      const int r = i / PIECES, p = i % PIECES, row = row0 + r;
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (r < nrow && p < kp)
+        v = __ldcg(reinterpret_cast<const uint4 *>(qg + ((size_t)(sv.q0 + row / G) * d.a[XA_LDQ] + (size_t)(ao.head * G + row % G) * kp * 8) * 2) + p);
+      *reinterpret_cast<uint4 *>(qs + r * PITCH + p * 16) = v;
+    }
+  }
+  consumer_sync();
+  stamp(c, task, 0);
+  const float scale = __int_as_float(d.a[XA_SCALE]), cap = __int_as_float(d.a[XA_CAP]);
+  const float cap2 = cap > 0.f ? 2.0f * 1.4426950408889634f / cap : 0.f;
+  uint32_t qf[D / 16][2];
+#pragma unroll
+  for (int kk = 0; kk < D / 16; ++kk)
+    ldmatrix_x2(qf[kk], smem_u32(qs) + (uint32_t)((lane & 7) * PITCH + ((lane >> 3) & 1) * 16 + kk * 32));
+  // this lane's two queries (columns of S^T) and the last key each sees
+  const int q0 = row0 + 2 * (lane & 3);
+  const int p_a = sv.pos0 + q0 / ao.G, p_b = sv.pos0 + (q0 + 1) / ao.G, p_all = min(sv.pos0 + row0 / ao.G, kend - 1);
+  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+  float o[D / 16][4];
+#pragma unroll
+  for (int i = 0; i < D / 16; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
+  const uint32_t k_off = (uint32_t)((lane & 15) * PITCH + (lane >> 4) * 16);
+  const uint32_t v_off = (uint32_t)(2 * OCT + ((lane & 7) + (lane >> 4) * 8) * PITCH + ((lane >> 3) & 1) * 16);
+#pragma unroll 1
+  for (int i = 0; i < mine; ++i) {
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncwarp();
+    const uint32_t st = ring + (i & 1) * 4 * OCT;
+    const int key0 = k0 + (warp + 8 * i) * 16;
+    float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int kk = 0; kk < D / 16; ++kk) {
+      uint32_t a[4];
+      ldmatrix_x4(a, st + k_off + kk * 32u);
+      if (kk & 1) mma_bf16_16816(s2, a, qf[kk][0], qf[kk][1]);
+      else mma_bf16_16816(s, a, qf[kk][0], qf[kk][1]);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s[e] = attn_score<HYB_BF16>(s[e] + s2[e], scale, cap, cap2);
+    if (key0 + 15 > p_all) {   // e: key g + 8 (e / 2), query 2 q + (e & 1)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int key = key0 + (lane >> 2) + (e >> 1) * 8;
+        if (key >= kend || key > ((e & 1) ? p_b : p_a)) s[e] = -INFINITY;
+      }
+    }
+    float x0 = fmaxf(s[0], s[2]), x1 = fmaxf(s[1], s[3]);
+#pragma unroll
+    for (int sh = 4; sh < 32; sh <<= 1) {
+      x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, sh));
+      x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, sh));
+    }
+    const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);
+    const float b0 = n0 == -INFINITY ? 0.f : n0, b1 = n1 == -INFINITY ? 0.f : n1;
+    const float c0 = exp2f(m0 - b0), c1 = exp2f(m1 - b1);
+    m0 = n0;
+    m1 = n1;
+    const float p0 = exp2f(s[0] - b0), p1 = exp2f(s[1] - b1), p2 = exp2f(s[2] - b0), p3 = exp2f(s[3] - b1);
+    if (__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) {   // (columns of O^T are queries as well: 2 q, 2 q + 1)
+      l0 *= c0;
+      l1 *= c1;
+#pragma unroll
+      for (int t = 0; t < D / 16; ++t) {
+        o[t][0] *= c0; o[t][1] *= c1;
+        o[t][2] *= c0; o[t][3] *= c1;
+      }
+    }
+    l0 += p0 + p2;
+    l1 += p1 + p3;
+    // weights as a bf16 value and a bf16 remainder
+    const uint32_t h0 = pack_bf16(p0, p1), h1 = pack_bf16(p2, p3);
+    const uint32_t r0 = pack_bf16(p0 - bf16_lo(h0), p1 - bf16_hi(h0)), r1 = pack_bf16(p2 - bf16_lo(h1), p3 - bf16_hi(h1));
+    const uint32_t hb0 = movmatrix_trans(h0), hb1 = movmatrix_trans(h1), rb0 = movmatrix_trans(r0), rb1 = movmatrix_trans(r1);
+#pragma unroll
+    for (int t = 0; t < D / 16; ++t) {
+      uint32_t a[4];
+      ldmatrix_x4_trans(a, st + v_off + t * 32u);
+      mma_bf16_16816(o[t], a, hb0, hb1);
+      mma_bf16_16816(o[t], a, rb0, rb1);
+    }
+    __syncwarp();   // every lane is done with the step that is refilled now
+    issue(i & 1);
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  consumer_sync();   // the rings become the combine area
+  stamp(c, task, 2);
+#pragma unroll
+  for (int sh = 4; sh < 32; sh <<= 1) {
+    l0 += __shfl_xor_sync(0xffffffffu, l0, sh);
+    l1 += __shfl_xor_sync(0xffffffffu, l1, sh);
+  }
+  float *comb = reinterpret_cast<float *>(qs + 16 * PITCH);   // [8 warps][8 queries][D + 2]
+  float *ca = comb + (size_t)(warp * 8 + 2 * (lane & 3)) * (D + 2), *cb = ca + (D + 2);
+  if (lane < 4) {
+    ca[0] = m0; ca[1] = l0;
+    cb[0] = m1; cb[1] = l1;
+  }
+#pragma unroll
+  for (int t = 0; t < D / 16; ++t) {
+    const int col = 2 + t * 16 + (lane >> 2);
+    ca[col] = o[t][0]; cb[col] = o[t][1];
+    ca[col + 8] = o[t][2]; cb[col + 8] = o[t][3];
+  }
+  consumer_sync();
+  attn_emit_splits<D>(c, d, ao, comb, 8, 8, row0, nrow);
+}
+
 // bf16: QK^T and PV on mma.sync.  Head sizes are padded to D columns in shared memory.  The eight warps are split over
 // row tiles (16 rows), key octets and, for D = 256, halves of the output columns; the key split is combined in shared
 // memory.  The probabilities enter PV as a bf16 value and a bf16 remainder, so that the weights keep 16 bits.
@@ -917,11 +1084,13 @@ __device__ __forceinline__ void run_ext_attention(const Ctx &c, const TaskDesc &
     const int w = max(d.a[XA_DIMP], d.a[XA_VDIMP]);
     const bool one = row1 - row0 <= 16 && (d.a[XA_PAGE] & 7) == 0;
     if (w <= 64) {
-      if (one && row1 - row0 <= 8) ext_attention_stream<64, false>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
+      if (one && row1 - row0 <= 8 && d.a[XA_STAGES] >= 3) ext_attention_decode<64>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
+      else if (one && row1 - row0 <= 8) ext_attention_stream<64, false>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
       else if (one) ext_attention_stream<64, true>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
       else ext_attention_mma<64>(c, d, sv, ao, k0, k1, row0, row1, task);
     } else if (w <= 128) {
-      if (one && row1 - row0 <= 8) ext_attention_stream<128, false>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
+      if (one && row1 - row0 <= 8 && d.a[XA_STAGES] >= 3) ext_attention_decode<128>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
+      else if (one && row1 - row0 <= 8) ext_attention_stream<128, false>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
       else if (one) ext_attention_stream<128, true>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
       else ext_attention_mma<128>(c, d, sv, ao, k0, k1, row0, row1, task);
     } else {

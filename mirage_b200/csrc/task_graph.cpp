@@ -1015,8 +1015,10 @@ struct Builder {
         if (g->hybrid == HYB_F32) return 8 * T[l.t[1]].dim(3) * 4;
         const int D = xattn_width(l), pitch = D * 2 + 16, keys = D > 128 ? 32 : 64, wmax = D > 128 ? 4 : 8;
         const int G = (int)(l.params[0] / std::max<int64_t>(l.params[1], 1));
-        return (int64_t)std::min(wmax * 16, ext_attention_rows(cfg.max_num_batched_tokens * G)) * pitch + xattn_stages() * 2 * keys * pitch +
-               kXaCells * 4;
+        const int64_t tile = (int64_t)std::min(wmax * 16, ext_attention_rows(cfg.max_num_batched_tokens * G)) * pitch +
+                             xattn_stages() * 2 * keys * pitch + kXaCells * 4;
+        // decoded tokens of graphs with room for it: sixteen query rows, two steps of 16 keys and values for each warp
+        return std::max(tile, xattn_stages() >= 3 && D <= 128 ? (int64_t)(16 + 8 * 64) * pitch : 0);
       }
       case MPK_OP_SHORT_CONV: return kMaxLinearTokens * 16 + (mbr + 1) * 4;
       case MPK_OP_RGLRU: {
