@@ -105,7 +105,7 @@ typedef enum {
    * are bit patterns.  Linears write float32 where the output tensor is float32; float32 linear inputs or
    * mixer outputs select 32-bit arithmetic for the whole graph. */
   MPK_OP_RESIDUAL_NORM = 32,    /* x += norm(y) | y; out = norm(x)   in: x (f32, in place), y, weight of y's norm, weight of the output norm
-                                   out: out   (all but x optional)   params: [eps, weights stored around zero] */
+                                   out: out, new stream (absent: x in place)   (all but x optional)   params: [eps, weights stored around zero] */
   MPK_OP_QKV_APPEND = 33,       /* rotate q and k, unit RMS norm, append k / v rows   in: projections, cos, sin  out: q, k_cache, v_cache
                                    tensors: proj, q, k_cache, v_cache, cos, sin
                                    params: [hq, hkv, dim, vdim, q_col, k_col, v_col, rotated dims, unit norm, eps] */

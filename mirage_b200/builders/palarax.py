@@ -251,13 +251,18 @@ class PalaraxBuilder:
         if tuple(sd["embed"].shape) != (c.vocab, c.width):
             raise ValueError(f"embedding is {tuple(sd['embed'].shape)}, configuration says {(c.vocab, c.width)}")
         table = self._weight("embed", [sd["embed"]])
-        x = self._buf("stream", c.width, float32)
+        # two stream buffers in turn: a norm reads one and writes the other
+        x, other = self._buf("stream", c.width, float32), self._buf("stream_b", c.width, float32)
         h = self._buf("normed", self._kpad(c.width), self.act)
         mpk.embed_layer(input=mpk.attach_input(mpk.meta_tensors["input_tokens"], name="input_token"), weight=table, output=x,
                         grid_dim=(1, 1, 1), block_dim=(128, 1, 1), input_source=1)
 
-        def norm(y: Optional[str], post: Optional[str], nxt: str):
-            mpk.residual_norm_layer(x, y, self._att(post) if post else None, self._att(nxt), h, eps=c.eps, zero_centered=True)
+        def norm(y: Optional[DTensor], post: Optional[str], nxt: str):
+            nonlocal x, other
+            mpk.residual_norm_layer(x, y, self._att(post) if post else None, self._att(nxt), h, eps=c.eps, zero_centered=True,
+                                    x_out=other if y is not None else None)
+            if y is not None:
+                x, other = other, x
 
         # a sublayer's closing norm and the next one's opening norm are one task
         y, post = None, None

@@ -135,6 +135,7 @@ __device__ __forceinline__ void residual_norm_rows(const Ctx &c, const TaskDesc 
   float *row = reinterpret_cast<float *>(c.s.xtile);
   for (int t = t0; t < t1; ++t) {
     float *x = reinterpret_cast<float *>(d.p[0]) + (size_t)t * d.a[3];
+    float *xo = reinterpret_cast<float *>(d.p[5]) + (size_t)t * d.a[8];
     const float *y = reinterpret_cast<const float *>(d.p[1]) + (size_t)t * d.a[4];
     float inv = 1.f;
     if (has_y && has_post) {
@@ -168,7 +169,7 @@ __device__ __forceinline__ void residual_norm_rows(const Ctx &c, const TaskDesc 
         if (has_y) xv[e] += has_post ? yv[e] * inv * (off + bf16_at(d.p[2], j + e)) : yv[e];
         ss += xv[e] * xv[e];
         row[j + e] = xv[e];
-        if (has_y) x[j + e] = xv[e];
+        if (has_y) xo[j + e] = xv[e];
       }
     }
     if (has_out) {
@@ -206,6 +207,7 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   for (int t = t0; t < t1; ++t) {
     float *x = reinterpret_cast<float *>(d.p[0]) + (size_t)t * d.a[3];
+    float *xo = reinterpret_cast<float *>(d.p[5]) + (size_t)t * d.a[8];
     const float *y = reinterpret_cast<const float *>(d.p[1]) + (size_t)t * d.a[4];
     float4 xv[NV], yv[NV], wp[NV], wn[NV];
 #pragma unroll
@@ -232,7 +234,7 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
         xv[i].x += yv[i].x * inv * ox; xv[i].y += yv[i].y * inv * oy;
         xv[i].z += yv[i].z * inv * oz; xv[i].w += yv[i].w * inv * ow;
         const int j = (i * kConsumerThreads + tid) * 4;
-        if (j < W) *reinterpret_cast<float4 *>(x + j) = xv[i];
+        if (j < W) *reinterpret_cast<float4 *>(xo + j) = xv[i];
       }
     }
     if (has_out) {
@@ -254,12 +256,12 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
 }
 template <int HYB>
 __device__ __noinline__ void run_residual_norm(const Ctx c, const TaskDesc &d) {
-  if (d.a[2] <= 4096 && ((d.a[2] | d.a[3] | d.a[4] | d.a[5]) & 3) == 0 && ((d.p[0] | d.p[1] | d.p[4]) & 15) == 0 &&
+  if (d.a[2] <= 4096 && ((d.a[2] | d.a[3] | d.a[4] | d.a[5] | d.a[8]) & 3) == 0 && ((d.p[0] | d.p[1] | d.p[4] | d.p[5]) & 15) == 0 &&
       ((d.p[2] | d.p[3]) & 7) == 0) {
     residual_norm_wide<HYB>(c, d);
     return;
   }
-  if (((d.a[2] | d.a[3] | d.a[4]) & 3) == 0 && ((d.p[0] | d.p[1]) & 15) == 0) residual_norm_rows<HYB, 4>(c, d);
+  if (((d.a[2] | d.a[3] | d.a[4] | d.a[8]) & 3) == 0 && ((d.p[0] | d.p[1] | d.p[5]) & 15) == 0) residual_norm_rows<HYB, 4>(c, d);
   else residual_norm_rows<HYB, 1>(c, d);
 }
 
@@ -1127,7 +1129,7 @@ __device__ __forceinline__ void short_conv_window(const Ctx &c, const TaskDesc &
 #pragma unroll
     for (int i = 0; i < 8 + kConvWindow; ++i) {   // x[i]: batch token t0 - kConvWindow + i
       const int t = t0 - kConvWindow + i;
-      x[i] = (ok && t >= 0 && i < n + kConvWindow) ? __ldcg(in + (size_t)t * d.a[4] + ch) + ib : 0.f;
+      x[i] = (ok && n > 0 && t >= 0 && i < n + kConvWindow) ? __ldcg(in + (size_t)t * d.a[4] + ch) + ib : 0.f;
     }
 #pragma unroll
     for (int u = 0; u < 8; ++u) {

@@ -387,6 +387,73 @@ __device__ __forceinline__ float gather_row(const Ctx &c, const TaskDesc &d, con
   return ss;
 }
 
+// PRO_RESNORM (hybrid graphs of a few tokens): the stream's residual sum and both norms in the consumer's prologue.  Every
+// task of the layer computes the same rows and writes the same values to x_out, which is another buffer than x.
+__device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d, int B) {
+  constexpr int NV = 4;   // rows of at most 4096 columns, in registers
+  const int tid = threadIdx.x, W = d.a[L_GROUPS], K = d.a[L_K], warp = tid >> 5;
+  const float eps = __int_as_float(d.a[L_EPS]), off = d.a[L_G_SLOT] ? 1.0f : 0.0f;
+  const bool has_y = d.p[6] != 0, has_post = d.p[3] != 0;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  auto weights = [&](uint64_t base, int j) {
+    const uint2 v = __ldg(reinterpret_cast<const uint2 *>(base + 2ull * j));
+    return make_float4(off + bf16_lo(v.x), off + bf16_hi(v.x), off + bf16_lo(v.y), off + bf16_hi(v.y));
+  };
+  auto total = [&](float v, float *slots) {
+    v = warp_sum(v);
+    if ((tid & 31) == 0) slots[warp] = v;
+    consumer_sync();
+    float t = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) t += slots[w];
+    return t;
+  };
+  for (int b = 0; b < B; ++b) {
+    const float *x = reinterpret_cast<const float *>(d.p[1]) + (size_t)b * d.a[L_LDX];
+    const float *y = reinterpret_cast<const float *>(d.p[6]) + (size_t)b * d.a[L_G_LDRES];
+    float *xo = reinterpret_cast<float *>(d.p[7]) + (size_t)b * d.a[L_G_LDOUT];
+    float4 xv[NV], yv[NV], wp[NV], wn[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int j = (i * kConsumerThreads + tid) * 4;
+      const bool in = j < W;
+      yv[i] = in && has_y ? __ldcg(reinterpret_cast<const float4 *>(y + j)) : zero;
+      xv[i] = in ? __ldcg(reinterpret_cast<const float4 *>(x + j)) : zero;
+      wp[i] = in && has_post ? weights(d.p[3], j) : make_float4(1.f, 1.f, 1.f, 1.f);
+      wn[i] = in ? weights(d.p[4], j) : zero;
+    }
+    if (has_y) {
+      float inv = 1.f;
+      if (has_post) {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) ss += yv[i].x * yv[i].x + yv[i].y * yv[i].y + yv[i].z * yv[i].z + yv[i].w * yv[i].w;
+        inv = 1.0f / sqrtf(total(ss, c.s.red) / (float)W + eps);
+      }
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        xv[i].x += yv[i].x * inv * wp[i].x; xv[i].y += yv[i].y * inv * wp[i].y;
+        xv[i].z += yv[i].z * inv * wp[i].z; xv[i].w += yv[i].w * inv * wp[i].w;
+        const int j = (i * kConsumerThreads + tid) * 4;
+        if (j < W) *reinterpret_cast<float4 *>(xo + j) = xv[i];
+      }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
+    const float inv = 1.0f / sqrtf(total(ss, c.s.red + 8) / (float)W + eps);
+    uint8_t *row = c.s.xtile + (size_t)b * (K * 2 + kRowPadBytes);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {   // (the padding columns behind the row come out as zeros)
+      const int j = (i * kConsumerThreads + tid) * 4;
+      if (j < K)
+        *reinterpret_cast<uint2 *>(row + 2 * j) = make_uint2(pack_bf16(xv[i].x * inv * wn[i].x, xv[i].y * inv * wn[i].y),
+                                                             pack_bf16(xv[i].z * inv * wn[i].z, xv[i].w * inv * wn[i].w));
+    }
+    consumer_sync();   // (also: the reduction slots are used again)
+  }
+}
+
 template <int MODE, bool TPX = false>
 __device__ void stage_x(const Ctx &c, const TaskDesc &d, int B, int k0, int KT, const uint4 (&gpre)[2]) {
   constexpr bool WIDE = MODE != 0;
@@ -742,7 +809,8 @@ __device__ __forceinline__ void run_linear(const Ctx &c, const TaskDesc &d, Line
   for (int kt = 0; kt < K; kt += KT) {
     if (B > 0 && !((d.flags & TF_SAME_X_AS_PREV) && !multi_tile)) {
       if (kt > 0) consumer_sync();   // everyone is done reading the previous tile
-      stage_x<WIDE ? 1 : 0, TPX>(c, d, B, kt, KT, gpre);
+      if (HYB && !WIDE && d.a[L_PRO] == PRO_RESNORM) stage_resnorm(c, d, B);
+      else stage_x<WIDE ? 1 : 0, TPX>(c, d, B, kt, KT, gpre);
     }
     if (tid == 0 && prof && kt == 0) P.profiler[(size_t)task * 8 + 4] = globaltimer_ns();
     int gi = 0;

@@ -96,7 +96,8 @@ enum : int {
 };
 
 // prologue applied while staging the activation tile of a linear task
-enum Prologue : int32_t { PRO_PLAIN = 0, PRO_RMSNORM = 1, PRO_SILU_MUL = 2 };
+enum Prologue : int32_t { PRO_PLAIN = 0, PRO_RMSNORM = 1, PRO_SILU_MUL = 2,
+                          PRO_RESNORM = 3 };   // hybrid graphs: x_out = x + norm(y) on the float32 stream, activation = norm(x_out)
 // epilogue of a linear task
 enum Epilogue : int32_t {
   EPI_STORE = 0,        // out = bf16(acc)
@@ -143,6 +144,8 @@ static_assert(sizeof(TaskDesc) == 16 * kDescVecs, "TaskDesc must stay 224 bytes 
 //  a[19] 1 + index of the allreduce whose pushed partials the prologue gathers (0: none); then p[6] residual,
 //        p[7] tensor that receives the reduced activations, a[20] ld residual, a[21] ld of that tensor,
 //        a[22] inbox slot stride of that allreduce (words)
+//  PRO_RESNORM: p[1] x f32  p[3] weight of y's norm or null  p[4] weight of the output norm  p[6] y f32 or null  p[7] x_out f32 (or
+//        null), a[20] ld y, a[21] ld x_out, a[22] 1: weights stored around zero, a[10] width (K minus the zero padding)
 //  a[15] allreduce index within the iteration  a[16] allreduces per iteration  a[17] stride between the two inbox buffers (floats)
 //  tcgen05 path (TF_TC): a[18] rows of one weight tile (the TMA box height, a multiple of 8, at most 128; the task's rows are
 //        cut into ceil(rows / a[18]) tiles, each one 128-lane accumulator), a[12] = 64 x (k blocks of 64 columns per ring slot),
@@ -195,8 +198,8 @@ enum { M_NEXP = 19, M_NTOPK, M_PER_SLOT, M_LDR, M_ESTRIDE };
 // ---- hybrid tasks --------------------------------------------------------------
 // ---- TASK_EMBED_F32: p[0] ids  p[1] table bf16  p[2] out f32;  a[E_*] as TASK_EMBED (a[E_AUX] = vocabulary)
 // ---- TASK_RESIDUAL_NORM: rows [a[0], a[1]), width a[2]; p[0] x f32 (in place)  p[1] y f32 or null  p[2] weight of y's norm or
-//      null (plain sum)  p[3] weight of the output norm or null  p[4] out (bf16, f32 with flag 1) or null;
-//      a[3] ld x  a[4] ld y  a[5] ld out  a[6] eps bits  a[7] flags (1: out f32, 2: weights stored around zero)
+//      null (plain sum)  p[3] weight of the output norm or null  p[4] out (bf16, f32 with flag 1) or null  p[5] new x (= p[0]: in place);
+//      a[3] ld x  a[4] ld y  a[5] ld out  a[6] eps bits  a[7] flags (1: out f32, 2: weights stored around zero)  a[8] ld of the new x
 // ---- TASK_LINEAR_F32: p[0] W bf16 [N, K]  p[1] x f32  p[2] out f32;  a[0] n0  a[1] n1  a[2] K  a[3] ldw  a[4] ld x  a[5] ld out
 //      a[6] activation (0 none, 1 squared relu)  a[7] tokens per shared-memory tile
 // ---- TASK_QKV_APPEND: tokens [a[0], a[1]); p[0] projections f32  p[1] q out  p[2] k cache  p[3] v cache  p[4] cos f32  p[5] sin f32

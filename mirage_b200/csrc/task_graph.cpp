@@ -116,7 +116,8 @@ struct Builder {
         } else {
           add(ins, l.prologue == PRO_PLAIN ? l.t[0] : l.pro_src);
         }
-        if (l.prologue == PRO_RMSNORM) add(ins, l.pro_gamma);
+        if (l.prologue == PRO_RMSNORM || l.prologue == PRO_RESNORM) add(ins, l.pro_gamma);
+        if (l.prologue == PRO_RESNORM) { add(ins, l.pro_y); add(ins, l.pro_post); add(outs, l.pro_xout); }
         add(ins, l.t[1]);
         const int y = l.op == MPK_OP_LINEAR_RESIDUAL ? l.t[3] : l.t[2];
         if (l.op == MPK_OP_LINEAR_RESIDUAL) add(ins, l.t[2]);
@@ -164,7 +165,7 @@ struct Builder {
       case MPK_OP_MLA_REDUCE: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); break;
       case MPK_OP_RESIDUAL_NORM:
         for (int i = 0; i < 4; ++i) add(ins, l.t[i]);
-        if (l.t[1] >= 0) add(outs, l.t[0]);
+        if (l.t[1] >= 0) add(outs, resnorm_out(l));
         add(outs, l.t[4]);
         break;
       case MPK_OP_QKV_APPEND: add(ins, l.t[0]); add(ins, l.t[4]); add(ins, l.t[5]); for (int i = 1; i < 4; ++i) add(outs, l.t[i]); break;
@@ -269,6 +270,48 @@ struct Builder {
           c.pro_groups = std::max(p.grid[0], 1);
         }
       }
+      p.folded = true;
+      g->num_folded++;
+    }
+  }
+
+  // Stream tensor a residual_norm layer writes: its own output (t[5]) or the input in place.
+  static int resnorm_out(const LayerInfo &l) { return l.t.size() > 5 && l.t[5] >= 0 ? l.t[5] : l.t[0]; }
+
+  // Hybrid graphs of one or two tokens: a residual_norm layer whose result feeds linears becomes their prologue, which
+  // spares the chain a task group.  (With more tokens the rows are spread over the workers instead of being formed by all.)
+  void fold_residual_norms() {
+    if (g->hybrid != HYB_BF16 || nb_max > 2 || cfg.max_num_batched_tokens > 2) return;
+    for (size_t i = 0; i < L.size(); ++i) {
+      LayerInfo &p = L[i];
+      if (p.op != MPK_OP_RESIDUAL_NORM || p.t[4] < 0 || p.t[3] < 0) continue;
+      const int x = p.t[0], y = p.t[1], out = p.t[4], xo = resnorm_out(p);
+      auto aligned = [&](int t) { return T[t].ld() % 4 == 0 && ((uint64_t)T[t].ptr & 15) == 0; };
+      const int64_t D = T[x].dim(1);
+      if (T[out].owner == 0 || D > 4096 || D % 4 || !aligned(x) || ((uint64_t)T[p.t[3]].ptr & 7) || p.params.size() < 2) continue;
+      if (y >= 0 && (T[xo].storage == T[x].storage || !aligned(y) || !aligned(xo) || T[xo].dtype != MPK_F32 || T[xo].dim(1) != D)) continue;
+      if (p.t[2] >= 0 && ((uint64_t)T[p.t[2]].ptr & 7)) continue;
+      std::vector<size_t> consumers;
+      bool ok = true;
+      for (size_t j = i + 1; j < L.size() && ok; ++j) {
+        const LayerInfo &c = L[j];
+        if (raw_reads(c, T[out].storage)) {
+          if (c.op != MPK_OP_LINEAR || c.prologue != PRO_PLAIN || c.t[0] != out || T[c.t[1]].dim(1) > 4096 ||
+              linear_tile_bytes(T[c.t[1]].dim(1)) > x_tile_cap()) ok = false;
+          else consumers.push_back(j);
+        }
+        if (raw_writes(c, T[out].storage)) break;
+      }
+      if (!ok || consumers.size() != 1) continue;
+      for (size_t j = i + 1; j < consumers[0] && ok; ++j)   // nothing in between may touch what the prologue reads or writes
+        for (int t : {x, y, xo})
+          if (t >= 0 && (raw_writes(L[j], T[t].storage) || (t == xo && y >= 0 && raw_reads(L[j], T[t].storage)))) ok = false;
+      if (!ok) continue;
+      LayerInfo &c = L[consumers[0]];
+      c.prologue = PRO_RESNORM;
+      c.pro_src = x; c.pro_y = y; c.pro_post = p.t[2]; c.pro_gamma = p.t[3];
+      c.pro_xout = y >= 0 ? xo : -1;
+      c.pro_eps = bits_of(p.params[0]); c.pro_zero = p.params[1] ? 1 : 0;
       p.folded = true;
       g->num_folded++;
     }
@@ -487,7 +530,7 @@ struct Builder {
       ++nkt;
     if (nkt > K / kq) return fail(MPK_ERR_UNSUPPORTED, "cannot tile K for " + w.name);
     const int KT = K / nkt;
-    if (l.prologue == PRO_RMSNORM && nkt != 1)
+    if ((l.prologue == PRO_RMSNORM || l.prologue == PRO_RESNORM) && nkt != 1)
       return fail(MPK_ERR_UNSUPPORTED, "rmsnorm prologue needs the whole row in shared memory: " + w.name);
     // k extent of a streamed chunk: the largest multiple of 16 that divides KT and fits a stage
     // Chunk geometry: 16 rows (one mma m-tile) x KC columns.  The copy engine handles a fixed number of bulk
@@ -503,7 +546,7 @@ struct Builder {
     if (l.prologue == PRO_SILU_MUL) {
       if (x.dim(1) != 2 * (int64_t)K || (K / l.pro_groups) % 8 != 0 || K % l.pro_groups != 0)
         return fail(MPK_ERR_INVALID, "silu_mul feeding " + w.name + ": bad gate|up width or group count");
-    } else if (x.dim(x.dims.size() - 1) != K) {
+    } else if (l.prologue != PRO_RESNORM && x.dim(x.dims.size() - 1) != K) {
       return fail(MPK_ERR_INVALID, "linear input width != K for " + w.name);
     }
     // (hybrid graphs: the output buffer may be padded to the k granularity of the next linear)
@@ -522,7 +565,7 @@ struct Builder {
       epi = EPI_RESIDUAL; res_ptr = (uint64_t)y.ptr; ldr = (int)y.ld();
     }
     if (l.push) epi = l.push_ll ? EPI_PUSH_LL : EPI_PUSH_F32;
-    if (x.dtype != MPK_BF16) return fail(MPK_ERR_UNSUPPORTED, "linear input must be bf16: " + w.name);
+    if (x.dtype != MPK_BF16 && l.prologue != PRO_RESNORM) return fail(MPK_ERR_UNSUPPORTED, "linear input must be bf16: " + w.name);
     if (l.op == MPK_OP_LINEAR && !l.params.empty() && l.params[0] != 0) {
       if (g->hybrid != HYB_BF16 || l.params[0] != 1 || y.dtype != MPK_BF16)
         return fail(MPK_ERR_UNSUPPORTED, "linear activation: squared relu into bf16, in hybrid graphs: " + w.name);
@@ -598,6 +641,15 @@ struct Builder {
           d.a[L_G_LDOUT] = (int)T[l.gather_out].ld();
           d.a[L_G_SLOT] = cfg.max_num_batched_tokens * K;
         }
+        if (l.prologue == PRO_RESNORM) {
+          d.p[3] = l.pro_post >= 0 ? (uint64_t)T[l.pro_post].ptr : 0;
+          d.p[4] = (uint64_t)T[l.pro_gamma].ptr;
+          d.p[6] = l.pro_y >= 0 ? (uint64_t)T[l.pro_y].ptr : 0;
+          d.p[7] = l.pro_xout >= 0 ? (uint64_t)T[l.pro_xout].ptr : 0;
+          d.a[L_G_LDRES] = l.pro_y >= 0 ? (int)T[l.pro_y].ld() : 0;
+          d.a[L_G_LDOUT] = l.pro_xout >= 0 ? (int)T[l.pro_xout].ld() : 0;
+          d.a[L_G_SLOT] = l.pro_zero;
+        }
         d.a[L_N0] = r;
         d.a[L_N1] = std::min(r + task_cap, row + cnt);
         d.a[L_K] = K;
@@ -607,8 +659,8 @@ struct Builder {
         d.a[L_LDR] = ldr;
         d.a[L_PRO] = l.prologue;
         d.a[L_EPI] = epi;
-        d.a[L_EPS] = float_bits(1e-6f);
-        d.a[L_GROUPS] = l.pro_groups;
+        d.a[L_EPS] = l.prologue == PRO_RESNORM ? l.pro_eps : float_bits(1e-6f);
+        d.a[L_GROUPS] = l.prologue == PRO_RESNORM ? (int)x.dim(1) : l.pro_groups;
         d.a[L_KT] = KT;
         d.a[L_KC] = KC;
         d.a[L_ROWS] = R;
@@ -975,7 +1027,7 @@ struct Builder {
     for (size_t i = 0; i < L.size(); ++i) {
       const LayerInfo &l = L[i];
       const int act_out = l.op == MPK_OP_RESIDUAL_NORM || l.op == MPK_OP_EXT_ATTENTION || l.op == MPK_OP_RGLRU || l.op == MPK_OP_MLSTM
-                              ? l.t.back() : -1;   // output of the graph's activation type
+                              ? (l.op == MPK_OP_RESIDUAL_NORM ? l.t[4] : l.t.back()) : -1;   // output of the graph's activation type
       if (act_out >= 0 && T[act_out].dtype == MPK_F32) f32 = true;
       if (hybrid_op(l.op) || l.op == MPK_OP_EMBED || l.op == MPK_OP_ARGMAX_PARTIAL || l.op == MPK_OP_ARGMAX_REDUCE ||
           l.op == MPK_OP_SAMPLING_PARTIAL || l.op == MPK_OP_SAMPLING_REDUCE) continue;
@@ -1069,9 +1121,12 @@ struct Builder {
       if (l.t[i] >= 0 && (T[l.t[i]].dtype != MPK_BF16 || T[l.t[i]].dim(0) != D)) return fail(MPK_ERR_INVALID, "residual_norm: weights must be bf16 [width]");
     if ((l.t[3] >= 0) != (l.t[4] >= 0)) return fail(MPK_ERR_INVALID, "residual_norm: output and its norm weight go together");
     if (l.t[4] >= 0 && (T[l.t[4]].dtype != act_dtype() || T[l.t[4]].dim(1) < D)) return fail(MPK_ERR_INVALID, "residual_norm: output type or width");
+    const TensorInfo &xo = T[resnorm_out(l)];
+    if (xo.dtype != MPK_F32 || xo.dim(1) != D) return fail(MPK_ERR_INVALID, "residual_norm: the new stream must be float32 of x's width");
     const int rows = (int)std::min<int64_t>(x.dim(0), cfg.max_num_batched_tokens), nt = std::min(rows, W);
     for (int i = 0; i < nt; ++i) {
       TaskDesc d = blank(TASK_RESIDUAL_NORM, li);
+      d.p[5] = (uint64_t)xo.ptr; d.a[8] = (int)xo.ld();
       d.p[0] = (uint64_t)x.ptr; d.p[1] = opt(1); d.p[2] = opt(2); d.p[3] = opt(3); d.p[4] = opt(4);
       d.a[0] = (int)((int64_t)rows * i / nt); d.a[1] = (int)((int64_t)rows * (i + 1) / nt); d.a[2] = D;
       d.a[3] = (int)x.ld(); d.a[4] = l.t[1] >= 0 ? (int)T[l.t[1]].ld() : 0; d.a[5] = l.t[4] >= 0 ? (int)T[l.t[4]].ld() : 0;
@@ -1576,6 +1631,7 @@ struct Builder {
     if (rc) return rc;
     for (const auto &l : L) if (l.folded) g->num_folded++;     // folded before materialisation (activation epilogue)
     fold_layers();
+    fold_residual_norms();
     rc = plan_allreduce();
     if (rc) return rc;
     rc = plan_smem();
@@ -1860,7 +1916,7 @@ std::string dump_task_graph(const CompiledGraph &g, const std::vector<TensorInfo
     for (size_t k = 0; k < x.deps.size(); ++k) os << (k ? ", " : "") << "[" << x.deps[k] << ", " << x.dep_need[k] << "]";
     os << "]";
     if (x.layer >= 0 && layers[x.layer].prologue != PRO_PLAIN)
-      os << ", \"prologue\": \"" << (layers[x.layer].prologue == PRO_RMSNORM ? "rmsnorm" : "silu_mul") << "\"";
+      os << ", \"prologue\": \"" << (layers[x.layer].prologue == PRO_RMSNORM ? "rmsnorm" : layers[x.layer].prologue == PRO_RESNORM ? "residual_norm" : "silu_mul") << "\"";
     if (x.layer >= 0 && layers[x.layer].silu_out >= 0) os << ", \"epilogue\": \"silu_mul\"";
     if (x.remote_trigger) os << ", \"push\": true";
     if (x.tc_rows > 0) os << ", \"tcgen05\": {\"tile_rows\": " << x.tc_rows << ", \"k_blocks_per_slot\": " << x.tc_kblocks << "}";

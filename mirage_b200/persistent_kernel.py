@@ -507,11 +507,13 @@ class PersistentKernel:
 
     def residual_norm_layer(self, x: DTensor, y: Optional[DTensor] = None, post_weight: Optional[DTensor] = None,
                             norm_weight: Optional[DTensor] = None, output: Optional[DTensor] = None, eps: float = 1e-6,
-                            zero_centered: bool = False):
+                            zero_centered: bool = False, x_out: Optional[DTensor] = None):
         """x += rmsnorm(y) * w_post on the float32 stream `x` (x += y without `post_weight`, x unchanged without `y`),
-        then output = rmsnorm(x) * w_norm.  `zero_centered`: both weights are stored around zero (1 + w is applied)."""
+        then output = rmsnorm(x) * w_norm.  `zero_centered`: both weights are stored around zero (1 + w is applied).
+        `x_out` receives the new stream instead of `x`; with it, graphs of one or two tokens fold the layer into the linear
+        that reads `output`."""
         assert x.num_dims == 2
-        self._layer(N.OP_RESIDUAL_NORM, [x, y, post_weight, norm_weight, output], (1, 1, 1),
+        self._layer(N.OP_RESIDUAL_NORM, [x, y, post_weight, norm_weight, output, x_out], (1, 1, 1),
                     [self._bits(eps), int(zero_centered)])
 
     def qkv_append_layer(self, proj: DTensor, q: DTensor, k_cache: DTensor, v_cache: DTensor, cos: DTensor, sin: DTensor,

@@ -105,3 +105,16 @@ def test_registry_picks_runner_and_kernel_family_by_config(tmp_path):
     with pytest.raises(KeyError):
         mi.runner_class(str(tmp_path / "u"))
     assert mi.get_builder("Palarax") is PalaraxBuilder
+
+
+def test_norms_fold_into_the_linears_of_single_token_graphs():
+    c = mixed_config()
+    pk = dry(c, mbt=1)
+    pk.compile()
+    ev = json.loads(pk.dump_task_graph())["events"]
+    assert "residual_norm" not in [e["type"] for e in ev]
+    assert sum(e.get("prologue") == "residual_norm" for e in ev) == pk.graph_info()["num_folded"] == 8     # 4 mixers, 3 feed-forwards, head
+    for kw in (dict(mbt=3), dict(mbt=1, dtype=torch.float32)):
+        pk = dry(c, **kw)
+        pk.compile()
+        assert pk.graph_info()["num_folded"] == 0
