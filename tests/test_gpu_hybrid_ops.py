@@ -98,7 +98,7 @@ def sources(width, seed):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads,dim,vdim", [(2, 16, 24), (1, 20, 7), (3, 130, 66), (1, 300, 40), (2, 64, 200)])
+@pytest.mark.parametrize("heads,dim,vdim", [(2, 16, 24), (1, 20, 7), (3, 130, 66), (1, 300, 40), (2, 64, 200), (1, 600, 530), (2, 256, 96)])
 def test_mlstm(dtype, heads, dim, vdim):
     qk, v = heads * dim, heads * vdim
     src = sources(2 * qk + 2 * v + 2 * heads, 11)
@@ -171,6 +171,33 @@ def test_rglru(dtype, blocks, size):
     assert float(out[:, :3].abs().max()) == 0.0
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_rglru_of_a_full_batch_in_several_token_groups(dtype):
+    """64 tokens of four requests against gates so wide that the task takes them in groups that cut through requests."""
+    size = width = 300
+    counts = [[29, 1, 20, 14], [3, 40, 1, 20]]
+    g = torch.Generator().manual_seed(8)
+    bf = lambda *s, std=1.0, mean=0.0: (mean + std * torch.randn(*s, generator=g)).to(torch.bfloat16)
+    ra, ri = bf(1, size, size, std=size ** -0.5), bf(1, size, size, std=size ** -0.5)
+    rab, rib, yb, lam = bf(1, size), bf(1, size), bf(width), bf(width, mean=-4.0)
+    src = [torch.randn(sum(c[r] for c in counts), 2 * width, generator=g).float() for r in range(4)]
+    b = Bench(4, tokens=64)
+    both, u, out = b.zeros(64, 2 * width), b.zeros(64, width), b.zeros(64, width, dtype=dtype)
+
+    class Split:
+        def __setitem__(self, row, v):
+            u[row], both[row] = v[:width].cuda(), v.cuda()
+    b.pk.rglru_layer(b.pk.attach_input(u, name="u"), b.pk.attach_input(both, name="proj"), b.inp(yb, "yb"), b.inp(ra, "ra"),
+                     b.inp(rab, "rab"), b.inp(ri, "ri"), b.inp(rib, "rib"), b.inp(lam, "lam"),
+                     b.pk.attach_input(b.zeros(4, width), name="st"), b.pk.attach_input(out, name="o"), y_col=width)
+    b.pk.compile()
+    got = feed(b, src, Split(), out, counts)
+    for r in range(4):
+        s = src[r].to(D)
+        S = ops.rglru(s[:, :width], ra.to(D), rab.to(D), ri.to(D), rib.to(D), lam.to(D))
+        assert err(got[r], S * ops.gelu_tanh(s[:, width:] + yb.to(D))) < TOL[dtype], r
+
+
 def attention_graph(b, dtype, H, G, dim, rot, base, scale, cap, sink, unit, eps, separate_v=False):
     vdim = dim
     width = (H + G) * dim + (G * vdim if separate_v else 0)
@@ -214,6 +241,20 @@ def test_attention(dtype, H, G, dim, rot, cap, sink, unit, sv):
         # bf16: q, k, v and the result are each rounded once
         assert err(got[r], attention_reference(src[r][:LENGTHS[r]], *args)) < (TOL[dtype] if dtype == torch.float32 else 1.5e-2), r
     assert float(out[:, :2].abs().max()) == 0.0
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,dim", [(8, 2, 128), (16, 1, 128), (4, 4, 96)])
+def test_attention_in_graphs_of_few_tokens(dtype, H, G, dim):
+    """At most eight batched tokens: the streams of one 16-row tile, with the upper rows in use (16 heads) and not."""
+    args = (H, G, dim, dim // 2, 900.0, 0.25, 30.0, True, True, 1e-5)
+    g = torch.Generator().manual_seed(15)
+    src = [torch.randn(n, (H + G) * dim, generator=g).float() for n in (150, 9)]
+    b = Bench(2, tokens=8, page=16, pages=32)
+    proj, out = attention_graph(b, dtype, *args)
+    got = feed(b, src, proj, out[:, 2:], [[8, 0]] * 17 + [[3, 2], [1, 1], [2, 1], [1, 1], [5, 3], [2, 1]])
+    for r in range(2):
+        assert err(got[r], attention_reference(src[r], *args)) < (TOL[dtype] if dtype == torch.float32 else 1.5e-2), r
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
