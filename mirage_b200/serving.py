@@ -55,18 +55,21 @@ class OnlineSession:
         """Runs the next tokens of each request: entries of (id, tokens, want), `want` indexing into `tokens`.  Returns
         per entry the float32 logits [len(want), vocabulary] (host memory).  Requests in `end` give back pages and slot."""
         todo: Dict[int, Tuple[int, int]] = {}                      # row -> (entry, length before this step)
+        ids = [rid for rid, tokens, _ in entries if len(tokens)]
+        if len(set(ids)) != len(ids):
+            raise ValueError("a request appears twice in one step")
+        for rid, tokens, _ in entries:                             # nothing is changed when a step is refused
+            have = self._live[rid].length if rid in self._live else 0
+            if have + len(tokens) >= self.max_length:
+                raise ValueError(f"request {rid!r} outgrows the token table ({self.max_length} positions)")
+        if sum(rid not in self._live for rid in ids) > len(self._free):
+            raise RuntimeError("no free row in the token table: too many live requests")
         for e, (rid, tokens, _) in enumerate(entries):
             if not len(tokens):
                 continue
             req = self._live.get(rid)
             if req is None:
-                if not self._free:
-                    raise RuntimeError("no free row in the token table: too many live requests")
                 req = self._live[rid] = _Request(self._free.pop(0), 0)
-            if req.row in todo:
-                raise ValueError(f"request {rid!r} appears twice in one step")
-            if req.length + len(tokens) >= self.max_length:
-                raise ValueError(f"request {rid!r} outgrows the token table ({self.max_length} positions)")
             todo[req.row] = (e, req.length)
             self.meta["tokens"][req.row, req.length:req.length + len(tokens)] = torch.tensor(
                 list(tokens), dtype=torch.int64, device=self.meta["tokens"].device)

@@ -84,10 +84,12 @@ def test_only_the_wanted_places_come_back_in_their_order(session, model):
 def test_errors_leave_the_session_usable(session, model):
     s, dt = session
     _, _, toks, ref = model
-    with pytest.raises(ValueError):
-        s.step([("x", [1] * 500, [])])
-    if "x" in s._live:
-        s._live.pop("x")
+    for bad in ([("x", [1] * 500, [])], [("x", [1], []), ("x", [2], [])]):
+        with pytest.raises(ValueError):
+            s.step(bad)
+    with pytest.raises(RuntimeError):
+        s.step([(f"x{i}", [1], []) for i in range(9)])
+    assert not s._live and len(s._free) + len(s._closing) == 8
     assert rel(s.step([("y", toks["c"], list(range(17)))], ["y"])[0], ref["c"]) < TOL[dt]
 
 
@@ -239,6 +241,35 @@ def test_online_scheduler_matches_its_oracle_bit_for_bit(model):
         assert eq("request_ctl", st.request_ctl) and eq("input_tokens", st.input_tokens[:st.num_active_tokens]), it
         st.output_tokens[:st.num_active_tokens] = m["output_tokens"].cpu().numpy().reshape(-1)[:st.num_active_tokens]
         assert eq("tokens", st.tokens.reshape(-1)), it
+
+
+def test_online_session_over_another_model():
+    """Qwen3 behind the same session: two requests in portions, one left out of a step, rows used again."""
+    from gpu_util import shape_of
+    from mirage_b200 import OnlineSession
+    from mirage_b200.builders.runner import Qwen3Runner
+    from oracle.qwen3_decoder import Qwen3Config, greedy_generate, make_weights
+    cfg = Qwen3Config.tiny()
+    w = make_weights(cfg, seed=9)
+    rng = random.Random(2)
+    prompts = [rng.choices(range(cfg.vocab_size), k=n) for n in (21, 14)]
+    ref = []
+    for p in prompts:
+        _, _, lg = greedy_generate(cfg, w, [p], 40, max_num_batched_requests=1, max_num_batched_tokens=1, max_num_pages=3, page_size=16,
+                                   max_iterations=len(p), keep_logits=True)
+        ref.append(torch.cat([l[:1] for l in lg]).float())
+    r = Qwen3Runner(shape_of(cfg), w, total_num_requests=4, max_seq_length=40, max_num_batched_requests=2, max_num_batched_tokens=16,
+                    max_num_pages=4, page_size=16, mode="online")
+    s = OnlineSession(r)
+    for turn in range(3):
+        a, b = f"a{turn}", f"b{turn}"
+        out = {0: [], 1: []}
+        for cut in ([(0, 0, 5)], [(0, 5, 6), (1, 0, 9)], [(1, 9, 10)], [(0, 6, 21), (1, 10, 14)]):
+            entries = [((a, b)[k], prompts[k][lo:hi], list(range(hi - lo))) for k, lo, hi in cut]
+            for (k, _, _), l in zip(cut, s.step(entries, [a, b] if cut[-1][2] == 14 else [])):
+                out[k].append(l)
+        for k in (0, 1):
+            assert float((torch.cat(out[k]) - ref[k]).abs().max()) <= 5e-2, (turn, k)
 
 
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
