@@ -57,10 +57,10 @@ typedef enum { MPK_IO_CUDA = 0, MPK_IO_SYMMETRIC = 1 } mpk_io_category;
 /* Layer operators: one per PersistentKernel.*_layer method on the decode path
  * (python/mirage/mpk/persistent_kernel.py, line of each method in the comment). */
 typedef enum {
-  MPK_OP_EMBED = 1,             /* embed_layer              :586  in: ids, table        out: y            params: [input_source]          */
+  MPK_OP_EMBED = 1,             /* embed_layer              :586  in: ids, table        out: y            params: [input_source, factor (hybrid graphs)] */
   MPK_OP_RMSNORM = 2,           /* rmsnorm_layer            :609  in: x, gamma          out: y                                            */
   MPK_OP_RMSNORM_LINEAR = 3,    /* rmsnorm_linear_layer     :627  in: x, gamma, W       out: y                                            */
-  MPK_OP_LINEAR = 4,            /* linear_layer             :1731 in: x, W              out: y            params: optional [activation: 0 none, 1 squared relu (hybrid graphs)] */
+  MPK_OP_LINEAR = 4,            /* linear_layer             :1731 in: x, W              out: y            params: optional [activation, soft cap] (hybrid graphs, mpk_activation)  */
   MPK_OP_LINEAR_RESIDUAL = 5,   /* linear_with_residual_layer :1762 in: x, W, residual  out: y            params: [enable_residual]       */
   MPK_OP_SPLITK_LINEAR = 6,     /* splitk_linear_layer      :1706 in: x, W              out: y (y += x W^T)                               */
   MPK_OP_ATTENTION = 7,         /* attention_layer          :648  in: qkv,k,v,qn,kn,cos,sin out: o       params: [hq, hkv, qk_norm, rope] */
@@ -74,9 +74,11 @@ typedef enum {
   MPK_OP_QUANTIZE_FP8 = 15,     /* quantize_fp8_layer       :1561 in: x               out: x_fp8, scale  params: [scale_ue8m0]            */
   MPK_OP_LINEAR_FP8 = 16,       /* linear_fp8_layer         :1584 in: x_fp8, x_scale, w_fp8, w_scale   out: y                            */
   MPK_OP_LINEAR_FP8_RESIDUAL = 17, /* linear_fp8_with_residual_layer :1611 in: x_fp8, x_scale, w_fp8, w_scale, residual  out: y           */
-  MPK_OP_MOE_TOPK_SIGMOID = 18, /* moe_topk_sigmoid_routing_layer :1408 in: logits, bias  out: topk_weight, routing_indices, mask  params: [num_groups, topk_group, scaling_bits] */
-  MPK_OP_MOE_W13_LINEAR = 19,   /* moe_w13_linear_layer     :1444 in: x, w, routing_indices, mask         out: y [B, topk, 2I]           */
-  MPK_OP_MOE_W2_LINEAR = 20,    /* moe_w2_linear_layer      :1652 in: x [B, topk, I], w, routing_indices, mask  out: y [B, topk, H]      */
+  MPK_OP_MOE_TOPK_SIGMOID = 18, /* moe_topk_sigmoid_routing_layer :1408 in: logits, bias  out: topk_weight, routing_indices, mask  params: [num_groups, topk_group, scaling_bits,
+                                   optional first, end of the experts this rank runs, optional 1: the logits are left as they are] */
+  MPK_OP_MOE_W13_LINEAR = 19,   /* moe_w13_linear_layer     :1444 in: x, w, routing_indices, mask         out: y [B, topk, 2I]  params: [first expert, activation
+                                   (hybrid graphs, mpk_activation: gated forms give y [B, topk, >= I])] */
+  MPK_OP_MOE_W2_LINEAR = 20,    /* moe_w2_linear_layer      :1652 in: x [B, topk, I], w, routing_indices, mask  out: y [B, topk, H] (float32 allowed in hybrid graphs) */
   MPK_OP_MOE_W13_FP8 = 21,      /* moe_w13_fp8_layer        :1475 in: x_fp8, x_scale, w_fp8, w_scale, routing_indices, mask  out: y      */
   MPK_OP_MOE_W2_FP8 = 22,       /* moe_w2_fp8_layer         :1518 in: x_fp8, x_scale, w_fp8, w_scale, routing_indices, mask  out: y      */
   MPK_OP_MOE_SILU_MUL = 23,     /* moe_silu_mul_layer       :1636 in: mid [B, topk, 2I]    out: act [B, topk, I]                         */
@@ -104,20 +106,37 @@ typedef enum {
    * A graph with one of these may hold, besides them, embed, linear, argmax and sampling layers; all floats in params
    * are bit patterns.  Linears write float32 where the output tensor is float32; float32 linear inputs or
    * mixer outputs select 32-bit arithmetic for the whole graph. */
-  MPK_OP_RESIDUAL_NORM = 32,    /* x += norm(y) | y; out = norm(x)   in: x (f32, in place), y, weight of y's norm, weight of the output norm
-                                   out: out, new stream (absent: x in place)   (all but x optional)   params: [eps, weights stored around zero] */
+  MPK_OP_RESIDUAL_NORM = 32,    /* x += sum of the given terms; out = norm(x)   tensors (all but x optional):
+                                   0 x f32  1 y f32  2 weight of y's norm  3 weight of the output norm  4 out  5 new stream (absent: x in place)
+                                   6 bias of the output norm  7 stream added as it is, f32 [tokens, width]  8 row added to every token, bf16 [width]
+                                   9 expert outputs f32 [tokens, slots, width]  10 their weights f32 [tokens, slots]
+                                   11 f32 [tokens, columns]: y is multiplied by sigmoid of column params[3]
+                                   params: [eps, weights stored around zero, 0 RMS norm | 1 layer norm, gate column] */
   MPK_OP_QKV_APPEND = 33,       /* rotate q and k, unit RMS norm, append k / v rows   in: projections, cos, sin  out: q, k_cache, v_cache
                                    tensors: proj, q, k_cache, v_cache, cos, sin
                                    params: [hq, hkv, dim, vdim, q_col, k_col, v_col, rotated dims, unit norm, eps] */
-  MPK_OP_EXT_ATTENTION = 34,    /* tensors: q, k_cache, v_cache, out
-                                   params: [hq, hkv, vdim, out_col, scale, soft cap (0: none), sink, out_scale] */
+  MPK_OP_EXT_ATTENTION = 34,    /* tensors: q, k_cache, v_cache (= k_cache: the leading vdim columns of a key are its value), out, sinks (optional)
+                                   params: [hq, hkv, vdim, out_col, scale, soft cap (0: none), sink, out_scale]
+                                   sink: exp(sinks[head]) joins the softmax denominator (bf16 [hq]; without the tensor: 1) */
   MPK_OP_SHORT_CONV = 35,       /* causal per-channel convolution   tensors: in, in_bias, taps, bias, state, out (biases optional)
                                    params: [in_col, activation: 0 none, 1 silu] */
   MPK_OP_RGLRU = 36,            /* gated diagonal recurrence        tensors: u, proj, y_bias, ra, ra_bias, ri, ri_bias, lambda, state, out
                                    params: [y_col, out_col, out_scale, decay constant] */
-  MPK_OP_MLSTM = 37             /* matrix-memory recurrence         tensors: proj, i_bias, f_bias, norm, state, n_m state, scratch, out
+  MPK_OP_MLSTM = 37,            /* matrix-memory recurrence         tensors: proj, i_bias, f_bias, norm, state, n_m state, scratch, out
                                    params: [heads, dim, vdim, q_col, k_col, v_col, gate_col, i_col, f_col, gate cap, eps, q scale, chunks] */
+  MPK_OP_GLA = 38,              /* gated linear attention, a decay per key channel   tensors: proj, a2, a2_bias, norm, state, scratch, out
+                                   params: [heads, dim, vdim, q_col, k_col, v_col, gate_col, a1_col, 1 / tau, eps, q scale, chunks] */
+  MPK_OP_LATENT_APPEND = 39,    /* latent attention: normed latents and rotated shared keys into the cache, rotated query parts into q
+                                   tensors: proj, latent norm weight, q, cache, cos, sin
+                                   params: [heads, latent size, rotated dims, q_col, kv_col, eps] */
+  MPK_OP_GROUPED_LINEAR = 40    /* one linear per group of columns   in: x [tokens, groups * x stride], W [groups, N, K]  out: y
+                                   params: [x stride, y column, y stride]: group g reads x[:, g * x stride + (0 .. K)] and writes
+                                   y[:, y column + g * y stride + (0 .. N)] */
 } mpk_op;
+
+/* Activations of linear layers in hybrid graphs.  The gated ones take weight rows interleaved as two gate rows, two up rows, and
+ * write act(gate) * up: half as many columns as the weight has rows. */
+typedef enum { MPK_ACT_NONE = 0, MPK_ACT_RELU2 = 1, MPK_ACT_SOFTCAP = 2, MPK_ACT_GATED_SILU = 3, MPK_ACT_GATED_GELU_TANH = 4 } mpk_activation;
 
 /* Value columns a task of an MPK_OP_MLSTM layer walks at a time; the layer's `chunks` parameter (and the second state
  * tensor [slots, heads, chunks, dim + 1]) may be at most ceil(vdim / this).  */

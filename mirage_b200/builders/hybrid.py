@@ -1,0 +1,117 @@
+"""What the builders of hybrid graphs share: buffers and weights padded for the tensor path, rotary tables, the head.
+
+Linear weights of a bf16 graph are padded to a multiple of 64 input columns (the tensor path's k granularity), the activation
+buffers in front of them likewise: what the padding columns hold is finite and meets zero weights.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Any, Dict, List, Optional, Tuple
+
+import torch
+
+from ..persistent_kernel import DTensor, PersistentKernel, bfloat16, float32, int64
+
+
+def round_up(n: int, m: int) -> int:
+    return -(-n // m) * m
+
+
+def k_padded(k: int, dtype: torch.dtype) -> int:
+    """Input columns a linear of a graph with activations of this type gives a weight of `k` columns."""
+    return round_up(k, 64) if dtype == torch.bfloat16 else k
+
+
+def rotary_tables(base: float, dims: int, positions: int, device) -> Tuple[torch.Tensor, torch.Tensor]:
+    """float32 cos / sin [positions, dims / 2] of position * base^(-2i / dims); the angles are formed in 64-bit."""
+    if dims == 0:
+        z = torch.zeros(1, 1, dtype=torch.float32, device=device)
+        return z, z.clone()
+    f = float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+    a = torch.arange(positions, dtype=torch.float64)[:, None] * f
+    return a.cos().float().to(device), a.sin().float().to(device)
+
+
+@dataclass
+class HybridModelConfig:
+    """What a builder needs beside the kernel: shapes, weights under their checkpoint names, state, activation type."""
+    config: Any
+    state_dict: Dict[str, torch.Tensor]
+    state: List[Dict[str, torch.Tensor]]   # one entry per layer run
+    dtype: torch.dtype = torch.bfloat16
+    sampling_seed: Optional[int] = None    # None: greedy argmax; an int: Gumbel-max sampling
+
+    def check_valid(self):
+        assert self.state_dict is not None and len(self.state) >= len(self.config.layers)
+        assert self.dtype in (torch.bfloat16, torch.float32)
+
+
+class HybridBuilder:
+    def __init__(self, mpk: PersistentKernel):
+        self.mpk = mpk
+        self.logits: Optional[DTensor] = None
+        self.hidden: Optional[DTensor] = None      # float32 residual stream
+        self._buffers: Dict[Tuple[str, tuple], DTensor] = {}
+        self._tables: Dict[Tuple[float, int], Tuple[DTensor, DTensor]] = {}
+        self._attached: Dict[str, DTensor] = {}
+
+    def _begin(self, mc: HybridModelConfig):
+        self.sd, self.eps, self.width, self.dtype = mc.state_dict, mc.config.eps, mc.config.width, mc.dtype
+        self.act = float32 if mc.dtype == torch.float32 else bfloat16
+
+    def _buf(self, tag: str, width, dt) -> DTensor:
+        """One buffer per purpose and row shape, shared by all layers."""
+        shape = width if isinstance(width, tuple) else (width,)
+        key = (tag, shape)
+        if key not in self._buffers:
+            self._buffers[key] = self.mpk.new_tensor(dims=(self.mpk.max_num_batched_tokens, *shape), dtype=dt,
+                                                     name="_".join([tag, *map(str, shape)]))
+        return self._buffers[key]
+
+    def _kpad(self, k: int) -> int:
+        return k_padded(k, self.dtype)
+
+    def _attach(self, name: str, make) -> DTensor:
+        """The tensor `make()` gives, once per name: a layer that runs several times has one set of weights."""
+        if name not in self._attached:
+            self._attached[name] = self.mpk.attach_input(make().contiguous(), name=name)
+        return self._attached[name]
+
+    def _weight(self, name: str, parts: List[torch.Tensor], dim: int = 0) -> DTensor:
+        """The parts side by side along `dim`, input columns padded."""
+        return self._attach(name, lambda: self._pad_k(torch.cat(parts, dim) if len(parts) > 1 else parts[0]))
+
+    def _pad_k(self, w: torch.Tensor) -> torch.Tensor:
+        pad = self._kpad(w.shape[-1]) - w.shape[-1]
+        return torch.nn.functional.pad(w, (0, pad)) if pad else w
+
+    def _att(self, name: str) -> DTensor:
+        return self._attach(name, lambda: self.sd[name])
+
+    def _linear(self, x: DTensor, w: DTensor, y: DTensor, activation: str = None, **kw):
+        self.mpk.linear_layer(input=x, weight=w, output=y, grid_dim=(96, 1, 1), block_dim=(128, 1, 1), activation=activation, **kw)
+
+    def _rotary(self, base: float, dims: int) -> Tuple[DTensor, DTensor]:
+        key = (base, dims)
+        if key not in self._tables:
+            dev = self.sd["embed"].device
+            cos, sin = rotary_tables(base, dims, self.mpk.max_seq_length, dev)
+            n = len(self._tables)
+            self._tables[key] = (self.mpk.attach_input(cos, name=f"cos_{n}"), self.mpk.attach_input(sin, name=f"sin_{n}"))
+        return self._tables[key]
+
+    def _head(self, h: DTensor, table: DTensor, vocab: int, sampling_seed: Optional[int], **linear):
+        """Logits from the normed stream, and the layers that choose the next token."""
+        mpk, mbt = self.mpk, self.mpk.max_num_batched_tokens
+        self.logits = mpk.new_tensor(dims=(mbt, vocab), dtype=float32, name="logits")
+        self._linear(h, table, self.logits, **linear)
+        out = mpk.attach_input(mpk.meta_tensors["output_tokens"], name="output_token")
+        if sampling_seed is not None:
+            mpk.sampling_sm100_layer(logits=self.logits, output=out, grid_dim=(mbt, 1, 1), block_dim=(256, 1, 1),
+                                     seed=sampling_seed)
+            return
+        parts = max(1, min(mpk.num_workers, vocab // 64))
+        part_v = mpk.new_tensor(dims=(mbt, parts), dtype=float32, name="argmax_part_value")
+        part_i = mpk.new_tensor(dims=(mbt, parts), dtype=int64, name="argmax_part_index")
+        mpk.argmax_partial_layer(input=self.logits, output=(part_v, part_i), grid_dim=(parts, 1, 1), block_dim=(128, 1, 1))
+        mpk.argmax_reduce_layer(input=(part_v, part_i), output=out, grid_dim=(1, 1, 1), block_dim=(128, 1, 1))

@@ -20,11 +20,8 @@ from typing import Any, Dict, List, Optional, Tuple
 import torch
 
 from ..mpk import register_model_builder
-from ..persistent_kernel import DTensor, PersistentKernel, bfloat16, float32, int64
-
-
-def _round_up(n: int, m: int) -> int:
-    return -(-n // m) * m
+from ..persistent_kernel import DTensor, PersistentKernel, bfloat16, float32
+from .hybrid import HybridBuilder, HybridModelConfig, round_up
 
 
 @dataclass(frozen=True)
@@ -108,16 +105,6 @@ class PalaraxConfig:
             return cls.from_dict(json.load(f))
 
 
-def _rotary_tables(base: float, dims: int, positions: int, device) -> Tuple[torch.Tensor, torch.Tensor]:
-    """float32 cos / sin [positions, dims / 2] of position * base^(-2i / dims); the angles are formed in 64-bit."""
-    if dims == 0:
-        z = torch.zeros(1, 1, dtype=torch.float32, device=device)
-        return z, z.clone()
-    f = float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
-    a = torch.arange(positions, dtype=torch.float64)[:, None] * f
-    return a.cos().float().to(device), a.sin().float().to(device)
-
-
 def allocate_state(c: PalaraxConfig, *, slots: int, max_num_pages: int, page_size: int, dtype: torch.dtype, device,
                    num_workers: int) -> List[Dict[str, torch.Tensor]]:
     """Per layer: what a sequence leaves behind.  Attention caches are paged [pages, page, kv heads, head size rounded up
@@ -128,10 +115,10 @@ def allocate_state(c: PalaraxConfig, *, slots: int, max_num_pages: int, page_siz
         m = layer.mixer
         if isinstance(m, MlstmSpec):
             chunks = PersistentKernel.mlstm_chunks(num_workers, slots, m.heads, m.dim, m.vdim)
-            out.append({"memory": z32(slots, m.heads, m.dim, _round_up(m.vdim, 4)),
+            out.append({"memory": z32(slots, m.heads, m.dim, round_up(m.vdim, 4)),
                         "normaliser": z32(slots, m.heads, chunks, m.dim + 1)})
         else:
-            shape = lambda d: (max_num_pages, page_size, m.left.kv_heads, _round_up(d, 8))
+            shape = lambda d: (max_num_pages, page_size, m.left.kv_heads, round_up(d, 8))
             out.append({"k": torch.zeros(shape(m.left.dim), dtype=dtype, device=device),
                         "v": torch.zeros(shape(m.left.vdim), dtype=dtype, device=device),
                         "conv": z32(slots, max(m.right.taps - 1, 1), m.right.width),
@@ -139,63 +126,11 @@ def allocate_state(c: PalaraxConfig, *, slots: int, max_num_pages: int, page_siz
     return out
 
 
-@dataclass
-class PalaraxModelConfig:
-    """What the builder needs beside the kernel: shapes, weights under their checkpoint names, state, activation type."""
-    config: PalaraxConfig
-    state_dict: Dict[str, torch.Tensor]
-    state: List[Dict[str, torch.Tensor]]
-    dtype: torch.dtype = torch.bfloat16
-    sampling_seed: Optional[int] = None    # None: greedy argmax; an int: Gumbel-max sampling
-
-    def check_valid(self):
-        assert self.state_dict is not None and len(self.state) == len(self.config.layers)
-        assert self.dtype in (torch.bfloat16, torch.float32)
+PalaraxModelConfig = HybridModelConfig
 
 
 @register_model_builder("palarax")
-class PalaraxBuilder:
-    def __init__(self, mpk: PersistentKernel):
-        self.mpk = mpk
-        self.logits: Optional[DTensor] = None
-        self.hidden: Optional[DTensor] = None      # float32 residual stream
-        self._buffers: Dict[Tuple[str, int], DTensor] = {}
-        self._tables: Dict[Tuple[float, int], Tuple[DTensor, DTensor]] = {}
-
-    # -- helpers
-    def _buf(self, tag: str, width: int, dt) -> DTensor:
-        """One buffer per purpose and width, shared by all layers."""
-        key = (tag, width)
-        if key not in self._buffers:
-            self._buffers[key] = self.mpk.new_tensor(dims=(self.mpk.max_num_batched_tokens, width), dtype=dt,
-                                                     name=f"{tag}_{width}")
-        return self._buffers[key]
-
-    def _kpad(self, k: int) -> int:
-        return _round_up(k, 64) if self.act is bfloat16 else k
-
-    def _weight(self, name: str, parts: List[torch.Tensor], dim: int = 0) -> DTensor:
-        """The parts side by side along `dim`, input columns padded."""
-        w = torch.cat(parts, dim) if len(parts) > 1 else parts[0]
-        pad = self._kpad(w.shape[1]) - w.shape[1]
-        w = torch.nn.functional.pad(w, (0, pad)) if pad else w
-        return self.mpk.attach_input(w.contiguous(), name=name)
-
-    def _att(self, name: str) -> DTensor:
-        return self.mpk.attach_input(self.sd[name].contiguous(), name=name)
-
-    def _linear(self, x: DTensor, w: DTensor, y: DTensor, activation: str = None):
-        self.mpk.linear_layer(input=x, weight=w, output=y, grid_dim=(96, 1, 1), block_dim=(128, 1, 1), activation=activation)
-
-    def _rotary(self, base: float, dims: int) -> Tuple[DTensor, DTensor]:
-        key = (base, dims)
-        if key not in self._tables:
-            dev = self.sd["embed"].device
-            cos, sin = _rotary_tables(base, dims, self.mpk.max_seq_length, dev)
-            n = len(self._tables)
-            self._tables[key] = (self.mpk.attach_input(cos, name=f"cos_{n}"), self.mpk.attach_input(sin, name=f"sin_{n}"))
-        return self._tables[key]
-
+class PalaraxBuilder(HybridBuilder):
     # -- mixers: `h` is the normed input; return the mixer's float32 output
     def _mlstm(self, p: str, m: MlstmSpec, st: Dict[str, torch.Tensor], h: DTensor) -> DTensor:
         mpk, sd = self.mpk, self.sd
@@ -245,9 +180,7 @@ class PalaraxBuilder:
 
     def build_from_config(self, mc: PalaraxModelConfig):
         mpk, c, sd = self.mpk, mc.config, mc.state_dict
-        self.sd, self.eps, self.width = sd, c.eps, c.width
-        self.act = float32 if mc.dtype == torch.float32 else bfloat16
-        mbt = mpk.max_num_batched_tokens
+        self._begin(mc)
         if tuple(sd["embed"].shape) != (c.vocab, c.width):
             raise ValueError(f"embedding is {tuple(sd['embed'].shape)}, configuration says {(c.vocab, c.width)}")
         table = self._weight("embed", [sd["embed"]])
@@ -280,15 +213,4 @@ class PalaraxBuilder:
                 self._linear(mid, self._weight(p + "mlp.down.padded", [sd[p + "mlp.down"]]), y)
         norm(y, post, "final.norm")
         self.hidden = x
-        self.logits = mpk.new_tensor(dims=(mbt, c.vocab), dtype=float32, name="logits")
-        self._linear(h, table, self.logits)
-        out = mpk.attach_input(mpk.meta_tensors["output_tokens"], name="output_token")
-        if mc.sampling_seed is not None:
-            mpk.sampling_sm100_layer(logits=self.logits, output=out, grid_dim=(mbt, 1, 1), block_dim=(256, 1, 1),
-                                     seed=mc.sampling_seed)
-            return
-        parts = max(1, min(mpk.num_workers, c.vocab // 64))
-        part_v = mpk.new_tensor(dims=(mbt, parts), dtype=float32, name="argmax_part_value")
-        part_i = mpk.new_tensor(dims=(mbt, parts), dtype=int64, name="argmax_part_index")
-        mpk.argmax_partial_layer(input=self.logits, output=(part_v, part_i), grid_dim=(parts, 1, 1), block_dim=(128, 1, 1))
-        mpk.argmax_reduce_layer(input=(part_v, part_i), output=out, grid_dim=(1, 1, 1), block_dim=(128, 1, 1))
+        self._head(h, table, c.vocab, mc.sampling_seed)

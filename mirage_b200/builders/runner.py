@@ -148,16 +148,21 @@ class Qwen3Runner(DecoderRunner):
                    sampling_seed=sampling_seed, fp8_state_dict=fp8 or None, presharded=True, **kw)
 
 
-class PalaraxRunner(DecoderRunner):
-    """Palarax on one GPU.  `dtype` torch.bfloat16 serves with bf16 matrix operands and KV cache; torch.float32 computes
-    everything in 32-bit floats (same graph, same scheduler, 32-bit task bodies)."""
+class HybridRunner(DecoderRunner):
+    """What the models on hybrid graphs share, on one GPU.  `dtype` torch.bfloat16 serves with bf16 matrix operands and KV
+    cache; torch.float32 computes everything in 32-bit floats (same graph, same scheduler, 32-bit task bodies).  A subclass
+    names its model module: configuration class, builder, builder configuration, state allocation."""
+
+    @classmethod
+    def _model(cls):
+        raise NotImplementedError
 
     def __init__(self, config, state_dict: Dict[str, torch.Tensor], *, total_num_requests: int, max_seq_length: int,
                  max_num_batched_requests: int, max_num_batched_tokens: int, max_num_pages: int, page_size: int,
                  eos_token_id: int = -1, dtype: torch.dtype = torch.bfloat16, device: Optional[int] = None,
                  num_workers: int = 0, sampling_seed: Optional[int] = None, mode: str = "offline",
                  profiler_tensor: Optional[torch.Tensor] = None):
-        from .palarax import PalaraxBuilder, PalaraxModelConfig, allocate_state
+        _, builder, model_config, allocate_state = self._model()
         dev = torch.device("cuda", torch.cuda.current_device() if device is None else device)
         self.device, self.config = dev, config
         sizes = dict(max_num_batched_requests=max_num_batched_requests, max_num_batched_tokens=max_num_batched_tokens,
@@ -169,16 +174,29 @@ class PalaraxRunner(DecoderRunner):
                                     profiler_tensor=profiler_tensor, **sizes)
         self.state = allocate_state(config, slots=max_num_batched_requests, max_num_pages=max_num_pages, page_size=page_size,
                                     dtype=dtype, device=dev, num_workers=self.mpk.num_workers)
-        self.builder = PalaraxBuilder(self.mpk)
-        self.builder.build_from_config(PalaraxModelConfig(config, {k: v.to(dev) for k, v in state_dict.items()}, self.state,
-                                                          dtype, sampling_seed))
+        self.builder = builder(self.mpk)
+        self.builder.build_from_config(model_config(config, {k: v.to(dev) for k, v in state_dict.items()}, self.state,
+                                                    dtype, sampling_seed))
         self.mpk.compile()
         self.logits = self.mpk.tensor_as_torch(self.builder.logits)
         self.vocab_first = 0
 
     @classmethod
-    def from_checkpoint(cls, path: str, **kw) -> "PalaraxRunner":
+    def from_checkpoint(cls, path: str, **kw) -> "HybridRunner":
         """Runner over a checkpoint directory (config.json + *.safetensors); keyword arguments are the constructor's."""
         from .checkpoint import load_sharded_state_dict
-        from .palarax import PalaraxConfig
-        return cls(PalaraxConfig.from_checkpoint(path), load_sharded_state_dict(path)[0], **kw)
+        return cls(cls._model()[0].from_checkpoint(path), load_sharded_state_dict(path)[0], **kw)
+
+
+class PalaraxRunner(HybridRunner):
+    @classmethod
+    def _model(cls):
+        from . import palarax as m
+        return m.PalaraxConfig, m.PalaraxBuilder, m.PalaraxModelConfig, m.allocate_state
+
+
+class LofiraxRunner(HybridRunner):
+    @classmethod
+    def _model(cls):
+        from . import lofirax as m
+        return m.LofiraxConfig, m.LofiraxBuilder, m.LofiraxModelConfig, m.allocate_state

@@ -1,10 +1,11 @@
 // Task bodies of hybrid graphs: decoders whose layers mix softmax attention with recurrent state.
 //
 //   float32 residual stream      TASK_EMBED_F32, TASK_RESIDUAL_NORM
-//   attention                    TASK_QKV_APPEND (rotation, unit norms, cache rows), TASK_EXT_ATTENTION (any head size,
-//                                score scale, soft cap, sink)
-//   recurrences                  TASK_SHORT_CONV, TASK_RGLRU (gated diagonal), TASK_MLSTM (matrix memory)
-//   32-bit graphs                TASK_LINEAR_F32
+//   attention                    TASK_QKV_APPEND (rotation, unit norms, cache rows), TASK_LATENT_APPEND (latent rows that serve
+//                                as keys and values), TASK_EXT_ATTENTION (any head size, score scale, soft cap, sinks)
+//   recurrences                  TASK_SHORT_CONV, TASK_RGLRU (gated diagonal), TASK_MLSTM and TASK_GLA (matrix memories)
+//   experts                      TASK_MOE_ROUTING, TASK_MOE_GEMM (megakernel.cuh); their sum is part of TASK_RESIDUAL_NORM
+//   32-bit graphs                TASK_LINEAR_F32, TASK_MOE_GEMM_F32
 //
 // A recurrent layer keeps its state in float32 tensors indexed by the request's state slot, which the batching task
 // hands out at admission; a request whose batch portion starts at position 0 starts from a zero state, so slots are
@@ -37,9 +38,8 @@ __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + lo
 // Decay factor exp(x), x <= 0, of a recurrence that applies it once per token: near 1 the last-bit error of expf has a
 // sign of its own and adds up over a long memory; 1 + expm1f(x) rounds to nearest.
 __device__ __forceinline__ float decay_exp(float x) { return x > -0.35f ? 1.0f + expm1f(x) : expf(x); }
-__device__ __forceinline__ float gelu_tanh_f(float x) {
-  return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
-}
+// A 64-bit value (pointer) kept in two of a descriptor's integers.
+__device__ __forceinline__ uint64_t wide_arg(const TaskDesc &d, int i) { return *reinterpret_cast<const uint64_t *>(&d.a[i]); }
 __device__ __forceinline__ float warp_max(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
@@ -114,16 +114,39 @@ __device__ __forceinline__ void run_embed_f32(const Ctx &c, const TaskDesc &d) {
   const int t0 = d.a[E_T0], t1 = min(d.a[E_T1], B), width = d.a[E_WIDTH];
   const int64_t *ids = reinterpret_cast<const int64_t *>(d.p[0]);
   float *out = reinterpret_cast<float *>(d.p[2]);
+  const float factor = __int_as_float(d.a[E_LDI2]);
   for (int t = t0; t < t1; ++t) {
     const long long id = __ldcg(reinterpret_cast<const long long *>(&ids[t]));
     const bool in_table = id >= 0 && id < (long long)d.a[E_AUX];   // ids outside the table read as a zero row
     for (int j = threadIdx.x; j < width; j += kConsumerThreads)
-      out[(size_t)t * d.a[E_LDO] + j] = in_table ? bf16_at(d.p[1], (size_t)id * d.a[E_LDI] + j) : 0.f;
+      out[(size_t)t * d.a[E_LDO] + j] = in_table ? bf16_at(d.p[1], (size_t)id * d.a[E_LDI] + j) * factor : 0.f;
   }
 }
 
-// x += norm(y) (or x += y, or nothing), then out = norm(x): one token row at a time.  VEC consecutive elements per
-// thread and step; the row stays in shared memory between the passes (every element is touched by one thread only).
+// What joins the stream beside the sublayer output y (pointers are null where a layer has no such term).
+struct NormTerms {
+  const float *add, *experts, *ew, *gate;   // added stream, expert outputs and their weights, logit whose sigmoid scales y
+  uint64_t row, bias;                       // row added to every token, bias of the output norm
+  int slots;
+};
+__device__ __forceinline__ NormTerms norm_terms(const TaskDesc &d, int t) {
+  NormTerms n;
+  n.slots = d.a[RN_SLOTS];
+  n.add = reinterpret_cast<const float *>(wide_arg(d, RN_ADD));
+  n.experts = reinterpret_cast<const float *>(wide_arg(d, RN_EXP));
+  n.ew = reinterpret_cast<const float *>(wide_arg(d, RN_EW));
+  n.gate = reinterpret_cast<const float *>(wide_arg(d, RN_GATE));
+  if (n.add) n.add += (size_t)t * d.a[RN_LDADD];
+  if (n.experts) n.experts += (size_t)t * n.slots * d.a[2];
+  if (n.ew) n.ew += (size_t)t * d.a[RN_LDEW];
+  if (n.gate) n.gate += (size_t)t * d.a[RN_LDGATE];
+  n.row = wide_arg(d, RN_ROW);
+  n.bias = wide_arg(d, RN_BIAS);
+  return n;
+}
+
+// x += the given terms, then out = norm(x): one token row at a time.  VEC consecutive elements per thread and step; the row
+// stays in shared memory between the passes (every element is touched by one thread only).
 template <int HYB, int VEC>
 __device__ __forceinline__ void residual_norm_rows(const Ctx &c, const TaskDesc &d) {
   typedef typename HybElt<HYB>::T T;
@@ -131,13 +154,16 @@ __device__ __forceinline__ void residual_norm_rows(const Ctx &c, const TaskDesc 
   const int t0 = d.a[0], t1 = min(d.a[1], B), W = d.a[2];
   const float eps = __int_as_float(d.a[6]);
   const float off = (d.a[7] & 2) ? 1.0f : 0.0f;
+  const bool layer_norm = (d.a[7] & 4) != 0;
   const bool has_y = d.p[1] != 0, has_post = d.p[2] != 0, has_out = d.p[3] != 0;
   float *row = reinterpret_cast<float *>(c.s.xtile);
   for (int t = t0; t < t1; ++t) {
     float *x = reinterpret_cast<float *>(d.p[0]) + (size_t)t * d.a[3];
     float *xo = reinterpret_cast<float *>(d.p[5]) + (size_t)t * d.a[8];
     const float *y = reinterpret_cast<const float *>(d.p[1]) + (size_t)t * d.a[4];
-    float inv = 1.f;
+    const NormTerms nt = norm_terms(d, t);
+    const bool moved = has_y || nt.add || nt.experts || nt.row;
+    float inv = nt.gate ? sigmoid_f(__ldcg(nt.gate)) : 1.f;
     if (has_y && has_post) {
       float ss = 0.f;
       for (int j = threadIdx.x * VEC; j < W; j += kConsumerThreads * VEC) {
@@ -153,7 +179,7 @@ __device__ __forceinline__ void residual_norm_rows(const Ctx &c, const TaskDesc 
       }
       inv = 1.0f / sqrtf(block_sum(ss, c.s.red) / (float)W + eps);
     }
-    float ss = 0.f;
+    float ss = 0.f, sum = 0.f;
     for (int j = threadIdx.x * VEC; j < W; j += kConsumerThreads * VEC) {
       float xv[VEC], yv[VEC];
       if (VEC == 4) {
@@ -166,18 +192,31 @@ __device__ __forceinline__ void residual_norm_rows(const Ctx &c, const TaskDesc 
       }
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
-        if (has_y) xv[e] += has_post ? yv[e] * inv * (off + bf16_at(d.p[2], j + e)) : yv[e];
+        if (has_y) xv[e] += has_post ? yv[e] * inv * (off + bf16_at(d.p[2], j + e)) : yv[e] * inv;
+        for (int k = 0; k < nt.slots; ++k) xv[e] = fmaf(__ldcg(nt.ew + k), __ldcg(nt.experts + (size_t)k * W + j + e), xv[e]);
+        if (nt.add) xv[e] += __ldcg(nt.add + j + e);
+        if (nt.row) xv[e] += bf16_at(nt.row, j + e);
         ss += xv[e] * xv[e];
+        sum += xv[e];
         row[j + e] = xv[e];
-        if (has_y) xo[j + e] = xv[e];
+        if (moved) xo[j + e] = xv[e];
       }
     }
     if (has_out) {
+      float mean = 0.f;
+      if (layer_norm) {   // the variance from deviations, not as a difference of two large sums
+        mean = block_sum(sum, c.s.red + 16) / (float)W;
+        ss = 0.f;
+        for (int j = threadIdx.x * VEC; j < W; j += kConsumerThreads * VEC)
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) { const float v = row[j + e] - mean; ss += v * v; }
+      }
       const float inv2 = 1.0f / sqrtf(block_sum(ss, c.s.red + 8) / (float)W + eps);
       T *out = reinterpret_cast<T *>(d.p[4]) + (size_t)t * d.a[5];
       for (int j = threadIdx.x * VEC; j < W; j += kConsumerThreads * VEC) {
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) store_elt(out + j + e, row[j + e] * inv2 * (off + bf16_at(d.p[3], j + e)));
+        for (int e = 0; e < VEC; ++e)
+          store_elt(out + j + e, (row[j + e] - mean) * inv2 * (off + bf16_at(d.p[3], j + e)) + (nt.bias ? bf16_at(nt.bias, j + e) : 0.f));
       }
     }
     consumer_sync();   // the reduction slots are used again by the next row
@@ -203,12 +242,17 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
   const int t0 = d.a[0], t1 = min(d.a[1], B), W = d.a[2], tid = threadIdx.x;
   const float eps = __int_as_float(d.a[6]);
   const float off = (d.a[7] & 2) ? 1.0f : 0.0f;
+  const bool layer_norm = (d.a[7] & 4) != 0;
   const bool has_y = d.p[1] != 0, has_post = d.p[2] != 0, has_out = d.p[3] != 0;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  auto fma4 = [](float4 &a, float w, const float4 &v) {
+    a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
+  };
   for (int t = t0; t < t1; ++t) {
     float *x = reinterpret_cast<float *>(d.p[0]) + (size_t)t * d.a[3];
     float *xo = reinterpret_cast<float *>(d.p[5]) + (size_t)t * d.a[8];
     const float *y = reinterpret_cast<const float *>(d.p[1]) + (size_t)t * d.a[4];
+    const NormTerms nt = norm_terms(d, t);
     float4 xv[NV], yv[NV], wp[NV], wn[NV];
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
@@ -220,7 +264,7 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
       wn[i] = in && has_out ? bf16x4_at(d.p[3], j) : zero;
     }
     if (has_y) {
-      float inv = 1.f;
+      float inv = nt.gate ? sigmoid_f(__ldcg(nt.gate)) : 1.f;
       if (has_post) {
         float ss = 0.f;
 #pragma unroll
@@ -233,11 +277,37 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
                     ow = has_post ? off + wp[i].w : 1.f;
         xv[i].x += yv[i].x * inv * ox; xv[i].y += yv[i].y * inv * oy;
         xv[i].z += yv[i].z * inv * oz; xv[i].w += yv[i].w * inv * ow;
+      }
+    }
+    if (nt.slots > 0 || nt.add || nt.row) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int j = (i * kConsumerThreads + tid) * 4;
+        if (j >= W) break;
+#pragma unroll 4
+        for (int k = 0; k < nt.slots; ++k)
+          fma4(xv[i], __ldcg(nt.ew + k), __ldcg(reinterpret_cast<const float4 *>(nt.experts + (size_t)k * W + j)));
+        if (nt.add) fma4(xv[i], 1.f, __ldcg(reinterpret_cast<const float4 *>(nt.add + j)));
+        if (nt.row) fma4(xv[i], 1.f, bf16x4_at(nt.row, j));
+      }
+    }
+    if (has_y || nt.slots > 0 || nt.add || nt.row) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
         const int j = (i * kConsumerThreads + tid) * 4;
         if (j < W) *reinterpret_cast<float4 *>(xo + j) = xv[i];
       }
     }
     if (has_out) {
+      if (layer_norm) {
+        float sum = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) sum += xv[i].x + xv[i].y + xv[i].z + xv[i].w;
+        const float mean = block_sum(sum, c.s.red + 16) / (float)W;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+          if ((i * kConsumerThreads + tid) * 4 < W) { xv[i].x -= mean; xv[i].y -= mean; xv[i].z -= mean; xv[i].w -= mean; }
+      }
       float ss = 0.f;
 #pragma unroll
       for (int i = 0; i < NV; ++i) ss += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
@@ -246,9 +316,10 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int j = (i * kConsumerThreads + tid) * 4;
-        if (j < W)
-          store_elt4(out + j, make_float4(xv[i].x * inv * (off + wn[i].x), xv[i].y * inv * (off + wn[i].y), xv[i].z * inv * (off + wn[i].z),
-                                          xv[i].w * inv * (off + wn[i].w)));
+        if (j >= W) break;
+        const float4 b = nt.bias ? bf16x4_at(nt.bias, j) : zero;
+        store_elt4(out + j, make_float4(xv[i].x * inv * (off + wn[i].x) + b.x, xv[i].y * inv * (off + wn[i].y) + b.y,
+                                        xv[i].z * inv * (off + wn[i].z) + b.z, xv[i].w * inv * (off + wn[i].w) + b.w));
       }
     }
     if (t + 1 < t1) consumer_sync();   // the reduction slots are used again by the next row
@@ -257,7 +328,8 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
 template <int HYB>
 __device__ __noinline__ void run_residual_norm(const Ctx c, const TaskDesc &d) {
   if (d.a[2] <= 4096 && ((d.a[2] | d.a[3] | d.a[4] | d.a[5] | d.a[8]) & 3) == 0 && ((d.p[0] | d.p[1] | d.p[4] | d.p[5]) & 15) == 0 &&
-      ((d.p[2] | d.p[3]) & 7) == 0) {
+      ((d.p[2] | d.p[3] | wide_arg(d, RN_BIAS) | wide_arg(d, RN_ROW)) & 7) == 0 && (d.a[RN_LDADD] & 3) == 0 &&
+      ((wide_arg(d, RN_ADD) | wide_arg(d, RN_EXP)) & 15) == 0) {
     residual_norm_wide<HYB>(c, d);
     return;
   }
@@ -266,12 +338,54 @@ __device__ __noinline__ void run_residual_norm(const Ctx c, const TaskDesc &d) {
 }
 
 // ---------------------------------------------------------------------------
-// linear layer in 32-bit arithmetic: one warp per weight row, eight tokens at a time
+// linear layers in 32-bit arithmetic: one warp per output column (one weight row, or a gate row and its up row), eight tokens
+// at a time
 // ---------------------------------------------------------------------------
-__device__ __forceinline__ void run_linear_f32(const Ctx &c, const TaskDesc &d) {
+// Products of weight row `wrow` with eight rows of xs [nt][K], starting at t8: acc[u] belongs to token min(t8 + u, nt - 1), its
+// sum over the lanes is still to be taken.
+__device__ __forceinline__ void dot8_f32(uint64_t w, size_t wrow, const float *xs, int K, int t8, int nt, float (&acc)[8]) {
+  const float *xr[8];
+#pragma unroll
+  for (int u = 0; u < 8; ++u) {
+    acc[u] = 0.f;
+    xr[u] = xs + (size_t)min(t8 + u, nt - 1) * K;
+  }
+  for (int k = threadIdx.x & 31; k < K; k += 32) {
+    const float v = bf16_at(w, wrow + k);
+#pragma unroll
+    for (int u = 0; u < 8; ++u) acc[u] = fmaf(v, xr[u][k], acc[u]);
+  }
+}
+// Output column n of `nt` tokens in xs; emit(t, value) is called by one lane.  W points to the weight's first row.
+template <class F>
+__device__ __forceinline__ void column_f32(uint64_t w, size_t ldw, const float *xs, int K, int n, int nt, int act, float cap, F emit) {
+  const int lane = threadIdx.x & 31;
+  const bool gated = act >= ACT_GATED_SILU;
+  const size_t row = gated ? (size_t)(n >> 1) * 4 + (n & 1) : n;
+  for (int t8 = 0; t8 < nt; t8 += 8) {
+    float acc[8], up[8];
+    dot8_f32(w, row * ldw, xs, K, t8, nt, acc);
+    if (gated) dot8_f32(w, (row + 2) * ldw, xs, K, t8, nt, up);
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+      float v = warp_sum(acc[u]);
+      if (gated) {
+        const float g = warp_sum(up[u]);
+        v = (act == ACT_GATED_SILU ? silu_exact_f(v) : gelu_tanh_f(v)) * g;
+      } else if (act == ACT_RELU2) {
+        v = fmaxf(v, 0.f);
+        v *= v;
+      } else if (act == ACT_SOFTCAP) {
+        v = cap * tanhf(v / cap);
+      }
+      if (lane == u && t8 + u < nt) emit(t8 + u, v);
+    }
+  }
+}
+__device__ __noinline__ void run_linear_f32(const Ctx c, const TaskDesc &d) {
   const int B = active_tokens(c.P);
-  const int n0 = d.a[0], n1 = d.a[1], K = d.a[2], act = d.a[6], TT = d.a[7];
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int n0 = d.a[0], n1 = d.a[1], K = d.a[2], TT = d.a[7];
+  const int tid = threadIdx.x, warp = tid >> 5;
   float *xs = reinterpret_cast<float *>(c.s.xtile);   // [TT][K]
   const float *x = reinterpret_cast<const float *>(d.p[1]);
   float *out = reinterpret_cast<float *>(d.p[2]);
@@ -281,30 +395,63 @@ __device__ __forceinline__ void run_linear_f32(const Ctx &c, const TaskDesc &d) 
     for (int t = 0; t < nt; ++t)
       for (int k = tid; k < K; k += kConsumerThreads) xs[(size_t)t * K + k] = __ldcg(x + (size_t)(tb + t) * d.a[4] + k);
     consumer_sync();
-    for (int n = n0 + warp; n < n1; n += 8) {
-      const size_t wrow = (size_t)n * d.a[3];
-      for (int t8 = 0; t8 < nt; t8 += 8) {
-        float acc[8];
-        const float *xr[8];
-#pragma unroll
-        for (int u = 0; u < 8; ++u) {
-          acc[u] = 0.f;
-          xr[u] = xs + (size_t)min(t8 + u, nt - 1) * K;
-        }
-        for (int k = lane; k < K; k += 32) {
-          const float w = bf16_at(d.p[0], wrow + k);
-#pragma unroll
-          for (int u = 0; u < 8; ++u) acc[u] = fmaf(w, xr[u][k], acc[u]);
-        }
-#pragma unroll
-        for (int u = 0; u < 8; ++u) {
-          float v = warp_sum(acc[u]);
-          if (act == 1) { v = fmaxf(v, 0.f); v *= v; }
-          if (lane == u && t8 + u < nt) out[(size_t)(tb + t8 + u) * d.a[5] + n] = v;
-        }
+    for (int n = n0 + warp; n < n1; n += 8)
+      column_f32(d.p[0], d.a[3], xs, K, n, nt, d.a[6], __int_as_float(d.a[8]), [&](int t, float v) { out[(size_t)(tb + t) * d.a[5] + n] = v; });
+  }
+}
+// Expert projections: the active experts one after the other, the tokens routed to each gathered in shared memory.
+__device__ __noinline__ void run_moe_gemm_f32(const Ctx c, const TaskDesc &d) {
+  const int B = min(active_tokens(c.P), kMaxLinearTokens);
+  const int n0 = d.a[0], n1 = d.a[1], K = d.a[2], TT = d.a[7], slots = d.a[9], ldr = d.a[10], E = d.a[11];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int *routing = reinterpret_cast<const int *>(d.p[4]), *active = reinterpret_cast<const int *>(d.p[5]);
+  float *xs = reinterpret_cast<float *>(c.s.xtile);                      // [TT][K]
+  int *list = reinterpret_cast<int *>(xs + (size_t)TT * K);              // [64] token * slots + slot
+  const float *x = reinterpret_cast<const float *>(d.p[1]);
+  float *out = reinterpret_cast<float *>(d.p[2]);
+  const int n_act = min(__ldcg(&active[E]), E);
+  for (int j = 0; j < n_act; ++j) {
+    const int e = __ldcg(&active[j]);
+    consumer_sync();   // the previous expert's readers are done
+    if (warp == 0) {
+      int cnt = 0;
+      for (int b = 0; b < B; b += 32) {
+        const int r = b + lane < B ? __ldcg(&routing[(size_t)e * ldr + b + lane]) : 0;
+        const unsigned bal = __ballot_sync(0xffffffffu, r != 0);
+        if (r != 0) list[cnt + __popc(bal & ((1u << lane) - 1u))] = (b + lane) * slots + r - 1;
+        cnt += __popc(bal);
       }
+      if (lane == 0) c.s.flags[8] = cnt;
+    }
+    consumer_sync();
+    const int cnt = c.s.flags[8];
+    for (int tb = 0; tb < cnt; tb += TT) {
+      const int nt = min(TT, cnt - tb);
+      if (tb > 0) consumer_sync();
+      for (int t = 0; t < nt; ++t) {
+        const int it = list[tb + t];
+        const float *xr = x + (size_t)(d.a[8] ? it : it / slots) * d.a[4];
+        for (int k = tid; k < K; k += kConsumerThreads) xs[(size_t)t * K + k] = __ldcg(xr + k);
+      }
+      consumer_sync();
+      for (int n = n0 + warp; n < n1; n += 8)
+        column_f32(d.p[0] + (uint64_t)e * d.a[12] * K * 2, K, xs, K, n, nt, d.a[6], 0.f,
+                   [&](int t, float v) { out[(size_t)list[tb + t] * d.a[5] + n] = v; });
     }
   }
+}
+
+// The request batch token t belongs to: as many requests end at or before the token.  Called by a whole warp.
+__device__ __forceinline__ int request_of(const KernelParams &P, int t) {
+  const int lane = threadIdx.x & 31, mbr = P.max_num_batched_requests;
+  int k = 0;
+  for (int b = 0; b < mbr; b += 32) {
+    const bool before = b + lane < mbr && __ldcg(&P.meta.qo_indptr[b + lane + 1]) <= t;
+    const int n = __popc(__ballot_sync(0xffffffffu, before));
+    k += n;
+    if (n < 32) break;
+  }
+  return k;
 }
 
 // ---------------------------------------------------------------------------
@@ -320,18 +467,10 @@ __device__ __noinline__ void run_qkv_append(const Ctx c, const TaskDesc &d) {
   const int hq = d.a[QA_HQ], hkv = d.a[QA_HKV], dim = d.a[QA_DIM], dimp = d.a[QA_DIMP], vdim = d.a[QA_VDIM], vdimp = d.a[QA_VDIMP];
   const int rot = d.a[QA_ROT], half = rot >> 1, page = d.a[QA_PAGE];
   const float eps = __int_as_float(d.a[QA_EPS]);
-  const int mbr = P.max_num_batched_requests;
   const int heads = hq + hkv, first = d.a[QA_T0], tasks = d.a[QA_T1];
   for (int item = first * 8 + warp; item < B * heads; item += tasks * 8) {
     const int t = item / heads, h = item - t * heads;
-    int k = 0;   // the request this token belongs to: as many requests end at or before the token
-    for (int b = 0; b < mbr; b += 32) {
-      const bool before = b + lane < mbr && __ldcg(&P.meta.qo_indptr[b + lane + 1]) <= t;
-      const int n = __popc(__ballot_sync(0xffffffffu, before));
-      k += n;
-      if (n < 32) break;
-    }
-    const SeqView s = seq_view(P, k);
+    const SeqView s = seq_view(P, request_of(P, t));
     const int pos = s.pos0 + t - s.q0;
     const bool is_q = h < hq;
     const float *src = reinterpret_cast<const float *>(d.p[0]) + (size_t)t * d.a[QA_LDP] +
@@ -366,6 +505,49 @@ __device__ __noinline__ void run_qkv_append(const Ctx c, const TaskDesc &d) {
 }
 
 // ---------------------------------------------------------------------------
+// TASK_LATENT_APPEND: one warp per (token, head) rotates the head's rotary query part into its columns of q (behind the
+// `rank` latent columns, which a grouped linear writes); one more warp per token writes the token's cache row: the latent,
+// RMS-normed, and the rotated key part all heads share.
+// ---------------------------------------------------------------------------
+template <int HYB>
+__device__ __noinline__ void run_latent_append(const Ctx c, const TaskDesc &d) {
+  typedef typename HybElt<HYB>::T T;
+  const KernelParams &P = c.P;
+  const int B = active_tokens(P);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int H = d.a[LA_H], rank = d.a[LA_RANK], rot = d.a[LA_ROT], half = rot >> 1, dimp = d.a[LA_DIMP], page = d.a[LA_PAGE];
+  for (int item = d.a[LA_T0] * 8 + warp; item < B * (H + 1); item += d.a[LA_T1] * 8) {
+    const int t = item / (H + 1), h = item - t * (H + 1);
+    const SeqView s = seq_view(P, request_of(P, t));
+    const int pos = s.pos0 + t - s.q0;
+    const float *row = reinterpret_cast<const float *>(d.p[0]) + (size_t)t * d.a[LA_LDP];
+    const float *src;   // what is rotated
+    T *dst;
+    if (h < H) {
+      src = row + d.a[LA_QOFF] + h * rot;
+      dst = reinterpret_cast<T *>(d.p[2]) + (size_t)t * d.a[LA_LDQ] + (size_t)h * dimp + rank;
+    } else {
+      const float *lat = row + d.a[LA_KVOFF];
+      const int pg = pos / page;
+      T *cell = reinterpret_cast<T *>(d.p[3]) + ((size_t)__ldcg(&P.meta.paged_kv_indices[s.kv0 + pg]) * page + (pos - pg * page)) * dimp;
+      float ss = 0.f;
+      for (int i = lane; i < rank; i += 32) { const float v = __ldcg(lat + i); ss += v * v; }
+      const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)rank + __int_as_float(d.a[LA_EPS]));
+      for (int i = lane; i < rank; i += 32) store_elt(cell + i, __ldcg(lat + i) * inv * bf16_at(d.p[1], i));
+      src = lat + rank;
+      dst = cell + rank;
+    }
+    const size_t trow = (size_t)min(pos, d.a[LA_ROWS] - 1) * half;
+    const float *cosT = reinterpret_cast<const float *>(d.p[4]) + trow, *sinT = reinterpret_cast<const float *>(d.p[5]) + trow;
+    for (int i = lane; i < half; i += 32) {
+      const float u = __ldcg(src + i), v = __ldcg(src + i + half), cs = __ldg(cosT + i), sn = __ldg(sinT + i);
+      store_elt(dst + i, u * cs - v * sn);
+      store_elt(dst + i + half, v * cs + u * sn);
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------
 // TASK_EXT_ATTENTION: (request, kv head, chunk of the keys).  The M rows of a task are the (token, query head of the
 // group) pairs, row r = token r / G, head r % G.  Chunks are merged by the last task of the (request, kv head) to
 // arrive.  Scores live in base 2 (bf16) or base e (float32): exp_dom undoes the same base everywhere.
@@ -383,6 +565,11 @@ __device__ __forceinline__ float attn_score(float dot, float scale, float cap, f
   return s * 1.4426950408889634f;
 }
 
+// Logit of the sink that joins head h's denominator, in the domain's base.
+template <int HYB>
+__device__ __forceinline__ float sink_logit(const TaskDesc &d, int h) {
+  return d.p[4] ? bf16_at(d.p[4], h) * (HYB == HYB_F32 ? 1.0f : 1.4426950408889634f) : 0.f;
+}
 struct AttnOut {   // where a task's rows go
   int hq, G, head, q0, NC, chunk, n_act, vdim, ldo, ocol, srec;
   float oscale;
@@ -395,9 +582,10 @@ __device__ __forceinline__ void attn_emit_row(const Ctx &c, const TaskDesc &d, c
   const int lane = threadIdx.x & 31;
   const int tok = o.q0 + r / o.G, hq_idx = o.head * o.G + r % o.G;
   if (o.n_act == 1) {
-    const float M = o.sink ? fmaxf(m, 0.f) : m;
+    const float sk = o.sink ? sink_logit<HYB>(d, hq_idx) : 0.f;
+    const float M = o.sink ? fmaxf(m, sk) : m;
     const float w = m == -INFINITY ? 0.f : exp_dom<HYB>(m - M);
-    const float L = l * w + (o.sink ? exp_dom<HYB>(-M) : 0.f);
+    const float L = l * w + (o.sink ? exp_dom<HYB>(sk - M) : 0.f);
     const float f = L > 0.f ? w / L * o.oscale : 0.f;
     T *out = reinterpret_cast<T *>(d.p[3]) + (size_t)tok * o.ldo + o.ocol + (size_t)hq_idx * o.vdim;
     for (int j0 = 0; j0 < o.vdim; j0 += 32) {   // (val may shuffle: the whole warp calls it)
@@ -451,9 +639,10 @@ __device__ __noinline__ void attn_merge(const Ctx c, const TaskDesc &d, const At
       for (int u = 0; u < 16; ++u) x2[u] = (16 + u < o.n_act && j < o.vdim) ? __ldcg(rec + (size_t)(16 + u) * o.srec + 2 + j) : 0.f;
     }
     float M = warp_max(m);
-    if (o.sink) M = fmaxf(M, 0.f);
+    const float sk = o.sink ? sink_logit<HYB>(d, hq_idx) : 0.f;
+    if (o.sink) M = fmaxf(M, sk);
     const float w = m == -INFINITY ? 0.f : exp_dom<HYB>(m - M);
-    const float L = warp_sum(l * w) + (o.sink ? exp_dom<HYB>(-M) : 0.f);
+    const float L = warp_sum(l * w) + (o.sink ? exp_dom<HYB>(sk - M) : 0.f);
     const float f = L > 0.f ? o.oscale / L : 0.f;
     float acc = 0.f;
 #pragma unroll
@@ -1475,11 +1664,11 @@ __device__ __forceinline__ float mlstm_log_i(float pre, float cap) { return cap 
 __device__ __forceinline__ float mlstm_log_f(float pre, float cap) { return -softplus_f(-cap * tanhf(pre / cap)); }
 
 // True for the task that finishes a (request, head).  Ends with a barrier.
-__device__ __forceinline__ bool mlstm_last(const Ctx &c, const TaskDesc &d, int chunks) {
+__device__ __forceinline__ bool last_of_head(const Ctx &c, int ticket_id, int chunks) {
   consumer_sync();
   if (chunks == 1) return true;
   if (threadIdx.x == 0) {
-    unsigned int *ticket = &c.P.attn_tickets[d.a[ML_TICKET]];
+    unsigned int *ticket = &c.P.attn_tickets[ticket_id];
     unsigned int old;
     asm volatile("atom.acq_rel.gpu.global.add.u32 %0, [%1], 1;" : "=r"(old) : "l"(ticket) : "memory");
     const bool last = old + 1u == (unsigned)chunks;
@@ -1648,7 +1837,7 @@ __device__ __noinline__ void mlstm_portion(const Ctx c, const TaskDesc &d, const
   }
   stamp(c, task, 1);
   // ---- output of the head
-  if (!mlstm_last(c, d, m.chunks)) return;
+  if (!last_of_head(c, d.a[ML_TICKET], m.chunks)) return;
   stamp(c, task, 2);
   const float eps = __int_as_float(d.a[ML_EPS]);
   T *out = reinterpret_cast<T *>(d.p[7]) + (size_t)sv.q0 * d.a[ML_LDO] + (size_t)m.h * m.vdim;
@@ -1768,7 +1957,7 @@ __device__ __noinline__ void mlstm_single(const Ctx c, const TaskDesc &d, const 
     }
   }
   stamp(c, task, 1);
-  if (!mlstm_last(c, d, m.chunks)) return;
+  if (!last_of_head(c, d.a[ML_TICKET], m.chunks)) return;
   stamp(c, task, 2);
   const float *gt = m.proj + d.a[ML_GOFF] + (size_t)m.h * m.vdim;
   T *out = reinterpret_cast<T *>(d.p[7]) + (size_t)sv.q0 * d.a[ML_LDO] + (size_t)m.h * m.vdim;
@@ -1797,6 +1986,283 @@ __device__ __forceinline__ void run_mlstm(const Ctx &c, const TaskDesc &d, int t
     case 8: mlstm_body<HYB, 8, 8>(c, d, sv, task); break;
     case 4: mlstm_body<HYB, 4, 8>(c, d, sv, task); break;
     default: mlstm_body<HYB, 2, 8>(c, d, sv, task); break;
+  }
+}
+
+// ---------------------------------------------------------------------------
+// TASK_GLA: (request, head, range of value columns).  Gated linear attention: the matrix memory S [dim, columns] decays by a
+// factor per key channel,
+//   S = diag(alpha) S + k v^T, o = S^T q,  alpha = sigmoid(a2 (a1 h) + b)^(1 / tau)
+// Thread layout and column walk are those of TASK_MLSTM.  The low-rank decay product is part of the task: a1 h is read from
+// the projections, a2's rows of the head from the weight.  The last task of the (request, head) to finish writes the head's
+// normed and gated output.
+// ---------------------------------------------------------------------------
+struct GlaView {
+  const float *proj;   // projections of the request's first token
+  float *S, *raw;
+  int ldp, H, h, dim, vdim, vdimp, V0, V1, chunks, rank;
+  bool fresh;
+};
+__device__ __forceinline__ GlaView gla_view(const TaskDesc &d, const SeqView &sv) {
+  GlaView m;
+  m.ldp = d.a[GA_LDP]; m.H = d.a[GA_H]; m.h = d.a[GA_HEAD]; m.dim = d.a[GA_DIM]; m.vdim = d.a[GA_VDIM]; m.vdimp = d.a[GA_VDIMP];
+  m.V0 = d.a[GA_V0]; m.V1 = d.a[GA_V1]; m.chunks = d.a[GA_NCHUNK]; m.rank = d.a[GA_RANK];
+  m.fresh = sv.pos0 == 0;
+  m.proj = reinterpret_cast<const float *>(d.p[0]) + (size_t)sv.q0 * m.ldp;
+  m.S = reinterpret_cast<float *>(d.p[4]) + (size_t)(sv.slot * m.H + m.h) * m.dim * m.vdimp;
+  m.raw = reinterpret_cast<float *>(d.p[6]) + (size_t)sv.q0 * d.a[GA_LDR] + (size_t)m.h * m.vdim;
+  return m;
+}
+__device__ __forceinline__ float gla_decay(float z, float inv_tau) { return decay_exp(-softplus_f(-z) * inv_tau); }
+
+// One step of S and the read-out for this thread's rows.
+template <int RPT>
+__device__ __forceinline__ float4 gla_step(float4 (&S)[RPT], const float *at, const float4 v, const float *kt, const float *qt) {
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < RPT; i += 4) {
+    const float4 a4 = *reinterpret_cast<const float4 *>(at + i), k4 = *reinterpret_cast<const float4 *>(kt + i),
+                 q4 = *reinterpret_cast<const float4 *>(qt + i);
+    const float a[4] = {a4.x, a4.y, a4.z, a4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w}, q[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float4 &s = S[i + e];
+      s.x = fmaf(a[e], s.x, k[e] * v.x); o.x = fmaf(q[e], s.x, o.x);
+      s.y = fmaf(a[e], s.y, k[e] * v.y); o.y = fmaf(q[e], s.y, o.y);
+      s.z = fmaf(a[e], s.z, k[e] * v.z); o.z = fmaf(q[e], s.z, o.z);
+      s.w = fmaf(a[e], s.w, k[e] * v.w); o.w = fmaf(q[e], s.w, o.w);
+    }
+  }
+  return o;
+}
+
+// Output of a head for token rows t0, t0 + step, ...: unit norm over the head, weight, silu of the gate.  One warp per token.
+template <int HYB>
+__device__ __forceinline__ void gla_emit(const TaskDesc &d, const GlaView &m, const SeqView &sv, int t0, int step) {
+  typedef typename HybElt<HYB>::T T;
+  const int lane = threadIdx.x & 31;
+  const float eps = __int_as_float(d.a[GA_EPS]);
+  T *out = reinterpret_cast<T *>(d.p[7]) + (size_t)sv.q0 * d.a[GA_LDO] + (size_t)m.h * m.vdim;
+  for (int t = t0; t < sv.nq; t += step) {
+    const float *rt = m.raw + (size_t)t * d.a[GA_LDR];
+    const float *gt = m.proj + (size_t)t * m.ldp + d.a[GA_GOFF] + (size_t)m.h * m.vdim;
+    float ss = 0.f;
+    if (m.vdim <= 512) {   // the row and its gates in registers, all loads in flight
+      float x[16], g[16];
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const bool in = i * 32 + lane < m.vdim;
+        x[i] = in ? __ldcg(rt + i * 32 + lane) : 0.f;
+        g[i] = in ? __ldcg(gt + i * 32 + lane) : 0.f;
+      }
+#pragma unroll
+      for (int i = 0; i < 16; ++i) ss += x[i] * x[i];
+      const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)m.vdim + eps);
+#pragma unroll
+      for (int i = 0; i < 16; ++i)
+        if (i * 32 + lane < m.vdim)
+          store_elt(out + (size_t)t * d.a[GA_LDO] + i * 32 + lane, x[i] * inv * bf16_at(d.p[3], i * 32 + lane) * silu_exact_f(g[i]));
+      continue;
+    }
+    for (int j = lane; j < m.vdim; j += 32) { const float v = __ldcg(rt + j); ss += v * v; }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)m.vdim + eps);
+    for (int j = lane; j < m.vdim; j += 32)
+      store_elt(out + (size_t)t * d.a[GA_LDO] + j, __ldcg(rt + j) * inv * bf16_at(d.p[3], j) * silu_exact_f(__ldcg(gt + j)));
+  }
+}
+
+// A portion of several tokens.
+template <int HYB, int CQ, int RPT>
+__device__ __noinline__ void gla_portion(const Ctx c, const TaskDesc &d, const SeqView sv, int task) {
+  constexpr int VC = 4 * CQ, RG = kConsumerThreads / CQ, ROWS = RG * RPT;
+  constexpr int GT = 8;   // tokens whose decays a thread forms together
+  const GlaView m = gla_view(d, sv);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int qd = tid % CQ, r0 = tid / CQ * RPT, TC = d.a[GA_TC];
+  // shared memory
+  float *as = reinterpret_cast<float *>(c.s.xtile);    // [TC][ROWS] decays
+  float *ks = as + (size_t)TC * ROWS;                  // [TC][ROWS]
+  float *qs = ks + (size_t)TC * ROWS;                  // [TC][ROWS]
+  float *vs = qs + (size_t)TC * ROWS;                  // [TC][VC]
+  float *red = vs + (size_t)TC * VC;                   // [TC][8 warps][VC]
+  float *low = red + (size_t)TC * 8 * VC;              // [TC][rank]
+  const float inv_tau = __int_as_float(d.a[GA_INVTAU]), qscale = __int_as_float(d.a[GA_QSCALE]);
+  stamp(c, task, 0);
+  for (int v0 = m.V0; v0 < m.V1; v0 += VC) {
+    const bool col_ok = v0 + 4 * qd < m.V1;
+    float4 S[RPT];
+    float *Sp = m.S + (size_t)r0 * m.vdimp + v0 + 4 * qd;
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+      S[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!m.fresh && col_ok && r0 + i < m.dim) S[i] = __ldcg(reinterpret_cast<const float4 *>(Sp + (size_t)i * m.vdimp));
+    }
+    for (int tb = 0; tb < sv.nq; tb += TC) {
+      const int nt = min(TC, sv.nq - tb);
+      consumer_sync();   // the previous trip's readers are done
+      // warp w takes tokens w, w + 8; a lane's loads of a token are independent and in flight together
+      const float *pk = m.proj + (size_t)tb * m.ldp + d.a[GA_KOFF] + m.h * m.dim, *pq = m.proj + (size_t)tb * m.ldp + d.a[GA_QOFF] + m.h * m.dim;
+      const float *pv = m.proj + (size_t)tb * m.ldp + d.a[GA_VOFF] + (size_t)m.h * m.vdim + v0;
+      const float *pa = m.proj + (size_t)tb * m.ldp + d.a[GA_AOFF];
+      for (int t = warp; t < nt; t += 8) {
+#pragma unroll 8
+        for (int r = lane; r < ROWS; r += 32) {
+          const bool ok = r < m.dim;
+          ks[(size_t)t * ROWS + r] = ok ? __ldcg(pk + (size_t)t * m.ldp + r) : 0.f;
+          qs[(size_t)t * ROWS + r] = ok ? __ldcg(pq + (size_t)t * m.ldp + r) * qscale : 0.f;
+        }
+#pragma unroll
+        for (int r = lane; r < VC; r += 32) vs[t * VC + r] = v0 + r < m.vdim ? __ldcg(pv + (size_t)t * m.ldp + r) : 0.f;
+        for (int j = lane; j < m.rank; j += 32) low[t * m.rank + j] = __ldcg(pa + (size_t)t * m.ldp + j);
+      }
+      consumer_sync();
+      // decays: an item is (row, GT tokens)
+      for (int it = tid; it < ROWS * ((nt + GT - 1) / GT); it += kConsumerThreads) {
+        const int r = it % ROWS, tg = it / ROWS * GT;
+        float z[GT];
+        const bool ok = r < m.dim;
+        const float bias = ok ? bf16_at(d.p[2], m.h * m.dim + r) : 0.f;
+#pragma unroll
+        for (int u = 0; u < GT; ++u) z[u] = bias;
+        if (ok) {
+          const size_t wr = (size_t)(m.h * m.dim + r) * m.rank;
+          for (int j = 0; j < m.rank; ++j) {
+            const float w = bf16_at(d.p[1], wr + j);
+#pragma unroll
+            for (int u = 0; u < GT; ++u) z[u] = fmaf(w, low[min(tg + u, nt - 1) * m.rank + j], z[u]);
+          }
+        }
+#pragma unroll
+        for (int u = 0; u < GT; ++u)
+          if (tg + u < nt) as[(size_t)(tg + u) * ROWS + r] = ok ? gla_decay(z[u], inv_tau) : 0.f;
+      }
+      consumer_sync();
+      for (int t = 0; t < nt; ++t) {
+        const float *at = as + (size_t)t * ROWS, *kt = ks + (size_t)t * ROWS, *qt = qs + (size_t)t * ROWS;
+        const float4 v = *reinterpret_cast<const float4 *>(vs + t * VC + 4 * qd);
+        const float4 o = mlstm_warp_rows<CQ>(gla_step<RPT>(S, at + r0, v, kt + r0, qt + r0));
+        if (lane < CQ) *reinterpret_cast<float4 *>(red + (size_t)(t * 8 + warp) * VC + 4 * lane) = o;
+      }
+      consumer_sync();
+      for (int i = tid; i < nt * VC; i += kConsumerThreads) {
+        const int t = i / VC, j = i % VC;
+        float s = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) s += red[(size_t)(t * 8 + w) * VC + j];
+        if (v0 + j < m.vdim && v0 + j < m.V1) __stcg(m.raw + (size_t)(tb + t) * d.a[GA_LDR] + v0 + j, s);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < RPT; ++i)
+      if (col_ok && r0 + i < m.dim) *reinterpret_cast<float4 *>(Sp + (size_t)i * m.vdimp) = S[i];
+  }
+  stamp(c, task, 1);
+  if (!last_of_head(c, d.a[GA_TICKET], m.chunks)) return;
+  stamp(c, task, 2);
+  gla_emit<HYB>(d, m, sv, warp, 8);
+}
+
+// One token (decoding): the state is what has to move, streamed as in mlstm_single.
+template <int HYB, int CQ, int RPT>
+__device__ __noinline__ void gla_single(const Ctx c, const TaskDesc &d, const SeqView sv, int task) {
+  constexpr int VC = 4 * CQ, RG = kConsumerThreads / CQ, ROWS = RG * RPT;
+  const GlaView m = gla_view(d, sv);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int qd = tid % CQ, r0 = tid / CQ * RPT;
+  float4 *ring = reinterpret_cast<float4 *>(c.s.xtile) + tid;                  // [2][RPT][256], this thread's cells
+  float *as = reinterpret_cast<float *>(c.s.xtile) + 8 * RPT * kConsumerThreads;   // [ROWS]
+  float *ks = as + ROWS;                                                       // [ROWS]
+  float *qs = ks + ROWS;                                                       // [ROWS]
+  float *red = qs + ROWS;                                                      // [2][8 warps][VC]
+  float *low = red + 16 * VC;                                                  // [rank]
+  const int nrow = min(RPT, m.dim - r0);                                       // real rows of this thread (may be <= 0)
+  float *Sp = m.S + (size_t)r0 * m.vdimp + m.V0 + 4 * qd;                      // its piece of the current sub-block
+  auto fetch = [&](int v0, int slot, const float *src) {
+    if (!m.fresh && v0 + 4 * qd < m.V1) {
+      const uint32_t dst = smem_u32(ring + slot * RPT * kConsumerThreads);
+#pragma unroll
+      for (int i = 0; i < RPT; ++i, src += m.vdimp)
+        if (i < nrow)
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + (uint32_t)(i * kConsumerThreads * 16)), "l"(src) : "memory");
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  fetch(m.V0, 0, Sp);
+  fetch(m.V0 + VC, 1, Sp + VC);
+  const float inv_tau = __int_as_float(d.a[GA_INVTAU]), qscale = __int_as_float(d.a[GA_QSCALE]);
+  for (int j = tid; j < m.rank; j += kConsumerThreads) low[j] = __ldcg(m.proj + d.a[GA_AOFF] + j);
+  for (int r = tid; r < ROWS; r += kConsumerThreads) {
+    const bool ok = r < m.dim;
+    ks[r] = ok ? __ldcg(m.proj + d.a[GA_KOFF] + m.h * m.dim + r) : 0.f;
+    qs[r] = ok ? __ldcg(m.proj + d.a[GA_QOFF] + m.h * m.dim + r) * qscale : 0.f;
+  }
+  consumer_sync();
+  for (int r = tid; r < ROWS; r += kConsumerThreads) {
+    float z = 0.f;
+    if (r < m.dim) {
+      z = bf16_at(d.p[2], m.h * m.dim + r);
+      const size_t wr = (size_t)(m.h * m.dim + r) * m.rank;
+#pragma unroll 16
+      for (int j = 0; j < m.rank; ++j) z = fmaf(bf16_at(d.p[1], wr + j), low[j], z);
+    }
+    as[r] = r < m.dim ? gla_decay(z, inv_tau) : 0.f;
+  }
+  consumer_sync();
+  stamp(c, task, 0);
+  int par = 0;
+  for (int v0 = m.V0; v0 < m.V1; v0 += VC, par ^= 1, Sp += VC) {
+    const bool col_ok = v0 + 4 * qd < m.V1;
+    float4 S[RPT];
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+#pragma unroll
+    for (int i = 0; i < RPT; ++i)
+      S[i] = !m.fresh && col_ok && i < nrow ? ring[(par * RPT + i) * kConsumerThreads] : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float *pv = m.proj + d.a[GA_VOFF] + (size_t)m.h * m.vdim + v0 + 4 * qd;
+    float4 v;
+    v.x = v0 + 4 * qd < m.vdim ? __ldcg(pv) : 0.f;
+    v.y = v0 + 4 * qd + 1 < m.vdim ? __ldcg(pv + 1) : 0.f;
+    v.z = v0 + 4 * qd + 2 < m.vdim ? __ldcg(pv + 2) : 0.f;
+    v.w = v0 + 4 * qd + 3 < m.vdim ? __ldcg(pv + 3) : 0.f;
+    const float4 o = mlstm_warp_rows<CQ>(gla_step<RPT>(S, as + r0, v, ks + r0, qs + r0));
+    fetch(v0 + 2 * VC, par, Sp + 2 * VC);
+    if (lane < CQ) *reinterpret_cast<float4 *>(red + (size_t)(par * 8 + warp) * VC + 4 * lane) = o;
+    float *dst = Sp;
+#pragma unroll
+    for (int i = 0; i < RPT; ++i, dst += m.vdimp)
+      if (col_ok && i < nrow) *reinterpret_cast<float4 *>(dst) = S[i];
+    consumer_sync();
+    if (tid < VC && v0 + tid < m.vdim && v0 + tid < m.V1) {
+      float s = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) s += red[(size_t)(par * 8 + w) * VC + tid];
+      __stcg(m.raw + v0 + tid, s);
+    }
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  stamp(c, task, 1);
+  if (!last_of_head(c, d.a[GA_TICKET], m.chunks)) return;
+  stamp(c, task, 2);
+  if (warp == 0) gla_emit<HYB>(d, m, sv, 0, 1);
+}
+
+template <int HYB, int CQ, int RPT>
+__device__ __forceinline__ void gla_body(const Ctx &c, const TaskDesc &d, const SeqView &sv, int task) {
+  if (sv.nq == 1) gla_single<HYB, CQ, RPT>(c, d, sv, task);
+  else gla_portion<HYB, CQ, RPT>(c, d, sv, task);
+}
+template <int HYB>
+__device__ __forceinline__ void run_gla(const Ctx &c, const TaskDesc &d, int task) {
+  const SeqView sv = seq_view(c.P, d.a[GA_SLOT]);
+  if (sv.nq <= 0) return;
+  const int dim = d.a[GA_DIM];
+  switch (mlstm_quads(dim)) {
+    case 16:
+      if (mlstm_rows_per_thread(dim) == 4) gla_body<HYB, 16, 4>(c, d, sv, task);
+      else gla_body<HYB, 16, 8>(c, d, sv, task);
+      break;
+    case 8: gla_body<HYB, 8, 8>(c, d, sv, task); break;
+    case 4: gla_body<HYB, 4, 8>(c, d, sv, task); break;
+    default: gla_body<HYB, 2, 8>(c, d, sv, task); break;
   }
 }
 
@@ -1838,6 +2304,8 @@ __device__ __forceinline__ void run_argmax_reduce_f32(const Ctx &c, const TaskDe
   }
 }
 
+__device__ __noinline__ void run_moe_routing_hybrid(const Ctx c, const TaskDesc &d) { run_moe_routing(c, d); }
+
 template <int HYB>
 __device__ __forceinline__ void run_hybrid_task(const Ctx &c, const TaskDesc &d, int task) {
   switch (d.type) {
@@ -1850,6 +2318,10 @@ __device__ __forceinline__ void run_hybrid_task(const Ctx &c, const TaskDesc &d,
     case TASK_EMBED_F32: run_embed_f32(c, d); break;
     case TASK_RESIDUAL_NORM: run_residual_norm<HYB>(c, d); break;
     case TASK_LINEAR_F32: if (HYB == HYB_F32) run_linear_f32(c, d); break;
+    case TASK_MOE_ROUTING: run_moe_routing_hybrid(c, d); break;
+    case TASK_MOE_GEMM_F32: if (HYB == HYB_F32) run_moe_gemm_f32(c, d); break;
+    case TASK_LATENT_APPEND: run_latent_append<HYB>(c, d); break;
+    case TASK_GLA: run_gla<HYB>(c, d, task); break;
     case TASK_QKV_APPEND: run_qkv_append<HYB>(c, d); break;
     case TASK_EXT_ATTENTION: run_ext_attention<HYB>(c, d, task); break;
     case TASK_SHORT_CONV: run_short_conv(c, d); break;

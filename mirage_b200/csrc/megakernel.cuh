@@ -133,6 +133,7 @@ __device__ void prefetch_attention_kv_l2(const Ctx &c, const TaskDesc *d, int la
 // are bank-conflict free.  Order: k tile (activation tile) -> 16-row group -> k chunk.
 template <bool GENERAL, int HYB>
 __device__ void streamer_loop(const Ctx &c, int t_begin, int t_end) {
+  constexpr bool kMoe = HYB ? HYB == HYB_BF16 : GENERAL;   // expert projections stream one panel per active expert
   const KernelParams &P = c.P;
   const int lane = threadIdx.x & 31;
   const uint64_t policy = l2_policy_evict_first();
@@ -148,7 +149,7 @@ __device__ void streamer_loop(const Ctx &c, int t_begin, int t_end) {
   for (int t = t_begin; t < t_end && ok; ++t) {
     const TaskDesc *d = &P.tasks[t];
     if (!HYB && d->type == TASK_ATTENTION && P.kv_l2_prefetch) prefetch_attention_kv_l2<GENERAL>(c, d, lane, t);
-    if (d->type != TASK_LINEAR && !(GENERAL && !HYB && d->type == TASK_MOE_GEMM)) continue;
+    if (d->type != TASK_LINEAR && !(kMoe && d->type == TASK_MOE_GEMM)) continue;
     if (d->flags & TF_STREAM_AFTER_DEP) {
       if (lane == 0)
         for (int i = 0; i < kMaxDeps && ok; ++i)
@@ -195,13 +196,13 @@ __device__ void streamer_loop(const Ctx &c, int t_begin, int t_end) {
     // an expert task repeats the panel loop once per active expert (the list is final: the task waited for it)
     int reps = 1;
     const int *act = nullptr;
-    if (GENERAL && !HYB && d->type == TASK_MOE_GEMM) {
+    if (kMoe && d->type == TASK_MOE_GEMM) {
       act = reinterpret_cast<const int *>(d->p[5]);
       reps = min(__ldcg(&act[d->a[M_NEXP]]), d->a[M_NEXP]);
     }
     for (int rep = 0; rep < reps && ok; ++rep) {
     const uint8_t *Wp = W;
-    if (GENERAL && !HYB && act != nullptr) Wp = W + (size_t)__ldcg(&act[rep]) * (size_t)d->a[M_ESTRIDE] * esz;
+    if (kMoe && act != nullptr) Wp = W + (size_t)__ldcg(&act[rep]) * (size_t)d->a[M_ESTRIDE] * esz;
     for (int kt = 0; kt < K && ok; kt += KT) {
       for (int r0 = n0; r0 < n1 && ok; r0 += R) {
         const int rows = min(R, n1 - r0);
@@ -288,6 +289,11 @@ __device__ __forceinline__ uint32_t ll_seq(unsigned long long iteration, int n_a
 
 // fast silu: x * sigmoid(x) with ex2.approx based exp and approximate divide (error far below bf16 rounding)
 __device__ __forceinline__ float silu_f(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
+// activations of hybrid graphs: float32 accuracy
+__device__ __forceinline__ float silu_exact_f(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float gelu_tanh_f(float x) {
+  return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+}
 
 // Stage the activation tile [B, KT] (bf16, rows padded by 16 bytes) for k range [k0, k0 + KT).
 // `gpre` holds this thread's first two gamma vectors, loaded before the dependency wait.
@@ -392,12 +398,15 @@ __device__ __forceinline__ float gather_row(const Ctx &c, const TaskDesc &d, con
 __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d, int B) {
   constexpr int NV = 4;   // rows of at most 4096 columns, in registers
   const int tid = threadIdx.x, W = d.a[L_GROUPS], K = d.a[L_K], warp = tid >> 5;
-  const float eps = __int_as_float(d.a[L_EPS]), off = d.a[L_G_SLOT] ? 1.0f : 0.0f;
-  const bool has_y = d.p[6] != 0, has_post = d.p[3] != 0;
+  const bool layer_norm = (d.a[L_G_SLOT] & 4) != 0;
+  const float eps = __int_as_float(d.a[L_EPS]), off = (d.a[L_G_SLOT] & 2) ? 1.0f : 0.0f;
+  const float *add = *reinterpret_cast<const float *const *>(&d.a[LR_ADD]);
+  const uint64_t rowp = *reinterpret_cast<const uint64_t *>(&d.a[LR_ROW]);
+  const bool has_y = d.p[6] != 0, has_post = d.p[3] != 0, moved = has_y || add != nullptr || rowp != 0;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  auto weights = [&](uint64_t base, int j) {
+  auto values = [&](uint64_t base, int j, float o) {
     const uint2 v = __ldg(reinterpret_cast<const uint2 *>(base + 2ull * j));
-    return make_float4(off + bf16_lo(v.x), off + bf16_hi(v.x), off + bf16_lo(v.y), off + bf16_hi(v.y));
+    return make_float4(o + bf16_lo(v.x), o + bf16_hi(v.x), o + bf16_lo(v.y), o + bf16_hi(v.y));
   };
   auto total = [&](float v, float *slots) {
     v = warp_sum(v);
@@ -419,8 +428,8 @@ __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d, int B
       const bool in = j < W;
       yv[i] = in && has_y ? __ldcg(reinterpret_cast<const float4 *>(y + j)) : zero;
       xv[i] = in ? __ldcg(reinterpret_cast<const float4 *>(x + j)) : zero;
-      wp[i] = in && has_post ? weights(d.p[3], j) : make_float4(1.f, 1.f, 1.f, 1.f);
-      wn[i] = in ? weights(d.p[4], j) : zero;
+      wp[i] = in && has_post ? values(d.p[3], j, off) : make_float4(1.f, 1.f, 1.f, 1.f);
+      wn[i] = in ? values(d.p[4], j, off) : zero;
     }
     if (has_y) {
       float inv = 1.f;
@@ -434,9 +443,33 @@ __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d, int B
       for (int i = 0; i < NV; ++i) {
         xv[i].x += yv[i].x * inv * wp[i].x; xv[i].y += yv[i].y * inv * wp[i].y;
         xv[i].z += yv[i].z * inv * wp[i].z; xv[i].w += yv[i].w * inv * wp[i].w;
+      }
+    }
+    if (add != nullptr || rowp != 0) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int j = (i * kConsumerThreads + tid) * 4;
+        if (j >= W) continue;
+        const float4 a = add != nullptr ? __ldcg(reinterpret_cast<const float4 *>(add + (size_t)b * d.a[LR_LDADD] + j)) : zero;
+        const float4 r = rowp != 0 ? values(rowp, j, 0.f) : zero;
+        xv[i].x = xv[i].x + a.x + r.x; xv[i].y = xv[i].y + a.y + r.y; xv[i].z = xv[i].z + a.z + r.z; xv[i].w = xv[i].w + a.w + r.w;
+      }
+    }
+    if (moved && d.p[7] != 0) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
         const int j = (i * kConsumerThreads + tid) * 4;
         if (j < W) *reinterpret_cast<float4 *>(xo + j) = xv[i];
       }
+    }
+    if (layer_norm) {
+      float s = 0.f;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) s += xv[i].x + xv[i].y + xv[i].z + xv[i].w;
+      const float mean = total(s, c.s.red + 16) / (float)W;
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if ((i * kConsumerThreads + tid) * 4 < W) { xv[i].x -= mean; xv[i].y -= mean; xv[i].z -= mean; xv[i].w -= mean; }
     }
     float ss = 0.f;
 #pragma unroll
@@ -446,9 +479,11 @@ __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d, int B
 #pragma unroll
     for (int i = 0; i < NV; ++i) {   // (the padding columns behind the row come out as zeros)
       const int j = (i * kConsumerThreads + tid) * 4;
+      const float4 bias = d.p[5] != 0 && j < W ? values(d.p[5], j, 0.f) : zero;
       if (j < K)
-        *reinterpret_cast<uint2 *>(row + 2 * j) = make_uint2(pack_bf16(xv[i].x * inv * wn[i].x, xv[i].y * inv * wn[i].y),
-                                                             pack_bf16(xv[i].z * inv * wn[i].z, xv[i].w * inv * wn[i].w));
+        *reinterpret_cast<uint2 *>(row + 2 * j) =
+            make_uint2(pack_bf16(xv[i].x * inv * wn[i].x + bias.x, xv[i].y * inv * wn[i].y + bias.y),
+                       pack_bf16(xv[i].z * inv * wn[i].z + bias.z, xv[i].w * inv * wn[i].w + bias.w));
     }
     consumer_sync();   // (also: the reduction slots are used again)
   }
@@ -772,6 +807,21 @@ __device__ __forceinline__ void linear_output(const Ctx &c, const TaskDesc &d, i
   } else if (HYB && epi == EPI_RELU2) {
     const float a = fmaxf(v, 0.f);
     reinterpret_cast<__nv_bfloat16 *>(d.p[2])[(size_t)b * d.a[L_LDO] + col] = __float2bfloat16_rn(a * a);
+  } else if (HYB && epi == EPI_SOFTCAP) {
+    const float cap = __int_as_float(d.a[L_CAP]);
+    reinterpret_cast<float *>(d.p[2])[(size_t)b * d.a[L_LDO] + col] = cap * tanhf(v / cap);
+  } else if (HYB && (epi == EPI_GATED_SILU || epi == EPI_GATED_GELU)) {
+    if ((r & 2) == 0) {
+      float u = 0.f;
+      if (WIDE) {
+        for (int w = b >> 3; w < 8; w += NT) u += part[(w * 16 + r + 2) * 8 + (b & 7)];
+      } else {
+#pragma unroll
+        for (int w = 0; w < 8; ++w) u += part[(w * 16 + r + 2) * 8 + b];
+      }
+      const float a = epi == EPI_GATED_SILU ? silu_exact_f(v) : gelu_tanh_f(v);
+      reinterpret_cast<__nv_bfloat16 *>(d.p[2])[(size_t)b * d.a[L_LDO] + ((col >> 2) << 1) + (r & 1)] = __float2bfloat16_rn(a * u);
+    }
   } else {
     __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(d.p[2]);
     if (epi == EPI_RESIDUAL) {
@@ -907,7 +957,7 @@ struct EmitArgs {
   __nv_bfloat16 *out;
   size_t push_off;      // element offset of (token 0, column 0) of this rank's slot in an inbox buffer
   int push_n;           // row length of the pushed matrix
-  uint32_t seq_hi;      // sequence number of the allreduce instance, already shifted to the high half
+  uint32_t seq_hi;      // sequence number of the allreduce instance, already shifted to the high half (EPI_SOFTCAP: cap bits)
 };
 
 __device__ __forceinline__ EmitArgs emit_args(const Ctx &c, const TaskDesc &d) {
@@ -919,7 +969,7 @@ __device__ __forceinline__ EmitArgs emit_args(const Ctx &c, const TaskDesc &d) {
   const unsigned long long inst = c.iteration * (unsigned)d.a[L_NAR] + (unsigned)d.a[L_ARIDX];
   e.push_off = (size_t)d.p[5] + (size_t)(inst & 1ull) * (size_t)d.a[L_PARSTRIDE] + (size_t)c.P.rank * (size_t)d.a[L_SLOT];
   e.push_n = d.a[L_N];
-  e.seq_hi = ll_seq(c.iteration, d.a[L_NAR], d.a[L_ARIDX]) << 16;
+  e.seq_hi = e.epi == EPI_SOFTCAP ? (uint32_t)d.a[L_CAP] : ll_seq(c.iteration, d.a[L_NAR], d.a[L_ARIDX]) << 16;
   return e;
 }
 
@@ -948,6 +998,13 @@ __device__ __forceinline__ void linear_emit(const Ctx &c, const EmitArgs &e, int
   } else if (HYB && e.epi == EPI_RELU2) {
     const float a = fmaxf(v, 0.f);
     e.out[(size_t)b * e.ldo + col] = __float2bfloat16_rn(a * a);
+  } else if (HYB && e.epi == EPI_SOFTCAP) {
+    const float cap = __uint_as_float(e.seq_hi);
+    reinterpret_cast<float *>(e.out)[(size_t)b * e.ldo + col] = cap * tanhf(v / cap);
+  } else if (HYB && (e.epi == EPI_GATED_SILU || e.epi == EPI_GATED_GELU)) {
+    if ((col & 2) == 0)
+      e.out[(size_t)b * e.ldo + ((col >> 2) << 1) + (col & 1)] =
+          __float2bfloat16_rn((e.epi == EPI_GATED_SILU ? silu_exact_f(v) : gelu_tanh_f(v)) * u);
   } else {
     e.out[(size_t)b * e.ldo + col] = __float2bfloat16_rn(v + resv);   // resv: the residual element, or 0
   }
@@ -1066,7 +1123,7 @@ __device__ void run_linear_tc(const Ctx &c, const TaskDesc &d, LinearState &ls, 
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
           const float v = __uint_as_float(r[j]);
-          const float u = (epi == EPI_SILU_PAIR) ? __shfl_down_sync(0xffffffffu, v, 2) : 0.f;
+          const float u = (epi == EPI_SILU_PAIR || (HYB && epi >= EPI_GATED_SILU)) ? __shfl_down_sync(0xffffffffu, v, 2) : 0.f;
           const int b = half * nh + c0 + j;
           if (row_ok && b < B) linear_emit<HYB>(c, ea, b, n0 + row, v, u, resv[j]);
         }
@@ -1529,6 +1586,7 @@ __device__ void run_moe_routing(const Ctx &c, const TaskDesc &d) {
   for (int i = tid; i < E * ldr; i += kConsumerThreads) routing[i] = 0;
   for (int i = tid; i < E; i += kConsumerThreads) mark[i] = 0;
   consumer_sync();
+  const bool keep_logits = d.a[12] != 0;
   const bool softmax = d.a[11] != 0;   // moe_topk_softmax_routing_layer: scores = softmax over the experts, no bias, logits kept
   for (int row = warp; row < B; row += 8) {
     float row_max = -INFINITY;
@@ -1537,11 +1595,11 @@ __device__ void run_moe_routing(const Ctx &c, const TaskDesc &d) {
       if (f32_in) {
         float *lp = reinterpret_cast<float *>(d.p[0]) + (size_t)row * ldl + e;
         logit = __ldcg(lp);
-        if (!softmax) *lp = 0.f;
+        if (!softmax && !keep_logits) *lp = 0.f;
       } else {
         __nv_bfloat16 *lp = reinterpret_cast<__nv_bfloat16 *>(d.p[0]) + (size_t)row * ldl + e;
         logit = bf16_to_f(__ldcg(lp));
-        if (!softmax) *lp = __float2bfloat16_rn(0.f);
+        if (!softmax && !keep_logits) *lp = __float2bfloat16_rn(0.f);
       }
       if (softmax) {
         sc[e] = logit;
@@ -1578,7 +1636,7 @@ __device__ void run_moe_routing(const Ctx &c, const TaskDesc &d) {
         if (v > t1) { t2 = t1; t1 = v; }
         else if (v > t2) t2 = v;
       }
-      gs[g] = t1 + t2;
+      gs[g] = per > 1 ? t1 + t2 : t1;
     }
     __syncwarp();
     unsigned long long selected = 0ull;
@@ -1657,12 +1715,13 @@ __device__ void run_moe_routing(const Ctx &c, const TaskDesc &d) {
 // by taking their exponent bits, as fp8_group_gemm_sm100.cuh:1378 does).  The task owns the row range [n0, n1) of
 // EVERY expert: all workers walk the same active list, so the load is balanced whatever the routing.  The
 // streamer walks the same list (it waits for the routing first) and streams the panel of each active expert.
+template <bool HYBRID>
 __device__ void run_moe_gemm(const Ctx &c, const TaskDesc &d, LinearState &ls, int task, bool ok) {
   const KernelParams &P = c.P;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   int stage = ls.stage;
   uint32_t phase = ls.phase;
-  const bool fp8 = (d.flags & TF_FP8) != 0;
+  const bool fp8 = !HYBRID && (d.flags & TF_FP8) != 0;
   const uint32_t esz = fp8 ? 1u : 2u;
   const int Bt = ok ? min(active_tokens(P), kMaxLinearTokens) : 0;
   const int n0 = d.a[L_N0], n1 = d.a[L_N1], K = d.a[L_K], N = d.a[L_N];
@@ -1894,7 +1953,18 @@ __device__ void run_moe_gemm(const Ctx &c, const TaskDesc &d, LinearState &ls, i
               float v = 0.f;
               for (int w = t >> 3; w < 8; w += NT) v += pp[(w * 16 + r) * 8 + (t & 7)];
               const int tmv = tokmap[t];
-              out[((size_t)(tmv & 0xff) * topk + (tmv >> 8)) * d.a[L_LDO] + rbase + r] = __float2bfloat16_rn(v);
+              const size_t orow = ((size_t)(tmv & 0xff) * topk + (tmv >> 8)) * d.a[L_LDO];
+              if (HYBRID && d.a[L_EPI] == EPI_STORE_F32) {
+                reinterpret_cast<float *>(out)[orow + rbase + r] = v;
+              } else if (HYBRID && d.a[L_EPI] >= EPI_GATED_SILU) {   // rows [gate, gate, up, up]
+                if (r & 2) continue;
+                float u = 0.f;
+                for (int w = t >> 3; w < 8; w += NT) u += pp[(w * 16 + r + 2) * 8 + (t & 7)];
+                const float a = d.a[L_EPI] == EPI_GATED_SILU ? silu_exact_f(v) : gelu_tanh_f(v);
+                out[orow + (((rbase + r) >> 2) << 1) + (r & 1)] = __float2bfloat16_rn(a * u);
+              } else {
+                out[orow + rbase + r] = __float2bfloat16_rn(v);
+              }
             }
           }
           if (r0 + R < n1) consumer_sync();   // further row groups reuse the buffers
@@ -1918,6 +1988,13 @@ __device__ void run_moe_gemm(const Ctx &c, const TaskDesc &d, LinearState &ls, i
 
 // TASK_MOE_SILU_MUL: rows of [gate | up] -> bf16(silu(gate)) * up  (tasks/ampere/silu_mul.cuh:20-42 on the
 // flattened [token x slot] rows, as register_moe_silu_mul_task sets it up)
+// Hybrid graphs (bf16 only): a function of its own, state of the stage ring by value, so that the linear loop's registers stay as
+// they are.
+__device__ __noinline__ LinearState run_moe_gemm_hybrid(const Ctx c, const TaskDesc &d, LinearState ls, int task, bool ok) {
+  run_moe_gemm<true>(c, d, ls, task, ok);
+  return ls;
+}
+
 __device__ void run_moe_silu_mul(const Ctx &c, const TaskDesc &d) {
   const int I = d.a[2], ldi = d.a[3], ldo = d.a[4];
   const int r1 = min(d.a[1], active_tokens(c.P) * d.a[5]);
@@ -3914,9 +3991,12 @@ __device__ void consumer_loop(const Ctx &c, int t_begin, int t_end) {
     TaskTimes tt{0, 0, (P.profiler != nullptr) && (uint64_t)(t + 1) * 8 <= P.profiler_entries};
     const uint32_t type = d.type;
     if (HYB != HYB_F32 && type == TASK_LINEAR) ok = task_linear<GENERAL, TPX, HYB>(c, d, t, ok, tt, ls);
-    else if (GENERAL && !HYB && type == TASK_MOE_GEMM) {
+    else if (HYB == HYB_BF16 && type == TASK_MOE_GEMM) {
       ok = wait_dependencies(c, d, t, ok, tt);
-      run_moe_gemm(c, d, ls, t, ok);
+      ls = run_moe_gemm_hybrid(c, d, ls, t, ok);
+    } else if (GENERAL && !HYB && type == TASK_MOE_GEMM) {
+      ok = wait_dependencies(c, d, t, ok, tt);
+      run_moe_gemm<false>(c, d, ls, t, ok);
     } else if (!HYB && type == TASK_ATTENTION) ok = task_attention<GENERAL>(c, d, t, ok, tt);
     else ok = task_other<GENERAL, TPX, HYB>(c, d, t, ok, tt);
     if (fetch) reinterpret_cast<uint4 *>(&c.s.desc[(t + 1 - t_begin) & 1])[tid - 224] = nxt;

@@ -63,6 +63,9 @@ enum TaskType : uint32_t {
   TASK_SHORT_CONV = 29,         // causal per-channel convolution with carried inputs
   TASK_RGLRU = 30,              // gated diagonal linear recurrence
   TASK_MLSTM = 31,              // matrix-memory recurrence with exponential gates
+  TASK_GLA = 32,                // gated linear attention (matrix state, a decay per key channel)
+  TASK_LATENT_APPEND = 33,      // latent attention: cache rows and rotated query parts
+  TASK_MOE_GEMM_F32 = 34,       // expert projections in 32-bit arithmetic
 };
 
 // Which family of megakernel instantiations runs a graph (template parameter HYB of the kernel).
@@ -85,6 +88,8 @@ MPK_HD constexpr int ext_attention_rows(int rows) {
 }
 
 enum : int { HYB_NONE = 0, HYB_BF16 = 1, HYB_F32 = 2 };
+// Activations of hybrid linears (mpk_activation of include/mpk_b200.h).
+enum : int { ACT_NONE = 0, ACT_RELU2 = 1, ACT_SOFTCAP = 2, ACT_GATED_SILU = 3, ACT_GATED_GELU = 4 };
 
 // Online mode: control word of a token-table row (KernelParams.meta.request_ctl[row], written by the host between
 // launches; request_ctl[rows + row] is the device's "live" flag).
@@ -106,6 +111,9 @@ enum Epilogue : int32_t {
   EPI_PUSH_LL = 3,      // {bf16 partial, 16-bit sequence} words pushed into every rank's inbox: self-validating
   EPI_STORE_F32 = 5,    // out = acc, float32 (hybrid graphs)
   EPI_RELU2 = 6,        // out = bf16(max(acc, 0)^2) (hybrid graphs)
+  EPI_SOFTCAP = 7,      // out = cap * tanh(acc / cap), float32 (hybrid graphs)
+  EPI_GATED_SILU = 8,   // rows [gate, gate, up, up]: out[2k + i] = bf16(silu(gate_i) * up_i) (hybrid graphs)
+  EPI_GATED_GELU = 9,   // the same with the tanh form of gelu
   EPI_SILU_PAIR = 4,    // rows interleaved [gate, gate, up, up]: out[2k + i] = bf16(silu(gate_i)) * up_i
 };
 
@@ -145,7 +153,9 @@ static_assert(sizeof(TaskDesc) == 16 * kDescVecs, "TaskDesc must stay 224 bytes 
 //        p[7] tensor that receives the reduced activations, a[20] ld residual, a[21] ld of that tensor,
 //        a[22] inbox slot stride of that allreduce (words)
 //  PRO_RESNORM: p[1] x f32  p[3] weight of y's norm or null  p[4] weight of the output norm  p[6] y f32 or null  p[7] x_out f32 (or
-//        null), a[20] ld y, a[21] ld x_out, a[22] 1: weights stored around zero, a[10] width (K minus the zero padding)
+//        null), a[20] ld y, a[21] ld x_out, a[22] flags (2: weights stored around zero, 4: layer norm), a[10] width (K minus the
+//        zero padding), p[5] norm bias or null, 64-bit values a[LR_ADD] added stream or null (ld a[LR_LDADD]), a[LR_ROW] added row or null
+//  EPI_SOFTCAP: a[23] cap bits
 //  a[15] allreduce index within the iteration  a[16] allreduces per iteration  a[17] stride between the two inbox buffers (floats)
 //  tcgen05 path (TF_TC): a[18] rows of one weight tile (the TMA box height, a multiple of 8, at most 128; the task's rows are
 //        cut into ceil(rows / a[18]) tiles, each one 128-lane accumulator), a[12] = 64 x (k blocks of 64 columns per ring slot),
@@ -153,6 +163,7 @@ static_assert(sizeof(TaskDesc) == 16 * kDescVecs, "TaskDesc must stay 224 bytes 
 enum { L_N0 = 0, L_N1, L_K, L_LDW, L_LDX, L_LDO, L_LDR, L_PRO, L_EPI, L_EPS, L_GROUPS, L_KT, L_KC, L_SLOT, L_N, L_ARIDX, L_NAR, L_PARSTRIDE, L_ROWS,
        L_GATHER, L_G_LDRES, L_G_LDOUT, L_G_SLOT, L_WS_S0, L_WS_S1, L_XS_S0, L_XS_S1, L_TMAP };
 static_assert(L_TMAP == 27, "TaskDesc::a has 28 entries");
+enum { LR_ADD = 14, LR_ROW = 16, L_CAP = 23, LR_LDADD = 25 };   // hybrid graphs (the fields of allreduces and FP8 tasks are free there)
 // ---- TASK_ATTENTION ----------------------------------------------------------
 //  p[0] qkv  p[1] k_cache  p[2] v_cache  p[3] q_norm  p[4] k_norm  p[5] cos  p[6] sin  p[7] out
 //  a[0] slot  a[1] kv head  a[2] chunk  a[3] num chunks  a[4] local q heads  a[5] local kv heads
@@ -167,9 +178,10 @@ enum { A_SLOT = 0, A_HEAD, A_CHUNK, A_NCHUNK, A_HQ, A_HKV, A_HD, A_PAGE, A_FLAGS
 enum { E_T0 = 0, E_T1, E_WIDTH, E_LDI, E_LDO, E_AUX, E_LDI2 };
 // ---- TASK_MOE_ROUTING: p[0] logits [B, E] (zeroed after reading)  p[1] bias f32 [E]  p[2] weights f32 [B, topk]
 //      p[3] routing i32 [E, ld]  p[4] active i32 [E + 1];  a[0] E  a[1] topk  a[2] groups  a[3] groups kept
-//      a[4] scaling bits  a[5] ld logits  a[6] ld weights  a[7] ld routing  a[8] logits are f32
+//      a[4] scaling bits  a[5] ld logits  a[6] ld weights  a[7] ld routing  a[8] logits are f32  a[12] logits stay as they are
 // ---- TASK_MOE_GEMM: linear-task fields (L_*) describe one expert's panel; p[0] weights [E, N, K]  p[1] x  p[2] out
 //      p[4] routing  p[5] active list  p[6] weight scales f32 [E, N, K/128]  p[7] x scales f32 [rows, K/128];
+//      a[L_EPI] EPI_STORE, EPI_STORE_F32, EPI_GATED_*
 //      a[M_NEXP] experts  a[M_NTOPK]  a[M_PER_SLOT] 1: x has one row per (token, slot)  a[M_LDR] ld routing
 //      a[M_ESTRIDE] elements between experts
 enum { M_NEXP = 19, M_NTOPK, M_PER_SLOT, M_LDR, M_ESTRIDE };
@@ -196,12 +208,18 @@ enum { M_NEXP = 19, M_NTOPK, M_PER_SLOT, M_LDR, M_ESTRIDE };
 //      exchange area inside an inbox buffer ([world][tokens] x {value | seq, index | seq} 64-bit words), a[L_ARIDX],
 //      a[L_NAR], a[L_PARSTRIDE] as for the allreduce
 // ---- hybrid tasks --------------------------------------------------------------
-// ---- TASK_EMBED_F32: p[0] ids  p[1] table bf16  p[2] out f32;  a[E_*] as TASK_EMBED (a[E_AUX] = vocabulary)
+// ---- TASK_EMBED_F32: p[0] ids  p[1] table bf16  p[2] out f32;  a[E_*] as TASK_EMBED (a[E_AUX] = vocabulary, a[E_LDI2] factor bits)
 // ---- TASK_RESIDUAL_NORM: rows [a[0], a[1]), width a[2]; p[0] x f32 (in place)  p[1] y f32 or null  p[2] weight of y's norm or
 //      null (plain sum)  p[3] weight of the output norm or null  p[4] out (bf16, f32 with flag 1) or null  p[5] new x (= p[0]: in place);
-//      a[3] ld x  a[4] ld y  a[5] ld out  a[6] eps bits  a[7] flags (1: out f32, 2: weights stored around zero)  a[8] ld of the new x
+//      a[3] ld x  a[4] ld y  a[5] ld out  a[6] eps bits  a[7] flags (1: out f32, 2: weights stored around zero, 4: layer norm)  a[8] ld
+//      of the new x;  64-bit values, 0 if absent: a[RN_BIAS] norm bias, a[RN_ADD] added stream, a[RN_ROW] added row, a[RN_EXP] expert
+//      outputs f32 [tokens, slots, width], a[RN_EW] their weights f32, a[RN_GATE] f32 column, y is multiplied by its sigmoid
+enum { RN_LDADD = 9, RN_BIAS = 10, RN_ADD = 12, RN_ROW = 14, RN_EXP = 16, RN_EW = 18, RN_GATE = 20, RN_SLOTS = 22, RN_LDEW, RN_LDGATE };
 // ---- TASK_LINEAR_F32: p[0] W bf16 [N, K]  p[1] x f32  p[2] out f32;  a[0] n0  a[1] n1  a[2] K  a[3] ldw  a[4] ld x  a[5] ld out
-//      a[6] activation (0 none, 1 squared relu)  a[7] tokens per shared-memory tile
+//      a[6] activation (mpk_activation)  a[7] tokens per shared-memory tile  a[8] soft cap bits
+// ---- TASK_MOE_GEMM_F32: p[0] W bf16 [E, N, K]  p[1] x f32  p[2] out f32  p[4] routing  p[5] active list;  a[0] n0  a[1] n1  a[2] K  a[4] ld x
+//      a[5] ld out (of a slot)  a[6] activation  a[7] tokens per shared-memory tile  a[8] x rows per (token, slot)  a[9] slots  a[10] ld routing
+//      a[11] experts  a[12] rows N of an expert
 // ---- TASK_QKV_APPEND: tokens [a[0], a[1]); p[0] projections f32  p[1] q out  p[2] k cache  p[3] v cache  p[4] cos f32  p[5] sin f32
 //      p[6] v source (null: the k columns before rotation and norm)
 //      a[QA_*] below
@@ -209,7 +227,7 @@ enum { QA_T0 = 0, QA_T1, QA_LDP, QA_QOFF, QA_KOFF, QA_VOFF, QA_HQ, QA_HKV, QA_DI
        QA_EPS, QA_PAGE, QA_LDQ, QA_ROWS };
 // ---- TASK_EXT_ATTENTION: p[0] q [tokens, hq * dimp]  p[1] k cache  p[2] v cache  p[3] out;  a[XA_*] below
 enum { XA_SLOT = 0, XA_HEAD, XA_CHUNK, XA_NCHUNK, XA_HQ, XA_HKV, XA_DIMP, XA_VDIM, XA_VDIMP, XA_PAGE, XA_LDQ, XA_LDO, XA_OCOL,
-       XA_SCALE, XA_CAP, XA_SINK, XA_OSCALE, XA_TICKET, XA_SREC, XA_STAGES };
+       XA_SCALE, XA_CAP, XA_SINK, XA_OSCALE, XA_TICKET, XA_SREC, XA_STAGES, XA_SHARED };   // p[4] sinks bf16 [hq] or null; XA_SHARED: values are key columns
 constexpr int kXaCells = 320;   // cache rows of a chunk's key octets kept in shared memory
 // ---- TASK_SHORT_CONV: channels [a[0], a[1]); p[0] in f32  p[1] in bias bf16 or null  p[2] taps bf16 [channels, taps]
 //      p[3] bias bf16 or null  p[4] carried inputs f32 [slots, taps - 1, channels]  p[5] out f32
@@ -223,6 +241,13 @@ enum { GL_BLOCK = 0, GL_C0, GL_C1, GL_BS, GL_WIDTH, GL_LDU, GL_LDP, GL_YOFF, GL_
 //      p[6] readout scratch f32 [tokens, heads * vdim]  p[7] out;  a[ML_*]
 enum { ML_SLOT = 0, ML_HEAD, ML_CHUNK, ML_NCHUNK, ML_H, ML_DIM, ML_VDIM, ML_VDIMP, ML_V0, ML_V1, ML_CAP, ML_EPS, ML_LDP, ML_QOFF,
        ML_KOFF, ML_VOFF, ML_GOFF, ML_IOFF, ML_FOFF, ML_LDO, ML_OUTF32, ML_QSCALE, ML_TICKET, ML_TC, ML_LDR };
+// ---- TASK_GLA: p[0] projections f32  p[1] a2 bf16 [heads * dim, rank]  p[2] a2 bias bf16  p[3] output norm weight bf16 [vdim]
+//      p[4] matrix state f32 [slots, heads, dim, vdimp]  p[6] readout scratch f32 [tokens, heads * vdim]  p[7] out;  a[GA_*]
+enum { GA_SLOT = 0, GA_HEAD, GA_CHUNK, GA_NCHUNK, GA_H, GA_DIM, GA_VDIM, GA_VDIMP, GA_V0, GA_V1, GA_EPS, GA_LDP, GA_QOFF, GA_KOFF, GA_VOFF,
+       GA_GOFF, GA_AOFF, GA_RANK, GA_LDO, GA_QSCALE, GA_TICKET, GA_TC, GA_LDR, GA_INVTAU };
+// ---- TASK_LATENT_APPEND: items [a[0] of a[1] tasks]; p[0] projections f32  p[1] latent norm weight bf16  p[2] q out  p[3] cache [pages, page, 1, dimp]
+//      p[4] cos f32  p[5] sin f32;  a[LA_*]
+enum { LA_T0 = 0, LA_T1, LA_LDP, LA_QOFF, LA_KVOFF, LA_H, LA_RANK, LA_ROT, LA_DIMP, LA_EPS, LA_PAGE, LA_LDQ, LA_ROWS };
 // ---- TASK_ALLREDUCE:       p[0] inbox base p[1] residual (or null) p[2] out
 //  a[0] c0 a[1] c1 (columns) a[2] world a[3] slot stride (floats) a[4] ld_out a[5] ld_res a[6] N
 //  a[7] allreduce index  a[8] allreduces per iteration  a[9] stride between the two inbox buffers (floats)

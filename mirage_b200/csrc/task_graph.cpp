@@ -117,7 +117,10 @@ struct Builder {
           add(ins, l.prologue == PRO_PLAIN ? l.t[0] : l.pro_src);
         }
         if (l.prologue == PRO_RMSNORM || l.prologue == PRO_RESNORM) add(ins, l.pro_gamma);
-        if (l.prologue == PRO_RESNORM) { add(ins, l.pro_y); add(ins, l.pro_post); add(outs, l.pro_xout); }
+        if (l.prologue == PRO_RESNORM) {
+          for (int t : {l.pro_y, l.pro_post, l.pro_bias, l.pro_add, l.pro_row}) add(ins, t);
+          add(outs, l.pro_xout);
+        }
         add(ins, l.t[1]);
         const int y = l.op == MPK_OP_LINEAR_RESIDUAL ? l.t[3] : l.t[2];
         if (l.op == MPK_OP_LINEAR_RESIDUAL) add(ins, l.t[2]);
@@ -151,7 +154,9 @@ struct Builder {
       case MPK_OP_QUANTIZE_FP8: add(ins, l.t[0]); add(outs, l.t[1]); add(outs, l.t[2]); break;
       case MPK_OP_LINEAR_FP8: for (int i = 0; i < 4; ++i) add(ins, l.t[i]); add(outs, l.t[4]); break;
       case MPK_OP_MOE_TOPK_SIGMOID:
-        add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[0]); add(outs, l.t[2]); add(outs, l.t[3]); add(outs, l.t[4]); break;
+        add(ins, l.t[0]); add(ins, l.t[1]);
+        if (!keeps_logits(l)) add(outs, l.t[0]);
+        add(outs, l.t[2]); add(outs, l.t[3]); add(outs, l.t[4]); break;
       case MPK_OP_MOE_TOPK_SOFTMAX:
         add(ins, l.t[0]); add(outs, l.t[1]); add(outs, l.t[2]); add(outs, l.t[3]); break;
       case MPK_OP_MOE_W13_LINEAR: case MPK_OP_MOE_W2_LINEAR:
@@ -164,15 +169,23 @@ struct Builder {
       case MPK_OP_MLA_DECODE: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); add(outs, l.t[3]); break;
       case MPK_OP_MLA_REDUCE: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); break;
       case MPK_OP_RESIDUAL_NORM:
-        for (int i = 0; i < 4; ++i) add(ins, l.t[i]);
-        if (l.t[1] >= 0) add(outs, resnorm_out(l));
+        for (int i = 0; i < 12; ++i) if (i != 4 && i != 5) add(ins, norm_tensor(l, i));
+        if (resnorm_moves(l)) add(outs, resnorm_out(l));
         add(outs, l.t[4]);
         break;
       case MPK_OP_QKV_APPEND: add(ins, l.t[0]); add(ins, l.t[4]); add(ins, l.t[5]); for (int i = 1; i < 4; ++i) add(outs, l.t[i]); break;
-      case MPK_OP_EXT_ATTENTION: for (int i = 0; i < 3; ++i) add(ins, l.t[i]); add(outs, l.t[3]); break;
+      case MPK_OP_EXT_ATTENTION:
+        for (int i = 0; i < 3; ++i) add(ins, l.t[i]);
+        if (l.t.size() > 4) add(ins, l.t[4]);
+        add(outs, l.t[3]);
+        break;
       case MPK_OP_SHORT_CONV: for (int i = 0; i < 5; ++i) add(ins, l.t[i]); add(outs, l.t[4]); add(outs, l.t[5]); break;
       case MPK_OP_RGLRU: for (int i = 0; i < 9; ++i) add(ins, l.t[i]); add(outs, l.t[8]); add(outs, l.t[9]); break;
       case MPK_OP_MLSTM: for (int i = 0; i < 6; ++i) add(ins, l.t[i]); for (int i = 4; i < 8; ++i) add(outs, l.t[i]); break;
+      case MPK_OP_GLA: for (int i = 0; i < 5; ++i) add(ins, l.t[i]); for (int i = 4; i < 7; ++i) add(outs, l.t[i]); break;
+      case MPK_OP_LATENT_APPEND:
+        add(ins, l.t[0]); add(ins, l.t[1]); add(ins, l.t[4]); add(ins, l.t[5]); add(outs, l.t[2]); add(outs, l.t[3]); break;
+      case MPK_OP_GROUPED_LINEAR: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); break;
       case MPK_OP_LINEAR_FP8_RESIDUAL: for (int i = 0; i < 5; ++i) add(ins, l.t[i]); add(outs, l.t[5]); break;
       default: break;
     }
@@ -205,7 +218,8 @@ struct Builder {
           {MPK_OP_MLA_KV_GATHER, 3}, {MPK_OP_MLA_DECODE, 4}, {MPK_OP_MLA_REDUCE, 3},
           {MPK_OP_SAMPLING_PARTIAL, 3}, {MPK_OP_SAMPLING_REDUCE, 3}, {MPK_OP_ARGMAX_EXCHANGE, 3},
           {MPK_OP_MOE_TOPK_SOFTMAX, 4}, {MPK_OP_RESIDUAL_NORM, 5}, {MPK_OP_QKV_APPEND, 6}, {MPK_OP_EXT_ATTENTION, 4},
-          {MPK_OP_SHORT_CONV, 6}, {MPK_OP_RGLRU, 10}, {MPK_OP_MLSTM, 8}};
+          {MPK_OP_SHORT_CONV, 6}, {MPK_OP_RGLRU, 10}, {MPK_OP_MLSTM, 8}, {MPK_OP_GLA, 7}, {MPK_OP_LATENT_APPEND, 6},
+          {MPK_OP_GROUPED_LINEAR, 3}};
       auto it = need.find(L[i].op);
       if (it == need.end()) return fail(MPK_ERR_UNSUPPORTED, "layer " + std::to_string(i) + ": unknown op");
       if ((int)L[i].t.size() < it->second)
@@ -276,7 +290,14 @@ struct Builder {
   }
 
   // Stream tensor a residual_norm layer writes: its own output (t[5]) or the input in place.
-  static int resnorm_out(const LayerInfo &l) { return l.t.size() > 5 && l.t[5] >= 0 ? l.t[5] : l.t[0]; }
+  static int norm_tensor(const LayerInfo &l, size_t i) { return i < l.t.size() ? l.t[i] : -1; }
+  static int resnorm_out(const LayerInfo &l) { return norm_tensor(l, 5) >= 0 ? l.t[5] : l.t[0]; }
+  // Does the layer add anything to the stream?
+  static bool resnorm_moves(const LayerInfo &l) {
+    return l.t[1] >= 0 || norm_tensor(l, 7) >= 0 || norm_tensor(l, 8) >= 0 || norm_tensor(l, 9) >= 0;
+  }
+  static int norm_flags(const LayerInfo &l) { return (l.params[1] ? 2 : 0) | (l.params.size() > 2 && l.params[2] == 1 ? 4 : 0); }
+  static bool keeps_logits(const LayerInfo &l) { return l.params.size() > 5 && l.params[5] != 0; }
 
   // Hybrid graphs of one or two tokens: a residual_norm layer whose result feeds linears becomes their prologue, which
   // spares the chain a task group.  (With more tokens the rows are spread over the workers instead of being formed by all.)
@@ -285,11 +306,15 @@ struct Builder {
     for (size_t i = 0; i < L.size(); ++i) {
       LayerInfo &p = L[i];
       if (p.op != MPK_OP_RESIDUAL_NORM || p.t[4] < 0 || p.t[3] < 0) continue;
-      const int x = p.t[0], y = p.t[1], out = p.t[4], xo = resnorm_out(p);
+      const int x = p.t[0], y = p.t[1], out = p.t[4], xo = resnorm_out(p), add = norm_tensor(p, 7), row = norm_tensor(p, 8), bias = norm_tensor(p, 6);
+      if (norm_tensor(p, 9) >= 0 || norm_tensor(p, 11) >= 0) continue;   // the sum over experts is formed once, not by every task
+      const bool moves = resnorm_moves(p);
       auto aligned = [&](int t) { return T[t].ld() % 4 == 0 && ((uint64_t)T[t].ptr & 15) == 0; };
       const int64_t D = T[x].dim(1);
       if (T[out].owner == 0 || D > 4096 || D % 4 || !aligned(x) || ((uint64_t)T[p.t[3]].ptr & 7) || p.params.size() < 2) continue;
-      if (y >= 0 && (T[xo].storage == T[x].storage || !aligned(y) || !aligned(xo) || T[xo].dtype != MPK_F32 || T[xo].dim(1) != D)) continue;
+      if (moves && (T[xo].storage == T[x].storage || !aligned(xo) || T[xo].dtype != MPK_F32 || T[xo].dim(1) != D)) continue;
+      if ((y >= 0 && !aligned(y)) || (add >= 0 && (!aligned(add) || T[add].dtype != MPK_F32 || T[add].dim(1) != D))) continue;
+      if ((bias >= 0 && ((uint64_t)T[bias].ptr & 7)) || (row >= 0 && ((uint64_t)T[row].ptr & 7))) continue;
       if (p.t[2] >= 0 && ((uint64_t)T[p.t[2]].ptr & 7)) continue;
       std::vector<size_t> consumers;
       bool ok = true;
@@ -304,14 +329,15 @@ struct Builder {
       }
       if (!ok || consumers.size() != 1) continue;
       for (size_t j = i + 1; j < consumers[0] && ok; ++j)   // nothing in between may touch what the prologue reads or writes
-        for (int t : {x, y, xo})
-          if (t >= 0 && (raw_writes(L[j], T[t].storage) || (t == xo && y >= 0 && raw_reads(L[j], T[t].storage)))) ok = false;
+        for (int t : {x, y, xo, add})
+          if (t >= 0 && (raw_writes(L[j], T[t].storage) || (t == xo && moves && raw_reads(L[j], T[t].storage)))) ok = false;
       if (!ok) continue;
       LayerInfo &c = L[consumers[0]];
       c.prologue = PRO_RESNORM;
       c.pro_src = x; c.pro_y = y; c.pro_post = p.t[2]; c.pro_gamma = p.t[3];
-      c.pro_xout = y >= 0 ? xo : -1;
-      c.pro_eps = bits_of(p.params[0]); c.pro_zero = p.params[1] ? 1 : 0;
+      c.pro_bias = bias; c.pro_add = add; c.pro_row = row;
+      c.pro_xout = moves ? xo : -1;
+      c.pro_eps = bits_of(p.params[0]); c.pro_flags = norm_flags(p);
       p.folded = true;
       g->num_folded++;
     }
@@ -428,6 +454,7 @@ struct Builder {
       if (l.folded) continue;
       if (hybrid_op(l.op)) {
         need = std::max<int64_t>(need, hybrid_smem(l) - kPartialBytes);
+        if (l.op == MPK_OP_GROUPED_LINEAR && g->hybrid == HYB_BF16 && tc_linear(T[l.t[1]].dim(2))) g->use_tmem = true;
       } else if (g->hybrid == HYB_F32 && l.op == MPK_OP_LINEAR) {
         const int64_t K = T[l.t[1]].dim(1);
         need = std::max<int64_t>(need, (int64_t)linear_f32_tokens(K) * K * 4 - kPartialBytes);
@@ -447,12 +474,15 @@ struct Builder {
         }
       } else if (l.op == MPK_OP_MOE_W13_FP8 || l.op == MPK_OP_MOE_W2_FP8) {
         need = std::max(need, std::min<int64_t>(moe_fp8_tile_bytes(ntok, T[l.t[2]].dim(2)), x_tile_cap()));
+      } else if (g->hybrid == HYB_F32 && (l.op == MPK_OP_MOE_W13_LINEAR || l.op == MPK_OP_MOE_W2_LINEAR)) {
+        const int64_t K = T[l.t[1]].dim(2);
+        need = std::max<int64_t>(need, (int64_t)linear_f32_tokens(K) * K * 4 + 256 - kPartialBytes);
       } else if (l.op == MPK_OP_MOE_W13_LINEAR || l.op == MPK_OP_MOE_W2_LINEAR) {
         need = std::max(need, std::min<int64_t>((int64_t)ntok * (T[l.t[1]].dim(2) * 2 + kRowPadBytes), x_tile_cap()));
       } else if (l.op == MPK_OP_MLA_DECODE) {
         need = std::max<int64_t>(need, 16 * (576 * 2 + 16) + 64 * (576 * 2 + 16) + 16 * (64 * 2 + 16) + 2 * 8 * 16 * 4);
       } else if (l.op == MPK_OP_MOE_TOPK_SIGMOID) {
-        const int64_t E = T[l.t[0]].dim(1);
+        const int64_t E = T[l.t[3]].dim(0);
         need = std::max(need, 8 * (2 * E + 64) * 4 + E * 4 + 64);
       } else if (l.op == MPK_OP_ATTENTION || l.op == MPK_OP_PAGED_ATTENTION) {
         const int G = (int)(l.params[0] / l.params[1]);
@@ -549,10 +579,8 @@ struct Builder {
     } else if (l.prologue != PRO_RESNORM && x.dim(x.dims.size() - 1) != K) {
       return fail(MPK_ERR_INVALID, "linear input width != K for " + w.name);
     }
-    // (hybrid graphs: the output buffer may be padded to the k granularity of the next linear)
-    if (g->hybrid ? y.dim(y.dims.size() - 1) < N : y.dim(y.dims.size() - 1) != N)
-      return fail(MPK_ERR_INVALID, "linear output width != N for " + w.name);
     int epi = EPI_STORE;
+    bool gated = false;
     uint64_t res_ptr = 0;
     int ldr = 0;
     if (l.op == MPK_OP_LINEAR_RESIDUAL) {
@@ -567,9 +595,11 @@ struct Builder {
     if (l.push) epi = l.push_ll ? EPI_PUSH_LL : EPI_PUSH_F32;
     if (x.dtype != MPK_BF16 && l.prologue != PRO_RESNORM) return fail(MPK_ERR_UNSUPPORTED, "linear input must be bf16: " + w.name);
     if (l.op == MPK_OP_LINEAR && !l.params.empty() && l.params[0] != 0) {
-      if (g->hybrid != HYB_BF16 || l.params[0] != 1 || y.dtype != MPK_BF16)
-        return fail(MPK_ERR_UNSUPPORTED, "linear activation: squared relu into bf16, in hybrid graphs: " + w.name);
-      epi = EPI_RELU2;
+      epi = activation_epilogue(l.params[0]);
+      if (g->hybrid != HYB_BF16 || epi == EPI_STORE || y.dtype != (epi == EPI_SOFTCAP ? MPK_F32 : MPK_BF16) || (epi == EPI_SOFTCAP && l.params.size() < 2))
+        return fail(MPK_ERR_UNSUPPORTED, "linear activation: in hybrid graphs, bf16 output (soft cap: float32): " + w.name);
+      gated = epi == EPI_GATED_SILU || epi == EPI_GATED_GELU;
+      if (gated && N % 4) return fail(MPK_ERR_INVALID, "gated linear: rows come as two gate rows, two up rows: " + w.name);
     } else if (y.dtype == MPK_F32) {
       if (g->hybrid != HYB_BF16 || epi != EPI_STORE) return fail(MPK_ERR_UNSUPPORTED, "float32 linear output needs a hybrid graph: " + w.name);
       epi = EPI_STORE_F32;
@@ -578,7 +608,11 @@ struct Builder {
     }
     uint64_t out_ptr = (uint64_t)y.ptr;
     int ldo = (int)y.ld();
-    const int unit = l.silu_out >= 0 ? 4 : 1;      // paired rows stay in one task
+    // (hybrid graphs: the output buffer may be padded to the k granularity of the next linear)
+    const int out_cols = gated ? N / 2 : N;
+    if (g->hybrid ? y.dim(y.dims.size() - 1) < out_cols : y.dim(y.dims.size() - 1) != N)
+      return fail(MPK_ERR_INVALID, "linear output width != N for " + w.name);
+    const int unit = l.silu_out >= 0 || gated ? 4 : 1;      // paired rows stay in one task
     if (l.silu_out >= 0) {
       if (epi != EPI_STORE || N % 4 != 0) return fail(MPK_ERR_INVALID, "activation epilogue on an unsupported linear: " + w.name);
       epi = EPI_SILU_PAIR;
@@ -648,7 +682,9 @@ struct Builder {
           d.p[7] = l.pro_xout >= 0 ? (uint64_t)T[l.pro_xout].ptr : 0;
           d.a[L_G_LDRES] = l.pro_y >= 0 ? (int)T[l.pro_y].ld() : 0;
           d.a[L_G_LDOUT] = l.pro_xout >= 0 ? (int)T[l.pro_xout].ld() : 0;
-          d.a[L_G_SLOT] = l.pro_zero;
+          d.a[L_G_SLOT] = l.pro_flags;
+          d.p[5] = l.pro_bias >= 0 ? (uint64_t)T[l.pro_bias].ptr : 0;
+          d.a[LR_LDADD] = l.pro_add >= 0 ? (int)T[l.pro_add].ld() : 0;
         }
         d.a[L_N0] = r;
         d.a[L_N1] = std::min(r + task_cap, row + cnt);
@@ -669,6 +705,11 @@ struct Builder {
         d.a[L_ARIDX] = std::max(l.ar_index, 0);
         d.a[L_NAR] = g->num_allreduce;
         d.a[L_PARSTRIDE] = (int)g->inbox_floats_per_buffer;
+        if (epi == EPI_SOFTCAP) d.a[L_CAP] = bits_of(l.params[1]);
+        if (l.prologue == PRO_RESNORM) {
+          put_wide(&d, LR_ADD, l.pro_add);
+          put_wide(&d, LR_ROW, l.pro_row);
+        }
         if (tc) {
           d.flags |= TF_TC;
           d.a[L_KC] = tc_nkb * kTcKBlock;
@@ -889,14 +930,26 @@ struct Builder {
     const int N = (int)w.dim(1), K = (int)w.dim(2), topk = (int)y.dim(1);
     if (ebase < 0 || ebase + EW > E) return fail(MPK_ERR_INVALID, "expert projection: weight experts outside the routing range: " + w.name);
     const int want = fp8 ? MPK_F8E4M3 : MPK_BF16;
-    if (w.dtype != want || x.dtype != want || y.dtype != MPK_BF16 || w.strides[2] != 1 || w.strides[1] != K ||
+    if (g->hybrid == HYB_F32) return emit_moe_gemm_f32(li, ex);
+    int epi = EPI_STORE, cols = N;
+    if (g->hybrid && !w2 && l.params.size() > 1 && l.params[1]) {
+      epi = activation_epilogue(l.params[1]);
+      if ((epi != EPI_GATED_SILU && epi != EPI_GATED_GELU) || N % 4) return fail(MPK_ERR_INVALID, "expert projection: gated activations only: " + w.name);
+      cols = N / 2;
+    } else if (g->hybrid && y.dtype == MPK_F32) {
+      epi = EPI_STORE_F32;
+    }
+    const int unit = cols < N ? 4 : 1;
+    if (g->hybrid && fp8) return fail(MPK_ERR_UNSUPPORTED, "expert projection: bf16 in hybrid graphs: " + w.name);
+    if (w.dtype != want || x.dtype != want || y.dtype != (epi == EPI_STORE_F32 ? MPK_F32 : MPK_BF16) || w.strides[2] != 1 || w.strides[1] != K ||
         w.strides[0] != (int64_t)N * K)
       return fail(MPK_ERR_UNSUPPORTED, "expert projection: dense " + std::string(fp8 ? "e4m3" : "bf16") + " weights, bf16 output: " + w.name);
-    if (x.dim(x.dims.size() - 1) != K || y.dim(2) != N || mask.dim(0) != E + 1 || idx.dtype != MPK_I32 ||
+    if (x.dim(x.dims.size() - 1) != K || (g->hybrid ? y.dim(2) < cols : y.dim(2) != N) || mask.dim(0) != E + 1 || idx.dtype != MPK_I32 ||
         mask.dtype != MPK_I32 || (w2 && x.dim(1) != topk) || topk > 255 || idx.dim(1) > 255)
       return fail(MPK_ERR_INVALID, "expert projection: shapes of " + w.name + " and its routing tensors disagree");
-    if (K % 128 != 0 || (int64_t)N * K >= (1ll << 31))
-      return fail(MPK_ERR_UNSUPPORTED, "expert projection: K must be a multiple of 128: " + w.name);
+    const int kstep = g->hybrid ? 64 : 128;
+    if (K % kstep != 0 || (int64_t)N * K >= (1ll << 31))
+      return fail(MPK_ERR_UNSUPPORTED, "expert projection: K must be a multiple of 128 (hybrid graphs: 64): " + w.name);
     if ((((uint64_t)x.ptr | (uint64_t)w.ptr) & 15u) != 0)     // rows are gathered / streamed with 16-byte copies
       return fail(MPK_ERR_UNSUPPORTED, "expert projection: input and weight must start on a 16-byte boundary: " + w.name);
     if (cfg.max_num_batched_tokens > kMaxLinearTokens)
@@ -913,19 +966,19 @@ struct Builder {
     const int ntok = std::min(std::max(cfg.max_num_batched_tokens, 1), (int)kMaxLinearTokens);
     auto tile_bytes = [&](int KT) { return fp8 ? moe_fp8_tile_bytes(ntok, KT) : (int64_t)ntok * (KT * 2 + kRowPadBytes); };
     int nkt = 1;
-    while (nkt <= K / 128 && !(K % nkt == 0 && (K / nkt) % 128 == 0 && tile_bytes(K / nkt) <= g->x_tile_bytes)) ++nkt;
-    if (nkt > K / 128) return fail(MPK_ERR_UNSUPPORTED, "cannot tile K for " + w.name);
+    while (nkt <= K / kstep && !(K % nkt == 0 && (K / nkt) % kstep == 0 && tile_bytes(K / nkt) <= g->x_tile_bytes)) ++nkt;
+    if (nkt > K / kstep) return fail(MPK_ERR_UNSUPPORTED, "cannot tile K for " + w.name);
     const int KT = K / nkt;
     const int R = kChunkRows;
     const int step = fp8 ? 128 : 64;
     int KC = std::min(KT, g->chunk_cols * (fp8 ? 2 : 1)) / step * step;
     while (KC > step && KT % KC != 0) KC -= step;
     const int cap = nkt > 1 ? 2 * R : kFp8TaskRows;
-    const int base = N / W, rem = N % W;
+    const int base = N / unit / W, rem = N / unit % W;
     int row = 0;
     for (int i = 0; i < W; ++i) {
       const int worker = (i + rot) % W;
-      const int cnt = base + (i < rem ? 1 : 0);
+      const int cnt = (base + (i < rem ? 1 : 0)) * unit;
       for (int r = row; r < row + cnt; r += cap) {
         TaskDesc d = blank(TASK_MOE_GEMM, li);
         d.flags |= TF_STREAM_AFTER_DEP | (fp8 ? TF_FP8 : 0u);
@@ -936,8 +989,8 @@ struct Builder {
           d.p[6] = (uint64_t)T[l.t[3]].ptr - (uint64_t)ebase * (uint64_t)N * (K / 128) * 4;
           d.p[7] = (uint64_t)T[l.t[1]].ptr;
         }
-        d.a[L_N0] = r; d.a[L_N1] = std::min(r + cap, row + cnt); d.a[L_K] = K; d.a[L_LDW] = K; d.a[L_LDX] = K;
-        d.a[L_LDO] = N; d.a[L_KT] = KT; d.a[L_KC] = KC; d.a[L_ROWS] = R; d.a[L_N] = N;
+        d.a[L_N0] = r; d.a[L_N1] = std::min(r + cap, row + cnt); d.a[L_K] = K; d.a[L_LDW] = K;
+        d.a[L_LDX] = (int)x.ld(); d.a[L_LDO] = (int)y.ld(); d.a[L_EPI] = epi; d.a[L_KT] = KT; d.a[L_KC] = KC; d.a[L_ROWS] = R; d.a[L_N] = N;
         d.a[M_NEXP] = E; d.a[M_NTOPK] = topk; d.a[M_PER_SLOT] = w2 ? 1 : 0; d.a[M_LDR] = (int)idx.dim(1);
         d.a[M_ESTRIDE] = N * K;
         put(worker, d, ex);
@@ -1013,7 +1066,22 @@ struct Builder {
   }
 
   // ---- hybrid graphs: recurrent layers, extended attention, float32 residual stream --------------------------
-  static bool hybrid_op(int op) { return op >= MPK_OP_RESIDUAL_NORM && op <= MPK_OP_MLSTM; }
+  static bool hybrid_op(int op) { return op >= MPK_OP_RESIDUAL_NORM && op <= MPK_OP_GROUPED_LINEAR; }
+  static bool expert_op(int op) { return op == MPK_OP_MOE_TOPK_SIGMOID || op == MPK_OP_MOE_W13_LINEAR || op == MPK_OP_MOE_W2_LINEAR; }
+  static int activation_epilogue(int64_t act) {
+    switch (act) {
+      case MPK_ACT_RELU2: return EPI_RELU2;
+      case MPK_ACT_SOFTCAP: return EPI_SOFTCAP;
+      case MPK_ACT_GATED_SILU: return EPI_GATED_SILU;
+      case MPK_ACT_GATED_GELU_TANH: return EPI_GATED_GELU;
+      default: return EPI_STORE;
+    }
+  }
+  // A tensor's address (0: absent) into two of a descriptor's integers.
+  void put_wide(TaskDesc *d, int i, int tensor) const {
+    const uint64_t p = tensor >= 0 ? (uint64_t)T[tensor].ptr : 0;
+    std::memcpy(&d->a[i], &p, 8);
+  }
   static int round_up(int64_t v, int m) { return (int)((v + m - 1) / m * m); }
   static int bits_of(int64_t p) { return (int)(uint32_t)p; }
 
@@ -1026,11 +1094,12 @@ struct Builder {
       return fail(MPK_ERR_UNSUPPORTED, "hybrid graphs batch at most 64 tokens");
     for (size_t i = 0; i < L.size(); ++i) {
       const LayerInfo &l = L[i];
-      const int act_out = l.op == MPK_OP_RESIDUAL_NORM || l.op == MPK_OP_EXT_ATTENTION || l.op == MPK_OP_RGLRU || l.op == MPK_OP_MLSTM
-                              ? (l.op == MPK_OP_RESIDUAL_NORM ? l.t[4] : l.t.back()) : -1;   // output of the graph's activation type
+      const int act_out = l.op == MPK_OP_RESIDUAL_NORM || l.op == MPK_OP_EXT_ATTENTION || l.op == MPK_OP_RGLRU || l.op == MPK_OP_MLSTM ||
+                                  l.op == MPK_OP_GLA
+                              ? (l.op == MPK_OP_RESIDUAL_NORM ? l.t[4] : l.op == MPK_OP_EXT_ATTENTION ? l.t[3] : l.t.back()) : -1;   // output of the graph's activation type
       if (act_out >= 0 && T[act_out].dtype == MPK_F32) f32 = true;
       if (hybrid_op(l.op) || l.op == MPK_OP_EMBED || l.op == MPK_OP_ARGMAX_PARTIAL || l.op == MPK_OP_ARGMAX_REDUCE ||
-          l.op == MPK_OP_SAMPLING_PARTIAL || l.op == MPK_OP_SAMPLING_REDUCE) continue;
+          l.op == MPK_OP_SAMPLING_PARTIAL || l.op == MPK_OP_SAMPLING_REDUCE || expert_op(l.op)) continue;
       if (l.op != MPK_OP_LINEAR) return fail(MPK_ERR_UNSUPPORTED, "layer " + std::to_string(i) + ": not available in a hybrid graph");
       if (T[l.t[0]].dtype == MPK_F32) f32 = true;
     }
@@ -1073,6 +1142,17 @@ struct Builder {
         return std::max(tile, xattn_stages() >= 3 && D <= 128 ? (int64_t)(16 + 8 * 64) * pitch : 0);
       }
       case MPK_OP_SHORT_CONV: return kMaxLinearTokens * 16 + (mbr + 1) * 4;
+      case MPK_OP_GROUPED_LINEAR: {
+        const int64_t K = T[l.t[1]].dim(2);
+        if (g->hybrid == HYB_F32) return (int64_t)linear_f32_tokens(K) * K * 4;
+        return std::min<int64_t>(linear_tile_bytes(K), x_tile_cap()) + kPartialBytes;   // (a linear task's partial sums stay behind the tile)
+      }
+      case MPK_OP_GLA: {
+        const int64_t dim = l.params[1], rank = T[l.t[1]].dim(1), vc = MPK_MLSTM_COLUMNS(dim), TC = mlstm_tokens(dim), rows = mlstm_rows((int)dim);
+        const int64_t portion = 4 * (TC * (3 * rows + vc) + TC * 8 * vc + TC * rank);
+        const int64_t single = (int64_t)mlstm_rows_per_thread((int)dim) * kConsumerThreads * 32 + 4 * (3 * rows + 16 * vc + rank);
+        return std::max(portion, single);
+      }
       case MPK_OP_RGLRU: {
         int C, TG;
         rglru_plan(l, &C, &TG);
@@ -1095,18 +1175,184 @@ struct Builder {
     if (w.dims.size() != 2 || w.dtype != MPK_BF16 || w.strides[1] != 1 || x.dtype != MPK_F32 || y.dtype != MPK_F32)
       return fail(MPK_ERR_UNSUPPORTED, "32-bit linear: float32 input and output, row-major bf16 weight: " + w.name);
     const int N = (int)w.dim(0), K = (int)w.dim(1);
-    if (x.dim(1) != K || y.dim(1) != N) return fail(MPK_ERR_INVALID, "32-bit linear: shapes disagree for " + w.name);
-    const int nt = std::min(W, N);
+    const int act = l.params.empty() ? 0 : (int)l.params[0];
+    const bool gated = act == MPK_ACT_GATED_SILU || act == MPK_ACT_GATED_GELU_TANH;
+    const int cols = gated ? N / 2 : N;
+    if (x.dim(1) != K || y.dim(1) < cols || (gated && N % 4) || act < 0 || act > MPK_ACT_GATED_GELU_TANH || (act == MPK_ACT_SOFTCAP && l.params.size() < 2))
+      return fail(MPK_ERR_INVALID, "32-bit linear: shapes or activation of " + w.name);
+    const int nt = std::min(W, cols);
     for (int i = 0; i < nt; ++i) {
       TaskDesc d = blank(TASK_LINEAR_F32, li);
       d.p[0] = (uint64_t)w.ptr; d.p[1] = (uint64_t)x.ptr; d.p[2] = (uint64_t)y.ptr;
-      d.a[0] = (int)((int64_t)N * i / nt); d.a[1] = (int)((int64_t)N * (i + 1) / nt);
+      d.a[0] = (int)((int64_t)cols * i / nt); d.a[1] = (int)((int64_t)cols * (i + 1) / nt);
       d.a[2] = K; d.a[3] = (int)w.ld(); d.a[4] = (int)x.ld(); d.a[5] = (int)y.ld();
-      d.a[6] = l.params.empty() ? 0 : (int)l.params[0];
+      d.a[6] = act;
       d.a[7] = linear_f32_tokens(K);
+      d.a[8] = l.params.size() > 1 ? bits_of(l.params[1]) : 0;
       put((i + rot) % W, d, ex);
     }
     g->weight_bytes += (int64_t)N * K * 2;
+    return MPK_OK;
+  }
+
+  int emit_moe_gemm_f32(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const bool w2 = l.op == MPK_OP_MOE_W2_LINEAR;
+    const TensorInfo &x = T[l.t[0]], &w = T[l.t[1]], &idx = T[l.t[2]], &mask = T[l.t[3]], &y = T[l.t[4]];
+    const int E = (int)idx.dim(0), N = (int)w.dim(1), K = (int)w.dim(2), slots = (int)y.dim(1);
+    const int act = !w2 && l.params.size() > 1 ? (int)l.params[1] : 0;
+    const bool gated = act == MPK_ACT_GATED_SILU || act == MPK_ACT_GATED_GELU_TANH;
+    const int cols = gated ? N / 2 : N;
+    if (w.dtype != MPK_BF16 || x.dtype != MPK_F32 || y.dtype != MPK_F32 || w.strides[2] != 1 || w.strides[1] != K || w.strides[0] != (int64_t)N * K)
+      return fail(MPK_ERR_UNSUPPORTED, "32-bit expert projection: float32 input and output, dense bf16 weights: " + w.name);
+    if (w.dim(0) != E || mask.dim(0) != E + 1 || idx.dtype != MPK_I32 || mask.dtype != MPK_I32 || x.dim(x.dims.size() - 1) < K || y.dim(2) < cols ||
+        (w2 && x.dim(1) != slots) || (act && !gated) || (gated && N % 4))
+      return fail(MPK_ERR_INVALID, "32-bit expert projection: shapes of " + w.name + " and its routing tensors disagree");
+    const int nt = std::min(W, cols);
+    for (int i = 0; i < nt; ++i) {
+      TaskDesc d = blank(TASK_MOE_GEMM_F32, li);
+      d.p[0] = (uint64_t)w.ptr; d.p[1] = (uint64_t)x.ptr; d.p[2] = (uint64_t)y.ptr; d.p[4] = (uint64_t)idx.ptr; d.p[5] = (uint64_t)mask.ptr;
+      d.a[0] = (int)((int64_t)cols * i / nt); d.a[1] = (int)((int64_t)cols * (i + 1) / nt); d.a[2] = K;
+      d.a[4] = (int)x.ld(); d.a[5] = (int)y.ld(); d.a[6] = act; d.a[7] = linear_f32_tokens(K); d.a[8] = w2 ? 1 : 0; d.a[9] = slots;
+      d.a[10] = (int)idx.dim(1); d.a[11] = E; d.a[12] = N;
+      put((i + rot) % W, d, ex);
+    }
+    return MPK_OK;
+  }
+
+  // One linear per group of columns: the same tasks as a linear layer's, cut at the group borders.
+  int emit_grouped_linear(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &x = T[l.t[0]], &w = T[l.t[1]], &y = T[l.t[2]];
+    if (l.params.size() < 3 || w.dims.size() != 3) return fail(MPK_ERR_INVALID, "grouped linear: weight [groups, N, K], params [x stride, y column, y stride]");
+    const int G = (int)w.dim(0), N = (int)w.dim(1), K = (int)w.dim(2);
+    const int64_t xs = l.params[0], yc = l.params[1], ys = l.params[2];
+    if (w.dtype != MPK_BF16 || w.strides[2] != 1 || w.strides[1] != K || w.strides[0] != (int64_t)N * K || x.dtype != act_dtype() ||
+        (y.dtype != act_dtype() && y.dtype != MPK_F32))
+      return fail(MPK_ERR_UNSUPPORTED, "grouped linear: dense bf16 weight, input and output of the graph's activation type: " + w.name);
+    if (xs < K || yc < 0 || ys < N || (G - 1) * xs + K > x.dim(1) || yc + (G - 1) * ys + N > y.dim(1))
+      return fail(MPK_ERR_INVALID, "grouped linear: columns outside the input or output: " + w.name);
+    const bool f32 = g->hybrid == HYB_F32;
+    if (!f32 && (K % 16 || xs % 8 || ((uint64_t)x.ptr & 15) || ((uint64_t)w.ptr & 15) || x.ld() % 8))
+      return fail(MPK_ERR_UNSUPPORTED, "grouped linear: K a multiple of 16, input columns on 16-byte boundaries: " + w.name);
+    const int64_t rows = (int64_t)G * N;
+    const bool tc = !f32 && g->use_tmem && tc_linear(K);
+    if (!f32 && linear_tile_bytes(K) > g->x_tile_bytes) return fail(MPK_ERR_UNSUPPORTED, "grouped linear: K too large: " + w.name);
+    const int esz_x = f32 ? 4 : 2, esz_y = y.dtype == MPK_F32 ? 4 : 2;
+    int KC = std::min(K, g->chunk_cols) / 16 * 16;
+    while (!f32 && KC > 16 && K % KC != 0) KC -= 16;
+    // tcgen05: row tiles of at most 128 rows; a task holds as many accumulators as fit
+    const int64_t widest = std::min<int64_t>((rows + W - 1) / W, N);
+    int rb = 0, nkb = 1;
+    if (tc) {
+      const int tiles = (int)((widest + 127) / 128);
+      rb = (int)std::min<int64_t>(128, ((widest + tiles - 1) / tiles + 7) / 8 * 8);
+      nkb = std::max(1, std::min(K / kTcKBlock, g->stage_bytes / (rb * 128)));
+      while (K / kTcKBlock % nkb) --nkb;
+      g->exec[ex].tc_rows = rb;
+      g->exec[ex].tc_kblocks = nkb;
+    }
+    const int cap = tc ? std::max(1, kTcAccCols / tc_np()) * rb : 1 << 20;
+    for (int i = 0; i < W; ++i) {
+      const int64_t end = rows * (i + 1) / W;
+      int last = -1;
+      for (int64_t r = rows * i / W; r < end;) {
+        const int grp = (int)(r / N), n0 = (int)(r - (int64_t)grp * N);
+        const int n1 = (int)std::min<int64_t>(std::min<int64_t>(N, end - (int64_t)grp * N), n0 + cap);
+        TaskDesc d = blank(f32 ? TASK_LINEAR_F32 : TASK_LINEAR, li);
+        d.p[0] = (uint64_t)w.ptr + (uint64_t)grp * N * K * 2;
+        d.p[1] = (uint64_t)x.ptr + (uint64_t)grp * xs * esz_x;
+        d.p[2] = (uint64_t)y.ptr + (uint64_t)(yc + grp * ys) * esz_y;
+        if (f32) {
+          d.a[0] = n0; d.a[1] = n1; d.a[2] = K; d.a[3] = K; d.a[4] = (int)x.ld(); d.a[5] = (int)y.ld(); d.a[7] = linear_f32_tokens(K);
+        } else {
+          if (grp == last) d.flags |= TF_SAME_X_AS_PREV;
+          d.a[L_N0] = n0; d.a[L_N1] = n1; d.a[L_K] = K; d.a[L_LDW] = K; d.a[L_LDX] = (int)x.ld(); d.a[L_LDO] = (int)y.ld();
+          d.a[L_PRO] = PRO_PLAIN; d.a[L_EPI] = y.dtype == MPK_F32 ? EPI_STORE_F32 : EPI_STORE; d.a[L_GROUPS] = 1;
+          d.a[L_KT] = K; d.a[L_KC] = KC; d.a[L_ROWS] = kChunkRows; d.a[L_N] = N;
+          if (tc) {
+            d.flags |= TF_TC;
+            d.a[L_KC] = nkb * kTcKBlock; d.a[L_ROWS] = rb; d.a[L_TMAP] = (int)g->tmaps.size();
+            TmapSpec m;
+            m.base = d.p[0] + (uint64_t)n0 * K * 2;
+            m.rows = n1 - n0; m.ld_bytes = (int64_t)K * 2; m.kblocks = K / kTcKBlock; m.box_rows = rb; m.box_kblocks = nkb; m.elt_bytes = 2;
+            g->tmaps.push_back(m);
+          }
+        }
+        put((i + rot) % W, d, ex);
+        last = grp;
+        r += n1 - n0;
+      }
+    }
+    g->weight_bytes += rows * K * 2;
+    return MPK_OK;
+  }
+
+  int emit_latent_append(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &pr = T[l.t[0]], &nw = T[l.t[1]], &q = T[l.t[2]], &kc = T[l.t[3]], &cs = T[l.t[4]], &sn = T[l.t[5]];
+    if (l.params.size() < 6) return fail(MPK_ERR_INVALID, "latent_append needs 6 parameters");
+    const int H = (int)l.params[0], rank = (int)l.params[1], rdim = (int)l.params[2];
+    if (!batch_meta_given()) return fail(MPK_ERR_INVALID, "latent_append needs the batch meta tensors");
+    if (pr.dtype != MPK_F32 || nw.dtype != MPK_BF16 || q.dtype != act_dtype() || kc.dtype != act_dtype() || cs.dtype != MPK_F32 || sn.dtype != MPK_F32)
+      return fail(MPK_ERR_INVALID, "latent_append: float32 projections and tables, bf16 norm weight, q and cache of the graph's activation type");
+    if (H < 1 || rank < 1 || rdim < 0 || rdim % 2 || nw.dim(0) < rank || kc.dims.size() != 4 || kc.dim(1) != cfg.page_size || kc.dim(2) != 1 ||
+        kc.dim(3) < rank + rdim || kc.dim(3) % 8 || q.dim(1) != H * kc.dim(3))
+      return fail(MPK_ERR_INVALID, "latent_append: cache [pages, page, 1, latent + rotated size rounded up to 8], q [tokens, heads x that]");
+    if (l.params[3] < 0 || l.params[4] < 0 || l.params[3] + (int64_t)H * rdim > pr.dim(1) || l.params[4] + rank + rdim > pr.dim(1))
+      return fail(MPK_ERR_INVALID, "latent_append: columns outside the projections");
+    if (rdim > 0 && (cs.dims.size() != 2 || cs.dim(1) != rdim / 2 || sn.dim(1) != rdim / 2 || cs.dim(0) != sn.dim(0)))
+      return fail(MPK_ERR_INVALID, "latent_append: cos / sin tables [positions, rotated dims / 2]");
+    const int nt = std::max(1, std::min(W, (nb_max * (H + 1) + 7) / 8));
+    for (int i = 0; i < nt; ++i) {
+      TaskDesc d = blank(TASK_LATENT_APPEND, li);
+      d.p[0] = (uint64_t)pr.ptr; d.p[1] = (uint64_t)nw.ptr; d.p[2] = (uint64_t)q.ptr; d.p[3] = (uint64_t)kc.ptr;
+      d.p[4] = (uint64_t)cs.ptr; d.p[5] = (uint64_t)sn.ptr;
+      d.a[LA_T0] = i; d.a[LA_T1] = nt; d.a[LA_LDP] = (int)pr.ld(); d.a[LA_QOFF] = (int)l.params[3]; d.a[LA_KVOFF] = (int)l.params[4];
+      d.a[LA_H] = H; d.a[LA_RANK] = rank; d.a[LA_ROT] = rdim; d.a[LA_DIMP] = (int)kc.dim(3); d.a[LA_EPS] = bits_of(l.params[5]);
+      d.a[LA_PAGE] = cfg.page_size; d.a[LA_LDQ] = (int)q.ld(); d.a[LA_ROWS] = rdim > 0 ? (int)cs.dim(0) : 1;
+      put((i + rot) % W, d, ex);
+    }
+    return MPK_OK;
+  }
+
+  int emit_gla(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &pr = T[l.t[0]], &a2 = T[l.t[1]], &S = T[l.t[4]], &raw = T[l.t[5]], &o = T[l.t[6]];
+    if (l.params.size() < 12 || a2.dims.size() != 2) return fail(MPK_ERR_INVALID, "gla: a2 [heads x dim, rank], 12 parameters");
+    const int H = (int)l.params[0], dim = (int)l.params[1], vdim = (int)l.params[2], chunks = (int)l.params[11], rank = (int)a2.dim(1);
+    const int slots = cfg.max_num_batched_requests;
+    if (!batch_meta_given()) return fail(MPK_ERR_INVALID, "gla needs the batch meta tensors");
+    if (H < 1 || dim < 1 || vdim < 1 || rank < 1) return fail(MPK_ERR_INVALID, "gla: head count or sizes");
+    if (dim > 1024 || rank > 512) return fail(MPK_ERR_UNSUPPORTED, "gla: key sizes up to 1024, decay rank up to 512");
+    if (pr.dtype != MPK_F32 || S.dtype != MPK_F32 || raw.dtype != MPK_F32 || o.dtype != act_dtype() || S.dims.size() != 4 || S.dim(0) < slots ||
+        S.dim(1) != H || S.dim(2) != dim || S.dim(3) < vdim || S.dim(3) % 4 || raw.dim(1) < (int64_t)H * vdim || o.dim(1) < (int64_t)H * vdim)
+      return fail(MPK_ERR_INVALID, "gla: state [slots, heads, dim, vdim rounded up to 4], scratch and output [tokens, heads x vdim]");
+    for (int i = 3; i < 8; ++i) {
+      const int64_t w = i < 5 ? (int64_t)H * dim : (i < 7 ? (int64_t)H * vdim : rank);
+      if (l.params[i] < 0 || l.params[i] + w > pr.dim(1)) return fail(MPK_ERR_INVALID, "gla: columns outside the projections");
+    }
+    if (a2.dtype != MPK_BF16 || a2.dim(0) != (int64_t)H * dim || a2.strides[0] != rank || a2.strides[1] != 1 || T[l.t[2]].dtype != MPK_BF16 ||
+        T[l.t[2]].dim(0) < (int64_t)H * dim || T[l.t[3]].dtype != MPK_BF16 || T[l.t[3]].dim(0) < vdim)
+      return fail(MPK_ERR_INVALID, "gla: bf16 a2 [heads x dim, rank], bias [heads x dim], norm [vdim]");
+    const int vc = MPK_MLSTM_COLUMNS(dim), nsub = (vdim + vc - 1) / vc;
+    if (chunks < 1 || chunks > nsub) return fail(MPK_ERR_INVALID, "gla: chunk count");
+    for (int s = 0; s < slots; ++s)
+      for (int h = 0; h < H; ++h)
+        for (int ch = 0; ch < chunks; ++ch) {
+          TaskDesc d = blank(TASK_GLA, li);
+          for (int k = 0; k < 5; ++k) d.p[k] = (uint64_t)T[l.t[k]].ptr;
+          d.p[6] = (uint64_t)raw.ptr; d.p[7] = (uint64_t)o.ptr;
+          d.a[GA_SLOT] = s; d.a[GA_HEAD] = h; d.a[GA_CHUNK] = ch; d.a[GA_NCHUNK] = chunks; d.a[GA_H] = H; d.a[GA_DIM] = dim;
+          d.a[GA_VDIM] = vdim; d.a[GA_VDIMP] = (int)S.dim(3); d.a[GA_V0] = nsub * ch / chunks * vc;
+          d.a[GA_V1] = std::min(nsub * (ch + 1) / chunks * vc, (int)S.dim(3));
+          d.a[GA_EPS] = bits_of(l.params[9]); d.a[GA_LDP] = (int)pr.ld(); d.a[GA_QOFF] = (int)l.params[3]; d.a[GA_KOFF] = (int)l.params[4];
+          d.a[GA_VOFF] = (int)l.params[5]; d.a[GA_GOFF] = (int)l.params[6]; d.a[GA_AOFF] = (int)l.params[7]; d.a[GA_RANK] = rank;
+          d.a[GA_LDO] = (int)o.ld(); d.a[GA_QSCALE] = bits_of(l.params[10]); d.a[GA_TICKET] = hybrid_tickets + s * H + h;
+          d.a[GA_TC] = mlstm_tokens(dim); d.a[GA_LDR] = (int)raw.ld(); d.a[GA_INVTAU] = bits_of(l.params[8]);
+          put(((s * H + h) * chunks + ch + rot) % W, d, ex);
+        }
+    hybrid_tickets += slots * H;
     return MPK_OK;
   }
 
@@ -1120,6 +1366,17 @@ struct Builder {
     for (int i = 2; i < 4; ++i)
       if (l.t[i] >= 0 && (T[l.t[i]].dtype != MPK_BF16 || T[l.t[i]].dim(0) != D)) return fail(MPK_ERR_INVALID, "residual_norm: weights must be bf16 [width]");
     if ((l.t[3] >= 0) != (l.t[4] >= 0)) return fail(MPK_ERR_INVALID, "residual_norm: output and its norm weight go together");
+    const int bias = norm_tensor(l, 6), add = norm_tensor(l, 7), row = norm_tensor(l, 8), exps = norm_tensor(l, 9), ew = norm_tensor(l, 10), gate = norm_tensor(l, 11);
+    if ((bias >= 0 && (l.t[3] < 0 || T[bias].dtype != MPK_BF16 || T[bias].dim(0) != D)) || (row >= 0 && (T[row].dtype != MPK_BF16 || T[row].dim(0) != D)) ||
+        (add >= 0 && (T[add].dtype != MPK_F32 || T[add].dims.size() != 2 || T[add].dim(1) != D)))
+      return fail(MPK_ERR_INVALID, "residual_norm: bf16 bias and row [width], float32 added stream [tokens, width]");
+    if ((exps >= 0) != (ew >= 0) || (exps >= 0 && (T[exps].dtype != MPK_F32 || T[exps].dims.size() != 3 || T[exps].dim(2) != D || T[exps].strides[1] != D ||
+                                                   T[exps].strides[0] != T[exps].dim(1) * D || T[ew].dtype != MPK_F32 || T[ew].dim(1) != T[exps].dim(1))))
+      return fail(MPK_ERR_INVALID, "residual_norm: expert outputs float32 [tokens, slots, width] with weights [tokens, slots]");
+    if (gate >= 0 && (l.t[1] < 0 || T[gate].dtype != MPK_F32 || l.params.size() < 4 || l.params[3] < 0 || l.params[3] >= T[gate].dim(1)))
+      return fail(MPK_ERR_INVALID, "residual_norm: gate column of a float32 tensor");
+    if (l.t[2] >= 0 && (exps >= 0 || gate >= 0 || (norm_flags(l) & 4)))
+      return fail(MPK_ERR_UNSUPPORTED, "residual_norm: a norm of y goes with RMS norms and without experts");
     if (l.t[4] >= 0 && (T[l.t[4]].dtype != act_dtype() || T[l.t[4]].dim(1) < D)) return fail(MPK_ERR_INVALID, "residual_norm: output type or width");
     const TensorInfo &xo = T[resnorm_out(l)];
     if (xo.dtype != MPK_F32 || xo.dim(1) != D) return fail(MPK_ERR_INVALID, "residual_norm: the new stream must be float32 of x's width");
@@ -1131,7 +1388,16 @@ struct Builder {
       d.a[0] = (int)((int64_t)rows * i / nt); d.a[1] = (int)((int64_t)rows * (i + 1) / nt); d.a[2] = D;
       d.a[3] = (int)x.ld(); d.a[4] = l.t[1] >= 0 ? (int)T[l.t[1]].ld() : 0; d.a[5] = l.t[4] >= 0 ? (int)T[l.t[4]].ld() : 0;
       d.a[6] = bits_of(l.params[0]);
-      d.a[7] = (g->hybrid == HYB_F32 ? 1 : 0) | (l.params[1] ? 2 : 0);
+      d.a[7] = (g->hybrid == HYB_F32 ? 1 : 0) | norm_flags(l);
+      put_wide(&d, RN_BIAS, bias); put_wide(&d, RN_ADD, add); put_wide(&d, RN_ROW, row); put_wide(&d, RN_EXP, exps); put_wide(&d, RN_EW, ew);
+      if (gate >= 0) {
+        const uint64_t gp = (uint64_t)T[gate].ptr + 4ull * l.params[3];
+        std::memcpy(&d.a[RN_GATE], &gp, 8);
+        d.a[RN_LDGATE] = (int)T[gate].ld();
+      }
+      d.a[RN_LDADD] = add >= 0 ? (int)T[add].ld() : 0;
+      d.a[RN_SLOTS] = exps >= 0 ? (int)T[exps].dim(1) : 0;
+      d.a[RN_LDEW] = ew >= 0 ? (int)T[ew].ld() : 0;
       put((i + rot) % W, d, ex);
     }
     return MPK_OK;
@@ -1181,8 +1447,11 @@ struct Builder {
       return fail(MPK_ERR_INVALID, "ext_attention: shapes of q, caches and output disagree");
     if (q.dtype != act_dtype() || kc.dtype != act_dtype() || vc.dtype != act_dtype() || o.dtype != act_dtype())
       return fail(MPK_ERR_INVALID, "ext_attention: q, caches and output must have the graph's activation type");
-    if (std::max(kc.dim(3), vc.dim(3)) > (g->hybrid == HYB_F32 ? 512 : 256))
-      return fail(MPK_ERR_UNSUPPORTED, "ext_attention: head sizes up to 256 (512 in 32-bit graphs)");
+    if (g->hybrid == HYB_F32 ? kc.dim(3) > 1024 || vdim > 512 : std::max(kc.dim(3), vc.dim(3)) > 256)
+      return fail(MPK_ERR_UNSUPPORTED, "ext_attention: head sizes up to 256 (32-bit graphs: keys up to 1024, values up to 512)");
+    const int sinks = l.t.size() > 4 ? l.t[4] : -1;
+    if (sinks >= 0 && (T[sinks].dtype != MPK_BF16 || T[sinks].dim(0) < hq || !l.params[6])) return fail(MPK_ERR_INVALID, "ext_attention: bf16 sinks [heads], sink = 1");
+    const bool shared = kc.storage == vc.storage;
     const int slots = cfg.max_num_batched_requests, max_seq = std::max(cfg.max_seq_length, 1);
     // chunks of a (request, kv head): enough to occupy the workers, at most ~2048 keys each, at least 64
     int NC = std::max(std::max(1, W / std::max(slots * hkv, 1)), (max_seq + 2047) / 2048);
@@ -1193,6 +1462,8 @@ struct Builder {
         for (int ch = 0; ch < NC; ++ch) {
           TaskDesc d = blank(TASK_EXT_ATTENTION, li);
           for (int i = 0; i < 4; ++i) d.p[i] = (uint64_t)T[l.t[i]].ptr;
+          d.p[4] = sinks >= 0 ? (uint64_t)T[sinks].ptr : 0;
+          d.a[XA_SHARED] = shared ? 1 : 0;
           d.a[XA_SLOT] = s; d.a[XA_HEAD] = h; d.a[XA_CHUNK] = ch; d.a[XA_NCHUNK] = NC; d.a[XA_HQ] = hq; d.a[XA_HKV] = hkv;
           d.a[XA_DIMP] = (int)kc.dim(3); d.a[XA_VDIM] = vdim; d.a[XA_VDIMP] = (int)vc.dim(3); d.a[XA_PAGE] = cfg.page_size;
           d.a[XA_LDQ] = (int)q.ld(); d.a[XA_LDO] = (int)o.ld(); d.a[XA_OCOL] = ocol;
@@ -1327,6 +1598,9 @@ struct Builder {
       case MPK_OP_SHORT_CONV: return emit_short_conv(li, ex);
       case MPK_OP_RGLRU: return emit_rglru(li, ex);
       case MPK_OP_MLSTM: return emit_mlstm(li, ex);
+      case MPK_OP_GLA: return emit_gla(li, ex);
+      case MPK_OP_LATENT_APPEND: return emit_latent_append(li, ex);
+      case MPK_OP_GROUPED_LINEAR: return emit_grouped_linear(li, ex);
       case MPK_OP_LINEAR_FP8: case MPK_OP_LINEAR_FP8_RESIDUAL:
         return emit_linear_fp8(li, ex);
       case MPK_OP_QUANTIZE_FP8:
@@ -1354,7 +1628,9 @@ struct Builder {
       case MPK_OP_MOE_TOPK_SIGMOID: {
         const TensorInfo &lg = T[l.t[0]], &bias = T[l.t[1]], &w = T[l.t[2]], &idx = T[l.t[3]], &mask = T[l.t[4]];
         if (l.params.size() < 3) return fail(MPK_ERR_INVALID, "sigmoid routing needs [num_groups, topk_group, scaling_bits]");
-        const int E = (int)lg.dim(1), topk = (int)w.dim(1), groups = (int)l.params[0], keep = (int)l.params[1];
+        // (hybrid graphs: the router's logits may be the leading columns of a wider tensor)
+        const int E = g->hybrid ? (int)idx.dim(0) : (int)lg.dim(1), topk = (int)w.dim(1), groups = (int)l.params[0], keep = (int)l.params[1];
+        if (lg.dim(1) < E || (g->hybrid && !keeps_logits(l))) return fail(MPK_ERR_INVALID, "sigmoid routing: fewer logits than experts, or (hybrid graphs) logits that are not kept");
         if ((lg.dtype != MPK_BF16 && lg.dtype != MPK_F32) || bias.dtype != MPK_F32 || w.dtype != MPK_F32 ||
             idx.dtype != MPK_I32 || mask.dtype != MPK_I32)
           return fail(MPK_ERR_INVALID, "sigmoid routing: logits bf16/f32, bias and weights f32, indices and mask int32");
@@ -1369,6 +1645,7 @@ struct Builder {
         // optional params [3], [4]: first and one-past-last expert this rank runs (expert parallelism)
         d.a[9] = l.params.size() > 4 ? (int)l.params[3] : 0;
         d.a[10] = l.params.size() > 4 ? (int)l.params[4] : E;
+        d.a[12] = keeps_logits(l) ? 1 : 0;
         if (d.a[9] < 0 || d.a[10] > E || d.a[9] >= d.a[10] || topk > 32)
           return fail(MPK_ERR_INVALID, "sigmoid routing: bad local expert range");
         put(rot % W, d, ex);
@@ -1476,7 +1753,7 @@ struct Builder {
           // the table may be wider than the stream (padded to the projections' k granularity)
           if (y.dtype != MPK_F32 || tab.dtype != MPK_BF16 || tab.dim(1) < y.dim(1)) return fail(MPK_ERR_INVALID, "embed in a hybrid graph: bf16 table, float32 output");
           emit_token_rows(TASK_EMBED_F32, li, ex, (uint64_t)T[l.t[0]].ptr, (uint64_t)tab.ptr, (uint64_t)y.ptr,
-                          (int)y.dim(1), (int)tab.ld(), (int)y.ld(), (int)tab.dim(0), 0, mbt);
+                          (int)y.dim(1), (int)tab.ld(), (int)y.ld(), (int)tab.dim(0), l.params.size() > 1 ? bits_of(l.params[1]) : float_bits(1.0f), mbt);
           return MPK_OK;
         }
         if (tab.dim(1) % 8 != 0) return fail(MPK_ERR_UNSUPPORTED, "embedding width must be a multiple of 8");
@@ -1618,8 +1895,17 @@ struct Builder {
   }
 
   // output tensor a layer writes only a column range of, and that range's first column
-  int sliced_output(const LayerInfo &l) const { return l.op == MPK_OP_EXT_ATTENTION ? l.t[3] : (l.op == MPK_OP_RGLRU ? l.t[9] : -1); }
+  int sliced_output(const LayerInfo &l) const {
+    switch (l.op) {
+      case MPK_OP_EXT_ATTENTION: return l.t[3];
+      case MPK_OP_RGLRU: return l.t[9];
+      case MPK_OP_LATENT_APPEND: return l.t[2];     // the rotated columns of every head
+      case MPK_OP_GROUPED_LINEAR: return l.t[2];    // N columns of every group
+      default: return -1;
+    }
+  }
   int slice_column(const LayerInfo &l) const {
+    // (a latent layer's rotated columns begin behind the latent ones, parameter 1)
     const size_t i = l.op == MPK_OP_EXT_ATTENTION ? 3 : 1;
     return l.params.size() > i ? (int)l.params[i] : 0;
   }

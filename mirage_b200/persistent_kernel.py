@@ -317,8 +317,10 @@ class PersistentKernel:
         return N.check(self._h, N.lib.mpk_add_layer(self._h, op, arr, n, grid, pr, len(params)))
 
     def embed_layer(self, input: DTensor, weight: DTensor, output: DTensor, grid_dim: tuple, block_dim: tuple,
-                    input_source: int = 0):
-        self._layer(N.OP_EMBED, [input, weight, output], grid_dim, [input_source])
+                    input_source: int = 0, factor: Optional[float] = None):
+        """`factor` (hybrid graphs) multiplies the rows."""
+        self._layer(N.OP_EMBED, [input, weight, output], grid_dim,
+                    [input_source] if factor is None else [input_source, self._bits(factor)])
 
     def rmsnorm_layer(self, input: DTensor, weight: DTensor, output: DTensor, grid_dim: tuple, block_dim: tuple):
         assert input.num_dims == 2 and output.num_dims == 2
@@ -329,14 +331,31 @@ class PersistentKernel:
         assert input.num_dims == 2 and weight_linear.num_dims == 2 and output.num_dims == 2
         self._layer(N.OP_RMSNORM_LINEAR, [input, weight_norm, weight_linear, output], grid_dim)
 
-    LINEAR_ACTIVATIONS = {None: 0, "relu2": 1}
+    # mpk_activation of include/mpk_b200.h
+    LINEAR_ACTIVATIONS = {None: 0, "relu2": 1, "softcap": 2, "gated_silu": 3, "gated_gelu_tanh": 4}
 
     def linear_layer(self, input: DTensor, weight: DTensor, output: DTensor, grid_dim: tuple, block_dim: tuple,
-                     activation: str = None):
-        """`activation` (squared relu, in hybrid graphs) is applied to the fp32 accumulator before the store."""
+                     activation: str = None, softcap: float = 0.0):
+        """`activation` (hybrid graphs) is applied to the fp32 accumulator before the store: squared relu, softcap * tanh(y /
+        softcap), or a gated form act(gate) * up over weight rows from `interleave_gated`, which has half as many outputs."""
         assert input.num_dims == 2 and weight.num_dims == 2 and output.num_dims == 2
         act = self.LINEAR_ACTIVATIONS[activation]
-        self._layer(N.OP_LINEAR, [input, weight, output], grid_dim, [act] if act else [])
+        params = [act, self._bits(softcap)] if activation == "softcap" else [act] if act else []
+        self._layer(N.OP_LINEAR, [input, weight, output], grid_dim, params)
+
+    @staticmethod
+    def interleave_gated(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+        """[.., I, K] x 2 -> [.., 2 I, K] in the row order of gated linears (two gate rows, two up rows, ...); I even."""
+        assert gate.shape == up.shape and gate.shape[-2] % 2 == 0
+        g, u = (t.unflatten(-2, (-1, 2)) for t in (gate, up))
+        return torch.cat([g, u], -2).flatten(-3, -2)
+
+    def grouped_linear_layer(self, input: DTensor, weight: DTensor, output: DTensor, *, in_stride: int, out_col: int = 0,
+                             out_stride: int):
+        """One linear per group: weight [groups, N, K]; group g maps input columns [g * in_stride, + K) to output columns
+        [out_col + g * out_stride, + N)."""
+        assert weight.num_dims == 3
+        self._layer(N.OP_GROUPED_LINEAR, [input, weight, output], (1, 1, 1), [in_stride, out_col, out_stride])
 
     def linear_with_residual_layer(self, input: DTensor, weight: DTensor, residual: DTensor, output: DTensor,
                                    grid_dim: tuple, block_dim: tuple):
@@ -507,14 +526,24 @@ class PersistentKernel:
 
     def residual_norm_layer(self, x: DTensor, y: Optional[DTensor] = None, post_weight: Optional[DTensor] = None,
                             norm_weight: Optional[DTensor] = None, output: Optional[DTensor] = None, eps: float = 1e-6,
-                            zero_centered: bool = False, x_out: Optional[DTensor] = None):
+                            zero_centered: bool = False, x_out: Optional[DTensor] = None, layer_norm: bool = False,
+                            norm_bias: Optional[DTensor] = None, added: Optional[DTensor] = None,
+                            added_row: Optional[DTensor] = None,
+                            experts: Optional[Tuple[DTensor, DTensor]] = None,
+                            y_gate: Optional[Tuple[DTensor, int]] = None):
         """x += rmsnorm(y) * w_post on the float32 stream `x` (x += y without `post_weight`, x unchanged without `y`),
         then output = rmsnorm(x) * w_norm.  `zero_centered`: both weights are stored around zero (1 + w is applied).
         `x_out` receives the new stream instead of `x`; with it, graphs of one or two tokens fold the layer into the linear
-        that reads `output`."""
+        that reads `output`.  `layer_norm` makes the output norm a layer norm (with `norm_bias`) instead of an RMS norm.
+        Further terms of the sum: `added` (float32 [tokens, width]), `added_row` (bf16 [width], for every token), `experts`
+        (outputs [tokens, slots, width] and weights [tokens, slots], both float32); `y_gate` = (float32 tensor, column)
+        multiplies `y` by the column's sigmoid."""
         assert x.num_dims == 2
-        self._layer(N.OP_RESIDUAL_NORM, [x, y, post_weight, norm_weight, output, x_out], (1, 1, 1),
-                    [self._bits(eps), int(zero_centered)])
+        gate, column = y_gate if y_gate else (None, 0)
+        exp_out, exp_w = experts if experts else (None, None)
+        self._layer(N.OP_RESIDUAL_NORM, [x, y, post_weight, norm_weight, output, x_out, norm_bias, added, added_row, exp_out,
+                                         exp_w, gate], (1, 1, 1),
+                    [self._bits(eps), int(zero_centered), int(layer_norm), column])
 
     def qkv_append_layer(self, proj: DTensor, q: DTensor, k_cache: DTensor, v_cache: DTensor, cos: DTensor, sin: DTensor,
                          *, heads: int, kv_heads: int, dim: int, vdim: int, q_col: int, k_col: int, v_col: int,
@@ -527,13 +556,23 @@ class PersistentKernel:
 
     def ext_attention_layer(self, q: DTensor, k_cache: DTensor, v_cache: DTensor, output: DTensor, *, heads: int,
                             kv_heads: int, vdim: int, scale: float, softcap: float = 0.0, sink: bool = False,
-                            out_col: int = 0, out_scale: float = 1.0):
-        """Causal paged attention over rows a qkv_append_layer wrote.  score = softcap * tanh(scale * q.k / softcap) (no
-        cap at 0); `sink` adds one to the softmax denominator; the result times `out_scale` goes to columns
-        [out_col, out_col + heads * vdim) of `output`."""
-        self._layer(N.OP_EXT_ATTENTION, [q, k_cache, v_cache, output], (1, 1, 1),
-                    [heads, kv_heads, vdim, out_col, self._bits(scale), self._bits(softcap or 0.0), int(sink),
-                     self._bits(out_scale)])
+                            sinks: Optional[DTensor] = None, out_col: int = 0, out_scale: float = 1.0):
+        """Causal paged attention over rows a qkv_append_layer or latent_append_layer wrote.  score = softcap *
+        tanh(scale * q.k / softcap) (no cap at 0); `sink` adds one to the softmax denominator, `sinks` (bf16 [heads]) adds
+        exp(sinks[head]); the result times `out_scale` goes to columns [out_col, out_col + heads * vdim) of `output`.
+        `v_cache` may be `k_cache`: the leading `vdim` columns of a key are then its value."""
+        self._layer(N.OP_EXT_ATTENTION, [q, k_cache, v_cache, output, sinks], (1, 1, 1),
+                    [heads, kv_heads, vdim, out_col, self._bits(scale), self._bits(softcap or 0.0),
+                     int(sink or sinks is not None), self._bits(out_scale)])
+
+    def latent_append_layer(self, proj: DTensor, latent_norm: DTensor, q: DTensor, cache: DTensor, cos: DTensor, sin: DTensor,
+                            *, heads: int, rank: int, rot_dims: int, q_col: int, kv_col: int, eps: float):
+        """Latent attention (DeepSeek-AI, "DeepSeek-V2: A Strong, Economical, and Efficient Mixture-of-Experts Language
+        Model"): columns [kv_col, + rank + rot_dims) of the float32 projections become a cache row [pages, page, 1, width]
+        (the RMS-normed latent, then the rotated key part all heads share); `rot_dims` columns per head from `q_col` are
+        rotated into q [tokens, heads * width] behind the head's `rank` latent columns."""
+        self._layer(N.OP_LATENT_APPEND, [proj, latent_norm, q, cache, cos, sin], (1, 1, 1),
+                    [heads, rank, rot_dims, q_col, kv_col, self._bits(eps)])
 
     def short_conv_layer(self, input: DTensor, taps: DTensor, state: DTensor, output: DTensor, *,
                          input_bias: Optional[DTensor] = None, bias: Optional[DTensor] = None, in_col: int = 0,
@@ -570,11 +609,24 @@ class PersistentKernel:
                     [heads, dim, vdim, q_col, k_col, v_col, gate_col, i_col, f_col, self._bits(gate_cap), self._bits(eps),
                      self._bits(q_scale), nm_state.dim(2)])
 
+    def gla_layer(self, proj: DTensor, a2: DTensor, a2_bias: DTensor, norm: DTensor, state: DTensor, scratch: DTensor,
+                  output: DTensor, *, heads: int, dim: int, vdim: int, q_col: int, k_col: int, v_col: int, gate_col: int,
+                  a1_col: int, tau: float, eps: float, q_scale: float, chunks: int):
+        """Gated linear attention (Yang et al., "Gated Linear Attention Transformers with Hardware-Efficient Training"): a
+        matrix state per head whose rows decay by sigmoid(a2 . proj[:, a1_col:] + a2_bias)^(1 / tau); float32 state [slots,
+        heads, dim, vdim up to a multiple of 4], per-head RMS norm with the shared weight `norm` [vdim], times silu of the
+        gate columns.  `chunks`: column ranges a head is cut into (`mlstm_chunks`)."""
+        self._layer(N.OP_GLA, [proj, a2, a2_bias, norm, state, scratch, output], (1, 1, 1),
+                    [heads, dim, vdim, q_col, k_col, v_col, gate_col, a1_col, self._bits(1.0 / tau), self._bits(eps),
+                     self._bits(q_scale), chunks])
+
     # ---- mixture of experts (persistent_kernel.py:1385-1704 of the reference) -------------------------------
     def moe_topk_sigmoid_routing_layer(self, input: DTensor, bias: DTensor, output: tuple, grid_dim: tuple,
                                        block_dim: tuple, num_groups: int = 8, topk_group: int = 4,
-                                       routed_scaling_factor: float = 2.5, local_experts: tuple = None):
-        """input [B, E] logits (zeroed by the task), bias [E] float32; output = (topk_weight [B, topk] float32,
+                                       routed_scaling_factor: float = 2.5, local_experts: tuple = None,
+                                       keep_logits: bool = False):
+        """input [B, E] logits (zeroed by the task unless `keep_logits`; hybrid graphs keep them, and may pass a wider tensor
+        whose leading columns they are), bias [E] float32; output = (topk_weight [B, topk] float32,
         routing_indices [E, B] int32 holding slot + 1 or 0, mask [E + 1] int32: active experts, count last)."""
         assert input.num_dims == 2 and bias.num_dims == 1 and len(output) == 3
         w, idx, mask = output
@@ -587,12 +639,18 @@ class PersistentKernel:
         params = [num_groups, topk_group, bits]
         if local_experts is not None:
             params += [int(local_experts[0]), int(local_experts[1])]
+        if keep_logits:
+            params = (params + [0, idx.dim(0)])[:5] + [1]
         self._layer(N.OP_MOE_TOPK_SIGMOID, [input, bias, w, idx, mask], grid_dim, params)
 
     def moe_w13_linear_layer(self, input: DTensor, weight: DTensor, moe_routing_indices: DTensor, moe_mask: DTensor,
-                             output: DTensor, grid_dim: tuple, block_dim: tuple, first_expert: int = 0):
+                             output: DTensor, grid_dim: tuple, block_dim: tuple, first_expert: int = 0,
+                             activation: str = None):
+        """`activation` (hybrid graphs): a gated form over rows from `interleave_gated`, output [B, topk, >= I]."""
         assert input.num_dims == 2 and weight.num_dims == 3 and output.num_dims == 3
-        self._layer(N.OP_MOE_W13_LINEAR, [input, weight, moe_routing_indices, moe_mask, output], grid_dim, [int(first_expert)])
+        act = self.LINEAR_ACTIVATIONS[activation]
+        self._layer(N.OP_MOE_W13_LINEAR, [input, weight, moe_routing_indices, moe_mask, output], grid_dim,
+                    [int(first_expert), act] if act else [int(first_expert)])
 
     def moe_w2_linear_layer(self, input: DTensor, weight: DTensor, moe_routing_indices: DTensor, moe_mask: DTensor,
                             output: DTensor, grid_dim: tuple, block_dim: tuple, first_expert: int = 0):

@@ -125,3 +125,71 @@ def mlstm_output(o: Tensor, norm: Tensor, gate: Tensor, eps: float) -> Tensor:
 
 def squared_relu(x: Tensor) -> Tensor:
     return torch.relu(x) ** 2
+
+
+def layer_norm(x: Tensor, w: Tensor, b: Tensor, eps: float) -> Tensor:
+    d = x - x.mean(-1, keepdim=True)
+    return d / torch.sqrt((d * d).mean(-1, keepdim=True) + eps) * w + b
+
+
+def attention_sinks(q: Tensor, k: Tensor, v: Tensor, scale: float, sinks: Tensor) -> Tensor:
+    """Causal attention as above, one key/value head per query head; exp(sinks[h]) joins head h's denominator."""
+    T, H = q.shape[:2]
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for h in range(H):
+        for t in range(T):
+            s = (k[:t + 1, h] @ q[t, h]) * scale
+            top = torch.maximum(s.max(), sinks[h])
+            e = torch.exp(s - top)
+            out[t, h] = (e / (e.sum() + torch.exp(sinks[h] - top))) @ v[:t + 1, h]
+    return out
+
+
+def latent_attention(h: Tensor, w_q: Tensor, w_dkv: Tensor, latent_norm: Tensor, w_uk: Tensor, w_uv: Tensor, sinks: Tensor, *,
+                     heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, base: float, scale: float,
+                     eps: float) -> Tensor:
+    """Keys and values expanded from the latents, per head; h [tokens, width] -> [tokens, heads * vdim]."""
+    T = h.shape[0]
+    pos = torch.arange(T)
+    q = (h @ w_q.T).view(T, heads, dim + rot_dim)
+    q_rot = rotate_half_split(q[..., dim:], pos, base, rot_dim)
+    down = h @ w_dkv.T
+    c = rms_unit(down[:, :kv_rank], eps) * latent_norm
+    k_rot = rotate_half_split(down[:, None, kv_rank:], pos, base, rot_dim).expand(T, heads, rot_dim)
+    k = torch.cat([(c @ w_uk.T).view(T, heads, dim), k_rot], -1)
+    v = (c @ w_uv.T).view(T, heads, vdim)
+    return attention_sinks(torch.cat([q[..., :dim], q_rot], -1), k, v, scale, sinks).reshape(T, heads * vdim)
+
+
+def gla(q: Tensor, k: Tensor, v: Tensor, z: Tensor, tau: float) -> Tensor:
+    """Gated linear attention: q (already scaled), k, gate pre-activations z [tokens, H, d], v [tokens, H, dv]."""
+    T, H, d = q.shape
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for h in range(H):
+        S = torch.zeros(d, v.shape[2], dtype=q.dtype)
+        for t in range(T):
+            S = (torch.sigmoid(z[t, h]) ** (1.0 / tau))[:, None] * S + torch.outer(k[t, h], v[t, h])
+            out[t, h] = q[t, h] @ S
+    return out
+
+
+def silu(z: Tensor) -> Tensor:
+    return z * torch.sigmoid(z)
+
+
+def gated_ff(h: Tensor, gate: Tensor, up: Tensor, down: Tensor, act) -> Tensor:
+    return (act(h @ gate.T) * (h @ up.T)) @ down.T
+
+
+def grouped_choice(scores: Tensor, correction: Tensor, groups: int, keep: int, top: int) -> list:
+    """Experts of one token: `scores` [experts]; groups of neighbours compete with the sum of their two best choice scores."""
+    choice = scores + correction
+    size = choice.shape[0] // groups
+    totals = [float(sum(sorted(choice[g * size:(g + 1) * size].tolist(), reverse=True)[:2])) for g in range(groups)]
+    kept = sorted(range(groups), key=lambda g: -totals[g])[:keep]
+    allowed = [e for e in range(choice.shape[0]) if e // size in kept]
+    return sorted(allowed, key=lambda e: -float(choice[e]))[:top]
+
+
+def softcap(z: Tensor, cap: float) -> Tensor:
+    return cap * torch.tanh(z / cap)

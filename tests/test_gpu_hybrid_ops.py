@@ -203,8 +203,8 @@ def attention_graph(b, dtype, H, G, dim, rot, base, scale, cap, sink, unit, eps,
     width = (H + G) * dim + (G * vdim if separate_v else 0)
     proj, out = b.zeros(b.B, width), b.zeros(b.B, H * vdim + 2, dtype=dtype)
     dp = (dim + 7) // 8 * 8
-    from mirage_b200.builders.palarax import _rotary_tables
-    cos, sin = _rotary_tables(base, rot, b.pk.max_seq_length, "cuda")
+    from mirage_b200.builders.hybrid import rotary_tables
+    cos, sin = rotary_tables(base, rot, b.pk.max_seq_length, "cuda")
     kc, vc = b.zeros(b.pk.max_num_pages, b.page, G, dp, dtype=dtype), b.zeros(b.pk.max_num_pages, b.page, G, dp, dtype=dtype)
     kct, vct = b.pk.attach_input(kc, name="kc"), b.pk.attach_input(vc, name="vc")
     q = b.pk.attach_input(b.zeros(b.B, H * dp, dtype=dtype), name="q")
