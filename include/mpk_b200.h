@@ -116,7 +116,7 @@ typedef enum {
                                    tensors: proj, q, k_cache, v_cache, cos, sin
                                    params: [hq, hkv, dim, vdim, q_col, k_col, v_col, rotated dims, unit norm, eps] */
   MPK_OP_EXT_ATTENTION = 34,    /* tensors: q, k_cache, v_cache (= k_cache: the leading vdim columns of a key are its value), out, sinks (optional)
-                                   params: [hq, hkv, vdim, out_col, scale, soft cap (0: none), sink, out_scale]
+                                   params: [hq, hkv, vdim, out_col, scale, soft cap (0: none), sink, out_scale, optional 1: an MPK_OP_ATTN_MERGE layer follows]
                                    sink: exp(sinks[head]) joins the softmax denominator (bf16 [hq]; without the tensor: 1) */
   MPK_OP_SHORT_CONV = 35,       /* causal per-channel convolution   tensors: in, in_bias, taps, bias, state, out (biases optional)
                                    params: [in_col, activation: 0 none, 1 silu] */
@@ -131,7 +131,9 @@ typedef enum {
                                    params: [heads, latent size, rotated dims, q_col, kv_col, eps] */
   MPK_OP_GROUPED_LINEAR = 40    /* one linear per group of columns   in: x [tokens, groups * x stride], W [groups, N, K]  out: y
                                    params: [x stride, y column, y stride]: group g reads x[:, g * x stride + (0 .. K)] and writes
-                                   y[:, y column + g * y stride + (0 .. N)] */
+                                   y[:, y column + g * y stride + (0 .. N)] */,
+  MPK_OP_ATTN_MERGE = 41        /* directly behind an MPK_OP_EXT_ATTENTION layer with its ninth parameter set: the same tensors and parameters;
+                                   merges the key chunks on all workers (for wide values) */
 } mpk_op;
 
 /* Activations of linear layers in hybrid graphs.  The gated ones take weight rows interleaved as two gate rows, two up rows, and

@@ -27,7 +27,8 @@ TARGETS = {
     "core": ("libmpk_b200.so", ["mpk_abi.cu", "task_graph.cpp", "shuffle_rows.cu", "noalloc_attention.cu"],
              HOST_HEADERS + ["device_utils.cuh"]),
     "decoder": ("libmpk_b200_decoder.so", ["decoder_kernels.cu"], KERNEL_HEADERS),
-    "hybrid": ("libmpk_b200_hybrid.so", ["hybrid_kernels.cu"], KERNEL_HEADERS),
+    "hybrid": ("libmpk_b200_hybrid.so", ["hybrid_kernels.cu", "hybrid_kernel_bf16.cu", "hybrid_kernel_bf16_wide.cu", "hybrid_kernel_f32.cu"],
+               KERNEL_HEADERS + ["hybrid_kernels.h"]),
 }
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 NVCC_FLAGS = [*ARCH, "-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr"]

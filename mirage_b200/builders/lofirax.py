@@ -179,7 +179,8 @@ class LofiraxBuilder(HybridBuilder):
         mpk.latent_append_layer(proj, self._att(p + "dkv.norm"), q, cache, cos, sin, heads=H, rank=rank, rot_dims=rot, q_col=0,
                                 kv_col=H * rot, eps=self.eps)
         mixed = self._buf("latent_out", H * rank_p, self.act)
-        mpk.ext_attention_layer(q, cache, cache, mixed, heads=H, kv_heads=1, vdim=rank_p, scale=m.scale, sinks=self._att(p + "sink"))
+        mpk.ext_attention_layer(q, cache, cache, mixed, heads=H, kv_heads=1, vdim=rank_p, scale=m.scale, sinks=self._att(p + "sink"),
+                                separate_merge=True)
         values = self._buf("mixed", self._kpad(H * m.vdim), self.act)
         uv = self._attach(p + "uv.heads", lambda: self._pad_k(sd[p + "uv"].view(H, m.vdim, rank)))
         mpk.grouped_linear_layer(mixed, uv, values, in_stride=rank_p, out_stride=m.vdim)

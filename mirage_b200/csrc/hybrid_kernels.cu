@@ -1,12 +1,11 @@
-// Megakernel instantiations of hybrid graphs (hybrid_tasks.cuh) and their launch entry points: bf16 with the narrow
-// linear body (up to 8 batched tokens), bf16 with the tcgen05 body (more), and 32-bit throughout.  Built as
-// libmpk_b200_hybrid.so, loaded by the C ABI library when such a graph is compiled.
-#include "megakernel.cuh"
+// Launch entry points of hybrid graphs (hybrid_tasks.cuh).  Their megakernel instantiations are in one source each, which nvcc
+// compiles side by side: bf16 with the narrow linear body (up to 8 batched tokens), bf16 with the tcgen05 body (more), and 32-bit
+// throughout.  Built as libmpk_b200_hybrid.so, loaded by the C ABI library when such a graph is compiled.
+#include "hybrid_kernels.h"
 
-typedef void (*HybridKernel)(const mpk::KernelParams);
-static HybridKernel pick(int hybrid, int general) {
-  if (hybrid == mpk::HYB_F32) return mpk::mpk_megakernel<false, false, mpk::HYB_F32>;
-  return general ? mpk::mpk_megakernel<true, false, mpk::HYB_BF16> : mpk::mpk_megakernel<false, false, mpk::HYB_BF16>;
+static mpk::MegaKernel pick(int hybrid, int general) {
+  if (hybrid == mpk::HYB_F32) return mpk::hybrid_kernel_f32();
+  return general ? mpk::hybrid_kernel_bf16_wide() : mpk::hybrid_kernel_bf16();
 }
 
 extern "C" int mpk_family_prepare(int smem_bytes, int) {
@@ -15,8 +14,8 @@ extern "C" int mpk_family_prepare(int smem_bytes, int) {
   if (e == cudaSuccess) e = cudaDeviceGetAttribute(&limit, cudaDevAttrMaxSharedMemoryPerBlockOptin, dev);
   if (e != cudaSuccess) return (int)e;
   if (smem_bytes > limit) return (int)cudaErrorInvalidValue;
-  const HybridKernel all[3] = {pick(mpk::HYB_BF16, 0), pick(mpk::HYB_BF16, 1), pick(mpk::HYB_F32, 0)};
-  for (HybridKernel k : all) {
+  const mpk::MegaKernel all[3] = {pick(mpk::HYB_BF16, 0), pick(mpk::HYB_BF16, 1), pick(mpk::HYB_F32, 0)};
+  for (mpk::MegaKernel k : all) {
     e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, limit);
     if (e != cudaSuccess) return (int)e;
   }

@@ -382,7 +382,7 @@ __device__ __forceinline__ void column_f32(uint64_t w, size_t ldw, const float *
     }
   }
 }
-__device__ __noinline__ void run_linear_f32(const Ctx c, const TaskDesc &d) {
+static __device__ __noinline__ void run_linear_f32(const Ctx c, const TaskDesc &d) {
   const int B = active_tokens(c.P);
   const int n0 = d.a[0], n1 = d.a[1], K = d.a[2], TT = d.a[7];
   const int tid = threadIdx.x, warp = tid >> 5;
@@ -400,7 +400,7 @@ __device__ __noinline__ void run_linear_f32(const Ctx c, const TaskDesc &d) {
   }
 }
 // Expert projections: the active experts one after the other, the tokens routed to each gathered in shared memory.
-__device__ __noinline__ void run_moe_gemm_f32(const Ctx c, const TaskDesc &d) {
+static __device__ __noinline__ void run_moe_gemm_f32(const Ctx c, const TaskDesc &d) {
   const int B = min(active_tokens(c.P), kMaxLinearTokens);
   const int n0 = d.a[0], n1 = d.a[1], K = d.a[2], TT = d.a[7], slots = d.a[9], ldr = d.a[10], E = d.a[11];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -550,7 +550,7 @@ __device__ __noinline__ void run_latent_append(const Ctx c, const TaskDesc &d) {
 // ---------------------------------------------------------------------------
 // TASK_EXT_ATTENTION: (request, kv head, chunk of the keys).  The M rows of a task are the (token, query head of the
 // group) pairs, row r = token r / G, head r % G.  Chunks are merged by the last task of the (request, kv head) to
-// arrive.  Scores live in base 2 (bf16) or base e (float32): exp_dom undoes the same base everywhere.
+// arrive, or by a layer of TASK_ATTN_MERGE.  Scores live in base 2 (bf16) or base e (float32): exp_dom undoes the same base everywhere.
 // ---------------------------------------------------------------------------
 template <int HYB>
 __device__ __forceinline__ float exp_dom(float x) { return HYB == HYB_F32 ? expf(x) : exp2f(x); }
@@ -571,10 +571,30 @@ __device__ __forceinline__ float sink_logit(const TaskDesc &d, int h) {
   return d.p[4] ? bf16_at(d.p[4], h) * (HYB == HYB_F32 ? 1.0f : 1.4426950408889634f) : 0.f;
 }
 struct AttnOut {   // where a task's rows go
-  int hq, G, head, q0, NC, chunk, n_act, vdim, ldo, ocol, srec;
+  int hq, G, head, q0, ks, chunk, n_act, vdim, ldo, ocol, srec, rec0;
   float oscale;
   bool sink;
 };
+// Partial record of a row (max, sum, then the unnormalised columns) of this task's chunk; the chunks of a row lie side by side.
+__device__ __forceinline__ float *attn_record(const KernelParams &P, const AttnOut &o, int r) {
+  return P.attn_scratch + ((size_t)o.rec0 + (size_t)r * o.ks + o.chunk) * o.srec;
+}
+// How the NC tasks of a (request, kv head) share its work: over the tiles of RT query rows first and over the keys with what is
+// left: a prompt portion has rows enough and needs no merge, a decoded token has one tile and all its tasks share the keys.
+struct AttnSplit {
+  int rows, tiles, parts, ks, per, n_act;   // rows, row tiles, row parts, key chunks at most, keys of a chunk, chunks with keys
+};
+__device__ __forceinline__ AttnSplit attn_split(const SeqView &sv, int G, int NC, int RT) {
+  AttnSplit a;
+  const int len = sv.pos0 + sv.nq;
+  a.rows = sv.nq * G;
+  a.tiles = (a.rows + RT - 1) / RT;
+  a.parts = min(NC, a.tiles);
+  a.ks = min(NC / a.parts, 32);
+  a.per = max(64, ((len + a.ks - 1) / a.ks + 63) & ~63);
+  a.n_act = (len + a.per - 1) / a.per;
+  return a;
+}
 // Row r with (max m, sum l); val(col) gives the unnormalised output column.  Called by one warp.
 template <int HYB, class F>
 __device__ __forceinline__ void attn_emit_row(const Ctx &c, const TaskDesc &d, const AttnOut &o, int r, float m, float l, F val) {
@@ -593,19 +613,19 @@ __device__ __forceinline__ void attn_emit_row(const Ctx &c, const TaskDesc &d, c
       if (j0 + lane < o.vdim) store_elt(out + j0 + lane, v * f);
     }
   } else {
-    float *rec = c.P.attn_scratch + (((size_t)tok * o.hq + hq_idx) * o.NC + o.chunk) * o.srec;
+    float *rec = attn_record(c.P, o, r);
     if (lane == 0) {
       __stcg(rec, m);
       __stcg(rec + 1, l);
     }
     for (int j0 = 0; j0 < o.vdim; j0 += 32) {
       const float v = val(j0 + lane);
-      if (j0 + lane < o.vdim) __stcg(rec + 2 + j0 + lane, v);
+      if (j0 + lane < o.vdim) __stcg(rec + kXaRecHead + j0 + lane, v);
     }
   }
 }
 
-// Merge of the chunks' records by the last arriver.  NC <= 32.
+// Merge of the chunks' records by the last arriver (at most 32 chunks).
 template <int HYB>
 __device__ __noinline__ void attn_merge(const Ctx c, const TaskDesc &d, const AttnOut &o, int part, int row0, int row1) {
   typedef typename HybElt<HYB>::T T;
@@ -627,16 +647,16 @@ __device__ __noinline__ void attn_merge(const Ctx c, const TaskDesc &d, const At
   for (int item = warp + row0 * cols; item < row1 * cols; item += 8) {
     const int r = item / cols, j = (item - r * cols) * 32 + lane;
     const int tok = o.q0 + r / o.G, hq_idx = o.head * o.G + r % o.G;
-    const float *rec = P.attn_scratch + ((size_t)tok * o.hq + hq_idx) * o.NC * o.srec;
+    const float *rec = P.attn_scratch + ((size_t)o.rec0 + (size_t)r * o.ks) * o.srec;
     const bool v = lane < o.n_act;
     const float m = v ? __ldcg(rec + (size_t)lane * o.srec) : -INFINITY;
     const float l = v ? __ldcg(rec + (size_t)lane * o.srec + 1) : 0.f;
     float x[16], x2[16];
 #pragma unroll
-    for (int u = 0; u < 16; ++u) x[u] = (u < o.n_act && j < o.vdim) ? __ldcg(rec + (size_t)u * o.srec + 2 + j) : 0.f;
+    for (int u = 0; u < 16; ++u) x[u] = (u < o.n_act && j < o.vdim) ? __ldcg(rec + (size_t)u * o.srec + kXaRecHead + j) : 0.f;
     if (o.n_act > 16) {
 #pragma unroll
-      for (int u = 0; u < 16; ++u) x2[u] = (16 + u < o.n_act && j < o.vdim) ? __ldcg(rec + (size_t)(16 + u) * o.srec + 2 + j) : 0.f;
+      for (int u = 0; u < 16; ++u) x2[u] = (16 + u < o.n_act && j < o.vdim) ? __ldcg(rec + (size_t)(16 + u) * o.srec + kXaRecHead + j) : 0.f;
     }
     float M = warp_max(m);
     const float sk = o.sink ? sink_logit<HYB>(d, hq_idx) : 0.f;
@@ -1178,8 +1198,247 @@ __device__ __noinline__ void ext_attention_mma(const Ctx c, const TaskDesc &d, c
   }
 }
 
+// Shared key / value rows (latent attention: one kv head, the leading vdim columns of a key are its value), bf16 on mma.sync.  A
+// tile of MT x 16 query rows meets KEYS keys at a time, and every key row is brought to shared memory once for both products:
+//   scores   the warps split the keys in groups of 16 and the row width KS ways; partial sums meet in shared memory
+//   softmax  a warp takes RT / 8 rows, online in base 2; weights go back as a bf16 value and a bf16 remainder, so that they
+//            keep 16 bits
+//   output   every warp owns eight-column tiles w, w + 8, ... of all rows
+template <int MT, int KEYS>
+__device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d, const SeqView sv, const AttnOut &ao, int k0, int k1,
+                                                  int row0, int nrow, int task) {
+  constexpr int RT = MT * 16, KW = KEYS / 16, KS = 8 / KW, SP = KEYS + 4, PP = KEYS * 2 + 16, NV = 8;
+  constexpr int RPW = RT * KEYS / 256;             // row sets a warp's lanes hold in the softmax (32 / KEYS rows at a time)
+  const KernelParams &P = c.P;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int G = ao.G, dimp = d.a[XA_DIMP], D = (dimp + 63) & ~63, page = d.a[XA_PAGE], nstg = d.a[XA_STAGES];
+  const uint32_t pitch = D * 2 + 16;
+  const int pieces = dimp >> 3;                    // 16-byte pieces of a row
+  uint8_t *qs = c.s.xtile;                         // [RT][pitch]
+  uint8_t *st = qs + RT * pitch;                   // [nstg][KEYS][pitch]
+  float *sp = reinterpret_cast<float *>(st + (size_t)nstg * KEYS * pitch);   // [KS][RT][SP]
+  uint8_t *ps = reinterpret_cast<uint8_t *>(sp + KS * RT * SP);              // [value, remainder][RT][PP]
+  float *corr_s = reinterpret_cast<float *>(ps + 2 * RT * PP);               // [RT] rescale factors; at the end m and l
+  int *cells = reinterpret_cast<int *>(corr_s + 2 * RT);                     // [kXaCells] cache row of every eighth key
+  const int kend = min(k1, sv.pos0 + (row0 + nrow - 1) / G + 1);
+  const int ntiles = kend > k0 ? (kend - k0 + KEYS - 1) / KEYS : 0;
+  const uint8_t *qg = reinterpret_cast<const uint8_t *>(d.p[0]), *kg = reinterpret_cast<const uint8_t *>(d.p[1]);
+  const int ncell = (page & 7) == 0 && k1 - k0 <= 8 * kXaCells ? (k1 - k0 + 7) >> 3 : 0;
+  auto cell_row = [&](int key) {
+    const int pg = key / page;
+    return __ldcg(&P.meta.paged_kv_indices[sv.kv0 + pg]) * page + (key - pg * page);
+  };
+  for (int i = tid; i < ncell; i += kConsumerThreads) cells[i] = cell_row(k0 + 8 * i);
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  for (int r = warp; r < RT; r += 8)
+    for (int p = lane; p < D >> 3; p += 32) {
+      uint4 v = zero;
+      if (r < nrow && p < pieces)
+        v = __ldcg(reinterpret_cast<const uint4 *>(qg + ((size_t)(sv.q0 + (row0 + r) / G) * d.a[XA_LDQ] + (size_t)((row0 + r) % G) * dimp) * 2) + p);
+      *reinterpret_cast<uint4 *>(qs + r * pitch + p * 16) = v;
+    }
+  if (pieces < D >> 3)   // columns no copy reaches
+    for (int r = warp; r < nstg * KEYS; r += 8)
+      for (int p = pieces + lane; p < D >> 3; p += 32) *reinterpret_cast<uint4 *>(st + (size_t)r * pitch + p * 16) = zero;
+  consumer_sync();
+  stamp(c, task, 0);
+  auto issue = [&](int it, int stg) {
+    if (it < ntiles) {
+#pragma unroll
+      for (int r = 0; r < KEYS / 8; ++r) {
+        const int key = k0 + it * KEYS + warp + 8 * r;
+        uint8_t *dst = st + (size_t)(stg * KEYS + warp + 8 * r) * pitch;
+        if (key < kend) {
+          const size_t cell = ncell > 0 ? (size_t)(cells[(key - k0) >> 3] + ((key - k0) & 7)) : (size_t)cell_row(key);
+          const uint8_t *src = kg + cell * dimp * 2;
+          for (int p = lane; p < pieces; p += 32)
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst + p * 16)), "l"(src + p * 16) : "memory");
+        } else {   // a masked key has weight 0, and 0 x NaN would be NaN
+          for (int p = lane; p < pieces; p += 32) *reinterpret_cast<uint4 *>(dst + p * 16) = zero;
+        }
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  for (int i = 0; i < nstg - 1; ++i) issue(i, i);
+  const float scale = __int_as_float(d.a[XA_SCALE]), cap = __int_as_float(d.a[XA_CAP]);
+  const float cap2 = cap > 0.f ? 2.0f * 1.4426950408889634f / cap : 0.f;
+  const int kw = warp % KW, ks = warp / KW, ksteps = D >> 4;
+  const uint32_t qa = smem_u32(qs) + (uint32_t)((lane & 15) * pitch + (lane >> 4) * 16);
+  const uint32_t pa = smem_u32(ps) + (uint32_t)((lane & 15) * PP + (lane >> 4) * 16);
+  // softmax: this lane's key of the tile and first row
+  const int skey = lane % KEYS, srow = warp * (RT / 8) + lane / KEYS;
+  float m_run[RPW], l_run[RPW];
+#pragma unroll
+  for (int i = 0; i < RPW; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
+  const int nv = (ao.vdim >> 3) > warp ? ((ao.vdim >> 3) - warp + 7) >> 3 : 0;   // this warp's column tiles
+  float o[MT][NV][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[m][i][e] = 0.f;
+  int stg = 0;
+#pragma unroll 1
+  for (int it = 0; it < ntiles; ++it) {
+    if (nstg >= 4) asm volatile("cp.async.wait_group 2;" ::: "memory");
+    else if (nstg == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
+    else asm volatile("cp.async.wait_group 0;" ::: "memory");
+    consumer_sync();   // the tile has landed for everyone, and everyone is done with the stage refilled next
+    if (it == 0) stamp(c, task, 1);
+    issue(it + nstg - 1, stg == 0 ? nstg - 1 : stg - 1);
+    const uint32_t kt = smem_u32(st + (size_t)stg * KEYS * pitch);
+    if (++stg == nstg) stg = 0;
+    {   // ---- scores
+      float s[MT][2][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[m][n][e] = 0.f;
+      const uint32_t ka = kt + (uint32_t)((kw * 16 + (lane & 7) + (lane >> 4) * 8) * pitch + ((lane >> 3) & 1) * 16);
+#pragma unroll 3
+      for (int kk = ks; kk < ksteps; kk += KS) {
+        uint32_t b[4];
+        ldmatrix_x4(b, ka + kk * 32u);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          uint32_t a[4];
+          ldmatrix_x4(a, qa + (uint32_t)(m * 16) * pitch + kk * 32u);
+          mma_bf16_16816(s[m][0], a, b[0], b[1]);
+          mma_bf16_16816(s[m][1], a, b[2], b[3]);
+        }
+      }
+      float *sr = sp + (size_t)(ks * RT + (lane >> 2)) * SP + kw * 16 + 2 * (lane & 3);
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          *reinterpret_cast<float2 *>(sr + m * 16 * SP + n * 8) = make_float2(s[m][n][0], s[m][n][1]);
+          *reinterpret_cast<float2 *>(sr + (m * 16 + 8) * SP + n * 8) = make_float2(s[m][n][2], s[m][n][3]);
+        }
+    }
+    consumer_sync();
+    {   // ---- softmax
+      const int key = k0 + it * KEYS + skey;
+#pragma unroll
+      for (int i = 0; i < RPW; ++i) {
+        const int r = srow + i * (32 / KEYS);
+        float v = 0.f;
+#pragma unroll
+        for (int p = 0; p < KS; ++p) v += sp[(size_t)(p * RT + r) * SP + skey];
+        v = attn_score<HYB_BF16>(v, scale, cap, cap2);
+        if (key >= kend || key > sv.pos0 + (row0 + r) / G) v = -INFINITY;
+        float mx = v;
+#pragma unroll
+        for (int sh = KEYS / 2; sh > 0; sh >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, sh));
+        const float mn = fmaxf(m_run[i], mx), ms = mn == -INFINITY ? 0.f : mn;
+        const float corr = exp2f(m_run[i] - ms), p = exp2f(v - ms);
+        m_run[i] = mn;
+        l_run[i] = l_run[i] * corr + p;
+        const __nv_bfloat16 hi = __float2bfloat16_rn(p);
+        *reinterpret_cast<__nv_bfloat16 *>(ps + r * PP + skey * 2) = hi;
+        *reinterpret_cast<__nv_bfloat16 *>(ps + (RT + r) * PP + skey * 2) = __float2bfloat16_rn(p - bf16_to_f(hi));
+        if (skey == 0) corr_s[r] = corr;
+      }
+    }
+    consumer_sync();
+    {   // ---- output
+      float cr[MT][2];
+      bool keep = true;
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          cr[m][h] = corr_s[m * 16 + h * 8 + (lane >> 2)];
+          keep = keep && cr[m][h] == 1.f;
+        }
+      if (!__all_sync(0xffffffffu, keep)) {
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int i = 0; i < NV; ++i) {
+            o[m][i][0] *= cr[m][0]; o[m][i][1] *= cr[m][0];
+            o[m][i][2] *= cr[m][1]; o[m][i][3] *= cr[m][1];
+          }
+      }
+      // 16 keys and two column tiles at a time (one past the last is read, not used)
+#pragma unroll
+      for (int k = 0; k < KW; ++k) {
+        uint32_t p[2][MT][4];
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+          for (int m = 0; m < MT; ++m) ldmatrix_x4(p[h][m], pa + (uint32_t)((h * RT + m * 16) * PP + k * 32));
+        const uint32_t va = kt + (uint32_t)(k * 16 + (lane & 15)) * pitch + warp * 16 + (lane >> 4) * 128u;
+#pragma unroll
+        for (int i = 0; i < NV; i += 2) {
+          if (i >= nv) break;
+          uint32_t b[4];
+          ldmatrix_x4_trans(b, va + i * 128u);
+#pragma unroll
+          for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+              mma_bf16_16816(o[m][i], p[h][m], b[0], b[1]);
+              if (i + 1 < nv) mma_bf16_16816(o[m][i + 1], p[h][m], b[2], b[3]);
+            }
+        }
+      }
+    }
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  consumer_sync();
+  stamp(c, task, 2);
+  // running maximum and sum of every row
+#pragma unroll
+  for (int i = 0; i < RPW; ++i) {
+    float l = l_run[i];
+#pragma unroll
+    for (int sh = KEYS / 2; sh > 0; sh >>= 1) l += __shfl_xor_sync(0xffffffffu, l, sh);
+    if (skey == 0) {
+      const int r = srow + i * (32 / KEYS);
+      corr_s[r] = m_run[i];
+      corr_s[RT + r] = l;
+    }
+  }
+  consumer_sync();
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int r = m * 16 + h * 8 + (lane >> 2), row = row0 + r;
+      if (r >= nrow) continue;
+      const float mx = corr_s[r], l = corr_s[RT + r];
+      const int col0 = warp * 8 + 2 * (lane & 3);
+      if (ao.n_act == 1) {
+        const int hq_idx = row % G;
+        const float sk = ao.sink ? sink_logit<HYB_BF16>(d, hq_idx) : 0.f;
+        const float M = ao.sink ? fmaxf(mx, sk) : mx;
+        const float w = mx == -INFINITY ? 0.f : exp2f(mx - M);
+        const float L = l * w + (ao.sink ? exp2f(sk - M) : 0.f);
+        const float f = L > 0.f ? w / L * ao.oscale : 0.f;
+        __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(d.p[3]) + (size_t)(sv.q0 + row / G) * ao.ldo + ao.ocol + (size_t)hq_idx * ao.vdim + col0;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+          if (i < nv) *reinterpret_cast<uint32_t *>(out + i * 64) = pack_bf16(o[m][i][2 * h] * f, o[m][i][2 * h + 1] * f);
+      } else {
+        float *rec = attn_record(P, ao, row);
+        if (warp == 0 && (lane & 3) == 0) {
+          __stcg(rec, mx);
+          __stcg(rec + 1, l);
+        }
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+          if (i < nv) __stcg(reinterpret_cast<float2 *>(rec + kXaRecHead + col0 + i * 64), make_float2(o[m][i][2 * h], o[m][i][2 * h + 1]));
+      }
+    }
+}
+
 // 32-bit: one warp per row, 32 keys at a time (a lane per key for the scores, a lane per output column for PV)
-__device__ __noinline__ void ext_attention_f32(const Ctx c, const TaskDesc &d, const SeqView sv, const AttnOut &ao, int k0, int k1,
+static __device__ __noinline__ void ext_attention_f32(const Ctx c, const TaskDesc &d, const SeqView sv, const AttnOut &ao, int k0, int k1,
                                                   int row0, int rows) {
   constexpr int NO = 16;   // output columns per lane: value sizes up to 512
   const KernelParams &P = c.P;
@@ -1247,30 +1506,40 @@ __device__ __forceinline__ void run_ext_attention(const Ctx &c, const TaskDesc &
   // shared by the block, in shared memory: in registers it would be live through the key loops (every thread writes the
   // same values, and the previous task is done with it)
   AttnOut &ao = *reinterpret_cast<AttnOut *>(c.s.red);
+  const int RT = d.a[XA_SHARED] ? d.a[XA_SHARED] : 16, NC = d.a[XA_NCHUNK];
   ao.hq = d.a[XA_HQ];
   ao.G = ao.hq / d.a[XA_HKV];
   ao.head = d.a[XA_HEAD];
   ao.q0 = sv.q0;
-  ao.NC = d.a[XA_NCHUNK];
   ao.vdim = d.a[XA_VDIM];
   ao.ldo = d.a[XA_LDO];
   ao.ocol = d.a[XA_OCOL];
   ao.srec = d.a[XA_SREC];
   ao.oscale = __int_as_float(d.a[XA_OSCALE]);
   ao.sink = d.a[XA_SINK] != 0;
-  // The NC tasks of a (request, kv head) are split over the 16-row query tiles first and over the keys with what is left:
-  // a prompt portion has rows enough and needs no merge, a decoded token has one tile and all its tasks share the keys.
-  const int len = sv.pos0 + sv.nq, rows = sv.nq * ao.G, tiles = (rows + 15) >> 4;
-  const int parts = min(ao.NC, tiles), ksplit = ao.NC / parts;
-  const int part = d.a[XA_CHUNK] % parts;
-  ao.chunk = d.a[XA_CHUNK] / parts;
-  const int per = max(64, ((len + ksplit - 1) / ksplit + 63) & ~63);   // keys of a chunk
-  ao.n_act = (len + per - 1) / per;
-  if (ao.chunk >= ao.n_act) return;   // (n_act <= ksplit: this also ends the tasks beyond parts * ksplit)
-  const int k0 = ao.chunk * per, k1 = min(len, k0 + per);
-  const int row0 = tiles * part / parts * 16, row1 = min(rows, tiles * (part + 1) / parts * 16);
+  const AttnSplit sp = attn_split(sv, ao.G, NC, RT);
+  const int part = d.a[XA_CHUNK] % sp.parts;
+  ao.chunk = d.a[XA_CHUNK] / sp.parts;
+  ao.ks = sp.ks;
+  ao.n_act = sp.n_act;
+  ao.rec0 = (d.a[XA_SLOT] * d.a[XA_HKV] + ao.head) * RT * NC;
+  if (ao.chunk >= ao.n_act) return;   // (n_act <= ks: this also ends the tasks beyond parts * ks)
+  const int k0 = ao.chunk * sp.per, k1 = min(sv.pos0 + sv.nq, k0 + sp.per);
+  const int row0 = sp.tiles * part / sp.parts * RT, row1 = min(sp.rows, sp.tiles * (part + 1) / sp.parts * RT);
   if (HYB == HYB_F32) {
     ext_attention_f32(c, d, sv, ao, k0, k1, row0, row1);
+  } else if (d.a[XA_SHARED]) {
+    for (int r = row0; r < row1; r += RT) {
+      const int n = min(RT, row1 - r);
+      if (r > row0) consumer_sync();
+      if (d.a[XA_KEYS] == 32) {
+        if (n <= 16) latent_attention_mma<1, 32>(c, d, sv, ao, k0, k1, r, n, task);
+        else latent_attention_mma<2, 32>(c, d, sv, ao, k0, k1, r, n, task);
+      } else {
+        if (n <= 16) latent_attention_mma<1, 16>(c, d, sv, ao, k0, k1, r, n, task);
+        else latent_attention_mma<2, 16>(c, d, sv, ao, k0, k1, r, n, task);
+      }
+    }
   } else {
     const int w = max(d.a[XA_DIMP], d.a[XA_VDIMP]);
     const bool one = row1 - row0 <= 16 && (d.a[XA_PAGE] & 7) == 0;
@@ -1289,7 +1558,47 @@ __device__ __forceinline__ void run_ext_attention(const Ctx &c, const TaskDesc &
     }
   }
   stamp(c, task, 3);
-  if (ao.n_act > 1) attn_merge<HYB>(c, d, ao, part, row0, row1);
+  if (ao.n_act > 1 && !d.a[XA_MERGE]) attn_merge<HYB>(c, d, ao, part, row0, row1);
+}
+
+// TASK_ATTN_MERGE: the chunks' records of an attention layer with wide values, spread over all workers.  A warp takes 128 columns
+// of a (token, query head).
+template <int HYB>
+__device__ __noinline__ void run_attn_merge(const Ctx c, const TaskDesc &d) {
+  typedef typename HybElt<HYB>::T T;
+  const KernelParams &P = c.P;
+  const int B = active_tokens(P), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int hq = d.a[XA_HQ], hkv = d.a[XA_HKV], G = hq / hkv, vdim = d.a[XA_VDIM], srec = d.a[XA_SREC], NC = d.a[XA_NCHUNK];
+  const int RT = d.a[XA_SHARED] ? d.a[XA_SHARED] : 16, cols = (vdim + 127) >> 7;
+  for (int item = d.a[XA_SLOT] * 8 + warp; item < B * hq * cols; item += d.a[XA_CHUNK] * 8) {
+    const int row = item / cols, j = (item - row * cols) * 128 + lane * 4, t = row / hq, h = row - t * hq;
+    const int k = request_of(P, t);
+    const SeqView sv = seq_view(P, k);
+    const AttnSplit a = attn_split(sv, G, NC, RT);
+    if (a.n_act == 1) continue;   // the attention task wrote the output
+    const int r = (t - sv.q0) * G + h % G;
+    const float *rec = P.attn_scratch + ((size_t)(k * hkv + h / G) * RT * NC + (size_t)r * a.ks) * srec;
+    const bool v = lane < a.n_act;
+    const float m = v ? __ldcg(rec + (size_t)lane * srec) : -INFINITY, l = v ? __ldcg(rec + (size_t)lane * srec + 1) : 0.f;
+    const float sk = d.a[XA_SINK] ? sink_logit<HYB>(d, h) : 0.f;
+    float M = warp_max(m);
+    if (d.a[XA_SINK]) M = fmaxf(M, sk);
+    const float w = m == -INFINITY ? 0.f : exp_dom<HYB>(m - M);
+    const float L = warp_sum(l * w) + (d.a[XA_SINK] ? exp_dom<HYB>(sk - M) : 0.f);
+    const float f = L > 0.f ? __int_as_float(d.a[XA_OSCALE]) / L : 0.f;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int u = 0; u < a.n_act; ++u) {
+      const float wu = __shfl_sync(0xffffffffu, w, u);
+      const float4 x = j < vdim ? __ldcg(reinterpret_cast<const float4 *>(rec + (size_t)u * srec + kXaRecHead + j)) : make_float4(0.f, 0.f, 0.f, 0.f);
+      acc.x = fmaf(wu, x.x, acc.x); acc.y = fmaf(wu, x.y, acc.y); acc.z = fmaf(wu, x.z, acc.z); acc.w = fmaf(wu, x.w, acc.w);
+    }
+    T *out = reinterpret_cast<T *>(d.p[3]) + (size_t)t * d.a[XA_LDO] + d.a[XA_OCOL] + (size_t)h * vdim + j;
+    const float o[4] = {acc.x * f, acc.y * f, acc.z * f, acc.w * f};
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      if (j + e < vdim) store_elt(out + e, o[e]);
+  }
 }
 
 // ---------------------------------------------------------------------------
@@ -1352,7 +1661,7 @@ __device__ __forceinline__ void short_conv_window(const Ctx &c, const TaskDesc &
   }
 }
 
-__device__ __noinline__ void run_short_conv(const Ctx c, const TaskDesc &d) {
+static __device__ __noinline__ void run_short_conv(const Ctx c, const TaskDesc &d) {
   const KernelParams &P = c.P;
   const int B = active_tokens(P);
   if (B <= 0) return;
@@ -2304,7 +2613,7 @@ __device__ __forceinline__ void run_argmax_reduce_f32(const Ctx &c, const TaskDe
   }
 }
 
-__device__ __noinline__ void run_moe_routing_hybrid(const Ctx c, const TaskDesc &d) { run_moe_routing(c, d); }
+static __device__ __noinline__ void run_moe_routing_hybrid(const Ctx c, const TaskDesc &d) { run_moe_routing(c, d); }
 
 template <int HYB>
 __device__ __forceinline__ void run_hybrid_task(const Ctx &c, const TaskDesc &d, int task) {
@@ -2322,6 +2631,7 @@ __device__ __forceinline__ void run_hybrid_task(const Ctx &c, const TaskDesc &d,
     case TASK_MOE_GEMM_F32: if (HYB == HYB_F32) run_moe_gemm_f32(c, d); break;
     case TASK_LATENT_APPEND: run_latent_append<HYB>(c, d); break;
     case TASK_GLA: run_gla<HYB>(c, d, task); break;
+    case TASK_ATTN_MERGE: run_attn_merge<HYB>(c, d); break;
     case TASK_QKV_APPEND: run_qkv_append<HYB>(c, d); break;
     case TASK_EXT_ATTENTION: run_ext_attention<HYB>(c, d, task); break;
     case TASK_SHORT_CONV: run_short_conv(c, d); break;

@@ -1,5 +1,5 @@
 // The decode megakernel: one launch executes one iteration of the task graph.  Included by the files that
-// instantiate it (decoder_kernels.cu, hybrid_kernels.cu).
+// instantiate it (decoder_kernels.cu, hybrid_kernel_*.cu).
 //
 // Replaces the reference's persistent runtime (worker/scheduler loops and queues,
 // include/mirage/persistent_kernel/persistent_kernel.cuh:513-1082) and the task bodies
@@ -81,7 +81,7 @@ struct Ctx {
 // ---------------------------------------------------------------------------
 // bounded waits
 // ---------------------------------------------------------------------------
-__device__ __noinline__ void report_timeout(DeviceStatus *st, int worker, int where, int task) {
+static __device__ __noinline__ void report_timeout(DeviceStatus *st, int worker, int where, int task) {
   if (atomicCAS(&st->error, 0, -4) == 0) {
     st->where = where;
     st->worker = worker;
@@ -395,7 +395,7 @@ __device__ __forceinline__ float gather_row(const Ctx &c, const TaskDesc &d, con
 
 // PRO_RESNORM (hybrid graphs of a few tokens): the stream's residual sum and both norms in the consumer's prologue.  Every
 // task of the layer computes the same rows and writes the same values to x_out, which is another buffer than x.
-__device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d, int B) {
+static __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d, int B) {
   constexpr int NV = 4;   // rows of at most 4096 columns, in registers
   const int tid = threadIdx.x, W = d.a[L_GROUPS], K = d.a[L_K], warp = tid >> 5;
   const bool layer_norm = (d.a[L_G_SLOT] & 4) != 0;
@@ -1145,7 +1145,7 @@ __device__ void run_linear_tc(const Ctx &c, const TaskDesc &d, LinearState &ls, 
 // belongs to one warp, which copies its scale words into its own eight tensor-memory columns and then issues the 16
 // MMAs in order behind the copy; super groups rotate over the issuing warps.
 // ---------------------------------------------------------------------------
-__device__ void run_linear_fp8_tc(const Ctx &c, const TaskDesc &d, LinearState &ls, int task, bool ok) {
+static __device__ void run_linear_fp8_tc(const Ctx &c, const TaskDesc &d, LinearState &ls, int task, bool ok) {
   const KernelParams &P = c.P;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int B = ok ? min(active_tokens(P), kMaxLinearTokens) : 0;
@@ -1363,7 +1363,7 @@ __device__ __forceinline__ uint32_t align16u(uint32_t v) { return (v + 15u) & ~1
 
 // Stage, for k range [k0, k0 + KT): the activation rows and their scale exponents (unless the previous task
 // left them in place), and the scale exponents of this task's weight rows.
-__device__ void stage_fp8(const Ctx &c, const TaskDesc &d, int B, int k0, int KT, bool with_x) {
+static __device__ void stage_fp8(const Ctx &c, const TaskDesc &d, int B, int k0, int KT, bool with_x) {
   const int tid = threadIdx.x;
   const uint32_t xstride = (uint32_t)KT + kRowPadBytes;
   const int NG = KT / 128, g0 = k0 / 128;
@@ -1506,7 +1506,7 @@ __device__ __forceinline__ void run_linear_fp8(const Ctx &c, const TaskDesc &d, 
 // Follows per_token_group_quantize_fp8 (include/mirage/persistent_kernel/tasks/blackwell/
 // per_token_group_quantize_fp8.cuh:33-160): amax clamped at 1e-10, scale = amax / 448, for UE8M0 rounded up
 // to a power of two (computed on the exponent bits, which is exact) and packed four to a uint32 word.
-__device__ void run_quantize_fp8(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_quantize_fp8(const Ctx &c, const TaskDesc &d) {
   const KernelParams &P = c.P;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int K = d.a[2], ldx = d.a[3], ldq = d.a[4], per_tok = d.a[6], s0 = d.a[7], s1 = d.a[8], pk = d.a[9];
@@ -1561,7 +1561,7 @@ __device__ void run_quantize_fp8(const Ctx &c, const TaskDesc &d) {
 // group), top-k experts by repeated argmax (ties: lowest expert), weights from the unbiased scores.  The list of
 // active experts is written in ascending order (the reference's order depends on atomics).  The logits are
 // zeroed after they are read, as the reference does for its accumulating gate projection.
-__device__ void run_moe_routing(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_moe_routing(const Ctx &c, const TaskDesc &d) {
   const KernelParams &P = c.P;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int E = d.a[0], topk = d.a[1], groups = d.a[2], keep = d.a[3];
@@ -1792,7 +1792,7 @@ __device__ void run_moe_gemm(const Ctx &c, const TaskDesc &d, LinearState &ls, i
                    "l"(reinterpret_cast<const uint4 *>(xg + (xrow * d.a[L_LDX] + kt) * esz) + v)
                    : "memory");
     }
-    if (fp8) {
+    if constexpr (!HYBRID) if (fp8) {
       const float *xs = reinterpret_cast<const float *>(d.p[7]);
       const float *ws = reinterpret_cast<const float *>(d.p[6]);
       const int g0 = kt / 128;
@@ -1990,12 +1990,12 @@ __device__ void run_moe_gemm(const Ctx &c, const TaskDesc &d, LinearState &ls, i
 // flattened [token x slot] rows, as register_moe_silu_mul_task sets it up)
 // Hybrid graphs (bf16 only): a function of its own, state of the stage ring by value, so that the linear loop's registers stay as
 // they are.
-__device__ __noinline__ LinearState run_moe_gemm_hybrid(const Ctx c, const TaskDesc &d, LinearState ls, int task, bool ok) {
+static __device__ __noinline__ LinearState run_moe_gemm_hybrid(const Ctx c, const TaskDesc &d, LinearState ls, int task, bool ok) {
   run_moe_gemm<true>(c, d, ls, task, ok);
   return ls;
 }
 
-__device__ void run_moe_silu_mul(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_moe_silu_mul(const Ctx &c, const TaskDesc &d) {
   const int I = d.a[2], ldi = d.a[3], ldo = d.a[4];
   const int r1 = min(d.a[1], active_tokens(c.P) * d.a[5]);
   const __nv_bfloat16 *in = reinterpret_cast<const __nv_bfloat16 *>(d.p[0]);
@@ -2010,7 +2010,7 @@ __device__ void run_moe_silu_mul(const Ctx &c, const TaskDesc &d) {
 }
 
 // TASK_MOE_MUL_SUM_ADD: out[b, h] = residual[b, h] + sum_k in[b, k, h] * w[b, k]  (mul_sum_add_sm100.cuh:19-49)
-__device__ void run_moe_mul_sum_add(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_moe_mul_sum_add(const Ctx &c, const TaskDesc &d) {
   const int c0 = d.a[0], c1 = d.a[1], H = d.a[2], topk = d.a[3], ldo = d.a[4], ldres = d.a[5], ldw = d.a[6];
   const int B = min(d.a[7], active_tokens(c.P));
   const __nv_bfloat16 *in = reinterpret_cast<const __nv_bfloat16 *>(d.p[0]);
@@ -2040,7 +2040,7 @@ constexpr int kMlaPRow = kMlaSub * 2 + 16;    // row stride of the probability t
 // TASK_MLA_APPEND: the request's new [c_latent | k_pe] rows go to their positions in the paged cache
 // (step 1 of mla_kv_cache_gather_sm100.cuh:36-128; the decode tasks read the paged cache in place, so the
 // reference's second step -- copying the whole sequence to a contiguous buffer -- has no counterpart).
-__device__ void run_mla_append(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_mla_append(const Ctx &c, const TaskDesc &d) {
   const KernelParams &P = c.P;
   const int slot = d.a[0], ldc = d.a[1], ldp = d.a[2], page = d.a[3], dk = d.a[4], dv = d.a[5];
   const int q0 = __ldcg(&P.meta.qo_indptr[slot]);
@@ -2077,7 +2077,7 @@ __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t sme
 // go through shared memory, the probabilities are written as a bf16 tile, and warp w accumulates output columns
 // [64w, 64w + 64) of P.V with V read transposed from the same kv tile.  Output: O normalised by the split's own
 // sum (bf16) and the split's log-sum-exp (fp32); TASK_MLA_REDUCE merges the splits.
-__device__ void run_mla_decode(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_mla_decode(const Ctx &c, const TaskDesc &d) {
   const KernelParams &P = c.P;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q = lane & 3;
   const int t = d.a[0], split = d.a[1], head0 = d.a[2], H = d.a[3], S = d.a[4], page = d.a[5], ldq = d.a[6];
@@ -2250,7 +2250,7 @@ __device__ void run_mla_decode(const Ctx &c, const TaskDesc &d) {
 
 // TASK_MLA_REDUCE: out[token, head] = sum_s w_s O_s with w_s = exp(lse_s - max) / sum: one warp per (token, head) row
 // (mla_reduce_sm100.cuh:28-76 / mla_mtp_reduce).
-__device__ void run_mla_reduce(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_mla_reduce(const Ctx &c, const TaskDesc &d) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int H = d.a[2], S = d.a[3], ldo = d.a[4];
   const int r1 = min(d.a[1], active_tokens(c.P) * H);
@@ -3017,7 +3017,7 @@ __device__ __forceinline__ void attn_step_mma(const uint8_t *ktile, const uint8_
   }
 }
 
-__device__ void attention_stream_body(const Ctx &c, const TaskDesc &d, AttnStream &a, int task) {
+static __device__ void attention_stream_body(const Ctx &c, const TaskDesc &d, AttnStream &a, int task) {
   const KernelParams &P = c.P;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const ReqView rv = a.rv;
@@ -3217,7 +3217,7 @@ __device__ __forceinline__ void run_attention_stream(const Ctx &c, const TaskDes
 // ---------------------------------------------------------------------------
 // small tasks
 // ---------------------------------------------------------------------------
-__device__ void run_embed(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_embed(const Ctx &c, const TaskDesc &d) {
   const int B = active_tokens(c.P);
   const int t0 = d.a[E_T0], t1 = min(d.a[E_T1], B), width = d.a[E_WIDTH];
   const int64_t *ids = reinterpret_cast<const int64_t *>(d.p[0]);
@@ -3235,7 +3235,7 @@ __device__ void run_embed(const Ctx &c, const TaskDesc &d) {
   }
 }
 
-__device__ void run_rmsnorm(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_rmsnorm(const Ctx &c, const TaskDesc &d) {
   const int B = active_tokens(c.P);
   const int t0 = d.a[E_T0], t1 = min(d.a[E_T1], B), width = d.a[E_WIDTH];
   const __nv_bfloat16 *in = reinterpret_cast<const __nv_bfloat16 *>(d.p[0]);
@@ -3275,7 +3275,7 @@ __device__ void run_rmsnorm(const Ctx &c, const TaskDesc &d) {
 }
 
 // silu_mul over columns [a[7], a[8]) of the activation (width a[2] = I), group-interleaved input
-__device__ void run_silu_mul(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_silu_mul(const Ctx &c, const TaskDesc &d) {
   const int B = active_tokens(c.P);
   const int t0 = d.a[E_T0], t1 = min(d.a[E_T1], B), I = d.a[E_WIDTH];
   const int groups = d.a[E_AUX];
@@ -3315,7 +3315,7 @@ __device__ void run_silu_mul(const Ctx &c, const TaskDesc &d) {
     }
 }
 
-__device__ void run_elementwise_add(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_elementwise_add(const Ctx &c, const TaskDesc &d) {
   const int B = active_tokens(c.P);
   const int t0 = d.a[E_T0], t1 = min(d.a[E_T1], B), width = d.a[E_WIDTH];
   const __nv_bfloat16 *a = reinterpret_cast<const __nv_bfloat16 *>(d.p[0]);
@@ -3327,7 +3327,7 @@ __device__ void run_elementwise_add(const Ctx &c, const TaskDesc &d) {
                                                            bf16_to_f(__ldcg(&b[(size_t)t * d.a[E_LDI2] + j])));
 }
 
-__device__ void run_tensor_init(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_tensor_init(const Ctx &c, const TaskDesc &d) {
   // zero rows [t0,t1) of width a[2] BYTES
   uint8_t *out = reinterpret_cast<uint8_t *>(d.p[2]);
   const size_t row_bytes = (size_t)d.a[E_WIDTH];
@@ -3344,7 +3344,7 @@ __device__ __forceinline__ void argmax_merge(float &v, long long &i, float v2, l
   }
 }
 
-__device__ void block_argmax(const Ctx &c, float &v, long long &i) {
+static __device__ void block_argmax(const Ctx &c, float &v, long long &i) {
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {
@@ -3448,7 +3448,7 @@ __device__ void run_sampling_partial(const Ctx &c, const TaskDesc &d) {
   }
 }
 
-__device__ void run_sampling_reduce(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_sampling_reduce(const Ctx &c, const TaskDesc &d) {
   const int B = active_tokens(c.P);
   const __nv_bfloat16 *pv = reinterpret_cast<const __nv_bfloat16 *>(d.p[0]);
   const long long *pi = reinterpret_cast<const long long *>(d.p[1]);
@@ -3470,7 +3470,7 @@ __device__ void run_sampling_reduce(const Ctx &c, const TaskDesc &d) {
   }
 }
 
-__device__ void run_argmax_partial(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_argmax_partial(const Ctx &c, const TaskDesc &d) {
   const int B = active_tokens(c.P);
   const __nv_bfloat16 *logits = reinterpret_cast<const __nv_bfloat16 *>(d.p[0]);
   __nv_bfloat16 *pv = reinterpret_cast<__nv_bfloat16 *>(d.p[1]);
@@ -3489,7 +3489,7 @@ __device__ void run_argmax_partial(const Ctx &c, const TaskDesc &d) {
   }
 }
 
-__device__ void run_argmax_reduce(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_argmax_reduce(const Ctx &c, const TaskDesc &d) {
   const int B = active_tokens(c.P);
   const __nv_bfloat16 *pv = reinterpret_cast<const __nv_bfloat16 *>(d.p[0]);
   const long long *pi = reinterpret_cast<const long long *>(d.p[1]);
@@ -3577,7 +3577,7 @@ __device__ __forceinline__ void run_argmax_exchange(const Ctx &c, const TaskDesc
 }
 
 // Sum the per-rank fp32 inbox slots in rank order (+ residual) -> bf16.
-__device__ void run_allreduce(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_allreduce(const Ctx &c, const TaskDesc &d) {
   const KernelParams &P = c.P;
   const int B = active_tokens(P);
   const int c0 = d.a[0], c1 = d.a[1], world = d.a[2], slot = d.a[3], ldo = d.a[4], ldr = d.a[5], N = d.a[6];
@@ -3597,7 +3597,7 @@ __device__ void run_allreduce(const Ctx &c, const TaskDesc &d) {
 
 // Push stage of an unfused allreduce: columns [c0, c1) of a local bf16 tensor go, as fp32, into this rank's slot of
 // every rank's inbox; the task's event is incremented on every rank once the stores are ordered (TF_REMOTE_TRIGGER).
-__device__ void run_ar_push(const Ctx &c, const TaskDesc &d) {
+static __device__ void run_ar_push(const Ctx &c, const TaskDesc &d) {
   const KernelParams &P = c.P;
   const int B = active_tokens(P);
   const int c0 = d.a[0], c1 = d.a[1], ldx = d.a[2], slot = d.a[3], N = d.a[6];
@@ -3623,7 +3623,7 @@ __device__ void run_ar_push(const Ctx &c, const TaskDesc &d) {
 //     while the loop runs (REQ_* in runtime_types.h), admitted in row order; a request advances no further than the
 //     tokens the host has supplied (REQ_HOLD) or decodes on its own (REQ_RUN), and never further than the free pages.
 // ---------------------------------------------------------------------------
-__device__ __noinline__ void run_batch(const Ctx c) {
+static __device__ __noinline__ void run_batch(const Ctx c) {
   if (c.tmem_base & 0x80000000u) {   // called for TASK_ARGMAX_EXCHANGE (see task_other)
     run_argmax_exchange(c, c.s.desc[c.tmem_base & 1u]);
     return;

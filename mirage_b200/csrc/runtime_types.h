@@ -66,6 +66,7 @@ enum TaskType : uint32_t {
   TASK_GLA = 32,                // gated linear attention (matrix state, a decay per key channel)
   TASK_LATENT_APPEND = 33,      // latent attention: cache rows and rotated query parts
   TASK_MOE_GEMM_F32 = 34,       // expert projections in 32-bit arithmetic
+  TASK_ATTN_MERGE = 35,         // merge of an attention layer's key chunks
 };
 
 // Which family of megakernel instantiations runs a graph (template parameter HYB of the kernel).
@@ -227,7 +228,10 @@ enum { QA_T0 = 0, QA_T1, QA_LDP, QA_QOFF, QA_KOFF, QA_VOFF, QA_HQ, QA_HKV, QA_DI
        QA_EPS, QA_PAGE, QA_LDQ, QA_ROWS };
 // ---- TASK_EXT_ATTENTION: p[0] q [tokens, hq * dimp]  p[1] k cache  p[2] v cache  p[3] out;  a[XA_*] below
 enum { XA_SLOT = 0, XA_HEAD, XA_CHUNK, XA_NCHUNK, XA_HQ, XA_HKV, XA_DIMP, XA_VDIM, XA_VDIMP, XA_PAGE, XA_LDQ, XA_LDO, XA_OCOL,
-       XA_SCALE, XA_CAP, XA_SINK, XA_OSCALE, XA_TICKET, XA_SREC, XA_STAGES, XA_SHARED };   // p[4] sinks bf16 [hq] or null; XA_SHARED: values are key columns
+       XA_SCALE, XA_CAP, XA_SINK, XA_OSCALE, XA_TICKET, XA_SREC, XA_STAGES, XA_SHARED, XA_KEYS, XA_MERGE };
+//      p[4] sinks bf16 [hq] or null; XA_SHARED: values are key columns, rows of a query tile (0: separate values); XA_KEYS: keys of a tile of
+//      theirs; XA_MERGE: a layer of TASK_ATTN_MERGE follows (its tasks: the same fields, task a[XA_SLOT] of a[XA_CHUNK])
+constexpr int kXaRecHead = 4;   // floats in front of a record's columns
 constexpr int kXaCells = 320;   // cache rows of a chunk's key octets kept in shared memory
 // ---- TASK_SHORT_CONV: channels [a[0], a[1]); p[0] in f32  p[1] in bias bf16 or null  p[2] taps bf16 [channels, taps]
 //      p[3] bias bf16 or null  p[4] carried inputs f32 [slots, taps - 1, channels]  p[5] out f32

@@ -43,6 +43,7 @@ struct Builder {
   std::vector<std::vector<TaskDesc>> per_worker;
   std::vector<std::vector<int>> per_worker_exec;
   int rot = 0;
+  TaskDesc xattn_task;      // the last extended-attention task (its merge layer shares the fields)
   int hybrid_tickets = 0;   // arrival tickets handed to the tasks of hybrid graphs
   std::map<int, std::map<int, int>> slices;   // storage -> (first column -> id) of outputs that layers write by column range
 
@@ -174,6 +175,7 @@ struct Builder {
         add(outs, l.t[4]);
         break;
       case MPK_OP_QKV_APPEND: add(ins, l.t[0]); add(ins, l.t[4]); add(ins, l.t[5]); for (int i = 1; i < 4; ++i) add(outs, l.t[i]); break;
+      case MPK_OP_ATTN_MERGE: add(ins, l.t[3]); add(outs, l.t[3]); break;
       case MPK_OP_EXT_ATTENTION:
         for (int i = 0; i < 3; ++i) add(ins, l.t[i]);
         if (l.t.size() > 4) add(ins, l.t[4]);
@@ -219,7 +221,7 @@ struct Builder {
           {MPK_OP_SAMPLING_PARTIAL, 3}, {MPK_OP_SAMPLING_REDUCE, 3}, {MPK_OP_ARGMAX_EXCHANGE, 3},
           {MPK_OP_MOE_TOPK_SOFTMAX, 4}, {MPK_OP_RESIDUAL_NORM, 5}, {MPK_OP_QKV_APPEND, 6}, {MPK_OP_EXT_ATTENTION, 4},
           {MPK_OP_SHORT_CONV, 6}, {MPK_OP_RGLRU, 10}, {MPK_OP_MLSTM, 8}, {MPK_OP_GLA, 7}, {MPK_OP_LATENT_APPEND, 6},
-          {MPK_OP_GROUPED_LINEAR, 3}};
+          {MPK_OP_GROUPED_LINEAR, 3}, {MPK_OP_ATTN_MERGE, 4}};
       auto it = need.find(L[i].op);
       if (it == need.end()) return fail(MPK_ERR_UNSUPPORTED, "layer " + std::to_string(i) + ": unknown op");
       if ((int)L[i].t.size() < it->second)
@@ -1066,7 +1068,7 @@ struct Builder {
   }
 
   // ---- hybrid graphs: recurrent layers, extended attention, float32 residual stream --------------------------
-  static bool hybrid_op(int op) { return op >= MPK_OP_RESIDUAL_NORM && op <= MPK_OP_GROUPED_LINEAR; }
+  static bool hybrid_op(int op) { return op >= MPK_OP_RESIDUAL_NORM && op <= MPK_OP_ATTN_MERGE; }
   static bool expert_op(int op) { return op == MPK_OP_MOE_TOPK_SIGMOID || op == MPK_OP_MOE_W13_LINEAR || op == MPK_OP_MOE_W2_LINEAR; }
   static int activation_epilogue(int64_t act) {
     switch (act) {
@@ -1117,6 +1119,27 @@ struct Builder {
   }
   // key / value tiles in flight: graphs of many tokens reserve a large activation tile anyway
   int xattn_stages() const { return nb_max > 8 ? 3 : 2; }
+  // Tiles of attention over shared key / value rows: the largest that leave the weight ring its size (graphs of many tokens
+  // reserve a large activation tile anyway; of few tokens what a ring of 32 KB stages leaves over).
+  struct LatentPlan { int rt, keys, stages; int64_t bytes; };
+  LatentPlan latent_plan(const LayerInfo &l) const {
+    const int64_t pitch = round_up(T[l.t[1]].dim(3), 64) * 2 + 16;
+    const int64_t rows = (int64_t)cfg.max_num_batched_tokens * l.params[0];
+    const int64_t budget = kPartialBytes + (nb_max > 8 ? 64 * (1024 * 2 + kRowPadBytes) : 90 * 1024);
+    LatentPlan p{0, 0, 0, 0};
+    for (const auto &c : {std::pair<int, int>{32, 32}, {16, 32}, {32, 16}, {16, 16}}) {
+      p.rt = c.first;
+      p.keys = c.second;
+      if (p.rt > 16 && rows <= 16) continue;
+      if (nb_max <= 8 && p.keys > 16) continue;
+      const int64_t fixed = p.rt * pitch + (int64_t)(8 / (p.keys / 16)) * p.rt * (p.keys + 4) * 4 + 2 * p.rt * (p.keys * 2 + 16) + 8 * p.rt + kXaCells * 4;
+      p.stages = (int)std::min<int64_t>(4, (budget - fixed) / (p.keys * pitch));
+      if (p.stages < 2 && p.rt + p.keys == 32) p.stages = 2;   // the smallest tiles: whatever they need
+      p.bytes = fixed + p.stages * p.keys * pitch;
+      if (p.stages >= 2) return p;
+    }
+    return p;
+  }
   // shared memory of a token: gate sums and u, as float32 or as three bf16 parts
   static int64_t rglru_token_bytes(int bs, int C) { return 16 * C + 6 * (round_up(bs, 16) + 8); }
   void rglru_plan(const LayerInfo &l, int *C, int *TG) const {
@@ -1134,6 +1157,7 @@ struct Builder {
       case MPK_OP_RESIDUAL_NORM: return T[l.t[0]].dim(1) * 4 + 16;
       case MPK_OP_EXT_ATTENTION: {
         if (g->hybrid == HYB_F32) return 8 * T[l.t[1]].dim(3) * 4;
+        if (T[l.t[1]].storage == T[l.t[2]].storage) return latent_plan(l).bytes;
         const int D = xattn_width(l), pitch = D * 2 + 16, keys = D > 128 ? 32 : 64, wmax = D > 128 ? 4 : 8;
         const int G = (int)(l.params[0] / std::max<int64_t>(l.params[1], 1));
         const int64_t tile = (int64_t)std::min(wmax * 16, ext_attention_rows(cfg.max_num_batched_tokens * G)) * pitch +
@@ -1447,23 +1471,31 @@ struct Builder {
       return fail(MPK_ERR_INVALID, "ext_attention: shapes of q, caches and output disagree");
     if (q.dtype != act_dtype() || kc.dtype != act_dtype() || vc.dtype != act_dtype() || o.dtype != act_dtype())
       return fail(MPK_ERR_INVALID, "ext_attention: q, caches and output must have the graph's activation type");
-    if (g->hybrid == HYB_F32 ? kc.dim(3) > 1024 || vdim > 512 : std::max(kc.dim(3), vc.dim(3)) > 256)
-      return fail(MPK_ERR_UNSUPPORTED, "ext_attention: head sizes up to 256 (32-bit graphs: keys up to 1024, values up to 512)");
+    const bool shared = kc.storage == vc.storage, bf16 = g->hybrid == HYB_BF16;
+    if (shared && bf16 && (hkv != 1 || vdim % 8 || (ocol | o.ld()) % 2)) return fail(MPK_ERR_UNSUPPORTED, "ext_attention: shared keys and values have one kv head and a value size of whole 16-byte pieces");
+    if (bf16 && !shared ? std::max(kc.dim(3), vc.dim(3)) > 256 : kc.dim(3) > 1024 || vdim > 512)
+      return fail(MPK_ERR_UNSUPPORTED, "ext_attention: head sizes up to 256 (32-bit graphs and shared keys and values: keys up to 1024, values up to 512)");
     const int sinks = l.t.size() > 4 ? l.t[4] : -1;
     if (sinks >= 0 && (T[sinks].dtype != MPK_BF16 || T[sinks].dim(0) < hq || !l.params[6])) return fail(MPK_ERR_INVALID, "ext_attention: bf16 sinks [heads], sink = 1");
-    const bool shared = kc.storage == vc.storage;
+    const bool merge = l.params.size() > 8 && l.params[8];
     const int slots = cfg.max_num_batched_requests, max_seq = std::max(cfg.max_seq_length, 1);
     // chunks of a (request, kv head): enough to occupy the workers, at most ~2048 keys each, at least 64
     int NC = std::max(std::max(1, W / std::max(slots * hkv, 1)), (max_seq + 2047) / 2048);
     NC = std::min(std::min(NC, std::max(1, max_seq / 64)), 32);
-    const int srec = vdim + 2;
+    LatentPlan lp{16, 0, xattn_stages(), 0};
+    if (shared && bf16) {   // row tiles of a prompt portion times key chunks of a decoded token
+      lp = latent_plan(l);
+      const int64_t tiles = ((int64_t)cfg.max_num_batched_tokens * hq + lp.rt - 1) / lp.rt;
+      NC = (int)std::min<int64_t>(std::max(1, W / slots), tiles * std::max(1, (max_seq + 63) / 64));
+    }
+    const int srec = round_up(vdim, 4) + kXaRecHead;
     for (int s = 0; s < slots; ++s)
       for (int h = 0; h < hkv; ++h)
         for (int ch = 0; ch < NC; ++ch) {
           TaskDesc d = blank(TASK_EXT_ATTENTION, li);
           for (int i = 0; i < 4; ++i) d.p[i] = (uint64_t)T[l.t[i]].ptr;
           d.p[4] = sinks >= 0 ? (uint64_t)T[sinks].ptr : 0;
-          d.a[XA_SHARED] = shared ? 1 : 0;
+          d.a[XA_SHARED] = shared && bf16 ? lp.rt : 0; d.a[XA_KEYS] = lp.keys; d.a[XA_MERGE] = merge ? 1 : 0;
           d.a[XA_SLOT] = s; d.a[XA_HEAD] = h; d.a[XA_CHUNK] = ch; d.a[XA_NCHUNK] = NC; d.a[XA_HQ] = hq; d.a[XA_HKV] = hkv;
           d.a[XA_DIMP] = (int)kc.dim(3); d.a[XA_VDIM] = vdim; d.a[XA_VDIMP] = (int)vc.dim(3); d.a[XA_PAGE] = cfg.page_size;
           d.a[XA_LDQ] = (int)q.ld(); d.a[XA_LDO] = (int)o.ld(); d.a[XA_OCOL] = ocol;
@@ -1471,11 +1503,29 @@ struct Builder {
           d.a[XA_OSCALE] = bits_of(l.params[7]);
           d.a[XA_TICKET] = hybrid_tickets + (s * hkv + h) * NC;   // one per part of the query rows
           d.a[XA_SREC] = srec;
-          d.a[XA_STAGES] = xattn_stages();
+          d.a[XA_STAGES] = lp.stages;
           put(((s * hkv + h) * NC + ch + rot) % W, d, ex);
+          xattn_task = d;
         }
     hybrid_tickets += slots * hkv * NC;
-    g->attn_scratch_floats = std::max<int64_t>(g->attn_scratch_floats, (int64_t)cfg.max_num_batched_tokens * hq * NC * srec);
+    // a (request, kv head) has at most one query tile's rows for each of its tasks in the scratch
+    g->attn_scratch_floats = std::max<int64_t>(g->attn_scratch_floats, (int64_t)slots * hkv * NC * lp.rt * srec);
+    return MPK_OK;
+  }
+
+  int emit_attn_merge(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const int at = li - 1;
+    if (at < 0 || L[at].op != MPK_OP_EXT_ATTENTION || L[at].t != l.t || L[at].params != l.params || l.params.size() < 9 || !l.params[8])
+      return fail(MPK_ERR_INVALID, "attn_merge: follows an ext_attention layer of the same tensors and parameters");
+    const int cols = (int)((l.params[2] + 127) / 128), nt = (int)std::max<int64_t>(1, std::min<int64_t>(W, ((int64_t)nb_max * l.params[0] * cols + 7) / 8));
+    for (int i = 0; i < nt; ++i) {
+      TaskDesc d = xattn_task;
+      d.type = TASK_ATTN_MERGE;
+      d.layer = li;
+      d.a[XA_SLOT] = i; d.a[XA_CHUNK] = nt;
+      put((i + rot) % W, d, ex);
+    }
     return MPK_OK;
   }
 
@@ -1601,6 +1651,7 @@ struct Builder {
       case MPK_OP_GLA: return emit_gla(li, ex);
       case MPK_OP_LATENT_APPEND: return emit_latent_append(li, ex);
       case MPK_OP_GROUPED_LINEAR: return emit_grouped_linear(li, ex);
+      case MPK_OP_ATTN_MERGE: return emit_attn_merge(li, ex);
       case MPK_OP_LINEAR_FP8: case MPK_OP_LINEAR_FP8_RESIDUAL:
         return emit_linear_fp8(li, ex);
       case MPK_OP_QUANTIZE_FP8:
@@ -2188,7 +2239,8 @@ std::string dump_task_graph(const CompiledGraph &g, const std::vector<TensorInfo
                                 "argmax_partial", "argmax_reduce", "allreduce", "elementwise_add", "tensor_init",
                                 "quantize_fp8", "moe_routing", "moe_gemm", "moe_silu_mul", "moe_mul_sum_add",
                                 "mla_append", "mla_decode", "mla_reduce", "sampling_partial", "sampling_reduce", "argmax_exchange", "ar_push",
-                                "embed_f32", "residual_norm", "linear_f32", "qkv_append", "ext_attention", "short_conv", "rglru", "mlstm"};
+                                "embed_f32", "residual_norm", "linear_f32", "qkv_append", "ext_attention", "short_conv", "rglru", "mlstm",
+                                "gla", "latent_append", "moe_gemm_f32", "attn_merge"};
   std::ostringstream os;
   os << "{\"num_workers\": " << g.num_workers << ", \"num_tasks\": " << g.tasks.size()
      << ", \"num_events\": " << g.num_events << ", \"num_layers\": " << layers.size()
@@ -2197,7 +2249,7 @@ std::string dump_task_graph(const CompiledGraph &g, const std::vector<TensorInfo
      << ",\n \"events\": [\n";
   for (size_t e = 0; e < g.exec.size(); ++e) {
     const ExecLayer &x = g.exec[e];
-    os << "  {\"event\": " << e << ", \"type\": \"" << names[x.type < 32 ? x.type : 0] << "\", \"layer\": " << x.layer
+    os << "  {\"event\": " << e << ", \"type\": \"" << names[x.type < sizeof(names) / sizeof(names[0]) ? x.type : 0] << "\", \"layer\": " << x.layer
        << ", \"tasks\": " << x.num_tasks << ", \"deps\": [";
     for (size_t k = 0; k < x.deps.size(); ++k) os << (k ? ", " : "") << "[" << x.deps[k] << ", " << x.dep_need[k] << "]";
     os << "]";

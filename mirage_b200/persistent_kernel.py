@@ -556,14 +556,19 @@ class PersistentKernel:
 
     def ext_attention_layer(self, q: DTensor, k_cache: DTensor, v_cache: DTensor, output: DTensor, *, heads: int,
                             kv_heads: int, vdim: int, scale: float, softcap: float = 0.0, sink: bool = False,
-                            sinks: Optional[DTensor] = None, out_col: int = 0, out_scale: float = 1.0):
+                            sinks: Optional[DTensor] = None, out_col: int = 0, out_scale: float = 1.0,
+                            separate_merge: bool = False):
         """Causal paged attention over rows a qkv_append_layer or latent_append_layer wrote.  score = softcap *
         tanh(scale * q.k / softcap) (no cap at 0); `sink` adds one to the softmax denominator, `sinks` (bf16 [heads]) adds
         exp(sinks[head]); the result times `out_scale` goes to columns [out_col, out_col + heads * vdim) of `output`.
-        `v_cache` may be `k_cache`: the leading `vdim` columns of a key are then its value."""
-        self._layer(N.OP_EXT_ATTENTION, [q, k_cache, v_cache, output, sinks], (1, 1, 1),
-                    [heads, kv_heads, vdim, out_col, self._bits(scale), self._bits(softcap or 0.0),
-                     int(sink or sinks is not None), self._bits(out_scale)])
+        `v_cache` may be `k_cache`: the leading `vdim` columns of a key are then its value.  `separate_merge`: the key chunks of
+        a request are merged by all workers in a layer of its own (for wide values) instead of by the last task to arrive."""
+        args = ([q, k_cache, v_cache, output, sinks], (1, 1, 1),
+                [heads, kv_heads, vdim, out_col, self._bits(scale), self._bits(softcap or 0.0), int(sink or sinks is not None),
+                 self._bits(out_scale), int(separate_merge)])
+        self._layer(N.OP_EXT_ATTENTION, *args)
+        if separate_merge:
+            self._layer(N.OP_ATTN_MERGE, *args)
 
     def latent_append_layer(self, proj: DTensor, latent_norm: DTensor, q: DTensor, cache: DTensor, cos: DTensor, sin: DTensor,
                             *, heads: int, rank: int, rot_dims: int, q_col: int, kv_col: int, eps: float):
