@@ -797,12 +797,74 @@ def palarax_case(z, dev):
     return c, w
 
 
-def run_palarax(args):
-    """Prefill (one request, 64 tokens per launch) and decode (batch 1, 16, 64 at --context) of Palarax and of Qwen3 layers of
-    equal size, with the spans of every kind of task group from the in-kernel profiler.  Timed launches carry no profiler."""
+# Lofirax at sizes like those: layers 2 and 3 run twice, so a launch runs 6 gated-linear-attention and 2 latent-attention layers
+# (cache rows of 512 + 64), half of them with experts; recurrent state, heads and width are Palarax's.
+LOFIRAX_SIZES = {
+    "4096": dict(heads=32, dim=128, rot=64, vdim=128, rank=512, ff=12288, experts=32, top=4, eff=1024, shared=2048),
+    "2048": dict(heads=16, dim=128, rot=64, vdim=128, rank=512, ff=6144, experts=64, top=6, eff=512, shared=1024),
+}
+
+
+def lofirax_case(size, dev):
+    """(config, device weights) of one size; random weights."""
     import torch
+    z, y = HYBRID_SIZES[size], LOFIRAX_SIZES[size]
+    D, E = z["width"], y["experts"]
+    moe = {"kind": "moe", "expert": {"ff": y["eff"]}, "shared": {"ff": y["shared"]},
+           "router": {"experts": E, "top": y["top"], "groups": {"count": 4, "keep": 2}}}
+    dense = {"kind": "dense", "ff": y["ff"]}
+    gla = {"type": "gla", "mixer": {"heads": z["mheads"], "dim": z["mdim"], "vdim": z["mvdim"], "tau": 16.0}}
+    lat = {"type": "latent_attention", "mixer": {"heads": y["heads"], "dim": y["dim"], "rot_dim": y["rot"], "vdim": y["vdim"],
+                                                 "kv_rank": y["rank"], "scale": (y["dim"] + y["rot"]) ** -0.5,
+                                                 "rot": {"base": 1e6, "dims": y["rot"]}}}
+    c = {"architecture": "Lofirax", "vocab": HYBRID_VOCAB, "width": D, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+         "logit_softcap": 30.0, "loop": {"start": 2, "stop": 4, "times": 2},
+         "layers": [dict(lat if n == 3 else gla, mlp=moe if n % 2 else dense) for n in range(6)]}
+    g = torch.Generator(device=dev).manual_seed(1)
+    rnd = lambda *s, std=None, mean=0.0: (mean + (s[-1] ** -0.5 if std is None else std) * torch.randn(
+        *s, generator=g, device=dev)).to(torch.bfloat16)
+    w = {"embed": rnd(HYBRID_VOCAB, D, std=1.0), "head": rnd(HYBRID_VOCAB, D), "loop.step": rnd(2, D, std=0.1)}
+
+    def norm(name):
+        w[name], w[name + ".b"] = rnd(D, std=0.1, mean=1.0), rnd(D, std=0.1)
+
+    def ff(p, n):
+        w[p + "gate"], w[p + "up"], w[p + "down"] = rnd(n, D), rnd(n, D), rnd(D, n)
+
+    norm("final.norm")
+    for n, layer in enumerate(c["layers"]):
+        p, m = f"l{n}.", layer["mixer"]
+        norm(p + "norm1"), norm(p + "norm2")
+        if layer["type"] == "gla":
+            H, d, dv = m["heads"], m["dim"], m["vdim"]
+            for nm, rows in (("q", H * d), ("k", H * d), ("v", H * dv), ("g", H * dv), ("a1", 16)):
+                w[p + "mix." + nm] = rnd(rows, D)
+            w[p + "mix.a2"], w[p + "mix.a2.b"], w[p + "mix.norm"] = rnd(H * d, 16), rnd(H * d, std=1.0, mean=2.0), rnd(dv, std=0.1, mean=1.0)
+            w[p + "mix.o"] = rnd(D, H * dv)
+        else:
+            H, rank, rot = m["heads"], m["kv_rank"], m["rot_dim"]
+            w[p + "mix.q"], w[p + "mix.dkv"] = rnd(H * (m["dim"] + rot), D), rnd(rank + rot, D)
+            w[p + "mix.dkv.norm"], w[p + "mix.sink"] = rnd(rank, std=0.1, mean=1.0), rnd(H, std=1.0)
+            w[p + "mix.uk"], w[p + "mix.uv"] = rnd(H * m["dim"], rank), rnd(H * m["vdim"], rank)
+            w[p + "mix.o"] = rnd(D, H * m["vdim"])
+        if n % 2 == 0:
+            ff(p + "mlp.", y["ff"])
+            continue
+        w[p + "mlp.router"], w[p + "mlp.correction"], w[p + "mlp.shared.sg"] = rnd(E, D), rnd(E, std=0.1), rnd(1, D)
+        ff(p + "mlp.shared.", y["shared"])
+        for e in range(E):
+            ff(f"{p}mlp.e{e}.", y["eff"])
+    return c, w
+
+
+def run_hybrid(args):
+    """Prefill (one request, 64 tokens per launch) and decode (batch 1, 16, 64 at --context) of a model on hybrid graphs and of
+    its closest neighbour at equal size (palarax: Qwen3 layers, lofirax: Palarax), with the spans of every kind of task group from
+    the in-kernel profiler.  Timed launches carry no profiler."""
+    import torch
+    from mirage_b200.builders.lofirax import LofiraxConfig
     from mirage_b200.builders.palarax import PalaraxConfig
-    from mirage_b200.builders.runner import DecoderShape, PalaraxRunner, Qwen3Runner
+    from mirage_b200.builders.runner import DecoderShape, LofiraxRunner, PalaraxRunner, Qwen3Runner
     from mirage_b200.profiler import event_spans
     torch.cuda.set_device(0)
     dev = torch.device("cuda", 0)
@@ -815,7 +877,7 @@ def run_palarax(args):
         max_seq = -(-(ctx + prompt + 2 * K + 4 * Wm + 16) // page) * page
         kw = dict(total_num_requests=B, max_seq_length=max_seq, max_num_batched_requests=B, max_num_batched_tokens=mbt,
                   max_num_pages=B * (max_seq // page), page_size=page)
-        spans, ms, clk = {}, None, None
+        spans, ms, clk, experts = {}, None, None, []
         for profiled in (False, True):
             prof = torch.zeros(1 << 20, dtype=torch.int64, device=dev) if profiled else None
             r = make(kw, prof)
@@ -829,9 +891,11 @@ def run_palarax(args):
                 r.step(ctx + Wm)
             st = r.mpk.status()
             assert st.active_tokens == (mbt if prompt > 1 else B), st.active_tokens
+            routing = [t[1] for k, t in getattr(r.builder, "_buffers", {}).items() if k[0] == "routing"]
             if profiled:
                 r.step(1)
                 r.mpk.status()
+                experts = [int(r.mpk.tensor_as_torch(t)[-1]) for t in routing]     # of the launch's last expert layer
                 info = r.mpk.graph_info()
                 for e in event_spans(prof, info["num_tasks"]).values():
                     spans.setdefault(e["type"], []).append(e["us"])
@@ -848,12 +912,15 @@ def run_palarax(args):
             wb = r.mpk.graph_info()["weight_bytes_per_step"]
             del r
             torch.cuda.empty_cache()
-        return ms, wb, {k: [len(v), round(sum(v) / len(v), 2)] for k, v in sorted(spans.items())}, clk
+        return ms, wb, {k: [len(v), round(sum(v) / len(v), 2)] for k, v in sorted(spans.items())}, clk, experts
 
     results, launches, clk = [], 0, None
     for size, z in HYBRID_SIZES.items():
-        for model in ("palarax", "qwen3"):
-            if model == "palarax":
+        for model in {"palarax": ("palarax", "qwen3"), "lofirax": ("lofirax", "palarax")}[args.workload]:
+            if model == "lofirax":
+                c, w = lofirax_case(size, dev)
+                make = lambda kw, prof: LofiraxRunner(LofiraxConfig.from_dict(c), w, profiler_tensor=prof, **kw)
+            elif model == "palarax":
                 c, w = palarax_case(z, dev)
                 make = lambda kw, prof: PalaraxRunner(PalaraxConfig.from_dict(c), w, profiler_tensor=prof, **kw)
             else:
@@ -866,19 +933,24 @@ def run_palarax(args):
                 full = f"{model}_{size}_{name}"
                 if args.cases not in full:
                     continue
-                ms, wb, spans, clk = case(make, B, mbt, prompt)
+                ms, wb, spans, clk, experts = case(make, B, mbt, prompt)
+                if experts:      # panels of the experts active in the last expert layer, taken for all four
+                    wb += 4 * experts[0] * 3 * LOFIRAX_SIZES[size]["eff"] * z["width"] * 2
                 n = mbt if prompt > 1 else B
                 results.append({"case": full, "ms_per_launch": round(ms, 4), "tok_s": round(n * 1e3 / ms, 1), "weight_gb": round(wb / 1e9, 3),
-                                "weight_roofline_frac": round(wb / (ms * 1e-3) / 1e9 / peak, 3), "groups_us": spans})
+                                "weight_roofline_frac": round(wb / (ms * 1e-3) / 1e9 / peak, 3), "groups_us": spans,
+                                **({"active_experts": experts} if experts else {})})
                 launches += K
             w = None
             torch.cuda.empty_cache()
-    head = [r for r in results if r["case"] == "palarax_4096_decode1"] or results
+    head = [r for r in results if r["case"] == args.workload + "_4096_decode1"] or results
     print(json.dumps({
-        "metric": "palarax_decode_ms_per_token_bs1", "value": head[0]["ms_per_launch"], "unit": "ms/token", "n_gpus": 1, "steps": K,
+        "metric": args.workload + "_decode_ms_per_token_bs1", "value": head[0]["ms_per_launch"], "unit": "ms/token", "n_gpus": 1, "steps": K,
         "warmup": Wm, "ms_per_step": head[0]["ms_per_launch"], "higher_is_better": False, "scaling": "strong", "vs_baseline": None,
         "dtype": "bf16", "data": "synthetic",
-        "config": {"workload": "Palarax 6 matrix-memory + 2 parallel layers beside 8 Qwen3 layers, width 4096 and 2048, context %d" % ctx,
+        "config": {"workload": {"palarax": "Palarax 6 matrix-memory + 2 parallel layers beside 8 Qwen3 layers, width 4096 and 2048, context %d",
+                                "lofirax": "Lofirax 6 gated-linear + 2 latent-attention layer runs (half with experts) beside Palarax 6 "
+                                           "matrix-memory + 2 parallel layers, width 4096 and 2048, context %d"}[args.workload] % ctx,
                    "l2": "weights of a launch exceed L2; every launch re-streams them"},
         "gpu_launches": launches, "clocks": clk, "peak_gbs": peak, "peak_kind": peak_kind, "results": results}))
 
@@ -906,11 +978,11 @@ def main():
                     help="N > 1: split the lm_head rows over the ranks and merge the ranks' argmax inside the kernel "
                          "(default: every rank keeps the whole lm_head, as the reference does)")
     ap.add_argument("--workload", default="qwen3", choices=["qwen3", "fp8_layer", "moe_block", "mla_decode", "deepseek_slice", "moe_w13", "mla_dense",
-                                                             "palarax"],
+                                                             "palarax", "lofirax"],
                     help="qwen3: the headline decode benchmark; the others time one block of the FP8 / MoE / MLA "
-                         "task bodies at the shapes of the DeepSeek-V3-style parity configurations (1 GPU); palarax: prefill "
-                         "and decode of Palarax at a few sizes beside Qwen3 layers of equal size (1 GPU)")
-    ap.add_argument("--cases", default="", help="palarax: only cases whose name contains this text")
+                         "task bodies at the shapes of the DeepSeek-V3-style parity configurations (1 GPU); palarax, lofirax: "
+                         "prefill and decode at a few sizes beside the closest other model's layers of equal size (Qwen3; Palarax) (1 GPU)")
+    ap.add_argument("--cases", default="", help="palarax, lofirax: only cases whose name contains this text")
     args = ap.parse_args()
     if args.impl == "reference":
         return run_reference(args)
@@ -918,8 +990,8 @@ def main():
         return run_ref_kernel(args)
     if args.workload == "deepseek_slice":
         return run_deepseek_slice(args)
-    if args.workload == "palarax":
-        return run_palarax(args)
+    if args.workload in ("palarax", "lofirax"):
+        return run_hybrid(args)
     if args.workload != "qwen3":
         return run_block_workload(args)
 
