@@ -279,14 +279,28 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
         xv[i].z += yv[i].z * inv * oz; xv[i].w += yv[i].w * inv * ow;
       }
     }
-    if (nt.slots > 0 || nt.add || nt.row) {
+    for (int k = 0; k < nt.slots; k += 2) {   // two experts' rows in flight
+      float4 e[2][NV];
+      float w[2];
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        w[u] = k + u < nt.slots ? __ldcg(nt.ew + k + u) : 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int j = (i * kConsumerThreads + tid) * 4;
+          e[u][i] = j < W && k + u < nt.slots ? __ldcg(reinterpret_cast<const float4 *>(nt.experts + (size_t)(k + u) * W + j)) : zero;
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int i = 0; i < NV; ++i) fma4(xv[i], w[u], e[u][i]);
+    }
+    if (nt.add || nt.row) {
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int j = (i * kConsumerThreads + tid) * 4;
         if (j >= W) break;
-#pragma unroll 4
-        for (int k = 0; k < nt.slots; ++k)
-          fma4(xv[i], __ldcg(nt.ew + k), __ldcg(reinterpret_cast<const float4 *>(nt.experts + (size_t)k * W + j)));
         if (nt.add) fma4(xv[i], 1.f, __ldcg(reinterpret_cast<const float4 *>(nt.add + j)));
         if (nt.row) fma4(xv[i], 1.f, bf16x4_at(nt.row, j));
       }
@@ -1204,74 +1218,97 @@ __device__ __noinline__ void ext_attention_mma(const Ctx c, const TaskDesc &d, c
 //   softmax  a warp takes RT / 8 rows, online in base 2; weights go back as a bf16 value and a bf16 remainder, so that they
 //            keep 16 bits
 //   output   every warp owns eight-column tiles w, w + 8, ... of all rows
+//
+// (with a few KB of L1 beside the shared memory a spilled variable of the key loop costs an L2 round trip: areas of fixed size
+// come first, so that their addresses are one base plus constants, and everything is addressed in 32 bits)
+__device__ __forceinline__ float lds_f32(uint32_t a) {
+  float v;
+  asm volatile("ld.shared.f32 %0, [%1];" : "=f"(v) : "r"(a));
+  return v;
+}
+__device__ __forceinline__ int lds_s32(uint32_t a) {
+  int v;
+  asm volatile("ld.shared.s32 %0, [%1];" : "=r"(v) : "r"(a));
+  return v;
+}
+__device__ __forceinline__ void sts_f32(uint32_t a, float v) { asm volatile("st.shared.f32 [%0], %1;" ::"r"(a), "f"(v) : "memory"); }
+__device__ __forceinline__ void sts_f32x2(uint32_t a, float v, float w) { asm volatile("st.shared.v2.f32 [%0], {%1, %2};" ::"r"(a), "f"(v), "f"(w) : "memory"); }
+__device__ __forceinline__ void sts_bf16(uint32_t a, __nv_bfloat16 v) {
+  asm volatile("st.shared.b16 [%0], %1;" ::"r"(a), "h"(__bfloat16_as_ushort(v)) : "memory");
+}
+__device__ __forceinline__ void sts_zero16(uint32_t a) { asm volatile("st.shared.v4.b32 [%0], {%1,%1,%1,%1};" ::"r"(a), "r"(0) : "memory"); }
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void *src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
 template <int MT, int KEYS>
 __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d, const SeqView sv, const AttnOut &ao, int k0, int k1,
                                                   int row0, int nrow, int task) {
   constexpr int RT = MT * 16, KW = KEYS / 16, KS = 8 / KW, SP = KEYS + 4, PP = KEYS * 2 + 16, NV = 8;
   constexpr int RPW = RT * KEYS / 256;             // row sets a warp's lanes hold in the softmax (32 / KEYS rows at a time)
-  const KernelParams &P = c.P;
+  // shared memory: partial scores [KS][RT][SP], weights [value, remainder][RT][PP], rescale factors [RT] (at the end m and l [2][RT]),
+  // cache row of every eighth key [kXaCells], queries [RT][pitch], ring of key tiles [stages][KEYS][pitch]
+  constexpr uint32_t oP = KS * RT * SP * 4, oC = oP + 2 * RT * PP, oCell = oC + 8 * RT, oQ = (oCell + kXaCells * 4 + 15) & ~15u;
+  const uint32_t sm = smem_u32(c.s.xtile);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int G = ao.G, dimp = d.a[XA_DIMP], D = (dimp + 63) & ~63, page = d.a[XA_PAGE], nstg = d.a[XA_STAGES];
-  const uint32_t pitch = D * 2 + 16;
-  const int pieces = dimp >> 3;                    // 16-byte pieces of a row
-  uint8_t *qs = c.s.xtile;                         // [RT][pitch]
-  uint8_t *st = qs + RT * pitch;                   // [nstg][KEYS][pitch]
-  float *sp = reinterpret_cast<float *>(st + (size_t)nstg * KEYS * pitch);   // [KS][RT][SP]
-  uint8_t *ps = reinterpret_cast<uint8_t *>(sp + KS * RT * SP);              // [value, remainder][RT][PP]
-  float *corr_s = reinterpret_cast<float *>(ps + 2 * RT * PP);               // [RT] rescale factors; at the end m and l
-  int *cells = reinterpret_cast<int *>(corr_s + 2 * RT);                     // [kXaCells] cache row of every eighth key
-  const int kend = min(k1, sv.pos0 + (row0 + nrow - 1) / G + 1);
+  const int pieces = d.a[XA_DIMP] >> 3, ksteps = (pieces + 7) / 8 * 4;   // 16-byte pieces of a cache row, 16-column steps of a padded one
+  const uint32_t pitch = ksteps * 32 + 16, tile = KEYS * pitch, ring = sm + oQ + RT * pitch;
+  const int nstg = d.a[XA_STAGES];
+  const int kend = min(k1, sv.pos0 + (row0 + nrow - 1) / ao.G + 1);
   const int ntiles = kend > k0 ? (kend - k0 + KEYS - 1) / KEYS : 0;
-  const uint8_t *qg = reinterpret_cast<const uint8_t *>(d.p[0]), *kg = reinterpret_cast<const uint8_t *>(d.p[1]);
-  const int ncell = (page & 7) == 0 && k1 - k0 <= 8 * kXaCells ? (k1 - k0 + 7) >> 3 : 0;
-  auto cell_row = [&](int key) {
-    const int pg = key / page;
-    return __ldcg(&P.meta.paged_kv_indices[sv.kv0 + pg]) * page + (key - pg * page);
-  };
-  for (int i = tid; i < ncell; i += kConsumerThreads) cells[i] = cell_row(k0 + 8 * i);
-  const uint4 zero = make_uint4(0, 0, 0, 0);
-  for (int r = warp; r < RT; r += 8)
-    for (int p = lane; p < D >> 3; p += 32) {
-      uint4 v = zero;
-      if (r < nrow && p < pieces)
-        v = __ldcg(reinterpret_cast<const uint4 *>(qg + ((size_t)(sv.q0 + (row0 + r) / G) * d.a[XA_LDQ] + (size_t)((row0 + r) % G) * dimp) * 2) + p);
-      *reinterpret_cast<uint4 *>(qs + r * pitch + p * 16) = v;
+  const uint4 *kg = reinterpret_cast<const uint4 *>(d.p[1]);
+  const int page = d.a[XA_PAGE];
+  const bool table = (page & 7) == 0 && k1 - k0 <= 8 * kXaCells;   // eight consecutive keys lie in one page
+  const int32_t *pages = c.P.meta.paged_kv_indices + sv.kv0;
+  auto cell_row = [&](int key) { return __ldcg(pages + key / page) * page + key % page; };
+  if (table)
+    for (int i = tid; i < (kend - k0 + 7) >> 3; i += kConsumerThreads)
+      asm volatile("st.shared.s32 [%0], %1;" ::"r"(sm + oCell + i * 4), "r"(cell_row(k0 + 8 * i)) : "memory");
+  {   // queries, and zeros where no copy reaches
+    const uint4 *qg = reinterpret_cast<const uint4 *>(d.p[0]);
+    const int G = ao.G, ldq = d.a[XA_LDQ] >> 3;
+    for (int r = warp; r < RT; r += 8) {
+      const uint32_t dst = sm + oQ + r * pitch;
+      const uint4 *src = qg + (size_t)(sv.q0 + (row0 + r) / G) * ldq + (size_t)((row0 + r) % G) * pieces;
+      for (int p = lane; p < ksteps * 2; p += 32) {
+        if (r < nrow && p < pieces) cp_async16(dst + p * 16, src + p);
+        else sts_zero16(dst + p * 16);
+      }
     }
-  if (pieces < D >> 3)   // columns no copy reaches
-    for (int r = warp; r < nstg * KEYS; r += 8)
-      for (int p = pieces + lane; p < D >> 3; p += 32) *reinterpret_cast<uint4 *>(st + (size_t)r * pitch + p * 16) = zero;
-  consumer_sync();
+    if (pieces < ksteps * 2)
+      for (int r = warp; r < nstg * KEYS; r += 8)
+        for (int p = pieces + lane; p < ksteps * 2; p += 32) sts_zero16(ring + r * pitch + p * 16);
+  }
+  consumer_sync();   // (the table of cache rows)
   stamp(c, task, 0);
   auto issue = [&](int it, int stg) {
     if (it < ntiles) {
 #pragma unroll
       for (int r = 0; r < KEYS / 8; ++r) {
-        const int key = k0 + it * KEYS + warp + 8 * r;
-        uint8_t *dst = st + (size_t)(stg * KEYS + warp + 8 * r) * pitch;
-        if (key < kend) {
-          const size_t cell = ncell > 0 ? (size_t)(cells[(key - k0) >> 3] + ((key - k0) & 7)) : (size_t)cell_row(key);
-          const uint8_t *src = kg + cell * dimp * 2;
-          for (int p = lane; p < pieces; p += 32)
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst + p * 16)), "l"(src + p * 16) : "memory");
+        const int kk = it * KEYS + warp + 8 * r;   // key relative to the chunk
+        const uint32_t dst = ring + stg * tile + (warp + 8 * r) * pitch;
+        if (k0 + kk < kend) {
+          const uint4 *src = kg + (size_t)(table ? lds_s32(sm + oCell + (kk >> 3) * 4) + (kk & 7) : cell_row(k0 + kk)) * pieces;
+          for (int p = lane; p < pieces; p += 32) cp_async16(dst + p * 16, src + p);
         } else {   // a masked key has weight 0, and 0 x NaN would be NaN
-          for (int p = lane; p < pieces; p += 32) *reinterpret_cast<uint4 *>(dst + p * 16) = zero;
+          for (int p = lane; p < pieces; p += 32) sts_zero16(dst + p * 16);
         }
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  for (int i = 0; i < nstg - 1; ++i) issue(i, i);
+  for (int i = 0; i < nstg - 1; ++i) issue(i, i);   // (the queries join the first group)
   const float scale = __int_as_float(d.a[XA_SCALE]), cap = __int_as_float(d.a[XA_CAP]);
-  const float cap2 = cap > 0.f ? 2.0f * 1.4426950408889634f / cap : 0.f;
-  const int kw = warp % KW, ks = warp / KW, ksteps = D >> 4;
-  const uint32_t qa = smem_u32(qs) + (uint32_t)((lane & 15) * pitch + (lane >> 4) * 16);
-  const uint32_t pa = smem_u32(ps) + (uint32_t)((lane & 15) * PP + (lane >> 4) * 16);
-  // softmax: this lane's key of the tile and first row
+  const int nv = (ao.vdim >> 3) > warp ? ((ao.vdim >> 3) - warp + 7) >> 3 : 0;   // this warp's column tiles
+  // softmax: this lane's key of the tile, its first row and the last keys that row set sees
   const int skey = lane % KEYS, srow = warp * (RT / 8) + lane / KEYS;
+  int seen[RPW];
   float m_run[RPW], l_run[RPW];
 #pragma unroll
-  for (int i = 0; i < RPW; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
-  const int nv = (ao.vdim >> 3) > warp ? ((ao.vdim >> 3) - warp + 7) >> 3 : 0;   // this warp's column tiles
+  for (int i = 0; i < RPW; ++i) {
+    m_run[i] = -INFINITY;
+    l_run[i] = 0.f;
+    seen[i] = min(kend - 1, sv.pos0 + (row0 + srow + i * (32 / KEYS)) / ao.G) - skey - k0;   // relative to the tile's first key
+  }
   float o[MT][NV][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -1288,9 +1325,10 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
     consumer_sync();   // the tile has landed for everyone, and everyone is done with the stage refilled next
     if (it == 0) stamp(c, task, 1);
     issue(it + nstg - 1, stg == 0 ? nstg - 1 : stg - 1);
-    const uint32_t kt = smem_u32(st + (size_t)stg * KEYS * pitch);
+    const uint32_t kt = ring + stg * tile;
     if (++stg == nstg) stg = 0;
     {   // ---- scores
+      const int kw = warp % KW, ks = warp / KW;
       float s[MT][2][4];
 #pragma unroll
       for (int m = 0; m < MT; ++m)
@@ -1299,7 +1337,8 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[m][n][e] = 0.f;
       const uint32_t ka = kt + (uint32_t)((kw * 16 + (lane & 7) + (lane >> 4) * 8) * pitch + ((lane >> 3) & 1) * 16);
-#pragma unroll 3
+      const uint32_t qa = sm + oQ + (uint32_t)((lane & 15) * pitch + (lane >> 4) * 16);
+#pragma unroll 2
       for (int kk = ks; kk < ksteps; kk += KS) {
         uint32_t b[4];
         ldmatrix_x4(b, ka + kk * 32u);
@@ -1311,26 +1350,27 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
           mma_bf16_16816(s[m][1], a, b[2], b[3]);
         }
       }
-      float *sr = sp + (size_t)(ks * RT + (lane >> 2)) * SP + kw * 16 + 2 * (lane & 3);
+      const uint32_t sr = sm + (uint32_t)(((ks * RT + (lane >> 2)) * SP + kw * 16 + 2 * (lane & 3)) * 4);
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
         for (int n = 0; n < 2; ++n) {
-          *reinterpret_cast<float2 *>(sr + m * 16 * SP + n * 8) = make_float2(s[m][n][0], s[m][n][1]);
-          *reinterpret_cast<float2 *>(sr + (m * 16 + 8) * SP + n * 8) = make_float2(s[m][n][2], s[m][n][3]);
+          sts_f32x2(sr + (m * 16 * SP + n * 8) * 4, s[m][n][0], s[m][n][1]);
+          sts_f32x2(sr + ((m * 16 + 8) * SP + n * 8) * 4, s[m][n][2], s[m][n][3]);
         }
     }
     consumer_sync();
     {   // ---- softmax
-      const int key = k0 + it * KEYS + skey;
+      const uint32_t sa = sm + (uint32_t)((srow * SP + skey) * 4), pa = sm + oP + (uint32_t)(srow * PP + skey * 2);
+      const float cap2 = cap > 0.f ? 2.0f * 1.4426950408889634f / cap : 0.f;
 #pragma unroll
       for (int i = 0; i < RPW; ++i) {
-        const int r = srow + i * (32 / KEYS);
+        const int r = i * (32 / KEYS);
         float v = 0.f;
 #pragma unroll
-        for (int p = 0; p < KS; ++p) v += sp[(size_t)(p * RT + r) * SP + skey];
+        for (int p = 0; p < KS; ++p) v += lds_f32(sa + (p * RT + r) * SP * 4);
         v = attn_score<HYB_BF16>(v, scale, cap, cap2);
-        if (key >= kend || key > sv.pos0 + (row0 + r) / G) v = -INFINITY;
+        if (it * KEYS > seen[i]) v = -INFINITY;
         float mx = v;
 #pragma unroll
         for (int sh = KEYS / 2; sh > 0; sh >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, sh));
@@ -1339,20 +1379,20 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
         m_run[i] = mn;
         l_run[i] = l_run[i] * corr + p;
         const __nv_bfloat16 hi = __float2bfloat16_rn(p);
-        *reinterpret_cast<__nv_bfloat16 *>(ps + r * PP + skey * 2) = hi;
-        *reinterpret_cast<__nv_bfloat16 *>(ps + (RT + r) * PP + skey * 2) = __float2bfloat16_rn(p - bf16_to_f(hi));
-        if (skey == 0) corr_s[r] = corr;
+        sts_bf16(pa + r * PP, hi);
+        sts_bf16(pa + (RT + r) * PP, __float2bfloat16_rn(p - bf16_to_f(hi)));
+        if (skey == 0) sts_f32(sm + oC + (srow + r) * 4, corr);
       }
     }
     consumer_sync();
     {   // ---- output
-      float cr[MT][2];
       bool keep = true;
+      float cr[MT][2];
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
-          cr[m][h] = corr_s[m * 16 + h * 8 + (lane >> 2)];
+          cr[m][h] = lds_f32(sm + oC + (m * 16 + h * 8 + (lane >> 2)) * 4);
           keep = keep && cr[m][h] == 1.f;
         }
       if (!__all_sync(0xffffffffu, keep)) {
@@ -1365,6 +1405,7 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
           }
       }
       // 16 keys and two column tiles at a time (one past the last is read, not used)
+      const uint32_t pa = sm + oP + (uint32_t)((lane & 15) * PP + (lane >> 4) * 16);
 #pragma unroll
       for (int k = 0; k < KW; ++k) {
         uint32_t p[2][MT][4];
@@ -1390,18 +1431,17 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
     }
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
-  consumer_sync();
   stamp(c, task, 2);
   // running maximum and sum of every row
+  consumer_sync();
 #pragma unroll
   for (int i = 0; i < RPW; ++i) {
     float l = l_run[i];
 #pragma unroll
     for (int sh = KEYS / 2; sh > 0; sh >>= 1) l += __shfl_xor_sync(0xffffffffu, l, sh);
     if (skey == 0) {
-      const int r = srow + i * (32 / KEYS);
-      corr_s[r] = m_run[i];
-      corr_s[RT + r] = l;
+      sts_f32(sm + oC + (srow + i * (32 / KEYS)) * 4, m_run[i]);
+      sts_f32(sm + oC + (RT + srow + i * (32 / KEYS)) * 4, l);
     }
   }
   consumer_sync();
@@ -1411,21 +1451,21 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
     for (int h = 0; h < 2; ++h) {
       const int r = m * 16 + h * 8 + (lane >> 2), row = row0 + r;
       if (r >= nrow) continue;
-      const float mx = corr_s[r], l = corr_s[RT + r];
+      const float mx = lds_f32(sm + oC + r * 4), l = lds_f32(sm + oC + (RT + r) * 4);
       const int col0 = warp * 8 + 2 * (lane & 3);
       if (ao.n_act == 1) {
-        const int hq_idx = row % G;
+        const int hq_idx = row % ao.G;
         const float sk = ao.sink ? sink_logit<HYB_BF16>(d, hq_idx) : 0.f;
         const float M = ao.sink ? fmaxf(mx, sk) : mx;
         const float w = mx == -INFINITY ? 0.f : exp2f(mx - M);
         const float L = l * w + (ao.sink ? exp2f(sk - M) : 0.f);
         const float f = L > 0.f ? w / L * ao.oscale : 0.f;
-        __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(d.p[3]) + (size_t)(sv.q0 + row / G) * ao.ldo + ao.ocol + (size_t)hq_idx * ao.vdim + col0;
+        __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(d.p[3]) + (size_t)(sv.q0 + row / ao.G) * ao.ldo + ao.ocol + (size_t)hq_idx * ao.vdim + col0;
 #pragma unroll
         for (int i = 0; i < NV; ++i)
           if (i < nv) *reinterpret_cast<uint32_t *>(out + i * 64) = pack_bf16(o[m][i][2 * h] * f, o[m][i][2 * h + 1] * f);
       } else {
-        float *rec = attn_record(P, ao, row);
+        float *rec = attn_record(c.P, ao, row);
         if (warp == 0 && (lane & 3) == 0) {
           __stcg(rec, mx);
           __stcg(rec + 1, l);

@@ -168,8 +168,30 @@ __device__ void streamer_loop(const Ctx &c, int t_begin, int t_end) {
       const int rows = d->a[L_N1] - d->a[L_N0], RB = d->a[L_ROWS];
       const int kbe = (!HYB && (d->flags & TF_FP8)) ? 2 * kTcKBlock : kTcKBlock;   // elements of one 128-byte k block
       const int nkb = d->a[L_KC] / kbe, kbt = d->a[L_KT] / kbe, kball = d->a[L_K] / kbe;
-      const int tiles = (rows + RB - 1) / RB;
       const uint32_t tx = (uint32_t)(nkb * RB * 128);
+      if (kMoe && d->type == TASK_MOE_GEMM) {
+        // expert projections on the tensor path: the row tiles of the active experts, dealt out to the layer's tasks in turn
+        const int *act = reinterpret_cast<const int *>(d->p[5]);
+        const int N = d->a[L_N], per = (N + RB - 1) / RB, items = min(__ldcg(&act[d->a[M_NEXP]]), d->a[M_NEXP]) * per;
+        for (int it = d->a[L_N0]; it < items && ok; it += d->a[L_N1]) {
+          const int row = __ldcg(&act[it / per]) * N + it % per * RB;
+          for (int kb = 0; kb < kball; kb += nkb) {
+            if (lane == 0) {
+              ok = wait_mbar(c, &c.s.empty[s], ph ^ 1u, t);
+              if (ok) {
+                mbar_arrive_expect_tx(&c.s.full[s], tx);
+                tma_load_3d(c.s.stages + (size_t)s * P.stage_bytes, tmap, 0, row, kb, &c.s.full[s], policy);
+              }
+            }
+            ok = __shfl_sync(0xffffffffu, (int)ok, 0) != 0;
+            if (!ok) break;
+            ++issued;
+            if (++s == NST) { s = 0; ph ^= 1u; }
+          }
+        }
+        continue;
+      }
+      const int tiles = (rows + RB - 1) / RB;
       for (int kb_t = 0; kb_t < kball && ok; kb_t += kbt)
         for (int tile = 0; tile < tiles && ok; ++tile)
           for (int kb = 0; kb < kbt; kb += nkb) {
@@ -1651,8 +1673,7 @@ static __device__ void run_moe_routing(const Ctx &c, const TaskDesc &d) {
       if (!((selected >> (e / per)) & 1ull)) bi[e] = -10000.f;
     __syncwarp();
     float total = 0.f;
-    if (lane < 32 && lane < topk) gs[32 + lane] = 0.f;
-    __syncwarp();
+    float mine = 0.f;   // lane k < topk: slot k's weight (0: its expert belongs to another rank)
     for (int k = 0; k < topk; ++k) {
       float mv = -3.0e38f;
       int me = E;
@@ -1666,27 +1687,22 @@ static __device__ void run_moe_routing(const Ctx &c, const TaskDesc &d) {
         const int oe = __shfl_xor_sync(0xffffffffu, me, o);
         if (ov > mv || (ov == mv && oe < me)) { mv = ov; me = oe; }
       }
+      const float orig = sc[me];
+      const bool local = me >= e_lo && me < e_hi;
+      total += orig;
+      if (lane == k && local) mine = orig;
+      __syncwarp();
       if (lane == 0) {
-        const float orig = sc[me];
-        wout[(size_t)row * ldw + k] = orig;
-        total += orig;
-        if (me >= e_lo && me < e_hi) {
+        if (local) {
           routing[(size_t)me * ldr + row] = k + 1;
           mark[me] = 1;
-        } else {
-          gs[32 + k] = -1.f;   // (group scores are dead by now: remember that slot k belongs to another rank)
         }
         bi[me] = -10000.f;
       }
       __syncwarp();
     }
-    if (lane == 0) {
-      const float inv = __fdiv_rn(1.0f, total + 1e-20f);
-      for (int k = 0; k < topk; ++k) {
-        const bool local = gs[32 + k] >= 0.f;
-        wout[(size_t)row * ldw + k] = local ? wout[(size_t)row * ldw + k] * inv * scaling : 0.f;
-      }
-    }
+    const float inv = __fdiv_rn(1.0f, total + 1e-20f);
+    if (lane < topk) wout[(size_t)row * ldw + lane] = mine * inv * scaling;
     __syncwarp();
   }
   consumer_sync();
@@ -1988,10 +2004,167 @@ __device__ void run_moe_gemm(const Ctx &c, const TaskDesc &d, LinearState &ls, i
 
 // TASK_MOE_SILU_MUL: rows of [gate | up] -> bf16(silu(gate)) * up  (tasks/ampere/silu_mul.cuh:20-42 on the
 // flattened [token x slot] rows, as register_moe_silu_mul_task sets it up)
+// Expert projections on tcgen05 (bf16 hybrid graphs of more than 8 batched tokens).  A row tile of an active expert is a linear of
+// RB <= 128 rows over the tokens routed to it: the weight tile streams through the ring as swizzled boxes, the tokens' rows are
+// gathered into the operand tile (N = their number rounded up to 16), eight warps issue MMAs into accumulators of their own, and the
+// epilogue scatters to (token, slot) rows.  Row tiles are dealt out to the workers in turn, whatever the routing; the next tile's
+// token rows are gathered while the current one's MMAs run where both fit.
+static __device__ void run_moe_gemm_tc(const Ctx &c, const TaskDesc &d, LinearState &ls, int task, bool ok) {
+  const KernelParams &P = c.P;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int B = ok ? min(active_tokens(P), kMaxLinearTokens) : 0;
+  const int K = d.a[L_K], RB = d.a[L_ROWS], N = d.a[L_N], E = d.a[M_NEXP], topk = d.a[M_NTOPK], ldr = d.a[M_LDR], ldx = d.a[L_LDX];
+  const int nkb = d.a[L_KC] / kTcKBlock, kball = K / kTcKBlock, per = (N + RB - 1) / RB, step = d.a[L_N1], epi = d.a[L_EPI], ldo = d.a[L_LDO];
+  const bool per_slot = d.a[M_PER_SLOT] != 0;
+  const int NST = P.num_stages, stage_bytes = P.stage_bytes, room = P.x_tile_bytes;
+  const int *routing = reinterpret_cast<const int *>(d.p[4]), *active = reinterpret_cast<const int *>(d.p[5]);
+  const uint8_t *xg = reinterpret_cast<const uint8_t *>(d.p[1]);
+  uint8_t *out = reinterpret_cast<uint8_t *>(d.p[2]);
+  const int items = ok ? min(__ldcg(&active[E]), E) * per : 0;
+  unsigned short *lists = reinterpret_cast<unsigned short *>(c.s.red);   // two lists of token | slot << 8
+  int *cnt_s = c.s.flags + 8;                                            // their lengths: [list][half]
+  const uint32_t x0 = smem_u32(c.s.xtile), st0 = smem_u32(c.s.stages), tmem = c.tmem_base;
+  const uint64_t desc_hi = umma_desc_k_sw128(0);
+  // warps 0 and 1: the expert's tokens; complete after the next barrier of the compute warps
+  auto build = [&](int it, int which) {
+    if (warp < 2) {
+      const int b = warp * 32 + lane;
+      const int r = b < B ? __ldcg(&routing[(size_t)__ldcg(&active[it / per]) * ldr + b]) : 0;
+      const unsigned bal = __ballot_sync(0xffffffffu, r != 0);
+      if (lane == 0) cnt_s[2 * which + warp] = __popc(bal);
+      asm volatile("bar.sync 2, 64;");
+      if (r != 0) lists[which * 64 + (warp ? cnt_s[2 * which] : 0) + __popc(bal & ((1u << lane) - 1u))] = (unsigned short)(b | ((r - 1) << 8));
+    }
+  };
+  // asynchronous copies of columns [k0, k0 + kn) of the list's token rows into the operand tile at `off` (committed)
+  auto gather = [&](int which, int cnt, int NP, int k0, int kn, uint32_t off) {
+    const int vecs = kn >> 3;
+    for (int i = tid; i < cnt * vecs; i += kConsumerThreads) {
+      const int t = i / vecs, v = i - t * vecs, tm = lists[which * 64 + t];
+      const size_t row = per_slot ? (size_t)(tm & 0xff) * topk + (tm >> 8) : (size_t)(tm & 0xff);
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(x0 + off + (uint32_t)((v >> 3) * NP * 128 + t * 128 + (((v & 7) ^ (t & 7)) << 4))),
+                   "l"(xg + (row * ldx + k0) * 2 + (size_t)v * 16)
+                   : "memory");
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  auto padded = [](int cnt) { return max(16, (cnt + 15) & ~15); };
+  int it = d.a[L_N0], which = 0, stage = ls.stage;
+  uint32_t phase = ls.phase, off = 0;
+  bool staged = false;
+  if (it < items) {
+    build(it, 0);
+    consumer_sync();
+  }
+  for (; it < items && ok; it += step, which ^= 1) {
+    const int cnt = cnt_s[2 * which] + cnt_s[2 * which + 1], NP = padded(cnt);
+    const int KT = min(K, room / (NP * 128) / nkb * nkb * kTcKBlock);
+    const int row0 = it % per * RB;
+    const uint32_t idesc = umma_idesc(1u, 128, NP);
+    const int sets = min(8, kTcAccCols / NP);
+    const bool more = it + step < items;
+    tc_fence_after_sync();
+    if (warp < 4) {
+      for (int col = 0; col < sets * NP; col += 16) tmem_st_zero_x16(tmem + ((uint32_t)(warp * 32) << 16) + (uint32_t)col);
+      tmem_st_wait();
+    }
+    tc_fence_before_sync();
+    uint32_t off_n = 0;
+    bool staged_n = false;
+    for (int k0 = 0; k0 < K; k0 += KT) {
+      const int kn = min(KT, K - k0);
+      if (!staged || k0 > 0) gather(which, cnt, NP, k0, kn, k0 > 0 ? 0u : off);
+      if (k0 == 0 && more) build(it + step, which ^ 1);
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+      fence_proxy_async_smem();   // the tile was written through the generic proxy; the MMA reads it through the async proxy
+      consumer_sync();
+      tc_fence_after_sync();
+      if (k0 == 0 && more && KT == K) {
+        const int cn = cnt_s[2 * (which ^ 1)] + cnt_s[2 * (which ^ 1) + 1], NPn = padded(cn);
+        const uint32_t mine = (uint32_t)(NP * 2 * K), next = (uint32_t)(NPn * 2 * K);
+        off_n = off + mine;
+        staged_n = off_n + next <= (uint32_t)room;
+        if (!staged_n && next <= off) { off_n = 0; staged_n = true; }
+        if (staged_n) gather(which ^ 1, cn, NPn, 0, K, off_n);
+        else off_n = 0;
+      }
+      const uint32_t xb = (x0 + (k0 > 0 ? 0u : off)) >> 4;
+      for (int kb = 0; kb < kn / kTcKBlock; kb += nkb) {
+        const int s = stage;
+        const uint32_t ph = phase;
+        if (++stage == NST) { stage = 0; phase ^= 1u; }
+        if (ok) ok = wait_mbar(c, &c.s.full[s], ph, task);
+        if (ok && lane == 0) {
+          tc_fence_after_sync();
+          const uint32_t a_base = (st0 + (uint32_t)(s * stage_bytes)) >> 4;
+          for (int m = warp; warp < sets && m < nkb * 4; m += sets) {
+            const int j = m >> 2, kk = m & 3;
+            umma_bf16_acc(tmem + (uint32_t)(warp * NP), desc_hi | (a_base + (uint32_t)(j * RB * 8 + kk * 2)),
+                          desc_hi | (xb + (uint32_t)((kb + j) * NP * 8 + kk * 2)), idesc);
+          }
+          umma_commit(&c.s.empty[s]);
+        }
+        __syncwarp();
+      }
+      // accumulators complete for these columns / operand tile free again: one arrival per warp
+      if (lane == 0) umma_commit(c.s.acc_bar);
+      if (!wait_mbar(c, c.s.acc_bar, ls.acc_phase, task)) ok = false;
+      ls.acc_phase ^= 1u;
+      if (!ok) c.s.flags[0] = 1;
+      consumer_sync();
+      ok = ok && (c.s.flags[0] == 0);
+      if (!ok) break;
+    }
+    if (!ok) break;
+    tc_fence_after_sync();
+    const int quad = warp & 3, half = warp >> 2, nh = NP >> 1, r = quad * 32 + lane, row = row0 + r;
+    if (quad * 32 < RB) {
+      const bool row_ok = r < RB && row < N;
+      const uint32_t taddr = tmem + ((uint32_t)(quad * 32) << 16) + (uint32_t)(half * nh);
+      for (int c0 = 0; c0 < nh && half * nh + c0 < cnt; c0 += 8) {
+        uint32_t v[8];
+        tmem_ld_x8(taddr + (uint32_t)c0, v);
+        for (int st = 1; st < sets; ++st) {   // the other issuers' accumulators, in set order
+          uint32_t v2[8];
+          tmem_ld_wait();
+          tmem_ld_x8(taddr + (uint32_t)(st * NP + c0), v2);
+          tmem_ld_wait();
+#pragma unroll
+          for (int j = 0; j < 8; ++j) v[j] = __float_as_uint(__uint_as_float(v[j]) + __uint_as_float(v2[j]));
+        }
+        tmem_ld_wait();
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          const float x = __uint_as_float(v[j]), u = __shfl_down_sync(0xffffffffu, x, 2);
+          const int t = half * nh + c0 + j;
+          if (!row_ok || t >= cnt) continue;
+          const int tm = lists[which * 64 + t];
+          const size_t orow = ((size_t)(tm & 0xff) * topk + (tm >> 8)) * ldo;
+          if (epi == EPI_STORE_F32) reinterpret_cast<float *>(out)[orow + row] = x;
+          else if (epi == EPI_STORE) reinterpret_cast<__nv_bfloat16 *>(out)[orow + row] = __float2bfloat16_rn(x);
+          else if ((row & 2) == 0)
+            reinterpret_cast<__nv_bfloat16 *>(out)[orow + ((row >> 2) << 1) + (row & 1)] =
+                __float2bfloat16_rn((epi == EPI_GATED_SILU ? silu_exact_f(x) : gelu_tanh_f(x)) * u);
+        }
+      }
+    }
+    tc_fence_before_sync();   // the accumulators have been read: the next item clears them after this barrier
+    consumer_sync();
+    staged = staged_n;
+    off = off_n;
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  if (!ok) c.s.flags[0] = 1;
+  ls.stage = stage;
+  ls.phase = phase;
+}
+
 // Hybrid graphs (bf16 only): a function of its own, state of the stage ring by value, so that the linear loop's registers stay as
 // they are.
-static __device__ __noinline__ LinearState run_moe_gemm_hybrid(const Ctx c, const TaskDesc &d, LinearState ls, int task, bool ok) {
-  run_moe_gemm<true>(c, d, ls, task, ok);
+template <bool GENERAL>
+__device__ __noinline__ LinearState run_moe_gemm_hybrid(const Ctx c, const TaskDesc &d, LinearState ls, int task, bool ok) {
+  if (GENERAL && (d.flags & TF_TC)) run_moe_gemm_tc(c, d, ls, task, ok);
+  else run_moe_gemm<true>(c, d, ls, task, ok);
   return ls;
 }
 
@@ -3993,7 +4166,7 @@ __device__ void consumer_loop(const Ctx &c, int t_begin, int t_end) {
     if (HYB != HYB_F32 && type == TASK_LINEAR) ok = task_linear<GENERAL, TPX, HYB>(c, d, t, ok, tt, ls);
     else if (HYB == HYB_BF16 && type == TASK_MOE_GEMM) {
       ok = wait_dependencies(c, d, t, ok, tt);
-      ls = run_moe_gemm_hybrid(c, d, ls, t, ok);
+      ls = run_moe_gemm_hybrid<GENERAL>(c, d, ls, t, ok);
     } else if (GENERAL && !HYB && type == TASK_MOE_GEMM) {
       ok = wait_dependencies(c, d, t, ok, tt);
       run_moe_gemm<false>(c, d, ls, t, ok);

@@ -480,7 +480,12 @@ struct Builder {
         const int64_t K = T[l.t[1]].dim(2);
         need = std::max<int64_t>(need, (int64_t)linear_f32_tokens(K) * K * 4 + 256 - kPartialBytes);
       } else if (l.op == MPK_OP_MOE_W13_LINEAR || l.op == MPK_OP_MOE_W2_LINEAR) {
-        need = std::max(need, std::min<int64_t>((int64_t)ntok * (T[l.t[1]].dim(2) * 2 + kRowPadBytes), x_tile_cap()));
+        const int64_t K = T[l.t[1]].dim(2);
+        need = std::max(need, std::min<int64_t>((int64_t)ntok * (K * 2 + kRowPadBytes), x_tile_cap()));
+        if (g->hybrid && tc_linear(K)) {
+          g->use_tmem = true;
+          need = std::max<int64_t>(need, (int64_t)tc_np() * kTcKBlock * 2 * 4);   // four k blocks of all tokens' rows at least
+        }
       } else if (l.op == MPK_OP_MLA_DECODE) {
         need = std::max<int64_t>(need, 16 * (576 * 2 + 16) + 64 * (576 * 2 + 16) + 16 * (64 * 2 + 16) + 2 * 8 * 16 * 4);
       } else if (l.op == MPK_OP_MOE_TOPK_SIGMOID) {
@@ -965,6 +970,31 @@ struct Builder {
       if ((K / 128) % 4 == 0 && (((uint64_t)xs.ptr | (uint64_t)ws.ptr) & 15u) != 0)
         return fail(MPK_ERR_UNSUPPORTED, "expert projection: scale tensors must start on a 16-byte boundary: " + w.name);
     }
+    if (g->hybrid && g->use_tmem && tc_linear(K)) {
+      // tensor path: row tiles of the active experts, dealt out to one task per worker.  Tall tiles share one gather of the token
+      // rows; short ones spread better when few experts are active.
+      const int rb = N % 128 == 0 && (int64_t)std::min<int64_t>(E, (int64_t)cfg.max_num_batched_tokens * topk) * (N / 128) >= 4 * W ? 128 : N > 32 ? 64 : 32;
+      int nkb = std::max(1, std::min(K / kTcKBlock, g->stage_bytes / (rb * 128)));
+      while (K / kTcKBlock % nkb) --nkb;
+      if (E * (int64_t)N >= (1ll << 31)) return fail(MPK_ERR_UNSUPPORTED, "expert projection: more rows than a tensor map holds: " + w.name);
+      TmapSpec m;
+      m.base = (uint64_t)w.ptr; m.rows = (int64_t)EW * N; m.ld_bytes = (int64_t)K * 2; m.kblocks = K / kTcKBlock; m.box_rows = rb; m.box_kblocks = nkb;
+      if (ebase) return fail(MPK_ERR_UNSUPPORTED, "expert projection: hybrid graphs hold all experts: " + w.name);
+      const int map = (int)g->tmaps.size();
+      g->tmaps.push_back(m);
+      g->exec[ex].tc_rows = rb;
+      g->exec[ex].tc_kblocks = nkb;
+      for (int i = 0; i < W; ++i) {
+        TaskDesc d = blank(TASK_MOE_GEMM, li);
+        d.flags |= TF_STREAM_AFTER_DEP | TF_TC;
+        d.p[0] = (uint64_t)w.ptr; d.p[1] = (uint64_t)x.ptr; d.p[2] = (uint64_t)y.ptr; d.p[4] = (uint64_t)idx.ptr; d.p[5] = (uint64_t)mask.ptr;
+        d.a[L_N0] = i; d.a[L_N1] = W; d.a[L_K] = K; d.a[L_LDX] = (int)x.ld(); d.a[L_LDO] = (int)y.ld(); d.a[L_EPI] = epi; d.a[L_KT] = K;
+        d.a[L_KC] = nkb * kTcKBlock; d.a[L_ROWS] = rb; d.a[L_N] = N; d.a[L_TMAP] = map;
+        d.a[M_NEXP] = E; d.a[M_NTOPK] = topk; d.a[M_PER_SLOT] = w2 ? 1 : 0; d.a[M_LDR] = (int)idx.dim(1);
+        put((i + rot) % W, d, ex);
+      }
+      return MPK_OK;
+    }
     const int ntok = std::min(std::max(cfg.max_num_batched_tokens, 1), (int)kMaxLinearTokens);
     auto tile_bytes = [&](int KT) { return fp8 ? moe_fp8_tile_bytes(ntok, KT) : (int64_t)ntok * (KT * 2 + kRowPadBytes); };
     int nkt = 1;
@@ -1132,7 +1162,7 @@ struct Builder {
       p.keys = c.second;
       if (p.rt > 16 && rows <= 16) continue;
       if (nb_max <= 8 && p.keys > 16) continue;
-      const int64_t fixed = p.rt * pitch + (int64_t)(8 / (p.keys / 16)) * p.rt * (p.keys + 4) * 4 + 2 * p.rt * (p.keys * 2 + 16) + 8 * p.rt + kXaCells * 4;
+      const int64_t fixed = 16 + p.rt * pitch + (int64_t)(8 / (p.keys / 16)) * p.rt * (p.keys + 4) * 4 + 2 * p.rt * (p.keys * 2 + 16) + 8 * p.rt + kXaCells * 4;
       p.stages = (int)std::min<int64_t>(4, (budget - fixed) / (p.keys * pitch));
       if (p.stages < 2 && p.rt + p.keys == 32) p.stages = 2;   // the smallest tiles: whatever they need
       p.bytes = fixed + p.stages * p.keys * pitch;
