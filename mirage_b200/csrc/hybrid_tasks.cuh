@@ -46,11 +46,11 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 // Phase stamp i (0..3) of a task's profiler record.
-__device__ __forceinline__ void stamp(const Ctx &c, int task, int i) {
-  const KernelParams &P = c.P;
+__device__ __forceinline__ void stamp(const KernelParams &P, int task, int i) {
   if (threadIdx.x == 0 && P.profiler != nullptr && (uint64_t)(task + 1) * 8 <= P.profiler_entries)
     P.profiler[(size_t)task * 8 + 4 + i] = globaltimer_ns();
 }
+__device__ __forceinline__ void stamp(const Ctx &c, int task, int i) { stamp(c.P, task, i); }
 // Sum over the 256 compute threads (slots: 8 floats of shared memory; the caller keeps two calls apart with a barrier
 // or with different slots).
 __device__ __forceinline__ float block_sum(float v, float *slots) {
@@ -1213,7 +1213,7 @@ __device__ __noinline__ void ext_attention_mma(const Ctx c, const TaskDesc &d, c
 }
 
 // Shared key / value rows (latent attention: one kv head, the leading vdim columns of a key are its value), bf16 on mma.sync.  A
-// tile of MT x 16 query rows meets KEYS keys at a time, and every key row is brought to shared memory once for both products:
+// tile of 16 query rows meets KEYS keys at a time, and every key row is brought to shared memory once for both products:
 //   scores   the warps split the keys in groups of 16 and the row width KS ways; partial sums meet in shared memory
 //   softmax  a warp takes RT / 8 rows, online in base 2; weights go back as a bf16 value and a bf16 remainder, so that they
 //            keep 16 bits
@@ -1240,25 +1240,30 @@ __device__ __forceinline__ void sts_zero16(uint32_t a) { asm volatile("st.shared
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void *src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
 }
-template <int MT, int KEYS>
-__device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d, const SeqView sv, const AttnOut &ao, int k0, int k1,
-                                                  int row0, int nrow, int task) {
-  constexpr int RT = MT * 16, KW = KEYS / 16, KS = 8 / KW, SP = KEYS + 4, PP = KEYS * 2 + 16, NV = 8;
+// (its arguments too: what the calling convention puts on the stack is read back from there in the loop)
+struct LatentArgs {   // in shared memory
+  AttnOut ao;
+  int q0, pos0, kv0, k0, k1, row0, nrow, task;
+};
+template <int KEYS>
+__device__ __noinline__ void latent_attention_mma(const KernelParams &P, uint32_t sm, const TaskDesc &d, const LatentArgs &la) {
+  constexpr int RT = 16, KW = KEYS / 16, KS = 8 / KW, SP = KEYS + 4, PP = KEYS * 2 + 16, NV = 8;
   constexpr int RPW = RT * KEYS / 256;             // row sets a warp's lanes hold in the softmax (32 / KEYS rows at a time)
   // shared memory: partial scores [KS][RT][SP], weights [value, remainder][RT][PP], rescale factors [RT] (at the end m and l [2][RT]),
   // cache row of every eighth key [kXaCells], queries [RT][pitch], ring of key tiles [stages][KEYS][pitch]
   constexpr uint32_t oP = KS * RT * SP * 4, oC = oP + 2 * RT * PP, oCell = oC + 8 * RT, oQ = (oCell + kXaCells * 4 + 15) & ~15u;
-  const uint32_t sm = smem_u32(c.s.xtile);
+  const AttnOut &ao = la.ao;
+  const int k0 = la.k0, row0 = la.row0, nrow = la.nrow;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int pieces = d.a[XA_DIMP] >> 3, ksteps = (pieces + 7) / 8 * 4;   // 16-byte pieces of a cache row, 16-column steps of a padded one
   const uint32_t pitch = ksteps * 32 + 16, tile = KEYS * pitch, ring = sm + oQ + RT * pitch;
   const int nstg = d.a[XA_STAGES];
-  const int kend = min(k1, sv.pos0 + (row0 + nrow - 1) / ao.G + 1);
+  const int kend = min(la.k1, la.pos0 + (row0 + nrow - 1) / ao.G + 1);
   const int ntiles = kend > k0 ? (kend - k0 + KEYS - 1) / KEYS : 0;
   const uint4 *kg = reinterpret_cast<const uint4 *>(d.p[1]);
   const int page = d.a[XA_PAGE];
-  const bool table = (page & 7) == 0 && k1 - k0 <= 8 * kXaCells;   // eight consecutive keys lie in one page
-  const int32_t *pages = c.P.meta.paged_kv_indices + sv.kv0;
+  const bool table = (page & 7) == 0 && la.k1 - k0 <= 8 * kXaCells;   // eight consecutive keys lie in one page
+  const int32_t *pages = P.meta.paged_kv_indices + la.kv0;
   auto cell_row = [&](int key) { return __ldcg(pages + key / page) * page + key % page; };
   if (table)
     for (int i = tid; i < (kend - k0 + 7) >> 3; i += kConsumerThreads)
@@ -1268,7 +1273,7 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
     const int G = ao.G, ldq = d.a[XA_LDQ] >> 3;
     for (int r = warp; r < RT; r += 8) {
       const uint32_t dst = sm + oQ + r * pitch;
-      const uint4 *src = qg + (size_t)(sv.q0 + (row0 + r) / G) * ldq + (size_t)((row0 + r) % G) * pieces;
+      const uint4 *src = qg + (size_t)(la.q0 + (row0 + r) / G) * ldq + (size_t)((row0 + r) % G) * pieces;
       for (int p = lane; p < ksteps * 2; p += 32) {
         if (r < nrow && p < pieces) cp_async16(dst + p * 16, src + p);
         else sts_zero16(dst + p * 16);
@@ -1279,7 +1284,7 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
         for (int p = pieces + lane; p < ksteps * 2; p += 32) sts_zero16(ring + r * pitch + p * 16);
   }
   consumer_sync();   // (the table of cache rows)
-  stamp(c, task, 0);
+  stamp(P, la.task, 0);
   auto issue = [&](int it, int stg) {
     if (it < ntiles) {
 #pragma unroll
@@ -1307,15 +1312,13 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
   for (int i = 0; i < RPW; ++i) {
     m_run[i] = -INFINITY;
     l_run[i] = 0.f;
-    seen[i] = min(kend - 1, sv.pos0 + (row0 + srow + i * (32 / KEYS)) / ao.G) - skey - k0;   // relative to the tile's first key
+    seen[i] = min(kend - 1, la.pos0 + (row0 + srow + i * (32 / KEYS)) / ao.G) - skey - k0;   // relative to the tile's first key
   }
-  float o[MT][NV][4];
+  float o[NV][4];
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+  for (int i = 0; i < NV; ++i)
 #pragma unroll
-    for (int i = 0; i < NV; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) o[m][i][e] = 0.f;
+    for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
   int stg = 0;
 #pragma unroll 1
   for (int it = 0; it < ntiles; ++it) {
@@ -1323,41 +1326,29 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
     else if (nstg == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
     else asm volatile("cp.async.wait_group 0;" ::: "memory");
     consumer_sync();   // the tile has landed for everyone, and everyone is done with the stage refilled next
-    if (it == 0) stamp(c, task, 1);
+    if (it == 0) stamp(P, la.task, 1);
     issue(it + nstg - 1, stg == 0 ? nstg - 1 : stg - 1);
     const uint32_t kt = ring + stg * tile;
     if (++stg == nstg) stg = 0;
     {   // ---- scores
       const int kw = warp % KW, ks = warp / KW;
-      float s[MT][2][4];
-#pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int n = 0; n < 2; ++n)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) s[m][n][e] = 0.f;
+      float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
       const uint32_t ka = kt + (uint32_t)((kw * 16 + (lane & 7) + (lane >> 4) * 8) * pitch + ((lane >> 3) & 1) * 16);
       const uint32_t qa = sm + oQ + (uint32_t)((lane & 15) * pitch + (lane >> 4) * 16);
 #pragma unroll 2
       for (int kk = ks; kk < ksteps; kk += KS) {
-        uint32_t b[4];
+        uint32_t a[4], b[4];
         ldmatrix_x4(b, ka + kk * 32u);
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          uint32_t a[4];
-          ldmatrix_x4(a, qa + (uint32_t)(m * 16) * pitch + kk * 32u);
-          mma_bf16_16816(s[m][0], a, b[0], b[1]);
-          mma_bf16_16816(s[m][1], a, b[2], b[3]);
-        }
+        ldmatrix_x4(a, qa + kk * 32u);
+        mma_bf16_16816(s[0], a, b[0], b[1]);
+        mma_bf16_16816(s[1], a, b[2], b[3]);
       }
       const uint32_t sr = sm + (uint32_t)(((ks * RT + (lane >> 2)) * SP + kw * 16 + 2 * (lane & 3)) * 4);
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          sts_f32x2(sr + (m * 16 * SP + n * 8) * 4, s[m][n][0], s[m][n][1]);
-          sts_f32x2(sr + ((m * 16 + 8) * SP + n * 8) * 4, s[m][n][2], s[m][n][3]);
-        }
+      for (int n = 0; n < 2; ++n) {
+        sts_f32x2(sr + n * 32, s[n][0], s[n][1]);
+        sts_f32x2(sr + (8 * SP + n * 8) * 4, s[n][2], s[n][3]);
+      }
     }
     consumer_sync();
     {   // ---- softmax
@@ -1386,33 +1377,21 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
     }
     consumer_sync();
     {   // ---- output
-      bool keep = true;
-      float cr[MT][2];
+      const float c0 = lds_f32(sm + oC + (lane >> 2) * 4), c1 = lds_f32(sm + oC + (8 + (lane >> 2)) * 4);
+      if (__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) {
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          cr[m][h] = lds_f32(sm + oC + (m * 16 + h * 8 + (lane >> 2)) * 4);
-          keep = keep && cr[m][h] == 1.f;
+        for (int i = 0; i < NV; ++i) {
+          o[i][0] *= c0; o[i][1] *= c0;
+          o[i][2] *= c1; o[i][3] *= c1;
         }
-      if (!__all_sync(0xffffffffu, keep)) {
-#pragma unroll
-        for (int m = 0; m < MT; ++m)
-#pragma unroll
-          for (int i = 0; i < NV; ++i) {
-            o[m][i][0] *= cr[m][0]; o[m][i][1] *= cr[m][0];
-            o[m][i][2] *= cr[m][1]; o[m][i][3] *= cr[m][1];
-          }
       }
       // 16 keys and two column tiles at a time (one past the last is read, not used)
       const uint32_t pa = sm + oP + (uint32_t)((lane & 15) * PP + (lane >> 4) * 16);
 #pragma unroll
       for (int k = 0; k < KW; ++k) {
-        uint32_t p[2][MT][4];
+        uint32_t p[2][4];
 #pragma unroll
-        for (int h = 0; h < 2; ++h)
-#pragma unroll
-          for (int m = 0; m < MT; ++m) ldmatrix_x4(p[h][m], pa + (uint32_t)((h * RT + m * 16) * PP + k * 32));
+        for (int h = 0; h < 2; ++h) ldmatrix_x4(p[h], pa + (uint32_t)(h * RT * PP + k * 32));
         const uint32_t va = kt + (uint32_t)(k * 16 + (lane & 15)) * pitch + warp * 16 + (lane >> 4) * 128u;
 #pragma unroll
         for (int i = 0; i < NV; i += 2) {
@@ -1420,18 +1399,16 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
           uint32_t b[4];
           ldmatrix_x4_trans(b, va + i * 128u);
 #pragma unroll
-          for (int m = 0; m < MT; ++m)
-#pragma unroll
-            for (int h = 0; h < 2; ++h) {
-              mma_bf16_16816(o[m][i], p[h][m], b[0], b[1]);
-              if (i + 1 < nv) mma_bf16_16816(o[m][i + 1], p[h][m], b[2], b[3]);
-            }
+          for (int h = 0; h < 2; ++h) {
+            mma_bf16_16816(o[i], p[h], b[0], b[1]);
+            if (i + 1 < nv) mma_bf16_16816(o[i + 1], p[h], b[2], b[3]);
+          }
         }
       }
     }
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
-  stamp(c, task, 2);
+  stamp(P, la.task, 2);
   // running maximum and sum of every row
   consumer_sync();
 #pragma unroll
@@ -1446,35 +1423,33 @@ __device__ __noinline__ void latent_attention_mma(const Ctx c, const TaskDesc &d
   }
   consumer_sync();
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+  for (int h = 0; h < 2; ++h) {
+    const int r = h * 8 + (lane >> 2), row = row0 + r;
+    if (r >= nrow) continue;
+    const float mx = lds_f32(sm + oC + r * 4), l = lds_f32(sm + oC + (RT + r) * 4);
+    const int col0 = warp * 8 + 2 * (lane & 3);
+    if (ao.n_act == 1) {
+      const int hq_idx = row % ao.G;
+      const float sk = ao.sink ? sink_logit<HYB_BF16>(d, hq_idx) : 0.f;
+      const float M = ao.sink ? fmaxf(mx, sk) : mx;
+      const float w = mx == -INFINITY ? 0.f : exp2f(mx - M);
+      const float L = l * w + (ao.sink ? exp2f(sk - M) : 0.f);
+      const float f = L > 0.f ? w / L * ao.oscale : 0.f;
+      __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(d.p[3]) + (size_t)(la.q0 + row / ao.G) * ao.ldo + ao.ocol + (size_t)hq_idx * ao.vdim + col0;
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const int r = m * 16 + h * 8 + (lane >> 2), row = row0 + r;
-      if (r >= nrow) continue;
-      const float mx = lds_f32(sm + oC + r * 4), l = lds_f32(sm + oC + (RT + r) * 4);
-      const int col0 = warp * 8 + 2 * (lane & 3);
-      if (ao.n_act == 1) {
-        const int hq_idx = row % ao.G;
-        const float sk = ao.sink ? sink_logit<HYB_BF16>(d, hq_idx) : 0.f;
-        const float M = ao.sink ? fmaxf(mx, sk) : mx;
-        const float w = mx == -INFINITY ? 0.f : exp2f(mx - M);
-        const float L = l * w + (ao.sink ? exp2f(sk - M) : 0.f);
-        const float f = L > 0.f ? w / L * ao.oscale : 0.f;
-        __nv_bfloat16 *out = reinterpret_cast<__nv_bfloat16 *>(d.p[3]) + (size_t)(sv.q0 + row / ao.G) * ao.ldo + ao.ocol + (size_t)hq_idx * ao.vdim + col0;
-#pragma unroll
-        for (int i = 0; i < NV; ++i)
-          if (i < nv) *reinterpret_cast<uint32_t *>(out + i * 64) = pack_bf16(o[m][i][2 * h] * f, o[m][i][2 * h + 1] * f);
-      } else {
-        float *rec = attn_record(c.P, ao, row);
-        if (warp == 0 && (lane & 3) == 0) {
-          __stcg(rec, mx);
-          __stcg(rec + 1, l);
-        }
-#pragma unroll
-        for (int i = 0; i < NV; ++i)
-          if (i < nv) __stcg(reinterpret_cast<float2 *>(rec + kXaRecHead + col0 + i * 64), make_float2(o[m][i][2 * h], o[m][i][2 * h + 1]));
+      for (int i = 0; i < NV; ++i)
+        if (i < nv) *reinterpret_cast<uint32_t *>(out + i * 64) = pack_bf16(o[i][2 * h] * f, o[i][2 * h + 1] * f);
+    } else {
+      float *rec = attn_record(P, ao, row);
+      if (warp == 0 && (lane & 3) == 0) {
+        __stcg(rec, mx);
+        __stcg(rec + 1, l);
       }
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (i < nv) __stcg(reinterpret_cast<float2 *>(rec + kXaRecHead + col0 + i * 64), make_float2(o[i][2 * h], o[i][2 * h + 1]));
     }
+  }
 }
 
 // 32-bit: one warp per row, 32 keys at a time (a lane per key for the scores, a lane per output column for PV)
@@ -1546,7 +1521,8 @@ __device__ __forceinline__ void run_ext_attention(const Ctx &c, const TaskDesc &
   // shared by the block, in shared memory: in registers it would be live through the key loops (every thread writes the
   // same values, and the previous task is done with it)
   AttnOut &ao = *reinterpret_cast<AttnOut *>(c.s.red);
-  const int RT = d.a[XA_SHARED] ? d.a[XA_SHARED] : 16, NC = d.a[XA_NCHUNK];
+  constexpr int RT = 16;
+  const int NC = d.a[XA_NCHUNK];
   ao.hq = d.a[XA_HQ];
   ao.G = ao.hq / d.a[XA_HKV];
   ao.head = d.a[XA_HEAD];
@@ -1569,16 +1545,12 @@ __device__ __forceinline__ void run_ext_attention(const Ctx &c, const TaskDesc &
   if (HYB == HYB_F32) {
     ext_attention_f32(c, d, sv, ao, k0, k1, row0, row1);
   } else if (d.a[XA_SHARED]) {
-    for (int r = row0; r < row1; r += RT) {
-      const int n = min(RT, row1 - r);
+    LatentArgs &la = *reinterpret_cast<LatentArgs *>(c.s.red);   // (begins with `ao`)
+    for (int r = row0; r < row1; r += 16) {
       if (r > row0) consumer_sync();
-      if (d.a[XA_KEYS] == 32) {
-        if (n <= 16) latent_attention_mma<1, 32>(c, d, sv, ao, k0, k1, r, n, task);
-        else latent_attention_mma<2, 32>(c, d, sv, ao, k0, k1, r, n, task);
-      } else {
-        if (n <= 16) latent_attention_mma<1, 16>(c, d, sv, ao, k0, k1, r, n, task);
-        else latent_attention_mma<2, 16>(c, d, sv, ao, k0, k1, r, n, task);
-      }
+      la.q0 = sv.q0; la.pos0 = sv.pos0; la.kv0 = sv.kv0; la.k0 = k0; la.k1 = k1; la.row0 = r; la.nrow = min(16, row1 - r); la.task = task;
+      if (d.a[XA_KEYS] == 32) latent_attention_mma<32>(c.P, smem_u32(c.s.xtile), d, la);
+      else latent_attention_mma<16>(c.P, smem_u32(c.s.xtile), d, la);
     }
   } else {
     const int w = max(d.a[XA_DIMP], d.a[XA_VDIMP]);
@@ -1609,7 +1581,7 @@ __device__ __noinline__ void run_attn_merge(const Ctx c, const TaskDesc &d) {
   const KernelParams &P = c.P;
   const int B = active_tokens(P), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int hq = d.a[XA_HQ], hkv = d.a[XA_HKV], G = hq / hkv, vdim = d.a[XA_VDIM], srec = d.a[XA_SREC], NC = d.a[XA_NCHUNK];
-  const int RT = d.a[XA_SHARED] ? d.a[XA_SHARED] : 16, cols = (vdim + 127) >> 7;
+  const int RT = 16, cols = (vdim + 127) >> 7;
   for (int item = d.a[XA_SLOT] * 8 + warp; item < B * hq * cols; item += d.a[XA_CHUNK] * 8) {
     const int row = item / cols, j = (item - row * cols) * 128 + lane * 4, t = row / hq, h = row - t * hq;
     const int k = request_of(P, t);

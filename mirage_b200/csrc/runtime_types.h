@@ -229,7 +229,7 @@ enum { QA_T0 = 0, QA_T1, QA_LDP, QA_QOFF, QA_KOFF, QA_VOFF, QA_HQ, QA_HKV, QA_DI
 // ---- TASK_EXT_ATTENTION: p[0] q [tokens, hq * dimp]  p[1] k cache  p[2] v cache  p[3] out;  a[XA_*] below
 enum { XA_SLOT = 0, XA_HEAD, XA_CHUNK, XA_NCHUNK, XA_HQ, XA_HKV, XA_DIMP, XA_VDIM, XA_VDIMP, XA_PAGE, XA_LDQ, XA_LDO, XA_OCOL,
        XA_SCALE, XA_CAP, XA_SINK, XA_OSCALE, XA_TICKET, XA_SREC, XA_STAGES, XA_SHARED, XA_KEYS, XA_MERGE };
-//      p[4] sinks bf16 [hq] or null; XA_SHARED: values are key columns, rows of a query tile (0: separate values); XA_KEYS: keys of a tile of
+//      p[4] sinks bf16 [hq] or null; XA_SHARED: values are key columns; XA_KEYS: keys of a tile of
 //      theirs; XA_MERGE: a layer of TASK_ATTN_MERGE follows (its tasks: the same fields, task a[XA_SLOT] of a[XA_CHUNK])
 constexpr int kXaRecHead = 4;   // floats in front of a record's columns
 constexpr int kXaCells = 320;   // cache rows of a chunk's key octets kept in shared memory

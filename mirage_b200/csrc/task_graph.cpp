@@ -1151,22 +1151,18 @@ struct Builder {
   int xattn_stages() const { return nb_max > 8 ? 3 : 2; }
   // Tiles of attention over shared key / value rows: the largest that leave the weight ring its size (graphs of many tokens
   // reserve a large activation tile anyway; of few tokens what a ring of 32 KB stages leaves over).
-  struct LatentPlan { int rt, keys, stages; int64_t bytes; };
+  struct LatentPlan { int keys, stages; int64_t bytes; };
   LatentPlan latent_plan(const LayerInfo &l) const {
     const int64_t pitch = round_up(T[l.t[1]].dim(3), 64) * 2 + 16;
-    const int64_t rows = (int64_t)cfg.max_num_batched_tokens * l.params[0];
     const int64_t budget = kPartialBytes + (nb_max > 8 ? 64 * (1024 * 2 + kRowPadBytes) : 90 * 1024);
-    LatentPlan p{0, 0, 0, 0};
-    for (const auto &c : {std::pair<int, int>{32, 32}, {16, 32}, {32, 16}, {16, 16}}) {
-      p.rt = c.first;
-      p.keys = c.second;
-      if (p.rt > 16 && rows <= 16) continue;
-      if (nb_max <= 8 && p.keys > 16) continue;
-      const int64_t fixed = 16 + p.rt * pitch + (int64_t)(8 / (p.keys / 16)) * p.rt * (p.keys + 4) * 4 + 2 * p.rt * (p.keys * 2 + 16) + 8 * p.rt + kXaCells * 4;
-      p.stages = (int)std::min<int64_t>(4, (budget - fixed) / (p.keys * pitch));
-      if (p.stages < 2 && p.rt + p.keys == 32) p.stages = 2;   // the smallest tiles: whatever they need
-      p.bytes = fixed + p.stages * p.keys * pitch;
-      if (p.stages >= 2) return p;
+    LatentPlan p{0, 0, 0};
+    for (int keys : {32, 16}) {
+      const int64_t fixed = 32 + 16 * pitch + (int64_t)(8 / (keys / 16)) * 16 * (keys + 4) * 4 + 2 * 16 * (keys * 2 + 16) + 8 * 16 + kXaCells * 4;
+      p.keys = keys;
+      p.stages = (int)std::min<int64_t>(4, (budget - fixed) / (keys * pitch));
+      if (p.stages < 2 && keys == 16) p.stages = 2;   // the smallest tiles: whatever they need
+      p.bytes = fixed + p.stages * keys * pitch;
+      if (p.stages >= (keys == 32 ? 3 : 2)) return p;
     }
     return p;
   }
@@ -1512,10 +1508,10 @@ struct Builder {
     // chunks of a (request, kv head): enough to occupy the workers, at most ~2048 keys each, at least 64
     int NC = std::max(std::max(1, W / std::max(slots * hkv, 1)), (max_seq + 2047) / 2048);
     NC = std::min(std::min(NC, std::max(1, max_seq / 64)), 32);
-    LatentPlan lp{16, 0, xattn_stages(), 0};
+    LatentPlan lp{0, xattn_stages(), 0};
     if (shared && bf16) {   // row tiles of a prompt portion times key chunks of a decoded token
       lp = latent_plan(l);
-      const int64_t tiles = ((int64_t)cfg.max_num_batched_tokens * hq + lp.rt - 1) / lp.rt;
+      const int64_t tiles = ((int64_t)cfg.max_num_batched_tokens * hq + 15) / 16;
       NC = (int)std::min<int64_t>(std::max(1, W / slots), tiles * std::max(1, (max_seq + 63) / 64));
     }
     const int srec = round_up(vdim, 4) + kXaRecHead;
@@ -1525,7 +1521,7 @@ struct Builder {
           TaskDesc d = blank(TASK_EXT_ATTENTION, li);
           for (int i = 0; i < 4; ++i) d.p[i] = (uint64_t)T[l.t[i]].ptr;
           d.p[4] = sinks >= 0 ? (uint64_t)T[sinks].ptr : 0;
-          d.a[XA_SHARED] = shared && bf16 ? lp.rt : 0; d.a[XA_KEYS] = lp.keys; d.a[XA_MERGE] = merge ? 1 : 0;
+          d.a[XA_SHARED] = shared && bf16 ? 1 : 0; d.a[XA_KEYS] = lp.keys; d.a[XA_MERGE] = merge ? 1 : 0;
           d.a[XA_SLOT] = s; d.a[XA_HEAD] = h; d.a[XA_CHUNK] = ch; d.a[XA_NCHUNK] = NC; d.a[XA_HQ] = hq; d.a[XA_HKV] = hkv;
           d.a[XA_DIMP] = (int)kc.dim(3); d.a[XA_VDIM] = vdim; d.a[XA_VDIMP] = (int)vc.dim(3); d.a[XA_PAGE] = cfg.page_size;
           d.a[XA_LDQ] = (int)q.ld(); d.a[XA_LDO] = (int)o.ld(); d.a[XA_OCOL] = ocol;
@@ -1539,7 +1535,7 @@ struct Builder {
         }
     hybrid_tickets += slots * hkv * NC;
     // a (request, kv head) has at most one query tile's rows for each of its tasks in the scratch
-    g->attn_scratch_floats = std::max<int64_t>(g->attn_scratch_floats, (int64_t)slots * hkv * NC * lp.rt * srec);
+    g->attn_scratch_floats = std::max<int64_t>(g->attn_scratch_floats, (int64_t)slots * hkv * NC * 16 * srec);
     return MPK_OK;
   }
 
