@@ -511,6 +511,24 @@ static __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d
   }
 }
 
+// Copies B rows of `vecs` 16-byte vectors into the activation tile, one warp per row, every copy in flight.  A function of its own:
+// at the register cap of the linear bodies its loop would reload spilled variables for each copy.
+template <int MODE>
+__device__ __noinline__ void stage_rows(uint32_t xs, const uint4 *src, int ld, int B, int vecs, int xstride, int np) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int b = warp; b < B; b += 8) {
+    const uint4 *row = src + (size_t)b * ld;
+    const uint32_t dst = MODE == 2 ? xs + b * 128 + (((lane & 7) ^ (b & 7)) << 4) : xs + b * xstride + lane * 16;
+#pragma unroll 4
+    for (int v = lane; v < vecs; v += 32)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + (MODE == 2 ? (uint32_t)((v >> 3) * np * 128) : (uint32_t)(v - lane) * 16u)),
+                   "l"(row + v)
+                   : "memory");
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+}
+
 template <int MODE, bool TPX = false>
 __device__ void stage_x(const Ctx &c, const TaskDesc &d, int B, int k0, int KT, const uint4 (&gpre)[2]) {
   constexpr bool WIDE = MODE != 0;
@@ -654,13 +672,7 @@ __device__ void stage_x(const Ctx &c, const TaskDesc &d, int B, int k0, int KT, 
   }
   if (WIDE && (pro == PRO_PLAIN || pro == PRO_RMSNORM)) {
     // many tokens: asynchronous 16-byte copies straight into shared memory (all in flight, no registers held)
-    for (int b = 0; b < B; ++b)
-      for (int v = tid; v < vec_per_row; v += kConsumerThreads)
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(x_vec<MODE>(xs, b, v, xstride, np))),
-                     "l"(reinterpret_cast<const uint4 *>(src + (size_t)b * ldx + k0) + v)
-                     : "memory");
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    stage_rows<MODE>(smem_u32(xs), reinterpret_cast<const uint4 *>(src + k0), ldx >> 3, B, vec_per_row, xstride, np);
     consumer_sync();
     if (pro == PRO_PLAIN) return;
     // RMSNorm in place.  Pass 1: one warp per token sums the squares and leaves 1 / rms in shared memory.  Pass 2:
