@@ -19,6 +19,8 @@
 // allocation, and every variant added makes the linear loop and the others spill.  They take the context by value: a
 // reference would keep it in local memory for the whole kernel.
 #pragma once
+#include <stddef.h>
+
 #include "megakernel.cuh"
 
 namespace mpk {
@@ -1217,18 +1219,18 @@ __device__ __noinline__ void ext_attention_mma(const Ctx c, const TaskDesc &d, c
 //   scores   the warps split the keys in groups of 16 and the row width KS ways; partial sums meet in shared memory
 //   softmax  a warp takes RT / 8 rows, online in base 2; weights go back as a bf16 value and a bf16 remainder, so that they
 //            keep 16 bits
-//   output   every warp owns eight-column tiles w, w + 8, ... of all rows
+//   output   every warp owns eight-column tiles w, w + 8, ... of all rows; a tile's output is formed beside the next one's scores
 //
 // (with a few KB of L1 beside the shared memory a spilled variable of the key loop costs an L2 round trip: areas of fixed size
 // come first, so that their addresses are one base plus constants, and everything is addressed in 32 bits)
 __device__ __forceinline__ float lds_f32(uint32_t a) {
   float v;
-  asm volatile("ld.shared.f32 %0, [%1];" : "=f"(v) : "r"(a));
+  asm volatile("ld.shared.f32 %0, [%1];" : "=f"(v) : "r"(a) : "memory");
   return v;
 }
 __device__ __forceinline__ int lds_s32(uint32_t a) {
   int v;
-  asm volatile("ld.shared.s32 %0, [%1];" : "=r"(v) : "r"(a));
+  asm volatile("ld.shared.s32 %0, [%1];" : "=r"(v) : "r"(a) : "memory");
   return v;
 }
 __device__ __forceinline__ void sts_f32(uint32_t a, float v) { asm volatile("st.shared.f32 [%0], %1;" ::"r"(a), "f"(v) : "memory"); }
@@ -1240,11 +1242,33 @@ __device__ __forceinline__ void sts_zero16(uint32_t a) { asm volatile("st.shared
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void *src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
 }
-// (its arguments too: what the calling convention puts on the stack is read back from there in the loop)
-struct LatentArgs {   // in shared memory
+// (the arguments and the loop's constants too: they stay in shared memory and are read where they are used)
+struct alignas(16) LatentArgs {
   AttnOut ao;
-  int q0, pos0, kv0, k0, k1, row0, nrow, task;
+  alignas(16) int keys;           // keys of the chunk the rows see
+  int pieces, table, ntiles;      // 16-byte pieces of a cache row, the table of cache rows is used, key tiles
+  const uint4 *rows;              // this layer's cache
+  const int32_t *pages;           // the request's pages
+  float scale, cap;
+  int page, k0;
+  int q0, pos0, row0, nrow, task, stages;
 };
+constexpr uint32_t kLatentHot = offsetof(LatentArgs, keys);
+static_assert(offsetof(LatentArgs, rows) == kLatentHot + 16, "read as one vector and one pointer");
+static_assert(sizeof(LatentArgs) <= 256, "the reduction slots hold 64 words");
+__device__ __forceinline__ int4 lds_v4(uint32_t a) {
+  int4 v;
+  asm volatile("ld.shared.v4.s32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "r"(a) : "memory");
+  return v;
+}
+__device__ __forceinline__ uint64_t lds_u64(uint32_t a) {
+  uint64_t v;
+  asm volatile("ld.shared.u64 %0, [%1];" : "=l"(v) : "r"(a) : "memory");
+  return v;
+}
+// Cache row of a key, where the table does not hold it (page sizes that are no multiple of eight, very long chunks).
+static __device__ __noinline__ int latent_cell(const int32_t *pages, int page, int key) { return __ldcg(pages + key / page) * page + key % page; }
+
 template <int KEYS>
 __device__ __noinline__ void latent_attention_mma(const KernelParams &P, uint32_t sm, const TaskDesc &d, const LatentArgs &la) {
   constexpr int RT = 16, KW = KEYS / 16, KS = 8 / KW, SP = KEYS + 4, PP = KEYS * 2 + 16, NV = 8;
@@ -1252,58 +1276,55 @@ __device__ __noinline__ void latent_attention_mma(const KernelParams &P, uint32_
   // shared memory: partial scores [KS][RT][SP], weights [value, remainder][RT][PP], rescale factors [RT] (at the end m and l [2][RT]),
   // cache row of every eighth key [kXaCells], queries [RT][pitch], ring of key tiles [stages][KEYS][pitch]
   constexpr uint32_t oP = KS * RT * SP * 4, oC = oP + 2 * RT * PP, oCell = oC + 8 * RT, oQ = (oCell + kXaCells * 4 + 15) & ~15u;
-  const AttnOut &ao = la.ao;
-  const int k0 = la.k0, row0 = la.row0, nrow = la.nrow;
+  const uint32_t args = smem_u32(&la);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int pieces = d.a[XA_DIMP] >> 3, ksteps = (pieces + 7) / 8 * 4;   // 16-byte pieces of a cache row, 16-column steps of a padded one
-  const uint32_t pitch = ksteps * 32 + 16, tile = KEYS * pitch, ring = sm + oQ + RT * pitch;
-  const int nstg = d.a[XA_STAGES];
-  const int kend = min(la.k1, la.pos0 + (row0 + nrow - 1) / ao.G + 1);
-  const int ntiles = kend > k0 ? (kend - k0 + KEYS - 1) / KEYS : 0;
-  const uint4 *kg = reinterpret_cast<const uint4 *>(d.p[1]);
-  const int page = d.a[XA_PAGE];
-  const bool table = (page & 7) == 0 && la.k1 - k0 <= 8 * kXaCells;   // eight consecutive keys lie in one page
-  const int32_t *pages = P.meta.paged_kv_indices + la.kv0;
-  auto cell_row = [&](int key) { return __ldcg(pages + key / page) * page + key % page; };
-  if (table)
-    for (int i = tid; i < (kend - k0 + 7) >> 3; i += kConsumerThreads)
-      asm volatile("st.shared.s32 [%0], %1;" ::"r"(sm + oCell + i * 4), "r"(cell_row(k0 + 8 * i)) : "memory");
-  {   // queries, and zeros where no copy reaches
+  const uint32_t pitch = ((la.pieces + 7) & ~7) * 16 + 16;   // rows padded to whole 64-column blocks
+  const uint32_t ring = sm + oQ + RT * pitch;
+  {
+    const int row0 = la.row0, nrow = la.nrow, pieces = la.pieces, padded = (pieces + 7) & ~7;
+    if (la.table)
+      for (int i = tid; i < (la.keys + 7) >> 3; i += kConsumerThreads)
+        asm volatile("st.shared.s32 [%0], %1;" ::"r"(sm + oCell + i * 4), "r"(latent_cell(la.pages, la.page, la.k0 + 8 * i)) : "memory");
+    // queries, and zeros where no copy reaches
     const uint4 *qg = reinterpret_cast<const uint4 *>(d.p[0]);
-    const int G = ao.G, ldq = d.a[XA_LDQ] >> 3;
+    const int G = la.ao.G, ldq = d.a[XA_LDQ] >> 3;
     for (int r = warp; r < RT; r += 8) {
       const uint32_t dst = sm + oQ + r * pitch;
       const uint4 *src = qg + (size_t)(la.q0 + (row0 + r) / G) * ldq + (size_t)((row0 + r) % G) * pieces;
-      for (int p = lane; p < ksteps * 2; p += 32) {
+      for (int p = lane; p < padded; p += 32) {
         if (r < nrow && p < pieces) cp_async16(dst + p * 16, src + p);
         else sts_zero16(dst + p * 16);
       }
     }
-    if (pieces < ksteps * 2)
-      for (int r = warp; r < nstg * KEYS; r += 8)
-        for (int p = pieces + lane; p < ksteps * 2; p += 32) sts_zero16(ring + r * pitch + p * 16);
+    if (pieces < padded)
+      for (int r = warp; r < la.stages * KEYS; r += 8)
+        for (int p = pieces + lane; p < padded; p += 32) sts_zero16(ring + r * pitch + p * 16);
   }
   consumer_sync();   // (the table of cache rows)
   stamp(P, la.task, 0);
-  auto issue = [&](int it, int stg) {
-    if (it < ntiles) {
+  auto issue = [&](int it, uint32_t dst) {
+    const int4 h = lds_v4(args + kLatentHot);   // keys, pieces, table, tiles
+    if (it < h.w) {
+      const uint4 *rows = reinterpret_cast<const uint4 *>(lds_u64(args + kLatentHot + 16)) + lane;
+      dst += warp * pitch + lane * 16;
 #pragma unroll
-      for (int r = 0; r < KEYS / 8; ++r) {
-        const int kk = it * KEYS + warp + 8 * r;   // key relative to the chunk
-        const uint32_t dst = ring + stg * tile + (warp + 8 * r) * pitch;
-        if (k0 + kk < kend) {
-          const uint4 *src = kg + (size_t)(table ? lds_s32(sm + oCell + (kk >> 3) * 4) + (kk & 7) : cell_row(k0 + kk)) * pieces;
-          for (int p = lane; p < pieces; p += 32) cp_async16(dst + p * 16, src + p);
+      for (int r = 0; r < KEYS / 8; ++r, dst += 8 * pitch) {
+        const int key = it * KEYS + warp + 8 * r;   // of the chunk
+        if (key < h.x) {
+          int cell;
+          if (h.z) cell = lds_s32(sm + oCell + (key >> 3) * 4) + (key & 7);
+          else cell = latent_cell(la.pages, la.page, la.k0 + key);
+          const uint4 *src = rows + (size_t)cell * h.y;
+          for (int p = lane; p < h.y; p += 32) cp_async16(dst + (p - lane) * 16, src + (p - lane));
         } else {   // a masked key has weight 0, and 0 x NaN would be NaN
-          for (int p = lane; p < pieces; p += 32) sts_zero16(dst + p * 16);
+          for (int p = lane; p < h.y; p += 32) sts_zero16(dst + (p - lane) * 16);
         }
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  for (int i = 0; i < nstg - 1; ++i) issue(i, i);   // (the queries join the first group)
-  const float scale = __int_as_float(d.a[XA_SCALE]), cap = __int_as_float(d.a[XA_CAP]);
-  const int nv = (ao.vdim >> 3) > warp ? ((ao.vdim >> 3) - warp + 7) >> 3 : 0;   // this warp's column tiles
+  for (int i = 0; i < la.stages - 2; ++i) issue(i, ring + i * KEYS * pitch);   // (the queries join the first group)
+  const int nv = (la.ao.vdim >> 3) > warp ? ((la.ao.vdim >> 3) - warp + 7) >> 3 : 0;   // this warp's column tiles
   // softmax: this lane's key of the tile, its first row and the last keys that row set sees
   const int skey = lane % KEYS, srow = warp * (RT / 8) + lane / KEYS;
   int seen[RPW];
@@ -1312,37 +1333,78 @@ __device__ __noinline__ void latent_attention_mma(const KernelParams &P, uint32_
   for (int i = 0; i < RPW; ++i) {
     m_run[i] = -INFINITY;
     l_run[i] = 0.f;
-    seen[i] = min(kend - 1, la.pos0 + (row0 + srow + i * (32 / KEYS)) / ao.G) - skey - k0;   // relative to the tile's first key
+    seen[i] = min(la.keys - 1, la.pos0 + (la.row0 + srow + i * (32 / KEYS)) / la.ao.G - la.k0) - skey;   // relative to the tile's first key
   }
   float o[NV][4];
 #pragma unroll
   for (int i = 0; i < NV; ++i)
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
-  int stg = 0;
+  // Trip `it`: scores of tile `it` and, in between, output of tile `it - 1`, whose weights the softmax left behind
+  uint32_t slot = 0, before = ring;   // ring slot of tile `it`, address of tile `it - 1`
 #pragma unroll 1
-  for (int it = 0; it < ntiles; ++it) {
-    if (nstg >= 4) asm volatile("cp.async.wait_group 2;" ::: "memory");
-    else if (nstg == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
+  for (int it = 0;; ++it) {
+    const uint32_t nstg = lds_s32(args + offsetof(LatentArgs, stages)), ntiles = lds_s32(args + offsetof(LatentArgs, ntiles));
+    if (nstg >= 4) asm volatile("cp.async.wait_group 1;" ::: "memory");
     else asm volatile("cp.async.wait_group 0;" ::: "memory");
-    consumer_sync();   // the tile has landed for everyone, and everyone is done with the stage refilled next
+    consumer_sync();   // the tile has landed for everyone, the weights of the one before are final, the one before that is free
     if (it == 0) stamp(P, la.task, 1);
-    issue(it + nstg - 1, stg == 0 ? nstg - 1 : stg - 1);
-    const uint32_t kt = ring + stg * tile;
-    if (++stg == nstg) stg = 0;
-    {   // ---- scores
-      const int kw = warp % KW, ks = warp / KW;
+    const uint32_t kt = ring + slot * (KEYS * pitch);
+    issue(it + nstg - 2, ring + (slot >= 2 ? slot - 2 : slot + nstg - 2) * (KEYS * pitch));
+    if (++slot == nstg) slot = 0;
+    {
+      const int kw = warp % KW, ks = warp / KW, ksteps = it < (int)ntiles ? (int)(pitch >> 5) : 0;   // 16-column steps of a row
       float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
       const uint32_t ka = kt + (uint32_t)((kw * 16 + (lane & 7) + (lane >> 4) * 8) * pitch + ((lane >> 3) & 1) * 16);
       const uint32_t qa = sm + oQ + (uint32_t)((lane & 15) * pitch + (lane >> 4) * 16);
+      int kk = ks;
+      if (it > 0) {
+        const float c0 = lds_f32(sm + oC + (lane >> 2) * 4), c1 = lds_f32(sm + oC + (8 + (lane >> 2)) * 4);
+        if (__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) {
+#pragma unroll
+          for (int i = 0; i < NV; ++i) {
+            o[i][0] *= c0; o[i][1] *= c0;
+            o[i][2] *= c1; o[i][3] *= c1;
+          }
+        }
+        // 16 keys and two column tiles at a time (one past the last is read, not used), a step of the scores beside each
+        const uint32_t pa = sm + oP + (uint32_t)((lane & 15) * PP + (lane >> 4) * 16);
+#pragma unroll
+        for (int k = 0; k < KW; ++k) {
+          uint32_t p[2][4];
+#pragma unroll
+          for (int h = 0; h < 2; ++h) ldmatrix_x4(p[h], pa + (uint32_t)(h * RT * PP + k * 32));
+          const uint32_t va = before + (uint32_t)(k * 16 + (lane & 15)) * pitch + warp * 16 + (lane >> 4) * 128u;
+#pragma unroll
+          for (int i = 0; i < NV; i += 2) {
+            if (i >= nv) break;
+            uint32_t v[4], a[4], b[4];
+            ldmatrix_x4_trans(v, va + i * 128u);
+            if (kk < ksteps) {
+              ldmatrix_x4(b, ka + kk * 32u);
+              ldmatrix_x4(a, qa + kk * 32u);
+              mma_bf16_16816(s[0], a, b[0], b[1]);
+              mma_bf16_16816(s[1], a, b[2], b[3]);
+              kk += KS;
+            }
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+              mma_bf16_16816(o[i], p[h], v[0], v[1]);
+              if (i + 1 < nv) mma_bf16_16816(o[i + 1], p[h], v[2], v[3]);
+            }
+          }
+        }
+      }
 #pragma unroll 2
-      for (int kk = ks; kk < ksteps; kk += KS) {
+      for (; kk < ksteps; kk += KS) {
         uint32_t a[4], b[4];
         ldmatrix_x4(b, ka + kk * 32u);
         ldmatrix_x4(a, qa + kk * 32u);
         mma_bf16_16816(s[0], a, b[0], b[1]);
         mma_bf16_16816(s[1], a, b[2], b[3]);
       }
+      before = kt;
+      if (it == (int)ntiles) break;
       const uint32_t sr = sm + (uint32_t)(((ks * RT + (lane >> 2)) * SP + kw * 16 + 2 * (lane & 3)) * 4);
 #pragma unroll
       for (int n = 0; n < 2; ++n) {
@@ -1353,6 +1415,7 @@ __device__ __noinline__ void latent_attention_mma(const KernelParams &P, uint32_
     consumer_sync();
     {   // ---- softmax
       const uint32_t sa = sm + (uint32_t)((srow * SP + skey) * 4), pa = sm + oP + (uint32_t)(srow * PP + skey * 2);
+      const float scale = lds_f32(args + offsetof(LatentArgs, scale)), cap = lds_f32(args + offsetof(LatentArgs, cap));
       const float cap2 = cap > 0.f ? 2.0f * 1.4426950408889634f / cap : 0.f;
 #pragma unroll
       for (int i = 0; i < RPW; ++i) {
@@ -1375,37 +1438,6 @@ __device__ __noinline__ void latent_attention_mma(const KernelParams &P, uint32_
         if (skey == 0) sts_f32(sm + oC + (srow + r) * 4, corr);
       }
     }
-    consumer_sync();
-    {   // ---- output
-      const float c0 = lds_f32(sm + oC + (lane >> 2) * 4), c1 = lds_f32(sm + oC + (8 + (lane >> 2)) * 4);
-      if (__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) {
-#pragma unroll
-        for (int i = 0; i < NV; ++i) {
-          o[i][0] *= c0; o[i][1] *= c0;
-          o[i][2] *= c1; o[i][3] *= c1;
-        }
-      }
-      // 16 keys and two column tiles at a time (one past the last is read, not used)
-      const uint32_t pa = sm + oP + (uint32_t)((lane & 15) * PP + (lane >> 4) * 16);
-#pragma unroll
-      for (int k = 0; k < KW; ++k) {
-        uint32_t p[2][4];
-#pragma unroll
-        for (int h = 0; h < 2; ++h) ldmatrix_x4(p[h], pa + (uint32_t)(h * RT * PP + k * 32));
-        const uint32_t va = kt + (uint32_t)(k * 16 + (lane & 15)) * pitch + warp * 16 + (lane >> 4) * 128u;
-#pragma unroll
-        for (int i = 0; i < NV; i += 2) {
-          if (i >= nv) break;
-          uint32_t b[4];
-          ldmatrix_x4_trans(b, va + i * 128u);
-#pragma unroll
-          for (int h = 0; h < 2; ++h) {
-            mma_bf16_16816(o[i], p[h], b[0], b[1]);
-            if (i + 1 < nv) mma_bf16_16816(o[i + 1], p[h], b[2], b[3]);
-          }
-        }
-      }
-    }
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   stamp(P, la.task, 2);
@@ -1422,10 +1454,11 @@ __device__ __noinline__ void latent_attention_mma(const KernelParams &P, uint32_
     }
   }
   consumer_sync();
+  const AttnOut &ao = la.ao;
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
-    const int r = h * 8 + (lane >> 2), row = row0 + r;
-    if (r >= nrow) continue;
+    const int r = h * 8 + (lane >> 2), row = la.row0 + r;
+    if (r >= la.nrow) continue;
     const float mx = lds_f32(sm + oC + r * 4), l = lds_f32(sm + oC + (RT + r) * 4);
     const int col0 = warp * 8 + 2 * (lane & 3);
     if (ao.n_act == 1) {
@@ -1546,10 +1579,20 @@ __device__ __forceinline__ void run_ext_attention(const Ctx &c, const TaskDesc &
     ext_attention_f32(c, d, sv, ao, k0, k1, row0, row1);
   } else if (d.a[XA_SHARED]) {
     LatentArgs &la = *reinterpret_cast<LatentArgs *>(c.s.red);   // (begins with `ao`)
+    const int keys = d.a[XA_KEYS];
     for (int r = row0; r < row1; r += 16) {
       if (r > row0) consumer_sync();
-      la.q0 = sv.q0; la.pos0 = sv.pos0; la.kv0 = sv.kv0; la.k0 = k0; la.k1 = k1; la.row0 = r; la.nrow = min(16, row1 - r); la.task = task;
-      if (d.a[XA_KEYS] == 32) latent_attention_mma<32>(c.P, smem_u32(c.s.xtile), d, la);
+      const int n = min(16, row1 - r), kend = min(k1, sv.pos0 + (r + n - 1) / ao.G + 1);   // keys past the last row's position are not needed
+      la.keys = max(kend - k0, 0);
+      la.pieces = d.a[XA_DIMP] >> 3;
+      la.table = (d.a[XA_PAGE] & 7) == 0 && la.keys <= 8 * kXaCells;   // eight consecutive keys lie in one page
+      la.ntiles = (la.keys + keys - 1) / keys;
+      la.rows = reinterpret_cast<const uint4 *>(d.p[1]);
+      la.pages = c.P.meta.paged_kv_indices + sv.kv0;
+      la.scale = __int_as_float(d.a[XA_SCALE]);
+      la.cap = __int_as_float(d.a[XA_CAP]);
+      la.page = d.a[XA_PAGE]; la.k0 = k0; la.q0 = sv.q0; la.pos0 = sv.pos0; la.row0 = r; la.nrow = n; la.task = task; la.stages = d.a[XA_STAGES];
+      if (keys == 32) latent_attention_mma<32>(c.P, smem_u32(c.s.xtile), d, la);
       else latent_attention_mma<16>(c.P, smem_u32(c.s.xtile), d, la);
     }
   } else {

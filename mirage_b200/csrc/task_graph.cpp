@@ -1154,15 +1154,15 @@ struct Builder {
   struct LatentPlan { int keys, stages; int64_t bytes; };
   LatentPlan latent_plan(const LayerInfo &l) const {
     const int64_t pitch = round_up(T[l.t[1]].dim(3), 64) * 2 + 16;
-    const int64_t budget = kPartialBytes + (nb_max > 8 ? 64 * (1024 * 2 + kRowPadBytes) : 90 * 1024);
+    const int64_t budget = nb_max > 8 ? kSmemBudget - kMiscBytes - 5 * kTcSlotBytes : kPartialBytes + 90 * 1024;
     LatentPlan p{0, 0, 0};
     for (int keys : {32, 16}) {
       const int64_t fixed = 32 + 16 * pitch + (int64_t)(8 / (keys / 16)) * 16 * (keys + 4) * 4 + 2 * 16 * (keys * 2 + 16) + 8 * 16 + kXaCells * 4;
       p.keys = keys;
       p.stages = (int)std::min<int64_t>(4, (budget - fixed) / (keys * pitch));
-      if (p.stages < 2 && keys == 16) p.stages = 2;   // the smallest tiles: whatever they need
+      if (p.stages < 3 && keys == 16) p.stages = 3;   // the smallest tiles: whatever they need
       p.bytes = fixed + p.stages * keys * pitch;
-      if (p.stages >= (keys == 32 ? 3 : 2)) return p;
+      if (p.stages >= 3) return p;
     }
     return p;
   }
