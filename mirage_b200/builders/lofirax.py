@@ -21,7 +21,7 @@ from typing import Any, Dict, List, Optional, Tuple
 import torch
 
 from ..mpk import register_model_builder
-from ..persistent_kernel import DTensor, PersistentKernel, bfloat16, float32, int32
+from ..persistent_kernel import DTensor, float32, int32
 from .hybrid import HybridBuilder, HybridModelConfig, k_padded, round_up
 
 

@@ -20,7 +20,7 @@ from typing import Any, Dict, List, Optional, Tuple
 import torch
 
 from ..mpk import register_model_builder
-from ..persistent_kernel import DTensor, PersistentKernel, bfloat16, float32
+from ..persistent_kernel import DTensor, PersistentKernel, float32
 from .hybrid import HybridBuilder, HybridModelConfig, round_up
 
 
