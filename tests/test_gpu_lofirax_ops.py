@@ -133,6 +133,23 @@ def test_latent_attention(dtype, tokens, H, dim, rot, vdim, rank):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+def test_latent_attention_on_pages_of_odd_size(dtype):
+    """Eight consecutive keys may lie in two pages."""
+    H, dim, rot, vdim, rank = 3, 16, 8, 8, 48
+    src = [s.to(torch.bfloat16).float() for s in sources(H * (dim + rot) + rank + rot, 33)]
+    g = torch.Generator().manual_seed(16)
+    args = (H, dim, rot, vdim, rank, 900.0, 0.15, 1e-4, RAND(g, rank, std=0.3, mean=1.0), RAND(g, H * dim, rank, std=rank ** -0.5),
+            RAND(g, H * vdim, rank, std=rank ** -0.5), RAND(g, H))
+    b = Bench(3, page=5)
+    dst, out = latent_graph(b, dtype, *args)
+    b.pk.compile()
+    got = feed(b, src, dst, out, SCHEDULE, RESTART)
+    for r in range(3):
+        ref = latent_reference(src[r][:LENGTHS[r]], *args)
+        assert err(got[r], ref) < (1e-5 if dtype == torch.float32 else 2.5e-2), r
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("tokens", [64, 4])
 @pytest.mark.parametrize("H,dim,rot,vdim,rank", [(4, 16, 8, 16, 64), (20, 32, 64, 16, 512)])
 def test_far_keys_stand_out(dtype, tokens, H, dim, rot, vdim, rank):
