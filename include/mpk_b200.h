@@ -60,7 +60,8 @@ typedef enum {
   MPK_OP_EMBED = 1,             /* embed_layer              :586  in: ids, table        out: y            params: [input_source, factor (hybrid graphs)] */
   MPK_OP_RMSNORM = 2,           /* rmsnorm_layer            :609  in: x, gamma          out: y                                            */
   MPK_OP_RMSNORM_LINEAR = 3,    /* rmsnorm_linear_layer     :627  in: x, gamma, W       out: y                                            */
-  MPK_OP_LINEAR = 4,            /* linear_layer             :1731 in: x, W              out: y            params: optional [activation, soft cap] (hybrid graphs, mpk_activation)  */
+  MPK_OP_LINEAR = 4,            /* linear_layer             :1731 in: x, W              out: y            params: optional [activation, soft cap] (hybrid graphs, mpk_activation)
+                                   hybrid graphs, optional fourth tensor: bf16 bias [rows of W], float32 y */
   MPK_OP_LINEAR_RESIDUAL = 5,   /* linear_with_residual_layer :1762 in: x, W, residual  out: y            params: [enable_residual]       */
   MPK_OP_SPLITK_LINEAR = 6,     /* splitk_linear_layer      :1706 in: x, W              out: y (y += x W^T)                               */
   MPK_OP_ATTENTION = 7,         /* attention_layer          :648  in: qkv,k,v,qn,kn,cos,sin out: o       params: [hq, hkv, qk_norm, rope] */
@@ -99,8 +100,8 @@ typedef enum {
   MPK_OP_ARGMAX_EXCHANGE = 30,  /* in: value, index (local columns)  out: token ids   params: [first column of this rank] */
   MPK_OP_MOE_TOPK_SOFTMAX = 31  /* moe_topk_softmax_routing_layer :1385 in: logits  out: topk_weight, routing_indices, mask
                                    (softmax over the experts, top-k by value with ties to the lower index, weights renormalised
-                                   over the selected experts; the logits are left as they are)  params: optional [first, end]
-                                   of the experts this rank runs */
+                                   over the selected experts; the logits are left as they are)  params: optional [first, end of the experts this rank runs,
+                                   1: weights are the probabilities, not renormalised, scaling_bits] */
   ,
   /* Hybrid graphs (no reference counterpart): float32 residual stream, attention with free head sizes, recurrent layers.
    * A graph with one of these may hold, besides them, embed, linear, argmax and sampling layers; all floats in params
@@ -111,14 +112,22 @@ typedef enum {
                                    6 bias of the output norm  7 stream added as it is, f32 [tokens, width]  8 row added to every token, bf16 [width]
                                    9 expert outputs f32 [tokens, slots, width]  10 their weights f32 [tokens, slots]
                                    11 f32 [tokens, columns]: y is multiplied by sigmoid of column params[3]
-                                   params: [eps, weights stored around zero, 0 RMS norm | 1 layer norm, gate column] */
-  MPK_OP_QKV_APPEND = 33,       /* rotate q and k, unit RMS norm, append k / v rows   in: projections, cos, sin  out: q, k_cache, v_cache
-                                   tensors: proj, q, k_cache, v_cache, cos, sin
-                                   params: [hq, hkv, dim, vdim, q_col, k_col, v_col, rotated dims, unit norm, eps] */
+                                   params: [eps, weights stored around zero, 0 RMS norm | 1 layer norm, gate column, factor of y's norm]
+                                   with a weight of y's norm: x += factor * norm(y + weighted sum of the experts) * weight
+                                   an output without a norm weight is the new stream as it is */
+  MPK_OP_QKV_APPEND = 33,       /* norm and rotate q and k, append k / v rows   in: projections, cos, sin  out: q, k_cache, v_cache
+                                   tensors: proj, q, k_cache, v_cache (caches absent: queries only), cos, sin, q norm, k norm (optional, bf16 [dim])
+                                   params: [hq, hkv, dim, vdim, q_col, k_col, v_col, rotated dims, unit norm (after the rotation), eps,
+                                   optional: 1 pairs are neighbours (0: halves), maps]
+                                   q / k norm: an RMS norm in front of the rotation.  maps = 2: q and k have two vectors per head; a cache row
+                                   holds both, a query row (two per head) has its own and zeros for the other */
   MPK_OP_EXT_ATTENTION = 34,    /* tensors: q, k_cache, v_cache (= k_cache: the leading vdim columns of a key are its value), out, sinks (optional)
-                                   params: [hq, hkv, vdim, out_col, scale, soft cap (0: none), sink, out_scale, optional 1: an MPK_OP_ATTN_MERGE layer follows]
+                                   params: [hq, hkv, vdim, out_col, scale, soft cap (0: none), sink, out_scale, optional 1: an MPK_OP_ATTN_MERGE layer follows,
+                                   optional window, kept]: with a window a position sees itself, the window - 1 before it and the first `kept`
+                                   out: the activation type, or float32
                                    sink: exp(sinks[head]) joins the softmax denominator (bf16 [hq]; without the tensor: 1) */
-  MPK_OP_SHORT_CONV = 35,       /* causal per-channel convolution   tensors: in, in_bias, taps, bias, state, out (biases optional)
+  MPK_OP_SHORT_CONV = 35,       /* causal per-channel convolution   tensors: in, in_bias, taps, bias, state, out, copy of out in the activation type
+                                   (biases and copy optional)
                                    params: [in_col, activation: 0 none, 1 silu] */
   MPK_OP_RGLRU = 36,            /* gated diagonal recurrence        tensors: u, proj, y_bias, ra, ra_bias, ri, ri_bias, lambda, state, out
                                    params: [y_col, out_col, out_scale, decay constant] */
@@ -133,7 +142,14 @@ typedef enum {
                                    params: [x stride, y column, y stride]: group g reads x[:, g * x stride + (0 .. K)] and writes
                                    y[:, y column + g * y stride + (0 .. N)] */,
   MPK_OP_ATTN_MERGE = 41        /* directly behind an MPK_OP_EXT_ATTENTION layer with its ninth parameter set: the same tensors and parameters;
-                                   merges the key chunks on all workers (for wide values) */
+                                   merges the key chunks on all workers (for wide values) */,
+  MPK_OP_SELECTIVE_SCAN = 42,   /* selective state space recurrence   tensors: u f32, low f32 [tokens, rank + 2 n], gate f32, dt weight [channels, rank],
+                                   dt bias, A_log [channels, n], D (bf16), state f32 [slots, channels, n up to a multiple of 4], out
+                                   params: [rank, n, gate column]
+                                   dt = softplus(dt weight . low[:, :rank] + dt bias), S = exp(-dt exp(A_log)) S + dt u B, out = (S C + D u) * silu(gate),
+                                   B and C the next 2 n columns of low */
+  MPK_OP_DIFF_COMBINE = 43      /* differential attention   in: maps f32 [tokens, heads * 2 * vdim]  out: y [tokens, >= heads * vdim]
+                                   params: [heads, vdim, lambda, factor, eps]: y = factor * unit norm(map 1 - lambda map 2) per head */
 } mpk_op;
 
 /* Activations of linear layers in hybrid graphs.  The gated ones take weight rows interleaved as two gate rows, two up rows, and

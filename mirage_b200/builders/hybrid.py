@@ -5,12 +5,13 @@ buffers in front of them likewise: what the padding columns hold is finite and m
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import Any, Dict, List, Optional, Tuple
 
 import torch
 
-from ..persistent_kernel import DTensor, PersistentKernel, bfloat16, float32, int64
+from ..persistent_kernel import DTensor, PersistentKernel, bfloat16, float32, int32, int64
 
 
 def round_up(n: int, m: int) -> int:
@@ -22,12 +23,30 @@ def k_padded(k: int, dtype: torch.dtype) -> int:
     return round_up(k, 64) if dtype == torch.bfloat16 else k
 
 
-def rotary_tables(base: float, dims: int, positions: int, device) -> Tuple[torch.Tensor, torch.Tensor]:
+@dataclass(frozen=True)
+class RotaryScaling:
+    """Frequencies for longer contexts as in Llama 3.1: wavelengths longer than original / low positions are stretched by `factor`,
+    those shorter than original / high are kept, the ones between are blended."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+    def apply(self, f: torch.Tensor) -> torch.Tensor:
+        turns = self.original * f / (2.0 * math.pi)           # original / wavelength
+        s = (turns - self.low) / (self.high - self.low)
+        blend = (1.0 - s) * f / self.factor + s * f
+        return torch.where(turns > self.high, f, torch.where(turns < self.low, f / self.factor, blend))
+
+
+def rotary_tables(base: float, dims: int, positions: int, device, scaling: Optional[RotaryScaling] = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """float32 cos / sin [positions, dims / 2] of position * base^(-2i / dims); the angles are formed in 64-bit."""
     if dims == 0:
         z = torch.zeros(1, 1, dtype=torch.float32, device=device)
         return z, z.clone()
     f = float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+    if scaling is not None:
+        f = scaling.apply(f)
     a = torch.arange(positions, dtype=torch.float64)[:, None] * f
     return a.cos().float().to(device), a.sin().float().to(device)
 
@@ -52,7 +71,7 @@ class HybridBuilder:
         self.logits: Optional[DTensor] = None
         self.hidden: Optional[DTensor] = None      # float32 residual stream
         self._buffers: Dict[Tuple[str, tuple], DTensor] = {}
-        self._tables: Dict[Tuple[float, int], Tuple[DTensor, DTensor]] = {}
+        self._tables: Dict[tuple, Tuple[DTensor, DTensor]] = {}
         self._attached: Dict[str, DTensor] = {}
 
     def _begin(self, mc: HybridModelConfig):
@@ -91,11 +110,44 @@ class HybridBuilder:
     def _linear(self, x: DTensor, w: DTensor, y: DTensor, activation: str = None, **kw):
         self.mpk.linear_layer(input=x, weight=w, output=y, grid_dim=(96, 1, 1), block_dim=(128, 1, 1), activation=activation, **kw)
 
-    def _rotary(self, base: float, dims: int) -> Tuple[DTensor, DTensor]:
-        key = (base, dims)
+    def _sublayer(self, x: DTensor, name: str, parts: List[torch.Tensor], bias: Optional[DTensor] = None) -> DTensor:
+        """A sublayer's output linear, float32."""
+        y = self._buf("sublayer", self.width, float32)
+        self._linear(x, self._weight(name + ".padded", parts), y, bias=bias)
+        return y
+
+    def _gated(self, x: DTensor, p: str, ff: int, activation: str) -> DTensor:
+        """down(act(gate x) * (up x)) for weights `p`gate / up / down."""
+        sd, mid = self.sd, self._buf("ff", self._kpad(round_up(ff, 2)), self.act)
+        even = lambda w: torch.nn.functional.pad(w, (0, 0, 0, ff % 2))
+        w = self._attach(p + "gate_up", lambda: self._pad_k(self.mpk.interleave_gated(even(sd[p + "gate"]), even(sd[p + "up"]))))
+        self._linear(x, w, mid, activation=activation)
+        return self._sublayer(mid, p + "down", [torch.nn.functional.pad(sd[p + "down"], (0, ff % 2))])
+
+    def _routing(self, experts: int, top: int) -> Tuple[DTensor, DTensor, DTensor]:
+        """(expert weights, routing table, active list) a routing layer fills."""
+        weights = self._buf("expert_weights", top, float32)
+        key = ("routing", (experts,))
+        if key not in self._buffers:
+            self._buffers[key] = (self.mpk.new_tensor(dims=(experts, self.mpk.max_num_batched_tokens), dtype=int32, name=f"routing_{experts}"),
+                                  self.mpk.new_tensor(dims=(experts + 1,), dtype=int32, name=f"active_{experts}"))
+        return (weights, *self._buffers[key])
+
+    def _experts(self, h: DTensor, routing: Tuple[DTensor, DTensor, DTensor], first: DTensor, second: DTensor, ff: int, top: int,
+                 activation: str) -> DTensor:
+        """Outputs [tokens, slots, width] of the chosen experts: second(act(first h)), `ff` columns in between (padded)."""
+        grid = dict(grid_dim=(1, 1, 1), block_dim=(128, 1, 1))
+        mid = self._buf("expert_mid", (top, ff), self.act)
+        self.mpk.moe_w13_linear_layer(h, first, *routing[1:], mid, **grid, activation=activation)
+        out = self._buf("expert_out", (top, self.width), float32)
+        self.mpk.moe_w2_linear_layer(mid, second, *routing[1:], out, **grid)
+        return out
+
+    def _rotary(self, base: float, dims: int, scaling: Optional[RotaryScaling] = None) -> Tuple[DTensor, DTensor]:
+        key = (base, dims, scaling)
         if key not in self._tables:
             dev = self.sd["embed"].device
-            cos, sin = rotary_tables(base, dims, self.mpk.max_seq_length, dev)
+            cos, sin = rotary_tables(base, dims, self.mpk.max_seq_length, dev, scaling)
             n = len(self._tables)
             self._tables[key] = (self.mpk.attach_input(cos, name=f"cos_{n}"), self.mpk.attach_input(sin, name=f"sin_{n}"))
         return self._tables[key]

@@ -21,7 +21,7 @@ from typing import Any, Dict, List, Optional, Tuple
 import torch
 
 from ..mpk import register_model_builder
-from ..persistent_kernel import DTensor, float32, int32
+from ..persistent_kernel import DTensor, float32
 from .hybrid import HybridBuilder, HybridModelConfig, k_padded, round_up
 
 
@@ -187,29 +187,16 @@ class LofiraxBuilder(HybridBuilder):
         return self._sublayer(values, p + "o", [sd[p + "o"]])
 
     # -- feed-forwards: return the terms that join the stream (arguments of residual_norm_layer)
-    def _gated(self, x: DTensor, p: str, ff: int, activation: str) -> DTensor:
-        """down(act(gate x) * (up x)) for weights `p`gate / up / down."""
-        sd, mid = self.sd, self._buf("ff", self._kpad(round_up(ff, 2)), self.act)
-        even = lambda w: torch.nn.functional.pad(w, (0, 0, 0, ff % 2))
-        w = self._attach(p + "gate_up", lambda: self._pad_k(self.mpk.interleave_gated(even(sd[p + "gate"]), even(sd[p + "up"]))))
-        self._linear(x, w, mid, activation=activation)
-        return self._sublayer(mid, p + "down", [torch.nn.functional.pad(sd[p + "down"], (0, ff % 2))])
-
     def _moe(self, h: DTensor, p: str, m: MoeSpec) -> Dict[str, Any]:
-        mpk, sd, mbt = self.mpk, self.sd, self.mpk.max_num_batched_tokens
+        mpk, sd = self.mpk, self.sd
         E, F = m.experts, self._kpad(round_up(m.ff, 2))
         shared = m.shared_ff is not None
         logits = self._buf("router", E + int(shared), float32)
         self._linear(h, self._weight(p + "router.sg", [sd[p + "router"]] + ([sd[p + "shared.sg"]] if shared else [])), logits)
-        weights = self._buf("expert_weights", m.top, float32)
-        key = ("routing", (E,))
-        if key not in self._buffers:
-            self._buffers[key] = (mpk.new_tensor(dims=(E, mbt), dtype=int32, name=f"routing_{E}"),
-                                  mpk.new_tensor(dims=(E + 1,), dtype=int32, name=f"active_{E}"))
-        routing, active = self._buffers[key]
+        routing = self._routing(E, m.top)
         grid = dict(grid_dim=(1, 1, 1), block_dim=(128, 1, 1))
         mpk.moe_topk_sigmoid_routing_layer(logits, self._attach(p + "correction.f32", lambda: sd[p + "correction"].float()),
-                                           (weights, routing, active), **grid, num_groups=m.groups, topk_group=m.keep,
+                                           routing, **grid, num_groups=m.groups, topk_group=m.keep,
                                            routed_scaling_factor=1.0, keep_logits=True)
         y = self._gated(h, p + "shared.", m.shared_ff, "gated_silu") if shared else None
         rows = lambda n, r: torch.nn.functional.pad(n, (0, 0, 0, r - n.shape[0]))
@@ -217,16 +204,8 @@ class LofiraxBuilder(HybridBuilder):
             [self._pad_k(mpk.interleave_gated(rows(sd[f"{p}e{e}.gate"], F), rows(sd[f"{p}e{e}.up"], F))) for e in range(E)]))
         w2 = self._attach(p + "experts.down", lambda: torch.stack(
             [torch.nn.functional.pad(sd[f"{p}e{e}.down"], (0, F - m.ff)) for e in range(E)]))
-        mid = self._buf("expert_mid", (m.top, F), self.act)
-        mpk.moe_w13_linear_layer(h, w13, routing, active, mid, **grid, activation="gated_silu")
-        out = self._buf("expert_out", (m.top, self.width), float32)
-        mpk.moe_w2_linear_layer(mid, w2, routing, active, out, **grid)
-        return {"y": y, "experts": (out, weights), "y_gate": (logits, E) if shared else None}
-
-    def _sublayer(self, x: DTensor, name: str, parts: List[torch.Tensor]) -> DTensor:
-        y = self._buf("sublayer", self.width, float32)
-        self._linear(x, self._weight(name + ".padded", parts), y)
-        return y
+        out = self._experts(h, routing, w13, w2, F, m.top, "gated_silu")
+        return {"y": y, "experts": (out, routing[0]), "y_gate": (logits, E) if shared else None}
 
     def build_from_config(self, mc: LofiraxModelConfig):
         mpk, c, sd = self.mpk, mc.config, mc.state_dict

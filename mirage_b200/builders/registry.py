@@ -9,6 +9,7 @@ import torch
 
 # architecture name -> (runner class in builders.runner, kernel family it runs on, activation types)
 _RUNNERS = {
+    "bebuzen": ("BebuzenRunner", "hybrid", (torch.bfloat16, torch.float32)),
     "lofirax": ("LofiraxRunner", "hybrid", (torch.bfloat16, torch.float32)),
     "palarax": ("PalaraxRunner", "hybrid", (torch.bfloat16, torch.float32)),
     "qwen3forcausallm": ("Qwen3Runner", "decoder", (torch.bfloat16,)),

@@ -200,3 +200,10 @@ class LofiraxRunner(HybridRunner):
     def _model(cls):
         from . import lofirax as m
         return m.LofiraxConfig, m.LofiraxBuilder, m.LofiraxModelConfig, m.allocate_state
+
+
+class BebuzenRunner(HybridRunner):
+    @classmethod
+    def _model(cls):
+        from . import bebuzen as m
+        return m.BebuzenConfig, m.BebuzenBuilder, m.BebuzenModelConfig, m.allocate_state

@@ -1,9 +1,11 @@
 // Task bodies of hybrid graphs: decoders whose layers mix softmax attention with recurrent state.
 //
 //   float32 residual stream      TASK_EMBED_F32, TASK_RESIDUAL_NORM
-//   attention                    TASK_QKV_APPEND (rotation, unit norms, cache rows), TASK_LATENT_APPEND (latent rows that serve
-//                                as keys and values), TASK_EXT_ATTENTION (any head size, score scale, soft cap, sinks)
-//   recurrences                  TASK_SHORT_CONV, TASK_RGLRU (gated diagonal), TASK_MLSTM and TASK_GLA (matrix memories)
+//   attention                    TASK_QKV_APPEND (norms, rotation, cache rows), TASK_LATENT_APPEND (latent rows that serve
+//                                as keys and values), TASK_EXT_ATTENTION (any head size, score scale, soft cap, sinks, sliding
+//                                window), TASK_DIFF_COMBINE (differential attention)
+//   recurrences                  TASK_SHORT_CONV, TASK_RGLRU (gated diagonal), TASK_SELECTIVE_SCAN (diagonal, input-dependent steps),
+//                                TASK_MLSTM and TASK_GLA (matrix memories)
 //   experts                      TASK_MOE_ROUTING, TASK_MOE_GEMM (megakernel.cuh); their sum is part of TASK_RESIDUAL_NORM
 //   32-bit graphs                TASK_LINEAR_F32, TASK_MOE_GEMM_F32
 //
@@ -130,10 +132,12 @@ struct NormTerms {
   const float *add, *experts, *ew, *gate;   // added stream, expert outputs and their weights, logit whose sigmoid scales y
   uint64_t row, bias;                       // row added to every token, bias of the output norm
   int slots;
+  float factor;                             // of y's norm
 };
 __device__ __forceinline__ NormTerms norm_terms(const TaskDesc &d, int t) {
   NormTerms n;
   n.slots = d.a[RN_SLOTS];
+  n.factor = __int_as_float(d.a[RN_POST]);
   n.add = reinterpret_cast<const float *>(wide_arg(d, RN_ADD));
   n.experts = reinterpret_cast<const float *>(wide_arg(d, RN_EXP));
   n.ew = reinterpret_cast<const float *>(wide_arg(d, RN_EW));
@@ -157,16 +161,26 @@ __device__ __forceinline__ void residual_norm_rows(const Ctx &c, const TaskDesc 
   const float eps = __int_as_float(d.a[6]);
   const float off = (d.a[7] & 2) ? 1.0f : 0.0f;
   const bool layer_norm = (d.a[7] & 4) != 0;
-  const bool has_y = d.p[1] != 0, has_post = d.p[2] != 0, has_out = d.p[3] != 0;
+  const bool has_y = d.p[1] != 0, has_post = d.p[2] != 0, has_out = d.p[3] != 0, has_copy = !has_out && d.p[4] != 0;
   float *row = reinterpret_cast<float *>(c.s.xtile);
   for (int t = t0; t < t1; ++t) {
     float *x = reinterpret_cast<float *>(d.p[0]) + (size_t)t * d.a[3];
     float *xo = reinterpret_cast<float *>(d.p[5]) + (size_t)t * d.a[8];
     const float *y = reinterpret_cast<const float *>(d.p[1]) + (size_t)t * d.a[4];
+    T *out = reinterpret_cast<T *>(d.p[4]) + (size_t)t * d.a[5];
     const NormTerms nt = norm_terms(d, t);
     const bool moved = has_y || nt.add || nt.experts || nt.row;
     float inv = nt.gate ? sigmoid_f(__ldcg(nt.gate)) : 1.f;
-    if (has_y && has_post) {
+    if (has_post && nt.slots > 0) {   // the experts' sum is part of what is normed
+      float ss = 0.f;
+      for (int j = threadIdx.x; j < W; j += kConsumerThreads) {
+        float v = has_y ? __ldcg(y + j) : 0.f;
+        for (int k = 0; k < nt.slots; ++k) v = fmaf(__ldcg(nt.ew + k), __ldcg(nt.experts + (size_t)k * W + j), v);
+        row[j] = v;
+        ss += v * v;
+      }
+      inv = nt.factor / sqrtf(block_sum(ss, c.s.red) / (float)W + eps);   // (its barrier: the row is complete)
+    } else if (has_y && has_post) {
       float ss = 0.f;
       for (int j = threadIdx.x * VEC; j < W; j += kConsumerThreads * VEC) {
         if (VEC == 4) {
@@ -179,29 +193,30 @@ __device__ __forceinline__ void residual_norm_rows(const Ctx &c, const TaskDesc 
           ss += v * v;
         }
       }
-      inv = 1.0f / sqrtf(block_sum(ss, c.s.red) / (float)W + eps);
+      inv = nt.factor / sqrtf(block_sum(ss, c.s.red) / (float)W + eps);
     }
     float ss = 0.f, sum = 0.f;
     for (int j = threadIdx.x * VEC; j < W; j += kConsumerThreads * VEC) {
       float xv[VEC], yv[VEC];
       if (VEC == 4) {
         *reinterpret_cast<float4 *>(xv) = __ldcg(reinterpret_cast<const float4 *>(x + j));
-        if (has_y) *reinterpret_cast<float4 *>(yv) = has_post ? *reinterpret_cast<const float4 *>(row + j)
+        if (has_y || has_post) *reinterpret_cast<float4 *>(yv) = has_post ? *reinterpret_cast<const float4 *>(row + j)
                                                               : __ldcg(reinterpret_cast<const float4 *>(y + j));
       } else {
         xv[0] = __ldcg(x + j);
-        if (has_y) yv[0] = has_post ? row[j] : __ldcg(y + j);
+        if (has_y || has_post) yv[0] = has_post ? row[j] : __ldcg(y + j);
       }
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
-        if (has_y) xv[e] += has_post ? yv[e] * inv * (off + bf16_at(d.p[2], j + e)) : yv[e] * inv;
-        for (int k = 0; k < nt.slots; ++k) xv[e] = fmaf(__ldcg(nt.ew + k), __ldcg(nt.experts + (size_t)k * W + j + e), xv[e]);
+        if (has_y || has_post) xv[e] += has_post ? yv[e] * inv * (off + bf16_at(d.p[2], j + e)) : yv[e] * inv;
+        for (int k = 0; k < (has_post ? 0 : nt.slots); ++k) xv[e] = fmaf(__ldcg(nt.ew + k), __ldcg(nt.experts + (size_t)k * W + j + e), xv[e]);
         if (nt.add) xv[e] += __ldcg(nt.add + j + e);
         if (nt.row) xv[e] += bf16_at(nt.row, j + e);
         ss += xv[e] * xv[e];
         sum += xv[e];
         row[j + e] = xv[e];
         if (moved) xo[j + e] = xv[e];
+        if (has_copy) store_elt(out + j + e, xv[e]);
       }
     }
     if (has_out) {
@@ -214,7 +229,6 @@ __device__ __forceinline__ void residual_norm_rows(const Ctx &c, const TaskDesc 
           for (int e = 0; e < VEC; ++e) { const float v = row[j + e] - mean; ss += v * v; }
       }
       const float inv2 = 1.0f / sqrtf(block_sum(ss, c.s.red + 8) / (float)W + eps);
-      T *out = reinterpret_cast<T *>(d.p[4]) + (size_t)t * d.a[5];
       for (int j = threadIdx.x * VEC; j < W; j += kConsumerThreads * VEC) {
 #pragma unroll
         for (int e = 0; e < VEC; ++e)
@@ -265,13 +279,34 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
       wp[i] = in && has_post ? bf16x4_at(d.p[2], j) : zero;
       wn[i] = in && has_out ? bf16x4_at(d.p[3], j) : zero;
     }
-    if (has_y) {
+    // the weighted sum over the experts: part of what is normed, or added to the stream
+    auto add_experts = [&](float4 (&to)[NV]) {
+      for (int k = 0; k < nt.slots; k += 2) {   // two experts' rows in flight
+        float4 e[2][NV];
+        float w[2];
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          w[u] = k + u < nt.slots ? __ldcg(nt.ew + k + u) : 0.f;
+#pragma unroll
+          for (int i = 0; i < NV; ++i) {
+            const int j = (i * kConsumerThreads + tid) * 4;
+            e[u][i] = j < W && k + u < nt.slots ? __ldcg(reinterpret_cast<const float4 *>(nt.experts + (size_t)(k + u) * W + j)) : zero;
+          }
+        }
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+          for (int i = 0; i < NV; ++i) fma4(to[i], w[u], e[u][i]);
+      }
+    };
+    if (has_post) add_experts(yv);
+    if (has_y || has_post) {
       float inv = nt.gate ? sigmoid_f(__ldcg(nt.gate)) : 1.f;
       if (has_post) {
         float ss = 0.f;
 #pragma unroll
         for (int i = 0; i < NV; ++i) ss += yv[i].x * yv[i].x + yv[i].y * yv[i].y + yv[i].z * yv[i].z + yv[i].w * yv[i].w;
-        inv = 1.0f / sqrtf(block_sum(ss, c.s.red) / (float)W + eps);
+        inv = nt.factor / sqrtf(block_sum(ss, c.s.red) / (float)W + eps);
       }
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
@@ -281,23 +316,7 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
         xv[i].z += yv[i].z * inv * oz; xv[i].w += yv[i].w * inv * ow;
       }
     }
-    for (int k = 0; k < nt.slots; k += 2) {   // two experts' rows in flight
-      float4 e[2][NV];
-      float w[2];
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        w[u] = k + u < nt.slots ? __ldcg(nt.ew + k + u) : 0.f;
-#pragma unroll
-        for (int i = 0; i < NV; ++i) {
-          const int j = (i * kConsumerThreads + tid) * 4;
-          e[u][i] = j < W && k + u < nt.slots ? __ldcg(reinterpret_cast<const float4 *>(nt.experts + (size_t)(k + u) * W + j)) : zero;
-        }
-      }
-#pragma unroll
-      for (int u = 0; u < 2; ++u)
-#pragma unroll
-        for (int i = 0; i < NV; ++i) fma4(xv[i], w[u], e[u][i]);
-    }
+    if (!has_post) add_experts(xv);
     if (nt.add || nt.row) {
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
@@ -312,6 +331,14 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
       for (int i = 0; i < NV; ++i) {
         const int j = (i * kConsumerThreads + tid) * 4;
         if (j < W) *reinterpret_cast<float4 *>(xo + j) = xv[i];
+      }
+    }
+    if (!has_out && d.p[4] != 0) {   // the stream as it is
+      T *out = reinterpret_cast<T *>(d.p[4]) + (size_t)t * d.a[5];
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int j = (i * kConsumerThreads + tid) * 4;
+        if (j < W) store_elt4(out + j, xv[i]);
       }
     }
     if (has_out) {
@@ -412,7 +439,7 @@ static __device__ __noinline__ void run_linear_f32(const Ctx c, const TaskDesc &
       for (int k = tid; k < K; k += kConsumerThreads) xs[(size_t)t * K + k] = __ldcg(x + (size_t)(tb + t) * d.a[4] + k);
     consumer_sync();
     for (int n = n0 + warp; n < n1; n += 8)
-      column_f32(d.p[0], d.a[3], xs, K, n, nt, d.a[6], __int_as_float(d.a[8]), [&](int t, float v) { out[(size_t)(tb + t) * d.a[5] + n] = v; });
+      column_f32(d.p[0], d.a[3], xs, K, n, nt, d.a[6], __int_as_float(d.a[8]), [&](int t, float v) { out[(size_t)(tb + t) * d.a[5] + n] = d.p[3] ? v + bf16_at(d.p[3], n) : v; });
   }
 }
 // Expert projections: the active experts one after the other, the tokens routed to each gathered in shared memory.
@@ -471,8 +498,10 @@ __device__ __forceinline__ int request_of(const KernelParams &P, int t) {
 }
 
 // ---------------------------------------------------------------------------
-// TASK_QKV_APPEND: one warp per (token, head).  q: rotate, normalise, store; k: rotate, normalise, store in the cache
-// page of its position together with the value row.
+// TASK_QKV_APPEND: one warp per (token, head, map).  q: norm, rotate, store; k: norm, rotate, store in the cache page of its
+// position together with the value row.  The norm is an RMS norm with a weight in front of the rotation, or a unit norm behind it.
+// Two maps (differential attention): a cache row holds both maps' keys side by side; a query row, one per map, has zeros where
+// the other map's key lies, so that attention over the whole row gives the map's own scores and a value row serves both.
 // ---------------------------------------------------------------------------
 template <int HYB>
 __device__ __noinline__ void run_qkv_append(const Ctx c, const TaskDesc &d) {
@@ -481,41 +510,51 @@ __device__ __noinline__ void run_qkv_append(const Ctx c, const TaskDesc &d) {
   const int B = active_tokens(P);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int hq = d.a[QA_HQ], hkv = d.a[QA_HKV], dim = d.a[QA_DIM], dimp = d.a[QA_DIMP], vdim = d.a[QA_VDIM], vdimp = d.a[QA_VDIMP];
-  const int rot = d.a[QA_ROT], half = rot >> 1, page = d.a[QA_PAGE];
+  const int rot = d.a[QA_ROT], half = rot >> 1, page = d.a[QA_PAGE], maps = d.a[QA_MAPS];
+  const bool pairs = d.a[QA_PAIRS] != 0;
   const float eps = __int_as_float(d.a[QA_EPS]);
-  const int heads = hq + hkv, first = d.a[QA_T0], tasks = d.a[QA_T1];
+  const int heads = (hq + (d.p[2] ? hkv : 0)) * maps, first = d.a[QA_T0], tasks = d.a[QA_T1];
   for (int item = first * 8 + warp; item < B * heads; item += tasks * 8) {
-    const int t = item / heads, h = item - t * heads;
+    const int t = item / heads, hm = item - t * heads, h = hm / maps, map = hm - h * maps;
     const SeqView s = seq_view(P, request_of(P, t));
     const int pos = s.pos0 + t - s.q0;
     const bool is_q = h < hq;
     const float *src = reinterpret_cast<const float *>(d.p[0]) + (size_t)t * d.a[QA_LDP] +
-                       (is_q ? d.a[QA_QOFF] + h * dim : d.a[QA_KOFF] + (h - hq) * dim);
+                       (is_q ? d.a[QA_QOFF] + hm * dim : d.a[QA_KOFF] + (hm - hq * maps) * dim);
+    const uint64_t norm = is_q ? d.p[6] : d.p[7];
     const size_t trow = (size_t)min(pos, d.a[QA_ROWS] - 1) * half;
     const float *cosT = reinterpret_cast<const float *>(d.p[4]) + trow, *sinT = reinterpret_cast<const float *>(d.p[5]) + trow;
+    auto value = [&](int i) { return norm ? __ldcg(src + i) * bf16_at(norm, i) : __ldcg(src + i); };   // (the norm's factor comes last)
     auto rotated = [&](int i) {
-      const float v = __ldcg(src + i);
+      const float v = value(i);
       if (i >= rot) return v;
-      if (i < half) return v * __ldg(cosT + i) - __ldcg(src + i + half) * __ldg(sinT + i);
-      return v * __ldg(cosT + i - half) + __ldcg(src + i - half) * __ldg(sinT + i - half);
+      const bool lower = pairs ? !(i & 1) : i < half;
+      const int f = pairs ? i >> 1 : (lower ? i : i - half);
+      const float w = value(pairs ? i ^ 1 : (lower ? i + half : i - half));
+      return lower ? v * __ldg(cosT + f) - w * __ldg(sinT + f) : v * __ldg(cosT + f) + w * __ldg(sinT + f);
     };
     float inv = 1.f;
-    if (d.a[QA_NORM]) {
+    if (norm || d.a[QA_NORM]) {
       float ss = 0.f;
-      for (int i = lane; i < dim; i += 32) { const float v = rotated(i); ss += v * v; }
+      for (int i = lane; i < dim; i += 32) { const float v = norm ? __ldcg(src + i) : rotated(i); ss += v * v; }
       inv = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
     }
     T *dst;
     if (is_q) {
-      dst = reinterpret_cast<T *>(d.p[1]) + (size_t)t * d.a[QA_LDQ] + (size_t)h * dimp;
+      dst = reinterpret_cast<T *>(d.p[1]) + (size_t)t * d.a[QA_LDQ] + (size_t)hm * dimp;
+      if (maps > 1)
+        for (int i = lane; i < dimp; i += 32)
+          if (i / dim != map) store_elt(dst + i, 0.f);
     } else {
       const int pg = pos / page;
       const size_t cell = ((size_t)__ldcg(&P.meta.paged_kv_indices[s.kv0 + pg]) * page + (pos - pg * page)) * hkv + (h - hq);
       dst = reinterpret_cast<T *>(d.p[2]) + cell * dimp;
       T *vdst = reinterpret_cast<T *>(d.p[3]) + cell * vdimp;
       const float *vsrc = reinterpret_cast<const float *>(d.p[0]) + (size_t)t * d.a[QA_LDP] + d.a[QA_VOFF] + (h - hq) * vdim;
-      for (int i = lane; i < vdim; i += 32) store_elt(vdst + i, __ldcg(vsrc + i));
+      if (map == 0)
+        for (int i = lane; i < vdim; i += 32) store_elt(vdst + i, __ldcg(vsrc + i));
     }
+    dst += map * dim;
     for (int i = lane; i < dim; i += 32) store_elt(dst + i, rotated(i) * inv);
   }
 }
@@ -586,11 +625,37 @@ template <int HYB>
 __device__ __forceinline__ float sink_logit(const TaskDesc &d, int h) {
   return d.p[4] ? bf16_at(d.p[4], h) * (HYB == HYB_F32 ? 1.0f : 1.4426950408889634f) : 0.f;
 }
-struct AttnOut {   // where a task's rows go
+// Keys of a request in the order the tasks walk them.  Without a window: positions 0, 1, ....  With one, positions that no token
+// of the portion sees are left out: first `kept` positions (a multiple of eight that covers the ones kept for good), then
+// everything from `shift` positions further on (a multiple of eight too, so that eight keys stay in one page).
+struct AttnKeys {
+  int kept, shift, len;   // len: keys in this order
+  __device__ __forceinline__ int pos(int i) const { return i < kept ? i : i + shift; }
+};
+__device__ __forceinline__ AttnKeys attn_keys(const TaskDesc &d, const SeqView &sv) {
+  AttnKeys k;
+  const int window = d.a[XA_WINDOW];
+  const int first = window > 0 ? max(0, sv.pos0 - window + 1) & ~7 : 0;
+  k.kept = min((d.a[XA_KEEP] + 7) & ~7, first);
+  k.shift = first - k.kept;
+  k.len = sv.pos0 + sv.nq - k.shift;
+  return k;
+}
+struct AttnOut {   // where a task's rows go, and the keys
   int hq, G, head, q0, ks, chunk, n_act, vdim, ldo, ocol, srec, rec0;
   float oscale;
-  bool sink;
+  bool sink, f32;
+  AttnKeys keys;
+  int window, keep;   // keys a position sees at most (very large without a window), first positions it sees all the same
+  // Does the row at position p not see the key at position `key` <= p?
+  __device__ __forceinline__ bool outside(int key, int p) const { return p - key >= window && key >= keep; }
 };
+// Element i of an output row that is float32 or of the activation type.
+template <class T>
+__device__ __forceinline__ void store_out(const TaskDesc &d, bool f32, size_t i, float v) {
+  if (f32) reinterpret_cast<float *>(d.p[3])[i] = v;
+  else store_elt(reinterpret_cast<T *>(d.p[3]) + i, v);
+}
 // Partial record of a row (max, sum, then the unnormalised columns) of this task's chunk; the chunks of a row lie side by side.
 __device__ __forceinline__ float *attn_record(const KernelParams &P, const AttnOut &o, int r) {
   return P.attn_scratch + ((size_t)o.rec0 + (size_t)r * o.ks + o.chunk) * o.srec;
@@ -600,9 +665,8 @@ __device__ __forceinline__ float *attn_record(const KernelParams &P, const AttnO
 struct AttnSplit {
   int rows, tiles, parts, ks, per, n_act;   // rows, row tiles, row parts, key chunks at most, keys of a chunk, chunks with keys
 };
-__device__ __forceinline__ AttnSplit attn_split(const SeqView &sv, int G, int NC, int RT) {
+__device__ __forceinline__ AttnSplit attn_split(const SeqView &sv, int len, int G, int NC, int RT) {
   AttnSplit a;
-  const int len = sv.pos0 + sv.nq;
   a.rows = sv.nq * G;
   a.tiles = (a.rows + RT - 1) / RT;
   a.parts = min(NC, a.tiles);
@@ -623,10 +687,10 @@ __device__ __forceinline__ void attn_emit_row(const Ctx &c, const TaskDesc &d, c
     const float w = m == -INFINITY ? 0.f : exp_dom<HYB>(m - M);
     const float L = l * w + (o.sink ? exp_dom<HYB>(sk - M) : 0.f);
     const float f = L > 0.f ? w / L * o.oscale : 0.f;
-    T *out = reinterpret_cast<T *>(d.p[3]) + (size_t)tok * o.ldo + o.ocol + (size_t)hq_idx * o.vdim;
+    const size_t out = (size_t)tok * o.ldo + o.ocol + (size_t)hq_idx * o.vdim;
     for (int j0 = 0; j0 < o.vdim; j0 += 32) {   // (val may shuffle: the whole warp calls it)
       const float v = val(j0 + lane);
-      if (j0 + lane < o.vdim) store_elt(out + j0 + lane, v * f);
+      if (j0 + lane < o.vdim) store_out<T>(d, o.f32, out + j0 + lane, v * f);
     }
   } else {
     float *rec = attn_record(c.P, o, r);
@@ -688,36 +752,38 @@ __device__ __noinline__ void attn_merge(const Ctx c, const TaskDesc &d, const At
       for (int u = 0; u < 16; ++u) acc = fmaf(__shfl_sync(0xffffffffu, w, 16 + u), x2[u], acc);
     }
     if (j < o.vdim)
-      store_elt(reinterpret_cast<T *>(d.p[3]) + (size_t)tok * o.ldo + o.ocol + (size_t)hq_idx * o.vdim + j, acc * f);
+      store_out<T>(d, o.f32, (size_t)tok * o.ldo + o.ocol + (size_t)hq_idx * o.vdim + j, acc * f);
   }
 }
 
 // What a warp's 16-row tile needs to know of its queries.
 struct AttnRows {
   float scale, cap, cap2;
-  int kend;         // keys of the task
-  int p_lo, p_hi;   // last key this lane's two rows see
-  int p_all;        // keys up to here are seen by every row of the tile
+  int kend;         // end of the task's keys
+  int p_lo, p_hi;   // positions of this lane's two rows
+  int p_all;        // keys up to here are not ahead of any row of the tile
+  int p_far;        // keys from here on are in the window of every row
   bool two;         // rows 8 .. 15 of the tile hold queries
 };
-__device__ __forceinline__ AttnRows attn_rows(const TaskDesc &d, const SeqView &sv, int G, int first, int n, int kend) {
+__device__ __forceinline__ AttnRows attn_rows(const TaskDesc &d, const SeqView &sv, const AttnOut &ao, int first, int n, int kend) {
   AttnRows w;
   w.scale = __int_as_float(d.a[XA_SCALE]);
   w.cap = __int_as_float(d.a[XA_CAP]);
   w.cap2 = w.cap > 0.f ? 2.0f * 1.4426950408889634f / w.cap : 0.f;
   w.kend = kend;
-  const int r = first + ((threadIdx.x & 31) >> 2);
+  const int r = first + ((threadIdx.x & 31) >> 2), G = ao.G;
   w.p_lo = sv.pos0 + r / G;
   w.p_hi = sv.pos0 + (r + 8) / G;
-  w.p_all = min(sv.pos0 + first / G, kend - 1);
+  w.p_all = sv.pos0 + first / G;
+  w.p_far = sv.pos0 + (first + n - 1) / G - ao.window + 1;
   w.two = n > 8;
   return w;
 }
 // Eight keys (rows at kaddr / vaddr, this lane's ldmatrix addresses) against a 16-row query tile: scores, online softmax,
-// P V.  key0 is below w.kend.
+// P V.  The first is number key0 (below w.kend) of the request's keys and lies at position `at`.
 template <int D, int ON, bool TWO>
-__device__ __forceinline__ void attn_octet(const AttnRows &w, const uint32_t (&qf)[TWO ? 1 : D / 16][2], uint32_t qa, uint32_t kaddr,
-                                           uint32_t vaddr, int key0, float (&m_run)[2], float (&l_run)[2], float (&o)[ON / 8][4]) {
+__device__ __forceinline__ void attn_octet(const AttnRows &w, const AttnOut &ao, const uint32_t (&qf)[TWO ? 1 : D / 16][2], uint32_t qa, uint32_t kaddr,
+                                           uint32_t vaddr, int key0, int at, float (&m_run)[2], float (&l_run)[2], float (&o)[ON / 8][4]) {
   float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
   for (int kk = 0; kk < D / 32; ++kk) {
@@ -742,12 +808,12 @@ __device__ __forceinline__ void attn_octet(const AttnRows &w, const uint32_t (&q
     if (e >= 2 && !(TWO && w.two)) { s[e] = -INFINITY; continue; }
     s[e] = attn_score<HYB_BF16>(s[e] + s2[e], w.scale, w.cap, w.cap2);
   }
-  if (key0 + 7 > w.p_all) {
-    const int key = key0 + 2 * (threadIdx.x & 3);
+  if (at + 7 > w.p_all || key0 + 8 > w.kend || at < w.p_far) {
+    const int off = 2 * (threadIdx.x & 3);
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int kpos = key + (e & 1);
-      if (kpos >= w.kend || kpos > (e < 2 ? w.p_lo : w.p_hi)) s[e] = -INFINITY;
+      const int o = off + (e & 1), p = e < 2 ? w.p_lo : w.p_hi;
+      if (key0 + o >= w.kend || at + o > p || ao.outside(at + o, p)) s[e] = -INFINITY;
     }
   }
   mx[0] = fmaxf(s[0], s[1]);
@@ -819,7 +885,8 @@ __device__ __noinline__ void ext_attention_stream(const Ctx c, const TaskDesc &d
   constexpr int PITCH = D * 2 + 16, STEP = 16 * PITCH, PIECES = D / 8, RSTEP = 32 / PIECES;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int nstg = d.a[XA_STAGES], page = d.a[XA_PAGE];
-  const int kend = min(k1, sv.pos0 + (row0 + nrow - 1) / ao.G + 1);
+  const AttnKeys keys = ao.keys;
+  const int kend = min(k1, sv.pos0 + (row0 + nrow - 1) / ao.G + 1 - keys.shift);
   const int noct = kend > k0 ? (kend - k0 + 7) >> 3 : 0, mine = noct > warp ? (noct - warp + 7) >> 3 : 0;
   uint8_t *qs = c.s.xtile;                                                      // [16][PITCH]
   const uint32_t ring = smem_u32(qs) + (16 + warp * nstg * 16) * PITCH;         // this warp's stages: eight K rows, then eight V rows
@@ -832,10 +899,10 @@ __device__ __noinline__ void ext_attention_stream(const Ctx c, const TaskDesc &d
   const int32_t *pages = c.P.meta.paged_kv_indices + sv.kv0;
   // page of the next octet to request, looked up one request ahead of its use
   int pos = k0 + warp * 8;
-  int pid = pos < kend ? __ldcg(pages + pos / page) : 0;
+  int pid = pos < kend ? __ldcg(pages + keys.pos(pos) / page) : 0;
   auto issue = [&](int slot) {
     if (pos < kend) {
-      const uint32_t row = (uint32_t)pid * page + pos % page;
+      const uint32_t row = (uint32_t)pid * page + keys.pos(pos) % page;
       const uint32_t dst = ring + slot * STEP + rl * PITCH + piece * 16;
       const int left = kend - pos - rl;   // rows of this lane's stride that exist
 #pragma unroll
@@ -848,7 +915,7 @@ __device__ __noinline__ void ext_attention_stream(const Ctx c, const TaskDesc &d
         else asm volatile("st.shared.v4.b32 [%0], {%1,%1,%1,%1};" ::"r"(vd), "r"(0) : "memory");
       }
       pos += 64;
-      pid = pos < kend ? __ldcg(pages + pos / page) : 0;
+      pid = pos < kend ? __ldcg(pages + keys.pos(pos) / page) : 0;
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -866,7 +933,7 @@ __device__ __noinline__ void ext_attention_stream(const Ctx c, const TaskDesc &d
   }
   consumer_sync();
   stamp(c, task, 0);
-  const AttnRows w = attn_rows(d, sv, ao.G, row0, nrow, kend);
+  const AttnRows w = attn_rows(d, sv, ao, row0, nrow, kend);
   const uint32_t qa = smem_u32(qs) + (uint32_t)((lane & 15) * PITCH + (lane >> 4) * 16);
   uint32_t qf[TWO ? 1 : D / 16][2];   // rows 0 .. 7 only: two of a fragment's four registers
   if (!TWO) {
@@ -890,7 +957,8 @@ __device__ __noinline__ void ext_attention_stream(const Ctx c, const TaskDesc &d
     __syncwarp();   // the octet has landed for every lane, and every lane is done with the slot refilled next
     issue(slot == 0 ? nstg - 1 : slot - 1);
     const uint32_t ka = ring + slot * STEP + lane_off;
-    attn_octet<D, D, TWO>(w, qf, qa, ka, ka + 8 * PITCH, k0 + (warp + 8 * i) * 8, m_run, l_run, o);
+    const int key0 = k0 + (warp + 8 * i) * 8;
+    attn_octet<D, D, TWO>(w, ao, qf, qa, ka, ka + 8 * PITCH, key0, keys.pos(key0), m_run, l_run, o);
     if (++slot == nstg) slot = 0;
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -931,7 +999,8 @@ __device__ __noinline__ void ext_attention_decode(const Ctx c, const TaskDesc &d
   constexpr int PITCH = D * 2 + 16, OCT = 8 * PITCH, PIECES = D / 8, RSTEP = 32 / PIECES, STEPS = 2;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int page = d.a[XA_PAGE];
-  const int kend = min(k1, sv.pos0 + (row0 + nrow - 1) / ao.G + 1);
+  const AttnKeys keys = ao.keys;
+  const int kend = min(k1, sv.pos0 + (row0 + nrow - 1) / ao.G + 1 - keys.shift);
   const int nstep = kend > k0 ? (kend - k0 + 15) >> 4 : 0, mine = nstep > warp ? (nstep - warp + 7) >> 3 : 0;
   uint8_t *qs = c.s.xtile;                                                   // [16][PITCH]
   // this warp's steps: sixteen K rows, then sixteen V rows
@@ -943,14 +1012,14 @@ __device__ __noinline__ void ext_attention_decode(const Ctx c, const TaskDesc &d
   const uint4 *vg = reinterpret_cast<const uint4 *>(d.p[2]) + ao.head * (d.a[XA_VDIMP] >> 3) + piece + rl * vrow;
   const int32_t *pages = c.P.meta.paged_kv_indices + sv.kv0;
   int pos = k0 + warp * 16;
-  auto page_of = [&](int key) { return key < kend ? __ldcg(pages + key / page) : 0; };
+  auto page_of = [&](int key) { return key < kend ? __ldcg(pages + keys.pos(key) / page) : 0; };
   int pid0 = page_of(pos), pid1 = page_of(pos + 8);   // of the next step to request
   auto issue = [&](int slot) {
     if (pos < kend) {
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
         const int p0 = pos + h * 8, left = kend - p0 - rl;
-        const uint32_t row = (uint32_t)(h ? pid1 : pid0) * page + p0 % page;
+        const uint32_t row = (uint32_t)(h ? pid1 : pid0) * page + keys.pos(p0) % page;
         const uint32_t dst = ring + slot * 4 * OCT + h * OCT + rl * PITCH + piece * 16;
 #pragma unroll
         for (int i = 0; i < 8 / RSTEP; ++i) {
@@ -989,9 +1058,10 @@ __device__ __noinline__ void ext_attention_decode(const Ctx c, const TaskDesc &d
 #pragma unroll
   for (int kk = 0; kk < D / 16; ++kk)
     ldmatrix_x2(qf[kk], smem_u32(qs) + (uint32_t)((lane & 7) * PITCH + ((lane >> 3) & 1) * 16 + kk * 32));
-  // this lane's two queries (columns of S^T) and the last key each sees
+  // this lane's two queries (columns of S^T), their positions, and the range of keys that needs no mask
   const int q0 = row0 + 2 * (lane & 3);
-  const int p_a = sv.pos0 + q0 / ao.G, p_b = sv.pos0 + (q0 + 1) / ao.G, p_all = min(sv.pos0 + row0 / ao.G, kend - 1);
+  const int p_a = sv.pos0 + q0 / ao.G, p_b = sv.pos0 + (q0 + 1) / ao.G, p_all = sv.pos0 + row0 / ao.G;
+  const int p_far = sv.pos0 + (row0 + nrow - 1) / ao.G - ao.window + 1;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
   float o[D / 16][4];
 #pragma unroll
@@ -1016,11 +1086,12 @@ __device__ __noinline__ void ext_attention_decode(const Ctx c, const TaskDesc &d
     }
 #pragma unroll
     for (int e = 0; e < 4; ++e) s[e] = attn_score<HYB_BF16>(s[e] + s2[e], scale, cap, cap2);
-    if (key0 + 15 > p_all) {   // e: key g + 8 (e / 2), query 2 q + (e & 1)
+    const int at0 = keys.pos(key0), at1 = keys.pos(key0 + 8);
+    if (at1 + 7 > p_all || key0 + 16 > kend || at0 < p_far) {   // e: key g + 8 (e / 2), query 2 q + (e & 1)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int key = key0 + (lane >> 2) + (e >> 1) * 8;
-        if (key >= kend || key > ((e & 1) ? p_b : p_a)) s[e] = -INFINITY;
+        const int at = (e >> 1 ? at1 : at0) + (lane >> 2), p = (e & 1) ? p_b : p_a;
+        if (key0 + (lane >> 2) + (e >> 1) * 8 >= kend || at > p || ao.outside(at, p)) s[e] = -INFINITY;
       }
     }
     float x0 = fmaxf(s[0], s[2]), x1 = fmaxf(s[1], s[3]);
@@ -1105,8 +1176,9 @@ __device__ __noinline__ void ext_attention_mma(const Ctx c, const TaskDesc &d, c
   const int kp = dimp >> 3, vp = vdimp >> 3;   // 16-byte pieces of a row
   // eight consecutive keys lie in one page when pages hold a multiple of eight positions
   const int ncell = (page & 7) == 0 && k1 - k0 <= 8 * kXaCells ? (k1 - k0 + 7) >> 3 : 0;
-  auto cell_row = [&](int key) {
-    const int pg = key / page;
+  const AttnKeys keys = ao.keys;
+  auto cell_row = [&](int i) {
+    const int key = keys.pos(i), pg = key / page;
     return __ldcg(&P.meta.paged_kv_indices[sv.kv0 + pg]) * page + (key - pg * page);
   };
   for (int i = tid; i < ncell; i += kConsumerThreads) cells[i] = cell_row(k0 + 8 * i);
@@ -1116,7 +1188,7 @@ __device__ __noinline__ void ext_attention_mma(const Ctx c, const TaskDesc &d, c
     const int WM = mt <= 1 ? 1 : (mt <= 2 ? 2 : (mt <= 4 ? 4 : WMAX));
     const int WK = WMAX / WM;                                      // <= NSUB
     const int wn = warp % WN, w2 = warp / WN, wm = w2 % WM, wk = w2 / WM;
-    const int kend = min(k1, sv.pos0 + (rb + nrow - 1) / G + 1);   // keys past the last row's position are not needed
+    const int kend = min(k1, sv.pos0 + (rb + nrow - 1) / G + 1 - keys.shift);   // keys past the last row's position are not needed
     if (rb > row0) consumer_sync();
     for (int i = tid; i < WM * 16 * (D / 8); i += kConsumerThreads) {
       const int r = i / (D / 8), p = i - r * (D / 8);
@@ -1153,7 +1225,7 @@ __device__ __noinline__ void ext_attention_mma(const Ctx c, const TaskDesc &d, c
     for (int i = 0; i < ON / 8; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
-    const AttnRows w = attn_rows(d, sv, G, rb + wm * 16, nrow - wm * 16, kend);
+    const AttnRows w = attn_rows(d, sv, ao, rb + wm * 16, min(nrow - wm * 16, 16), kend);
     const int ntiles = kend > k0 ? (kend - k0 + KEYS - 1) / KEYS : 0;
     consumer_sync();   // queries and cells
     stamp(c, task, 0);
@@ -1183,7 +1255,7 @@ __device__ __noinline__ void ext_attention_mma(const Ctx c, const TaskDesc &d, c
       for (int j = wk; j < NSUB; j += WK) {
         const int key0 = base + j * 8;
         if (key0 >= kend) break;
-        attn_octet<D, ON, true>(w, qf, qa, kt + (uint32_t)(j * 8 * PITCH), vt + (uint32_t)(j * 8 * PITCH), key0, m_run, l_run, o);
+        attn_octet<D, ON, true>(w, ao, qf, qa, kt + (uint32_t)(j * 8 * PITCH), vt + (uint32_t)(j * 8 * PITCH), key0, keys.pos(key0), m_run, l_run, o);
       }
     }
     consumer_sync();   // the stages become the combine area
@@ -1496,12 +1568,13 @@ static __device__ __noinline__ void ext_attention_f32(const Ctx c, const TaskDes
   float *q = reinterpret_cast<float *>(c.s.xtile) + warp * dimp;
   const float *qg = reinterpret_cast<const float *>(d.p[0]);
   const float *kg = reinterpret_cast<const float *>(d.p[1]), *vg = reinterpret_cast<const float *>(d.p[2]);
+  const AttnKeys keys = ao.keys;
   auto cell_of = [&](int key) {
     const int pg = key / page;
     return ((size_t)__ldcg(&P.meta.paged_kv_indices[sv.kv0 + pg]) * page + (key - pg * page)) * hkv + ao.head;
   };
   for (int r = row0 + warp; r < rows; r += 8) {
-    const int kend = min(k1, sv.pos0 + r / G + 1);
+    const int pos = sv.pos0 + r / G, kend = min(k1, pos + 1 - keys.shift);
     __syncwarp();
     for (int i = lane; i < dimp; i += 32) q[i] = __ldcg(qg + (size_t)(sv.q0 + r / G) * d.a[XA_LDQ] + (size_t)(ao.head * G + r % G) * dimp + i);
     __syncwarp();
@@ -1509,11 +1582,12 @@ static __device__ __noinline__ void ext_attention_f32(const Ctx c, const TaskDes
 #pragma unroll
     for (int i = 0; i < NO; ++i) o[i] = 0.f;
     for (int kb = k0; kb < kend; kb += 32) {
-      const int key = kb + lane;
+      const int at = keys.pos(kb + lane);
+      const bool seen = kb + lane < kend && !ao.outside(at, pos);
       float s = -INFINITY;
       size_t cell = 0;
-      if (key < kend) {
-        cell = cell_of(key);
+      if (seen) {
+        cell = cell_of(at);
         const float4 *kr = reinterpret_cast<const float4 *>(kg + cell * dimp);
         float dot = 0.f;
         for (int i = 0; i < dimp >> 2; ++i) {
@@ -1523,7 +1597,8 @@ static __device__ __noinline__ void ext_attention_f32(const Ctx c, const TaskDes
         s = attn_score<HYB_F32>(dot, scale, cap, 0.f);
       }
       const float mn = fmaxf(m, warp_max(s));
-      const float corr = expf(m - mn), p = key < kend ? expf(s - mn) : 0.f;
+      if (mn == -INFINITY) continue;   // none of these keys is seen
+      const float corr = expf(m - mn), p = seen ? expf(s - mn) : 0.f;
       l = l * corr + warp_sum(p);
       m = mn;
 #pragma unroll
@@ -1566,14 +1641,18 @@ __device__ __forceinline__ void run_ext_attention(const Ctx &c, const TaskDesc &
   ao.srec = d.a[XA_SREC];
   ao.oscale = __int_as_float(d.a[XA_OSCALE]);
   ao.sink = d.a[XA_SINK] != 0;
-  const AttnSplit sp = attn_split(sv, ao.G, NC, RT);
+  ao.f32 = d.a[XA_OUTF32] != 0;
+  ao.window = d.a[XA_WINDOW] > 0 ? d.a[XA_WINDOW] : 1 << 30;
+  ao.keep = d.a[XA_KEEP];
+  ao.keys = attn_keys(d, sv);
+  const AttnSplit sp = attn_split(sv, ao.keys.len, ao.G, NC, RT);
   const int part = d.a[XA_CHUNK] % sp.parts;
   ao.chunk = d.a[XA_CHUNK] / sp.parts;
   ao.ks = sp.ks;
   ao.n_act = sp.n_act;
   ao.rec0 = (d.a[XA_SLOT] * d.a[XA_HKV] + ao.head) * RT * NC;
   if (ao.chunk >= ao.n_act) return;   // (n_act <= ks: this also ends the tasks beyond parts * ks)
-  const int k0 = ao.chunk * sp.per, k1 = min(sv.pos0 + sv.nq, k0 + sp.per);
+  const int k0 = ao.chunk * sp.per, k1 = min(ao.keys.len, k0 + sp.per);
   const int row0 = sp.tiles * part / sp.parts * RT, row1 = min(sp.rows, sp.tiles * (part + 1) / sp.parts * RT);
   if (HYB == HYB_F32) {
     ext_attention_f32(c, d, sv, ao, k0, k1, row0, row1);
@@ -1629,7 +1708,7 @@ __device__ __noinline__ void run_attn_merge(const Ctx c, const TaskDesc &d) {
     const int row = item / cols, j = (item - row * cols) * 128 + lane * 4, t = row / hq, h = row - t * hq;
     const int k = request_of(P, t);
     const SeqView sv = seq_view(P, k);
-    const AttnSplit a = attn_split(sv, G, NC, RT);
+    const AttnSplit a = attn_split(sv, attn_keys(d, sv).len, G, NC, RT);
     if (a.n_act == 1) continue;   // the attention task wrote the output
     const int r = (t - sv.q0) * G + h % G;
     const float *rec = P.attn_scratch + ((size_t)(k * hkv + h / G) * RT * NC + (size_t)r * a.ks) * srec;
@@ -1648,11 +1727,46 @@ __device__ __noinline__ void run_attn_merge(const Ctx c, const TaskDesc &d) {
       const float4 x = j < vdim ? __ldcg(reinterpret_cast<const float4 *>(rec + (size_t)u * srec + kXaRecHead + j)) : make_float4(0.f, 0.f, 0.f, 0.f);
       acc.x = fmaf(wu, x.x, acc.x); acc.y = fmaf(wu, x.y, acc.y); acc.z = fmaf(wu, x.z, acc.z); acc.w = fmaf(wu, x.w, acc.w);
     }
-    T *out = reinterpret_cast<T *>(d.p[3]) + (size_t)t * d.a[XA_LDO] + d.a[XA_OCOL] + (size_t)h * vdim + j;
+    const size_t out = (size_t)t * d.a[XA_LDO] + d.a[XA_OCOL] + (size_t)h * vdim + j;
     const float o[4] = {acc.x * f, acc.y * f, acc.z * f, acc.w * f};
 #pragma unroll
     for (int e = 0; e < 4; ++e)
-      if (j + e < vdim) store_elt(out + e, o[e]);
+      if (j + e < vdim) store_out<T>(d, d.a[XA_OUTF32] != 0, out + e, o[e]);
+  }
+}
+
+// ---------------------------------------------------------------------------
+// TASK_DIFF_COMBINE (Ye et al., "Differential Transformer"): per token and head, the difference of the two maps' outputs, divided
+// by its root mean square over the head's values, times a factor.  One warp per (token, head).
+// ---------------------------------------------------------------------------
+template <int HYB>
+__device__ __noinline__ void run_diff_combine(const Ctx c, const TaskDesc &d) {
+  typedef typename HybElt<HYB>::T T;
+  const int B = active_tokens(c.P), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int H = d.a[2], vdim = d.a[3];
+  const float lambda = __int_as_float(d.a[6]), factor = __int_as_float(d.a[7]), eps = __int_as_float(d.a[8]);
+  for (int item = d.a[0] * 8 + warp; item < B * H; item += d.a[1] * 8) {
+    const int t = item / H, h = item - t * H;
+    const float *a = reinterpret_cast<const float *>(d.p[0]) + (size_t)t * d.a[4] + (size_t)2 * h * vdim;
+    T *out = reinterpret_cast<T *>(d.p[1]) + (size_t)t * d.a[5] + (size_t)h * vdim;
+    float ss = 0.f;
+    if (vdim <= 256) {   // the row in registers, all loads in flight
+      float x[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int j = i * 32 + lane;
+        x[i] = j < vdim ? __ldcg(a + j) - lambda * __ldcg(a + vdim + j) : 0.f;
+        ss += x[i] * x[i];
+      }
+      const float f = factor / sqrtf(warp_sum(ss) / (float)vdim + eps);
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (i * 32 + lane < vdim) store_elt(out + i * 32 + lane, x[i] * f);
+      continue;
+    }
+    for (int j = lane; j < vdim; j += 32) { const float x = __ldcg(a + j) - lambda * __ldcg(a + vdim + j); ss += x * x; }
+    const float f = factor / sqrtf(warp_sum(ss) / (float)vdim + eps);
+    for (int j = lane; j < vdim; j += 32) store_elt(out + j, (__ldcg(a + j) - lambda * __ldcg(a + vdim + j)) * f);
   }
 }
 
@@ -1664,7 +1778,9 @@ __device__ __noinline__ void run_attn_merge(const Ctx c, const TaskDesc &d) {
 // needs (the tokens of its run, the ones before them, carried ones where a request starts) in registers before anything
 // is stored.
 constexpr int kConvWindow = 4;
+template <int HYB>
 __device__ __forceinline__ void short_conv_window(const Ctx &c, const TaskDesc &d, const TokenRec *rec, int B) {
+  typedef typename HybElt<HYB>::T T;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int C = d.a[2], taps = d.a[3], hist = taps - 1;
   const float *in = reinterpret_cast<const float *>(d.p[0]) + d.a[5];
@@ -1707,6 +1823,7 @@ __device__ __forceinline__ void short_conv_window(const Ctx &c, const TaskDesc &
       for (int j = 0; j < kConvWindow; ++j) v = fmaf(w[j + 1], prev[u][j], v);
       if (d.a[7] == 1) v = v * sigmoid_f(v);
       out[(size_t)(t0 + u) * d.a[6] + ch] = v;
+      if (d.p[6]) store_elt(reinterpret_cast<T *>(d.p[6]) + (size_t)(t0 + u) * d.a[8] + ch, v);
       if (r.flags & 2) {   // the last `hist` inputs, oldest first
 #pragma unroll
         for (int j = 0; j < kConvWindow; ++j)
@@ -1716,14 +1833,16 @@ __device__ __forceinline__ void short_conv_window(const Ctx &c, const TaskDesc &
   }
 }
 
-static __device__ __noinline__ void run_short_conv(const Ctx c, const TaskDesc &d) {
+template <int HYB>
+__device__ __noinline__ void run_short_conv(const Ctx c, const TaskDesc &d) {
+  typedef typename HybElt<HYB>::T T;
   const KernelParams &P = c.P;
   const int B = active_tokens(P);
   if (B <= 0) return;
   TokenRec *rec = reinterpret_cast<TokenRec *>(c.s.xtile);
   token_map(P, B, rec, reinterpret_cast<int *>(c.s.xtile + kTokenMapBytes));
   if (d.a[3] <= kConvWindow + 1) {
-    short_conv_window(c, d, rec, B);
+    short_conv_window<HYB>(c, d, rec, B);
     return;
   }
   const int c0 = d.a[0], nc = d.a[1] - c0, C = d.a[2], taps = d.a[3], hist = taps - 1;
@@ -1743,6 +1862,7 @@ static __device__ __noinline__ void run_short_conv(const Ctx c, const TaskDesc &
     for (int j = 0; j < taps; ++j) v = fmaf(bf16_at(d.p[2], (size_t)ch * taps + j), input(r, t - hist + j, ch, bias), v);
     if (d.a[7] == 1) v = v * sigmoid_f(v);
     out[(size_t)t * d.a[6] + ch] = v;
+    if (d.p[6]) store_elt(reinterpret_cast<T *>(d.p[6]) + (size_t)t * d.a[8] + ch, v);
   }
   consumer_sync();   // the carried inputs have been read
   for (int i = threadIdx.x; i < B * nc; i += kConsumerThreads) {
@@ -1995,6 +2115,189 @@ __device__ __noinline__ void run_rglru(const Ctx c, const TaskDesc &d) {
       store_elt(outp + (size_t)(tb + t) * d.a[GL_LDO] + d.a[GL_OCOL] + gch + ch, S * gelu_tanh_f(yp + chp[192 + ch]) * oscale);
     }
     consumer_sync();
+  }
+}
+
+// ---------------------------------------------------------------------------
+// TASK_SELECTIVE_SCAN (Gu and Dao, "Mamba: Linear-Time Sequence Modeling with Selective State Spaces"): a channel range of every
+// request.  Per channel c and state n
+//   dt = softplus(W_dt low + b),  S = exp(-dt exp(A_log)) S + dt u B,  y = (sum_n S C + D u) * silu(z)
+// SS_LANES neighbouring lanes share a channel, four states each, so that a block walks 256 / SS_LANES channels at a time through the
+// tokens of the batch; the step sizes' low-rank product is part of the task.  A request's state enters at its first token of the
+// batch and is written back at its last; every thread copies its own piece of the states to come into its own cells of a ring.
+// ---------------------------------------------------------------------------
+// Adds columns [r0, r0 + rn) of the low-rank product to dts [B][CP] (B <= 8: a warp takes a channel, its lanes the columns; else a
+// thread takes a channel and eight tokens).  low: [B][rn] in shared memory, rows of `pitch` floats.
+__device__ __forceinline__ void scan_steps(const TaskDesc &d, const float *low, int pitch, float *dts, int CP, int cb, int nc, int B, int r0, int rn) {
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rank = d.a[SS_RANK];
+  const bool vec = (rank & 7) == 0 && (d.p[3] & 15) == 0;   // rows of whole 16-byte pieces
+  auto eight = [&](size_t row, int k, float (&w)[8]) {      // weights k .. k + 7 of the chunk, zeros past its end
+    if (vec) {
+      const uint4 v = __ldg(reinterpret_cast<const uint4 *>(d.p[3] + 2 * (row * rank + r0 + k)));
+      const uint32_t p[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+      for (int e = 0; e < 8; ++e) w[e] = e & 1 ? bf16_hi(p[e >> 1]) : bf16_lo(p[e >> 1]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) w[e] = k + e < rn ? bf16_at(d.p[3], row * rank + r0 + k + e) : 0.f;
+    }
+  };
+  if (B <= 8) {
+    for (int c = warp; c < nc; c += 8) {
+      float acc[8];
+#pragma unroll
+      for (int u = 0; u < 8; ++u) acc[u] = 0.f;
+      for (int k = lane * 8; k < rn; k += 256) {
+        float w[8];
+        eight(cb + c, k, w);
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+          if (u >= B) break;
+#pragma unroll
+          for (int e = 0; e < 8; ++e) acc[u] = fmaf(w[e], low[u * pitch + k + e], acc[u]);
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < 8; ++u) {
+        if (u >= B) break;
+        const float v = warp_sum(acc[u]);
+        if (lane == 0) dts[u * CP + c] += v;
+      }
+    }
+    return;
+  }
+  for (int it = tid; it < nc * ((B + 7) >> 3); it += kConsumerThreads) {
+    const int c = it % nc, t0 = it / nc * 8;
+    float acc[8];
+#pragma unroll
+    for (int u = 0; u < 8; ++u) acc[u] = 0.f;
+    for (int k = 0; k < rn; k += 8) {
+      float w[8];
+      eight(cb + c, k, w);
+#pragma unroll
+      for (int u = 0; u < 8; ++u) {
+        const float4 *x = reinterpret_cast<const float4 *>(low + min(t0 + u, B - 1) * pitch + k);
+        const float4 a = x[0], b = x[1];
+        acc[u] = fmaf(w[3], a.w, fmaf(w[2], a.z, fmaf(w[1], a.y, fmaf(w[0], a.x, acc[u]))));
+        acc[u] = fmaf(w[7], b.w, fmaf(w[6], b.z, fmaf(w[5], b.y, fmaf(w[4], b.x, acc[u]))));
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < 8; ++u)
+      if (t0 + u < B) dts[(t0 + u) * CP + c] += acc[u];
+  }
+}
+
+template <int HYB>
+__device__ __noinline__ void run_selective_scan(const Ctx c, const TaskDesc &d, int task) {
+  typedef typename HybElt<HYB>::T T;
+  const KernelParams &P = c.P;
+  const int B = active_tokens(P);
+  if (B <= 0) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int C = d.a[SS_C], rank = d.a[SS_RANK], N = d.a[SS_N], NP = d.a[SS_NP], LPC = d.a[SS_LANES], CP = kConsumerThreads / LPC;
+  const int mbr = P.max_num_batched_requests, RC = min(kScanRank, (rank + 7) & ~7);
+  // shared memory
+  TokenRec *rec = reinterpret_cast<TokenRec *>(c.s.xtile);
+  int *qo = reinterpret_cast<int *>(c.s.xtile + kTokenMapBytes);
+  int *seqs = qo + ((mbr + 4) & ~3);                                          // [64] state slot of the batch's requests in order, -1: starts from zeros
+  float4 *ring = reinterpret_cast<float4 *>(seqs + kMaxLinearTokens) + tid;   // [kScanRing][256], this thread's cells
+  float *bc = reinterpret_cast<float *>(ring - tid + kScanRing * kConsumerThreads);   // [B][2 NP]: B, C
+  float *low = bc + B * 2 * NP;                                               // [B][RC]
+  float *dts = low + B * RC;                                                  // [B][CP] step sizes
+  float *us = dts + B * CP;                                                   // [B][CP] inputs, then read-outs
+  float *state = reinterpret_cast<float *>(wide_arg(d, SS_STATE));
+  token_map(P, B, rec, qo);
+  if (warp == 0) {
+    const int f0 = lane < B ? rec[lane].flags : 0, f1 = 32 + lane < B ? rec[32 + lane].flags : 0;
+    const unsigned b0 = __ballot_sync(0xffffffffu, f0 & 1), b1 = __ballot_sync(0xffffffffu, f1 & 1), before = (1u << lane) - 1u;
+    seqs[lane] = seqs[32 + lane] = -1;
+    __syncwarp();
+    if (f0 & 1) seqs[__popc(b0 & before)] = f0 & 4 ? -1 : rec[lane].slot;
+    if (f1 & 1) seqs[__popc(b0) + __popc(b1 & before)] = f1 & 4 ? -1 : rec[32 + lane].slot;
+  }
+  for (int i = tid; i < B * 2 * NP; i += kConsumerThreads) {
+    const int t = i / (2 * NP), j = i - t * 2 * NP, n = j % NP;
+    bc[i] = n < N ? __ldcg(reinterpret_cast<const float *>(d.p[1]) + (size_t)t * d.a[SS_LDL] + rank + (j < NP ? n : N + n)) : 0.f;
+  }
+  consumer_sync();
+  stamp(c, task, 0);
+  const int q = tid % LPC, ch = tid / LPC, n0 = 4 * q;
+  for (int cb = d.a[SS_C0]; cb < d.a[SS_C1]; cb += CP) {
+    const int nc = min(CP, d.a[SS_C1] - cb);
+    const bool on = ch < nc && n0 < NP;       // this thread holds states
+    float *mine = state + (size_t)(cb + ch) * NP + n0;
+    auto fetch = [&](int j) {
+      const int slot = j < kMaxLinearTokens ? seqs[j] : -1;
+      if (on && slot >= 0) cp_async16(smem_u32(ring + (j % kScanRing) * kConsumerThreads), mine + (size_t)slot * C * NP);
+      asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+#pragma unroll
+    for (int j = 0; j < kScanRing - 1; ++j) fetch(j);
+    float4 A = make_float4(0.f, 0.f, 0.f, 0.f);
+    float D = 0.f;
+    if (on) {
+      float *a = reinterpret_cast<float *>(&A);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) a[e] = n0 + e < N ? -expf(bf16_at(d.p[5], (size_t)(cb + ch) * N + n0 + e)) : 0.f;
+      D = bf16_at(d.p[6], cb + ch);
+    }
+    // step sizes and inputs
+    for (int i = tid; i < B * nc; i += kConsumerThreads) {
+      const int t = i / nc, k = i - t * nc;
+      us[t * CP + k] = __ldcg(reinterpret_cast<const float *>(d.p[0]) + (size_t)t * d.a[SS_LDU] + cb + k);
+      dts[t * CP + k] = bf16_at(d.p[4], cb + k);
+    }
+    for (int r0 = 0; r0 < rank; r0 += RC) {
+      const int rn = min(RC, rank - r0);
+      for (int t = warp; t < B; t += 8)
+        for (int k = lane; k < RC; k += 32) low[t * RC + k] = k < rn ? __ldcg(reinterpret_cast<const float *>(d.p[1]) + (size_t)t * d.a[SS_LDL] + r0 + k) : 0.f;
+      consumer_sync();
+      scan_steps(d, low, RC, dts, CP, cb, nc, B, r0, rn);
+      consumer_sync();
+    }
+    for (int i = tid; i < B * nc; i += kConsumerThreads) {
+      const int t = i / nc, k = t * CP + i - t * nc;
+      dts[k] = softplus_f(dts[k]);
+    }
+    consumer_sync();
+    stamp(c, task, 1);
+    // the recurrence: lanes of a channel meet in the read-out only
+    float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
+    int seq = 0;
+    for (int t = 0; t < B; ++t) {
+      const int flags = rec[t].flags;
+      if (flags & 1) {
+        fetch(seq + kScanRing - 1);
+        asm volatile("cp.async.wait_group %0;" ::"n"(kScanRing - 1) : "memory");
+        S = on && seqs[seq] >= 0 ? ring[(seq % kScanRing) * kConsumerThreads] : make_float4(0.f, 0.f, 0.f, 0.f);
+        ++seq;
+      }
+      float y = 0.f, u = 0.f;
+      if (on) {
+        const float dt = dts[t * CP + ch];
+        u = us[t * CP + ch];
+        const float4 b = *reinterpret_cast<const float4 *>(bc + t * 2 * NP + n0), k = *reinterpret_cast<const float4 *>(bc + t * 2 * NP + NP + n0);
+        const float du = dt * u;
+        S.x = fmaf(decay_exp(dt * A.x), S.x, du * b.x);
+        S.y = fmaf(decay_exp(dt * A.y), S.y, du * b.y);
+        S.z = fmaf(decay_exp(dt * A.z), S.z, du * b.z);
+        S.w = fmaf(decay_exp(dt * A.w), S.w, du * b.w);
+        y = fmaf(S.x, k.x, fmaf(S.y, k.y, fmaf(S.z, k.z, S.w * k.w)));
+        if (flags & 2) *reinterpret_cast<float4 *>(mine + (size_t)rec[t].slot * C * NP) = S;
+      }
+      for (int s = LPC >> 1; s > 0; s >>= 1) y += __shfl_xor_sync(0xffffffffu, y, s);
+      if (on && q == 0) us[t * CP + ch] = fmaf(D, u, y);   // (the other lanes of the channel read u before the shuffles)
+    }
+    consumer_sync();
+    stamp(c, task, 2);
+    for (int i = tid; i < B * nc; i += kConsumerThreads) {
+      const int t = i / nc, k = i - t * nc;
+      const float z = __ldcg(reinterpret_cast<const float *>(d.p[2]) + (size_t)t * d.a[SS_LDG] + d.a[SS_GOFF] + cb + k);
+      store_elt(reinterpret_cast<T *>(d.p[7]) + (size_t)t * d.a[SS_LDO] + cb + k, us[t * CP + k] * silu_exact_f(z));
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    consumer_sync();   // the next channels reuse the arrays and the ring
   }
 }
 
@@ -2689,7 +2992,9 @@ __device__ __forceinline__ void run_hybrid_task(const Ctx &c, const TaskDesc &d,
     case TASK_ATTN_MERGE: run_attn_merge<HYB>(c, d); break;
     case TASK_QKV_APPEND: run_qkv_append<HYB>(c, d); break;
     case TASK_EXT_ATTENTION: run_ext_attention<HYB>(c, d, task); break;
-    case TASK_SHORT_CONV: run_short_conv(c, d); break;
+    case TASK_SHORT_CONV: run_short_conv<HYB>(c, d); break;
+    case TASK_SELECTIVE_SCAN: run_selective_scan<HYB>(c, d, task); break;
+    case TASK_DIFF_COMBINE: run_diff_combine<HYB>(c, d); break;
     case TASK_RGLRU: run_rglru<HYB>(c, d); break;
     case TASK_MLSTM: run_mlstm<HYB>(c, d, task); break;
     case TASK_ARGMAX_PARTIAL: run_argmax_partial_f32(c, d); break;

@@ -421,7 +421,7 @@ static __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d
   constexpr int NV = 4;   // rows of at most 4096 columns, in registers
   const int tid = threadIdx.x, W = d.a[L_GROUPS], K = d.a[L_K], warp = tid >> 5;
   const bool layer_norm = (d.a[L_G_SLOT] & 4) != 0;
-  const float eps = __int_as_float(d.a[L_EPS]), off = (d.a[L_G_SLOT] & 2) ? 1.0f : 0.0f;
+  const float eps = __int_as_float(d.a[L_EPS]), off = (d.a[L_G_SLOT] & 2) ? 1.0f : 0.0f, factor = __int_as_float(d.a[LR_POST]);
   const float *add = *reinterpret_cast<const float *const *>(&d.a[LR_ADD]);
   const uint64_t rowp = *reinterpret_cast<const uint64_t *>(&d.a[LR_ROW]);
   const bool has_y = d.p[6] != 0, has_post = d.p[3] != 0, moved = has_y || add != nullptr || rowp != 0;
@@ -451,7 +451,7 @@ static __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d
       yv[i] = in && has_y ? __ldcg(reinterpret_cast<const float4 *>(y + j)) : zero;
       xv[i] = in ? __ldcg(reinterpret_cast<const float4 *>(x + j)) : zero;
       wp[i] = in && has_post ? values(d.p[3], j, off) : make_float4(1.f, 1.f, 1.f, 1.f);
-      wn[i] = in ? values(d.p[4], j, off) : zero;
+      wn[i] = !in ? zero : d.p[4] != 0 ? values(d.p[4], j, off) : make_float4(1.f, 1.f, 1.f, 1.f);
     }
     if (has_y) {
       float inv = 1.f;
@@ -459,7 +459,7 @@ static __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d
         float ss = 0.f;
 #pragma unroll
         for (int i = 0; i < NV; ++i) ss += yv[i].x * yv[i].x + yv[i].y * yv[i].y + yv[i].z * yv[i].z + yv[i].w * yv[i].w;
-        inv = 1.0f / sqrtf(total(ss, c.s.red) / (float)W + eps);
+        inv = factor / sqrtf(total(ss, c.s.red) / (float)W + eps);
       }
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
@@ -493,10 +493,13 @@ static __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d
       for (int i = 0; i < NV; ++i)
         if ((i * kConsumerThreads + tid) * 4 < W) { xv[i].x -= mean; xv[i].y -= mean; xv[i].z -= mean; xv[i].w -= mean; }
     }
-    float ss = 0.f;
+    float inv = 1.f;   // (no norm weight: the stream as it is)
+    if (d.p[4] != 0) {
+      float ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < NV; ++i) ss += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
-    const float inv = 1.0f / sqrtf(total(ss, c.s.red + 8) / (float)W + eps);
+      for (int i = 0; i < NV; ++i) ss += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
+      inv = 1.0f / sqrtf(total(ss, c.s.red + 8) / (float)W + eps);
+    }
     uint8_t *row = c.s.xtile + (size_t)b * (K * 2 + kRowPadBytes);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {   // (the padding columns behind the row come out as zeros)
@@ -838,6 +841,9 @@ __device__ __forceinline__ void linear_output(const Ctx &c, const TaskDesc &d, i
     }
   } else if (HYB && epi == EPI_STORE_F32) {
     reinterpret_cast<float *>(d.p[2])[(size_t)b * d.a[L_LDO] + col] = v;
+  } else if (HYB && epi == EPI_BIAS_F32) {
+    const __nv_bfloat16 *bias = *reinterpret_cast<const __nv_bfloat16 *const *>(&d.a[LR_BIAS]);
+    reinterpret_cast<float *>(d.p[2])[(size_t)b * d.a[L_LDO] + col] = v + bf16_to_f(__ldg(bias + col));
   } else if (HYB && epi == EPI_RELU2) {
     const float a = fmaxf(v, 0.f);
     reinterpret_cast<__nv_bfloat16 *>(d.p[2])[(size_t)b * d.a[L_LDO] + col] = __float2bfloat16_rn(a * a);
@@ -1027,8 +1033,8 @@ __device__ __forceinline__ void linear_emit(const Ctx &c, const EmitArgs &e, int
       const float a = round_bf16(silu_f(round_bf16(v)));
       e.out[(size_t)b * e.ldo + ((col >> 2) << 1) + (col & 1)] = __float2bfloat16_rn(a * round_bf16(u));
     }
-  } else if (HYB && e.epi == EPI_STORE_F32) {
-    reinterpret_cast<float *>(e.out)[(size_t)b * e.ldo + col] = v;
+  } else if (HYB && (e.epi == EPI_STORE_F32 || e.epi == EPI_BIAS_F32)) {
+    reinterpret_cast<float *>(e.out)[(size_t)b * e.ldo + col] = v + resv;   // resv: the bias, or 0
   } else if (HYB && e.epi == EPI_RELU2) {
     const float a = fmaxf(v, 0.f);
     e.out[(size_t)b * e.ldo + col] = __float2bfloat16_rn(a * a);
@@ -1131,6 +1137,8 @@ __device__ void run_linear_tc(const Ctx &c, const TaskDesc &d, LinearState &ls, 
       const int row = tile * RB + r_in_tile;
       const bool row_ok = r_in_tile < RB && row < rows;
       const uint32_t taddr = c.tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)(tile * NP + half * nh);
+      float bias = 0.f;
+      if (HYB && epi == EPI_BIAS_F32 && row_ok) bias = bf16_to_f(__ldg(*reinterpret_cast<const __nv_bfloat16 *const *>(&d.a[LR_BIAS]) + n0 + row));
       for (int c0 = 0; c0 < nh; c0 += 8) {
         uint32_t r[8];
         tmem_ld_x8(taddr + (uint32_t)c0, r);
@@ -1148,7 +1156,7 @@ __device__ void run_linear_tc(const Ctx &c, const TaskDesc &d, LinearState &ls, 
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
           const int b = half * nh + c0 + j;
-          resv[j] = 0.f;
+          resv[j] = HYB ? bias : 0.f;
           if (epi == EPI_RESIDUAL && row_ok && b < B)
             resv[j] = bf16_to_f(__ldcg(resp + (size_t)b * ldr + n0 + row));
         }
@@ -1157,7 +1165,7 @@ __device__ void run_linear_tc(const Ctx &c, const TaskDesc &d, LinearState &ls, 
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
           const float v = __uint_as_float(r[j]);
-          const float u = (epi == EPI_SILU_PAIR || (HYB && epi >= EPI_GATED_SILU)) ? __shfl_down_sync(0xffffffffu, v, 2) : 0.f;
+          const float u = (epi == EPI_SILU_PAIR || (HYB && (epi == EPI_GATED_SILU || epi == EPI_GATED_GELU))) ? __shfl_down_sync(0xffffffffu, v, 2) : 0.f;
           const int b = half * nh + c0 + j;
           if (row_ok && b < B) linear_emit<HYB>(c, ea, b, n0 + row, v, u, resv[j]);
         }
@@ -1663,27 +1671,29 @@ static __device__ void run_moe_routing(const Ctx &c, const TaskDesc &d) {
       }
     }
     __syncwarp();
-    for (int g = lane; g < groups; g += 32) {
-      float t1 = bi[g * per], t2 = -1e30f;
-      for (int i = 1; i < per; ++i) {
-        const float v = bi[g * per + i];
-        if (v > t1) { t2 = t1; t1 = v; }
-        else if (v > t2) t2 = v;
+    if (groups > 1) {   // (one group: nothing to choose between)
+      for (int g = lane; g < groups; g += 32) {
+        float t1 = bi[g * per], t2 = -1e30f;
+        for (int i = 1; i < per; ++i) {
+          const float v = bi[g * per + i];
+          if (v > t1) { t2 = t1; t1 = v; }
+          else if (v > t2) t2 = v;
+        }
+        gs[g] = per > 1 ? t1 + t2 : t1;
       }
-      gs[g] = per > 1 ? t1 + t2 : t1;
+      __syncwarp();
+      unsigned long long selected = 0ull;
+      for (int k = 0; k < keep; ++k) {
+        int best = 0;
+        float best_s = -1e30f;
+        for (int g = 0; g < groups; ++g)
+          if (!((selected >> g) & 1ull) && gs[g] > best_s) { best_s = gs[g]; best = g; }
+        selected |= 1ull << best;
+      }
+      for (int e = lane; e < E; e += 32)
+        if (!((selected >> (e / per)) & 1ull)) bi[e] = -10000.f;
+      __syncwarp();
     }
-    __syncwarp();
-    unsigned long long selected = 0ull;
-    for (int k = 0; k < keep; ++k) {
-      int best = 0;
-      float best_s = -1e30f;
-      for (int g = 0; g < groups; ++g)
-        if (!((selected >> g) & 1ull) && gs[g] > best_s) { best_s = gs[g]; best = g; }
-      selected |= 1ull << best;
-    }
-    for (int e = lane; e < E; e += 32)
-      if (!((selected >> (e / per)) & 1ull)) bi[e] = -10000.f;
-    __syncwarp();
     float total = 0.f;
     float mine = 0.f;   // lane k < topk: slot k's weight (0: its expert belongs to another rank)
     for (int k = 0; k < topk; ++k) {
@@ -1713,7 +1723,7 @@ static __device__ void run_moe_routing(const Ctx &c, const TaskDesc &d) {
       }
       __syncwarp();
     }
-    const float inv = __fdiv_rn(1.0f, total + 1e-20f);
+    const float inv = d.a[13] ? 1.0f : __fdiv_rn(1.0f, total + 1e-20f);
     if (lane < topk) wout[(size_t)row * ldw + lane] = mine * inv * scaling;
     __syncwarp();
   }
@@ -1984,6 +1994,9 @@ __device__ void run_moe_gemm(const Ctx &c, const TaskDesc &d, LinearState &ls, i
               const size_t orow = ((size_t)(tmv & 0xff) * topk + (tmv >> 8)) * d.a[L_LDO];
               if (HYBRID && d.a[L_EPI] == EPI_STORE_F32) {
                 reinterpret_cast<float *>(out)[orow + rbase + r] = v;
+              } else if (HYBRID && d.a[L_EPI] == EPI_RELU2) {
+                const float a = fmaxf(v, 0.f);
+                out[orow + rbase + r] = __float2bfloat16_rn(a * a);
               } else if (HYBRID && d.a[L_EPI] >= EPI_GATED_SILU) {   // rows [gate, gate, up, up]
                 if (r & 2) continue;
                 float u = 0.f;
@@ -2154,6 +2167,7 @@ static __device__ void run_moe_gemm_tc(const Ctx &c, const TaskDesc &d, LinearSt
           const size_t orow = ((size_t)(tm & 0xff) * topk + (tm >> 8)) * ldo;
           if (epi == EPI_STORE_F32) reinterpret_cast<float *>(out)[orow + row] = x;
           else if (epi == EPI_STORE) reinterpret_cast<__nv_bfloat16 *>(out)[orow + row] = __float2bfloat16_rn(x);
+          else if (epi == EPI_RELU2) reinterpret_cast<__nv_bfloat16 *>(out)[orow + row] = __float2bfloat16_rn(fmaxf(x, 0.f) * fmaxf(x, 0.f));
           else if ((row & 2) == 0)
             reinterpret_cast<__nv_bfloat16 *>(out)[orow + ((row >> 2) << 1) + (row & 1)] =
                 __float2bfloat16_rn((epi == EPI_GATED_SILU ? silu_exact_f(x) : gelu_tanh_f(x)) * u);

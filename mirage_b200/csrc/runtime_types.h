@@ -67,6 +67,8 @@ enum TaskType : uint32_t {
   TASK_LATENT_APPEND = 33,      // latent attention: cache rows and rotated query parts
   TASK_MOE_GEMM_F32 = 34,       // expert projections in 32-bit arithmetic
   TASK_ATTN_MERGE = 35,         // merge of an attention layer's key chunks
+  TASK_SELECTIVE_SCAN = 36,     // selective state space recurrence
+  TASK_DIFF_COMBINE = 37,       // differential attention: difference of the two maps' outputs, unit norm per head
 };
 
 // Which family of megakernel instantiations runs a graph (template parameter HYB of the kernel).
@@ -87,6 +89,15 @@ MPK_HD constexpr int ext_attention_rows(int rows) {
   while (r < rows) r *= 2;
   return r;
 }
+
+// Selective scan: lanes that share a channel's state (four values each), slots of the ring of states to come, columns of the
+// low-rank step sizes staged at a time.
+MPK_HD constexpr int scan_lanes(int n) {
+  int l = 1;
+  while (4 * l < n) l *= 2;
+  return l;
+}
+constexpr int kScanRing = 8, kScanRank = 128;
 
 enum : int { HYB_NONE = 0, HYB_BF16 = 1, HYB_F32 = 2 };
 // Activations of hybrid linears (mpk_activation of include/mpk_b200.h).
@@ -115,6 +126,7 @@ enum Epilogue : int32_t {
   EPI_SOFTCAP = 7,      // out = cap * tanh(acc / cap), float32 (hybrid graphs)
   EPI_GATED_SILU = 8,   // rows [gate, gate, up, up]: out[2k + i] = bf16(silu(gate_i) * up_i) (hybrid graphs)
   EPI_GATED_GELU = 9,   // the same with the tanh form of gelu
+  EPI_BIAS_F32 = 10,    // out = acc + bias, float32 (hybrid graphs)
   EPI_SILU_PAIR = 4,    // rows interleaved [gate, gate, up, up]: out[2k + i] = bf16(silu(gate_i)) * up_i
 };
 
@@ -156,7 +168,8 @@ static_assert(sizeof(TaskDesc) == 16 * kDescVecs, "TaskDesc must stay 224 bytes 
 //  PRO_RESNORM: p[1] x f32  p[3] weight of y's norm or null  p[4] weight of the output norm  p[6] y f32 or null  p[7] x_out f32 (or
 //        null), a[20] ld y, a[21] ld x_out, a[22] flags (2: weights stored around zero, 4: layer norm), a[10] width (K minus the
 //        zero padding), p[5] norm bias or null, 64-bit values a[LR_ADD] added stream or null (ld a[LR_LDADD]), a[LR_ROW] added row or null
-//  EPI_SOFTCAP: a[23] cap bits
+//        a[LR_POST] factor of y's norm (bits); p[4] null: the activation is the stream as it is
+//  EPI_SOFTCAP: a[23] cap bits;  EPI_BIAS_F32: 64-bit value a[LR_BIAS]
 //  a[15] allreduce index within the iteration  a[16] allreduces per iteration  a[17] stride between the two inbox buffers (floats)
 //  tcgen05 path (TF_TC): a[18] rows of one weight tile (the TMA box height, a multiple of 8, at most 128; the task's rows are
 //        cut into ceil(rows / a[18]) tiles, each one 128-lane accumulator), a[12] = 64 x (k blocks of 64 columns per ring slot),
@@ -164,7 +177,7 @@ static_assert(sizeof(TaskDesc) == 16 * kDescVecs, "TaskDesc must stay 224 bytes 
 enum { L_N0 = 0, L_N1, L_K, L_LDW, L_LDX, L_LDO, L_LDR, L_PRO, L_EPI, L_EPS, L_GROUPS, L_KT, L_KC, L_SLOT, L_N, L_ARIDX, L_NAR, L_PARSTRIDE, L_ROWS,
        L_GATHER, L_G_LDRES, L_G_LDOUT, L_G_SLOT, L_WS_S0, L_WS_S1, L_XS_S0, L_XS_S1, L_TMAP };
 static_assert(L_TMAP == 27, "TaskDesc::a has 28 entries");
-enum { LR_ADD = 14, LR_ROW = 16, L_CAP = 23, LR_LDADD = 25 };   // hybrid graphs (the fields of allreduces and FP8 tasks are free there)
+enum { LR_POST = 13, LR_ADD = 14, LR_ROW = 16, L_CAP = 23, LR_BIAS = 24, LR_LDADD = 26 };   // hybrid graphs (the fields of allreduces and FP8 tasks are free there)
 // ---- TASK_ATTENTION ----------------------------------------------------------
 //  p[0] qkv  p[1] k_cache  p[2] v_cache  p[3] q_norm  p[4] k_norm  p[5] cos  p[6] sin  p[7] out
 //  a[0] slot  a[1] kv head  a[2] chunk  a[3] num chunks  a[4] local q heads  a[5] local kv heads
@@ -180,9 +193,10 @@ enum { E_T0 = 0, E_T1, E_WIDTH, E_LDI, E_LDO, E_AUX, E_LDI2 };
 // ---- TASK_MOE_ROUTING: p[0] logits [B, E] (zeroed after reading)  p[1] bias f32 [E]  p[2] weights f32 [B, topk]
 //      p[3] routing i32 [E, ld]  p[4] active i32 [E + 1];  a[0] E  a[1] topk  a[2] groups  a[3] groups kept
 //      a[4] scaling bits  a[5] ld logits  a[6] ld weights  a[7] ld routing  a[8] logits are f32  a[12] logits stay as they are
+//      a[13] weights are the scores, not renormalised over the chosen experts
 // ---- TASK_MOE_GEMM: linear-task fields (L_*) describe one expert's panel; p[0] weights [E, N, K]  p[1] x  p[2] out
 //      p[4] routing  p[5] active list  p[6] weight scales f32 [E, N, K/128]  p[7] x scales f32 [rows, K/128];
-//      a[L_EPI] EPI_STORE, EPI_STORE_F32, EPI_GATED_*
+//      a[L_EPI] EPI_STORE, EPI_STORE_F32, EPI_RELU2, EPI_GATED_*
 //      a[M_NEXP] experts  a[M_NTOPK]  a[M_PER_SLOT] 1: x has one row per (token, slot)  a[M_LDR] ld routing
 //      a[M_ESTRIDE] elements between experts
 enum { M_NEXP = 19, M_NTOPK, M_PER_SLOT, M_LDR, M_ESTRIDE };
@@ -211,31 +225,32 @@ enum { M_NEXP = 19, M_NTOPK, M_PER_SLOT, M_LDR, M_ESTRIDE };
 // ---- hybrid tasks --------------------------------------------------------------
 // ---- TASK_EMBED_F32: p[0] ids  p[1] table bf16  p[2] out f32;  a[E_*] as TASK_EMBED (a[E_AUX] = vocabulary, a[E_LDI2] factor bits)
 // ---- TASK_RESIDUAL_NORM: rows [a[0], a[1]), width a[2]; p[0] x f32 (in place)  p[1] y f32 or null  p[2] weight of y's norm or
-//      null (plain sum)  p[3] weight of the output norm or null  p[4] out (bf16, f32 with flag 1) or null  p[5] new x (= p[0]: in place);
+//      null (plain sum)  p[3] weight of the output norm or null (out is the new x)  p[4] out (bf16, f32 with flag 1) or null  p[5] new x (= p[0]: in place);
 //      a[3] ld x  a[4] ld y  a[5] ld out  a[6] eps bits  a[7] flags (1: out f32, 2: weights stored around zero, 4: layer norm)  a[8] ld
 //      of the new x;  64-bit values, 0 if absent: a[RN_BIAS] norm bias, a[RN_ADD] added stream, a[RN_ROW] added row, a[RN_EXP] expert
 //      outputs f32 [tokens, slots, width], a[RN_EW] their weights f32, a[RN_GATE] f32 column, y is multiplied by its sigmoid
-enum { RN_LDADD = 9, RN_BIAS = 10, RN_ADD = 12, RN_ROW = 14, RN_EXP = 16, RN_EW = 18, RN_GATE = 20, RN_SLOTS = 22, RN_LDEW, RN_LDGATE };
+//      a[RN_POST] factor of y's norm (bits); with that norm the experts' sum is part of what is normed
+enum { RN_LDADD = 9, RN_BIAS = 10, RN_ADD = 12, RN_ROW = 14, RN_EXP = 16, RN_EW = 18, RN_GATE = 20, RN_SLOTS = 22, RN_LDEW, RN_LDGATE, RN_POST };
 // ---- TASK_LINEAR_F32: p[0] W bf16 [N, K]  p[1] x f32  p[2] out f32;  a[0] n0  a[1] n1  a[2] K  a[3] ldw  a[4] ld x  a[5] ld out
 //      a[6] activation (mpk_activation)  a[7] tokens per shared-memory tile  a[8] soft cap bits
 // ---- TASK_MOE_GEMM_F32: p[0] W bf16 [E, N, K]  p[1] x f32  p[2] out f32  p[4] routing  p[5] active list;  a[0] n0  a[1] n1  a[2] K  a[4] ld x
 //      a[5] ld out (of a slot)  a[6] activation  a[7] tokens per shared-memory tile  a[8] x rows per (token, slot)  a[9] slots  a[10] ld routing
 //      a[11] experts  a[12] rows N of an expert
 // ---- TASK_QKV_APPEND: tokens [a[0], a[1]); p[0] projections f32  p[1] q out  p[2] k cache  p[3] v cache  p[4] cos f32  p[5] sin f32
-//      p[6] v source (null: the k columns before rotation and norm)
-//      a[QA_*] below
+//      p[6] q norm  p[7] k norm (bf16 [dim], null: none);  p[2] null: queries only;  a[QA_*] below
 enum { QA_T0 = 0, QA_T1, QA_LDP, QA_QOFF, QA_KOFF, QA_VOFF, QA_HQ, QA_HKV, QA_DIM, QA_DIMP, QA_VDIM, QA_VDIMP, QA_ROT, QA_NORM,
-       QA_EPS, QA_PAGE, QA_LDQ, QA_ROWS };
+       QA_EPS, QA_PAGE, QA_LDQ, QA_ROWS, QA_PAIRS, QA_MAPS };
 // ---- TASK_EXT_ATTENTION: p[0] q [tokens, hq * dimp]  p[1] k cache  p[2] v cache  p[3] out;  a[XA_*] below
 enum { XA_SLOT = 0, XA_HEAD, XA_CHUNK, XA_NCHUNK, XA_HQ, XA_HKV, XA_DIMP, XA_VDIM, XA_VDIMP, XA_PAGE, XA_LDQ, XA_LDO, XA_OCOL,
-       XA_SCALE, XA_CAP, XA_SINK, XA_OSCALE, XA_TICKET, XA_SREC, XA_STAGES, XA_SHARED, XA_KEYS, XA_MERGE };
+       XA_SCALE, XA_CAP, XA_SINK, XA_OSCALE, XA_TICKET, XA_SREC, XA_STAGES, XA_SHARED, XA_KEYS, XA_MERGE, XA_WINDOW, XA_KEEP, XA_OUTF32 };
 //      p[4] sinks bf16 [hq] or null; XA_SHARED: values are key columns; XA_KEYS: keys of a tile of
-//      theirs; XA_MERGE: a layer of TASK_ATTN_MERGE follows (its tasks: the same fields, task a[XA_SLOT] of a[XA_CHUNK])
+//      theirs; XA_MERGE: a layer of TASK_ATTN_MERGE follows (its tasks: the same fields, task a[XA_SLOT] of a[XA_CHUNK]);
+//      XA_WINDOW: keys a position sees at most, itself included (0: all)  XA_KEEP: first keys it sees all the same
 constexpr int kXaRecHead = 4;   // floats in front of a record's columns
 constexpr int kXaCells = 320;   // cache rows of a chunk's key octets kept in shared memory
 // ---- TASK_SHORT_CONV: channels [a[0], a[1]); p[0] in f32  p[1] in bias bf16 or null  p[2] taps bf16 [channels, taps]
-//      p[3] bias bf16 or null  p[4] carried inputs f32 [slots, taps - 1, channels]  p[5] out f32
-//      a[2] channels  a[3] taps  a[4] ld in  a[5] in column offset  a[6] ld out  a[7] activation (0 none, 1 silu)
+//      p[3] bias bf16 or null  p[4] carried inputs f32 [slots, taps - 1, channels]  p[5] out f32  p[6] copy of out in the activation type or null
+//      a[2] channels  a[3] taps  a[4] ld in  a[5] in column offset  a[6] ld out  a[7] activation (0 none, 1 silu)  a[8] ld copy
 // ---- TASK_RGLRU: p[0] u f32 [tokens, width]  p[1] projections f32 (output branch)  p[2] y bias bf16  p[3] ra  p[4] ra bias  p[5] ri
 //      p[6] ri bias  p[7] lambda (bf16, all);  a[GL_*]; state and output pointers are 64-bit values in a[GL_STATE], a[GL_OUT]
 enum { GL_BLOCK = 0, GL_C0, GL_C1, GL_BS, GL_WIDTH, GL_LDU, GL_LDP, GL_YOFF, GL_LDO, GL_OCOL, GL_OSCALE, GL_OUTF32, GL_GATE_C, GL_TG,
@@ -252,6 +267,11 @@ enum { GA_SLOT = 0, GA_HEAD, GA_CHUNK, GA_NCHUNK, GA_H, GA_DIM, GA_VDIM, GA_VDIM
 // ---- TASK_LATENT_APPEND: items [a[0] of a[1] tasks]; p[0] projections f32  p[1] latent norm weight bf16  p[2] q out  p[3] cache [pages, page, 1, dimp]
 //      p[4] cos f32  p[5] sin f32;  a[LA_*]
 enum { LA_T0 = 0, LA_T1, LA_LDP, LA_QOFF, LA_KVOFF, LA_H, LA_RANK, LA_ROT, LA_DIMP, LA_EPS, LA_PAGE, LA_LDQ, LA_ROWS };
+// ---- TASK_SELECTIVE_SCAN: channels [a[SS_C0], a[SS_C1]) of all requests; p[0] u f32  p[1] low f32 [tokens, rank | B | C]  p[2] gate f32
+//      p[3] dt weight bf16 [channels, rank]  p[4] dt bias  p[5] A_log [channels, n]  p[6] D  p[7] out;  64-bit value a[SS_STATE] f32 [slots, channels, np]
+enum { SS_C0 = 0, SS_C1, SS_C, SS_RANK, SS_N, SS_NP, SS_LANES, SS_LDU, SS_LDL, SS_LDG, SS_GOFF, SS_LDO, SS_STATE };
+// ---- TASK_DIFF_COMBINE: task a[0] of a[1]; p[0] maps f32 [tokens, heads * 2 * vdim]  p[1] out;  a[2] heads  a[3] vdim  a[4] ld in  a[5] ld out
+//      a[6] lambda  a[7] factor  a[8] eps (bits)
 // ---- TASK_ALLREDUCE:       p[0] inbox base p[1] residual (or null) p[2] out
 //  a[0] c0 a[1] c1 (columns) a[2] world a[3] slot stride (floats) a[4] ld_out a[5] ld_res a[6] N
 //  a[7] allreduce index  a[8] allreduces per iteration  a[9] stride between the two inbox buffers (floats)

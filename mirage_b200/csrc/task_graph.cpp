@@ -125,6 +125,7 @@ struct Builder {
         add(ins, l.t[1]);
         const int y = l.op == MPK_OP_LINEAR_RESIDUAL ? l.t[3] : l.t[2];
         if (l.op == MPK_OP_LINEAR_RESIDUAL) add(ins, l.t[2]);
+        if (l.op == MPK_OP_LINEAR) add(ins, norm_tensor(l, 3));
         if (l.op == MPK_OP_SPLITK_LINEAR) add(ins, y);
         if (!l.push) add(outs, l.silu_out >= 0 ? l.silu_out : y);
         break;
@@ -174,14 +175,16 @@ struct Builder {
         if (resnorm_moves(l)) add(outs, resnorm_out(l));
         add(outs, l.t[4]);
         break;
-      case MPK_OP_QKV_APPEND: add(ins, l.t[0]); add(ins, l.t[4]); add(ins, l.t[5]); for (int i = 1; i < 4; ++i) add(outs, l.t[i]); break;
+      case MPK_OP_QKV_APPEND: add(ins, l.t[0]); for (int i = 4; i < 8; ++i) add(ins, norm_tensor(l, i)); for (int i = 1; i < 4; ++i) add(outs, l.t[i]); break;
       case MPK_OP_ATTN_MERGE: add(ins, l.t[3]); add(outs, l.t[3]); break;
       case MPK_OP_EXT_ATTENTION:
         for (int i = 0; i < 3; ++i) add(ins, l.t[i]);
         if (l.t.size() > 4) add(ins, l.t[4]);
         add(outs, l.t[3]);
         break;
-      case MPK_OP_SHORT_CONV: for (int i = 0; i < 5; ++i) add(ins, l.t[i]); add(outs, l.t[4]); add(outs, l.t[5]); break;
+      case MPK_OP_SHORT_CONV: for (int i = 0; i < 5; ++i) add(ins, l.t[i]); add(outs, l.t[4]); add(outs, l.t[5]); add(outs, norm_tensor(l, 6)); break;
+      case MPK_OP_SELECTIVE_SCAN: for (int i = 0; i < 8; ++i) add(ins, l.t[i]); add(outs, l.t[7]); add(outs, l.t[8]); break;
+      case MPK_OP_DIFF_COMBINE: add(ins, l.t[0]); add(outs, l.t[1]); break;
       case MPK_OP_RGLRU: for (int i = 0; i < 9; ++i) add(ins, l.t[i]); add(outs, l.t[8]); add(outs, l.t[9]); break;
       case MPK_OP_MLSTM: for (int i = 0; i < 6; ++i) add(ins, l.t[i]); for (int i = 4; i < 8; ++i) add(outs, l.t[i]); break;
       case MPK_OP_GLA: for (int i = 0; i < 5; ++i) add(ins, l.t[i]); for (int i = 4; i < 7; ++i) add(outs, l.t[i]); break;
@@ -221,7 +224,7 @@ struct Builder {
           {MPK_OP_SAMPLING_PARTIAL, 3}, {MPK_OP_SAMPLING_REDUCE, 3}, {MPK_OP_ARGMAX_EXCHANGE, 3},
           {MPK_OP_MOE_TOPK_SOFTMAX, 4}, {MPK_OP_RESIDUAL_NORM, 5}, {MPK_OP_QKV_APPEND, 6}, {MPK_OP_EXT_ATTENTION, 4},
           {MPK_OP_SHORT_CONV, 6}, {MPK_OP_RGLRU, 10}, {MPK_OP_MLSTM, 8}, {MPK_OP_GLA, 7}, {MPK_OP_LATENT_APPEND, 6},
-          {MPK_OP_GROUPED_LINEAR, 3}, {MPK_OP_ATTN_MERGE, 4}};
+          {MPK_OP_GROUPED_LINEAR, 3}, {MPK_OP_ATTN_MERGE, 4}, {MPK_OP_SELECTIVE_SCAN, 9}, {MPK_OP_DIFF_COMBINE, 2}};
       auto it = need.find(L[i].op);
       if (it == need.end()) return fail(MPK_ERR_UNSUPPORTED, "layer " + std::to_string(i) + ": unknown op");
       if ((int)L[i].t.size() < it->second)
@@ -299,6 +302,7 @@ struct Builder {
     return l.t[1] >= 0 || norm_tensor(l, 7) >= 0 || norm_tensor(l, 8) >= 0 || norm_tensor(l, 9) >= 0;
   }
   static int norm_flags(const LayerInfo &l) { return (l.params[1] ? 2 : 0) | (l.params.size() > 2 && l.params[2] == 1 ? 4 : 0); }
+  static int norm_factor(const LayerInfo &l) { return l.params.size() > 4 ? bits_of(l.params[4]) : 0x3f800000; }   // (1.0f)
   static bool keeps_logits(const LayerInfo &l) { return l.params.size() > 5 && l.params[5] != 0; }
 
   // Hybrid graphs of one or two tokens: a residual_norm layer whose result feeds linears becomes their prologue, which
@@ -307,13 +311,13 @@ struct Builder {
     if (g->hybrid != HYB_BF16 || nb_max > 2 || cfg.max_num_batched_tokens > 2) return;
     for (size_t i = 0; i < L.size(); ++i) {
       LayerInfo &p = L[i];
-      if (p.op != MPK_OP_RESIDUAL_NORM || p.t[4] < 0 || p.t[3] < 0) continue;
+      if (p.op != MPK_OP_RESIDUAL_NORM || p.t[4] < 0) continue;
       const int x = p.t[0], y = p.t[1], out = p.t[4], xo = resnorm_out(p), add = norm_tensor(p, 7), row = norm_tensor(p, 8), bias = norm_tensor(p, 6);
       if (norm_tensor(p, 9) >= 0 || norm_tensor(p, 11) >= 0) continue;   // the sum over experts is formed once, not by every task
       const bool moves = resnorm_moves(p);
       auto aligned = [&](int t) { return T[t].ld() % 4 == 0 && ((uint64_t)T[t].ptr & 15) == 0; };
       const int64_t D = T[x].dim(1);
-      if (T[out].owner == 0 || D > 4096 || D % 4 || !aligned(x) || ((uint64_t)T[p.t[3]].ptr & 7) || p.params.size() < 2) continue;
+      if (T[out].owner == 0 || D > 4096 || D % 4 || !aligned(x) || (p.t[3] >= 0 && ((uint64_t)T[p.t[3]].ptr & 7)) || p.params.size() < 2) continue;
       if (moves && (T[xo].storage == T[x].storage || !aligned(xo) || T[xo].dtype != MPK_F32 || T[xo].dim(1) != D)) continue;
       if ((y >= 0 && !aligned(y)) || (add >= 0 && (!aligned(add) || T[add].dtype != MPK_F32 || T[add].dim(1) != D))) continue;
       if ((bias >= 0 && ((uint64_t)T[bias].ptr & 7)) || (row >= 0 && ((uint64_t)T[row].ptr & 7))) continue;
@@ -339,7 +343,7 @@ struct Builder {
       c.pro_src = x; c.pro_y = y; c.pro_post = p.t[2]; c.pro_gamma = p.t[3];
       c.pro_bias = bias; c.pro_add = add; c.pro_row = row;
       c.pro_xout = moves ? xo : -1;
-      c.pro_eps = bits_of(p.params[0]); c.pro_flags = norm_flags(p);
+      c.pro_eps = bits_of(p.params[0]); c.pro_flags = norm_flags(p); c.pro_factor = norm_factor(p);
       p.folded = true;
       g->num_folded++;
     }
@@ -488,8 +492,8 @@ struct Builder {
         }
       } else if (l.op == MPK_OP_MLA_DECODE) {
         need = std::max<int64_t>(need, 16 * (576 * 2 + 16) + 64 * (576 * 2 + 16) + 16 * (64 * 2 + 16) + 2 * 8 * 16 * 4);
-      } else if (l.op == MPK_OP_MOE_TOPK_SIGMOID) {
-        const int64_t E = T[l.t[3]].dim(0);
+      } else if (l.op == MPK_OP_MOE_TOPK_SIGMOID || l.op == MPK_OP_MOE_TOPK_SOFTMAX) {
+        const int64_t E = T[l.t[l.op == MPK_OP_MOE_TOPK_SIGMOID ? 3 : 2]].dim(0);
         need = std::max(need, 8 * (2 * E + 64) * 4 + E * 4 + 64);
       } else if (l.op == MPK_OP_ATTENTION || l.op == MPK_OP_PAGED_ATTENTION) {
         const int G = (int)(l.params[0] / l.params[1]);
@@ -588,6 +592,9 @@ struct Builder {
     }
     int epi = EPI_STORE;
     bool gated = false;
+    const int bias = l.op == MPK_OP_LINEAR ? norm_tensor(l, 3) : -1;
+    if (bias >= 0 && (y.dtype != MPK_F32 || T[bias].dtype != MPK_BF16 || T[bias].dim(0) < N || (!l.params.empty() && l.params[0])))
+      return fail(MPK_ERR_INVALID, "linear bias: bf16 [rows], float32 output, no activation: " + w.name);
     uint64_t res_ptr = 0;
     int ldr = 0;
     if (l.op == MPK_OP_LINEAR_RESIDUAL) {
@@ -609,7 +616,7 @@ struct Builder {
       if (gated && N % 4) return fail(MPK_ERR_INVALID, "gated linear: rows come as two gate rows, two up rows: " + w.name);
     } else if (y.dtype == MPK_F32) {
       if (g->hybrid != HYB_BF16 || epi != EPI_STORE) return fail(MPK_ERR_UNSUPPORTED, "float32 linear output needs a hybrid graph: " + w.name);
-      epi = EPI_STORE_F32;
+      epi = bias >= 0 ? EPI_BIAS_F32 : EPI_STORE_F32;
     } else if (y.dtype != MPK_BF16) {
       return fail(MPK_ERR_UNSUPPORTED, "linear output must be bf16 or float32: " + w.name);
     }
@@ -684,7 +691,7 @@ struct Builder {
         }
         if (l.prologue == PRO_RESNORM) {
           d.p[3] = l.pro_post >= 0 ? (uint64_t)T[l.pro_post].ptr : 0;
-          d.p[4] = (uint64_t)T[l.pro_gamma].ptr;
+          d.p[4] = l.pro_gamma >= 0 ? (uint64_t)T[l.pro_gamma].ptr : 0;
           d.p[6] = l.pro_y >= 0 ? (uint64_t)T[l.pro_y].ptr : 0;
           d.p[7] = l.pro_xout >= 0 ? (uint64_t)T[l.pro_xout].ptr : 0;
           d.a[L_G_LDRES] = l.pro_y >= 0 ? (int)T[l.pro_y].ld() : 0;
@@ -713,7 +720,9 @@ struct Builder {
         d.a[L_NAR] = g->num_allreduce;
         d.a[L_PARSTRIDE] = (int)g->inbox_floats_per_buffer;
         if (epi == EPI_SOFTCAP) d.a[L_CAP] = bits_of(l.params[1]);
+        if (epi == EPI_BIAS_F32) put_wide(&d, LR_BIAS, bias);
         if (l.prologue == PRO_RESNORM) {
+          d.a[LR_POST] = l.pro_factor;
           put_wide(&d, LR_ADD, l.pro_add);
           put_wide(&d, LR_ROW, l.pro_row);
         }
@@ -941,8 +950,9 @@ struct Builder {
     int epi = EPI_STORE, cols = N;
     if (g->hybrid && !w2 && l.params.size() > 1 && l.params[1]) {
       epi = activation_epilogue(l.params[1]);
-      if ((epi != EPI_GATED_SILU && epi != EPI_GATED_GELU) || N % 4) return fail(MPK_ERR_INVALID, "expert projection: gated activations only: " + w.name);
-      cols = N / 2;
+      const bool gated = epi == EPI_GATED_SILU || epi == EPI_GATED_GELU;
+      if ((!gated && epi != EPI_RELU2) || (gated && N % 4)) return fail(MPK_ERR_INVALID, "expert projection: gated activations or squared relu: " + w.name);
+      if (gated) cols = N / 2;
     } else if (g->hybrid && y.dtype == MPK_F32) {
       epi = EPI_STORE_F32;
     }
@@ -1098,8 +1108,8 @@ struct Builder {
   }
 
   // ---- hybrid graphs: recurrent layers, extended attention, float32 residual stream --------------------------
-  static bool hybrid_op(int op) { return op >= MPK_OP_RESIDUAL_NORM && op <= MPK_OP_ATTN_MERGE; }
-  static bool expert_op(int op) { return op == MPK_OP_MOE_TOPK_SIGMOID || op == MPK_OP_MOE_W13_LINEAR || op == MPK_OP_MOE_W2_LINEAR; }
+  static bool hybrid_op(int op) { return op >= MPK_OP_RESIDUAL_NORM && op <= MPK_OP_DIFF_COMBINE; }
+  static bool expert_op(int op) { return op == MPK_OP_MOE_TOPK_SIGMOID || op == MPK_OP_MOE_TOPK_SOFTMAX || op == MPK_OP_MOE_W13_LINEAR || op == MPK_OP_MOE_W2_LINEAR; }
   static int activation_epilogue(int64_t act) {
     switch (act) {
       case MPK_ACT_RELU2: return EPI_RELU2;
@@ -1127,8 +1137,8 @@ struct Builder {
     for (size_t i = 0; i < L.size(); ++i) {
       const LayerInfo &l = L[i];
       const int act_out = l.op == MPK_OP_RESIDUAL_NORM || l.op == MPK_OP_EXT_ATTENTION || l.op == MPK_OP_RGLRU || l.op == MPK_OP_MLSTM ||
-                                  l.op == MPK_OP_GLA
-                              ? (l.op == MPK_OP_RESIDUAL_NORM ? l.t[4] : l.op == MPK_OP_EXT_ATTENTION ? l.t[3] : l.t.back()) : -1;   // output of the graph's activation type
+                                  l.op == MPK_OP_GLA || l.op == MPK_OP_SELECTIVE_SCAN || l.op == MPK_OP_DIFF_COMBINE
+                              ? (l.op == MPK_OP_RESIDUAL_NORM ? l.t[4] : l.op == MPK_OP_EXT_ATTENTION ? l.t[0] : l.t.back()) : -1;   // tensor of the graph's activation type
       if (act_out >= 0 && T[act_out].dtype == MPK_F32) f32 = true;
       if (hybrid_op(l.op) || l.op == MPK_OP_EMBED || l.op == MPK_OP_ARGMAX_PARTIAL || l.op == MPK_OP_ARGMAX_REDUCE ||
           l.op == MPK_OP_SAMPLING_PARTIAL || l.op == MPK_OP_SAMPLING_REDUCE || expert_op(l.op)) continue;
@@ -1192,6 +1202,11 @@ struct Builder {
         return std::max(tile, xattn_stages() >= 3 && D <= 128 ? (int64_t)(16 + 8 * 64) * pitch : 0);
       }
       case MPK_OP_SHORT_CONV: return kMaxLinearTokens * 16 + (mbr + 1) * 4;
+      case MPK_OP_SELECTIVE_SCAN: {
+        const int64_t np = round_up(l.params[1], 4), cp = kConsumerThreads / scan_lanes((int)l.params[1]);
+        return kMaxLinearTokens * 16 + round_up(mbr + 1, 4) * 4 + kMaxLinearTokens * 4 + 4 * nb_max * (2 * cp + 2 * np) +
+               4 * nb_max * std::min<int64_t>(kScanRank, round_up(l.params[0], 8)) + kScanRing * kConsumerThreads * 16;
+      }
       case MPK_OP_GROUPED_LINEAR: {
         const int64_t K = T[l.t[1]].dim(2);
         if (g->hybrid == HYB_F32) return (int64_t)linear_f32_tokens(K) * K * 4;
@@ -1230,10 +1245,12 @@ struct Builder {
     const int cols = gated ? N / 2 : N;
     if (x.dim(1) != K || y.dim(1) < cols || (gated && N % 4) || act < 0 || act > MPK_ACT_GATED_GELU_TANH || (act == MPK_ACT_SOFTCAP && l.params.size() < 2))
       return fail(MPK_ERR_INVALID, "32-bit linear: shapes or activation of " + w.name);
+    const int bias = norm_tensor(l, 3);
+    if (bias >= 0 && (act || T[bias].dtype != MPK_BF16 || T[bias].dim(0) < N)) return fail(MPK_ERR_INVALID, "linear bias: bf16 [rows], no activation: " + w.name);
     const int nt = std::min(W, cols);
     for (int i = 0; i < nt; ++i) {
       TaskDesc d = blank(TASK_LINEAR_F32, li);
-      d.p[0] = (uint64_t)w.ptr; d.p[1] = (uint64_t)x.ptr; d.p[2] = (uint64_t)y.ptr;
+      d.p[0] = (uint64_t)w.ptr; d.p[1] = (uint64_t)x.ptr; d.p[2] = (uint64_t)y.ptr; d.p[3] = bias >= 0 ? (uint64_t)T[bias].ptr : 0;
       d.a[0] = (int)((int64_t)cols * i / nt); d.a[1] = (int)((int64_t)cols * (i + 1) / nt);
       d.a[2] = K; d.a[3] = (int)w.ld(); d.a[4] = (int)x.ld(); d.a[5] = (int)y.ld();
       d.a[6] = act;
@@ -1256,7 +1273,7 @@ struct Builder {
     if (w.dtype != MPK_BF16 || x.dtype != MPK_F32 || y.dtype != MPK_F32 || w.strides[2] != 1 || w.strides[1] != K || w.strides[0] != (int64_t)N * K)
       return fail(MPK_ERR_UNSUPPORTED, "32-bit expert projection: float32 input and output, dense bf16 weights: " + w.name);
     if (w.dim(0) != E || mask.dim(0) != E + 1 || idx.dtype != MPK_I32 || mask.dtype != MPK_I32 || x.dim(x.dims.size() - 1) < K || y.dim(2) < cols ||
-        (w2 && x.dim(1) != slots) || (act && !gated) || (gated && N % 4))
+        (w2 && x.dim(1) != slots) || (act && !gated && act != MPK_ACT_RELU2) || (gated && N % 4))
       return fail(MPK_ERR_INVALID, "32-bit expert projection: shapes of " + w.name + " and its routing tensors disagree");
     const int nt = std::min(W, cols);
     for (int i = 0; i < nt; ++i) {
@@ -1415,7 +1432,7 @@ struct Builder {
     if (l.t[1] >= 0 && (T[l.t[1]].dtype != MPK_F32 || T[l.t[1]].dim(1) != D)) return fail(MPK_ERR_INVALID, "residual_norm: y must be float32 of x's width");
     for (int i = 2; i < 4; ++i)
       if (l.t[i] >= 0 && (T[l.t[i]].dtype != MPK_BF16 || T[l.t[i]].dim(0) != D)) return fail(MPK_ERR_INVALID, "residual_norm: weights must be bf16 [width]");
-    if ((l.t[3] >= 0) != (l.t[4] >= 0)) return fail(MPK_ERR_INVALID, "residual_norm: output and its norm weight go together");
+    if (l.t[3] >= 0 && l.t[4] < 0) return fail(MPK_ERR_INVALID, "residual_norm: a norm weight needs an output");
     const int bias = norm_tensor(l, 6), add = norm_tensor(l, 7), row = norm_tensor(l, 8), exps = norm_tensor(l, 9), ew = norm_tensor(l, 10), gate = norm_tensor(l, 11);
     if ((bias >= 0 && (l.t[3] < 0 || T[bias].dtype != MPK_BF16 || T[bias].dim(0) != D)) || (row >= 0 && (T[row].dtype != MPK_BF16 || T[row].dim(0) != D)) ||
         (add >= 0 && (T[add].dtype != MPK_F32 || T[add].dims.size() != 2 || T[add].dim(1) != D)))
@@ -1425,8 +1442,8 @@ struct Builder {
       return fail(MPK_ERR_INVALID, "residual_norm: expert outputs float32 [tokens, slots, width] with weights [tokens, slots]");
     if (gate >= 0 && (l.t[1] < 0 || T[gate].dtype != MPK_F32 || l.params.size() < 4 || l.params[3] < 0 || l.params[3] >= T[gate].dim(1)))
       return fail(MPK_ERR_INVALID, "residual_norm: gate column of a float32 tensor");
-    if (l.t[2] >= 0 && (exps >= 0 || gate >= 0 || (norm_flags(l) & 4)))
-      return fail(MPK_ERR_UNSUPPORTED, "residual_norm: a norm of y goes with RMS norms and without experts");
+    if (l.t[2] >= 0 && (gate >= 0 || (norm_flags(l) & 4) || (l.t[1] < 0 && exps < 0)))
+      return fail(MPK_ERR_UNSUPPORTED, "residual_norm: a norm of y (or of the experts' sum) goes with RMS norms and without a gate");
     if (l.t[4] >= 0 && (T[l.t[4]].dtype != act_dtype() || T[l.t[4]].dim(1) < D)) return fail(MPK_ERR_INVALID, "residual_norm: output type or width");
     const TensorInfo &xo = T[resnorm_out(l)];
     if (xo.dtype != MPK_F32 || xo.dim(1) != D) return fail(MPK_ERR_INVALID, "residual_norm: the new stream must be float32 of x's width");
@@ -1448,6 +1465,7 @@ struct Builder {
       d.a[RN_LDADD] = add >= 0 ? (int)T[add].ld() : 0;
       d.a[RN_SLOTS] = exps >= 0 ? (int)T[exps].dim(1) : 0;
       d.a[RN_LDEW] = ew >= 0 ? (int)T[ew].ld() : 0;
+      d.a[RN_POST] = norm_factor(l);
       put((i + rot) % W, d, ex);
     }
     return MPK_OK;
@@ -1455,29 +1473,39 @@ struct Builder {
 
   int emit_qkv_append(int li, int ex) {
     const LayerInfo &l = L[li];
-    const TensorInfo &pr = T[l.t[0]], &q = T[l.t[1]], &kc = T[l.t[2]], &vc = T[l.t[3]], &cs = T[l.t[4]], &sn = T[l.t[5]];
+    const bool caches = l.t[2] >= 0;   // else queries only
+    if (caches != (l.t[3] >= 0)) return fail(MPK_ERR_INVALID, "qkv_append: both caches or none");
+    const TensorInfo &pr = T[l.t[0]], &q = T[l.t[1]], &kc = T[l.t[caches ? 2 : 1]], &vc = T[l.t[caches ? 3 : 1]], &cs = T[l.t[4]], &sn = T[l.t[5]];
     if (l.params.size() < 10) return fail(MPK_ERR_INVALID, "qkv_append needs 10 parameters");
     const int hq = (int)l.params[0], hkv = (int)l.params[1], dim = (int)l.params[2], vdim = (int)l.params[3], rdim = (int)l.params[7];
+    const int pairs = l.params.size() > 10 ? (int)l.params[10] : 0, maps = l.params.size() > 11 ? (int)l.params[11] : 1;
     if (!batch_meta_given()) return fail(MPK_ERR_INVALID, "qkv_append needs the batch meta tensors");
-    if (pr.dtype != MPK_F32 || q.dtype != act_dtype() || kc.dtype != act_dtype() || vc.dtype != act_dtype() || cs.dtype != MPK_F32 || sn.dtype != MPK_F32)
+    if (pr.dtype != MPK_F32 || q.dtype != act_dtype() || (caches && (kc.dtype != act_dtype() || vc.dtype != act_dtype())) || cs.dtype != MPK_F32 || sn.dtype != MPK_F32)
       return fail(MPK_ERR_INVALID, "qkv_append: float32 projections and tables, q and caches of the graph's activation type");
-    if (hq < 1 || hkv < 1 || hq % hkv || dim < 1 || vdim < 1 || rdim < 0 || rdim > dim || rdim % 2)
+    if (hq < 1 || hkv < 1 || hq % hkv || dim < 1 || vdim < 1 || rdim < 0 || rdim > dim || rdim % 2 || maps < 1 || maps > 2)
       return fail(MPK_ERR_INVALID, "qkv_append: head counts or sizes");
-    if (kc.dims.size() != 4 || vc.dims.size() != 4 || kc.dim(1) != cfg.page_size || vc.dim(1) != cfg.page_size || kc.dim(2) != hkv ||
-        vc.dim(2) != hkv || kc.dim(3) < dim || vc.dim(3) < vdim || kc.dim(3) % 8 || vc.dim(3) % 8 || q.dim(1) != hq * kc.dim(3))
+    const int dimp = caches && kc.dims.size() == 4 ? (int)kc.dim(3) : (int)q.dim(1) / (hq * maps);
+    for (int i : {6, 7})
+      if (norm_tensor(l, i) >= 0 && (T[l.t[i]].dtype != MPK_BF16 || T[l.t[i]].dim(0) < dim || l.params[8])) return fail(MPK_ERR_INVALID, "qkv_append: bf16 norm weights [dim], no unit norm beside them");
+    if (!caches) {
+      if (dimp < maps * dim || dimp % 8 || q.dim(1) != (int64_t)hq * maps * dimp || l.params[4] + (int64_t)hq * maps * dim > pr.dim(1)) return fail(MPK_ERR_INVALID, "qkv_append: q [tokens, heads x head size rounded up to 8], columns inside the projections");
+    } else if (kc.dims.size() != 4 || vc.dims.size() != 4 || kc.dim(1) != cfg.page_size || vc.dim(1) != cfg.page_size || kc.dim(2) != hkv ||
+        vc.dim(2) != hkv || kc.dim(3) < maps * dim || vc.dim(3) < vdim || kc.dim(3) % 8 || vc.dim(3) % 8 || q.dim(1) != hq * maps * kc.dim(3))
       return fail(MPK_ERR_INVALID, "qkv_append: caches [pages, page, kv_heads, head size rounded up to 8], q [tokens, heads x that]");
-    if (l.params[4] + (int64_t)hq * dim > pr.dim(1) || l.params[5] + (int64_t)hkv * dim > pr.dim(1) || l.params[6] + (int64_t)hkv * vdim > pr.dim(1))
+    else if (l.params[4] + (int64_t)hq * maps * dim > pr.dim(1) || l.params[5] + (int64_t)hkv * maps * dim > pr.dim(1) || l.params[6] + (int64_t)hkv * vdim > pr.dim(1))
       return fail(MPK_ERR_INVALID, "qkv_append: columns outside the projections");
     if (rdim > 0 && (cs.dims.size() != 2 || cs.dim(1) != rdim / 2 || sn.dim(1) != rdim / 2 || cs.dim(0) != sn.dim(0)))
       return fail(MPK_ERR_INVALID, "qkv_append: cos / sin tables [positions, rotated dims / 2]");
-    const int nt = std::max(1, std::min(W, (nb_max * (hq + hkv) + 7) / 8));
+    const int nt = std::max(1, std::min(W, (nb_max * (hq + (caches ? hkv : 0)) * maps + 7) / 8));
     for (int i = 0; i < nt; ++i) {
       TaskDesc d = blank(TASK_QKV_APPEND, li);
-      d.p[0] = (uint64_t)pr.ptr; d.p[1] = (uint64_t)q.ptr; d.p[2] = (uint64_t)kc.ptr; d.p[3] = (uint64_t)vc.ptr;
+      d.p[0] = (uint64_t)pr.ptr; d.p[1] = (uint64_t)q.ptr; d.p[2] = caches ? (uint64_t)kc.ptr : 0; d.p[3] = caches ? (uint64_t)vc.ptr : 0;
       d.p[4] = (uint64_t)cs.ptr; d.p[5] = (uint64_t)sn.ptr;
+      for (int k : {6, 7}) d.p[k] = norm_tensor(l, k) >= 0 ? (uint64_t)T[l.t[k]].ptr : 0;
+      d.a[QA_PAIRS] = pairs; d.a[QA_MAPS] = maps;
       d.a[QA_T0] = i; d.a[QA_T1] = nt; d.a[QA_LDP] = (int)pr.ld();
       d.a[QA_QOFF] = (int)l.params[4]; d.a[QA_KOFF] = (int)l.params[5]; d.a[QA_VOFF] = (int)l.params[6];
-      d.a[QA_HQ] = hq; d.a[QA_HKV] = hkv; d.a[QA_DIM] = dim; d.a[QA_DIMP] = (int)kc.dim(3); d.a[QA_VDIM] = vdim; d.a[QA_VDIMP] = (int)vc.dim(3);
+      d.a[QA_HQ] = hq; d.a[QA_HKV] = hkv; d.a[QA_DIM] = dim; d.a[QA_DIMP] = dimp; d.a[QA_VDIM] = vdim; d.a[QA_VDIMP] = caches ? (int)vc.dim(3) : 0;
       d.a[QA_ROT] = rdim; d.a[QA_NORM] = (int)l.params[8]; d.a[QA_EPS] = bits_of(l.params[9]); d.a[QA_PAGE] = cfg.page_size;
       d.a[QA_LDQ] = (int)q.ld(); d.a[QA_ROWS] = rdim > 0 ? (int)cs.dim(0) : 1;
       put((i + rot) % W, d, ex);
@@ -1495,9 +1523,12 @@ struct Builder {
         kc.dim(1) != cfg.page_size || vc.dim(1) != cfg.page_size || kc.dim(3) % 8 || vc.dim(3) % 8 || vc.dim(3) < vdim ||
         q.dim(1) != hq * kc.dim(3) || ocol < 0 || ocol + (int64_t)hq * vdim > o.dim(1))
       return fail(MPK_ERR_INVALID, "ext_attention: shapes of q, caches and output disagree");
-    if (q.dtype != act_dtype() || kc.dtype != act_dtype() || vc.dtype != act_dtype() || o.dtype != act_dtype())
-      return fail(MPK_ERR_INVALID, "ext_attention: q, caches and output must have the graph's activation type");
+    if (q.dtype != act_dtype() || kc.dtype != act_dtype() || vc.dtype != act_dtype() || (o.dtype != act_dtype() && o.dtype != MPK_F32))
+      return fail(MPK_ERR_INVALID, "ext_attention: q and caches of the graph's activation type, output of that or float32");
+    const int64_t window = l.params.size() > 9 ? l.params[9] : 0, keep = l.params.size() > 10 ? l.params[10] : 0;
+    if (window < 0 || keep < 0 || window > (1 << 30) || keep > (1 << 30)) return fail(MPK_ERR_INVALID, "ext_attention: window or kept positions");
     const bool shared = kc.storage == vc.storage, bf16 = g->hybrid == HYB_BF16;
+    if (shared && bf16 && (window > 0 || o.dtype == MPK_F32)) return fail(MPK_ERR_UNSUPPORTED, "ext_attention: no window and no float32 output with shared keys and values");
     if (shared && bf16 && (hkv != 1 || vdim % 8 || (ocol | o.ld()) % 2)) return fail(MPK_ERR_UNSUPPORTED, "ext_attention: shared keys and values have one kv head and a value size of whole 16-byte pieces");
     if (bf16 && !shared ? std::max(kc.dim(3), vc.dim(3)) > 256 : kc.dim(3) > 1024 || vdim > 512)
       return fail(MPK_ERR_UNSUPPORTED, "ext_attention: head sizes up to 256 (32-bit graphs and shared keys and values: keys up to 1024, values up to 512)");
@@ -1521,6 +1552,7 @@ struct Builder {
           TaskDesc d = blank(TASK_EXT_ATTENTION, li);
           for (int i = 0; i < 4; ++i) d.p[i] = (uint64_t)T[l.t[i]].ptr;
           d.p[4] = sinks >= 0 ? (uint64_t)T[sinks].ptr : 0;
+          d.a[XA_WINDOW] = (int)window; d.a[XA_KEEP] = (int)keep; d.a[XA_OUTF32] = o.dtype == MPK_F32 ? 1 : 0;
           d.a[XA_SHARED] = shared && bf16 ? 1 : 0; d.a[XA_KEYS] = lp.keys; d.a[XA_MERGE] = merge ? 1 : 0;
           d.a[XA_SLOT] = s; d.a[XA_HEAD] = h; d.a[XA_CHUNK] = ch; d.a[XA_NCHUNK] = NC; d.a[XA_HQ] = hq; d.a[XA_HKV] = hkv;
           d.a[XA_DIMP] = (int)kc.dim(3); d.a[XA_VDIM] = vdim; d.a[XA_VDIMP] = (int)vc.dim(3); d.a[XA_PAGE] = cfg.page_size;
@@ -1566,12 +1598,63 @@ struct Builder {
       return fail(MPK_ERR_INVALID, "short_conv: float32 input, output and state [slots, taps - 1, channels], bf16 taps");
     for (int i : {1, 3})
       if (l.t[i] >= 0 && (T[l.t[i]].dtype != MPK_BF16 || T[l.t[i]].dim(0) != C)) return fail(MPK_ERR_INVALID, "short_conv: bf16 biases [channels]");
+    const int copy = norm_tensor(l, 6);
+    if (copy >= 0 && (T[copy].dtype != act_dtype() || T[copy].dim(1) < C)) return fail(MPK_ERR_INVALID, "short_conv: copy of the output in the graph's activation type");
     const int nt = std::max(1, std::min(W, C / 32));
     for (int i = 0; i < nt; ++i) {
       TaskDesc d = blank(TASK_SHORT_CONV, li);
       for (int k = 0; k < 6; ++k) d.p[k] = l.t[k] >= 0 ? (uint64_t)T[l.t[k]].ptr : 0;
+      d.p[6] = copy >= 0 ? (uint64_t)T[copy].ptr : 0; d.a[8] = copy >= 0 ? (int)T[copy].ld() : 0;
       d.a[0] = (int)((int64_t)C * i / nt); d.a[1] = (int)((int64_t)C * (i + 1) / nt); d.a[2] = C; d.a[3] = taps;
       d.a[4] = (int)x.ld(); d.a[5] = (int)l.params[0]; d.a[6] = (int)o.ld(); d.a[7] = (int)l.params[1];
+      put((i + rot) % W, d, ex);
+    }
+    return MPK_OK;
+  }
+
+  int emit_selective_scan(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &u = T[l.t[0]], &low = T[l.t[1]], &gate = T[l.t[2]], &dt = T[l.t[3]], &st = T[l.t[7]], &o = T[l.t[8]];
+    if (l.params.size() < 3 || dt.dims.size() != 2) return fail(MPK_ERR_INVALID, "selective_scan: dt weight [channels, rank], params [rank, n, gate column]");
+    const int C = (int)dt.dim(0), rank = (int)l.params[0], n = (int)l.params[1], np = round_up(n, 4);
+    if (!batch_meta_given()) return fail(MPK_ERR_INVALID, "selective_scan needs the batch meta tensors");
+    if (n > 128) return fail(MPK_ERR_UNSUPPORTED, "selective_scan: state sizes up to 128");
+    if (rank < 1 || n < 1 || u.dtype != MPK_F32 || low.dtype != MPK_F32 || gate.dtype != MPK_F32 || st.dtype != MPK_F32 || o.dtype != act_dtype() ||
+        u.dim(1) < C || low.dim(1) < rank + 2 * n || l.params[2] < 0 || l.params[2] + C > gate.dim(1) || o.dim(1) < C || st.dims.size() != 3 ||
+        st.dim(0) < cfg.max_num_batched_requests || st.dim(1) != C || st.dim(2) != np)
+      return fail(MPK_ERR_INVALID, "selective_scan: float32 inputs and state [slots, channels, n rounded up to 4], output of the activation type");
+    for (int i = 3; i < 7; ++i)
+      if (T[l.t[i]].dtype != MPK_BF16 || (int64_t)(T[l.t[i]].bytes / 2) != (int64_t)C * (i == 3 ? rank : i == 5 ? n : 1) ||
+          (T[l.t[i]].dims.size() == 2 && T[l.t[i]].strides[1] != 1))
+        return fail(MPK_ERR_INVALID, "selective_scan: bf16 dt weight [channels, rank], dt bias, A_log [channels, n] and D");
+    const int nt = std::max(1, std::min(W, C / 8));
+    for (int i = 0; i < nt; ++i) {
+      TaskDesc d = blank(TASK_SELECTIVE_SCAN, li);
+      for (int k = 0; k < 7; ++k) d.p[k] = (uint64_t)T[l.t[k]].ptr;
+      d.p[7] = (uint64_t)o.ptr;
+      put_wide(&d, SS_STATE, l.t[7]);
+      d.a[SS_C0] = (int)((int64_t)C * i / nt); d.a[SS_C1] = (int)((int64_t)C * (i + 1) / nt); d.a[SS_C] = C; d.a[SS_RANK] = rank; d.a[SS_N] = n;
+      d.a[SS_NP] = np; d.a[SS_LANES] = scan_lanes(n); d.a[SS_LDU] = (int)u.ld(); d.a[SS_LDL] = (int)low.ld(); d.a[SS_LDG] = (int)gate.ld();
+      d.a[SS_GOFF] = (int)l.params[2]; d.a[SS_LDO] = (int)o.ld();
+      put((i + rot) % W, d, ex);
+    }
+    g->weight_bytes += (int64_t)C * (rank + n + 2) * 2;
+    return MPK_OK;
+  }
+
+  int emit_diff_combine(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &x = T[l.t[0]], &o = T[l.t[1]];
+    if (l.params.size() < 5) return fail(MPK_ERR_INVALID, "diff_combine needs 5 parameters");
+    const int H = (int)l.params[0], vdim = (int)l.params[1];
+    if (H < 1 || vdim < 1 || x.dtype != MPK_F32 || o.dtype != act_dtype() || x.dim(1) < (int64_t)2 * H * vdim || o.dim(1) < (int64_t)H * vdim)
+      return fail(MPK_ERR_INVALID, "diff_combine: float32 maps [tokens, heads x 2 x vdim], output [tokens, heads x vdim] of the activation type");
+    const int nt = std::max(1, std::min(W, (nb_max * H + 7) / 8));
+    for (int i = 0; i < nt; ++i) {
+      TaskDesc d = blank(TASK_DIFF_COMBINE, li);
+      d.p[0] = (uint64_t)x.ptr; d.p[1] = (uint64_t)o.ptr;
+      d.a[0] = i; d.a[1] = nt; d.a[2] = H; d.a[3] = vdim; d.a[4] = (int)x.ld(); d.a[5] = (int)o.ld();
+      for (int k = 0; k < 3; ++k) d.a[6 + k] = bits_of(l.params[2 + k]);
       put((i + rot) % W, d, ex);
     }
     return MPK_OK;
@@ -1673,6 +1756,8 @@ struct Builder {
       case MPK_OP_EXT_ATTENTION: return emit_ext_attention(li, ex);
       case MPK_OP_SHORT_CONV: return emit_short_conv(li, ex);
       case MPK_OP_RGLRU: return emit_rglru(li, ex);
+      case MPK_OP_SELECTIVE_SCAN: return emit_selective_scan(li, ex);
+      case MPK_OP_DIFF_COMBINE: return emit_diff_combine(li, ex);
       case MPK_OP_MLSTM: return emit_mlstm(li, ex);
       case MPK_OP_GLA: return emit_gla(li, ex);
       case MPK_OP_LATENT_APPEND: return emit_latent_append(li, ex);
@@ -1687,17 +1772,18 @@ struct Builder {
       case MPK_OP_MOE_TOPK_SOFTMAX: {
         // the same task as the sigmoid routing with one group, no bias and scaling 1: only the score function differs
         const TensorInfo &lg = T[l.t[0]], &w = T[l.t[1]], &idx = T[l.t[2]], &mask = T[l.t[3]];
-        const int E = (int)lg.dim(1), topk = (int)w.dim(1);
-        if ((lg.dtype != MPK_BF16 && lg.dtype != MPK_F32) || w.dtype != MPK_F32 || idx.dtype != MPK_I32 || mask.dtype != MPK_I32 ||
+        const int E = g->hybrid ? (int)idx.dim(0) : (int)lg.dim(1), topk = (int)w.dim(1);
+        if (lg.dim(1) < E || (lg.dtype != MPK_BF16 && lg.dtype != MPK_F32) || w.dtype != MPK_F32 || idx.dtype != MPK_I32 || mask.dtype != MPK_I32 ||
             E > 1024 || idx.dim(0) != E || mask.dim(0) != E + 1 || topk <= 0 || topk > std::min(E, 32) || idx.dim(1) > kMaxLinearTokens)
           return fail(MPK_ERR_UNSUPPORTED, "softmax routing: logits bf16/f32 [B, E <= 1024], weights f32 [B, topk <= 32], indices and mask int32");
         TaskDesc d = blank(TASK_MOE_ROUTING, li);
         d.p[0] = (uint64_t)lg.ptr; d.p[1] = 0; d.p[2] = (uint64_t)w.ptr; d.p[3] = (uint64_t)idx.ptr; d.p[4] = (uint64_t)mask.ptr;
-        d.a[0] = E; d.a[1] = topk; d.a[2] = 1; d.a[3] = 1; d.a[4] = float_bits(1.0f); d.a[5] = (int)lg.ld();
+        d.a[0] = E; d.a[1] = topk; d.a[2] = 1; d.a[3] = 1; d.a[4] = l.params.size() > 3 ? bits_of(l.params[3]) : float_bits(1.0f); d.a[5] = (int)lg.ld();
         d.a[6] = (int)w.ld(); d.a[7] = (int)idx.dim(1); d.a[8] = lg.dtype == MPK_F32 ? 1 : 0;
         d.a[9] = l.params.size() > 1 ? (int)l.params[0] : 0;
         d.a[10] = l.params.size() > 1 ? (int)l.params[1] : E;
         d.a[11] = 1;   // softmax scores, logits left in place
+        d.a[13] = l.params.size() > 2 ? (int)l.params[2] : 0;
         if (d.a[9] < 0 || d.a[10] > E || d.a[9] >= d.a[10]) return fail(MPK_ERR_INVALID, "softmax routing: bad local expert range");
         put(rot % W, d, ex);
         return MPK_OK;
@@ -2266,7 +2352,7 @@ std::string dump_task_graph(const CompiledGraph &g, const std::vector<TensorInfo
                                 "quantize_fp8", "moe_routing", "moe_gemm", "moe_silu_mul", "moe_mul_sum_add",
                                 "mla_append", "mla_decode", "mla_reduce", "sampling_partial", "sampling_reduce", "argmax_exchange", "ar_push",
                                 "embed_f32", "residual_norm", "linear_f32", "qkv_append", "ext_attention", "short_conv", "rglru", "mlstm",
-                                "gla", "latent_append", "moe_gemm_f32", "attn_merge"};
+                                "gla", "latent_append", "moe_gemm_f32", "attn_merge", "selective_scan", "diff_combine"};
   std::ostringstream os;
   os << "{\"num_workers\": " << g.num_workers << ", \"num_tasks\": " << g.tasks.size()
      << ", \"num_events\": " << g.num_events << ", \"num_layers\": " << layers.size()

@@ -335,13 +335,14 @@ class PersistentKernel:
     LINEAR_ACTIVATIONS = {None: 0, "relu2": 1, "softcap": 2, "gated_silu": 3, "gated_gelu_tanh": 4}
 
     def linear_layer(self, input: DTensor, weight: DTensor, output: DTensor, grid_dim: tuple, block_dim: tuple,
-                     activation: str = None, softcap: float = 0.0):
+                     activation: str = None, softcap: float = 0.0, bias: Optional[DTensor] = None):
         """`activation` (hybrid graphs) is applied to the fp32 accumulator before the store: squared relu, softcap * tanh(y /
-        softcap), or a gated form act(gate) * up over weight rows from `interleave_gated`, which has half as many outputs."""
+        softcap), or a gated form act(gate) * up over weight rows from `interleave_gated`, which has half as many outputs.
+        `bias` (hybrid graphs, bf16 [rows of the weight]) joins a float32 output."""
         assert input.num_dims == 2 and weight.num_dims == 2 and output.num_dims == 2
         act = self.LINEAR_ACTIVATIONS[activation]
         params = [act, self._bits(softcap)] if activation == "softcap" else [act] if act else []
-        self._layer(N.OP_LINEAR, [input, weight, output], grid_dim, params)
+        self._layer(N.OP_LINEAR, [input, weight, output] + ([bias] if bias is not None else []), grid_dim, params)
 
     @staticmethod
     def interleave_gated(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
@@ -435,16 +436,19 @@ class PersistentKernel:
                                    block_dim=block_dim)
 
     def moe_topk_softmax_routing_layer(self, input: DTensor, output: tuple, grid_dim: tuple, block_dim: tuple,
-                                       local_experts: tuple = None):
+                                       local_experts: tuple = None, renormalize: bool = True, scale: float = 1.0):
         """Softmax top-k routing (python/mirage/mpk/persistent_kernel.py:1385-1406, tasks/blackwell/topk_softmax_sm100.cuh):
         softmax over the experts in fp32, the k largest probabilities (ties to the lower expert), weights renormalised over
         the selected ones; routing_indices[e, b] = 1-based slot or 0, the list of active experts with its count in the last
         entry.  The logits are left untouched.  `local_experts`: as for the sigmoid routing (the reference task's
-        start_expert / end_expert)."""
+        start_expert / end_expert).  `renormalize=False` keeps the probabilities as weights; `scale` multiplies the weights.  Hybrid
+        graphs may pass a wider tensor whose leading columns are the logits."""
         assert input.num_dims == 2 and len(output) == 3
         w, idx, mask = output
         assert w.num_dims == 2 and idx.num_dims == 2 and mask.num_dims == 1
         params = [] if local_experts is None else [int(local_experts[0]), int(local_experts[1])]
+        if not renormalize or scale != 1.0:
+            params = (params or [0, idx.dim(0)]) + [int(not renormalize), self._bits(scale)]
         self._layer(N.OP_MOE_TOPK_SOFTMAX, [input, w, idx, mask], grid_dim, params)
 
     def silu_mul_layer(self, input: DTensor, output: DTensor, grid_dim: tuple, block_dim: tuple):
@@ -530,45 +534,57 @@ class PersistentKernel:
                             norm_bias: Optional[DTensor] = None, added: Optional[DTensor] = None,
                             added_row: Optional[DTensor] = None,
                             experts: Optional[Tuple[DTensor, DTensor]] = None,
-                            y_gate: Optional[Tuple[DTensor, int]] = None):
-        """x += rmsnorm(y) * w_post on the float32 stream `x` (x += y without `post_weight`, x unchanged without `y`),
-        then output = rmsnorm(x) * w_norm.  `zero_centered`: both weights are stored around zero (1 + w is applied).
+                            y_gate: Optional[Tuple[DTensor, int]] = None, post_factor: float = 1.0):
+        """x += post_factor * rmsnorm(y) * w_post on the float32 stream `x` (x += y without `post_weight`, x unchanged without `y`),
+        then output = rmsnorm(x) * w_norm (without `norm_weight`: x as it is).  `zero_centered`: both weights are stored around zero (1 + w is applied).
         `x_out` receives the new stream instead of `x`; with it, graphs of one or two tokens fold the layer into the linear
         that reads `output`.  `layer_norm` makes the output norm a layer norm (with `norm_bias`) instead of an RMS norm.
         Further terms of the sum: `added` (float32 [tokens, width]), `added_row` (bf16 [width], for every token), `experts`
         (outputs [tokens, slots, width] and weights [tokens, slots], both float32); `y_gate` = (float32 tensor, column)
-        multiplies `y` by the column's sigmoid."""
+        multiplies `y` by the column's sigmoid.  With `post_weight` the experts' weighted sum joins `y` in front of its norm."""
         assert x.num_dims == 2
         gate, column = y_gate if y_gate else (None, 0)
         exp_out, exp_w = experts if experts else (None, None)
         self._layer(N.OP_RESIDUAL_NORM, [x, y, post_weight, norm_weight, output, x_out, norm_bias, added, added_row, exp_out,
                                          exp_w, gate], (1, 1, 1),
-                    [self._bits(eps), int(zero_centered), int(layer_norm), column])
+                    [self._bits(eps), int(zero_centered), int(layer_norm), column, self._bits(post_factor)])
 
-    def qkv_append_layer(self, proj: DTensor, q: DTensor, k_cache: DTensor, v_cache: DTensor, cos: DTensor, sin: DTensor,
-                         *, heads: int, kv_heads: int, dim: int, vdim: int, q_col: int, k_col: int, v_col: int,
-                         rot_dims: int, unit_norm: bool, eps: float):
+    def qkv_append_layer(self, proj: DTensor, q: DTensor, k_cache: Optional[DTensor], v_cache: Optional[DTensor], cos: DTensor,
+                         sin: DTensor, *, heads: int, kv_heads: int, dim: int, vdim: int, q_col: int, k_col: int = 0, v_col: int = 0,
+                         rot_dims: int, unit_norm: bool = False, eps: float, q_norm: Optional[DTensor] = None,
+                         k_norm: Optional[DTensor] = None, interleaved: bool = False, maps: int = 1):
         """Takes q / k / v columns of the float32 projections: rotates the first `rot_dims` of q and k (half-split pairs,
         float32 tables [positions, rot_dims / 2]), divides them by their RMS (`unit_norm`), and writes q and the cache
-        rows of the new positions.  Values are taken as projected; `v_col == k_col` makes the keys the values."""
-        self._layer(N.OP_QKV_APPEND, [proj, q, k_cache, v_cache, cos, sin], (1, 1, 1),
-                    [heads, kv_heads, dim, vdim, q_col, k_col, v_col, rot_dims, int(unit_norm), self._bits(eps)])
+        rows of the new positions.  Values are taken as projected; `v_col == k_col` makes the keys the values.  Without caches
+        only queries are formed (a layer that reads another layer's keys and values).  `q_norm`, `k_norm` (bf16 [dim]): RMS norms
+        in front of the rotation instead.  `interleaved`: neighbours are rotated together.  `maps=2` (differential attention):
+        heads have two vectors of `dim` columns side by side in the projections; a cache row holds both, and `q` has two rows
+        per head, each with its own vector and zeros for the other."""
+        self._layer(N.OP_QKV_APPEND, [proj, q, k_cache, v_cache, cos, sin, q_norm, k_norm], (1, 1, 1),
+                    [heads, kv_heads, dim, vdim, q_col, k_col, v_col, rot_dims, int(unit_norm), self._bits(eps), int(interleaved), maps])
 
     def ext_attention_layer(self, q: DTensor, k_cache: DTensor, v_cache: DTensor, output: DTensor, *, heads: int,
                             kv_heads: int, vdim: int, scale: float, softcap: float = 0.0, sink: bool = False,
                             sinks: Optional[DTensor] = None, out_col: int = 0, out_scale: float = 1.0,
-                            separate_merge: bool = False):
+                            separate_merge: bool = False, window: int = 0, keep_first: int = 0):
         """Causal paged attention over rows a qkv_append_layer or latent_append_layer wrote.  score = softcap *
         tanh(scale * q.k / softcap) (no cap at 0); `sink` adds one to the softmax denominator, `sinks` (bf16 [heads]) adds
         exp(sinks[head]); the result times `out_scale` goes to columns [out_col, out_col + heads * vdim) of `output`.
         `v_cache` may be `k_cache`: the leading `vdim` columns of a key are then its value.  `separate_merge`: the key chunks of
-        a request are merged by all workers in a layer of its own (for wide values) instead of by the last task to arrive."""
+        a request are merged by all workers in a layer of its own (for wide values) instead of by the last task to arrive.
+        `window` > 0: a position sees itself, the window - 1 positions before it and the first `keep_first`; keys outside are
+        not read.  A float32 `output` is allowed in bf16 graphs."""
         args = ([q, k_cache, v_cache, output, sinks], (1, 1, 1),
                 [heads, kv_heads, vdim, out_col, self._bits(scale), self._bits(softcap or 0.0), int(sink or sinks is not None),
-                 self._bits(out_scale), int(separate_merge)])
+                 self._bits(out_scale), int(separate_merge), int(window), int(keep_first)])
         self._layer(N.OP_EXT_ATTENTION, *args)
         if separate_merge:
             self._layer(N.OP_ATTN_MERGE, *args)
+
+    def diff_combine_layer(self, maps: DTensor, output: DTensor, *, heads: int, vdim: int, lam: float, factor: float, eps: float):
+        """Differential attention (Ye et al., "Differential Transformer"): `maps` (float32 [tokens, heads * 2 * vdim], two rows
+        per head) -> factor * unit norm of (map 1 - lam * map 2) per head."""
+        self._layer(N.OP_DIFF_COMBINE, [maps, output], (1, 1, 1), [heads, vdim, self._bits(lam), self._bits(factor), self._bits(eps)])
 
     def latent_append_layer(self, proj: DTensor, latent_norm: DTensor, q: DTensor, cache: DTensor, cos: DTensor, sin: DTensor,
                             *, heads: int, rank: int, rot_dims: int, q_col: int, kv_col: int, eps: float):
@@ -581,10 +597,11 @@ class PersistentKernel:
 
     def short_conv_layer(self, input: DTensor, taps: DTensor, state: DTensor, output: DTensor, *,
                          input_bias: Optional[DTensor] = None, bias: Optional[DTensor] = None, in_col: int = 0,
-                         activation: str = None):
+                         activation: str = None, copy: Optional[DTensor] = None):
         """Causal convolution per channel over columns [in_col, in_col + channels) of `input` (+ `input_bias`); the last
-        taps - 1 inputs of a request live in `state` [slots, taps - 1, channels]."""
-        self._layer(N.OP_SHORT_CONV, [input, input_bias, taps, bias, state, output], (1, 1, 1),
+        taps - 1 inputs of a request live in `state` [slots, taps - 1, channels].  `copy` receives the output in the activation
+        type (the operand of a linear behind it)."""
+        self._layer(N.OP_SHORT_CONV, [input, input_bias, taps, bias, state, output, copy], (1, 1, 1),
                     [in_col, {None: 0, "silu": 1}[activation]])
 
     def rglru_layer(self, u: DTensor, proj: DTensor, y_bias: DTensor, ra: DTensor, ra_bias: DTensor, ri: DTensor,
@@ -595,6 +612,14 @@ class PersistentKernel:
         log a = -decay * r * softplus(lam), output out_scale * S * gelu_tanh(proj[:, y_col:] + y_bias)."""
         self._layer(N.OP_RGLRU, [u, proj, y_bias, ra, ra_bias, ri, ri_bias, lam, state, output], (1, 1, 1),
                     [y_col, out_col, self._bits(out_scale), self._bits(decay)])
+
+    def selective_scan_layer(self, u: DTensor, low: DTensor, gate: DTensor, dt: DTensor, dt_bias: DTensor, a_log: DTensor, d: DTensor,
+                             state: DTensor, output: DTensor, *, rank: int, n: int, gate_col: int):
+        """Selective state space recurrence (Gu and Dao, "Mamba: Linear-Time Sequence Modeling with Selective State Spaces"): a
+        state of `n` values per channel, float32 [slots, channels, n up to a multiple of 4].  `low` holds [step sizes' low-rank
+        part | B | C]; step sizes softplus(dt . low[:, :rank] + dt_bias), decays exp(-step * exp(a_log)); the read-out plus d * u is
+        multiplied by silu of the gate columns."""
+        self._layer(N.OP_SELECTIVE_SCAN, [u, low, gate, dt, dt_bias, a_log, d, state, output], (1, 1, 1), [rank, n, gate_col])
 
     @staticmethod
     def mlstm_chunks(num_workers: int, slots: int, heads: int, dim: int, vdim: int) -> int:
@@ -651,7 +676,7 @@ class PersistentKernel:
     def moe_w13_linear_layer(self, input: DTensor, weight: DTensor, moe_routing_indices: DTensor, moe_mask: DTensor,
                              output: DTensor, grid_dim: tuple, block_dim: tuple, first_expert: int = 0,
                              activation: str = None):
-        """`activation` (hybrid graphs): a gated form over rows from `interleave_gated`, output [B, topk, >= I]."""
+        """`activation` (hybrid graphs): a gated form over rows from `interleave_gated`, or squared relu; output [B, topk, >= I]."""
         assert input.num_dims == 2 and weight.num_dims == 3 and output.num_dims == 3
         act = self.LINEAR_ACTIVATIONS[activation]
         self._layer(N.OP_MOE_W13_LINEAR, [input, weight, moe_routing_indices, moe_mask, output], grid_dim,

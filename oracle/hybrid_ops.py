@@ -6,7 +6,7 @@ float64).  Shares nothing with the product path.
 from __future__ import annotations
 
 import math
-from typing import Dict, Optional, Tuple
+from typing import Dict, Optional, Sequence, Tuple
 
 import torch
 
@@ -193,3 +193,88 @@ def grouped_choice(scores: Tensor, correction: Tensor, groups: int, keep: int, t
 
 def softcap(z: Tensor, cap: float) -> Tensor:
     return cap * torch.tanh(z / cap)
+
+
+def rms_norm(x: Tensor, w: Tensor, eps: float) -> Tensor:
+    return rms_unit(x, eps) * w
+
+
+def rotary_frequencies(base: float, dims: int, scaling: Optional[Dict[str, float]] = None) -> list:
+    """Angle per position of every pair.  `scaling`: long wavelengths are stretched by `factor`, short ones kept, those between
+    original / high and original / low blended."""
+    out = []
+    for i in range(dims // 2):
+        f = base ** (-2.0 * i / dims)
+        if scaling:
+            waves = scaling["original"] * f / (2 * math.pi)        # turns within the original length
+            if waves < scaling["low"]:
+                f = f / scaling["factor"]
+            elif waves <= scaling["high"]:
+                s = (waves - scaling["low"]) / (scaling["high"] - scaling["low"])
+                f = (1 - s) * f / scaling["factor"] + s * f
+        out.append(f)
+    return out
+
+
+def rotate_pairs(x: Tensor, pos: Tensor, freqs: Sequence[float], interleaved: bool) -> Tensor:
+    """x [tokens, heads, size]; pair i is (i, i + n) of the first 2 n components, or (2 i, 2 i + 1), n = len(freqs)."""
+    out = x.clone()
+    for i, f in enumerate(freqs):
+        a, b = (2 * i, 2 * i + 1) if interleaved else (i, i + len(freqs))
+        c, s = torch.cos(pos.to(x.dtype) * f)[:, None], torch.sin(pos.to(x.dtype) * f)[:, None]
+        out[..., a] = x[..., a] * c - x[..., b] * s
+        out[..., b] = x[..., b] * c + x[..., a] * s
+    return out
+
+
+def visible(i: int, window: int = 0, keep_first: int = 0) -> list:
+    """Keys position i sees: itself and the window - 1 before it (all before it without a window), and the first `keep_first`."""
+    return [j for j in range(i + 1) if not window or i - j < window or j < keep_first]
+
+
+def window_attention(q: Tensor, k: Tensor, v: Tensor, scale: float, window: int = 0, keep_first: int = 0, sink: bool = False) -> Tensor:
+    """Grouped heads over the visible keys; `sink` adds one to the softmax denominator."""
+    T, H = q.shape[:2]
+    G = k.shape[1]
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for t in range(T):
+        at = torch.tensor(visible(t, window, keep_first))
+        for h in range(H):
+            g = h // (H // G)
+            s = (k[at, g] @ q[t, h]) * scale
+            top = torch.clamp(s.max(), min=0.0) if sink else s.max()
+            e = torch.exp(s - top)
+            out[t, h] = (e / (e.sum() + (torch.exp(-top) if sink else 0.0))) @ v[at, g]
+    return out
+
+
+def diff_lambda(lq1: Tensor, lk1: Tensor, lq2: Tensor, lk2: Tensor, diff: float) -> Tensor:
+    return torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum()) + diff
+
+
+def diff_combine(a1: Tensor, a2: Tensor, lam: Tensor, diff: float, eps: float) -> Tensor:
+    """The two maps' outputs [.., vdim] -> unit norm of their difference, times 1 - diff."""
+    return rms_unit(a1 - lam * a2, eps) * (1 - diff)
+
+
+def diff_attention(q: Tensor, k: Tensor, v: Tensor, scale: float, lam: Tensor, diff: float, eps: float, window: int = 0) -> Tensor:
+    """q [tokens, H, 2, d], k [tokens, G, 2, d], v [tokens, G, dv]: one attention per map over the same values."""
+    a1, a2 = (window_attention(q[:, :, m], k[:, :, m], v, scale, window) for m in range(2))
+    return diff_combine(a1, a2, lam, diff, eps)
+
+
+def selective_scan(x: Tensor, dt: Tensor, A: Tensor, B: Tensor, C: Tensor, D: Tensor) -> Tensor:
+    """x, dt [tokens, channels], A [channels, n], B, C [tokens, n] -> read-outs [tokens, channels]."""
+    S = torch.zeros_like(A)
+    out = torch.zeros_like(x)
+    for t in range(x.shape[0]):
+        S = torch.exp(dt[t][:, None] * A) * S + (dt[t] * x[t])[:, None] * B[t][None, :]
+        out[t] = S @ C[t] + D * x[t]
+    return out
+
+
+def softmax_choice(logits: Tensor, top: int) -> Tuple[list, Tensor]:
+    """Experts of one token with their weights: the largest probabilities, as they are."""
+    p = torch.softmax(logits, -1)
+    chosen = sorted(range(p.shape[0]), key=lambda e: -float(p[e]))[:top]
+    return chosen, p[torch.tensor(chosen)]
