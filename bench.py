@@ -857,14 +857,69 @@ def lofirax_case(size, dev):
     return c, w
 
 
+# Bebuzen at sizes like those: 4 selective-scan layers, 2 layers of windowed attention with a sink, 2 of differential attention over one
+# cache; every second feed-forward with (ungated) experts of the same bytes as Lofirax's gated ones.
+BEBUZEN_SIZES = {
+    "4096": dict(inner=8192, state=16, rank=256, heads=32, kv=8, dim=128, dheads=16, ff=12288, experts=32, top=4, eff=1536, shared=3072),
+    "2048": dict(inner=4096, state=16, rank=128, heads=16, kv=8, dim=128, dheads=8, ff=6144, experts=64, top=6, eff=768, shared=1536),
+}
+
+
+def bebuzen_case(size, dev):
+    """(config, device weights) of one size; random weights."""
+    import torch
+    z, y = HYBRID_SIZES[size], BEBUZEN_SIZES[size]
+    D, E = z["width"], y["experts"]
+    moe = {"kind": "moe", "expert": {"ff": y["eff"]}, "shared": {"ff": y["shared"]}, "router": {"experts": E, "top": y["top"], "scale": 1.0}}
+    dense = {"kind": "dense", "ff": y["ff"]}
+    scan = {"type": "mamba1", "mixer": {"inner": y["inner"], "state": y["state"], "dt_rank": y["rank"], "conv": 4}}
+    sink = {"type": "attention_2", "mixer": {"heads": y["heads"], "kv_heads": y["kv"], "dim": y["dim"], "vdim": y["dim"], "scale": y["dim"] ** -0.5,
+                                             "mask": {"size": 1024, "keep_first": 4}, "rot": {"base": 1e4, "dims": y["dim"]}}}
+    diff = {"heads": y["dheads"], "kv_heads": y["kv"], "dim": y["dim"] // 2, "vdim": y["dim"], "scale": (y["dim"] // 2) ** -0.5, "conv": 4, "diff": 0.5,
+            "mask": {"size": 1024}, "rot": {"base": 5e5, "dims": y["dim"] // 2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    mixers = [scan, sink, scan, {"type": "attention", "mixer": diff}, scan, {"type": "attention", "mixer": dict(diff, kv_from=3)}, scan, sink]
+    c = {"architecture": "Bebuzen", "vocab": HYBRID_VOCAB, "width": D, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+         "layers": [dict(m, mlp=moe if n % 2 else dense) for n, m in enumerate(mixers)]}
+    g = torch.Generator(device=dev).manual_seed(1)
+    rnd = lambda *s, std=None, mean=0.0: (mean + (s[-1] ** -0.5 if std is None else std) * torch.randn(
+        *s, generator=g, device=dev)).to(torch.bfloat16)
+    one = lambda n: rnd(n, std=0.1, mean=1.0)
+    w = {"embed": rnd(HYBRID_VOCAB, D, std=1.0), "head": rnd(HYBRID_VOCAB, D), "final.norm": one(D)}
+    for n, layer in enumerate(c["layers"]):
+        p, m, mlp = f"l{n}.mix.", layer["mixer"], f"l{n}.mlp."
+        w[f"l{n}.norm1"], w[f"l{n}.norm2"] = one(D), one(D)
+        if layer["type"] == "mamba1":
+            C, N, R = m["inner"], m["state"], m["dt_rank"]
+            w[p + "in"], w[p + "conv"], w[p + "conv.b"], w[p + "x"] = rnd(2 * C, D), rnd(C, 4, std=0.5), rnd(C, std=0.2), rnd(R + 2 * N, C)
+            w[p + "dt"], w[p + "dt.b"], w[p + "A_log"], w[p + "D"] = rnd(C, R), rnd(C, std=1.0, mean=-3.0), rnd(C, N, std=0.8), one(C)
+            w[p + "o"] = rnd(D, C)
+        else:
+            maps = 2 if layer["type"] == "attention" else 1
+            names = [("q", m["heads"] * maps * m["dim"])] + ([] if "kv_from" in m else [("k", m["kv_heads"] * maps * m["dim"]),
+                                                                                        ("v", m["kv_heads"] * m["vdim"])])
+            for nm, rows in names:
+                w[p + nm], w[p + nm + ".b"], w[f"{p}{nm}.conv"], w[f"{p}{nm}.norm"] = rnd(rows, D), rnd(rows, std=0.2), rnd(rows, 4, std=0.5), one(m["dim"])
+            for nm in ("lq1", "lk1", "lq2", "lk2"):
+                w[p + nm] = rnd(m["dim"], std=0.1)
+            w[p + "o"], w[p + "o.b"] = rnd(D, m["heads"] * m["vdim"]), rnd(D, std=0.1)
+        if n % 2 == 0:
+            w[mlp + "gate"], w[mlp + "up"], w[mlp + "down"] = rnd(y["ff"], D), rnd(y["ff"], D), rnd(D, y["ff"])
+            continue
+        w[mlp + "router"] = rnd(E, D)
+        for nm, ff in [("shared", y["shared"])] + [(f"e{e}", y["eff"]) for e in range(E)]:
+            w[f"{mlp}{nm}.up"], w[f"{mlp}{nm}.down"] = rnd(ff, D), rnd(D, ff)
+    return c, w
+
+
 def run_hybrid(args):
     """Prefill (one request, 64 tokens per launch) and decode (batch 1, 16, 64 at --context) of a model on hybrid graphs and of
-    its closest neighbour at equal size (palarax: Qwen3 layers, lofirax: Palarax), with the spans of every kind of task group from
-    the in-kernel profiler.  Timed launches carry no profiler."""
+    its closest neighbours at equal size (palarax: Qwen3 layers, lofirax: Palarax, bebuzen: Lofirax and Palarax), with the spans of
+    every kind of task group from the in-kernel profiler.  Timed launches carry no profiler."""
     import torch
+    from mirage_b200.builders.bebuzen import BebuzenConfig
     from mirage_b200.builders.lofirax import LofiraxConfig
     from mirage_b200.builders.palarax import PalaraxConfig
-    from mirage_b200.builders.runner import DecoderShape, LofiraxRunner, PalaraxRunner, Qwen3Runner
+    from mirage_b200.builders.runner import BebuzenRunner, DecoderShape, LofiraxRunner, PalaraxRunner, Qwen3Runner
     from mirage_b200.profiler import event_spans
     torch.cuda.set_device(0)
     dev = torch.device("cuda", 0)
@@ -916,8 +971,14 @@ def run_hybrid(args):
 
     results, launches, clk = [], 0, None
     for size, z in HYBRID_SIZES.items():
-        for model in {"palarax": ("palarax", "qwen3"), "lofirax": ("lofirax", "palarax")}[args.workload]:
-            if model == "lofirax":
+        for model in {"palarax": ("palarax", "qwen3"), "lofirax": ("lofirax", "palarax"),
+                      "bebuzen": ("bebuzen", "lofirax", "palarax")}[args.workload]:
+            if not any(args.cases in f"{model}_{size}_{k}" for k in ("prefill64", "decode1", "decode16", "decode64")):
+                continue
+            if model == "bebuzen":
+                c, w = bebuzen_case(size, dev)
+                make = lambda kw, prof: BebuzenRunner(BebuzenConfig.from_dict(c), w, profiler_tensor=prof, **kw)
+            elif model == "lofirax":
                 c, w = lofirax_case(size, dev)
                 make = lambda kw, prof: LofiraxRunner(LofiraxConfig.from_dict(c), w, profiler_tensor=prof, **kw)
             elif model == "palarax":
@@ -935,7 +996,8 @@ def run_hybrid(args):
                     continue
                 ms, wb, spans, clk, experts = case(make, B, mbt, prompt)
                 if experts:      # panels of the experts active in the last expert layer, taken for all four
-                    wb += 4 * experts[0] * 3 * LOFIRAX_SIZES[size]["eff"] * z["width"] * 2
+                    panel = 3 * LOFIRAX_SIZES[size]["eff"] if model == "lofirax" else 2 * BEBUZEN_SIZES[size]["eff"]
+                    wb += 4 * experts[0] * panel * z["width"] * 2
                 n = mbt if prompt > 1 else B
                 results.append({"case": full, "ms_per_launch": round(ms, 4), "tok_s": round(n * 1e3 / ms, 1), "weight_gb": round(wb / 1e9, 3),
                                 "weight_roofline_frac": round(wb / (ms * 1e-3) / 1e9 / peak, 3), "groups_us": spans,
@@ -950,7 +1012,9 @@ def run_hybrid(args):
         "dtype": "bf16", "data": "synthetic",
         "config": {"workload": {"palarax": "Palarax 6 matrix-memory + 2 parallel layers beside 8 Qwen3 layers, width 4096 and 2048, context %d",
                                 "lofirax": "Lofirax 6 gated-linear + 2 latent-attention layer runs (half with experts) beside Palarax 6 "
-                                           "matrix-memory + 2 parallel layers, width 4096 and 2048, context %d"}[args.workload] % ctx,
+                                           "matrix-memory + 2 parallel layers, width 4096 and 2048, context %d",
+                                "bebuzen": "Bebuzen 4 selective-scan + 2 windowed + 2 differential attention layers (half with experts) beside "
+                                           "Lofirax and Palarax layers, width 4096 and 2048, context %d"}[args.workload] % ctx,
                    "l2": "weights of a launch exceed L2; every launch re-streams them"},
         "gpu_launches": launches, "clocks": clk, "peak_gbs": peak, "peak_kind": peak_kind, "results": results}))
 
@@ -978,11 +1042,12 @@ def main():
                     help="N > 1: split the lm_head rows over the ranks and merge the ranks' argmax inside the kernel "
                          "(default: every rank keeps the whole lm_head, as the reference does)")
     ap.add_argument("--workload", default="qwen3", choices=["qwen3", "fp8_layer", "moe_block", "mla_decode", "deepseek_slice", "moe_w13", "mla_dense",
-                                                             "palarax", "lofirax"],
+                                                             "palarax", "lofirax", "bebuzen"],
                     help="qwen3: the headline decode benchmark; the others time one block of the FP8 / MoE / MLA "
-                         "task bodies at the shapes of the DeepSeek-V3-style parity configurations (1 GPU); palarax, lofirax: "
-                         "prefill and decode at a few sizes beside the closest other model's layers of equal size (Qwen3; Palarax) (1 GPU)")
-    ap.add_argument("--cases", default="", help="palarax, lofirax: only cases whose name contains this text")
+                         "task bodies at the shapes of the DeepSeek-V3-style parity configurations (1 GPU); palarax, lofirax, "
+                         "bebuzen: prefill and decode at a few sizes beside the closest other models' layers of equal size (Qwen3; Palarax; "
+                         "Lofirax and Palarax) (1 GPU)")
+    ap.add_argument("--cases", default="", help="palarax, lofirax, bebuzen: only cases whose name contains this text")
     args = ap.parse_args()
     if args.impl == "reference":
         return run_reference(args)
@@ -990,7 +1055,7 @@ def main():
         return run_ref_kernel(args)
     if args.workload == "deepseek_slice":
         return run_deepseek_slice(args)
-    if args.workload in ("palarax", "lofirax"):
+    if args.workload in ("palarax", "lofirax", "bebuzen"):
         return run_hybrid(args)
     if args.workload != "qwen3":
         return run_block_workload(args)

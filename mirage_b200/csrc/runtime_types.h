@@ -90,10 +90,10 @@ MPK_HD constexpr int ext_attention_rows(int rows) {
   return r;
 }
 
-// Selective scan: lanes that share a channel's state (four values each), slots of the ring of states to come, columns of the
+// Selective scan: lanes that share a channel's state (four values each; at least four, so that the channels of a pass fit), slots of the ring of states to come, columns of the
 // low-rank step sizes staged at a time.
 MPK_HD constexpr int scan_lanes(int n) {
-  int l = 1;
+  int l = 4;
   while (4 * l < n) l *= 2;
   return l;
 }

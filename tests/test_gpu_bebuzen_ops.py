@@ -82,14 +82,16 @@ def test_scan_states_of_many_requests_stream_through_the_ring(dtype):
 
 
 def test_scan_memory_of_a_thousand_tokens():
-    """Decays near one: what the first token wrote is read after a thousand steps, its decay accurate to the last bits."""
+    """Decays near one: what the first token wrote is read after a thousand steps.  (Steps that vary: a constant one would be rounded
+    the same way every time.)"""
     channels, n, T = 8, 4, 1024
     b = Bench(1, tokens=64, page=64, pages=16, max_seq=1024)
     u, low, gate, out = b.zeros(64, channels), b.zeros(64, 1 + 2 * n), b.zeros(64, channels), b.zeros(64, channels)
     bias = torch.linspace(-9.0, -6.0, channels).to(torch.bfloat16)          # steps of 1e-4 .. 2e-3
-    zero = lambda *s: torch.zeros(*s, dtype=torch.bfloat16)
+    w, zero = torch.full((channels, 1), 0.25, dtype=torch.bfloat16), lambda *s: torch.zeros(*s, dtype=torch.bfloat16)
+    z = torch.randn(T, generator=torch.Generator().manual_seed(1))
     b.pk.selective_scan_layer(b.pk.attach_input(u, name="u"), b.pk.attach_input(low, name="low"), b.pk.attach_input(gate, name="gate"),
-                              b.inp(zero(channels, 1), "w"), b.inp(bias, "bias"), b.inp(zero(channels, n), "a"), b.inp(zero(channels), "d"),
+                              b.inp(w, "w"), b.inp(bias, "bias"), b.inp(zero(channels, n), "a"), b.inp(zero(channels), "d"),
                               b.pk.attach_input(b.zeros(1, channels, n), name="S"), b.pk.attach_input(out, name="out"), rank=1, n=n, gate_col=0)
     mark_type(b, torch.float32)
     b.pk.compile()
@@ -97,13 +99,14 @@ def test_scan_memory_of_a_thousand_tokens():
     low[:, 1 + n:] = 1.0
     for t in range(T // 64):
         u.zero_(), low[:, 1:1 + n].zero_()
+        low[:, 0] = z[64 * t:64 * t + 64].cuda()
         if t == 0:
             u[0], low[0, 1:1 + n] = 1.0, 1.0
         b.describe([64])
         b.pk.step(1)
         b.pk.status()
-    dt = torch.nn.functional.softplus(bias.to(D))
-    ref = n * dt * torch.exp(-dt * (T - 1)) * ops.silu(torch.tensor(2.0, dtype=D))
+    dt = torch.nn.functional.softplus(bias.to(D) + 0.25 * z.to(D)[:, None])
+    ref = n * dt[0] * torch.exp(-dt[1:].sum(0)) * ops.silu(torch.tensor(2.0, dtype=D))
     assert float(((out[63].double().cpu() - ref) / ref).abs().max()) < 5e-6
 
 
@@ -204,7 +207,7 @@ def test_windowed_attention(dtype, tokens, case):
 
 
 DIFF = [(4, 2, 16, 24, 8, False, 0.3, 9, 0, False), (3, 3, 20, 12, 20, False, 0.25, 13, 0, False), (2, 1, 64, 128, 32, True, 0.1, 17, 0, False),
-        (4, 1, 48, 96, 48, False, 0.15, 7, 2, True), (5, 1, 100, 260, 10, False, 0.1, 0, 0, False), (1, 1, 9, 5, 2, False, 0.3, 6, 0, False)]
+        (4, 1, 56, 88, 56, False, 0.15, 7, 2, True), (5, 1, 100, 260, 10, False, 0.1, 0, 0, False), (1, 1, 9, 5, 2, False, 0.3, 6, 0, False)]
 
 
 @DT
@@ -230,7 +233,7 @@ def test_differential_attention(dtype, tokens, second, case):
 @DT
 @pytest.mark.parametrize("page", [8, 6])
 @pytest.mark.parametrize("maps", [1, 2])
-@pytest.mark.parametrize("window,keep", [(40, 6), (64, 0), (137, 9), (256, 64)])
+@pytest.mark.parametrize("window,keep", [(45, 5), (64, 0), (139, 9), (256, 64)])
 def test_keys_at_the_edges_of_the_window_and_of_the_kept_tokens(dtype, window, keep, maps, page):
     """Keys that stand out just inside and just outside the window and at the last kept and the next position, asked for from a prompt's
     portion and by decoded tokens, at contexts far beyond the window and before it is full."""
