@@ -1300,6 +1300,16 @@ __device__ __forceinline__ float lds_f32(uint32_t a) {
   asm volatile("ld.shared.f32 %0, [%1];" : "=f"(v) : "r"(a) : "memory");
   return v;
 }
+__device__ __forceinline__ float4 lds_f32x4(uint32_t a) {
+  float4 v;
+  asm volatile("ld.shared.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(a) : "memory");
+  return v;
+}
+__device__ __forceinline__ float2 lds_f32x2(uint32_t a) {
+  float2 v;
+  asm volatile("ld.shared.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(a) : "memory");
+  return v;
+}
 __device__ __forceinline__ int lds_s32(uint32_t a) {
   int v;
   asm volatile("ld.shared.s32 %0, [%1];" : "=r"(v) : "r"(a) : "memory");
@@ -2125,179 +2135,303 @@ __device__ __noinline__ void run_rglru(const Ctx c, const TaskDesc &d) {
 // SS_LANES neighbouring lanes share a channel, four states each, so that a block walks 256 / SS_LANES channels at a time through the
 // tokens of the batch; the step sizes' low-rank product is part of the task.  A request's state enters at its first token of the
 // batch and is written back at its last; every thread copies its own piece of the states to come into its own cells of a ring.
+// The phases are functions of their own, called one after the other: what one keeps in registers is not spilled in another's loop (a
+// further level of calls would cost every task body registers).
 // ---------------------------------------------------------------------------
-// Adds columns [r0, r0 + rn) of the low-rank product to dts [B][CP] (B <= 8: a warp takes a channel, its lanes the columns; else a
-// thread takes a channel and eight tokens).  low: [B][rn] in shared memory, rows of `pitch` floats.
-__device__ __forceinline__ void scan_steps(const TaskDesc &d, const float *low, int pitch, float *dts, int CP, int cb, int nc, int B, int r0, int rn) {
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rank = d.a[SS_RANK];
-  const bool vec = (rank & 7) == 0 && (d.p[3] & 15) == 0;   // rows of whole 16-byte pieces
-  auto eight = [&](size_t row, int k, float (&w)[8]) {      // weights k .. k + 7 of the chunk, zeros past its end
-    if (vec) {
-      const uint4 v = __ldg(reinterpret_cast<const uint4 *>(d.p[3] + 2 * (row * rank + r0 + k)));
-      const uint32_t p[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-      for (int e = 0; e < 8; ++e) w[e] = e & 1 ? bf16_hi(p[e >> 1]) : bf16_lo(p[e >> 1]);
-    } else {
-#pragma unroll
-      for (int e = 0; e < 8; ++e) w[e] = k + e < rn ? bf16_at(d.p[3], row * rank + r0 + k + e) : 0.f;
+// Shared memory of a task.
+struct ScanMem {
+  TokenRec *rec;        // [64]
+  int *seqs;            // [64] state slot of the batch's requests in order, -1: starts from zeros
+  int *tok;             // [64] state slot << 2 | first token of its request in the batch << 1 | last one
+  int *qo;              // [requests + 1]
+  float4 *ring;         // [kScanRing][256] states to come
+  __nv_bfloat16 *w;     // [CP][scan_pitch] weights of the step sizes (in the ring's place, before it is used)
+  float *bc;            // [B][2 NP] B, C
+  float *us;            // [B][CP] inputs
+  float *dts;           // [B][CP] step sizes, then read-outs
+  float *low;           // [B][scan_pitch] columns of the low-rank part; later the gate [B][CP]
+};
+__device__ __forceinline__ ScanMem scan_mem(const Ctx &c, const TaskDesc &d, int B) {
+  const int NP = d.a[SS_NP], CP = kConsumerThreads / d.a[SS_LANES];
+  ScanMem m;
+  m.rec = reinterpret_cast<TokenRec *>(c.s.xtile);
+  m.seqs = reinterpret_cast<int *>(c.s.xtile + kTokenMapBytes);
+  m.tok = m.seqs + kMaxLinearTokens;
+  m.qo = m.tok + kMaxLinearTokens;
+  m.ring = reinterpret_cast<float4 *>(m.qo + ((c.P.max_num_batched_requests + 4) & ~3));
+  m.w = reinterpret_cast<__nv_bfloat16 *>(m.ring);
+  m.bc = reinterpret_cast<float *>(reinterpret_cast<uint8_t *>(m.ring) + scan_ring_bytes(d.a[SS_RANK], CP));
+  m.us = m.bc + B * 2 * NP;
+  m.dts = m.us + B * CP;
+  m.low = m.dts + B * CP;
+  return m;
+}
+// `rows` rows of `cols` floats: 16-byte asynchronous copies where everything is aligned.
+__device__ __forceinline__ void scan_copy(float *dst, int pitch, const float *src, int ld, int rows, int cols, bool vec) {
+  const int v = vec ? cols >> 2 : cols;
+#pragma unroll 1
+  for (int i = threadIdx.x; i < rows * v; i += kConsumerThreads) {
+    const int t = i / v, j = i - t * v;
+    if (vec) cp_async16(smem_u32(dst + t * pitch + 4 * j), src + (size_t)t * ld + 4 * j);
+    else dst[t * pitch + j] = __ldcg(src + (size_t)t * ld + j);
+  }
+}
+__device__ __forceinline__ bool scan_aligned(const TaskDesc &d) {
+  return ((d.a[SS_C0] | d.a[SS_C] | d.a[SS_N] | d.a[SS_LDU] | d.a[SS_LDL] | d.a[SS_LDG] | d.a[SS_GOFF]) & 3) == 0 && (d.a[SS_RANK] & 7) == 0 &&
+         ((d.p[0] | d.p[1] | d.p[2] | d.p[3]) & 15) == 0;
+}
+// Requests what the task needs for channels [cb, cb + nc): inputs, B and C, columns [r0, ..) of the low-rank part and of its weights;
+// then the places of the batch's tokens.
+template <int HYB>
+__device__ __noinline__ void scan_load(const Ctx c, const TaskDesc &d, int B, int cb, int nc, int r0) {
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int rank = d.a[SS_RANK], NP = d.a[SS_NP], N = d.a[SS_N], CP = kConsumerThreads / d.a[SS_LANES], pitch = scan_pitch(rank);
+  const int rn = min(pitch - 8, rank - r0), rpad = (rn + 15) & ~15;
+  const bool vec = scan_aligned(d);
+  const ScanMem m = scan_mem(c, d, B);
+  const float *low = reinterpret_cast<const float *>(d.p[1]);
+  if (HYB == HYB_BF16) {
+    const __nv_bfloat16 *w = reinterpret_cast<const __nv_bfloat16 *>(d.p[3]) + (size_t)cb * rank + r0;
+    const int v = vec ? rn >> 3 : rn;
+#pragma unroll 1
+    for (int i = tid; i < nc * v; i += kConsumerThreads) {
+      const int t = i / v, j = i - t * v;
+      if (vec) cp_async16(smem_u32(m.w + t * pitch + 8 * j), w + (size_t)t * rank + 8 * j);
+      else m.w[t * pitch + j] = __ldg(w + (size_t)t * rank + j);
     }
-  };
-  if (B <= 8) {
-    for (int c = warp; c < nc; c += 8) {
-      float acc[8];
+  }
+  scan_copy(m.low, pitch, low + r0, d.a[SS_LDL], B, rn, vec);
+  if (rpad > rn) {   // columns up to a whole 16: zeros on both sides
+    const int z = rpad - rn;
+    for (int i = tid; i < B * z; i += kConsumerThreads) m.low[i / z * pitch + rn + i % z] = 0.f;
+    if (HYB == HYB_BF16)
+      for (int i = tid; i < nc * z; i += kConsumerThreads) m.w[i / z * pitch + rn + i % z] = __float2bfloat16_rn(0.f);
+  }
+  if (r0 == 0) scan_copy(m.us, CP, reinterpret_cast<const float *>(d.p[0]) + cb, d.a[SS_LDU], B, nc, vec);
+  const bool first = r0 == 0 && cb == d.a[SS_C0];
+  if (first) {
+    if (vec) {
+      scan_copy(m.bc, 2 * NP, low + rank, d.a[SS_LDL], B, 2 * NP, true);
+    } else {
+      for (int i = tid; i < B * 2 * NP; i += kConsumerThreads) {
+        const int t = i / (2 * NP), j = i - t * 2 * NP, n = j % NP;
+        m.bc[i] = n < N ? __ldcg(low + (size_t)t * d.a[SS_LDL] + rank + (j < NP ? n : N + n)) : 0.f;
+      }
+    }
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  if (first) {
+    token_map(c.P, B, m.rec, m.qo);
+    if (warp == 0) {
+      const int f0 = lane < B ? m.rec[lane].flags : 0, f1 = 32 + lane < B ? m.rec[32 + lane].flags : 0;
+      const unsigned b0 = __ballot_sync(0xffffffffu, f0 & 1), b1 = __ballot_sync(0xffffffffu, f1 & 1), before = (1u << lane) - 1u;
+      m.seqs[lane] = m.seqs[32 + lane] = -1;
+      __syncwarp();
+      if (f0 & 1) m.seqs[__popc(b0 & before)] = f0 & 4 ? -1 : m.rec[lane].slot;
+      if (f1 & 1) m.seqs[__popc(b0) + __popc(b1 & before)] = f1 & 4 ? -1 : m.rec[32 + lane].slot;
+      if (lane < B) m.tok[lane] = m.rec[lane].slot << 2 | (f0 & 1) << 1 | (f0 & 2) >> 1;
+      if (32 + lane < B) m.tok[32 + lane] = m.rec[32 + lane].slot << 2 | (f1 & 1) << 1 | (f1 & 2) >> 1;
+    }
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  consumer_sync();
+}
+// Three bf16 parts of two neighbouring values; their sum is the float32 value.
+__device__ __forceinline__ void split3(const float2 v, uint32_t (&p)[3]) {
+  p[0] = pack_bf16(v.x, v.y);
+  const float a = v.x - bf16_lo(p[0]), b = v.y - bf16_hi(p[0]);
+  p[1] = pack_bf16(a, b);
+  p[2] = pack_bf16(a - bf16_lo(p[1]), b - bf16_hi(p[1]));
+}
+// Step sizes from the columns at hand (added to what earlier columns gave).  Tensor cores, without losing 32-bit precision: the
+// weights are bf16 as they are, the low-rank part is split into three bf16 numbers.  A unit of a warp is 16 channels x 32 tokens.
+template <int HYB>
+__device__ __noinline__ void scan_steps(const Ctx c, const TaskDesc &d, int B, int cb, int nc, int r0) {
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int rank = d.a[SS_RANK], CP = kConsumerThreads / d.a[SS_LANES], pitch = scan_pitch(rank), rn = min(pitch - 8, rank - r0);
+  const ScanMem m = scan_mem(c, d, B);
+  if (HYB == HYB_BF16) {
+    const int groups = (B + 31) >> 5, units = ((nc + 15) >> 4) * groups;
+#pragma unroll 1
+    for (int u = warp; u < units; u += 8) {
+      const int t0 = u % groups * 32, c0 = u / groups * 16;
+      // (rows past the channels or the batch repeat the last one; what they give is not stored)
+      const uint32_t wa = smem_u32(m.w + min(c0 + (lane & 15), nc - 1) * pitch) + (uint32_t)(lane >> 4) * 16u;
+      uint32_t xa[4];
 #pragma unroll
-      for (int u = 0; u < 8; ++u) acc[u] = 0.f;
-      for (int k = lane * 8; k < rn; k += 256) {
-        float w[8];
-        eight(cb + c, k, w);
+      for (int n = 0; n < 4; ++n) xa[n] = smem_u32(m.low + min(t0 + 8 * n + (lane >> 2), B - 1) * pitch + 2 * (lane & 3));
+      float acc[4][4];
 #pragma unroll
-        for (int u = 0; u < 8; ++u) {
-          if (u >= B) break;
+      for (int n = 0; n < 4; ++n)
 #pragma unroll
-          for (int e = 0; e < 8; ++e) acc[u] = fmaf(w[e], low[u * pitch + k + e], acc[u]);
+        for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
+#pragma unroll 1
+      for (int k = 0; k < rn; k += 16) {
+        uint32_t a[4];
+        ldmatrix_x4(a, wa + 2 * k);
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+          if (t0 + 8 * n >= B) break;
+          uint32_t p0[3], p1[3];
+          split3(lds_f32x2(xa[n] + 4 * k), p0);
+          split3(lds_f32x2(xa[n] + 4 * k + 32), p1);
+#pragma unroll
+          for (int h = 0; h < 3; ++h) mma_bf16_16816(acc[n], a, p0[h], p1[h]);
         }
       }
 #pragma unroll
-      for (int u = 0; u < 8; ++u) {
-        if (u >= B) break;
-        const float v = warp_sum(acc[u]);
-        if (lane == 0) dts[u * CP + c] += v;
-      }
+      for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int t = t0 + 8 * n + 2 * (lane & 3) + (e & 1), ch = c0 + (lane >> 2) + (e >> 1) * 8;
+          if (t < B && ch < nc) m.dts[t * CP + ch] = r0 > 0 ? m.dts[t * CP + ch] + acc[n][e] : acc[n][e];
+        }
     }
-    return;
-  }
-  for (int it = tid; it < nc * ((B + 7) >> 3); it += kConsumerThreads) {
-    const int c = it % nc, t0 = it / nc * 8;
-    float acc[8];
+  } else {
+#pragma unroll 1
+    for (int i = tid; i < nc * ((B + 7) >> 3); i += kConsumerThreads) {   // a channel, eight tokens
+      const int ch = i % nc, t0 = i / nc * 8;
+      const size_t row = (size_t)(cb + ch) * rank + r0;
+      float acc[8];
 #pragma unroll
-    for (int u = 0; u < 8; ++u) acc[u] = 0.f;
-    for (int k = 0; k < rn; k += 8) {
-      float w[8];
-      eight(cb + c, k, w);
+      for (int u = 0; u < 8; ++u) acc[u] = 0.f;
+#pragma unroll 8
+      for (int k = 0; k < rn; ++k) {
+        const float w = bf16_at(d.p[3], row + k);
 #pragma unroll
-      for (int u = 0; u < 8; ++u) {
-        const float4 *x = reinterpret_cast<const float4 *>(low + min(t0 + u, B - 1) * pitch + k);
-        const float4 a = x[0], b = x[1];
-        acc[u] = fmaf(w[3], a.w, fmaf(w[2], a.z, fmaf(w[1], a.y, fmaf(w[0], a.x, acc[u]))));
-        acc[u] = fmaf(w[7], b.w, fmaf(w[6], b.z, fmaf(w[5], b.y, fmaf(w[4], b.x, acc[u]))));
+        for (int u = 0; u < 8; ++u) acc[u] = fmaf(w, m.low[min(t0 + u, B - 1) * pitch + k], acc[u]);
       }
-    }
 #pragma unroll
-    for (int u = 0; u < 8; ++u)
-      if (t0 + u < B) dts[(t0 + u) * CP + c] += acc[u];
+      for (int u = 0; u < 8; ++u)
+        if (t0 + u < B) m.dts[(t0 + u) * CP + ch] = r0 > 0 ? m.dts[(t0 + u) * CP + ch] + acc[u] : acc[u];
+    }
   }
+  consumer_sync();
+  if (r0 + rn < rank) return;
+  // the gate travels while the recurrence is walked
+  if (scan_aligned(d)) scan_copy(m.low, CP, reinterpret_cast<const float *>(d.p[2]) + d.a[SS_GOFF] + cb, d.a[SS_LDG], B, nc, true);
+#pragma unroll 1
+  for (int i = tid; i < B * nc; i += kConsumerThreads) {
+    const int t = i / nc, k = i - t * nc;
+    m.dts[t * CP + k] = softplus_f(m.dts[t * CP + k] + bf16_at(d.p[4], cb + k));
+  }
+  consumer_sync();
+}
+
+// exp(x) for x <= 0, to the last bit near 1 (a decay that is applied once per token must not be off to one side): argument reduced by
+// multiples of ln 2 in two parts (Cody and Waite, "Software Manual for the Elementary Functions"), Taylor series, no branch.
+__device__ __forceinline__ float scan_decay(float x) {
+  x = fmaxf(x, -87.0f);
+  const float n = rintf(x * 1.44269504f);
+  const float r = fmaf(n, 2.12194440e-4f, fmaf(n, -0.693359375f, x));   // |r| <= 0.35
+  float p = fmaf(r, 1.0f / 5040.0f, 1.0f / 720.0f);
+  p = fmaf(p, r, 1.0f / 120.0f);
+  p = fmaf(p, r, 1.0f / 24.0f);
+  p = fmaf(p, r, 1.0f / 6.0f);
+  p = fmaf(p, r, 0.5f);
+  p = fmaf(p * r, r, r);                                                // exp(r) - 1
+  const float s = __int_as_float(((int)n + 127) << 23);
+  return fmaf(s, p, s);
+}
+
+// The recurrence over channels [cb, cb + nc).
+static __device__ __noinline__ void scan_walk(const Ctx c, const TaskDesc &d, int B, int cb, int nc) {
+  const int tid = threadIdx.x, N = d.a[SS_N], NP = d.a[SS_NP], LPC = d.a[SS_LANES], CP = kConsumerThreads / LPC, stride = d.a[SS_C] * NP;
+  const int ch = tid / LPC, n0 = tid % LPC * 4;
+  const bool on = ch < nc && n0 < NP;          // this thread holds states (the others walk along and write nothing)
+  const bool writes = on && n0 == 0;
+  float a[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int e = 0; e < 4; ++e)
+    if (on && n0 + e < N) a[e] = bf16_at(d.p[5], (size_t)(cb + ch) * N + n0 + e);
+  const ScanMem m = scan_mem(c, d, B);
+  float *mine = reinterpret_cast<float *>(wide_arg(d, SS_STATE)) + (on ? (size_t)(cb + ch) * NP + n0 : 0);
+  const uint32_t ring = smem_u32(m.ring + tid), seqs = smem_u32(m.seqs), rows = (uint32_t)(B * CP) * 4u, step = (uint32_t)CP * 4u, bstep = (uint32_t)NP * 8u;
+  uint32_t tok = smem_u32(m.tok), bc = smem_u32(m.bc + min(n0, NP - 4)), cell = smem_u32(m.us + ch);   // (dts lies `rows` bytes behind us)
+  auto fetch = [&](int j) {
+    const int slot = on && j < kMaxLinearTokens ? lds_s32(seqs + 4 * j) : -1;
+    if (slot >= 0) cp_async16(ring + (uint32_t)(j % kScanRing) * (kConsumerThreads * 16), mine + (size_t)slot * stride);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+#pragma unroll 1
+  for (int j = 0; j < kScanRing - 1; ++j) fetch(j);   // (the gate's copies join the first group)
+  const float4 A = make_float4(-expf(a[0]), -expf(a[1]), -expf(a[2]), -expf(a[3]));
+  float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
+  int seq = 0;
+#pragma unroll 1
+  for (int t = 0; t < B; ++t) {
+    const int info = lds_s32(tok);
+    const float dt = lds_f32(cell + rows), du = dt * lds_f32(cell);
+    const float4 b = lds_f32x4(bc), k = lds_f32x4(bc + NP * 4u);
+    if (info & 2) {
+      fetch(seq + kScanRing - 1);
+      asm volatile("cp.async.wait_group %0;" ::"n"(kScanRing - 1) : "memory");
+      S = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (on && lds_s32(seqs + 4 * seq) >= 0) S = lds_f32x4(ring + (uint32_t)(seq % kScanRing) * (kConsumerThreads * 16));
+      ++seq;
+    }
+    S.x = fmaf(scan_decay(dt * A.x), S.x, du * b.x);
+    S.y = fmaf(scan_decay(dt * A.y), S.y, du * b.y);
+    S.z = fmaf(scan_decay(dt * A.z), S.z, du * b.z);
+    S.w = fmaf(scan_decay(dt * A.w), S.w, du * b.w);
+    if ((info & 1) && on) *reinterpret_cast<float4 *>(mine + (size_t)(info >> 2) * stride) = S;
+    float y = on ? fmaf(S.x, k.x, S.y * k.y) + fmaf(S.z, k.z, S.w * k.w) : 0.f;
+    for (int s = LPC >> 1; s > 0; s >>= 1) y += __shfl_xor_sync(0xffffffffu, y, s);
+    if (writes) sts_f32(cell + rows, y);   // (the other lanes of the channel have read dt before the shuffles)
+    cell += step;
+    bc += bstep;
+    tok += 4;
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  consumer_sync();
+}
+
+// (y + D u) * silu(z)
+template <int HYB>
+__device__ __noinline__ void scan_emit(const Ctx c, const TaskDesc &d, int B, int cb, int nc) {
+  typedef typename HybElt<HYB>::T T;
+  const int tid = threadIdx.x, CP = kConsumerThreads / d.a[SS_LANES];
+  const ScanMem m = scan_mem(c, d, B);
+  T *out = reinterpret_cast<T *>(d.p[7]) + cb;
+  if (scan_aligned(d) && (d.a[SS_LDO] & 3) == 0 && ((d.p[6] | d.p[7]) & 15) == 0) {
+    const int v = nc >> 2;
+#pragma unroll 1
+    for (int i = tid; i < B * v; i += kConsumerThreads) {
+      const int t = i / v, j = (i - t * v) * 4;
+      const float4 D = bf16x4_at(d.p[6], cb + j);
+      const float4 y = *reinterpret_cast<const float4 *>(m.dts + t * CP + j), u = *reinterpret_cast<const float4 *>(m.us + t * CP + j);
+      const float4 z = *reinterpret_cast<const float4 *>(m.low + t * CP + j);
+      store_elt4(out + (size_t)t * d.a[SS_LDO] + j, make_float4(fmaf(D.x, u.x, y.x) * silu_exact_f(z.x), fmaf(D.y, u.y, y.y) * silu_exact_f(z.y),
+                                                                fmaf(D.z, u.z, y.z) * silu_exact_f(z.z), fmaf(D.w, u.w, y.w) * silu_exact_f(z.w)));
+    }
+  } else {
+#pragma unroll 1
+    for (int i = tid; i < B * nc; i += kConsumerThreads) {
+      const int t = i / nc, j = i - t * nc;
+      const float z = __ldcg(reinterpret_cast<const float *>(d.p[2]) + (size_t)t * d.a[SS_LDG] + d.a[SS_GOFF] + cb + j);
+      store_elt(out + (size_t)t * d.a[SS_LDO] + j, fmaf(bf16_at(d.p[6], cb + j), m.us[t * CP + j], m.dts[t * CP + j]) * silu_exact_f(z));
+    }
+  }
+  consumer_sync();   // the next channels reuse the arrays and the ring
 }
 
 template <int HYB>
-__device__ __noinline__ void run_selective_scan(const Ctx c, const TaskDesc &d, int task) {
-  typedef typename HybElt<HYB>::T T;
-  const KernelParams &P = c.P;
-  const int B = active_tokens(P);
+__device__ __forceinline__ void run_selective_scan(const Ctx &c, const TaskDesc &d, int task) {
+  const int B = min(active_tokens(c.P), kMaxLinearTokens);
   if (B <= 0) return;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int C = d.a[SS_C], rank = d.a[SS_RANK], N = d.a[SS_N], NP = d.a[SS_NP], LPC = d.a[SS_LANES], CP = kConsumerThreads / LPC;
-  const int mbr = P.max_num_batched_requests, RC = min(kScanRank, (rank + 7) & ~7);
-  // shared memory
-  TokenRec *rec = reinterpret_cast<TokenRec *>(c.s.xtile);
-  int *qo = reinterpret_cast<int *>(c.s.xtile + kTokenMapBytes);
-  int *seqs = qo + ((mbr + 4) & ~3);                                          // [64] state slot of the batch's requests in order, -1: starts from zeros
-  float4 *ring = reinterpret_cast<float4 *>(seqs + kMaxLinearTokens) + tid;   // [kScanRing][256], this thread's cells
-  float *bc = reinterpret_cast<float *>(ring - tid + kScanRing * kConsumerThreads);   // [B][2 NP]: B, C
-  float *low = bc + B * 2 * NP;                                               // [B][RC]
-  float *dts = low + B * RC;                                                  // [B][CP] step sizes
-  float *us = dts + B * CP;                                                   // [B][CP] inputs, then read-outs
-  float *state = reinterpret_cast<float *>(wide_arg(d, SS_STATE));
-  token_map(P, B, rec, qo);
-  if (warp == 0) {
-    const int f0 = lane < B ? rec[lane].flags : 0, f1 = 32 + lane < B ? rec[32 + lane].flags : 0;
-    const unsigned b0 = __ballot_sync(0xffffffffu, f0 & 1), b1 = __ballot_sync(0xffffffffu, f1 & 1), before = (1u << lane) - 1u;
-    seqs[lane] = seqs[32 + lane] = -1;
-    __syncwarp();
-    if (f0 & 1) seqs[__popc(b0 & before)] = f0 & 4 ? -1 : rec[lane].slot;
-    if (f1 & 1) seqs[__popc(b0) + __popc(b1 & before)] = f1 & 4 ? -1 : rec[32 + lane].slot;
-  }
-  for (int i = tid; i < B * 2 * NP; i += kConsumerThreads) {
-    const int t = i / (2 * NP), j = i - t * 2 * NP, n = j % NP;
-    bc[i] = n < N ? __ldcg(reinterpret_cast<const float *>(d.p[1]) + (size_t)t * d.a[SS_LDL] + rank + (j < NP ? n : N + n)) : 0.f;
-  }
-  consumer_sync();
-  stamp(c, task, 0);
-  const int q = tid % LPC, ch = tid / LPC, n0 = 4 * q;
-  for (int cb = d.a[SS_C0]; cb < d.a[SS_C1]; cb += CP) {
-    const int nc = min(CP, d.a[SS_C1] - cb);
-    const bool on = ch < nc && n0 < NP;       // this thread holds states
-    float *mine = state + (size_t)(cb + ch) * NP + n0;
-    auto fetch = [&](int j) {
-      const int slot = j < kMaxLinearTokens ? seqs[j] : -1;
-      if (on && slot >= 0) cp_async16(smem_u32(ring + (j % kScanRing) * kConsumerThreads), mine + (size_t)slot * C * NP);
-      asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-#pragma unroll
-    for (int j = 0; j < kScanRing - 1; ++j) fetch(j);
-    float4 A = make_float4(0.f, 0.f, 0.f, 0.f);
-    float D = 0.f;
-    if (on) {
-      float *a = reinterpret_cast<float *>(&A);
-#pragma unroll
-      for (int e = 0; e < 4; ++e) a[e] = n0 + e < N ? -expf(bf16_at(d.p[5], (size_t)(cb + ch) * N + n0 + e)) : 0.f;
-      D = bf16_at(d.p[6], cb + ch);
+#pragma unroll 1
+  for (int cb = d.a[SS_C0]; cb < d.a[SS_C1]; cb += kConsumerThreads / d.a[SS_LANES]) {
+    const int nc = min(kConsumerThreads / d.a[SS_LANES], d.a[SS_C1] - cb);
+#pragma unroll 1
+    for (int r0 = 0; r0 < d.a[SS_RANK]; r0 += kScanRank) {
+      scan_load<HYB>(c, d, B, cb, nc, r0);
+      stamp(c, task, 0);
+      scan_steps<HYB>(c, d, B, cb, nc, r0);
     }
-    // step sizes and inputs
-    for (int i = tid; i < B * nc; i += kConsumerThreads) {
-      const int t = i / nc, k = i - t * nc;
-      us[t * CP + k] = __ldcg(reinterpret_cast<const float *>(d.p[0]) + (size_t)t * d.a[SS_LDU] + cb + k);
-      dts[t * CP + k] = bf16_at(d.p[4], cb + k);
-    }
-    for (int r0 = 0; r0 < rank; r0 += RC) {
-      const int rn = min(RC, rank - r0);
-      for (int t = warp; t < B; t += 8)
-        for (int k = lane; k < RC; k += 32) low[t * RC + k] = k < rn ? __ldcg(reinterpret_cast<const float *>(d.p[1]) + (size_t)t * d.a[SS_LDL] + r0 + k) : 0.f;
-      consumer_sync();
-      scan_steps(d, low, RC, dts, CP, cb, nc, B, r0, rn);
-      consumer_sync();
-    }
-    for (int i = tid; i < B * nc; i += kConsumerThreads) {
-      const int t = i / nc, k = t * CP + i - t * nc;
-      dts[k] = softplus_f(dts[k]);
-    }
-    consumer_sync();
     stamp(c, task, 1);
-    // the recurrence: lanes of a channel meet in the read-out only
-    float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
-    int seq = 0;
-    for (int t = 0; t < B; ++t) {
-      const int flags = rec[t].flags;
-      if (flags & 1) {
-        fetch(seq + kScanRing - 1);
-        asm volatile("cp.async.wait_group %0;" ::"n"(kScanRing - 1) : "memory");
-        S = on && seqs[seq] >= 0 ? ring[(seq % kScanRing) * kConsumerThreads] : make_float4(0.f, 0.f, 0.f, 0.f);
-        ++seq;
-      }
-      float y = 0.f, u = 0.f;
-      if (on) {
-        const float dt = dts[t * CP + ch];
-        u = us[t * CP + ch];
-        const float4 b = *reinterpret_cast<const float4 *>(bc + t * 2 * NP + n0), k = *reinterpret_cast<const float4 *>(bc + t * 2 * NP + NP + n0);
-        const float du = dt * u;
-        S.x = fmaf(decay_exp(dt * A.x), S.x, du * b.x);
-        S.y = fmaf(decay_exp(dt * A.y), S.y, du * b.y);
-        S.z = fmaf(decay_exp(dt * A.z), S.z, du * b.z);
-        S.w = fmaf(decay_exp(dt * A.w), S.w, du * b.w);
-        y = fmaf(S.x, k.x, fmaf(S.y, k.y, fmaf(S.z, k.z, S.w * k.w)));
-        if (flags & 2) *reinterpret_cast<float4 *>(mine + (size_t)rec[t].slot * C * NP) = S;
-      }
-      for (int s = LPC >> 1; s > 0; s >>= 1) y += __shfl_xor_sync(0xffffffffu, y, s);
-      if (on && q == 0) us[t * CP + ch] = fmaf(D, u, y);   // (the other lanes of the channel read u before the shuffles)
-    }
-    consumer_sync();
+    scan_walk(c, d, B, cb, nc);
     stamp(c, task, 2);
-    for (int i = tid; i < B * nc; i += kConsumerThreads) {
-      const int t = i / nc, k = i - t * nc;
-      const float z = __ldcg(reinterpret_cast<const float *>(d.p[2]) + (size_t)t * d.a[SS_LDG] + d.a[SS_GOFF] + cb + k);
-      store_elt(reinterpret_cast<T *>(d.p[7]) + (size_t)t * d.a[SS_LDO] + cb + k, us[t * CP + k] * silu_exact_f(z));
-    }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    consumer_sync();   // the next channels reuse the arrays and the ring
+    scan_emit<HYB>(c, d, B, cb, nc);
   }
 }
 

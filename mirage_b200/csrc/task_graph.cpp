@@ -1204,8 +1204,9 @@ struct Builder {
       case MPK_OP_SHORT_CONV: return kMaxLinearTokens * 16 + (mbr + 1) * 4;
       case MPK_OP_SELECTIVE_SCAN: {
         const int64_t np = round_up(l.params[1], 4), cp = kConsumerThreads / scan_lanes((int)l.params[1]);
-        return kMaxLinearTokens * 16 + round_up(mbr + 1, 4) * 4 + kMaxLinearTokens * 4 + 4 * nb_max * (2 * cp + 2 * np) +
-               4 * nb_max * std::min<int64_t>(kScanRank, round_up(l.params[0], 8)) + kScanRing * kConsumerThreads * 16;
+        const int rank = (int)l.params[0];
+        return kMaxLinearTokens * (16 + 8) + round_up(mbr + 1, 4) * 4 + scan_ring_bytes(rank, (int)cp) +
+               4 * nb_max * (2 * np + 2 * cp + std::max<int64_t>(scan_pitch(rank), cp));
       }
       case MPK_OP_GROUPED_LINEAR: {
         const int64_t K = T[l.t[1]].dim(2);
@@ -1627,13 +1628,13 @@ struct Builder {
       if (T[l.t[i]].dtype != MPK_BF16 || (int64_t)(T[l.t[i]].bytes / 2) != (int64_t)C * (i == 3 ? rank : i == 5 ? n : 1) ||
           (T[l.t[i]].dims.size() == 2 && T[l.t[i]].strides[1] != 1))
         return fail(MPK_ERR_INVALID, "selective_scan: bf16 dt weight [channels, rank], dt bias, A_log [channels, n] and D");
-    const int nt = std::max(1, std::min(W, C / 8));
+    const int blocks = (C + 7) / 8, nt = std::min(W, blocks);   // eight channels: rows of whole 16-byte pieces
     for (int i = 0; i < nt; ++i) {
       TaskDesc d = blank(TASK_SELECTIVE_SCAN, li);
       for (int k = 0; k < 7; ++k) d.p[k] = (uint64_t)T[l.t[k]].ptr;
       d.p[7] = (uint64_t)o.ptr;
       put_wide(&d, SS_STATE, l.t[7]);
-      d.a[SS_C0] = (int)((int64_t)C * i / nt); d.a[SS_C1] = (int)((int64_t)C * (i + 1) / nt); d.a[SS_C] = C; d.a[SS_RANK] = rank; d.a[SS_N] = n;
+      d.a[SS_C0] = (int)((int64_t)blocks * i / nt) * 8; d.a[SS_C1] = std::min(C, (int)((int64_t)blocks * (i + 1) / nt) * 8); d.a[SS_C] = C; d.a[SS_RANK] = rank; d.a[SS_N] = n;
       d.a[SS_NP] = np; d.a[SS_LANES] = scan_lanes(n); d.a[SS_LDU] = (int)u.ld(); d.a[SS_LDL] = (int)low.ld(); d.a[SS_LDG] = (int)gate.ld();
       d.a[SS_GOFF] = (int)l.params[2]; d.a[SS_LDO] = (int)o.ld();
       put((i + rot) % W, d, ex);
