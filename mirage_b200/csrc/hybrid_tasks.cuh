@@ -2144,12 +2144,13 @@ struct ScanMem {
   int *seqs;            // [64] state slot of the batch's requests in order, -1: starts from zeros
   int *tok;             // [64] state slot << 2 | first token of its request in the batch << 1 | last one
   int *qo;              // [requests + 1]
-  float4 *ring;         // [kScanRing][256] states to come
-  __nv_bfloat16 *w;     // [CP][scan_pitch] weights of the step sizes (in the ring's place, before it is used)
   float *bc;            // [B][2 NP] B, C
   float *us;            // [B][CP] inputs
   float *dts;           // [B][CP] step sizes, then read-outs
-  float *low;           // [B][scan_pitch] columns of the low-rank part; later the gate [B][CP]
+  float *low;           // [B][scan_pitch] columns of the low-rank part
+  __nv_bfloat16 *w;     // [CP][scan_pitch] weights of the step sizes
+  float *gate;          // [B][CP] (in the place of low and w, once the step sizes are there)
+  float4 *ring;         // [kScanRing][256] states to come (likewise)
 };
 __device__ __forceinline__ ScanMem scan_mem(const Ctx &c, const TaskDesc &d, int B) {
   const int NP = d.a[SS_NP], CP = kConsumerThreads / d.a[SS_LANES];
@@ -2158,23 +2159,25 @@ __device__ __forceinline__ ScanMem scan_mem(const Ctx &c, const TaskDesc &d, int
   m.seqs = reinterpret_cast<int *>(c.s.xtile + kTokenMapBytes);
   m.tok = m.seqs + kMaxLinearTokens;
   m.qo = m.tok + kMaxLinearTokens;
-  m.ring = reinterpret_cast<float4 *>(m.qo + ((c.P.max_num_batched_requests + 4) & ~3));
-  m.w = reinterpret_cast<__nv_bfloat16 *>(m.ring);
-  m.bc = reinterpret_cast<float *>(reinterpret_cast<uint8_t *>(m.ring) + scan_ring_bytes(d.a[SS_RANK], CP));
+  m.bc = reinterpret_cast<float *>(m.qo + ((c.P.max_num_batched_requests + 4) & ~3));
   m.us = m.bc + B * 2 * NP;
   m.dts = m.us + B * CP;
-  m.low = m.dts + B * CP;
+  m.low = m.gate = m.dts + B * CP;
+  m.w = reinterpret_cast<__nv_bfloat16 *>(m.low + B * scan_pitch(d.a[SS_RANK]));
+  m.ring = reinterpret_cast<float4 *>(m.gate + B * CP);
   return m;
 }
-// `rows` rows of `cols` floats: 16-byte asynchronous copies where everything is aligned.
-__device__ __forceinline__ void scan_copy(float *dst, int pitch, const float *src, int ld, int rows, int cols, bool vec) {
-  const int v = vec ? cols >> 2 : cols;
+// `rows` rows of `bytes` bytes, 16-byte asynchronous copies: one warp per row, or WIDE (a power of two) neighbouring threads per row.
+template <int WIDE = 32>
+__device__ __forceinline__ void scan_copy(uint32_t dst, int pitch, const void *src, int ld, int rows, int bytes) {
 #pragma unroll 1
-  for (int i = threadIdx.x; i < rows * v; i += kConsumerThreads) {
-    const int t = i / v, j = i - t * v;
-    if (vec) cp_async16(smem_u32(dst + t * pitch + 4 * j), src + (size_t)t * ld + 4 * j);
-    else dst[t * pitch + j] = __ldcg(src + (size_t)t * ld + j);
-  }
+  for (int t = threadIdx.x / WIDE; t < rows; t += kConsumerThreads / WIDE)
+    for (int j = threadIdx.x % WIDE * 16; j < bytes; j += WIDE * 16)
+      cp_async16(dst + t * pitch + j, reinterpret_cast<const uint8_t *>(src) + (size_t)t * ld + j);
+}
+// The same for floats at any alignment.
+__device__ __forceinline__ void scan_copy_plain(float *dst, int pitch, const float *src, int ld, int rows, int cols) {
+  for (int i = threadIdx.x; i < rows * cols; i += kConsumerThreads) dst[i / cols * pitch + i % cols] = __ldcg(src + (size_t)(i / cols) * ld + i % cols);
 }
 __device__ __forceinline__ bool scan_aligned(const TaskDesc &d) {
   return ((d.a[SS_C0] | d.a[SS_C] | d.a[SS_N] | d.a[SS_LDU] | d.a[SS_LDL] | d.a[SS_LDG] | d.a[SS_GOFF]) & 3) == 0 && (d.a[SS_RANK] & 7) == 0 &&
@@ -2190,34 +2193,30 @@ __device__ __noinline__ void scan_load(const Ctx c, const TaskDesc &d, int B, in
   const bool vec = scan_aligned(d);
   const ScanMem m = scan_mem(c, d, B);
   const float *low = reinterpret_cast<const float *>(d.p[1]);
-  if (HYB == HYB_BF16) {
-    const __nv_bfloat16 *w = reinterpret_cast<const __nv_bfloat16 *>(d.p[3]) + (size_t)cb * rank + r0;
-    const int v = vec ? rn >> 3 : rn;
-#pragma unroll 1
-    for (int i = tid; i < nc * v; i += kConsumerThreads) {
-      const int t = i / v, j = i - t * v;
-      if (vec) cp_async16(smem_u32(m.w + t * pitch + 8 * j), w + (size_t)t * rank + 8 * j);
-      else m.w[t * pitch + j] = __ldg(w + (size_t)t * rank + j);
-    }
+  const float *u = reinterpret_cast<const float *>(d.p[0]) + cb;
+  const __nv_bfloat16 *w = reinterpret_cast<const __nv_bfloat16 *>(d.p[3]) + (size_t)cb * rank + r0;
+  const bool first = r0 == 0 && cb == d.a[SS_C0];
+  if (vec) {
+    if (HYB == HYB_BF16) scan_copy(smem_u32(m.w), pitch * 2, w, rank * 2, nc, rn * 2);
+    scan_copy(smem_u32(m.low), pitch * 4, low + r0, d.a[SS_LDL] * 4, B, rn * 4);
+    if (r0 == 0) scan_copy<16>(smem_u32(m.us), CP * 4, u, d.a[SS_LDU] * 4, B, nc * 4);
+    if (first) scan_copy<8>(smem_u32(m.bc), NP * 8, low + rank, d.a[SS_LDL] * 4, B, NP * 8);
+  } else {
+    if (HYB == HYB_BF16)
+      for (int i = tid; i < nc * rn; i += kConsumerThreads) m.w[i / rn * pitch + i % rn] = __ldg(w + (size_t)(i / rn) * rank + i % rn);
+    scan_copy_plain(m.low, pitch, low + r0, d.a[SS_LDL], B, rn);
+    if (r0 == 0) scan_copy_plain(m.us, CP, u, d.a[SS_LDU], B, nc);
+    if (first)
+      for (int i = tid; i < B * 2 * NP; i += kConsumerThreads) {
+        const int t = i / (2 * NP), j = i - t * 2 * NP, n = j % NP;
+        m.bc[i] = n < N ? __ldcg(low + (size_t)t * d.a[SS_LDL] + rank + (j < NP ? n : N + n)) : 0.f;
+      }
   }
-  scan_copy(m.low, pitch, low + r0, d.a[SS_LDL], B, rn, vec);
   if (rpad > rn) {   // columns up to a whole 16: zeros on both sides
     const int z = rpad - rn;
     for (int i = tid; i < B * z; i += kConsumerThreads) m.low[i / z * pitch + rn + i % z] = 0.f;
     if (HYB == HYB_BF16)
       for (int i = tid; i < nc * z; i += kConsumerThreads) m.w[i / z * pitch + rn + i % z] = __float2bfloat16_rn(0.f);
-  }
-  if (r0 == 0) scan_copy(m.us, CP, reinterpret_cast<const float *>(d.p[0]) + cb, d.a[SS_LDU], B, nc, vec);
-  const bool first = r0 == 0 && cb == d.a[SS_C0];
-  if (first) {
-    if (vec) {
-      scan_copy(m.bc, 2 * NP, low + rank, d.a[SS_LDL], B, 2 * NP, true);
-    } else {
-      for (int i = tid; i < B * 2 * NP; i += kConsumerThreads) {
-        const int t = i / (2 * NP), j = i - t * 2 * NP, n = j % NP;
-        m.bc[i] = n < N ? __ldcg(low + (size_t)t * d.a[SS_LDL] + rank + (j < NP ? n : N + n)) : 0.f;
-      }
-    }
   }
   asm volatile("cp.async.commit_group;" ::: "memory");
   if (first) {
@@ -2244,49 +2243,59 @@ __device__ __forceinline__ void split3(const float2 v, uint32_t (&p)[3]) {
   p[2] = pack_bf16(a - bf16_lo(p[1]), b - bf16_hi(p[1]));
 }
 // Step sizes from the columns at hand (added to what earlier columns gave).  Tensor cores, without losing 32-bit precision: the
-// weights are bf16 as they are, the low-rank part is split into three bf16 numbers.  A unit of a warp is 16 channels x 32 tokens.
+// weights are bf16 as they are, the low-rank part is split into three bf16 numbers.  A unit of a warp is 16 MT channels x 8 tokens.
+template <int MT>
+__device__ __forceinline__ void scan_products(const ScanMem &m, int B, int nc, int CP, int pitch, int rn, bool add) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int groups = (B + 7) >> 3, units = (nc + 16 * MT - 1) / (16 * MT) * groups;
+#pragma unroll 1
+  for (int u = warp; u < units; u += 8) {
+    const int t0 = u % groups * 8, c0 = u / groups * 16 * MT;
+    // (rows past the channels or the batch repeat the last one; what they give is not stored)
+    uint32_t wa[MT];
+#pragma unroll
+    for (int i = 0; i < MT; ++i) wa[i] = smem_u32(m.w + min(c0 + 16 * i + (lane & 15), nc - 1) * pitch) + (uint32_t)(lane >> 4) * 16u;
+    const uint32_t xa = smem_u32(m.low + min(t0 + (lane >> 2), B - 1) * pitch + 2 * (lane & 3));
+    float acc[MT][4];
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+#pragma unroll 1
+    for (int k = 0; k < rn; k += 16) {
+      uint32_t a[MT][4], p0[3], p1[3];
+      split3(lds_f32x2(xa + 4 * k), p0);
+      split3(lds_f32x2(xa + 4 * k + 32), p1);
+#pragma unroll
+      for (int i = 0; i < MT; ++i) ldmatrix_x4(a[i], wa[i] + 2 * k);
+#pragma unroll
+      for (int h = 0; h < 3; ++h)
+#pragma unroll
+        for (int i = 0; i < MT; ++i) mma_bf16_16816(acc[i], a[i], p0[h], p1[h]);
+    }
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int t = t0 + 2 * (lane & 3) + (e & 1), ch = c0 + 16 * i + (lane >> 2) + (e >> 1) * 8;
+        if (t < B && ch < nc) m.dts[t * CP + ch] = add ? m.dts[t * CP + ch] + acc[i][e] : acc[i][e];
+      }
+  }
+}
 template <int HYB>
 __device__ __noinline__ void scan_steps(const Ctx c, const TaskDesc &d, int B, int cb, int nc, int r0) {
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x;
   const int rank = d.a[SS_RANK], CP = kConsumerThreads / d.a[SS_LANES], pitch = scan_pitch(rank), rn = min(pitch - 8, rank - r0);
   const ScanMem m = scan_mem(c, d, B);
+  const bool last = r0 + rn >= rank;
+  // a thread keeps its channel in what follows
+  const int ch = tid % CP, tstep = kConsumerThreads / CP;
+  const float bias = last && ch < nc ? bf16_at(d.p[4], cb + ch) : 0.f;
   if (HYB == HYB_BF16) {
-    const int groups = (B + 31) >> 5, units = ((nc + 15) >> 4) * groups;
-#pragma unroll 1
-    for (int u = warp; u < units; u += 8) {
-      const int t0 = u % groups * 32, c0 = u / groups * 16;
-      // (rows past the channels or the batch repeat the last one; what they give is not stored)
-      const uint32_t wa = smem_u32(m.w + min(c0 + (lane & 15), nc - 1) * pitch) + (uint32_t)(lane >> 4) * 16u;
-      uint32_t xa[4];
-#pragma unroll
-      for (int n = 0; n < 4; ++n) xa[n] = smem_u32(m.low + min(t0 + 8 * n + (lane >> 2), B - 1) * pitch + 2 * (lane & 3));
-      float acc[4][4];
-#pragma unroll
-      for (int n = 0; n < 4; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
-#pragma unroll 1
-      for (int k = 0; k < rn; k += 16) {
-        uint32_t a[4];
-        ldmatrix_x4(a, wa + 2 * k);
-#pragma unroll
-        for (int n = 0; n < 4; ++n) {
-          if (t0 + 8 * n >= B) break;
-          uint32_t p0[3], p1[3];
-          split3(lds_f32x2(xa[n] + 4 * k), p0);
-          split3(lds_f32x2(xa[n] + 4 * k + 32), p1);
-#pragma unroll
-          for (int h = 0; h < 3; ++h) mma_bf16_16816(acc[n], a, p0[h], p1[h]);
-        }
-      }
-#pragma unroll
-      for (int n = 0; n < 4; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int t = t0 + 8 * n + 2 * (lane & 3) + (e & 1), ch = c0 + (lane >> 2) + (e >> 1) * 8;
-          if (t < B && ch < nc) m.dts[t * CP + ch] = r0 > 0 ? m.dts[t * CP + ch] + acc[n][e] : acc[n][e];
-        }
-    }
+    // (as many units as warps, if there are channels enough)
+    if (B <= 16) scan_products<1>(m, B, nc, CP, pitch, rn, r0 > 0);
+    else if (B <= 32) scan_products<2>(m, B, nc, CP, pitch, rn, r0 > 0);
+    else scan_products<4>(m, B, nc, CP, pitch, rn, r0 > 0);
   } else {
 #pragma unroll 1
     for (int i = tid; i < nc * ((B + 7) >> 3); i += kConsumerThreads) {   // a channel, eight tokens
@@ -2307,80 +2316,189 @@ __device__ __noinline__ void scan_steps(const Ctx c, const TaskDesc &d, int B, i
     }
   }
   consumer_sync();
-  if (r0 + rn < rank) return;
+  if (!last) return;
   // the gate travels while the recurrence is walked
-  if (scan_aligned(d)) scan_copy(m.low, CP, reinterpret_cast<const float *>(d.p[2]) + d.a[SS_GOFF] + cb, d.a[SS_LDG], B, nc, true);
-#pragma unroll 1
-  for (int i = tid; i < B * nc; i += kConsumerThreads) {
-    const int t = i / nc, k = i - t * nc;
-    m.dts[t * CP + k] = softplus_f(m.dts[t * CP + k] + bf16_at(d.p[4], cb + k));
-  }
+  if (scan_aligned(d)) scan_copy<16>(smem_u32(m.gate), CP * 4, reinterpret_cast<const float *>(d.p[2]) + d.a[SS_GOFF] + cb, d.a[SS_LDG] * 4, B, nc * 4);
+#pragma unroll 2
+  for (int t = ch < nc ? tid / CP : B; t < B; t += tstep) m.dts[t * CP + ch] = softplus_f(m.dts[t * CP + ch] + bias);
   consumer_sync();
 }
 
-// exp(x) for x <= 0, to the last bit near 1 (a decay that is applied once per token must not be off to one side): argument reduced by
-// multiples of ln 2 in two parts (Cody and Waite, "Software Manual for the Elementary Functions"), Taylor series, no branch.
-__device__ __forceinline__ float scan_decay(float x) {
-  x = fmaxf(x, -87.0f);
-  const float n = rintf(x * 1.44269504f);
-  const float r = fmaf(n, 2.12194440e-4f, fmaf(n, -0.693359375f, x));   // |r| <= 0.35
-  float p = fmaf(r, 1.0f / 5040.0f, 1.0f / 720.0f);
-  p = fmaf(p, r, 1.0f / 120.0f);
-  p = fmaf(p, r, 1.0f / 24.0f);
-  p = fmaf(p, r, 1.0f / 6.0f);
-  p = fmaf(p, r, 0.5f);
-  p = fmaf(p * r, r, r);                                                // exp(r) - 1
-  const float s = __int_as_float(((int)n + 127) << 23);
-  return fmaf(s, p, s);
+// Two float32 values in one 64-bit register, and the arithmetic that takes both at once.
+__device__ __forceinline__ uint64_t f2(float x, float y) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+  return r;
+}
+__device__ __forceinline__ float2 f2_parts(uint64_t v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+// exp(x) for x <= 0, to the last bit near 1 (a decay that is applied once per token must not be off to one side): exp(x) = 2^n exp(r)
+// with n = round(x / ln 2) and the Taylor series of exp(r) - 1, without branches and conversions.
+__device__ __forceinline__ uint64_t scan_decay2(uint64_t v) {
+  constexpr float kRound = 12582912.0f;   // 1.5 x 2^23: added, it leaves the nearest integer in the low bits
+  auto both = [](float x) { return f2(x, x); };
+  const float2 u = f2_parts(v);
+  const uint64_t x = f2(fmaxf(u.x, -87.0f), fmaxf(u.y, -87.0f));
+  const uint64_t t = fma2(x, both(1.44269504f), both(kRound));
+  const uint64_t r = fma2(add2(t, both(-kRound)), both(-0.69314718f), x);   // |r| <= 0.35
+  uint64_t p = fma2(r, both(1.0f / 720.0f), both(1.0f / 120.0f));
+  p = fma2(p, r, both(1.0f / 24.0f));
+  p = fma2(p, r, both(1.0f / 6.0f));
+  p = fma2(p, r, both(0.5f));
+  p = fma2(p, mul2(r, r), r);                                               // exp(r) - 1
+  const float2 n = f2_parts(t);
+  const uint64_t s = f2(__int_as_float((__float_as_int(n.x) << 23) + 0x3f800000), __int_as_float((__float_as_int(n.y) << 23) + 0x3f800000));
+  return fma2(s, p, s);
+}
+struct ScanState { uint64_t a, b; };   // four states of a thread
+__device__ __forceinline__ ScanState scan_state(const float4 v) { return ScanState{f2(v.x, v.y), f2(v.z, v.w)}; }
+__device__ __forceinline__ ScanState lds_state(uint32_t a) {
+  ScanState v;
+  asm volatile("ld.shared.v2.b64 {%0, %1}, [%2];" : "=l"(v.a), "=l"(v.b) : "r"(a) : "memory");
+  return v;
+}
+__device__ __forceinline__ void scan_update(ScanState &S, const ScanState &e, const ScanState &x) {
+  S.a = fma2(e.a, S.a, x.a);
+  S.b = fma2(e.b, S.b, x.b);
+}
+__device__ __forceinline__ float scan_read(const ScanState &S, const ScanState &k) {
+  const float2 y = f2_parts(fma2(S.a, k.a, mul2(S.b, k.b)));
+  return y.x + y.y;
 }
 
-// The recurrence over channels [cb, cb + nc).
+// The recurrence over channels [cb, cb + nc).  Four tokens at a time where none of them begins or ends a request, or where all of them
+// are single tokens of requests of their own; else one by one.
 static __device__ __noinline__ void scan_walk(const Ctx c, const TaskDesc &d, int B, int cb, int nc) {
   const int tid = threadIdx.x, N = d.a[SS_N], NP = d.a[SS_NP], LPC = d.a[SS_LANES], CP = kConsumerThreads / LPC, stride = d.a[SS_C] * NP;
-  const int ch = tid / LPC, n0 = tid % LPC * 4;
+  const int ch = tid / LPC, n0 = tid % LPC * 4, q = tid & 3;
   const bool on = ch < nc && n0 < NP;          // this thread holds states (the others walk along and write nothing)
-  const bool writes = on && n0 == 0;
   float a[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
   for (int e = 0; e < 4; ++e)
     if (on && n0 + e < N) a[e] = bf16_at(d.p[5], (size_t)(cb + ch) * N + n0 + e);
   const ScanMem m = scan_mem(c, d, B);
   float *mine = reinterpret_cast<float *>(wide_arg(d, SS_STATE)) + (on ? (size_t)(cb + ch) * NP + n0 : 0);
-  const uint32_t ring = smem_u32(m.ring + tid), seqs = smem_u32(m.seqs), rows = (uint32_t)(B * CP) * 4u, step = (uint32_t)CP * 4u, bstep = (uint32_t)NP * 8u;
+  const uint32_t ring = smem_u32(m.ring + tid), rows = (uint32_t)(B * CP) * 4u, step = (uint32_t)CP * 4u, bstep = (uint32_t)NP * 8u;
+  constexpr uint32_t kSlot = kConsumerThreads * 16;
   uint32_t tok = smem_u32(m.tok), bc = smem_u32(m.bc + min(n0, NP - 4)), cell = smem_u32(m.us + ch);   // (dts lies `rows` bytes behind us)
-  auto fetch = [&](int j) {
-    const int slot = on && j < kMaxLinearTokens ? lds_s32(seqs + 4 * j) : -1;
-    if (slot >= 0) cp_async16(ring + (uint32_t)(j % kScanRing) * (kConsumerThreads * 16), mine + (size_t)slot * stride);
+  uint32_t put = ring, get = ring, next = smem_u32(m.seqs), seq = next;   // ring cells and requests to fetch and to use next
+  const uint32_t end = next + 4 * kMaxLinearTokens;
+  auto turn = [&](uint32_t at) { return at + kSlot == ring + kScanRing * kSlot ? ring : at + kSlot; };
+  auto slot_of = [&](uint32_t at) { return on && at < end ? lds_s32(min(at, end - 4)) : -1; };   // of a request, -1: nothing to fetch
+  auto fetch = [&](int slot) {
+    asm volatile("{\n.reg .pred p;\nsetp.ge.s32 p, %2, 0;\n@p cp.async.cg.shared.global [%0], [%1], 16;\n}" ::"r"(put), "l"(mine + (size_t)max(slot, 0) * stride), "r"(slot)
+                 : "memory");
     asm volatile("cp.async.commit_group;" ::: "memory");
+    next += 4;
+    put = turn(put);
+  };
+  auto entering = [&](int slot) {   // the state a request brings
+    const ScanState s = lds_state(get);
+    get = turn(get);
+    return ScanState{slot >= 0 ? s.a : 0ull, slot >= 0 ? s.b : 0ull};
+  };
+  auto leaving = [&](const ScanState &S, int slot) {
+    const float2 lo = f2_parts(S.a), hi = f2_parts(S.b);
+    *reinterpret_cast<float4 *>(mine + (size_t)slot * stride) = make_float4(lo.x, lo.y, hi.x, hi.y);
   };
 #pragma unroll 1
-  for (int j = 0; j < kScanRing - 1; ++j) fetch(j);   // (the gate's copies join the first group)
-  const float4 A = make_float4(-expf(a[0]), -expf(a[1]), -expf(a[2]), -expf(a[3]));
-  float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
-  int seq = 0;
+  for (int j = 0; j < kScanRing - 1; ++j) fetch(slot_of(next));   // (the gate's copies join the first group)
+  const ScanState A = scan_state(make_float4(-expf(a[0]), -expf(a[1]), -expf(a[2]), -expf(a[3])));
+  ScanState S{0ull, 0ull};
 #pragma unroll 1
-  for (int t = 0; t < B; ++t) {
-    const int info = lds_s32(tok);
-    const float dt = lds_f32(cell + rows), du = dt * lds_f32(cell);
-    const float4 b = lds_f32x4(bc), k = lds_f32x4(bc + NP * 4u);
-    if (info & 2) {
-      fetch(seq + kScanRing - 1);
-      asm volatile("cp.async.wait_group %0;" ::"n"(kScanRing - 1) : "memory");
-      S = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (on && lds_s32(seqs + 4 * seq) >= 0) S = lds_f32x4(ring + (uint32_t)(seq % kScanRing) * (kConsumerThreads * 16));
-      ++seq;
+  for (int t = 0; t < B;) {
+    const int4 info = lds_v4(tok & ~15u);
+    const bool four = (t & 3) == 0 && t + 4 <= B, plain = four && ((info.x | info.y | info.z | info.w) & 3) == 0;
+    if (plain || (four && (info.x & info.y & info.z & info.w & 3) == 3)) {
+      ScanState e[4], x[4], k[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float dt = lds_f32(cell + rows + i * step), du = dt * lds_f32(cell + i * step);
+        const ScanState b = lds_state(bc + i * bstep);
+        k[i] = lds_state(bc + i * bstep + NP * 4u);
+        e[i].a = scan_decay2(mul2(f2(dt, dt), A.a));
+        e[i].b = scan_decay2(mul2(f2(dt, dt), A.b));
+        x[i].a = mul2(f2(du, du), b.a);
+        x[i].b = mul2(f2(du, du), b.b);
+      }
+      float y[4];
+      if (plain) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          scan_update(S, e[i], x[i]);
+          y[i] = scan_read(S, k[i]);
+        }
+      } else {
+        const int slot[4] = {info.x >> 2, info.y >> 2, info.z >> 2, info.w >> 2};
+        int from[4], then[4];
+        ScanState s[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          from[i] = slot_of(seq + 4 * i);
+          then[i] = slot_of(next + 4 * i);
+        }
+        seq += 16;
+        asm volatile("cp.async.wait_group %0;" ::"n"(kScanRing - 5) : "memory");   // the four oldest of kScanRing - 1
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s[i] = entering(from[i]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) scan_update(s[i], e[i], x[i]);
+        if (on)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) leaving(s[i], slot[i]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          y[i] = scan_read(s[i], k[i]);
+          fetch(then[i]);
+        }
+      }
+      // sums over the lanes of a channel; lane q of the last four ends up with token q's
+#pragma unroll
+      for (int i = 0; i < 4; ++i) y[i] = on ? y[i] : 0.f;
+      for (int s = LPC >> 1; s > 2; s >>= 1)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) y[i] += __shfl_xor_sync(0xffffffffu, y[i], s);
+      float y0 = q & 2 ? y[2] : y[0], y1 = q & 2 ? y[3] : y[1];
+      y0 += __shfl_xor_sync(0xffffffffu, q & 2 ? y[0] : y[2], 2);
+      y1 += __shfl_xor_sync(0xffffffffu, q & 2 ? y[1] : y[3], 2);
+      const float sum = (q & 1 ? y1 : y0) + __shfl_xor_sync(0xffffffffu, q & 1 ? y0 : y1, 1);
+      if (ch < nc && n0 < 16) sts_f32(cell + rows + q * step, sum);   // (the step sizes there have been read before the shuffles)
+      t += 4; cell += 4 * step; bc += 4 * bstep; tok += 16;
+      continue;
     }
-    S.x = fmaf(scan_decay(dt * A.x), S.x, du * b.x);
-    S.y = fmaf(scan_decay(dt * A.y), S.y, du * b.y);
-    S.z = fmaf(scan_decay(dt * A.z), S.z, du * b.z);
-    S.w = fmaf(scan_decay(dt * A.w), S.w, du * b.w);
-    if ((info & 1) && on) *reinterpret_cast<float4 *>(mine + (size_t)(info >> 2) * stride) = S;
-    float y = on ? fmaf(S.x, k.x, S.y * k.y) + fmaf(S.z, k.z, S.w * k.w) : 0.f;
+    const int here = lds_s32(tok);
+    const float dt = lds_f32(cell + rows), du = dt * lds_f32(cell);
+    const ScanState b = lds_state(bc), k = lds_state(bc + NP * 4u);
+    if (here & 2) {
+      fetch(slot_of(next));
+      asm volatile("cp.async.wait_group %0;" ::"n"(kScanRing - 1) : "memory");
+      S = entering(slot_of(seq));
+      seq += 4;
+    }
+    scan_update(S, ScanState{scan_decay2(mul2(f2(dt, dt), A.a)), scan_decay2(mul2(f2(dt, dt), A.b))}, ScanState{mul2(f2(du, du), b.a), mul2(f2(du, du), b.b)});
+    if ((here & 1) && on) leaving(S, here >> 2);
+    float y = on ? scan_read(S, k) : 0.f;
     for (int s = LPC >> 1; s > 0; s >>= 1) y += __shfl_xor_sync(0xffffffffu, y, s);
-    if (writes) sts_f32(cell + rows, y);   // (the other lanes of the channel have read dt before the shuffles)
-    cell += step;
-    bc += bstep;
-    tok += 4;
+    if (ch < nc && n0 == 0) sts_f32(cell + rows, y);
+    ++t; cell += step; bc += bstep; tok += 4;
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   consumer_sync();
@@ -2394,13 +2512,12 @@ __device__ __noinline__ void scan_emit(const Ctx c, const TaskDesc &d, int B, in
   const ScanMem m = scan_mem(c, d, B);
   T *out = reinterpret_cast<T *>(d.p[7]) + cb;
   if (scan_aligned(d) && (d.a[SS_LDO] & 3) == 0 && ((d.p[6] | d.p[7]) & 15) == 0) {
-    const int v = nc >> 2;
-#pragma unroll 1
-    for (int i = tid; i < B * v; i += kConsumerThreads) {
-      const int t = i / v, j = (i - t * v) * 4;
-      const float4 D = bf16x4_at(d.p[6], cb + j);
+    const int j = tid % (CP >> 2) * 4;   // a thread keeps its channels
+    const float4 D = j < nc ? bf16x4_at(d.p[6], cb + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 2
+    for (int t = j < nc ? tid / (CP >> 2) : B; t < B; t += kConsumerThreads * 4 / CP) {
       const float4 y = *reinterpret_cast<const float4 *>(m.dts + t * CP + j), u = *reinterpret_cast<const float4 *>(m.us + t * CP + j);
-      const float4 z = *reinterpret_cast<const float4 *>(m.low + t * CP + j);
+      const float4 z = *reinterpret_cast<const float4 *>(m.gate + t * CP + j);
       store_elt4(out + (size_t)t * d.a[SS_LDO] + j, make_float4(fmaf(D.x, u.x, y.x) * silu_exact_f(z.x), fmaf(D.y, u.y, y.y) * silu_exact_f(z.y),
                                                                 fmaf(D.z, u.z, y.z) * silu_exact_f(z.z), fmaf(D.w, u.w, y.w) * silu_exact_f(z.w)));
     }

@@ -97,11 +97,12 @@ MPK_HD constexpr int scan_lanes(int n) {
   while (4 * l < n) l *= 2;
   return l;
 }
-constexpr int kScanRing = 6, kScanRank = 256;
+constexpr int kScanRing = 12, kScanRank = 256;
 MPK_HD constexpr int scan_pitch(int rank) { return (rank < kScanRank ? (rank + 15) / 16 * 16 : kScanRank) + 8; }   // of staged rows, elements
-MPK_HD constexpr int scan_ring_bytes(int rank, int channels) {   // the weights are staged where the ring will be
-  const int w = channels * scan_pitch(rank) * 2, r = kScanRing * kConsumerThreads * 16;
-  return ((w > r ? w : r) + 15) & ~15;
+// The low-rank part and its weights are staged where the gate and the ring will be.
+MPK_HD constexpr int scan_staged_bytes(int tokens, int rank, int channels) {
+  const int a = tokens * scan_pitch(rank) * 4 + channels * scan_pitch(rank) * 2, b = tokens * channels * 4, ring = kScanRing * kConsumerThreads * 16;
+  return a > b + ring ? a : b + ring;
 }
 
 enum : int { HYB_NONE = 0, HYB_BF16 = 1, HYB_F32 = 2 };

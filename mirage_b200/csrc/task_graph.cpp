@@ -1204,9 +1204,8 @@ struct Builder {
       case MPK_OP_SHORT_CONV: return kMaxLinearTokens * 16 + (mbr + 1) * 4;
       case MPK_OP_SELECTIVE_SCAN: {
         const int64_t np = round_up(l.params[1], 4), cp = kConsumerThreads / scan_lanes((int)l.params[1]);
-        const int rank = (int)l.params[0];
-        return kMaxLinearTokens * (16 + 8) + round_up(mbr + 1, 4) * 4 + scan_ring_bytes(rank, (int)cp) +
-               4 * nb_max * (2 * np + 2 * cp + std::max<int64_t>(scan_pitch(rank), cp));
+        return kMaxLinearTokens * (16 + 8) + round_up(mbr + 1, 4) * 4 + 4 * nb_max * (2 * np + 2 * cp) +
+               scan_staged_bytes(nb_max, (int)l.params[0], (int)cp);
       }
       case MPK_OP_GROUPED_LINEAR: {
         const int64_t K = T[l.t[1]].dim(2);
