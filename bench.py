@@ -874,9 +874,9 @@ def bebuzen_case(size, dev):
     dense = {"kind": "dense", "ff": y["ff"]}
     scan = {"type": "mamba1", "mixer": {"inner": y["inner"], "state": y["state"], "dt_rank": y["rank"], "conv": 4}}
     sink = {"type": "attention_2", "mixer": {"heads": y["heads"], "kv_heads": y["kv"], "dim": y["dim"], "vdim": y["dim"], "scale": y["dim"] ** -0.5,
-                                             "mask": {"size": 1024, "keep_first": 4}, "rot": {"base": 1e4, "dims": y["dim"]}}}
-    diff = {"heads": y["dheads"], "kv_heads": y["kv"], "dim": y["dim"] // 2, "vdim": y["dim"], "scale": (y["dim"] // 2) ** -0.5, "conv": 4, "diff": 0.5,
-            "mask": {"size": 1024}, "rot": {"base": 5e5, "dims": y["dim"] // 2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+                                             "mask": {"size": 1024, "keep_first": 4}, "rot": {"base": 2e4, "dims": y["dim"]}}}
+    diff = {"heads": y["dheads"], "kv_heads": y["kv"], "dim": y["dim"] // 2, "vdim": y["dim"], "scale": (y["dim"] // 2) ** -0.5, "conv": 4, "diff": 0.6,
+            "mask": {"size": 1024}, "rot": {"base": 1e6, "dims": y["dim"] // 2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
     mixers = [scan, sink, scan, {"type": "attention", "mixer": diff}, scan, {"type": "attention", "mixer": dict(diff, kv_from=3)}, scan, sink]
     c = {"architecture": "Bebuzen", "vocab": HYBRID_VOCAB, "width": D, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
          "layers": [dict(m, mlp=moe if n % 2 else dense) for n, m in enumerate(mixers)]}
