@@ -278,3 +278,58 @@ def softmax_choice(logits: Tensor, top: int) -> Tuple[list, Tensor]:
     p = torch.softmax(logits, -1)
     chosen = sorted(range(p.shape[0]), key=lambda e: -float(p[e]))[:top]
     return chosen, p[torch.tensor(chosen)]
+
+
+def bigram_rows(tokens: Sequence[int], buckets: int, mul_prev: int, mul_cur: int) -> list:
+    """Row of the bigram table for every token of a sequence; the first token has the row behind the buckets."""
+    return [buckets] + [(a * mul_prev + b * mul_cur) % buckets for a, b in zip(tokens, tokens[1:])]
+
+
+def sinusoids(tokens: int, width: int, dtype: torch.dtype) -> Tensor:
+    """[tokens, width]: sine and cosine, in turn, of position * 10000^(-2 i / width)."""
+    out = torch.zeros(tokens, width, dtype=dtype)
+    for p in range(tokens):
+        for j in range(width):
+            a = p * 10000.0 ** (-2.0 * (j // 2) / width)
+            out[p, j] = math.cos(a) if j % 2 else math.sin(a)
+    return out
+
+
+def depth_average(history: Sequence[Tensor], weights: Tensor) -> Tensor:
+    """Weighted sum of the embedding output and all layers' results so far."""
+    assert len(history) == weights.shape[0]
+    out = torch.zeros_like(history[0])
+    for x, w in zip(history, weights):
+        out = out + w * x
+    return out
+
+
+def query_temperature(position: int, coef: float, every: int) -> float:
+    return 1.0 + coef * math.log((position + 1) // every + 1)
+
+
+def biased_attention(q: Tensor, k: Tensor, v: Tensor, scale: float, window: int, r1: Tensor, r2: Tensor) -> Tensor:
+    """Grouped heads over the visible keys; a key d positions back has r1[h] * ln(1 + r2[h] * d) taken off its score."""
+    T, H = q.shape[:2]
+    G = k.shape[1]
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for t in range(T):
+        at = torch.tensor(visible(t, window))
+        for h in range(H):
+            g = h // (H // G)
+            s = (k[at, g] @ q[t, h]) * scale - r1[h] * torch.log(1 + r2[h] * (t - at).to(q.dtype))
+            out[t, h] = torch.softmax(s, 0) @ v[at, g]
+    return out
+
+
+def latent_window_attention(q: Tensor, c: Tensor, w_uk: Tensor, w_uv: Tensor, scale: float, window: int) -> Tensor:
+    """q [tokens, H, d], latents c [tokens, rank]: keys and values expanded per head -> [tokens, H, dv]."""
+    T, H, d = q.shape
+    k = (c @ w_uk.T).view(T, H, d)
+    v = (c @ w_uv.T).view(T, H, -1)
+    return window_attention(q, k, v, scale, window)
+
+
+def poly_norm(z: Tensor, coef: Tensor, eps: float) -> Tensor:
+    """Weighted sum of the first three powers of z, each divided by its root mean square, and a constant (four numbers)."""
+    return coef[0] * rms_unit(z, eps) + coef[1] * rms_unit(z ** 2, eps) + coef[2] * rms_unit(z ** 3, eps) + coef[3]
