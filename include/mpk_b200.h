@@ -57,10 +57,15 @@ typedef enum { MPK_IO_CUDA = 0, MPK_IO_SYMMETRIC = 1 } mpk_io_category;
 /* Layer operators: one per PersistentKernel.*_layer method on the decode path
  * (python/mirage/mpk/persistent_kernel.py, line of each method in the comment). */
 typedef enum {
-  MPK_OP_EMBED = 1,             /* embed_layer              :586  in: ids, table        out: y            params: [input_source, factor (hybrid graphs)] */
+  MPK_OP_EMBED = 1,             /* embed_layer              :586  in: ids, table        out: y            params: [input_source, factor (hybrid graphs)]
+                                   hybrid graphs, optional tensors 3-5: bigram table bf16 [buckets + 1, width], position frequencies int64 [(width + 1) / 2], copy of y
+                                   (f32 [.., tokens, width], its first rows), then params [.., mul_prev, mul_cur] and 64-bit arithmetic: y = factor * table[id] +
+                                   bigram[(previous id * mul_prev + id * mul_cur) mod buckets] (a sequence's first token: the last row) + [sin, cos, sin, ..] of
+                                   position * frequency (turns in units of 2^-64).  The previous id is read from the token table (config `tokens`) */
   MPK_OP_RMSNORM = 2,           /* rmsnorm_layer            :609  in: x, gamma          out: y                                            */
   MPK_OP_RMSNORM_LINEAR = 3,    /* rmsnorm_linear_layer     :627  in: x, gamma, W       out: y                                            */
   MPK_OP_LINEAR = 4,            /* linear_layer             :1731 in: x, W              out: y            params: optional [activation, soft cap] (hybrid graphs, mpk_activation)
+                                   (scale: the second parameter is the factor of a float32 y)
                                    hybrid graphs, optional fourth tensor: bf16 bias [rows of W], float32 y */
   MPK_OP_LINEAR_RESIDUAL = 5,   /* linear_with_residual_layer :1762 in: x, W, residual  out: y            params: [enable_residual]       */
   MPK_OP_SPLITK_LINEAR = 6,     /* splitk_linear_layer      :1706 in: x, W              out: y (y += x W^T)                               */
@@ -114,17 +119,22 @@ typedef enum {
                                    11 f32 [tokens, columns]: y is multiplied by sigmoid of column params[3]
                                    params: [eps, weights stored around zero, 0 RMS norm | 1 layer norm, gate column, factor of y's norm]
                                    with a weight of y's norm: x += factor * norm(y + weighted sum of the experts) * weight
-                                   an output without a norm weight is the new stream as it is */
+                                   an output without a norm weight is the new stream as it is
+                                   optional params[5]: columns of x that are normed (0: all; the leading ones, with nothing added)
+                                   tensors 12, 13: results f32 [results, tokens, width], weights bf16 [n]: x + y becomes result n - 1, the new stream is the
+                                   weighted sum of results 0 .. n - 1 */
   MPK_OP_QKV_APPEND = 33,       /* norm and rotate q and k, append k / v rows   in: projections, cos, sin  out: q, k_cache, v_cache
                                    tensors: proj, q, k_cache, v_cache (caches absent: queries only), cos, sin, q norm, k norm (optional, bf16 [dim])
                                    params: [hq, hkv, dim, vdim, q_col, k_col, v_col, rotated dims, unit norm (after the rotation), eps,
                                    optional: 1 pairs are neighbours (0: halves), maps]
                                    q / k norm: an RMS norm in front of the rotation.  maps = 2: q and k have two vectors per head; a cache row
-                                   holds both, a query row (two per head) has its own and zeros for the other */
+                                   holds both, a query row (two per head) has its own and zeros for the other
+                                   optional params[12..14]: 1 the norms span all heads (weights [heads x dim], nothing rotated), temperature coefficient c, step s:
+                                   queries times 1 + c ln(floor((position + 1) / s) + 1) (s = 0: none) */
   MPK_OP_EXT_ATTENTION = 34,    /* tensors: q, k_cache, v_cache (= k_cache: the leading vdim columns of a key are its value), out, sinks (optional)
                                    params: [hq, hkv, vdim, out_col, scale, soft cap (0: none), sink, out_scale, optional 1: an MPK_OP_ATTN_MERGE layer follows,
                                    optional window, kept]: with a window a position sees itself, the window - 1 before it and the first `kept`
-                                   out: the activation type, or float32
+                                   out: the activation type, or float32; tensors 5, 6: distance bias, bf16 [hq] each: score - r1 ln(1 + r2 distance)
                                    sink: exp(sinks[head]) joins the softmax denominator (bf16 [hq]; without the tensor: 1) */
   MPK_OP_SHORT_CONV = 35,       /* causal per-channel convolution   tensors: in, in_bias, taps, bias, state, out, copy of out in the activation type
                                    (biases and copy optional)
@@ -140,7 +150,8 @@ typedef enum {
                                    params: [heads, latent size, rotated dims, q_col, kv_col, eps] */
   MPK_OP_GROUPED_LINEAR = 40    /* one linear per group of columns   in: x [tokens, groups * x stride], W [groups, N, K]  out: y
                                    params: [x stride, y column, y stride]: group g reads x[:, g * x stride + (0 .. K)] and writes
-                                   y[:, y column + g * y stride + (0 .. N)] */,
+                                   y[:, y column + g * y stride + (0 .. N)];  optional fourth tensor f32 with params [.., gate column, gate stride]:
+                                   the result is multiplied by the sigmoid of the gate's columns gate column + g * gate stride + (0 .. N) */,
   MPK_OP_ATTN_MERGE = 41        /* directly behind an MPK_OP_EXT_ATTENTION layer with its ninth parameter set: the same tensors and parameters;
                                    merges the key chunks on all workers (for wide values) */,
   MPK_OP_SELECTIVE_SCAN = 42,   /* selective state space recurrence   tensors: u f32, low f32 [tokens, rank + 2 n], gate f32, dt weight [channels, rank],
@@ -148,13 +159,15 @@ typedef enum {
                                    params: [rank, n, gate column]
                                    dt = softplus(dt weight . low[:, :rank] + dt bias), S = exp(-dt exp(A_log)) S + dt u B, out = (S C + D u) * silu(gate),
                                    B and C the next 2 n columns of low */
-  MPK_OP_DIFF_COMBINE = 43      /* differential attention   in: maps f32 [tokens, heads * 2 * vdim]  out: y [tokens, >= heads * vdim]
+  MPK_OP_DIFF_COMBINE = 43,     /* differential attention   in: maps f32 [tokens, heads * 2 * vdim]  out: y [tokens, >= heads * vdim]
                                    params: [heads, vdim, lambda, factor, eps]: y = factor * unit norm(map 1 - lambda map 2) per head */
+  MPK_OP_POLY_NORM = 44         /* activation   tensors: z f32 [tokens, n], coefficients bf16 [4] (a, b, c, e), y [tokens, >= n] of the activation type   params: [eps]
+                                   y = a N(z) + b N(z^2) + c N(z^3) + e, N dividing a token's values by their root mean square */
 } mpk_op;
 
 /* Activations of linear layers in hybrid graphs.  The gated ones take weight rows interleaved as two gate rows, two up rows, and
  * write act(gate) * up: half as many columns as the weight has rows. */
-typedef enum { MPK_ACT_NONE = 0, MPK_ACT_RELU2 = 1, MPK_ACT_SOFTCAP = 2, MPK_ACT_GATED_SILU = 3, MPK_ACT_GATED_GELU_TANH = 4 } mpk_activation;
+typedef enum { MPK_ACT_NONE = 0, MPK_ACT_RELU2 = 1, MPK_ACT_SOFTCAP = 2, MPK_ACT_GATED_SILU = 3, MPK_ACT_GATED_GELU_TANH = 4, MPK_ACT_SCALE = 5 } mpk_activation;
 
 /* Value columns a task of an MPK_OP_MLSTM layer walks at a time; the layer's `chunks` parameter (and the second state
  * tensor [slots, heads, chunks, dim + 1]) may be at most ceil(vdim / this).  */

@@ -31,7 +31,7 @@ OP_ARGMAX_EXCHANGE = 30
 OP_MOE_TOPK_SOFTMAX = 31
 OP_RESIDUAL_NORM, OP_QKV_APPEND, OP_EXT_ATTENTION, OP_SHORT_CONV, OP_RGLRU, OP_MLSTM = 32, 33, 34, 35, 36, 37
 OP_GLA, OP_LATENT_APPEND, OP_GROUPED_LINEAR, OP_ATTN_MERGE = 38, 39, 40, 41
-OP_SELECTIVE_SCAN, OP_DIFF_COMBINE = 42, 43
+OP_SELECTIVE_SCAN, OP_DIFF_COMBINE, OP_POLY_NORM = 42, 43, 44
 IO_CUDA, IO_SYMMETRIC = 0, 1
 MODE_OFFLINE, MODE_ONLINE_NOTOKEN, MODE_ONLINE = 0, 1, 2
 # control words of online mode (request_ctl)

@@ -1,4 +1,4 @@
-"""What the builders of hybrid graphs share: buffers and weights padded for the tensor path, rotary tables, the head.
+"""What the builders of hybrid graphs share: buffers and weights padded for the tensor path, rotary tables, the mLSTM mixer, the head.
 
 Linear weights of a bf16 graph are padded to a multiple of 64 input columns (the tensor path's k granularity), the activation
 buffers in front of them likewise: what the padding columns hold is finite and meets zero weights.
@@ -49,6 +49,25 @@ def rotary_tables(base: float, dims: int, positions: int, device, scaling: Optio
         f = scaling.apply(f)
     a = torch.arange(positions, dtype=torch.float64)[:, None] * f
     return a.cos().float().to(device), a.sin().float().to(device)
+
+
+@dataclass(frozen=True)
+class MlstmSpec:
+    """Sizes of a matrix-memory mixer."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    @classmethod
+    def from_dict(cls, m: Dict[str, Any]) -> "MlstmSpec":
+        return cls(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"]))
+
+    def state(self, slots: int, num_workers: int, device) -> Dict[str, torch.Tensor]:
+        """float32, indexed by state slot: the memory, and normaliser and running maximum of every task of a head."""
+        chunks = PersistentKernel.mlstm_chunks(num_workers, slots, self.heads, self.dim, self.vdim)
+        z = lambda *s: torch.zeros(*s, dtype=torch.float32, device=device)
+        return {"memory": z(slots, self.heads, self.dim, round_up(self.vdim, 4)), "normaliser": z(slots, self.heads, chunks, self.dim + 1)}
 
 
 @dataclass
@@ -115,6 +134,19 @@ class HybridBuilder:
         y = self._buf("sublayer", self.width, float32)
         self._linear(x, self._weight(name + ".padded", parts), y, bias=bias)
         return y
+
+    def _mlstm(self, p: str, m: MlstmSpec, st: Dict[str, torch.Tensor], h: DTensor) -> DTensor:
+        """[q | k | v | gate | i | f] in one linear -> recurrence with its head norm and gate -> output linear."""
+        mpk, sd = self.mpk, self.sd
+        qk, v = m.heads * m.dim, m.heads * m.vdim
+        proj = self._buf("proj", 2 * qk + 2 * v + 2 * m.heads, float32)
+        self._linear(h, self._weight(p + "qkvgif", [sd[p + n] for n in ("q", "k", "v", "g", "i", "f")]), proj)
+        out = self._buf("mixed", self._kpad(v), self.act)
+        mpk.mlstm_layer(proj, self._att(p + "i.b"), self._att(p + "f.b"), self._att(p + "norm"), mpk.attach_input(st["memory"], name=p + "memory"),
+                        mpk.attach_input(st["normaliser"], name=p + "normaliser"), self._buf("readout", v, float32), out,
+                        heads=m.heads, dim=m.dim, vdim=m.vdim, q_col=0, k_col=qk, v_col=2 * qk, gate_col=2 * qk + v,
+                        i_col=2 * qk + 2 * v, f_col=2 * qk + 2 * v + m.heads, gate_cap=m.gate_cap, eps=self.eps, q_scale=m.dim ** -0.5)
+        return self._sublayer(out, p + "o", [sd[p + "o"]])
 
     def _gated(self, x: DTensor, p: str, ff: int, activation: str) -> DTensor:
         """down(act(gate x) * (up x)) for weights `p`gate / up / down."""

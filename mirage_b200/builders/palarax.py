@@ -20,16 +20,8 @@ from typing import Any, Dict, List, Optional, Tuple
 import torch
 
 from ..mpk import register_model_builder
-from ..persistent_kernel import DTensor, PersistentKernel, float32
-from .hybrid import HybridBuilder, HybridModelConfig, round_up
-
-
-@dataclass(frozen=True)
-class MlstmSpec:
-    heads: int
-    dim: int
-    vdim: int
-    gate_cap: float
+from ..persistent_kernel import DTensor, float32
+from .hybrid import HybridBuilder, HybridModelConfig, MlstmSpec, round_up
 
 
 @dataclass(frozen=True)
@@ -80,7 +72,7 @@ class PalaraxConfig:
         for n, entry in enumerate(c["layers"]):
             m = entry["mixer"]
             if entry["type"] == "mlstm":
-                mixer = MlstmSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"]))
+                mixer = MlstmSpec.from_dict(m)
             elif entry["type"] == "parallel":
                 l, r = m["left"], m["right"]
                 left = AttentionSpec(int(l["heads"]), int(l["kv_heads"]), int(l["dim"]), int(l["vdim"]),
@@ -114,9 +106,7 @@ def allocate_state(c: PalaraxConfig, *, slots: int, max_num_pages: int, page_siz
     for layer in c.layers:
         m = layer.mixer
         if isinstance(m, MlstmSpec):
-            chunks = PersistentKernel.mlstm_chunks(num_workers, slots, m.heads, m.dim, m.vdim)
-            out.append({"memory": z32(slots, m.heads, m.dim, round_up(m.vdim, 4)),
-                        "normaliser": z32(slots, m.heads, chunks, m.dim + 1)})
+            out.append(m.state(slots, num_workers, device))
         else:
             shape = lambda d: (max_num_pages, page_size, m.left.kv_heads, round_up(d, 8))
             out.append({"k": torch.zeros(shape(m.left.dim), dtype=dtype, device=device),
@@ -132,22 +122,6 @@ PalaraxModelConfig = HybridModelConfig
 @register_model_builder("palarax")
 class PalaraxBuilder(HybridBuilder):
     # -- mixers: `h` is the normed input; return the mixer's float32 output
-    def _mlstm(self, p: str, m: MlstmSpec, st: Dict[str, torch.Tensor], h: DTensor) -> DTensor:
-        mpk, sd = self.mpk, self.sd
-        qk, v = m.heads * m.dim, m.heads * m.vdim
-        proj = self._buf("proj", 2 * qk + 2 * v + 2 * m.heads, float32)
-        self._linear(h, self._weight(p + "qkvgif", [sd[p + n] for n in ("q", "k", "v", "g", "i", "f")]), proj)
-        out = self._buf("mixed", self._kpad(v), self.act)
-        mpk.mlstm_layer(proj, self._att(p + "i.b"), self._att(p + "f.b"), self._att(p + "norm"),
-                        mpk.attach_input(st["memory"], name=p + "memory"),
-                        mpk.attach_input(st["normaliser"], name=p + "normaliser"), self._buf("readout", v, float32), out,
-                        heads=m.heads, dim=m.dim, vdim=m.vdim, q_col=0, k_col=qk, v_col=2 * qk, gate_col=2 * qk + v,
-                        i_col=2 * qk + 2 * v, f_col=2 * qk + 2 * v + m.heads, gate_cap=m.gate_cap, eps=self.eps,
-                        q_scale=m.dim ** -0.5)
-        y = self._buf("sublayer", self.width, float32)
-        self._linear(out, self._weight(p + "o.padded", [sd[p + "o"]]), y)
-        return y
-
     def _parallel(self, p: str, m: ParallelSpec, st: Dict[str, torch.Tensor], h: DTensor) -> DTensor:
         mpk, sd = self.mpk, self.sd
         l, r, pl, pr = m.left, m.right, p + "left.", p + "right."

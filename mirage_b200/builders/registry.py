@@ -12,6 +12,7 @@ _RUNNERS = {
     "bebuzen": ("BebuzenRunner", "hybrid", (torch.bfloat16, torch.float32)),
     "lofirax": ("LofiraxRunner", "hybrid", (torch.bfloat16, torch.float32)),
     "palarax": ("PalaraxRunner", "hybrid", (torch.bfloat16, torch.float32)),
+    "ruludra": ("RuludraRunner", "hybrid", (torch.bfloat16, torch.float32)),
     "qwen3forcausallm": ("Qwen3Runner", "decoder", (torch.bfloat16,)),
 }
 

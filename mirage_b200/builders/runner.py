@@ -207,3 +207,10 @@ class BebuzenRunner(HybridRunner):
     def _model(cls):
         from . import bebuzen as m
         return m.BebuzenConfig, m.BebuzenBuilder, m.BebuzenModelConfig, m.allocate_state
+
+
+class RuludraRunner(HybridRunner):
+    @classmethod
+    def _model(cls):
+        from . import ruludra as m
+        return m.RuludraConfig, m.RuludraBuilder, m.RuludraModelConfig, m.allocate_state

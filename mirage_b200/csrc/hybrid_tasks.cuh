@@ -3,7 +3,8 @@
 //   float32 residual stream      TASK_EMBED_F32, TASK_RESIDUAL_NORM
 //   attention                    TASK_QKV_APPEND (norms, rotation, cache rows), TASK_LATENT_APPEND (latent rows that serve
 //                                as keys and values), TASK_EXT_ATTENTION (any head size, score scale, soft cap, sinks, sliding
-//                                window), TASK_DIFF_COMBINE (differential attention)
+//                                window, distance bias), TASK_DIFF_COMBINE (differential attention)
+//   activations                  TASK_POLY_NORM (beside those in the epilogues of linears)
 //   recurrences                  TASK_SHORT_CONV, TASK_RGLRU (gated diagonal), TASK_SELECTIVE_SCAN (diagonal, input-dependent steps),
 //                                TASK_MLSTM and TASK_GLA (matrix memories)
 //   experts                      TASK_MOE_ROUTING, TASK_MOE_GEMM (megakernel.cuh); their sum is part of TASK_RESIDUAL_NORM
@@ -83,6 +84,19 @@ __device__ __forceinline__ SeqView seq_view(const KernelParams &P, int k) {
   return s;
 }
 
+// The request batch token t belongs to: as many requests end at or before the token.  Called by a whole warp.
+__device__ __forceinline__ int request_of(const KernelParams &P, int t) {
+  const int lane = threadIdx.x & 31, mbr = P.max_num_batched_requests;
+  int k = 0;
+  for (int b = 0; b < mbr; b += 32) {
+    const bool before = b + lane < mbr && __ldcg(&P.meta.qo_indptr[b + lane + 1]) <= t;
+    const int n = __popc(__ballot_sync(0xffffffffu, before));
+    k += n;
+    if (n < 32) break;
+  }
+  return k;
+}
+
 // Per-token view for bodies that take all tokens of the batch at once (filled by token_map, shared memory).
 struct TokenRec {
   int q0;      // first token of this token's request
@@ -127,12 +141,50 @@ __device__ __forceinline__ void run_embed_f32(const Ctx &c, const TaskDesc &d) {
   }
 }
 
+// Rows with further terms: the bigram of the token and the one before it, and sines and cosines of the position.  Angles are turns in
+// units of 2^-64, position times frequency, so that their reduction is exact.
+static __device__ __noinline__ void run_embed_sum(const Ctx c, const TaskDesc &d) {
+  const KernelParams &P = c.P;
+  const int B = active_tokens(P);
+  const int t1 = min(d.a[E_T1], B), width = d.a[E_WIDTH];
+  const long long *ids = reinterpret_cast<const long long *>(d.p[0]);
+  const long long *freq = reinterpret_cast<const long long *>(d.p[4]);
+  const float factor = __int_as_float(d.a[E_LDI2]);
+  for (int t = d.a[E_T0]; t < t1; ++t) {
+    const long long id = __ldcg(ids + t);
+    const bool in_table = id >= 0 && id < (long long)d.a[E_AUX];
+    const int k = request_of(P, t);
+    const SeqView s = seq_view(P, k);
+    const int pos = s.pos0 + t - s.q0;
+    unsigned long long pair = (unsigned)d.a[E_BUCKETS];
+    if (d.p[3] && pos > 0) {
+      const int row = P.meta_static ? k : __ldcg(&P.meta.request_ids[k]);
+      const unsigned long long prev = t > s.q0 ? __ldcg(ids + t - 1) : __ldcg(reinterpret_cast<const long long *>(P.meta.tokens) + (size_t)row * P.max_seq_length + pos - 1);
+      pair = (prev * wide_arg(d, E_PREV) + (unsigned long long)id * wide_arg(d, E_CUR)) % pair;
+    }
+    float *out = reinterpret_cast<float *>(d.p[2]) + (size_t)t * d.a[E_LDO], *copy = reinterpret_cast<float *>(d.p[5]) + (size_t)t * d.a[E_LDC];
+#pragma unroll 4
+    for (int j = threadIdx.x; j < width; j += kConsumerThreads) {
+      float v = in_table ? bf16_at(d.p[1], (size_t)id * d.a[E_LDI] + j) * factor : 0.f;
+      if (d.p[3]) v += bf16_at(d.p[3], (size_t)pair * d.a[E_LDB] + j);
+      if (freq) {
+        const unsigned long long turns = (unsigned long long)pos * (unsigned long long)__ldg(freq + (j >> 1));
+        const float half_turns = (float)(int)(turns >> 32) * (1.0f / 2147483648.0f);
+        v += (j & 1) ? cospif(half_turns) : sinpif(half_turns);
+      }
+      out[j] = v;
+      if (d.p[5]) copy[j] = v;
+    }
+  }
+}
+
 // What joins the stream beside the sublayer output y (pointers are null where a layer has no such term).
 struct NormTerms {
   const float *add, *experts, *ew, *gate;   // added stream, expert outputs and their weights, logit whose sigmoid scales y
   uint64_t row, bias;                       // row added to every token, bias of the output norm
   int slots;
   float factor;                             // of y's norm
+  float *results;                           // this token's row of the earlier results, or null: their weighted sum becomes the stream
 };
 __device__ __forceinline__ NormTerms norm_terms(const TaskDesc &d, int t) {
   NormTerms n;
@@ -148,6 +200,8 @@ __device__ __forceinline__ NormTerms norm_terms(const TaskDesc &d, int t) {
   if (n.gate) n.gate += (size_t)t * d.a[RN_LDGATE];
   n.row = wide_arg(d, RN_ROW);
   n.bias = wide_arg(d, RN_BIAS);
+  n.results = reinterpret_cast<float *>(d.p[6]);
+  if (n.results) n.results += (size_t)t * d.a[2];
   return n;
 }
 
@@ -212,6 +266,12 @@ __device__ __forceinline__ void residual_norm_rows(const Ctx &c, const TaskDesc 
         for (int k = 0; k < (has_post ? 0 : nt.slots); ++k) xv[e] = fmaf(__ldcg(nt.ew + k), __ldcg(nt.experts + (size_t)k * W + j + e), xv[e]);
         if (nt.add) xv[e] += __ldcg(nt.add + j + e);
         if (nt.row) xv[e] += bf16_at(nt.row, j + e);
+        if (nt.results) {
+          const int last = d.a[RN_TERMS] - 1;
+          nt.results[(size_t)last * d.a[RN_HSTRIDE] + j + e] = xv[e];
+          xv[e] *= bf16_at(d.p[7], last);
+          for (int k = 0; k < last; ++k) xv[e] = fmaf(bf16_at(d.p[7], k), __ldcg(nt.results + (size_t)k * d.a[RN_HSTRIDE] + j + e), xv[e]);
+        }
         ss += xv[e] * xv[e];
         sum += xv[e];
         row[j + e] = xv[e];
@@ -326,6 +386,32 @@ __device__ __forceinline__ void residual_norm_wide(const Ctx &c, const TaskDesc 
         if (nt.row) fma4(xv[i], 1.f, bf16x4_at(nt.row, j));
       }
     }
+    if (nt.results) {
+      const int last = d.a[RN_TERMS] - 1;
+      const float w = bf16_at(d.p[7], last);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int j = (i * kConsumerThreads + tid) * 4;
+        if (j < W) *reinterpret_cast<float4 *>(nt.results + (size_t)last * d.a[RN_HSTRIDE] + j) = xv[i];
+        xv[i].x *= w; xv[i].y *= w; xv[i].z *= w; xv[i].w *= w;
+      }
+      for (int k = 0; k < last; k += 2) {   // two earlier results in flight
+        float4 e[2][NV];
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+          for (int i = 0; i < NV; ++i) {
+            const int j = (i * kConsumerThreads + tid) * 4;
+            e[u][i] = j < W && k + u < last ? __ldcg(reinterpret_cast<const float4 *>(nt.results + (size_t)(k + u) * d.a[RN_HSTRIDE] + j)) : zero;
+          }
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          const float wk = k + u < last ? bf16_at(d.p[7], k + u) : 0.f;
+#pragma unroll
+          for (int i = 0; i < NV; ++i) fma4(xv[i], wk, e[u][i]);
+        }
+      }
+    }
     if (has_y || nt.slots > 0 || nt.add || nt.row) {
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
@@ -372,7 +458,7 @@ template <int HYB>
 __device__ __noinline__ void run_residual_norm(const Ctx c, const TaskDesc &d) {
   if (d.a[2] <= 4096 && ((d.a[2] | d.a[3] | d.a[4] | d.a[5] | d.a[8]) & 3) == 0 && ((d.p[0] | d.p[1] | d.p[4] | d.p[5]) & 15) == 0 &&
       ((d.p[2] | d.p[3] | wide_arg(d, RN_BIAS) | wide_arg(d, RN_ROW)) & 7) == 0 && (d.a[RN_LDADD] & 3) == 0 &&
-      ((wide_arg(d, RN_ADD) | wide_arg(d, RN_EXP)) & 15) == 0) {
+      ((wide_arg(d, RN_ADD) | wide_arg(d, RN_EXP) | d.p[6]) & 15) == 0 && (d.a[RN_HSTRIDE] & 3) == 0) {
     residual_norm_wide<HYB>(c, d);
     return;
   }
@@ -403,7 +489,7 @@ __device__ __forceinline__ void dot8_f32(uint64_t w, size_t wrow, const float *x
 template <class F>
 __device__ __forceinline__ void column_f32(uint64_t w, size_t ldw, const float *xs, int K, int n, int nt, int act, float cap, F emit) {
   const int lane = threadIdx.x & 31;
-  const bool gated = act >= ACT_GATED_SILU;
+  const bool gated = act == ACT_GATED_SILU || act == ACT_GATED_GELU;
   const size_t row = gated ? (size_t)(n >> 1) * 4 + (n & 1) : n;
   for (int t8 = 0; t8 < nt; t8 += 8) {
     float acc[8], up[8];
@@ -420,6 +506,8 @@ __device__ __forceinline__ void column_f32(uint64_t w, size_t ldw, const float *
         v *= v;
       } else if (act == ACT_SOFTCAP) {
         v = cap * tanhf(v / cap);
+      } else if (act == ACT_SCALE) {
+        v *= cap;
       }
       if (lane == u && t8 + u < nt) emit(t8 + u, v);
     }
@@ -439,7 +527,10 @@ static __device__ __noinline__ void run_linear_f32(const Ctx c, const TaskDesc &
       for (int k = tid; k < K; k += kConsumerThreads) xs[(size_t)t * K + k] = __ldcg(x + (size_t)(tb + t) * d.a[4] + k);
     consumer_sync();
     for (int n = n0 + warp; n < n1; n += 8)
-      column_f32(d.p[0], d.a[3], xs, K, n, nt, d.a[6], __int_as_float(d.a[8]), [&](int t, float v) { out[(size_t)(tb + t) * d.a[5] + n] = d.p[3] ? v + bf16_at(d.p[3], n) : v; });
+      column_f32(d.p[0], d.a[3], xs, K, n, nt, d.a[6], __int_as_float(d.a[8]), [&](int t, float v) {
+        if (d.p[4]) v *= sigmoid_f(__ldcg(reinterpret_cast<const float *>(d.p[4]) + (size_t)(tb + t) * d.a[9] + n));
+        out[(size_t)(tb + t) * d.a[5] + n] = d.p[3] ? v + bf16_at(d.p[3], n) : v;
+      });
   }
 }
 // Expert projections: the active experts one after the other, the tokens routed to each gathered in shared memory.
@@ -482,19 +573,6 @@ static __device__ __noinline__ void run_moe_gemm_f32(const Ctx c, const TaskDesc
                    [&](int t, float v) { out[(size_t)list[tb + t] * d.a[5] + n] = v; });
     }
   }
-}
-
-// The request batch token t belongs to: as many requests end at or before the token.  Called by a whole warp.
-__device__ __forceinline__ int request_of(const KernelParams &P, int t) {
-  const int lane = threadIdx.x & 31, mbr = P.max_num_batched_requests;
-  int k = 0;
-  for (int b = 0; b < mbr; b += 32) {
-    const bool before = b + lane < mbr && __ldcg(&P.meta.qo_indptr[b + lane + 1]) <= t;
-    const int n = __popc(__ballot_sync(0xffffffffu, before));
-    k += n;
-    if (n < 32) break;
-  }
-  return k;
 }
 
 // ---------------------------------------------------------------------------
@@ -559,6 +637,60 @@ __device__ __noinline__ void run_qkv_append(const Ctx c, const TaskDesc &d) {
   }
 }
 
+// The norms span all heads and nothing is rotated: a block takes a token's queries, or its keys and values.
+template <int HYB>
+__device__ __noinline__ void run_qkv_append_whole(const Ctx c, const TaskDesc &d) {
+  typedef typename HybElt<HYB>::T T;
+  constexpr int NR = 16;   // a row's first 4096 columns, in registers
+  const KernelParams &P = c.P;
+  const int B = active_tokens(P), tid = threadIdx.x;
+  const int hq = d.a[QA_HQ], hkv = d.a[QA_HKV], dim = d.a[QA_DIM], dimp = d.a[QA_DIMP], vdim = d.a[QA_VDIM], vdimp = d.a[QA_VDIMP], page = d.a[QA_PAGE];
+  const int parts = d.p[2] ? 2 : 1;
+  for (int item = d.a[QA_T0]; item < B * parts; item += d.a[QA_T1]) {
+    const int t = item / parts;
+    const bool is_q = item == t * parts;
+    const SeqView s = seq_view(P, request_of(P, t));
+    const int pos = s.pos0 + t - s.q0, n = (is_q ? hq : hkv) * dim;
+    const float *row = reinterpret_cast<const float *>(d.p[0]) + (size_t)t * d.a[QA_LDP];
+    const float *src = row + (is_q ? d.a[QA_QOFF] : d.a[QA_KOFF]);
+    const uint64_t norm = is_q ? d.p[6] : d.p[7];
+    float x[NR], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int j = i * kConsumerThreads + tid;
+      x[i] = j < n ? __ldcg(src + j) : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < NR; ++i) ss += x[i] * x[i];
+    for (int j = NR * kConsumerThreads + tid; j < n; j += kConsumerThreads) { const float v = __ldcg(src + j); ss += v * v; }
+    float inv = 1.0f / sqrtf(block_sum(ss, c.s.red) / (float)n + __int_as_float(d.a[QA_EPS]));
+    if (is_q && d.a[QA_EVERY] > 0) inv *= 1.0f + __int_as_float(d.a[QA_TEMP]) * logf((float)((pos + 1) / d.a[QA_EVERY] + 1));
+    T *dst = reinterpret_cast<T *>(d.p[1]) + (size_t)t * d.a[QA_LDQ], *vdst = nullptr;
+    if (!is_q) {
+      const int pg = pos / page;
+      const size_t cell = ((size_t)__ldcg(&P.meta.paged_kv_indices[s.kv0 + pg]) * page + (pos - pg * page)) * hkv;
+      dst = reinterpret_cast<T *>(d.p[2]) + cell * dimp;
+      vdst = reinterpret_cast<T *>(d.p[3]) + cell * vdimp;
+    }
+    // the keys as projected are the values: they are in registers already
+    const bool same = !is_q && d.a[QA_VOFF] == d.a[QA_KOFF] && vdim == dim;
+    auto place = [&](int j, float v) {
+      const int h = dim == dimp && (is_q || vdim == vdimp) ? 0 : j / dim;
+      store_elt(dst + j + h * (dimp - dim), v * bf16_at(norm, j) * inv);
+      if (same) store_elt(vdst + j + h * (vdimp - vdim), v);
+    };
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int j = i * kConsumerThreads + tid;
+      if (j < n) place(j, x[i]);
+    }
+    for (int j = NR * kConsumerThreads + tid; j < n; j += kConsumerThreads) place(j, __ldcg(src + j));
+    if (!is_q && !same)
+      for (int j = tid; j < hkv * vdim; j += kConsumerThreads) store_elt(vdst + j + j / vdim * (vdimp - vdim), __ldcg(row + d.a[QA_VOFF] + j));
+    consumer_sync();   // the reduction slots are used again
+  }
+}
+
 // ---------------------------------------------------------------------------
 // TASK_LATENT_APPEND: one warp per (token, head) rotates the head's rotary query part into its columns of q (behind the
 // `rank` latent columns, which a grouped linear writes); one more warp per token writes the token's cache row: the latent,
@@ -570,7 +702,8 @@ __device__ __noinline__ void run_latent_append(const Ctx c, const TaskDesc &d) {
   const KernelParams &P = c.P;
   const int B = active_tokens(P);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int H = d.a[LA_H], rank = d.a[LA_RANK], rot = d.a[LA_ROT], half = rot >> 1, dimp = d.a[LA_DIMP], page = d.a[LA_PAGE];
+  const int rank = d.a[LA_RANK], rot = d.a[LA_ROT], half = rot >> 1, dimp = d.a[LA_DIMP], page = d.a[LA_PAGE];
+  const int H = rot > 0 ? d.a[LA_H] : 0;   // heads with something to rotate
   for (int item = d.a[LA_T0] * 8 + warp; item < B * (H + 1); item += d.a[LA_T1] * 8) {
     const int t = item / (H + 1), h = item - t * (H + 1);
     const SeqView s = seq_view(P, request_of(P, t));
@@ -585,10 +718,17 @@ __device__ __noinline__ void run_latent_append(const Ctx c, const TaskDesc &d) {
       const float *lat = row + d.a[LA_KVOFF];
       const int pg = pos / page;
       T *cell = reinterpret_cast<T *>(d.p[3]) + ((size_t)__ldcg(&P.meta.paged_kv_indices[s.kv0 + pg]) * page + (pos - pg * page)) * dimp;
-      float ss = 0.f;
-      for (int i = lane; i < rank; i += 32) { const float v = __ldcg(lat + i); ss += v * v; }
+      float x[16], ss = 0.f;   // 512 columns in registers, all loads in flight
+#pragma unroll
+      for (int u = 0; u < 16; ++u) x[u] = u * 32 + lane < rank ? __ldcg(lat + u * 32 + lane) : 0.f;
+#pragma unroll
+      for (int u = 0; u < 16; ++u) ss += x[u] * x[u];
+      for (int i = 512 + lane; i < rank; i += 32) { const float v = __ldcg(lat + i); ss += v * v; }
       const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)rank + __int_as_float(d.a[LA_EPS]));
-      for (int i = lane; i < rank; i += 32) store_elt(cell + i, __ldcg(lat + i) * inv * bf16_at(d.p[1], i));
+#pragma unroll
+      for (int u = 0; u < 16; ++u)
+        if (u * 32 + lane < rank) store_elt(cell + u * 32 + lane, x[u] * inv * bf16_at(d.p[1], u * 32 + lane));
+      for (int i = 512 + lane; i < rank; i += 32) store_elt(cell + i, __ldcg(lat + i) * inv * bf16_at(d.p[1], i));
       src = lat + rank;
       dst = cell + rank;
     }
@@ -624,6 +764,12 @@ __device__ __forceinline__ float attn_score(float dot, float scale, float cap, f
 template <int HYB>
 __device__ __forceinline__ float sink_logit(const TaskDesc &d, int h) {
   return d.p[4] ? bf16_at(d.p[4], h) * (HYB == HYB_F32 ? 1.0f : 1.4426950408889634f) : 0.f;
+}
+// What a distance takes off a score, in the domain's base: r1 ln(1 + r2 distance).
+template <int HYB>
+__device__ __forceinline__ float distance_bias(float r1, float r2, int distance) {
+  const float x = r2 * (float)max(distance, 0);
+  return r1 * (HYB == HYB_F32 ? log1pf(x) : __log2f(1.0f + x));
 }
 // Keys of a request in the order the tasks walk them.  Without a window: positions 0, 1, ....  With one, positions that no token
 // of the portion sees are left out: first `kept` positions (a multiple of eight that covers the ones kept for good), then
@@ -764,7 +910,9 @@ struct AttnRows {
   int p_all;        // keys up to here are not ahead of any row of the tile
   int p_far;        // keys from here on are in the window of every row
   bool two;         // rows 8 .. 15 of the tile hold queries
+  float r1[2], r2[2];   // distance bias of this lane's two rows
 };
+template <bool BIAS>
 __device__ __forceinline__ AttnRows attn_rows(const TaskDesc &d, const SeqView &sv, const AttnOut &ao, int first, int n, int kend) {
   AttnRows w;
   w.scale = __int_as_float(d.a[XA_SCALE]);
@@ -777,11 +925,19 @@ __device__ __forceinline__ AttnRows attn_rows(const TaskDesc &d, const SeqView &
   w.p_all = sv.pos0 + first / G;
   w.p_far = sv.pos0 + (first + n - 1) / G - ao.window + 1;
   w.two = n > 8;
+  if (BIAS) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int h = ao.head * G + (r + 8 * i) % G;
+      w.r1[i] = bf16_at(d.p[5], h);
+      w.r2[i] = bf16_at(d.p[6], h);
+    }
+  }
   return w;
 }
 // Eight keys (rows at kaddr / vaddr, this lane's ldmatrix addresses) against a 16-row query tile: scores, online softmax,
 // P V.  The first is number key0 (below w.kend) of the request's keys and lies at position `at`.
-template <int D, int ON, bool TWO>
+template <int D, int ON, bool TWO, bool BIAS>
 __device__ __forceinline__ void attn_octet(const AttnRows &w, const AttnOut &ao, const uint32_t (&qf)[TWO ? 1 : D / 16][2], uint32_t qa, uint32_t kaddr,
                                            uint32_t vaddr, int key0, int at, float (&m_run)[2], float (&l_run)[2], float (&o)[ON / 8][4]) {
   float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
@@ -807,6 +963,7 @@ __device__ __forceinline__ void attn_octet(const AttnRows &w, const AttnOut &ao,
   for (int e = 0; e < 4; ++e) {
     if (e >= 2 && !(TWO && w.two)) { s[e] = -INFINITY; continue; }
     s[e] = attn_score<HYB_BF16>(s[e] + s2[e], w.scale, w.cap, w.cap2);
+    if (BIAS) s[e] -= distance_bias<HYB_BF16>(w.r1[e >> 1], w.r2[e >> 1], (e < 2 ? w.p_lo : w.p_hi) - at - 2 * ((int)threadIdx.x & 3) - (e & 1));
   }
   if (at + 7 > w.p_all || key0 + 8 > w.kend || at < w.p_far) {
     const int off = 2 * (threadIdx.x & 3);
@@ -879,7 +1036,7 @@ __device__ __forceinline__ void attn_emit_splits(const Ctx &c, const TaskDesc &d
 
 // One tile of query rows (decoding, or a task's share of a prompt portion): every warp streams its own octets of keys, w,
 // w + 8, ..., through its own ring -- no block barrier in the loop -- and the eight partial results are combined at the end.
-template <int D, bool TWO>
+template <int D, bool TWO, bool BIAS>
 __device__ __noinline__ void ext_attention_stream(const Ctx c, const TaskDesc &d, const SeqView sv, const AttnOut &ao, int k0, int k1,
                                                   int row0, int nrow, int task) {
   constexpr int PITCH = D * 2 + 16, STEP = 16 * PITCH, PIECES = D / 8, RSTEP = 32 / PIECES;
@@ -933,7 +1090,7 @@ __device__ __noinline__ void ext_attention_stream(const Ctx c, const TaskDesc &d
   }
   consumer_sync();
   stamp(c, task, 0);
-  const AttnRows w = attn_rows(d, sv, ao, row0, nrow, kend);
+  const AttnRows w = attn_rows<BIAS>(d, sv, ao, row0, nrow, kend);
   const uint32_t qa = smem_u32(qs) + (uint32_t)((lane & 15) * PITCH + (lane >> 4) * 16);
   uint32_t qf[TWO ? 1 : D / 16][2];   // rows 0 .. 7 only: two of a fragment's four registers
   if (!TWO) {
@@ -958,7 +1115,7 @@ __device__ __noinline__ void ext_attention_stream(const Ctx c, const TaskDesc &d
     issue(slot == 0 ? nstg - 1 : slot - 1);
     const uint32_t ka = ring + slot * STEP + lane_off;
     const int key0 = k0 + (warp + 8 * i) * 8;
-    attn_octet<D, D, TWO>(w, ao, qf, qa, ka, ka + 8 * PITCH, key0, keys.pos(key0), m_run, l_run, o);
+    attn_octet<D, D, TWO, BIAS>(w, ao, qf, qa, ka, ka + 8 * PITCH, key0, keys.pos(key0), m_run, l_run, o);
     if (++slot == nstg) slot = 0;
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -993,7 +1150,7 @@ __device__ __forceinline__ uint32_t movmatrix_trans(uint32_t v) {
   asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
   return r;
 }
-template <int D>
+template <int D, bool BIAS>
 __device__ __noinline__ void ext_attention_decode(const Ctx c, const TaskDesc &d, const SeqView sv, const AttnOut &ao, int k0, int k1,
                                                   int row0, int nrow, int task) {
   constexpr int PITCH = D * 2 + 16, OCT = 8 * PITCH, PIECES = D / 8, RSTEP = 32 / PIECES, STEPS = 2;
@@ -1062,6 +1219,15 @@ __device__ __noinline__ void ext_attention_decode(const Ctx c, const TaskDesc &d
   const int q0 = row0 + 2 * (lane & 3);
   const int p_a = sv.pos0 + q0 / ao.G, p_b = sv.pos0 + (q0 + 1) / ao.G, p_all = sv.pos0 + row0 / ao.G;
   const int p_far = sv.pos0 + (row0 + nrow - 1) / ao.G - ao.window + 1;
+  float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};   // distance bias of the two
+  if (BIAS) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int h = ao.head * ao.G + (q0 + i) % ao.G;
+      r1[i] = bf16_at(d.p[5], h);
+      r2[i] = bf16_at(d.p[6], h);
+    }
+  }
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
   float o[D / 16][4];
 #pragma unroll
@@ -1087,6 +1253,10 @@ __device__ __noinline__ void ext_attention_decode(const Ctx c, const TaskDesc &d
 #pragma unroll
     for (int e = 0; e < 4; ++e) s[e] = attn_score<HYB_BF16>(s[e] + s2[e], scale, cap, cap2);
     const int at0 = keys.pos(key0), at1 = keys.pos(key0 + 8);
+    if (BIAS) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[e] -= distance_bias<HYB_BF16>(r1[e & 1], r2[e & 1], ((e & 1) ? p_b : p_a) - (e >> 1 ? at1 : at0) - (lane >> 2));
+    }
     if (at1 + 7 > p_all || key0 + 16 > kend || at0 < p_far) {   // e: key g + 8 (e / 2), query 2 q + (e & 1)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
@@ -1158,7 +1328,7 @@ __device__ __noinline__ void ext_attention_decode(const Ctx c, const TaskDesc &d
 // bf16: QK^T and PV on mma.sync.  Head sizes are padded to D columns in shared memory.  The eight warps are split over
 // row tiles (16 rows), key octets and, for D = 256, halves of the output columns; the key split is combined in shared
 // memory.  The probabilities enter PV as a bf16 value and a bf16 remainder, so that the weights keep 16 bits.
-template <int D>
+template <int D, bool BIAS>
 __device__ __noinline__ void ext_attention_mma(const Ctx c, const TaskDesc &d, const SeqView sv, const AttnOut &ao, int k0, int k1,
                                                   int row0, int rows, int task) {
   constexpr int ON = D < 128 ? D : 128, WN = D / ON, KEYS = D > 128 ? 32 : 64, NSUB = KEYS / 8, PITCH = D * 2 + 16;
@@ -1225,7 +1395,7 @@ __device__ __noinline__ void ext_attention_mma(const Ctx c, const TaskDesc &d, c
     for (int i = 0; i < ON / 8; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
-    const AttnRows w = attn_rows(d, sv, ao, rb + wm * 16, min(nrow - wm * 16, 16), kend);
+    const AttnRows w = attn_rows<BIAS>(d, sv, ao, rb + wm * 16, min(nrow - wm * 16, 16), kend);
     const int ntiles = kend > k0 ? (kend - k0 + KEYS - 1) / KEYS : 0;
     consumer_sync();   // queries and cells
     stamp(c, task, 0);
@@ -1255,7 +1425,7 @@ __device__ __noinline__ void ext_attention_mma(const Ctx c, const TaskDesc &d, c
       for (int j = wk; j < NSUB; j += WK) {
         const int key0 = base + j * 8;
         if (key0 >= kend) break;
-        attn_octet<D, ON, true>(w, ao, qf, qa, kt + (uint32_t)(j * 8 * PITCH), vt + (uint32_t)(j * 8 * PITCH), key0, keys.pos(key0), m_run, l_run, o);
+        attn_octet<D, ON, true, BIAS>(w, ao, qf, qa, kt + (uint32_t)(j * 8 * PITCH), vt + (uint32_t)(j * 8 * PITCH), key0, keys.pos(key0), m_run, l_run, o);
       }
     }
     consumer_sync();   // the stages become the combine area
@@ -1407,7 +1577,7 @@ __device__ __noinline__ void latent_attention_mma(const KernelParams &P, uint32_
   };
   for (int i = 0; i < la.stages - 2; ++i) issue(i, ring + i * KEYS * pitch);   // (the queries join the first group)
   const int nv = (la.ao.vdim >> 3) > warp ? ((la.ao.vdim >> 3) - warp + 7) >> 3 : 0;   // this warp's column tiles
-  // softmax: this lane's key of the tile, its first row and the last keys that row set sees
+  // softmax: this lane's key of the tile, its first row and how far behind that row set the key lies
   const int skey = lane % KEYS, srow = warp * (RT / 8) + lane / KEYS;
   int seen[RPW];
   float m_run[RPW], l_run[RPW];
@@ -1415,7 +1585,7 @@ __device__ __noinline__ void latent_attention_mma(const KernelParams &P, uint32_
   for (int i = 0; i < RPW; ++i) {
     m_run[i] = -INFINITY;
     l_run[i] = 0.f;
-    seen[i] = min(la.keys - 1, la.pos0 + (la.row0 + srow + i * (32 / KEYS)) / la.ao.G - la.k0) - skey;   // relative to the tile's first key
+    seen[i] = la.pos0 + (la.row0 + srow + i * (32 / KEYS)) / la.ao.G - la.k0 - skey;   // distance from this lane's key of the first tile
   }
   float o[NV][4];
 #pragma unroll
@@ -1499,6 +1669,8 @@ __device__ __noinline__ void latent_attention_mma(const KernelParams &P, uint32_
       const uint32_t sa = sm + (uint32_t)((srow * SP + skey) * 4), pa = sm + oP + (uint32_t)(srow * PP + skey * 2);
       const float scale = lds_f32(args + offsetof(LatentArgs, scale)), cap = lds_f32(args + offsetof(LatentArgs, cap));
       const float cap2 = cap > 0.f ? 2.0f * 1.4426950408889634f / cap : 0.f;
+      // keys past the chunk's end are in nobody's window
+      const int window = it * KEYS + skey < lds_s32(args + kLatentHot) ? lds_s32(args + offsetof(LatentArgs, ao) + offsetof(AttnOut, window)) : 0;
 #pragma unroll
       for (int i = 0; i < RPW; ++i) {
         const int r = i * (32 / KEYS);
@@ -1506,7 +1678,7 @@ __device__ __noinline__ void latent_attention_mma(const KernelParams &P, uint32_
 #pragma unroll
         for (int p = 0; p < KS; ++p) v += lds_f32(sa + (p * RT + r) * SP * 4);
         v = attn_score<HYB_BF16>(v, scale, cap, cap2);
-        if (it * KEYS > seen[i]) v = -INFINITY;
+        if ((unsigned)(seen[i] - it * KEYS) >= (unsigned)window) v = -INFINITY;
         float mx = v;
 #pragma unroll
         for (int sh = KEYS / 2; sh > 0; sh >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, sh));
@@ -1579,6 +1751,7 @@ static __device__ __noinline__ void ext_attention_f32(const Ctx c, const TaskDes
   const float *qg = reinterpret_cast<const float *>(d.p[0]);
   const float *kg = reinterpret_cast<const float *>(d.p[1]), *vg = reinterpret_cast<const float *>(d.p[2]);
   const AttnKeys keys = ao.keys;
+  const bool bias = d.p[5] != 0;
   auto cell_of = [&](int key) {
     const int pg = key / page;
     return ((size_t)__ldcg(&P.meta.paged_kv_indices[sv.kv0 + pg]) * page + (key - pg * page)) * hkv + ao.head;
@@ -1588,6 +1761,8 @@ static __device__ __noinline__ void ext_attention_f32(const Ctx c, const TaskDes
     __syncwarp();
     for (int i = lane; i < dimp; i += 32) q[i] = __ldcg(qg + (size_t)(sv.q0 + r / G) * d.a[XA_LDQ] + (size_t)(ao.head * G + r % G) * dimp + i);
     __syncwarp();
+    const int hb = ao.head * G + r % G;
+    const float r1 = bias ? bf16_at(d.p[5], hb) : 0.f, r2 = bias ? bf16_at(d.p[6], hb) : 0.f;
     float m = -INFINITY, l = 0.f, o[NO];
 #pragma unroll
     for (int i = 0; i < NO; ++i) o[i] = 0.f;
@@ -1605,6 +1780,7 @@ static __device__ __noinline__ void ext_attention_f32(const Ctx c, const TaskDes
           dot += kv.x * qv.x + kv.y * qv.y + kv.z * qv.z + kv.w * qv.w;
         }
         s = attn_score<HYB_F32>(dot, scale, cap, 0.f);
+        if (bias) s -= distance_bias<HYB_F32>(r1, r2, pos - at);
       }
       const float mn = fmaxf(m, warp_max(s));
       if (mn == -INFINITY) continue;   // none of these keys is seen
@@ -1630,6 +1806,22 @@ static __device__ __noinline__ void ext_attention_f32(const Ctx c, const TaskDes
       return v;
     });
   }
+}
+
+// Head sizes padded to D columns, bf16: the body for the task's rows.
+template <int D, bool BIAS>
+__device__ __forceinline__ void ext_attention_sized(const Ctx &c, const TaskDesc &d, const SeqView &sv, const AttnOut &ao, int k0, int k1, int row0,
+                                                    int row1, int task) {
+  if constexpr (D <= 128) {
+    const int n = row1 - row0;
+    if (n <= 16 && (d.a[XA_PAGE] & 7) == 0) {
+      if (n <= 8 && d.a[XA_STAGES] >= 3) ext_attention_decode<D, BIAS>(c, d, sv, ao, k0, k1, row0, n, task);
+      else if (n <= 8) ext_attention_stream<D, false, BIAS>(c, d, sv, ao, k0, k1, row0, n, task);
+      else ext_attention_stream<D, true, BIAS>(c, d, sv, ao, k0, k1, row0, n, task);
+      return;
+    }
+  }
+  ext_attention_mma<D, BIAS>(c, d, sv, ao, k0, k1, row0, row1, task);
 }
 
 template <int HYB>
@@ -1671,8 +1863,10 @@ __device__ __forceinline__ void run_ext_attention(const Ctx &c, const TaskDesc &
     const int keys = d.a[XA_KEYS];
     for (int r = row0; r < row1; r += 16) {
       if (r > row0) consumer_sync();
-      const int n = min(16, row1 - r), kend = min(k1, sv.pos0 + (r + n - 1) / ao.G + 1);   // keys past the last row's position are not needed
-      la.keys = max(kend - k0, 0);
+      // keys in front of the first row's window and past the last row's position are not needed
+      const int n = min(16, row1 - r), shift = ao.keys.shift, kend = min(k1 + shift, sv.pos0 + (r + n - 1) / ao.G + 1);
+      const int first = max(k0 + shift, (sv.pos0 + r / ao.G - ao.window + 1) & ~7);
+      la.keys = max(kend - first, 0);
       la.pieces = d.a[XA_DIMP] >> 3;
       la.table = (d.a[XA_PAGE] & 7) == 0 && la.keys <= 8 * kXaCells;   // eight consecutive keys lie in one page
       la.ntiles = (la.keys + keys - 1) / keys;
@@ -1680,25 +1874,20 @@ __device__ __forceinline__ void run_ext_attention(const Ctx &c, const TaskDesc &
       la.pages = c.P.meta.paged_kv_indices + sv.kv0;
       la.scale = __int_as_float(d.a[XA_SCALE]);
       la.cap = __int_as_float(d.a[XA_CAP]);
-      la.page = d.a[XA_PAGE]; la.k0 = k0; la.q0 = sv.q0; la.pos0 = sv.pos0; la.row0 = r; la.nrow = n; la.task = task; la.stages = d.a[XA_STAGES];
+      la.page = d.a[XA_PAGE]; la.k0 = first; la.q0 = sv.q0; la.pos0 = sv.pos0; la.row0 = r; la.nrow = n; la.task = task; la.stages = d.a[XA_STAGES];
       if (keys == 32) latent_attention_mma<32>(c.P, smem_u32(c.s.xtile), d, la);
       else latent_attention_mma<16>(c.P, smem_u32(c.s.xtile), d, la);
     }
   } else {
     const int w = max(d.a[XA_DIMP], d.a[XA_VDIMP]);
-    const bool one = row1 - row0 <= 16 && (d.a[XA_PAGE] & 7) == 0;
-    if (w <= 64) {
-      if (one && row1 - row0 <= 8 && d.a[XA_STAGES] >= 3) ext_attention_decode<64>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
-      else if (one && row1 - row0 <= 8) ext_attention_stream<64, false>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
-      else if (one) ext_attention_stream<64, true>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
-      else ext_attention_mma<64>(c, d, sv, ao, k0, k1, row0, row1, task);
-    } else if (w <= 128) {
-      if (one && row1 - row0 <= 8 && d.a[XA_STAGES] >= 3) ext_attention_decode<128>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
-      else if (one && row1 - row0 <= 8) ext_attention_stream<128, false>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
-      else if (one) ext_attention_stream<128, true>(c, d, sv, ao, k0, k1, row0, row1 - row0, task);
-      else ext_attention_mma<128>(c, d, sv, ao, k0, k1, row0, row1, task);
+    if (d.p[5]) {
+      if (w <= 64) ext_attention_sized<64, true>(c, d, sv, ao, k0, k1, row0, row1, task);
+      else if (w <= 128) ext_attention_sized<128, true>(c, d, sv, ao, k0, k1, row0, row1, task);
+      else ext_attention_sized<256, true>(c, d, sv, ao, k0, k1, row0, row1, task);
     } else {
-      ext_attention_mma<256>(c, d, sv, ao, k0, k1, row0, row1, task);
+      if (w <= 64) ext_attention_sized<64, false>(c, d, sv, ao, k0, k1, row0, row1, task);
+      else if (w <= 128) ext_attention_sized<128, false>(c, d, sv, ao, k0, k1, row0, row1, task);
+      else ext_attention_sized<256, false>(c, d, sv, ao, k0, k1, row0, row1, task);
     }
   }
   stamp(c, task, 3);
@@ -1777,6 +1966,70 @@ __device__ __noinline__ void run_diff_combine(const Ctx c, const TaskDesc &d) {
     for (int j = lane; j < vdim; j += 32) { const float x = __ldcg(a + j) - lambda * __ldcg(a + vdim + j); ss += x * x; }
     const float f = factor / sqrtf(warp_sum(ss) / (float)vdim + eps);
     for (int j = lane; j < vdim; j += 32) store_elt(out + j, (__ldcg(a + j) - lambda * __ldcg(a + vdim + j)) * f);
+  }
+}
+
+// ---------------------------------------------------------------------------
+// TASK_POLY_NORM: a N(z) + b N(z^2) + c N(z^3) + e, N dividing a token's values by their root mean square.  One block per token; with the
+// three factors known the sum is a cubic in z.
+// ---------------------------------------------------------------------------
+template <int HYB>
+__device__ __noinline__ void run_poly_norm(const Ctx c, const TaskDesc &d) {
+  typedef typename HybElt<HYB>::T T;
+  constexpr int NV = 16;   // 16384 columns in registers, all loads in flight
+  const int B = active_tokens(c.P), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int t1 = min(d.a[1], B), N = d.a[2];
+  const float eps = __int_as_float(d.a[5]), k1 = bf16_at(d.p[1], 0), k2 = bf16_at(d.p[1], 1), k3 = bf16_at(d.p[1], 2), k0 = bf16_at(d.p[1], 3);
+  const bool vec = N <= NV * kConsumerThreads * 4 && ((N | d.a[3] | d.a[4]) & 3) == 0 && ((d.p[0] | d.p[2]) & 15) == 0;
+  for (int t = d.a[0]; t < t1; ++t) {
+    const float *z = reinterpret_cast<const float *>(d.p[0]) + (size_t)t * d.a[3];
+    T *out = reinterpret_cast<T *>(d.p[2]) + (size_t)t * d.a[4];
+    float4 x[NV];
+    float s[3] = {0.f, 0.f, 0.f};
+    auto powers = [&](float v) {
+      const float q = v * v;
+      s[0] += q;
+      s[1] = fmaf(q, q, s[1]);
+      s[2] = fmaf(q * q, q, s[2]);
+    };
+    if (vec) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int j = (i * kConsumerThreads + tid) * 4;
+        x[i] = j < N ? __ldcg(reinterpret_cast<const float4 *>(z + j)) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+#pragma unroll
+      for (int i = 0; i < NV; ++i) { powers(x[i].x); powers(x[i].y); powers(x[i].z); powers(x[i].w); }
+    } else {
+#pragma unroll 4
+      for (int j = tid; j < N; j += kConsumerThreads) powers(__ldcg(z + j));
+    }
+#pragma unroll
+    for (int k = 0; k < 3; ++k) {
+      s[k] = warp_sum(s[k]);
+      if (lane == 0) c.s.red[8 * k + warp] = s[k];
+    }
+    consumer_sync();
+    float f[3];
+#pragma unroll
+    for (int k = 0; k < 3; ++k) {
+      float v = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) v += c.s.red[8 * k + w];
+      f[k] = (k == 0 ? k1 : k == 1 ? k2 : k3) / sqrtf(v / (float)N + eps);
+    }
+    auto cubic = [&](float v) { return fmaf(v, fmaf(v, fmaf(v, f[2], f[1]), f[0]), k0); };
+    if (vec) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int j = (i * kConsumerThreads + tid) * 4;
+        if (j < N) store_elt4(out + j, make_float4(cubic(x[i].x), cubic(x[i].y), cubic(x[i].z), cubic(x[i].w)));
+      }
+    } else {
+#pragma unroll 4
+      for (int j = tid; j < N; j += kConsumerThreads) store_elt(out + j, cubic(__ldcg(z + j)));
+    }
+    consumer_sync();   // the reduction slots are used again
   }
 }
 
@@ -3233,7 +3486,11 @@ __device__ __forceinline__ void run_hybrid_task(const Ctx &c, const TaskDesc &d,
       run_batch(cc);
       break;
     }
-    case TASK_EMBED_F32: run_embed_f32(c, d); break;
+    case TASK_EMBED_F32:
+      if (d.p[3] | d.p[4] | d.p[5]) run_embed_sum(c, d);
+      else run_embed_f32(c, d);
+      break;
+    case TASK_POLY_NORM: run_poly_norm<HYB>(c, d); break;
     case TASK_RESIDUAL_NORM: run_residual_norm<HYB>(c, d); break;
     case TASK_LINEAR_F32: if (HYB == HYB_F32) run_linear_f32(c, d); break;
     case TASK_MOE_ROUTING: run_moe_routing_hybrid(c, d); break;
@@ -3241,7 +3498,10 @@ __device__ __forceinline__ void run_hybrid_task(const Ctx &c, const TaskDesc &d,
     case TASK_LATENT_APPEND: run_latent_append<HYB>(c, d); break;
     case TASK_GLA: run_gla<HYB>(c, d, task); break;
     case TASK_ATTN_MERGE: run_attn_merge<HYB>(c, d); break;
-    case TASK_QKV_APPEND: run_qkv_append<HYB>(c, d); break;
+    case TASK_QKV_APPEND:
+      if (d.a[QA_WHOLE]) run_qkv_append_whole<HYB>(c, d);
+      else run_qkv_append<HYB>(c, d);
+      break;
     case TASK_EXT_ATTENTION: run_ext_attention<HYB>(c, d, task); break;
     case TASK_SHORT_CONV: run_short_conv<HYB>(c, d); break;
     case TASK_SELECTIVE_SCAN: run_selective_scan<HYB>(c, d, task); break;

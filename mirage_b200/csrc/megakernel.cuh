@@ -850,6 +850,11 @@ __device__ __forceinline__ void linear_output(const Ctx &c, const TaskDesc &d, i
   } else if (HYB && epi == EPI_SOFTCAP) {
     const float cap = __int_as_float(d.a[L_CAP]);
     reinterpret_cast<float *>(d.p[2])[(size_t)b * d.a[L_LDO] + col] = cap * tanhf(v / cap);
+  } else if (HYB && epi == EPI_SCALE_F32) {
+    reinterpret_cast<float *>(d.p[2])[(size_t)b * d.a[L_LDO] + col] = __int_as_float(d.a[L_CAP]) * v;
+  } else if (HYB && epi == EPI_GATE_SIGMOID) {
+    const float g = __ldcg(reinterpret_cast<const float *>(d.p[3]) + (size_t)b * d.a[L_LDR] + col);
+    reinterpret_cast<__nv_bfloat16 *>(d.p[2])[(size_t)b * d.a[L_LDO] + col] = __float2bfloat16_rn(v / (1.0f + expf(-g)));
   } else if (HYB && (epi == EPI_GATED_SILU || epi == EPI_GATED_GELU)) {
     if ((r & 2) == 0) {
       float u = 0.f;
@@ -997,7 +1002,7 @@ struct EmitArgs {
   __nv_bfloat16 *out;
   size_t push_off;      // element offset of (token 0, column 0) of this rank's slot in an inbox buffer
   int push_n;           // row length of the pushed matrix
-  uint32_t seq_hi;      // sequence number of the allreduce instance, already shifted to the high half (EPI_SOFTCAP: cap bits)
+  uint32_t seq_hi;      // sequence number of the allreduce instance, already shifted to the high half (EPI_SOFTCAP, EPI_SCALE_F32: cap / factor bits)
 };
 
 __device__ __forceinline__ EmitArgs emit_args(const Ctx &c, const TaskDesc &d) {
@@ -1009,7 +1014,7 @@ __device__ __forceinline__ EmitArgs emit_args(const Ctx &c, const TaskDesc &d) {
   const unsigned long long inst = c.iteration * (unsigned)d.a[L_NAR] + (unsigned)d.a[L_ARIDX];
   e.push_off = (size_t)d.p[5] + (size_t)(inst & 1ull) * (size_t)d.a[L_PARSTRIDE] + (size_t)c.P.rank * (size_t)d.a[L_SLOT];
   e.push_n = d.a[L_N];
-  e.seq_hi = e.epi == EPI_SOFTCAP ? (uint32_t)d.a[L_CAP] : ll_seq(c.iteration, d.a[L_NAR], d.a[L_ARIDX]) << 16;
+  e.seq_hi = e.epi == EPI_SOFTCAP || e.epi == EPI_SCALE_F32 ? (uint32_t)d.a[L_CAP] : ll_seq(c.iteration, d.a[L_NAR], d.a[L_ARIDX]) << 16;
   return e;
 }
 
@@ -1041,6 +1046,10 @@ __device__ __forceinline__ void linear_emit(const Ctx &c, const EmitArgs &e, int
   } else if (HYB && e.epi == EPI_SOFTCAP) {
     const float cap = __uint_as_float(e.seq_hi);
     reinterpret_cast<float *>(e.out)[(size_t)b * e.ldo + col] = cap * tanhf(v / cap);
+  } else if (HYB && e.epi == EPI_SCALE_F32) {
+    reinterpret_cast<float *>(e.out)[(size_t)b * e.ldo + col] = __uint_as_float(e.seq_hi) * v;
+  } else if (HYB && e.epi == EPI_GATE_SIGMOID) {
+    e.out[(size_t)b * e.ldo + col] = __float2bfloat16_rn(v / (1.0f + expf(-resv)));   // resv: the gate
   } else if (HYB && (e.epi == EPI_GATED_SILU || e.epi == EPI_GATED_GELU)) {
     if ((col & 2) == 0)
       e.out[(size_t)b * e.ldo + ((col >> 2) << 1) + (col & 1)] =
@@ -1159,6 +1168,7 @@ __device__ void run_linear_tc(const Ctx &c, const TaskDesc &d, LinearState &ls, 
           resv[j] = HYB ? bias : 0.f;
           if (epi == EPI_RESIDUAL && row_ok && b < B)
             resv[j] = bf16_to_f(__ldcg(resp + (size_t)b * ldr + n0 + row));
+          if (HYB && epi == EPI_GATE_SIGMOID && row_ok && b < B) resv[j] = __ldcg(reinterpret_cast<const float *>(resp) + (size_t)b * ldr + n0 + row);
         }
         tmem_ld_wait();
         if (tid == 0 && prof && tile == 0 && c0 == 0) P.profiler[(size_t)task * 8 + 6] = globaltimer_ns();

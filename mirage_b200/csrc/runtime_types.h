@@ -69,6 +69,7 @@ enum TaskType : uint32_t {
   TASK_ATTN_MERGE = 35,         // merge of an attention layer's key chunks
   TASK_SELECTIVE_SCAN = 36,     // selective state space recurrence
   TASK_DIFF_COMBINE = 37,       // differential attention: difference of the two maps' outputs, unit norm per head
+  TASK_POLY_NORM = 38,          // activation: weighted sum of the normed powers of a token's values
 };
 
 // Which family of megakernel instantiations runs a graph (template parameter HYB of the kernel).
@@ -107,7 +108,7 @@ MPK_HD constexpr int scan_staged_bytes(int tokens, int rank, int channels) {
 
 enum : int { HYB_NONE = 0, HYB_BF16 = 1, HYB_F32 = 2 };
 // Activations of hybrid linears (mpk_activation of include/mpk_b200.h).
-enum : int { ACT_NONE = 0, ACT_RELU2 = 1, ACT_SOFTCAP = 2, ACT_GATED_SILU = 3, ACT_GATED_GELU = 4 };
+enum : int { ACT_NONE = 0, ACT_RELU2 = 1, ACT_SOFTCAP = 2, ACT_GATED_SILU = 3, ACT_GATED_GELU = 4, ACT_SCALE = 5 };
 
 // Online mode: control word of a token-table row (KernelParams.meta.request_ctl[row], written by the host between
 // launches; request_ctl[rows + row] is the device's "live" flag).
@@ -133,6 +134,8 @@ enum Epilogue : int32_t {
   EPI_GATED_SILU = 8,   // rows [gate, gate, up, up]: out[2k + i] = bf16(silu(gate_i) * up_i) (hybrid graphs)
   EPI_GATED_GELU = 9,   // the same with the tanh form of gelu
   EPI_BIAS_F32 = 10,    // out = acc + bias, float32 (hybrid graphs)
+  EPI_SCALE_F32 = 11,   // out = factor * acc, float32 (hybrid graphs)
+  EPI_GATE_SIGMOID = 12,  // out = bf16(acc * sigmoid(gate)), the gate float32 (hybrid graphs)
   EPI_SILU_PAIR = 4,    // rows interleaved [gate, gate, up, up]: out[2k + i] = bf16(silu(gate_i)) * up_i
 };
 
@@ -175,7 +178,7 @@ static_assert(sizeof(TaskDesc) == 16 * kDescVecs, "TaskDesc must stay 224 bytes 
 //        null), a[20] ld y, a[21] ld x_out, a[22] flags (2: weights stored around zero, 4: layer norm), a[10] width (K minus the
 //        zero padding), p[5] norm bias or null, 64-bit values a[LR_ADD] added stream or null (ld a[LR_LDADD]), a[LR_ROW] added row or null
 //        a[LR_POST] factor of y's norm (bits); p[4] null: the activation is the stream as it is
-//  EPI_SOFTCAP: a[23] cap bits;  EPI_BIAS_F32: 64-bit value a[LR_BIAS]
+//  EPI_SOFTCAP, EPI_SCALE_F32: a[23] cap / factor bits;  EPI_BIAS_F32: 64-bit value a[LR_BIAS];  EPI_GATE_SIGMOID: p[3] gate f32, a[6] its ld
 //  a[15] allreduce index within the iteration  a[16] allreduces per iteration  a[17] stride between the two inbox buffers (floats)
 //  tcgen05 path (TF_TC): a[18] rows of one weight tile (the TMA box height, a multiple of 8, at most 128; the task's rows are
 //        cut into ceil(rows / a[18]) tiles, each one 128-lane accumulator), a[12] = 64 x (k blocks of 64 columns per ring slot),
@@ -230,28 +233,37 @@ enum { M_NEXP = 19, M_NTOPK, M_PER_SLOT, M_LDR, M_ESTRIDE };
 //      a[L_NAR], a[L_PARSTRIDE] as for the allreduce
 // ---- hybrid tasks --------------------------------------------------------------
 // ---- TASK_EMBED_F32: p[0] ids  p[1] table bf16  p[2] out f32;  a[E_*] as TASK_EMBED (a[E_AUX] = vocabulary, a[E_LDI2] factor bits)
+//      p[3] bigram table bf16 [buckets + 1, a[E_LDB]] or null  p[4] position frequencies int64 [(width + 1) / 2] or null  p[5] second copy of the output
+//      or null, a[E_LDC] its ld;  bigram row (previous id * mul_prev + id * mul_cur) mod buckets, 64-bit values a[E_PREV], a[E_CUR]
+enum { E_LDB = 7, E_BUCKETS, E_LDC, E_PREV = 10, E_CUR = 12 };
 // ---- TASK_RESIDUAL_NORM: rows [a[0], a[1]), width a[2]; p[0] x f32 (in place)  p[1] y f32 or null  p[2] weight of y's norm or
 //      null (plain sum)  p[3] weight of the output norm or null (out is the new x)  p[4] out (bf16, f32 with flag 1) or null  p[5] new x (= p[0]: in place);
 //      a[3] ld x  a[4] ld y  a[5] ld out  a[6] eps bits  a[7] flags (1: out f32, 2: weights stored around zero, 4: layer norm)  a[8] ld
 //      of the new x;  64-bit values, 0 if absent: a[RN_BIAS] norm bias, a[RN_ADD] added stream, a[RN_ROW] added row, a[RN_EXP] expert
 //      outputs f32 [tokens, slots, width], a[RN_EW] their weights f32, a[RN_GATE] f32 column, y is multiplied by its sigmoid
 //      a[RN_POST] factor of y's norm (bits); with that norm the experts' sum is part of what is normed
-enum { RN_LDADD = 9, RN_BIAS = 10, RN_ADD = 12, RN_ROW = 14, RN_EXP = 16, RN_EW = 18, RN_GATE = 20, RN_SLOTS = 22, RN_LDEW, RN_LDGATE, RN_POST };
+//      p[6] earlier results f32 or null (then a[RN_TERMS] >= 2 of them, a[RN_HSTRIDE] floats apart, rows of `width`), p[7] their weights bf16: the sum
+//      x + y goes to the last of the a[RN_TERMS] results, and the new stream is the weighted sum of all of them
+enum { RN_LDADD = 9, RN_BIAS = 10, RN_ADD = 12, RN_ROW = 14, RN_EXP = 16, RN_EW = 18, RN_GATE = 20, RN_SLOTS = 22, RN_LDEW, RN_LDGATE, RN_POST, RN_TERMS, RN_HSTRIDE };
 // ---- TASK_LINEAR_F32: p[0] W bf16 [N, K]  p[1] x f32  p[2] out f32;  a[0] n0  a[1] n1  a[2] K  a[3] ldw  a[4] ld x  a[5] ld out
-//      a[6] activation (mpk_activation)  a[7] tokens per shared-memory tile  a[8] soft cap bits
+//      a[6] activation (mpk_activation)  a[7] tokens per shared-memory tile  a[8] soft cap / factor bits  p[3] bias bf16 or null  p[4] gate f32 or null (the output
+//      is multiplied by its sigmoid)  a[9] ld gate
 // ---- TASK_MOE_GEMM_F32: p[0] W bf16 [E, N, K]  p[1] x f32  p[2] out f32  p[4] routing  p[5] active list;  a[0] n0  a[1] n1  a[2] K  a[4] ld x
 //      a[5] ld out (of a slot)  a[6] activation  a[7] tokens per shared-memory tile  a[8] x rows per (token, slot)  a[9] slots  a[10] ld routing
 //      a[11] experts  a[12] rows N of an expert
 // ---- TASK_QKV_APPEND: tokens [a[0], a[1]); p[0] projections f32  p[1] q out  p[2] k cache  p[3] v cache  p[4] cos f32  p[5] sin f32
 //      p[6] q norm  p[7] k norm (bf16 [dim], null: none);  p[2] null: queries only;  a[QA_*] below
+//      QA_WHOLE: the norms span all heads (weights [heads * dim]), nothing is rotated;  queries are multiplied by
+//      1 + QA_TEMP (bits) * ln(floor((position + 1) / QA_EVERY) + 1) where QA_EVERY > 0
 enum { QA_T0 = 0, QA_T1, QA_LDP, QA_QOFF, QA_KOFF, QA_VOFF, QA_HQ, QA_HKV, QA_DIM, QA_DIMP, QA_VDIM, QA_VDIMP, QA_ROT, QA_NORM,
-       QA_EPS, QA_PAGE, QA_LDQ, QA_ROWS, QA_PAIRS, QA_MAPS };
+       QA_EPS, QA_PAGE, QA_LDQ, QA_ROWS, QA_PAIRS, QA_MAPS, QA_WHOLE, QA_TEMP, QA_EVERY };
 // ---- TASK_EXT_ATTENTION: p[0] q [tokens, hq * dimp]  p[1] k cache  p[2] v cache  p[3] out;  a[XA_*] below
 enum { XA_SLOT = 0, XA_HEAD, XA_CHUNK, XA_NCHUNK, XA_HQ, XA_HKV, XA_DIMP, XA_VDIM, XA_VDIMP, XA_PAGE, XA_LDQ, XA_LDO, XA_OCOL,
        XA_SCALE, XA_CAP, XA_SINK, XA_OSCALE, XA_TICKET, XA_SREC, XA_STAGES, XA_SHARED, XA_KEYS, XA_MERGE, XA_WINDOW, XA_KEEP, XA_OUTF32 };
 //      p[4] sinks bf16 [hq] or null; XA_SHARED: values are key columns; XA_KEYS: keys of a tile of
 //      theirs; XA_MERGE: a layer of TASK_ATTN_MERGE follows (its tasks: the same fields, task a[XA_SLOT] of a[XA_CHUNK]);
 //      XA_WINDOW: keys a position sees at most, itself included (0: all)  XA_KEEP: first keys it sees all the same
+//      p[5], p[6] distance bias bf16 [hq] or null: r1 * ln(1 + r2 * distance) comes off the score
 constexpr int kXaRecHead = 4;   // floats in front of a record's columns
 constexpr int kXaCells = 320;   // cache rows of a chunk's key octets kept in shared memory
 // ---- TASK_SHORT_CONV: channels [a[0], a[1]); p[0] in f32  p[1] in bias bf16 or null  p[2] taps bf16 [channels, taps]
@@ -278,6 +290,7 @@ enum { LA_T0 = 0, LA_T1, LA_LDP, LA_QOFF, LA_KVOFF, LA_H, LA_RANK, LA_ROT, LA_DI
 enum { SS_C0 = 0, SS_C1, SS_C, SS_RANK, SS_N, SS_NP, SS_LANES, SS_LDU, SS_LDL, SS_LDG, SS_GOFF, SS_LDO, SS_STATE };
 // ---- TASK_DIFF_COMBINE: task a[0] of a[1]; p[0] maps f32 [tokens, heads * 2 * vdim]  p[1] out;  a[2] heads  a[3] vdim  a[4] ld in  a[5] ld out
 //      a[6] lambda  a[7] factor  a[8] eps (bits)
+// ---- TASK_POLY_NORM: rows [a[0], a[1]), width a[2]; p[0] z f32  p[1] coefficients bf16 [4]  p[2] out (activation type);  a[3] ld z  a[4] ld out  a[5] eps bits
 // ---- TASK_ALLREDUCE:       p[0] inbox base p[1] residual (or null) p[2] out
 //  a[0] c0 a[1] c1 (columns) a[2] world a[3] slot stride (floats) a[4] ld_out a[5] ld_res a[6] N
 //  a[7] allreduce index  a[8] allreduces per iteration  a[9] stride between the two inbox buffers (floats)

@@ -106,7 +106,7 @@ struct Builder {
   void layer_io(const LayerInfo &l, std::vector<int> *ins, std::vector<int> *outs) const {
     auto add = [](std::vector<int> *v, int t) { if (t >= 0) v->push_back(t); };
     switch (l.op) {
-      case MPK_OP_EMBED: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); break;
+      case MPK_OP_EMBED: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); add(ins, norm_tensor(l, 3)); add(ins, norm_tensor(l, 4)); add(outs, norm_tensor(l, 5)); break;
       case MPK_OP_RMSNORM: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); break;
       case MPK_OP_RMSNORM_LINEAR:
         add(ins, l.t[0]); add(ins, l.t[1]); add(ins, l.t[2]); add(outs, l.t[3]); break;
@@ -171,26 +171,28 @@ struct Builder {
       case MPK_OP_MLA_DECODE: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); add(outs, l.t[3]); break;
       case MPK_OP_MLA_REDUCE: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); break;
       case MPK_OP_RESIDUAL_NORM:
-        for (int i = 0; i < 12; ++i) if (i != 4 && i != 5) add(ins, norm_tensor(l, i));
+        for (int i = 0; i < 14; ++i) if (i != 4 && i != 5) add(ins, norm_tensor(l, i));
         if (resnorm_moves(l)) add(outs, resnorm_out(l));
+        add(outs, norm_tensor(l, 12));
         add(outs, l.t[4]);
         break;
       case MPK_OP_QKV_APPEND: add(ins, l.t[0]); for (int i = 4; i < 8; ++i) add(ins, norm_tensor(l, i)); for (int i = 1; i < 4; ++i) add(outs, l.t[i]); break;
       case MPK_OP_ATTN_MERGE: add(ins, l.t[3]); add(outs, l.t[3]); break;
       case MPK_OP_EXT_ATTENTION:
         for (int i = 0; i < 3; ++i) add(ins, l.t[i]);
-        if (l.t.size() > 4) add(ins, l.t[4]);
+        for (int i = 4; i < 7; ++i) add(ins, norm_tensor(l, i));
         add(outs, l.t[3]);
         break;
       case MPK_OP_SHORT_CONV: for (int i = 0; i < 5; ++i) add(ins, l.t[i]); add(outs, l.t[4]); add(outs, l.t[5]); add(outs, norm_tensor(l, 6)); break;
       case MPK_OP_SELECTIVE_SCAN: for (int i = 0; i < 8; ++i) add(ins, l.t[i]); add(outs, l.t[7]); add(outs, l.t[8]); break;
       case MPK_OP_DIFF_COMBINE: add(ins, l.t[0]); add(outs, l.t[1]); break;
+      case MPK_OP_POLY_NORM: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); break;
       case MPK_OP_RGLRU: for (int i = 0; i < 9; ++i) add(ins, l.t[i]); add(outs, l.t[8]); add(outs, l.t[9]); break;
       case MPK_OP_MLSTM: for (int i = 0; i < 6; ++i) add(ins, l.t[i]); for (int i = 4; i < 8; ++i) add(outs, l.t[i]); break;
       case MPK_OP_GLA: for (int i = 0; i < 5; ++i) add(ins, l.t[i]); for (int i = 4; i < 7; ++i) add(outs, l.t[i]); break;
       case MPK_OP_LATENT_APPEND:
         add(ins, l.t[0]); add(ins, l.t[1]); add(ins, l.t[4]); add(ins, l.t[5]); add(outs, l.t[2]); add(outs, l.t[3]); break;
-      case MPK_OP_GROUPED_LINEAR: add(ins, l.t[0]); add(ins, l.t[1]); add(outs, l.t[2]); break;
+      case MPK_OP_GROUPED_LINEAR: add(ins, l.t[0]); add(ins, l.t[1]); add(ins, norm_tensor(l, 3)); add(outs, l.t[2]); break;
       case MPK_OP_LINEAR_FP8_RESIDUAL: for (int i = 0; i < 5; ++i) add(ins, l.t[i]); add(outs, l.t[5]); break;
       default: break;
     }
@@ -224,7 +226,8 @@ struct Builder {
           {MPK_OP_SAMPLING_PARTIAL, 3}, {MPK_OP_SAMPLING_REDUCE, 3}, {MPK_OP_ARGMAX_EXCHANGE, 3},
           {MPK_OP_MOE_TOPK_SOFTMAX, 4}, {MPK_OP_RESIDUAL_NORM, 5}, {MPK_OP_QKV_APPEND, 6}, {MPK_OP_EXT_ATTENTION, 4},
           {MPK_OP_SHORT_CONV, 6}, {MPK_OP_RGLRU, 10}, {MPK_OP_MLSTM, 8}, {MPK_OP_GLA, 7}, {MPK_OP_LATENT_APPEND, 6},
-          {MPK_OP_GROUPED_LINEAR, 3}, {MPK_OP_ATTN_MERGE, 4}, {MPK_OP_SELECTIVE_SCAN, 9}, {MPK_OP_DIFF_COMBINE, 2}};
+          {MPK_OP_GROUPED_LINEAR, 3}, {MPK_OP_ATTN_MERGE, 4}, {MPK_OP_SELECTIVE_SCAN, 9}, {MPK_OP_DIFF_COMBINE, 2},
+          {MPK_OP_POLY_NORM, 3}};
       auto it = need.find(L[i].op);
       if (it == need.end()) return fail(MPK_ERR_UNSUPPORTED, "layer " + std::to_string(i) + ": unknown op");
       if ((int)L[i].t.size() < it->second)
@@ -302,6 +305,8 @@ struct Builder {
     return l.t[1] >= 0 || norm_tensor(l, 7) >= 0 || norm_tensor(l, 8) >= 0 || norm_tensor(l, 9) >= 0;
   }
   static int norm_flags(const LayerInfo &l) { return (l.params[1] ? 2 : 0) | (l.params.size() > 2 && l.params[2] == 1 ? 4 : 0); }
+  // columns of x a residual_norm layer works on
+  int64_t norm_columns(const LayerInfo &l) const { return l.params.size() > 5 && l.params[5] > 0 ? l.params[5] : T[l.t[0]].dim(1); }
   static int norm_factor(const LayerInfo &l) { return l.params.size() > 4 ? bits_of(l.params[4]) : 0x3f800000; }   // (1.0f)
   static bool keeps_logits(const LayerInfo &l) { return l.params.size() > 5 && l.params[5] != 0; }
 
@@ -313,10 +318,11 @@ struct Builder {
       LayerInfo &p = L[i];
       if (p.op != MPK_OP_RESIDUAL_NORM || p.t[4] < 0) continue;
       const int x = p.t[0], y = p.t[1], out = p.t[4], xo = resnorm_out(p), add = norm_tensor(p, 7), row = norm_tensor(p, 8), bias = norm_tensor(p, 6);
-      if (norm_tensor(p, 9) >= 0 || norm_tensor(p, 11) >= 0) continue;   // the sum over experts is formed once, not by every task
+      // the sums over experts or earlier results are formed once, not by every task
+      if (norm_tensor(p, 9) >= 0 || norm_tensor(p, 11) >= 0 || norm_tensor(p, 12) >= 0) continue;
       const bool moves = resnorm_moves(p);
       auto aligned = [&](int t) { return T[t].ld() % 4 == 0 && ((uint64_t)T[t].ptr & 15) == 0; };
-      const int64_t D = T[x].dim(1);
+      const int64_t D = norm_columns(p);
       if (T[out].owner == 0 || D > 4096 || D % 4 || !aligned(x) || (p.t[3] >= 0 && ((uint64_t)T[p.t[3]].ptr & 7)) || p.params.size() < 2) continue;
       if (moves && (T[xo].storage == T[x].storage || !aligned(xo) || T[xo].dtype != MPK_F32 || T[xo].dim(1) != D)) continue;
       if ((y >= 0 && !aligned(y)) || (add >= 0 && (!aligned(add) || T[add].dtype != MPK_F32 || T[add].dim(1) != D))) continue;
@@ -343,6 +349,7 @@ struct Builder {
       c.pro_src = x; c.pro_y = y; c.pro_post = p.t[2]; c.pro_gamma = p.t[3];
       c.pro_bias = bias; c.pro_add = add; c.pro_row = row;
       c.pro_xout = moves ? xo : -1;
+      c.pro_cols = (int)D;
       c.pro_eps = bits_of(p.params[0]); c.pro_flags = norm_flags(p); c.pro_factor = norm_factor(p);
       p.folded = true;
       g->num_folded++;
@@ -610,8 +617,8 @@ struct Builder {
     if (x.dtype != MPK_BF16 && l.prologue != PRO_RESNORM) return fail(MPK_ERR_UNSUPPORTED, "linear input must be bf16: " + w.name);
     if (l.op == MPK_OP_LINEAR && !l.params.empty() && l.params[0] != 0) {
       epi = activation_epilogue(l.params[0]);
-      if (g->hybrid != HYB_BF16 || epi == EPI_STORE || y.dtype != (epi == EPI_SOFTCAP ? MPK_F32 : MPK_BF16) || (epi == EPI_SOFTCAP && l.params.size() < 2))
-        return fail(MPK_ERR_UNSUPPORTED, "linear activation: in hybrid graphs, bf16 output (soft cap: float32): " + w.name);
+      if (g->hybrid != HYB_BF16 || epi == EPI_STORE || y.dtype != (capped(epi) ? MPK_F32 : MPK_BF16) || (capped(epi) && l.params.size() < 2))
+        return fail(MPK_ERR_UNSUPPORTED, "linear activation: in hybrid graphs, bf16 output (soft cap, scale: float32): " + w.name);
       gated = epi == EPI_GATED_SILU || epi == EPI_GATED_GELU;
       if (gated && N % 4) return fail(MPK_ERR_INVALID, "gated linear: rows come as two gate rows, two up rows: " + w.name);
     } else if (y.dtype == MPK_F32) {
@@ -710,7 +717,7 @@ struct Builder {
         d.a[L_PRO] = l.prologue;
         d.a[L_EPI] = epi;
         d.a[L_EPS] = l.prologue == PRO_RESNORM ? l.pro_eps : float_bits(1e-6f);
-        d.a[L_GROUPS] = l.prologue == PRO_RESNORM ? (int)x.dim(1) : l.pro_groups;
+        d.a[L_GROUPS] = l.prologue == PRO_RESNORM ? l.pro_cols : l.pro_groups;
         d.a[L_KT] = KT;
         d.a[L_KC] = KC;
         d.a[L_ROWS] = R;
@@ -719,7 +726,7 @@ struct Builder {
         d.a[L_ARIDX] = std::max(l.ar_index, 0);
         d.a[L_NAR] = g->num_allreduce;
         d.a[L_PARSTRIDE] = (int)g->inbox_floats_per_buffer;
-        if (epi == EPI_SOFTCAP) d.a[L_CAP] = bits_of(l.params[1]);
+        if (capped(epi)) d.a[L_CAP] = bits_of(l.params[1]);
         if (epi == EPI_BIAS_F32) put_wide(&d, LR_BIAS, bias);
         if (l.prologue == PRO_RESNORM) {
           d.a[LR_POST] = l.pro_factor;
@@ -1108,17 +1115,20 @@ struct Builder {
   }
 
   // ---- hybrid graphs: recurrent layers, extended attention, float32 residual stream --------------------------
-  static bool hybrid_op(int op) { return op >= MPK_OP_RESIDUAL_NORM && op <= MPK_OP_DIFF_COMBINE; }
+  static bool hybrid_op(int op) { return op >= MPK_OP_RESIDUAL_NORM && op <= MPK_OP_POLY_NORM; }
   static bool expert_op(int op) { return op == MPK_OP_MOE_TOPK_SIGMOID || op == MPK_OP_MOE_TOPK_SOFTMAX || op == MPK_OP_MOE_W13_LINEAR || op == MPK_OP_MOE_W2_LINEAR; }
   static int activation_epilogue(int64_t act) {
     switch (act) {
       case MPK_ACT_RELU2: return EPI_RELU2;
       case MPK_ACT_SOFTCAP: return EPI_SOFTCAP;
+      case MPK_ACT_SCALE: return EPI_SCALE_F32;
       case MPK_ACT_GATED_SILU: return EPI_GATED_SILU;
       case MPK_ACT_GATED_GELU_TANH: return EPI_GATED_GELU;
       default: return EPI_STORE;
     }
   }
+  // Epilogues with a number of their own and a float32 output.
+  static bool capped(int epi) { return epi == EPI_SOFTCAP || epi == EPI_SCALE_F32; }
   // A tensor's address (0: absent) into two of a descriptor's integers.
   void put_wide(TaskDesc *d, int i, int tensor) const {
     const uint64_t p = tensor >= 0 ? (uint64_t)T[tensor].ptr : 0;
@@ -1137,7 +1147,7 @@ struct Builder {
     for (size_t i = 0; i < L.size(); ++i) {
       const LayerInfo &l = L[i];
       const int act_out = l.op == MPK_OP_RESIDUAL_NORM || l.op == MPK_OP_EXT_ATTENTION || l.op == MPK_OP_RGLRU || l.op == MPK_OP_MLSTM ||
-                                  l.op == MPK_OP_GLA || l.op == MPK_OP_SELECTIVE_SCAN || l.op == MPK_OP_DIFF_COMBINE
+                                  l.op == MPK_OP_GLA || l.op == MPK_OP_SELECTIVE_SCAN || l.op == MPK_OP_DIFF_COMBINE || l.op == MPK_OP_POLY_NORM
                               ? (l.op == MPK_OP_RESIDUAL_NORM ? l.t[4] : l.op == MPK_OP_EXT_ATTENTION ? l.t[0] : l.t.back()) : -1;   // tensor of the graph's activation type
       if (act_out >= 0 && T[act_out].dtype == MPK_F32) f32 = true;
       if (hybrid_op(l.op) || l.op == MPK_OP_EMBED || l.op == MPK_OP_ARGMAX_PARTIAL || l.op == MPK_OP_ARGMAX_REDUCE ||
@@ -1190,7 +1200,7 @@ struct Builder {
   int64_t hybrid_smem(const LayerInfo &l) const {
     const int64_t mbr = cfg.max_num_batched_requests;
     switch (l.op) {
-      case MPK_OP_RESIDUAL_NORM: return T[l.t[0]].dim(1) * 4 + 16;
+      case MPK_OP_RESIDUAL_NORM: return norm_columns(l) * 4 + 16;
       case MPK_OP_EXT_ATTENTION: {
         if (g->hybrid == HYB_F32) return 8 * T[l.t[1]].dim(3) * 4;
         if (T[l.t[1]].storage == T[l.t[2]].storage) return latent_plan(l).bytes;
@@ -1243,7 +1253,7 @@ struct Builder {
     const int act = l.params.empty() ? 0 : (int)l.params[0];
     const bool gated = act == MPK_ACT_GATED_SILU || act == MPK_ACT_GATED_GELU_TANH;
     const int cols = gated ? N / 2 : N;
-    if (x.dim(1) != K || y.dim(1) < cols || (gated && N % 4) || act < 0 || act > MPK_ACT_GATED_GELU_TANH || (act == MPK_ACT_SOFTCAP && l.params.size() < 2))
+    if (x.dim(1) != K || y.dim(1) < cols || (gated && N % 4) || act < 0 || act > MPK_ACT_SCALE || ((act == MPK_ACT_SOFTCAP || act == MPK_ACT_SCALE) && l.params.size() < 2))
       return fail(MPK_ERR_INVALID, "32-bit linear: shapes or activation of " + w.name);
     const int bias = norm_tensor(l, 3);
     if (bias >= 0 && (act || T[bias].dtype != MPK_BF16 || T[bias].dim(0) < N)) return fail(MPK_ERR_INVALID, "linear bias: bf16 [rows], no activation: " + w.name);
@@ -1299,6 +1309,10 @@ struct Builder {
       return fail(MPK_ERR_UNSUPPORTED, "grouped linear: dense bf16 weight, input and output of the graph's activation type: " + w.name);
     if (xs < K || yc < 0 || ys < N || (G - 1) * xs + K > x.dim(1) || yc + (G - 1) * ys + N > y.dim(1))
       return fail(MPK_ERR_INVALID, "grouped linear: columns outside the input or output: " + w.name);
+    const int gate = norm_tensor(l, 3);
+    const int64_t gc = l.params.size() > 3 ? l.params[3] : 0, gs = l.params.size() > 4 ? l.params[4] : N;
+    if (gate >= 0 && (T[gate].dtype != MPK_F32 || y.dtype != act_dtype() || gc < 0 || gs < N || gc + (G - 1) * gs + N > T[gate].dim(1)))
+      return fail(MPK_ERR_INVALID, "grouped linear: float32 gate columns inside their tensor, output of the graph's activation type: " + w.name);
     const bool f32 = g->hybrid == HYB_F32;
     if (!f32 && (K % 16 || xs % 8 || ((uint64_t)x.ptr & 15) || ((uint64_t)w.ptr & 15) || x.ld() % 8))
       return fail(MPK_ERR_UNSUPPORTED, "grouped linear: K a multiple of 16, input columns on 16-byte boundaries: " + w.name);
@@ -1330,12 +1344,15 @@ struct Builder {
         d.p[0] = (uint64_t)w.ptr + (uint64_t)grp * N * K * 2;
         d.p[1] = (uint64_t)x.ptr + (uint64_t)grp * xs * esz_x;
         d.p[2] = (uint64_t)y.ptr + (uint64_t)(yc + grp * ys) * esz_y;
+        const uint64_t gp = gate >= 0 ? (uint64_t)T[gate].ptr + (uint64_t)(gc + grp * gs) * 4 : 0;
         if (f32) {
+          d.p[4] = gp; d.a[9] = gate >= 0 ? (int)T[gate].ld() : 0;
           d.a[0] = n0; d.a[1] = n1; d.a[2] = K; d.a[3] = K; d.a[4] = (int)x.ld(); d.a[5] = (int)y.ld(); d.a[7] = linear_f32_tokens(K);
         } else {
           if (grp == last) d.flags |= TF_SAME_X_AS_PREV;
           d.a[L_N0] = n0; d.a[L_N1] = n1; d.a[L_K] = K; d.a[L_LDW] = K; d.a[L_LDX] = (int)x.ld(); d.a[L_LDO] = (int)y.ld();
-          d.a[L_PRO] = PRO_PLAIN; d.a[L_EPI] = y.dtype == MPK_F32 ? EPI_STORE_F32 : EPI_STORE; d.a[L_GROUPS] = 1;
+          d.a[L_PRO] = PRO_PLAIN; d.a[L_EPI] = gate >= 0 ? EPI_GATE_SIGMOID : y.dtype == MPK_F32 ? EPI_STORE_F32 : EPI_STORE; d.a[L_GROUPS] = 1;
+          d.p[3] = gp; d.a[L_LDR] = gate >= 0 ? (int)T[gate].ld() : 0;
           d.a[L_KT] = K; d.a[L_KC] = KC; d.a[L_ROWS] = kChunkRows; d.a[L_N] = N;
           if (tc) {
             d.flags |= TF_TC;
@@ -1357,20 +1374,22 @@ struct Builder {
 
   int emit_latent_append(int li, int ex) {
     const LayerInfo &l = L[li];
-    const TensorInfo &pr = T[l.t[0]], &nw = T[l.t[1]], &q = T[l.t[2]], &kc = T[l.t[3]], &cs = T[l.t[4]], &sn = T[l.t[5]];
     if (l.params.size() < 6) return fail(MPK_ERR_INVALID, "latent_append needs 6 parameters");
     const int H = (int)l.params[0], rank = (int)l.params[1], rdim = (int)l.params[2];
+    for (int i : {2, 4, 5})   // (nothing to rotate: they stand for themselves)
+      if (l.t[i] < 0 && rdim) return fail(MPK_ERR_INVALID, "latent_append: q and tables are absent, but there is a rotated part");
+    const TensorInfo &pr = T[l.t[0]], &nw = T[l.t[1]], &kc = T[l.t[3]], &q = T[l.t[l.t[2] >= 0 ? 2 : 3]], &cs = T[l.t[l.t[4] >= 0 ? 4 : 0]], &sn = T[l.t[l.t[5] >= 0 ? 5 : 0]];
     if (!batch_meta_given()) return fail(MPK_ERR_INVALID, "latent_append needs the batch meta tensors");
     if (pr.dtype != MPK_F32 || nw.dtype != MPK_BF16 || q.dtype != act_dtype() || kc.dtype != act_dtype() || cs.dtype != MPK_F32 || sn.dtype != MPK_F32)
       return fail(MPK_ERR_INVALID, "latent_append: float32 projections and tables, bf16 norm weight, q and cache of the graph's activation type");
     if (H < 1 || rank < 1 || rdim < 0 || rdim % 2 || nw.dim(0) < rank || kc.dims.size() != 4 || kc.dim(1) != cfg.page_size || kc.dim(2) != 1 ||
-        kc.dim(3) < rank + rdim || kc.dim(3) % 8 || q.dim(1) != H * kc.dim(3))
+        kc.dim(3) < rank + rdim || kc.dim(3) % 8 || (rdim > 0 && q.dim(1) != H * kc.dim(3)))
       return fail(MPK_ERR_INVALID, "latent_append: cache [pages, page, 1, latent + rotated size rounded up to 8], q [tokens, heads x that]");
     if (l.params[3] < 0 || l.params[4] < 0 || l.params[3] + (int64_t)H * rdim > pr.dim(1) || l.params[4] + rank + rdim > pr.dim(1))
       return fail(MPK_ERR_INVALID, "latent_append: columns outside the projections");
     if (rdim > 0 && (cs.dims.size() != 2 || cs.dim(1) != rdim / 2 || sn.dim(1) != rdim / 2 || cs.dim(0) != sn.dim(0)))
       return fail(MPK_ERR_INVALID, "latent_append: cos / sin tables [positions, rotated dims / 2]");
-    const int nt = std::max(1, std::min(W, (nb_max * (H + 1) + 7) / 8));
+    const int nt = std::max(1, std::min(W, (nb_max * (rdim > 0 ? H + 1 : 1) + 7) / 8));
     for (int i = 0; i < nt; ++i) {
       TaskDesc d = blank(TASK_LATENT_APPEND, li);
       d.p[0] = (uint64_t)pr.ptr; d.p[1] = (uint64_t)nw.ptr; d.p[2] = (uint64_t)q.ptr; d.p[3] = (uint64_t)kc.ptr;
@@ -1427,7 +1446,7 @@ struct Builder {
     const LayerInfo &l = L[li];
     const TensorInfo &x = T[l.t[0]];
     auto opt = [&](int i) { return l.t[i] >= 0 ? (uint64_t)T[l.t[i]].ptr : 0; };
-    const int D = (int)x.dim(1);
+    const int D = (int)norm_columns(l);
     if (l.params.size() < 2 || x.dtype != MPK_F32 || x.dims.size() != 2) return fail(MPK_ERR_INVALID, "residual_norm: x must be float32 [tokens, width]");
     if (l.t[1] >= 0 && (T[l.t[1]].dtype != MPK_F32 || T[l.t[1]].dim(1) != D)) return fail(MPK_ERR_INVALID, "residual_norm: y must be float32 of x's width");
     for (int i = 2; i < 4; ++i)
@@ -1445,8 +1464,13 @@ struct Builder {
     if (l.t[2] >= 0 && (gate >= 0 || (norm_flags(l) & 4) || (l.t[1] < 0 && exps < 0)))
       return fail(MPK_ERR_UNSUPPORTED, "residual_norm: a norm of y (or of the experts' sum) goes with RMS norms and without a gate");
     if (l.t[4] >= 0 && (T[l.t[4]].dtype != act_dtype() || T[l.t[4]].dim(1) < D)) return fail(MPK_ERR_INVALID, "residual_norm: output type or width");
+    const int results = norm_tensor(l, 12), rw = norm_tensor(l, 13), terms = rw >= 0 ? (int)T[rw].dim(0) : 0;
+    if ((results >= 0) != (rw >= 0) || (results >= 0 && (T[results].dtype != MPK_F32 || T[results].dims.size() != 3 || T[results].dim(2) != D || T[results].strides[1] != D ||
+                                                         T[results].dim(1) < cfg.max_num_batched_tokens || T[rw].dtype != MPK_BF16 || terms < 2 || terms > T[results].dim(0) || l.t[1] < 0)))
+      return fail(MPK_ERR_INVALID, "residual_norm: results float32 [results, tokens, width], at least two of them with bf16 weights, and a y");
+    if (D > x.dim(1) || (D < x.dim(1) && resnorm_moves(l))) return fail(MPK_ERR_INVALID, "residual_norm: leading columns of x, with nothing added");
     const TensorInfo &xo = T[resnorm_out(l)];
-    if (xo.dtype != MPK_F32 || xo.dim(1) != D) return fail(MPK_ERR_INVALID, "residual_norm: the new stream must be float32 of x's width");
+    if (resnorm_moves(l) && (xo.dtype != MPK_F32 || xo.dim(1) != D)) return fail(MPK_ERR_INVALID, "residual_norm: the new stream must be float32 of x's width");
     const int rows = (int)std::min<int64_t>(x.dim(0), cfg.max_num_batched_tokens), nt = std::min(rows, W);
     for (int i = 0; i < nt; ++i) {
       TaskDesc d = blank(TASK_RESIDUAL_NORM, li);
@@ -1466,6 +1490,9 @@ struct Builder {
       d.a[RN_SLOTS] = exps >= 0 ? (int)T[exps].dim(1) : 0;
       d.a[RN_LDEW] = ew >= 0 ? (int)T[ew].ld() : 0;
       d.a[RN_POST] = norm_factor(l);
+      if (results >= 0) {
+        d.p[6] = (uint64_t)T[results].ptr; d.p[7] = (uint64_t)T[rw].ptr; d.a[RN_TERMS] = terms; d.a[RN_HSTRIDE] = (int)T[results].strides[0];
+      }
       put((i + rot) % W, d, ex);
     }
     return MPK_OK;
@@ -1475,18 +1502,24 @@ struct Builder {
     const LayerInfo &l = L[li];
     const bool caches = l.t[2] >= 0;   // else queries only
     if (caches != (l.t[3] >= 0)) return fail(MPK_ERR_INVALID, "qkv_append: both caches or none");
-    const TensorInfo &pr = T[l.t[0]], &q = T[l.t[1]], &kc = T[l.t[caches ? 2 : 1]], &vc = T[l.t[caches ? 3 : 1]], &cs = T[l.t[4]], &sn = T[l.t[5]];
+    const TensorInfo &pr = T[l.t[0]], &q = T[l.t[1]], &kc = T[l.t[caches ? 2 : 1]], &vc = T[l.t[caches ? 3 : 1]];
     if (l.params.size() < 10) return fail(MPK_ERR_INVALID, "qkv_append needs 10 parameters");
     const int hq = (int)l.params[0], hkv = (int)l.params[1], dim = (int)l.params[2], vdim = (int)l.params[3], rdim = (int)l.params[7];
     const int pairs = l.params.size() > 10 ? (int)l.params[10] : 0, maps = l.params.size() > 11 ? (int)l.params[11] : 1;
+    if ((l.t[4] < 0 || l.t[5] < 0) && rdim) return fail(MPK_ERR_INVALID, "qkv_append: no tables, but rotated dimensions");
+    const TensorInfo &cs = T[l.t[l.t[4] >= 0 ? 4 : 0]], &sn = T[l.t[l.t[5] >= 0 ? 5 : 0]];   // (nothing to rotate: absent)
+    const bool whole = l.params.size() > 12 && l.params[12];
+    const int temp = l.params.size() > 13 ? bits_of(l.params[13]) : 0, every = l.params.size() > 14 ? (int)l.params[14] : 0;
     if (!batch_meta_given()) return fail(MPK_ERR_INVALID, "qkv_append needs the batch meta tensors");
+    if ((whole && (rdim || maps != 1 || l.params[8] || norm_tensor(l, 6) < 0 || (caches && norm_tensor(l, 7) < 0))) || (!whole && every) || every < 0)
+      return fail(MPK_ERR_UNSUPPORTED, "qkv_append: norms over all heads go with q and k weights and without rotation, the query temperature with such norms");
     if (pr.dtype != MPK_F32 || q.dtype != act_dtype() || (caches && (kc.dtype != act_dtype() || vc.dtype != act_dtype())) || cs.dtype != MPK_F32 || sn.dtype != MPK_F32)
       return fail(MPK_ERR_INVALID, "qkv_append: float32 projections and tables, q and caches of the graph's activation type");
     if (hq < 1 || hkv < 1 || hq % hkv || dim < 1 || vdim < 1 || rdim < 0 || rdim > dim || rdim % 2 || maps < 1 || maps > 2)
       return fail(MPK_ERR_INVALID, "qkv_append: head counts or sizes");
     const int dimp = caches && kc.dims.size() == 4 ? (int)kc.dim(3) : (int)q.dim(1) / (hq * maps);
     for (int i : {6, 7})
-      if (norm_tensor(l, i) >= 0 && (T[l.t[i]].dtype != MPK_BF16 || T[l.t[i]].dim(0) < dim || l.params[8])) return fail(MPK_ERR_INVALID, "qkv_append: bf16 norm weights [dim], no unit norm beside them");
+      if (norm_tensor(l, i) >= 0 && (T[l.t[i]].dtype != MPK_BF16 || T[l.t[i]].dim(0) < (whole ? (int64_t)dim * (i == 6 ? hq : hkv) : dim) || l.params[8])) return fail(MPK_ERR_INVALID, "qkv_append: bf16 norm weights [dim], no unit norm beside them");
     if (!caches) {
       if (dimp < maps * dim || dimp % 8 || q.dim(1) != (int64_t)hq * maps * dimp || l.params[4] + (int64_t)hq * maps * dim > pr.dim(1)) return fail(MPK_ERR_INVALID, "qkv_append: q [tokens, heads x head size rounded up to 8], columns inside the projections");
     } else if (kc.dims.size() != 4 || vc.dims.size() != 4 || kc.dim(1) != cfg.page_size || vc.dim(1) != cfg.page_size || kc.dim(2) != hkv ||
@@ -1496,13 +1529,13 @@ struct Builder {
       return fail(MPK_ERR_INVALID, "qkv_append: columns outside the projections");
     if (rdim > 0 && (cs.dims.size() != 2 || cs.dim(1) != rdim / 2 || sn.dim(1) != rdim / 2 || cs.dim(0) != sn.dim(0)))
       return fail(MPK_ERR_INVALID, "qkv_append: cos / sin tables [positions, rotated dims / 2]");
-    const int nt = std::max(1, std::min(W, (nb_max * (hq + (caches ? hkv : 0)) * maps + 7) / 8));
+    const int nt = std::max(1, std::min(W, whole ? nb_max * (caches ? 2 : 1) : (nb_max * (hq + (caches ? hkv : 0)) * maps + 7) / 8));
     for (int i = 0; i < nt; ++i) {
       TaskDesc d = blank(TASK_QKV_APPEND, li);
       d.p[0] = (uint64_t)pr.ptr; d.p[1] = (uint64_t)q.ptr; d.p[2] = caches ? (uint64_t)kc.ptr : 0; d.p[3] = caches ? (uint64_t)vc.ptr : 0;
       d.p[4] = (uint64_t)cs.ptr; d.p[5] = (uint64_t)sn.ptr;
       for (int k : {6, 7}) d.p[k] = norm_tensor(l, k) >= 0 ? (uint64_t)T[l.t[k]].ptr : 0;
-      d.a[QA_PAIRS] = pairs; d.a[QA_MAPS] = maps;
+      d.a[QA_PAIRS] = pairs; d.a[QA_MAPS] = maps; d.a[QA_WHOLE] = whole ? 1 : 0; d.a[QA_TEMP] = temp; d.a[QA_EVERY] = every;
       d.a[QA_T0] = i; d.a[QA_T1] = nt; d.a[QA_LDP] = (int)pr.ld();
       d.a[QA_QOFF] = (int)l.params[4]; d.a[QA_KOFF] = (int)l.params[5]; d.a[QA_VOFF] = (int)l.params[6];
       d.a[QA_HQ] = hq; d.a[QA_HKV] = hkv; d.a[QA_DIM] = dim; d.a[QA_DIMP] = dimp; d.a[QA_VDIM] = vdim; d.a[QA_VDIMP] = caches ? (int)vc.dim(3) : 0;
@@ -1528,7 +1561,11 @@ struct Builder {
     const int64_t window = l.params.size() > 9 ? l.params[9] : 0, keep = l.params.size() > 10 ? l.params[10] : 0;
     if (window < 0 || keep < 0 || window > (1 << 30) || keep > (1 << 30)) return fail(MPK_ERR_INVALID, "ext_attention: window or kept positions");
     const bool shared = kc.storage == vc.storage, bf16 = g->hybrid == HYB_BF16;
-    if (shared && bf16 && (window > 0 || o.dtype == MPK_F32)) return fail(MPK_ERR_UNSUPPORTED, "ext_attention: no window and no float32 output with shared keys and values");
+    const int r1 = norm_tensor(l, 5), r2 = norm_tensor(l, 6);
+    if ((r1 >= 0) != (r2 >= 0) || (r1 >= 0 && (T[r1].dtype != MPK_BF16 || T[r2].dtype != MPK_BF16 || T[r1].dim(0) < hq || T[r2].dim(0) < hq)))
+      return fail(MPK_ERR_INVALID, "ext_attention: distance bias of two bf16 tensors [heads]");
+    if (shared && (keep > 0 || r1 >= 0 || (bf16 && o.dtype == MPK_F32)))
+      return fail(MPK_ERR_UNSUPPORTED, "ext_attention: no kept positions, distance bias or float32 output with shared keys and values");
     if (shared && bf16 && (hkv != 1 || vdim % 8 || (ocol | o.ld()) % 2)) return fail(MPK_ERR_UNSUPPORTED, "ext_attention: shared keys and values have one kv head and a value size of whole 16-byte pieces");
     if (bf16 && !shared ? std::max(kc.dim(3), vc.dim(3)) > 256 : kc.dim(3) > 1024 || vdim > 512)
       return fail(MPK_ERR_UNSUPPORTED, "ext_attention: head sizes up to 256 (32-bit graphs and shared keys and values: keys up to 1024, values up to 512)");
@@ -1552,6 +1589,7 @@ struct Builder {
           TaskDesc d = blank(TASK_EXT_ATTENTION, li);
           for (int i = 0; i < 4; ++i) d.p[i] = (uint64_t)T[l.t[i]].ptr;
           d.p[4] = sinks >= 0 ? (uint64_t)T[sinks].ptr : 0;
+          d.p[5] = r1 >= 0 ? (uint64_t)T[r1].ptr : 0; d.p[6] = r2 >= 0 ? (uint64_t)T[r2].ptr : 0;
           d.a[XA_WINDOW] = (int)window; d.a[XA_KEEP] = (int)keep; d.a[XA_OUTF32] = o.dtype == MPK_F32 ? 1 : 0;
           d.a[XA_SHARED] = shared && bf16 ? 1 : 0; d.a[XA_KEYS] = lp.keys; d.a[XA_MERGE] = merge ? 1 : 0;
           d.a[XA_SLOT] = s; d.a[XA_HEAD] = h; d.a[XA_CHUNK] = ch; d.a[XA_NCHUNK] = NC; d.a[XA_HQ] = hq; d.a[XA_HKV] = hkv;
@@ -1660,6 +1698,22 @@ struct Builder {
     return MPK_OK;
   }
 
+  int emit_poly_norm(int li, int ex) {
+    const LayerInfo &l = L[li];
+    const TensorInfo &z = T[l.t[0]], &co = T[l.t[1]], &o = T[l.t[2]];
+    const int N = (int)z.dim(1), rows = (int)std::min<int64_t>(z.dim(0), cfg.max_num_batched_tokens), nt = std::min(rows, W);
+    if (l.params.empty() || z.dtype != MPK_F32 || z.dims.size() != 2 || co.dtype != MPK_BF16 || co.dim(0) != 4 || o.dtype != act_dtype() || o.dim(1) < N || o.dim(0) < rows)
+      return fail(MPK_ERR_INVALID, "poly_norm: float32 values [tokens, n], four bf16 coefficients, output [tokens, >= n] of the activation type");
+    for (int i = 0; i < nt; ++i) {
+      TaskDesc d = blank(TASK_POLY_NORM, li);
+      for (int k = 0; k < 3; ++k) d.p[k] = (uint64_t)T[l.t[k]].ptr;
+      d.a[0] = (int)((int64_t)rows * i / nt); d.a[1] = (int)((int64_t)rows * (i + 1) / nt); d.a[2] = N; d.a[3] = (int)z.ld(); d.a[4] = (int)o.ld();
+      d.a[5] = bits_of(l.params[0]);
+      put((i + rot) % W, d, ex);
+    }
+    return MPK_OK;
+  }
+
   int emit_rglru(int li, int ex) {
     const LayerInfo &l = L[li];
     const TensorInfo &u = T[l.t[0]], &pr = T[l.t[1]], &ra = T[l.t[3]], &st = T[l.t[8]], &o = T[l.t[9]];
@@ -1758,6 +1812,7 @@ struct Builder {
       case MPK_OP_RGLRU: return emit_rglru(li, ex);
       case MPK_OP_SELECTIVE_SCAN: return emit_selective_scan(li, ex);
       case MPK_OP_DIFF_COMBINE: return emit_diff_combine(li, ex);
+      case MPK_OP_POLY_NORM: return emit_poly_norm(li, ex);
       case MPK_OP_MLSTM: return emit_mlstm(li, ex);
       case MPK_OP_GLA: return emit_gla(li, ex);
       case MPK_OP_LATENT_APPEND: return emit_latent_append(li, ex);
@@ -1915,8 +1970,29 @@ struct Builder {
         if (g->hybrid) {
           // the table may be wider than the stream (padded to the projections' k granularity)
           if (y.dtype != MPK_F32 || tab.dtype != MPK_BF16 || tab.dim(1) < y.dim(1)) return fail(MPK_ERR_INVALID, "embed in a hybrid graph: bf16 table, float32 output");
-          emit_token_rows(TASK_EMBED_F32, li, ex, (uint64_t)T[l.t[0]].ptr, (uint64_t)tab.ptr, (uint64_t)y.ptr,
-                          (int)y.dim(1), (int)tab.ld(), (int)y.ld(), (int)tab.dim(0), l.params.size() > 1 ? bits_of(l.params[1]) : float_bits(1.0f), mbt);
+          const int pairs = norm_tensor(l, 3), freq = norm_tensor(l, 4), copy = norm_tensor(l, 5);
+          if (pairs >= 0 && (T[pairs].dtype != MPK_BF16 || T[pairs].dims.size() != 2 || T[pairs].dim(0) < 2 || T[pairs].dim(1) < y.dim(1) || l.params.size() < 4))
+            return fail(MPK_ERR_INVALID, "embed: bigram table bf16 [buckets + 1, width], two multipliers");
+          if (pairs >= 0 && !cfg.dry_run && !cfg.tokens) return fail(MPK_ERR_INVALID, "embed: bigrams need the token table");
+          if (freq >= 0 && (T[freq].dtype != MPK_I64 || T[freq].dim(0) < (y.dim(1) + 1) / 2)) return fail(MPK_ERR_INVALID, "embed: position frequencies int64 [(width + 1) / 2]");
+          if (copy >= 0 && (T[copy].dtype != MPK_F32 || T[copy].dims.size() < 2 || T[copy].dims.back() < y.dim(1) || T[copy].dim((int)T[copy].dims.size() - 2) < mbt))
+            return fail(MPK_ERR_INVALID, "embed: copy of the output float32 [.., tokens, width]");
+          if ((pairs >= 0 || freq >= 0) && !batch_meta_given()) return fail(MPK_ERR_INVALID, "embed: bigrams and positions need the batch meta tensors");
+          const int nt = std::min(mbt, W);
+          for (int i = 0; i < nt; ++i) {
+            TaskDesc d = blank(TASK_EMBED_F32, li);
+            for (int k = 0; k < 6; ++k) d.p[k] = norm_tensor(l, k) >= 0 ? (uint64_t)T[l.t[k]].ptr : 0;
+            d.a[E_T0] = (int)((int64_t)mbt * i / nt); d.a[E_T1] = (int)((int64_t)mbt * (i + 1) / nt);
+            d.a[E_WIDTH] = (int)y.dim(1); d.a[E_LDI] = (int)tab.ld(); d.a[E_LDO] = (int)y.ld(); d.a[E_AUX] = (int)tab.dim(0);
+            d.a[E_LDI2] = l.params.size() > 1 ? bits_of(l.params[1]) : float_bits(1.0f);
+            d.a[E_LDC] = copy >= 0 ? (int)T[copy].ld() : 0;
+            if (pairs >= 0) {
+              d.a[E_LDB] = (int)T[pairs].ld(); d.a[E_BUCKETS] = (int)T[pairs].dim(0) - 1;
+              std::memcpy(&d.a[E_PREV], &l.params[2], 8);
+              std::memcpy(&d.a[E_CUR], &l.params[3], 8);
+            }
+            put((i + rot) % W, d, ex);
+          }
           return MPK_OK;
         }
         if (tab.dim(1) % 8 != 0) return fail(MPK_ERR_UNSUPPORTED, "embedding width must be a multiple of 8");
@@ -2352,7 +2428,7 @@ std::string dump_task_graph(const CompiledGraph &g, const std::vector<TensorInfo
                                 "quantize_fp8", "moe_routing", "moe_gemm", "moe_silu_mul", "moe_mul_sum_add",
                                 "mla_append", "mla_decode", "mla_reduce", "sampling_partial", "sampling_reduce", "argmax_exchange", "ar_push",
                                 "embed_f32", "residual_norm", "linear_f32", "qkv_append", "ext_attention", "short_conv", "rglru", "mlstm",
-                                "gla", "latent_append", "moe_gemm_f32", "attn_merge", "selective_scan", "diff_combine"};
+                                "gla", "latent_append", "moe_gemm_f32", "attn_merge", "selective_scan", "diff_combine", "poly_norm"};
   std::ostringstream os;
   os << "{\"num_workers\": " << g.num_workers << ", \"num_tasks\": " << g.tasks.size()
      << ", \"num_events\": " << g.num_events << ", \"num_layers\": " << layers.size()

@@ -317,10 +317,26 @@ class PersistentKernel:
         return N.check(self._h, N.lib.mpk_add_layer(self._h, op, arr, n, grid, pr, len(params)))
 
     def embed_layer(self, input: DTensor, weight: DTensor, output: DTensor, grid_dim: tuple, block_dim: tuple,
-                    input_source: int = 0, factor: Optional[float] = None):
-        """`factor` (hybrid graphs) multiplies the rows."""
-        self._layer(N.OP_EMBED, [input, weight, output], grid_dim,
-                    [input_source] if factor is None else [input_source, self._bits(factor)])
+                    input_source: int = 0, factor: Optional[float] = None, bigram: Optional[Tuple[DTensor, int, int]] = None,
+                    positions: Optional[DTensor] = None, copy: Optional[DTensor] = None):
+        """Hybrid graphs: `factor` multiplies the rows; `bigram` = (table [buckets + 1, width], multiplier of the previous id, multiplier of
+        the id) adds row (previous id * m_prev + id * m_cur) mod buckets, for a sequence's first token the last row; `positions` (int64,
+        `position_frequencies`) adds sines and cosines of the position in turn; `copy` (float32 [.., tokens, width]) receives the output as well."""
+        params = [input_source] if factor is None else [input_source, self._bits(factor)]
+        if bigram is None and positions is None and copy is None:
+            return self._layer(N.OP_EMBED, [input, weight, output], grid_dim, params)
+        table, m_prev, m_cur = bigram or (None, 0, 0)
+        if table is not None and not self.dry_run:
+            tokens = self.meta_tensors.get("tokens")   # the previous id of a portion's first token is read from it
+            if tokens is None or tuple(tokens.shape)[1] != self.max_seq_length or tokens.shape[0] < (self.max_num_batched_requests if self.mode == "online_notoken" else 1):
+                raise ValueError("bigrams need meta_tensors['tokens'] [requests, max_seq_length]")
+        self._layer(N.OP_EMBED, [input, weight, output, table, positions, copy], grid_dim,
+                    [input_source, self._bits(1.0 if factor is None else factor), int(m_prev), int(m_cur)])
+
+    @staticmethod
+    def position_frequencies(width: int, base: float = 10000.0) -> torch.Tensor:
+        """int64 [(width + 1) / 2]: base^(-2 i / width) radians per position, as turns in units of 2^-64."""
+        return torch.tensor([round(base ** (-2.0 * i / width) / (2.0 * math.pi) * 2 ** 64) for i in range((width + 1) // 2)], dtype=torch.int64)
 
     def rmsnorm_layer(self, input: DTensor, weight: DTensor, output: DTensor, grid_dim: tuple, block_dim: tuple):
         assert input.num_dims == 2 and output.num_dims == 2
@@ -332,16 +348,18 @@ class PersistentKernel:
         self._layer(N.OP_RMSNORM_LINEAR, [input, weight_norm, weight_linear, output], grid_dim)
 
     # mpk_activation of include/mpk_b200.h
-    LINEAR_ACTIVATIONS = {None: 0, "relu2": 1, "softcap": 2, "gated_silu": 3, "gated_gelu_tanh": 4}
+    LINEAR_ACTIVATIONS = {None: 0, "relu2": 1, "softcap": 2, "gated_silu": 3, "gated_gelu_tanh": 4, "scale": 5}
 
     def linear_layer(self, input: DTensor, weight: DTensor, output: DTensor, grid_dim: tuple, block_dim: tuple,
-                     activation: str = None, softcap: float = 0.0, bias: Optional[DTensor] = None):
+                     activation: str = None, softcap: float = 0.0, bias: Optional[DTensor] = None, scale: float = 1.0):
         """`activation` (hybrid graphs) is applied to the fp32 accumulator before the store: squared relu, softcap * tanh(y /
-        softcap), or a gated form act(gate) * up over weight rows from `interleave_gated`, which has half as many outputs.
+        softcap), scale * y, or a gated form act(gate) * up over weight rows from `interleave_gated`, which has half as many outputs.
         `bias` (hybrid graphs, bf16 [rows of the weight]) joins a float32 output."""
         assert input.num_dims == 2 and weight.num_dims == 2 and output.num_dims == 2
         act = self.LINEAR_ACTIVATIONS[activation]
-        params = [act, self._bits(softcap)] if activation == "softcap" else [act] if act else []
+        params = [act] if act else []
+        if activation in ("softcap", "scale"):
+            params.append(self._bits(softcap if activation == "softcap" else scale))
         self._layer(N.OP_LINEAR, [input, weight, output] + ([bias] if bias is not None else []), grid_dim, params)
 
     @staticmethod
@@ -352,11 +370,12 @@ class PersistentKernel:
         return torch.cat([g, u], -2).flatten(-3, -2)
 
     def grouped_linear_layer(self, input: DTensor, weight: DTensor, output: DTensor, *, in_stride: int, out_col: int = 0,
-                             out_stride: int):
+                             out_stride: int, gate: Optional[DTensor] = None, gate_col: int = 0, gate_stride: Optional[int] = None):
         """One linear per group: weight [groups, N, K]; group g maps input columns [g * in_stride, + K) to output columns
-        [out_col + g * out_stride, + N)."""
+        [out_col + g * out_stride, + N).  `gate` (float32) multiplies them by the sigmoid of its columns [gate_col + g * gate_stride, + N)."""
         assert weight.num_dims == 3
-        self._layer(N.OP_GROUPED_LINEAR, [input, weight, output], (1, 1, 1), [in_stride, out_col, out_stride])
+        self._layer(N.OP_GROUPED_LINEAR, [input, weight, output] + ([gate] if gate is not None else []), (1, 1, 1),
+                    [in_stride, out_col, out_stride] + ([gate_col, weight.dim(1) if gate_stride is None else gate_stride] if gate is not None else []))
 
     def linear_with_residual_layer(self, input: DTensor, weight: DTensor, residual: DTensor, output: DTensor,
                                    grid_dim: tuple, block_dim: tuple):
@@ -534,47 +553,59 @@ class PersistentKernel:
                             norm_bias: Optional[DTensor] = None, added: Optional[DTensor] = None,
                             added_row: Optional[DTensor] = None,
                             experts: Optional[Tuple[DTensor, DTensor]] = None,
-                            y_gate: Optional[Tuple[DTensor, int]] = None, post_factor: float = 1.0):
+                            y_gate: Optional[Tuple[DTensor, int]] = None, post_factor: float = 1.0, columns: int = 0,
+                            average: Optional[Tuple[DTensor, DTensor]] = None):
         """x += post_factor * rmsnorm(y) * w_post on the float32 stream `x` (x += y without `post_weight`, x unchanged without `y`),
         then output = rmsnorm(x) * w_norm (without `norm_weight`: x as it is).  `zero_centered`: both weights are stored around zero (1 + w is applied).
         `x_out` receives the new stream instead of `x`; with it, graphs of one or two tokens fold the layer into the linear
         that reads `output`.  `layer_norm` makes the output norm a layer norm (with `norm_bias`) instead of an RMS norm.
         Further terms of the sum: `added` (float32 [tokens, width]), `added_row` (bf16 [width], for every token), `experts`
         (outputs [tokens, slots, width] and weights [tokens, slots], both float32); `y_gate` = (float32 tensor, column)
-        multiplies `y` by the column's sigmoid.  With `post_weight` the experts' weighted sum joins `y` in front of its norm."""
+        multiplies `y` by the column's sigmoid.  With `post_weight` the experts' weighted sum joins `y` in front of its norm.
+        `columns`: the norm is that of the leading columns of `x` (nothing is added then).  `average` = (results float32 [results,
+        tokens, width], weights bf16 [n]): x + y is kept as result n - 1 and the new stream is the weighted sum of results 0 .. n - 1."""
         assert x.num_dims == 2
         gate, column = y_gate if y_gate else (None, 0)
         exp_out, exp_w = experts if experts else (None, None)
         self._layer(N.OP_RESIDUAL_NORM, [x, y, post_weight, norm_weight, output, x_out, norm_bias, added, added_row, exp_out,
-                                         exp_w, gate], (1, 1, 1),
-                    [self._bits(eps), int(zero_centered), int(layer_norm), column, self._bits(post_factor)])
+                                         exp_w, gate, *(average or ())], (1, 1, 1),
+                    [self._bits(eps), int(zero_centered), int(layer_norm), column, self._bits(post_factor), int(columns)])
 
-    def qkv_append_layer(self, proj: DTensor, q: DTensor, k_cache: Optional[DTensor], v_cache: Optional[DTensor], cos: DTensor,
-                         sin: DTensor, *, heads: int, kv_heads: int, dim: int, vdim: int, q_col: int, k_col: int = 0, v_col: int = 0,
+    def qkv_append_layer(self, proj: DTensor, q: DTensor, k_cache: Optional[DTensor], v_cache: Optional[DTensor],
+                         cos: Optional[DTensor], sin: Optional[DTensor], *, heads: int, kv_heads: int, dim: int, vdim: int, q_col: int, k_col: int = 0, v_col: int = 0,
                          rot_dims: int, unit_norm: bool = False, eps: float, q_norm: Optional[DTensor] = None,
-                         k_norm: Optional[DTensor] = None, interleaved: bool = False, maps: int = 1):
+                         k_norm: Optional[DTensor] = None, interleaved: bool = False, maps: int = 1, whole_norm: bool = False,
+                         temperature: Optional[Tuple[float, int]] = None):
         """Takes q / k / v columns of the float32 projections: rotates the first `rot_dims` of q and k (half-split pairs,
         float32 tables [positions, rot_dims / 2]), divides them by their RMS (`unit_norm`), and writes q and the cache
         rows of the new positions.  Values are taken as projected; `v_col == k_col` makes the keys the values.  Without caches
         only queries are formed (a layer that reads another layer's keys and values).  `q_norm`, `k_norm` (bf16 [dim]): RMS norms
         in front of the rotation instead.  `interleaved`: neighbours are rotated together.  `maps=2` (differential attention):
         heads have two vectors of `dim` columns side by side in the projections; a cache row holds both, and `q` has two rows
-        per head, each with its own vector and zeros for the other."""
+        per head, each with its own vector and zeros for the other.  `whole_norm`: one norm over all heads of q (of k), with weights
+        [heads * dim] and without rotation; `temperature` = (coef, every) then multiplies the queries by
+        1 + coef * ln(floor((position + 1) / every) + 1).  The tables are absent where nothing is rotated."""
+        coef, every = temperature or (0.0, 0)
+        if temperature and every < 1:
+            raise ValueError(f"query temperature: a step of {every} positions")
         self._layer(N.OP_QKV_APPEND, [proj, q, k_cache, v_cache, cos, sin, q_norm, k_norm], (1, 1, 1),
-                    [heads, kv_heads, dim, vdim, q_col, k_col, v_col, rot_dims, int(unit_norm), self._bits(eps), int(interleaved), maps])
+                    [heads, kv_heads, dim, vdim, q_col, k_col, v_col, rot_dims, int(unit_norm), self._bits(eps), int(interleaved), maps,
+                     int(whole_norm), self._bits(coef), int(every)])
 
     def ext_attention_layer(self, q: DTensor, k_cache: DTensor, v_cache: DTensor, output: DTensor, *, heads: int,
                             kv_heads: int, vdim: int, scale: float, softcap: float = 0.0, sink: bool = False,
                             sinks: Optional[DTensor] = None, out_col: int = 0, out_scale: float = 1.0,
-                            separate_merge: bool = False, window: int = 0, keep_first: int = 0):
+                            separate_merge: bool = False, window: int = 0, keep_first: int = 0,
+                            distance_bias: Optional[Tuple[DTensor, DTensor]] = None):
         """Causal paged attention over rows a qkv_append_layer or latent_append_layer wrote.  score = softcap *
         tanh(scale * q.k / softcap) (no cap at 0); `sink` adds one to the softmax denominator, `sinks` (bf16 [heads]) adds
         exp(sinks[head]); the result times `out_scale` goes to columns [out_col, out_col + heads * vdim) of `output`.
         `v_cache` may be `k_cache`: the leading `vdim` columns of a key are then its value.  `separate_merge`: the key chunks of
         a request are merged by all workers in a layer of its own (for wide values) instead of by the last task to arrive.
         `window` > 0: a position sees itself, the window - 1 positions before it and the first `keep_first`; keys outside are
-        not read.  A float32 `output` is allowed in bf16 graphs."""
-        args = ([q, k_cache, v_cache, output, sinks], (1, 1, 1),
+        not read.  A float32 `output` is allowed in bf16 graphs.  `distance_bias` = (r1, r2), bf16 [heads]: r1 * ln(1 + r2 * distance)
+        comes off the score."""
+        args = ([q, k_cache, v_cache, output, sinks, *(distance_bias or ())], (1, 1, 1),
                 [heads, kv_heads, vdim, out_col, self._bits(scale), self._bits(softcap or 0.0), int(sink or sinks is not None),
                  self._bits(out_scale), int(separate_merge), int(window), int(keep_first)])
         self._layer(N.OP_EXT_ATTENTION, *args)
@@ -586,12 +617,17 @@ class PersistentKernel:
         per head) -> factor * unit norm of (map 1 - lam * map 2) per head."""
         self._layer(N.OP_DIFF_COMBINE, [maps, output], (1, 1, 1), [heads, vdim, self._bits(lam), self._bits(factor), self._bits(eps)])
 
-    def latent_append_layer(self, proj: DTensor, latent_norm: DTensor, q: DTensor, cache: DTensor, cos: DTensor, sin: DTensor,
-                            *, heads: int, rank: int, rot_dims: int, q_col: int, kv_col: int, eps: float):
+    def poly_norm_layer(self, z: DTensor, coefficients: DTensor, output: DTensor, *, eps: float):
+        """Activation a N(z) + b N(z^2) + c N(z^3) + e of float32 `z` [tokens, n] with the bf16 coefficients (a, b, c, e); N divides a
+        token's values by their root mean square."""
+        self._layer(N.OP_POLY_NORM, [z, coefficients, output], (1, 1, 1), [self._bits(eps)])
+
+    def latent_append_layer(self, proj: DTensor, latent_norm: DTensor, q: Optional[DTensor], cache: DTensor, cos: Optional[DTensor],
+                            sin: Optional[DTensor], *, heads: int, rank: int, rot_dims: int, q_col: int, kv_col: int, eps: float):
         """Latent attention (DeepSeek-AI, "DeepSeek-V2: A Strong, Economical, and Efficient Mixture-of-Experts Language
         Model"): columns [kv_col, + rank + rot_dims) of the float32 projections become a cache row [pages, page, 1, width]
         (the RMS-normed latent, then the rotated key part all heads share); `rot_dims` columns per head from `q_col` are
-        rotated into q [tokens, heads * width] behind the head's `rank` latent columns."""
+        rotated into q [tokens, heads * width] behind the head's `rank` latent columns.  Without a rotated part q and tables are absent."""
         self._layer(N.OP_LATENT_APPEND, [proj, latent_norm, q, cache, cos, sin], (1, 1, 1),
                     [heads, rank, rot_dims, q_col, kv_col, self._bits(eps)])
 
