@@ -911,15 +911,68 @@ def bebuzen_case(size, dev):
     return c, w
 
 
+# Ruludra at sizes like those: 3 matrix-memory layers as Palarax's, 2 layers of windowed attention with Palarax's heads, 3 of latent
+# attention with Lofirax's heads and latents, the last of which reads the first one's; feed-forwards of Palarax's width.
+RULUDRA_SIZES = {
+    "4096": dict(q_rank=1536, rank=512, ldim=128, lheads=32),
+    "2048": dict(q_rank=768, rank=512, ldim=128, lheads=16),
+}
+
+
+def ruludra_case(size, dev):
+    """(config, device weights) of one size; random weights."""
+    import torch
+    z, y = HYBRID_SIZES[size], RULUDRA_SIZES[size]
+    D, F, mask, buckets = z["width"], z["ff"], {"size": 1024}, 65536
+    ml = {"type": "mlstm", "mixer": {"heads": z["mheads"], "dim": z["mdim"], "vdim": z["mvdim"], "gate_cap": 15.0}}
+    at = {"type": "attention", "mixer": {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+                                         "mask": mask, "q_temp": {"coef": 0.1, "every": 4096}}}
+    la = {"heads": y["lheads"], "dim": y["ldim"], "vdim": y["ldim"], "q_rank": y["q_rank"], "kv_rank": y["rank"], "scale": y["ldim"] ** -0.5, "mask": mask}
+    lat = {"type": "latent_attention", "mixer": la}
+    layers = [ml, lat, ml, at, lat, ml, at, {"type": "latent_attention", "mixer": dict(la, kv_from=1)}]
+    c = {"architecture": "Ruludra", "vocab": HYBRID_VOCAB, "width": D, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+         "embedding": {"bigram": {"buckets": buckets, "mul_prev": 31337, "mul_cur": 13}}, "layers": [dict(m, mlp={"kind": "dense", "ff": F}) for m in layers]}
+    g = torch.Generator(device=dev).manual_seed(1)
+    rnd = lambda *s, std=None, mean=0.0: (mean + (s[-1] ** -0.5 if std is None else std) * torch.randn(
+        *s, generator=g, device=dev)).to(torch.bfloat16)
+    one = lambda n: rnd(n, std=0.1, mean=1.0)
+    w = {"embed": rnd(HYBRID_VOCAB, D, std=1.0), "bigram": rnd(buckets + 1, D, std=0.5), "head": rnd(HYBRID_VOCAB, D), "final.norm": one(D)}
+    for n, layer in enumerate(c["layers"]):
+        p, m = f"l{n}.mix.", layer["mixer"]
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        for nm in ("norm1", "norm1b", "norm2", "norm2b"):
+            w[f"l{n}.{nm}"] = one(D)
+        if layer["type"] == "mlstm":
+            for nm, rows in (("q", H * d), ("k", H * d), ("v", H * dv), ("g", H * dv), ("i", H), ("f", H)):
+                w[p + nm] = rnd(rows, D)
+            w[p + "o"], w[p + "norm"], w[p + "i.b"], w[p + "f.b"] = rnd(D, H * dv), one(H * dv), rnd(H, std=1.0), rnd(H, std=1.0, mean=4.0)
+        elif layer["type"] == "attention":
+            for nm, rows in (("q", H * d), ("k", m["kv_heads"] * d)):
+                w[p + nm], w[f"{p}{nm}.norm"] = rnd(rows, D), one(rows)
+            w[p + "r1"], w[p + "r2"], w[p + "o"] = rnd(H, std=0.1, mean=1.0), rnd(H, std=0.01, mean=0.1), rnd(D, H * d)
+        else:
+            w[p + "dq"], w[p + "dq.norm"], w[p + "uq"] = rnd(m["q_rank"], D), one(m["q_rank"]), rnd(H * d, m["q_rank"])
+            if "kv_from" not in m:
+                w[p + "dkv"], w[p + "dkv.norm"] = rnd(m["kv_rank"], D), one(m["kv_rank"])
+            w[p + "uk"], w[p + "uv"], w[p + "g"], w[p + "o"] = rnd(H * d, m["kv_rank"]), rnd(H * dv, m["kv_rank"]), rnd(H * dv, D), rnd(D, H * dv)
+        q = f"l{n}.mlp."
+        w[q + "up"], w[q + "down"], w[q + "act"] = rnd(F, D), rnd(D, F), torch.tensor([0.6, 0.3, 0.4, 0.1], device=dev).to(torch.bfloat16)
+        w[f"l{n}.dwa"] = rnd(n + 2, std=0.1)
+        w[f"l{n}.dwa"][-1] += 0.9
+    return c, w
+
+
 def run_hybrid(args):
     """Prefill (one request, 64 tokens per launch) and decode (batch 1, 16, 64 at --context) of a model on hybrid graphs and of
-    its closest neighbours at equal size (palarax: Qwen3 layers, lofirax: Palarax, bebuzen: Lofirax and Palarax), with the spans of
-    every kind of task group from the in-kernel profiler.  Timed launches carry no profiler."""
+    its closest neighbours at equal size (palarax: Qwen3 layers, lofirax: Palarax, bebuzen and ruludra: Lofirax and Palarax), with the spans of
+    every kind of task group from the in-kernel profiler (attention over shared rows and norms that form an average under names of their own).
+    Timed launches carry no profiler."""
     import torch
     from mirage_b200.builders.bebuzen import BebuzenConfig
     from mirage_b200.builders.lofirax import LofiraxConfig
     from mirage_b200.builders.palarax import PalaraxConfig
-    from mirage_b200.builders.runner import BebuzenRunner, DecoderShape, LofiraxRunner, PalaraxRunner, Qwen3Runner
+    from mirage_b200.builders.runner import BebuzenRunner, DecoderShape, LofiraxRunner, PalaraxRunner, Qwen3Runner, RuludraRunner
+    from mirage_b200.builders.ruludra import RuludraConfig
     from mirage_b200.profiler import event_spans
     torch.cuda.set_device(0)
     dev = torch.device("cuda", 0)
@@ -952,8 +1005,10 @@ def run_hybrid(args):
                 r.mpk.status()
                 experts = [int(r.mpk.tensor_as_torch(t)[-1]) for t in routing]     # of the launch's last expert layer
                 info = r.mpk.graph_info()
-                for e in event_spans(prof, info["num_tasks"]).values():
-                    spans.setdefault(e["type"], []).append(e["us"])
+                graph = json.loads(r.mpk.dump_task_graph())["events"]
+                for i, e in event_spans(prof, info["num_tasks"]).items():
+                    merged = i + 1 < len(graph) and graph[i + 1]["type"] == "attn_merge"
+                    spans.setdefault(e["type"] + ("_shared" if merged else "_average" if graph[i].get("average") else ""), []).append(e["us"])
                 continue
             e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             torch.cuda.synchronize()
@@ -972,12 +1027,15 @@ def run_hybrid(args):
     results, launches, clk = [], 0, None
     for size, z in HYBRID_SIZES.items():
         for model in {"palarax": ("palarax", "qwen3"), "lofirax": ("lofirax", "palarax"),
-                      "bebuzen": ("bebuzen", "lofirax", "palarax")}[args.workload]:
+                      "bebuzen": ("bebuzen", "lofirax", "palarax"), "ruludra": ("ruludra", "lofirax", "palarax")}[args.workload]:
             if not any(args.cases in f"{model}_{size}_{k}" for k in ("prefill64", "decode1", "decode16", "decode64")):
                 continue
             if model == "bebuzen":
                 c, w = bebuzen_case(size, dev)
                 make = lambda kw, prof: BebuzenRunner(BebuzenConfig.from_dict(c), w, profiler_tensor=prof, **kw)
+            elif model == "ruludra":
+                c, w = ruludra_case(size, dev)
+                make = lambda kw, prof: RuludraRunner(RuludraConfig.from_dict(c), w, profiler_tensor=prof, **kw)
             elif model == "lofirax":
                 c, w = lofirax_case(size, dev)
                 make = lambda kw, prof: LofiraxRunner(LofiraxConfig.from_dict(c), w, profiler_tensor=prof, **kw)
@@ -1014,7 +1072,9 @@ def run_hybrid(args):
                                 "lofirax": "Lofirax 6 gated-linear + 2 latent-attention layer runs (half with experts) beside Palarax 6 "
                                            "matrix-memory + 2 parallel layers, width 4096 and 2048, context %d",
                                 "bebuzen": "Bebuzen 4 selective-scan + 2 windowed + 2 differential attention layers (half with experts) beside "
-                                           "Lofirax and Palarax layers, width 4096 and 2048, context %d"}[args.workload] % ctx,
+                                           "Lofirax and Palarax layers, width 4096 and 2048, context %d",
+                                "ruludra": "Ruludra 3 matrix-memory + 2 windowed + 3 latent attention layers beside Lofirax and Palarax layers, width "
+                                           "4096 and 2048, context %d"}[args.workload] % ctx,
                    "l2": "weights of a launch exceed L2; every launch re-streams them"},
         "gpu_launches": launches, "clocks": clk, "peak_gbs": peak, "peak_kind": peak_kind, "results": results}))
 
@@ -1042,12 +1102,12 @@ def main():
                     help="N > 1: split the lm_head rows over the ranks and merge the ranks' argmax inside the kernel "
                          "(default: every rank keeps the whole lm_head, as the reference does)")
     ap.add_argument("--workload", default="qwen3", choices=["qwen3", "fp8_layer", "moe_block", "mla_decode", "deepseek_slice", "moe_w13", "mla_dense",
-                                                             "palarax", "lofirax", "bebuzen"],
+                                                             "palarax", "lofirax", "bebuzen", "ruludra"],
                     help="qwen3: the headline decode benchmark; the others time one block of the FP8 / MoE / MLA "
                          "task bodies at the shapes of the DeepSeek-V3-style parity configurations (1 GPU); palarax, lofirax, "
-                         "bebuzen: prefill and decode at a few sizes beside the closest other models' layers of equal size (Qwen3; Palarax; "
+                         "bebuzen, ruludra: prefill and decode at a few sizes beside the closest other models' layers of equal size (Qwen3; Palarax; "
                          "Lofirax and Palarax) (1 GPU)")
-    ap.add_argument("--cases", default="", help="palarax, lofirax, bebuzen: only cases whose name contains this text")
+    ap.add_argument("--cases", default="", help="palarax, lofirax, bebuzen, ruludra: only cases whose name contains this text")
     args = ap.parse_args()
     if args.impl == "reference":
         return run_reference(args)
@@ -1055,7 +1115,7 @@ def main():
         return run_ref_kernel(args)
     if args.workload == "deepseek_slice":
         return run_deepseek_slice(args)
-    if args.workload in ("palarax", "lofirax", "bebuzen"):
+    if args.workload in ("palarax", "lofirax", "bebuzen", "ruludra"):
         return run_hybrid(args)
     if args.workload != "qwen3":
         return run_block_workload(args)

@@ -68,6 +68,16 @@ __device__ __forceinline__ float block_sum(float v, float *slots) {
   return t;
 }
 
+// Four bf16 values as floats (8-byte aligned).
+__device__ __forceinline__ float4 bf16x4_at(uint64_t base, int i) {
+  const uint2 v = __ldg(reinterpret_cast<const uint2 *>(base + 2ull * i));
+  return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y));
+}
+__device__ __forceinline__ void store_elt4(__nv_bfloat16 *p, float4 v) {
+  *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+}
+__device__ __forceinline__ void store_elt4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+
 // One request of the batch: its tokens [q0, q0 + nq), the position of the first, its cache pages and its state slot.
 struct SeqView {
   int q0, nq, pos0, kv0, slot;
@@ -150,6 +160,7 @@ static __device__ __noinline__ void run_embed_sum(const Ctx c, const TaskDesc &d
   const long long *ids = reinterpret_cast<const long long *>(d.p[0]);
   const long long *freq = reinterpret_cast<const long long *>(d.p[4]);
   const float factor = __int_as_float(d.a[E_LDI2]);
+  const bool vec = ((width | d.a[E_LDI] | d.a[E_LDB] | d.a[E_LDO] | d.a[E_LDC]) & 3) == 0 && ((d.p[1] | d.p[3]) & 7) == 0 && ((d.p[2] | d.p[5]) & 15) == 0;
   for (int t = d.a[E_T0]; t < t1; ++t) {
     const long long id = __ldcg(ids + t);
     const bool in_table = id >= 0 && id < (long long)d.a[E_AUX];
@@ -163,15 +174,41 @@ static __device__ __noinline__ void run_embed_sum(const Ctx c, const TaskDesc &d
       pair = (prev * wide_arg(d, E_PREV) + (unsigned long long)id * wide_arg(d, E_CUR)) % pair;
     }
     float *out = reinterpret_cast<float *>(d.p[2]) + (size_t)t * d.a[E_LDO], *copy = reinterpret_cast<float *>(d.p[5]) + (size_t)t * d.a[E_LDC];
-#pragma unroll 4
-    for (int j = threadIdx.x; j < width; j += kConsumerThreads) {
-      float v = in_table ? bf16_at(d.p[1], (size_t)id * d.a[E_LDI] + j) * factor : 0.f;
-      if (d.p[3]) v += bf16_at(d.p[3], (size_t)pair * d.a[E_LDB] + j);
-      if (freq) {
-        const unsigned long long turns = (unsigned long long)pos * (unsigned long long)__ldg(freq + (j >> 1));
-        const float half_turns = (float)(int)(turns >> 32) * (1.0f / 2147483648.0f);
-        v += (j & 1) ? cospif(half_turns) : sinpif(half_turns);
+    const uint64_t row1 = d.p[1] + 2ull * (size_t)id * d.a[E_LDI], row2 = d.p[3] + 2ull * (size_t)pair * d.a[E_LDB];
+    auto angle = [&](int i) {   // of columns 2 i and 2 i + 1, in half turns
+      return (float)(int)((unsigned long long)pos * (unsigned long long)__ldg(freq + i) >> 32) * (1.0f / 2147483648.0f);
+    };
+    if (vec) {
+      constexpr int NV = 4;   // 4096 columns at a time
+      for (int j0 = threadIdx.x * 4; j0 < width; j0 += NV * kConsumerThreads * 4) {
+        float4 a[NV], b[NV];
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int j = j0 + i * kConsumerThreads * 4;
+          a[i] = j < width && in_table ? bf16x4_at(row1, j) : make_float4(0.f, 0.f, 0.f, 0.f);
+          b[i] = j < width && d.p[3] ? bf16x4_at(row2, j) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int j = j0 + i * kConsumerThreads * 4;
+          if (j >= width) break;
+          float4 v = make_float4(fmaf(a[i].x, factor, b[i].x), fmaf(a[i].y, factor, b[i].y), fmaf(a[i].z, factor, b[i].z), fmaf(a[i].w, factor, b[i].w));
+          if (freq) {
+            float s0, c0, s1, c1;
+            sincospif(angle(j >> 1), &s0, &c0);
+            sincospif(angle((j >> 1) + 1), &s1, &c1);
+            v.x += s0; v.y += c0; v.z += s1; v.w += c1;
+          }
+          *reinterpret_cast<float4 *>(out + j) = v;
+          if (d.p[5]) *reinterpret_cast<float4 *>(copy + j) = v;
+        }
       }
+      continue;
+    }
+    for (int j = threadIdx.x; j < width; j += kConsumerThreads) {
+      float v = in_table ? bf16_at(row1, j) * factor : 0.f;
+      if (d.p[3]) v += bf16_at(row2, j);
+      if (freq) v += (j & 1) ? cospif(angle(j >> 1)) : sinpif(angle(j >> 1));
       out[j] = v;
       if (d.p[5]) copy[j] = v;
     }
@@ -298,16 +335,6 @@ __device__ __forceinline__ void residual_norm_rows(const Ctx &c, const TaskDesc 
     consumer_sync();   // the reduction slots are used again by the next row
   }
 }
-// Four bf16 values as floats (8-byte aligned).
-__device__ __forceinline__ float4 bf16x4_at(uint64_t base, int i) {
-  const uint2 v = __ldg(reinterpret_cast<const uint2 *>(base + 2ull * i));
-  return make_float4(bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y));
-}
-__device__ __forceinline__ void store_elt4(__nv_bfloat16 *p, float4 v) {
-  *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
-}
-__device__ __forceinline__ void store_elt4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
-
 // The same for aligned rows of at most 4096 columns: row, sublayer output and both weights sit in registers, every load of
 // a row is in flight before the first reduction.
 template <int HYB>
@@ -1973,63 +2000,84 @@ __device__ __noinline__ void run_diff_combine(const Ctx c, const TaskDesc &d) {
 // TASK_POLY_NORM: a N(z) + b N(z^2) + c N(z^3) + e, N dividing a token's values by their root mean square.  One block per token; with the
 // three factors known the sum is a cubic in z.
 // ---------------------------------------------------------------------------
+// One token: emit4(column, values) or emit(column, value) receives the activations of the row's N columns.  Ends with a barrier.
+template <class F4, class F>
+__device__ __forceinline__ void poly_norm_row(const Ctx &c, const float *z, int N, bool vec, uint64_t coefficients, float eps, F4 emit4, F emit) {
+  constexpr int NV = 16;   // 16384 columns in registers, all loads in flight
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  float4 x[NV];
+  float s[3] = {0.f, 0.f, 0.f};
+  auto powers = [&](float v) {
+    const float q = v * v;
+    s[0] += q;
+    s[1] = fmaf(q, q, s[1]);
+    s[2] = fmaf(q * q, q, s[2]);
+  };
+  vec = vec && N <= NV * kConsumerThreads * 4;
+  if (vec) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int j = (i * kConsumerThreads + tid) * 4;
+      x[i] = j < N ? __ldcg(reinterpret_cast<const float4 *>(z + j)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      if (i * kConsumerThreads * 4 >= N) break;
+      powers(x[i].x); powers(x[i].y); powers(x[i].z); powers(x[i].w);
+    }
+  } else {
+#pragma unroll 4
+    for (int j = tid; j < N; j += kConsumerThreads) powers(__ldcg(z + j));
+  }
+#pragma unroll
+  for (int k = 0; k < 3; ++k) {
+    s[k] = warp_sum(s[k]);
+    if (lane == 0) c.s.red[8 * k + warp] = s[k];
+  }
+  consumer_sync();
+  float f[3];
+#pragma unroll
+  for (int k = 0; k < 3; ++k) {
+    float v = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) v += c.s.red[8 * k + w];
+    f[k] = bf16_at(coefficients, k) / sqrtf(v / (float)N + eps);
+  }
+  const float k0 = bf16_at(coefficients, 3);
+  auto cubic = [&](float v) { return fmaf(v, fmaf(v, fmaf(v, f[2], f[1]), f[0]), k0); };
+  if (vec) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int j = (i * kConsumerThreads + tid) * 4;
+      if (i * kConsumerThreads * 4 >= N) break;
+      if (j < N) emit4(j, make_float4(cubic(x[i].x), cubic(x[i].y), cubic(x[i].z), cubic(x[i].w)));
+    }
+  } else {
+#pragma unroll 4
+    for (int j = tid; j < N; j += kConsumerThreads) emit(j, cubic(__ldcg(z + j)));
+  }
+  consumer_sync();   // the reduction slots are used again
+}
 template <int HYB>
 __device__ __noinline__ void run_poly_norm(const Ctx c, const TaskDesc &d) {
   typedef typename HybElt<HYB>::T T;
-  constexpr int NV = 16;   // 16384 columns in registers, all loads in flight
-  const int B = active_tokens(c.P), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int t1 = min(d.a[1], B), N = d.a[2];
-  const float eps = __int_as_float(d.a[5]), k1 = bf16_at(d.p[1], 0), k2 = bf16_at(d.p[1], 1), k3 = bf16_at(d.p[1], 2), k0 = bf16_at(d.p[1], 3);
-  const bool vec = N <= NV * kConsumerThreads * 4 && ((N | d.a[3] | d.a[4]) & 3) == 0 && ((d.p[0] | d.p[2]) & 15) == 0;
+  const int t1 = min(d.a[1], active_tokens(c.P)), N = d.a[2];
+  const bool vec = ((N | d.a[3] | d.a[4]) & 3) == 0 && ((d.p[0] | d.p[2]) & 15) == 0;
   for (int t = d.a[0]; t < t1; ++t) {
-    const float *z = reinterpret_cast<const float *>(d.p[0]) + (size_t)t * d.a[3];
     T *out = reinterpret_cast<T *>(d.p[2]) + (size_t)t * d.a[4];
-    float4 x[NV];
-    float s[3] = {0.f, 0.f, 0.f};
-    auto powers = [&](float v) {
-      const float q = v * v;
-      s[0] += q;
-      s[1] = fmaf(q, q, s[1]);
-      s[2] = fmaf(q * q, q, s[2]);
-    };
-    if (vec) {
-#pragma unroll
-      for (int i = 0; i < NV; ++i) {
-        const int j = (i * kConsumerThreads + tid) * 4;
-        x[i] = j < N ? __ldcg(reinterpret_cast<const float4 *>(z + j)) : make_float4(0.f, 0.f, 0.f, 0.f);
-      }
-#pragma unroll
-      for (int i = 0; i < NV; ++i) { powers(x[i].x); powers(x[i].y); powers(x[i].z); powers(x[i].w); }
-    } else {
-#pragma unroll 4
-      for (int j = tid; j < N; j += kConsumerThreads) powers(__ldcg(z + j));
-    }
-#pragma unroll
-    for (int k = 0; k < 3; ++k) {
-      s[k] = warp_sum(s[k]);
-      if (lane == 0) c.s.red[8 * k + warp] = s[k];
-    }
-    consumer_sync();
-    float f[3];
-#pragma unroll
-    for (int k = 0; k < 3; ++k) {
-      float v = 0.f;
-#pragma unroll
-      for (int w = 0; w < 8; ++w) v += c.s.red[8 * k + w];
-      f[k] = (k == 0 ? k1 : k == 1 ? k2 : k3) / sqrtf(v / (float)N + eps);
-    }
-    auto cubic = [&](float v) { return fmaf(v, fmaf(v, fmaf(v, f[2], f[1]), f[0]), k0); };
-    if (vec) {
-#pragma unroll
-      for (int i = 0; i < NV; ++i) {
-        const int j = (i * kConsumerThreads + tid) * 4;
-        if (j < N) store_elt4(out + j, make_float4(cubic(x[i].x), cubic(x[i].y), cubic(x[i].z), cubic(x[i].w)));
-      }
-    } else {
-#pragma unroll 4
-      for (int j = tid; j < N; j += kConsumerThreads) store_elt(out + j, cubic(__ldcg(z + j)));
-    }
-    consumer_sync();   // the reduction slots are used again
+    poly_norm_row(c, reinterpret_cast<const float *>(d.p[0]) + (size_t)t * d.a[3], N, vec, d.p[1], __int_as_float(d.a[5]),
+                  [&](int j, float4 v) { store_elt4(out + j, v); }, [&](int j, float v) { store_elt(out + j, v); });
+  }
+}
+// PRO_POLY (graphs of one or two tokens): the same rows as the activation tile of the linear behind them, zeros in the padding columns.
+static __device__ __noinline__ void stage_poly(const Ctx c, const TaskDesc &d, int B) {
+  const int N = d.a[L_GROUPS], K = d.a[L_K];
+  const bool vec = ((N | d.a[L_LDX]) & 3) == 0 && (d.p[1] & 15) == 0;
+  for (int b = 0; b < B; ++b) {
+    __nv_bfloat16 *row = reinterpret_cast<__nv_bfloat16 *>(c.s.xtile + (size_t)b * (K * 2 + kRowPadBytes));
+    for (int j = N + threadIdx.x; j < K; j += kConsumerThreads) store_elt(row + j, 0.f);
+    poly_norm_row(c, reinterpret_cast<const float *>(d.p[1]) + (size_t)b * d.a[L_LDX], N, vec, d.p[4], __int_as_float(d.a[L_EPS]),
+                  [&](int j, float4 v) { store_elt4(row + j, v); }, [&](int j, float v) { store_elt(row + j, v); });
   }
 }
 

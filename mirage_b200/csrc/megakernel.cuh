@@ -424,7 +424,7 @@ static __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d
   const float eps = __int_as_float(d.a[L_EPS]), off = (d.a[L_G_SLOT] & 2) ? 1.0f : 0.0f, factor = __int_as_float(d.a[LR_POST]);
   const float *add = *reinterpret_cast<const float *const *>(&d.a[LR_ADD]);
   const uint64_t rowp = *reinterpret_cast<const uint64_t *>(&d.a[LR_ROW]);
-  const bool has_y = d.p[6] != 0, has_post = d.p[3] != 0, moved = has_y || add != nullptr || rowp != 0;
+  const bool has_y = d.p[6] != 0, has_post = d.p[3] != 0, moved = has_y || add != nullptr || rowp != 0, average = (d.a[L_G_SLOT] & 8) != 0;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   auto values = [&](uint64_t base, int j, float o) {
     const uint2 v = __ldg(reinterpret_cast<const uint2 *>(base + 2ull * j));
@@ -467,7 +467,37 @@ static __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d
         xv[i].z += yv[i].z * inv * wp[i].z; xv[i].w += yv[i].w * inv * wp[i].w;
       }
     }
-    if (add != nullptr || rowp != 0) {
+    if (average) {
+      float *res = const_cast<float *>(add) + (size_t)b * W;
+      const int last = d.a[L_LDR] - 1, step = d.a[LR_LDADD];
+      auto weight = [&](int k) { return bf16_to_f(__ldg(reinterpret_cast<const __nv_bfloat16 *>(rowp) + k)); };
+      const float wl = weight(last);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int j = (i * kConsumerThreads + tid) * 4;
+        if (j < W) *reinterpret_cast<float4 *>(res + (size_t)last * step + j) = xv[i];
+        xv[i].x *= wl; xv[i].y *= wl; xv[i].z *= wl; xv[i].w *= wl;
+      }
+      for (int k = 0; k < last; k += 2) {   // two results in flight
+        float4 e[2][NV];
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+          for (int i = 0; i < NV; ++i) {
+            const int j = (i * kConsumerThreads + tid) * 4;
+            e[u][i] = j < W && k + u < last ? __ldcg(reinterpret_cast<const float4 *>(res + (size_t)(k + u) * step + j)) : zero;
+          }
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          const float wk = k + u < last ? weight(k + u) : 0.f;
+#pragma unroll
+          for (int i = 0; i < NV; ++i) {
+            xv[i].x = fmaf(wk, e[u][i].x, xv[i].x); xv[i].y = fmaf(wk, e[u][i].y, xv[i].y);
+            xv[i].z = fmaf(wk, e[u][i].z, xv[i].z); xv[i].w = fmaf(wk, e[u][i].w, xv[i].w);
+          }
+        }
+      }
+    } else if (add != nullptr || rowp != 0) {
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int j = (i * kConsumerThreads + tid) * 4;
@@ -513,6 +543,9 @@ static __device__ __noinline__ void stage_resnorm(const Ctx c, const TaskDesc &d
     consumer_sync();   // (also: the reduction slots are used again)
   }
 }
+
+// PRO_POLY (hybrid_tasks.cuh).
+static __device__ __noinline__ void stage_poly(const Ctx c, const TaskDesc &d, int B);
 
 // Copies B rows of `vecs` 16-byte vectors into the activation tile, one warp per row, every copy in flight.  A function of its own:
 // at the register cap of the linear bodies its loop would reload spilled variables for each copy.
@@ -905,6 +938,7 @@ __device__ __forceinline__ void run_linear(const Ctx &c, const TaskDesc &d, Line
     if (B > 0 && !((d.flags & TF_SAME_X_AS_PREV) && !multi_tile)) {
       if (kt > 0) consumer_sync();   // everyone is done reading the previous tile
       if (HYB && !WIDE && d.a[L_PRO] == PRO_RESNORM) stage_resnorm(c, d, B);
+      else if (HYB && !WIDE && d.a[L_PRO] == PRO_POLY) stage_poly(c, d, B);
       else stage_x<WIDE ? 1 : 0, TPX>(c, d, B, kt, KT, gpre);
     }
     if (tid == 0 && prof && kt == 0) P.profiler[(size_t)task * 8 + 4] = globaltimer_ns();

@@ -121,7 +121,8 @@ enum : int {
 
 // prologue applied while staging the activation tile of a linear task
 enum Prologue : int32_t { PRO_PLAIN = 0, PRO_RMSNORM = 1, PRO_SILU_MUL = 2,
-                          PRO_RESNORM = 3 };   // hybrid graphs: x_out = x + norm(y) on the float32 stream, activation = norm(x_out)
+                          PRO_RESNORM = 3,   // hybrid graphs: x_out = x + norm(y) on the float32 stream, activation = norm(x_out)
+                          PRO_POLY = 4 };      // hybrid graphs: activation = sum of normed powers of float32 values (TASK_POLY_NORM)
 // epilogue of a linear task
 enum Epilogue : int32_t {
   EPI_STORE = 0,        // out = bf16(acc)
@@ -178,6 +179,9 @@ static_assert(sizeof(TaskDesc) == 16 * kDescVecs, "TaskDesc must stay 224 bytes 
 //        null), a[20] ld y, a[21] ld x_out, a[22] flags (2: weights stored around zero, 4: layer norm), a[10] width (K minus the
 //        zero padding), p[5] norm bias or null, 64-bit values a[LR_ADD] added stream or null (ld a[LR_LDADD]), a[LR_ROW] added row or null
 //        a[LR_POST] factor of y's norm (bits); p[4] null: the activation is the stream as it is
+//        flag 8: the stream is the weighted sum of a[L_LDR] results: a[LR_ADD] results f32 (a[LR_LDADD] floats apart, rows of a[10]; the last is
+//        written), a[LR_ROW] their weights bf16
+//  PRO_POLY: p[1] z f32  p[4] coefficients bf16 [4], a[10] columns of z (K minus the zero padding), a[9] eps bits
 //  EPI_SOFTCAP, EPI_SCALE_F32: a[23] cap / factor bits;  EPI_BIAS_F32: 64-bit value a[LR_BIAS];  EPI_GATE_SIGMOID: p[3] gate f32, a[6] its ld
 //  a[15] allreduce index within the iteration  a[16] allreduces per iteration  a[17] stride between the two inbox buffers (floats)
 //  tcgen05 path (TF_TC): a[18] rows of one weight tile (the TMA box height, a multiple of 8, at most 128; the task's rows are

@@ -43,6 +43,7 @@ struct Builder {
   std::vector<std::vector<TaskDesc>> per_worker;
   std::vector<std::vector<int>> per_worker_exec;
   int rot = 0;
+  static constexpr int kMaxFoldedTerms = 16;   // results a linear's prologue averages at most: every task of the linear reads them all
   TaskDesc xattn_task;      // the last extended-attention task (its merge layer shares the fields)
   int hybrid_tickets = 0;   // arrival tickets handed to the tasks of hybrid graphs
   std::map<int, std::map<int, int>> slices;   // storage -> (first column -> id) of outputs that layers write by column range
@@ -117,10 +118,11 @@ struct Builder {
         } else {
           add(ins, l.prologue == PRO_PLAIN ? l.t[0] : l.pro_src);
         }
-        if (l.prologue == PRO_RMSNORM || l.prologue == PRO_RESNORM) add(ins, l.pro_gamma);
+        if (l.prologue == PRO_RMSNORM || l.prologue == PRO_RESNORM || l.prologue == PRO_POLY) add(ins, l.pro_gamma);
         if (l.prologue == PRO_RESNORM) {
           for (int t : {l.pro_y, l.pro_post, l.pro_bias, l.pro_add, l.pro_row}) add(ins, t);
           add(outs, l.pro_xout);
+          if (l.pro_terms > 0) add(outs, l.pro_add);   // the results it averages: one of them is its own
         }
         add(ins, l.t[1]);
         const int y = l.op == MPK_OP_LINEAR_RESIDUAL ? l.t[3] : l.t[2];
@@ -318,8 +320,9 @@ struct Builder {
       LayerInfo &p = L[i];
       if (p.op != MPK_OP_RESIDUAL_NORM || p.t[4] < 0) continue;
       const int x = p.t[0], y = p.t[1], out = p.t[4], xo = resnorm_out(p), add = norm_tensor(p, 7), row = norm_tensor(p, 8), bias = norm_tensor(p, 6);
-      // the sums over experts or earlier results are formed once, not by every task
-      if (norm_tensor(p, 9) >= 0 || norm_tensor(p, 11) >= 0 || norm_tensor(p, 12) >= 0) continue;
+      if (norm_tensor(p, 9) >= 0 || norm_tensor(p, 11) >= 0) continue;   // the sum over experts is formed once, not by every task
+      const int results = norm_tensor(p, 12), terms = results >= 0 ? (int)T[p.t[13]].dim(0) : 0;
+      if (results >= 0 && (add >= 0 || row >= 0 || terms > kMaxFoldedTerms || ((uint64_t)T[results].ptr & 15) || T[results].strides[0] % 4)) continue;
       const bool moves = resnorm_moves(p);
       auto aligned = [&](int t) { return T[t].ld() % 4 == 0 && ((uint64_t)T[t].ptr & 15) == 0; };
       const int64_t D = norm_columns(p);
@@ -341,7 +344,7 @@ struct Builder {
       }
       if (!ok || consumers.size() != 1) continue;
       for (size_t j = i + 1; j < consumers[0] && ok; ++j)   // nothing in between may touch what the prologue reads or writes
-        for (int t : {x, y, xo, add})
+        for (int t : {x, y, xo, add, results})
           if (t >= 0 && (raw_writes(L[j], T[t].storage) || (t == xo && moves && raw_reads(L[j], T[t].storage)))) ok = false;
       if (!ok) continue;
       LayerInfo &c = L[consumers[0]];
@@ -350,7 +353,38 @@ struct Builder {
       c.pro_bias = bias; c.pro_add = add; c.pro_row = row;
       c.pro_xout = moves ? xo : -1;
       c.pro_cols = (int)D;
-      c.pro_eps = bits_of(p.params[0]); c.pro_flags = norm_flags(p); c.pro_factor = norm_factor(p);
+      c.pro_terms = terms;
+      if (terms > 0) { c.pro_add = results; c.pro_row = p.t[13]; }
+      c.pro_eps = bits_of(p.params[0]); c.pro_flags = norm_flags(p) | (terms > 0 ? 8 : 0); c.pro_factor = norm_factor(p);
+      p.folded = true;
+      g->num_folded++;
+    }
+  }
+
+  // The same for the sum of normed powers in front of a linear.
+  void fold_poly_norms() {
+    if (g->hybrid != HYB_BF16 || nb_max > 2 || cfg.max_num_batched_tokens > 2) return;
+    for (size_t i = 0; i < L.size(); ++i) {
+      LayerInfo &p = L[i];
+      if (p.op != MPK_OP_POLY_NORM || p.params.empty() || T[p.t[2]].owner == 0) continue;
+      const int z = p.t[0], out = p.t[2];
+      std::vector<size_t> consumers;
+      bool ok = true;
+      for (size_t j = i + 1; j < L.size() && ok; ++j) {
+        const LayerInfo &c = L[j];
+        if (raw_reads(c, T[out].storage)) {
+          if (c.op != MPK_OP_LINEAR || c.prologue != PRO_PLAIN || c.t[0] != out || linear_tile_bytes(T[c.t[1]].dim(1)) > x_tile_cap()) ok = false;
+          else consumers.push_back(j);
+        }
+        if (raw_writes(c, T[out].storage)) break;
+      }
+      if (!ok || consumers.size() != 1) continue;
+      for (size_t j = i + 1; j < consumers[0] && ok; ++j)
+        if (raw_writes(L[j], T[z].storage)) ok = false;
+      if (!ok || T[z].dtype != MPK_F32 || T[p.t[1]].dtype != MPK_BF16 || T[p.t[1]].dim(0) != 4 || T[z].dim(1) > T[L[consumers[0]].t[1]].dim(1)) continue;
+      LayerInfo &c = L[consumers[0]];
+      c.prologue = PRO_POLY;
+      c.pro_src = z; c.pro_gamma = p.t[1]; c.pro_cols = (int)T[z].dim(1); c.pro_eps = bits_of(p.params[0]);
       p.folded = true;
       g->num_folded++;
     }
@@ -578,7 +612,8 @@ struct Builder {
       ++nkt;
     if (nkt > K / kq) return fail(MPK_ERR_UNSUPPORTED, "cannot tile K for " + w.name);
     const int KT = K / nkt;
-    if ((l.prologue == PRO_RMSNORM || l.prologue == PRO_RESNORM) && nkt != 1)
+    const bool f32_source = l.prologue == PRO_RESNORM || l.prologue == PRO_POLY;   // formed from float32 values by the prologue
+    if ((l.prologue == PRO_RMSNORM || f32_source) && nkt != 1)
       return fail(MPK_ERR_UNSUPPORTED, "rmsnorm prologue needs the whole row in shared memory: " + w.name);
     // k extent of a streamed chunk: the largest multiple of 16 that divides KT and fits a stage
     // Chunk geometry: 16 rows (one mma m-tile) x KC columns.  The copy engine handles a fixed number of bulk
@@ -594,7 +629,7 @@ struct Builder {
     if (l.prologue == PRO_SILU_MUL) {
       if (x.dim(1) != 2 * (int64_t)K || (K / l.pro_groups) % 8 != 0 || K % l.pro_groups != 0)
         return fail(MPK_ERR_INVALID, "silu_mul feeding " + w.name + ": bad gate|up width or group count");
-    } else if (l.prologue != PRO_RESNORM && x.dim(x.dims.size() - 1) != K) {
+    } else if (!f32_source && x.dim(x.dims.size() - 1) != K) {
       return fail(MPK_ERR_INVALID, "linear input width != K for " + w.name);
     }
     int epi = EPI_STORE;
@@ -614,7 +649,7 @@ struct Builder {
       epi = EPI_RESIDUAL; res_ptr = (uint64_t)y.ptr; ldr = (int)y.ld();
     }
     if (l.push) epi = l.push_ll ? EPI_PUSH_LL : EPI_PUSH_F32;
-    if (x.dtype != MPK_BF16 && l.prologue != PRO_RESNORM) return fail(MPK_ERR_UNSUPPORTED, "linear input must be bf16: " + w.name);
+    if (x.dtype != MPK_BF16 && !f32_source) return fail(MPK_ERR_UNSUPPORTED, "linear input must be bf16: " + w.name);
     if (l.op == MPK_OP_LINEAR && !l.params.empty() && l.params[0] != 0) {
       epi = activation_epilogue(l.params[0]);
       if (g->hybrid != HYB_BF16 || epi == EPI_STORE || y.dtype != (capped(epi) ? MPK_F32 : MPK_BF16) || (capped(epi) && l.params.size() < 2))
@@ -686,7 +721,7 @@ struct Builder {
         d.p[1] = (uint64_t)x.ptr;
         d.p[2] = out_ptr;
         d.p[3] = res_ptr;
-        d.p[4] = l.prologue == PRO_RMSNORM ? (uint64_t)T[l.pro_gamma].ptr : 0;
+        d.p[4] = l.prologue == PRO_RMSNORM || l.prologue == PRO_POLY ? (uint64_t)T[l.pro_gamma].ptr : 0;
         d.p[5] = in.inbox_base_floats;
         if (l.gather_ar >= 0) {
           d.p[6] = l.gather_res >= 0 ? (uint64_t)T[l.gather_res].ptr : 0;
@@ -705,7 +740,7 @@ struct Builder {
           d.a[L_G_LDOUT] = l.pro_xout >= 0 ? (int)T[l.pro_xout].ld() : 0;
           d.a[L_G_SLOT] = l.pro_flags;
           d.p[5] = l.pro_bias >= 0 ? (uint64_t)T[l.pro_bias].ptr : 0;
-          d.a[LR_LDADD] = l.pro_add >= 0 ? (int)T[l.pro_add].ld() : 0;
+          d.a[LR_LDADD] = l.pro_terms > 0 ? (int)T[l.pro_add].strides[0] : l.pro_add >= 0 ? (int)T[l.pro_add].ld() : 0;
         }
         d.a[L_N0] = r;
         d.a[L_N1] = std::min(r + task_cap, row + cnt);
@@ -713,11 +748,11 @@ struct Builder {
         d.a[L_LDW] = ldw;
         d.a[L_LDX] = (int)x.ld();
         d.a[L_LDO] = ldo;
-        d.a[L_LDR] = ldr;
+        d.a[L_LDR] = l.prologue == PRO_RESNORM ? l.pro_terms : ldr;
         d.a[L_PRO] = l.prologue;
         d.a[L_EPI] = epi;
-        d.a[L_EPS] = l.prologue == PRO_RESNORM ? l.pro_eps : float_bits(1e-6f);
-        d.a[L_GROUPS] = l.prologue == PRO_RESNORM ? l.pro_cols : l.pro_groups;
+        d.a[L_EPS] = f32_source ? l.pro_eps : float_bits(1e-6f);
+        d.a[L_GROUPS] = f32_source ? l.pro_cols : l.pro_groups;
         d.a[L_KT] = KT;
         d.a[L_KC] = KC;
         d.a[L_ROWS] = R;
@@ -2157,6 +2192,7 @@ struct Builder {
     for (const auto &l : L) if (l.folded) g->num_folded++;     // folded before materialisation (activation epilogue)
     fold_layers();
     fold_residual_norms();
+    fold_poly_norms();
     rc = plan_allreduce();
     if (rc) return rc;
     rc = plan_smem();
@@ -2442,8 +2478,9 @@ std::string dump_task_graph(const CompiledGraph &g, const std::vector<TensorInfo
     for (size_t k = 0; k < x.deps.size(); ++k) os << (k ? ", " : "") << "[" << x.deps[k] << ", " << x.dep_need[k] << "]";
     os << "]";
     if (x.layer >= 0 && layers[x.layer].prologue != PRO_PLAIN)
-      os << ", \"prologue\": \"" << (layers[x.layer].prologue == PRO_RMSNORM ? "rmsnorm" : layers[x.layer].prologue == PRO_RESNORM ? "residual_norm" : "silu_mul") << "\"";
+      os << ", \"prologue\": \"" << (layers[x.layer].prologue == PRO_RMSNORM ? "rmsnorm" : layers[x.layer].prologue == PRO_RESNORM ? "residual_norm" : layers[x.layer].prologue == PRO_POLY ? "poly_norm" : "silu_mul") << "\"";
     if (x.layer >= 0 && layers[x.layer].silu_out >= 0) os << ", \"epilogue\": \"silu_mul\"";
+    if (x.layer >= 0 && layers[x.layer].op == MPK_OP_RESIDUAL_NORM && layers[x.layer].t.size() > 12 && layers[x.layer].t[12] >= 0) os << ", \"average\": true";
     if (x.remote_trigger) os << ", \"push\": true";
     if (x.tc_rows > 0) os << ", \"tcgen05\": {\"tile_rows\": " << x.tc_rows << ", \"k_blocks_per_slot\": " << x.tc_kblocks << "}";
     if (x.layer >= 0 && !layers[x.layer].t.empty()) {

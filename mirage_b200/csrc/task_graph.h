@@ -47,7 +47,7 @@ struct LayerInfo {
   int pro_y = -1, pro_post = -1, pro_xout = -1;   // PRO_RESNORM: sublayer output, weight of its norm, new stream
   int pro_bias = -1, pro_add = -1, pro_row = -1;  // PRO_RESNORM: bias of the norm, added stream, added row
   int pro_eps = 0, pro_flags = 0, pro_factor = 0;
-  int pro_cols = 0;            // PRO_RESNORM: columns of the row
+  int pro_cols = 0, pro_terms = 0;   // PRO_RESNORM: columns of the row, results in the average (then pro_add, pro_row: the results, their weights)
   bool push = false;           // linear: epilogue pushes fp32 partials to the peers' inboxes
   int ar_index = -1;           // allreduce ordinal within the iteration
   int ar_producer = -1;        // allreduce: exec layer of the pushing linear

@@ -17,7 +17,7 @@ TASK_NAMES = ["nop", "batch", "embed", "rmsnorm", "linear", "attention", "silu_m
               "allreduce", "elementwise_add", "tensor_init", "quantize_fp8", "moe_routing", "moe_gemm", "moe_silu_mul",
               "moe_mul_sum_add", "mla_append", "mla_decode", "mla_reduce", "sampling_partial", "sampling_reduce", "argmax_exchange", "ar_push",
               "embed_f32", "residual_norm", "linear_f32", "qkv_append", "ext_attention", "short_conv", "rglru", "mlstm",
-              "gla", "latent_append", "moe_gemm_f32", "attn_merge", "selective_scan", "diff_combine"]
+              "gla", "latent_append", "moe_gemm_f32", "attn_merge", "selective_scan", "diff_combine", "poly_norm"]
 
 
 def decode_records(profiler_buffer: torch.Tensor, num_tasks: int) -> List[Dict[str, int]]:

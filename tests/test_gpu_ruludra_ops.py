@@ -67,7 +67,7 @@ def test_attention_with_norms_over_all_heads_and_a_distance_bias(dtype, tokens, 
 
 def test_norm_over_more_columns_than_registers_hold():
     """Rows of more than 4096 columns, queries only and with caches."""
-    H, G, dim, n = 70, 36, 120, 5
+    H, G, dim, n = 70, 35, 120, 5
     g = torch.Generator().manual_seed(1)
     b = Bench(1, tokens=8)
     x = torch.randn(8, (H + G) * dim, generator=g)
@@ -282,6 +282,51 @@ def test_average_over_the_layers_results(dtype, tokens, width, terms, post):
     assert err(kept[terms - 1], own) < TOL[torch.float32] and torch.equal(kept[:terms - 1], hist[:terms - 1].double()) and torch.equal(kept[terms:], hist[terms:].double())
     assert err(xo.double().cpu(), new) < TOL[torch.float32]
     assert err(out[:, :width].double().cpu(), ops.rms_norm(new, wn.double(), 1e-3)) < TOL[dtype] and float(out[:, width:].abs().max()) == 0.0
+
+
+@pytest.mark.parametrize("tokens", [1, 2])
+@pytest.mark.parametrize("terms", [2, 5, 16, 17])
+def test_average_over_the_layers_results_folds_into_a_linear(tokens, terms):
+    g = torch.Generator().manual_seed(15)
+    width, N = 100, 70
+    x, y, hist = torch.randn(tokens, width, generator=g), 3 * torch.randn(tokens, width, generator=g), torch.randn(terms + 1, tokens, width, generator=g)
+    w, wp, wn, lin = RAND(g, terms), RAND(g, width, std=0.3, mean=1.0), RAND(g, width, std=0.3, mean=1.0), RAND(g, N, width, std=0.1)
+    b = Bench(1, tokens=tokens)
+    results, xo, out = hist.cuda(), b.zeros(tokens, width), b.zeros(tokens, N)
+    h = b.pk.new_tensor(dims=(tokens, 128), name="h")
+    b.pk.residual_norm_layer(b.inp(x, "x"), b.inp(y, "y"), b.inp(wp, "wp"), b.inp(wn, "wn"), h, eps=1e-4, x_out=b.pk.attach_input(xo, name="xo"),
+                             average=(b.pk.attach_input(results, name="results"), b.inp(w, "w")))
+    b.pk.linear_layer(input=h, weight=b.inp(pad_k(lin, torch.bfloat16), "lin"), output=b.pk.attach_input(out, name="o"), grid_dim=(1, 1, 1),
+                      block_dim=(128, 1, 1))
+    b.pk.compile()
+    assert b.pk.graph_info()["num_folded"] == int(terms <= 16)
+    b.describe([tokens])
+    b.pk.step(1)
+    b.pk.status()
+    own = x.double() + ops.rms_norm(y.double(), wp.double(), 1e-4)
+    new = ops.depth_average([*hist[:terms - 1].double(), own], w.double())
+    kept = results.double().cpu()
+    assert err(kept[terms - 1], own) < TOL[torch.float32] and torch.equal(kept[:terms - 1], hist[:terms - 1].double()) and torch.equal(kept[terms], hist[terms].double())
+    assert err(xo.double().cpu(), new) < TOL[torch.float32]
+    assert err(out.double().cpu(), ops.rms_norm(new, wn.double(), 1e-4) @ lin.double().T) < TOL[torch.bfloat16]
+
+
+@pytest.mark.parametrize("tokens", [1, 2])
+@pytest.mark.parametrize("n", [1, 37, 64, 1030, 16384])
+def test_normed_powers_fold_into_a_linear(tokens, n):
+    g = torch.Generator().manual_seed(16)
+    z, co, lin = 2.0 * torch.randn(tokens, n, generator=g), torch.tensor([0.6, -0.8, 1.1, 0.3]).to(torch.bfloat16), RAND(g, 70, n, std=n ** -0.5)
+    b = Bench(1, tokens=tokens)
+    padded, out = pad_k(lin, torch.bfloat16), b.zeros(tokens, 70)
+    h = b.pk.new_tensor(dims=(tokens, padded.shape[1]), name="h")
+    b.pk.poly_norm_layer(b.inp(z, "z"), b.inp(co, "co"), h, eps=1e-3)
+    b.pk.linear_layer(input=h, weight=b.inp(padded, "lin"), output=b.pk.attach_input(out, name="o"), grid_dim=(1, 1, 1), block_dim=(128, 1, 1))
+    b.pk.compile()
+    assert b.pk.graph_info()["num_folded"] == 1
+    b.describe([tokens])
+    b.pk.step(1)
+    b.pk.status()
+    assert err(out.double().cpu(), ops.poly_norm(z.double(), co.double(), 1e-3) @ lin.double().T) < TOL[torch.bfloat16]
 
 
 @DT

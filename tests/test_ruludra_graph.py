@@ -56,9 +56,13 @@ def test_norms_fold_into_the_linears_of_single_token_graphs():
     c = mixed_config()
     pk = dry(c, mbt=1)
     ev = events(pk)
-    # the first norm, two query latents, three in front of a feed-forward; those that form an average (one per layer) stay
-    assert sum(e.get("prologue") == "residual_norm" for e in ev) == pk.graph_info()["num_folded"] == 6
-    assert sum(e["type"] == "residual_norm" for e in ev) == len(c["layers"])
+    # the first norm, two query latents, three in front of a feed-forward, one with an average per layer; and three activations
+    kinds = [e.get("prologue") for e in ev]
+    assert (kinds.count("residual_norm"), kinds.count("poly_norm")) == (6 + len(c["layers"]), 3) and pk.graph_info()["num_folded"] == 15
+    assert not {"residual_norm", "poly_norm"} & {e["type"] for e in ev}
+    # an average over many results is formed once, not by every task of the linear behind it
+    deep = dry(P.config(32, 64, [P.mlstm_layer(1, 8, 8, ff=None)] * 17), mbt=1)
+    assert [e["type"] for e in events(deep)].count("residual_norm") == 2
     pk = dry(c, mbt=3)
     pk.compile()
     assert pk.graph_info()["num_folded"] == 0
