@@ -15,7 +15,7 @@ from .persistent_kernel import (  # noqa: F401
 
 from .noalloc import paged_decode_attention_noalloc  # noqa: F401,E402
 from .mpk import MPK, MPKMetadata, get_builder, register_model_builder  # noqa: F401,E402
-from .builders import bebuzen as _bebuzen_builder, lofirax as _lofirax_builder, palarax as _palarax_builder, qwen3 as _qwen3_builder  # noqa: F401,E402  (file the graph builders)
+from .builders import bebuzen as _bebuzen_builder, lofirax as _lofirax_builder, palarax as _palarax_builder, qwen3 as _qwen3_builder, ruludra as _ruludra_builder  # noqa: F401,E402  (file the graph builders)
 from .builders.registry import load_runner, runner_class  # noqa: F401,E402
 from .serving import OnlineSession  # noqa: F401,E402
 
